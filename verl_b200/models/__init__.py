@@ -13,3 +13,13 @@ def make_flat_params(cfg: ModelConfig, **kw):
         kw.pop("grad_buffer", None)
         return ModuleFlatParams(cfg, **kw)
     return FlatParams(cfg, **kw)
+
+
+def build_decoder(cfg: ModelConfig, params, **kw):
+    """The hand-scheduled model of a natively supported configuration: :class:`DecoderModel`, or
+    :class:`~verl_b200.models.mixer_stack.MixerStackModel` for decoders whose layers differ."""
+    if cfg.is_stack:
+        from .mixer_stack import MixerStackModel
+
+        return MixerStackModel(cfg, params, **kw)
+    return DecoderModel(cfg, params, **kw)

@@ -12,6 +12,8 @@ import os
 from dataclasses import asdict, dataclass, field
 from typing import Any, Optional
 
+from .mixer_stack_config import StackSpec, is_stack_config, parse_stack
+
 __all__ = ["ModelConfig", "PRESETS", "get_preset", "NATIVE_FAMILIES"]
 
 # architectures with a hand-scheduled decoder (own kernels, own backward, paged rollout engine); every other causal language
@@ -49,6 +51,8 @@ class ModelConfig:
     pad_token_id: Optional[int] = None
     initializer_range: float = 0.02
     extra: dict = field(default_factory=dict)
+    # decoders whose layers differ (``mixer_stack_config.DESIGNS``): the typed layer list
+    stack: Optional[StackSpec] = None
     # model-parallel shard description (a full model has both ends and local = global expert count)
     has_embedding: bool = True    # pipeline stage owns the token embedding
     has_head: bool = True         # pipeline stage owns the final norm and the LM/value head
@@ -101,6 +105,11 @@ class ModelConfig:
         return bool(self.extra.get("generic"))
 
     @property
+    def is_stack(self) -> bool:
+        """True for mixer stacks (``models/mixer_stack.py``): per-layer mixers, own cache layout, served forward-only."""
+        return self.stack is not None
+
+    @property
     def q_size(self) -> int:
         return self.num_attention_heads * self.head_dim
 
@@ -114,6 +123,10 @@ class ModelConfig:
 
     def num_parameters(self, value_head: bool = False) -> int:
         h, v = self.hidden_size, self.vocab_size
+        if self.is_stack:
+            from .weights import build_param_specs
+
+            return sum(s.numel for s in build_param_specs(self))
         per_layer = 2 * h + self.qkv_size * h + self.q_size * h
         if self.attention_bias:
             per_layer += self.qkv_size
@@ -140,6 +153,8 @@ class ModelConfig:
     # ------------------------------------------------------------------ HF interchange
     @classmethod
     def from_hf_dict(cls, d: dict[str, Any]) -> "ModelConfig":
+        if is_stack_config(d):
+            return cls._stack_from_dict(d)
         mt = d.get("model_type", "llama")
         if mt not in NATIVE_FAMILIES:
             return cls._generic_from_hf_dict(d)
@@ -192,6 +207,18 @@ class ModelConfig:
         return cfg
 
     @classmethod
+    def _stack_from_dict(cls, d: dict[str, Any]) -> "ModelConfig":
+        """A mixer stack: the layer list in typed form; the framework-wide sizes summarise it (planning, reports)."""
+        spec = parse_stack(d)
+        heads = max(l.mixer.heads for l in spec.layers)
+        return cls(model_type=spec.design.lower(), vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+                   intermediate_size=max((l.mlp.ff for l in spec.layers if l.mlp is not None), default=0), num_hidden_layers=len(spec.layers),
+                   num_attention_heads=heads, num_key_value_heads=heads, head_dim=max(l.mixer.vdim for l in spec.layers),
+                   rms_norm_eps=spec.norm_eps, bos_token_id=d.get("bos_token_id"), eos_token_id=d.get("eos_token_id"),
+                   pad_token_id=d.get("pad_token_id"), max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)), stack=spec,
+                   extra={"hf_config": dict(d), "_explicit": ("attention_bias",)})
+
+    @classmethod
     def _generic_from_hf_dict(cls, d: dict[str, Any]) -> "ModelConfig":
         """Description of an architecture outside ``NATIVE_FAMILIES``: the sizes the framework reports and plans with
         (FLOPs estimate, token ids) are read leniently; the complete library configuration travels in ``extra``."""
@@ -216,7 +243,7 @@ class ModelConfig:
             return cls.from_hf_dict(json.load(f))
 
     def to_hf_dict(self) -> dict[str, Any]:
-        if self.is_generic:
+        if self.is_generic or self.is_stack:
             return dict(self.extra["hf_config"])
         arch = {
             "qwen2": "Qwen2ForCausalLM",

@@ -31,7 +31,7 @@ ALIGN = 128  # elements; keeps every view 256-byte aligned in bf16 and shard bou
 class ParamSpec:
     name: str
     shape: tuple
-    init: str = "normal"  # normal | ones | zeros
+    init: str = "normal"  # normal | ones | zeros | fill:<value>
     decay: bool = True
     layer: int = -1  # -1: embedding/pre, num_layers: final norm/head
 
@@ -40,7 +40,23 @@ class ParamSpec:
         return int(math.prod(self.shape))
 
 
+def _stack_param_specs(cfg: ModelConfig) -> list[ParamSpec]:
+    """Mixer stacks: checkpoint names throughout, projections of the same input fused (``mixer_stack_config.fused_rows``)."""
+    from .mixer_stack_config import layer_tensors
+
+    h, L = cfg.hidden_size, cfg.num_hidden_layers
+    specs = [ParamSpec("embed", (cfg.vocab_size, h), "normal", True, -1)]
+    for i, l in enumerate(cfg.stack.layers):
+        if l.owner == i:
+            specs += [ParamSpec(n, shape, init, decay, i) for n, shape, init, decay in layer_tensors(cfg.stack, h, i)]
+    return specs + [ParamSpec("final.norm", (h,), "ones", False, L), ParamSpec("final.norm.b", (h,), "zeros", False, L),
+                    ParamSpec("final.norm.alpha", (1,), "fill:0.5", False, L), ParamSpec("head", (cfg.vocab_size, h), "normal", True, L)]
+
+
 def build_param_specs(cfg: ModelConfig, value_head: bool = False) -> list[ParamSpec]:
+    if cfg.is_stack:
+        assert not value_head, f"{cfg.stack.design}: no value head"
+        return _stack_param_specs(cfg)
     h = cfg.hidden_size
     L = cfg.num_hidden_layers
     specs = []
@@ -170,6 +186,8 @@ class FlatParams:
 
     @property
     def lm_head_weight(self) -> torch.Tensor:
+        if self.cfg.is_stack:
+            return self.views["head"]
         return self.views["embed_tokens.weight"] if "lm_head.weight" not in self.views else self.views["lm_head.weight"]
 
     # ------------------------------------------------------------------ init
@@ -183,6 +201,8 @@ class FlatParams:
                 v.fill_(1.0)
             elif s.init == "zeros":
                 v.zero_()
+            elif s.init.startswith("fill:"):
+                v.fill_(float(s.init[5:]))
             else:
                 if v.is_cuda:
                     g = torch.Generator(device=v.device)
@@ -195,6 +215,18 @@ class FlatParams:
     def hf_views(self, prefix: str = "model.") -> Iterator[tuple[str, torch.Tensor]]:
         """HF-named tensors as zero-copy views of the fused storage."""
         cfg = self.cfg
+        if cfg.is_stack:
+            from .mixer_stack_config import checkpoint_parts
+
+            parts = checkpoint_parts(cfg.stack)
+            for s in self.specs:
+                v = self.views[s.name]
+                if s.name in parts:
+                    for name, r0, rows in parts[s.name]:
+                        yield name, v[r0 : r0 + rows]
+                else:
+                    yield s.name, (v.view(()) if s.name.endswith(".alpha") else v)
+            return
         q, kv = cfg.q_size, cfg.kv_size
         mixtral, phi3 = cfg.model_type == "mixtral", cfg.model_type == "phi3"
         for s in self.specs:

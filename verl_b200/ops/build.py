@@ -35,6 +35,13 @@ NVCC_FLAGS = [
     "-v",
 ]
 
+# sources whose transcendental functions, divisions and square roots keep full fp32 accuracy
+PRECISE_MATH = ("gemm_simt", "mixer_kernels", "latent_attention_simt", "mlstm_chunk", "latent_decode", "latent_prefill_tcgen05")
+
+
+def _nvcc_flags(stem: str) -> list:
+    return [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and stem in PRECISE_MATH)]
+
 
 def _nvcc() -> str:
     cand = os.environ.get("NVCC") or shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
@@ -89,11 +96,11 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     for src in cu:
         obj = BUILD / (src.stem + ".o")
         tag = BUILD / (src.stem + ".hash")
-        want = _hash([src], hdr_hash)
+        want = _hash([src], hdr_hash + " ".join(_nvcc_flags(src.stem)))
         objs.append(obj)
         if obj.exists() and tag.exists() and tag.read_text() == want and not force:
             continue
-        cmd = [_nvcc(), *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
+        cmd = [_nvcc(), *_nvcc_flags(src.stem), "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
         jobs.append((cmd, BUILD / (src.stem + ".log"), tag, want))
     inc = []
     for p in ce.include_paths(device_type="cuda") if "device_type" in ce.include_paths.__code__.co_varnames else ce.include_paths(cuda=True):

@@ -1,0 +1,327 @@
+// torch.ops.verl_b200.* bindings of the mixer-stack kernels.
+#include <ATen/ATen.h>
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/library.h>
+
+#include "launchers.h"
+#include "mixers.h"
+
+namespace {
+
+using at::Tensor;
+using OptTensor = c10::optional<at::Tensor>;
+
+inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
+inline void* ptr(const OptTensor& t) { return t.has_value() ? t->data_ptr() : nullptr; }
+inline int* iptr(const OptTensor& t) { return t.has_value() ? t->data_ptr<int>() : nullptr; }
+inline const long long* lptr(const Tensor& t) { return reinterpret_cast<const long long*>(t.data_ptr<int64_t>()); }
+int dtype_of(const Tensor& t) {
+  TORCH_CHECK(t.is_cuda(), "expected a CUDA tensor");
+  if (t.scalar_type() == at::kFloat) return 0;
+  TORCH_CHECK(t.scalar_type() == at::kBFloat16, "expected an fp32 or bf16 tensor");
+  return 1;
+}
+void same(const Tensor& a, const Tensor& b, const char* what) { TORCH_CHECK(b.is_cuda() && a.scalar_type() == b.scalar_type(), what, ": types differ"); }
+#define CHECK_RC(rc, what) TORCH_CHECK((rc) == 0, what " failed with code ", (rc))
+#define CHECK_F32(x) TORCH_CHECK((x).is_cuda() && (x).scalar_type() == at::kFloat, #x " must be a CUDA fp32 tensor")
+#define CHECK_I32(x) TORCH_CHECK((x).is_cuda() && (x).scalar_type() == at::kInt && (x).is_contiguous(), #x " must be a contiguous int32 CUDA tensor")
+
+// D = epilogue(a w^T): tensor cores where the sizes allow, the fp32-pipeline kernel otherwise.
+void run_gemm(const Tensor& a, const Tensor& w, const VbEpiArgs& e) {
+  const int dt = dtype_of(a);
+  same(a, w, "linear");
+  TORCH_CHECK(a.dim() == 2 && w.dim() == 2 && a.stride(1) == 1 && w.stride(1) == 1 && a.size(1) == w.size(1), "linear: a [M, K], w [N, K]");
+  const int M = (int)a.size(0), K = (int)a.size(1), N = (int)w.size(0);
+  if (M == 0 || N == 0) return;
+  vb_count_launches(1);
+  int rc = -1;
+  if (dt == 1) {
+    if (M <= 1024 && N % 8 == 0 && K % 8 == 0 && a.stride(0) % 8 == 0 && w.stride(0) % 8 == 0) {
+      const int s = vb_gemm_skinny_splits(M, N, K);
+      if (s >= 1) {
+        Tensor ws;
+        if (s > 1) ws = at::empty({s, M, N}, a.options().dtype(at::kFloat));
+        rc = vb_gemm_skinny_epi(a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), w.stride(0), &e, s, s > 1 ? ws.data_ptr<float>() : nullptr, cur_stream());
+      }
+    }
+    if (rc < 0) rc = vb_gemm_bf16_epi(a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), w.stride(0), &e, cur_stream());
+  }
+  if (rc < 0) rc = vb_gemm_simt(dt, a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), w.stride(0), 0, 1, 0, 0, 0, &e, cur_stream());
+  TORCH_CHECK(rc == 0, "linear with epilogue ", e.mode, " failed with code ", rc, " (M=", M, " N=", N, " K=", K, ")");
+}
+
+Tensor linear_act(const Tensor& a, const Tensor& w, bool gelu, bool out_f32) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  Tensor d = at::empty({a.size(0), w.size(0)}, out_f32 ? a.options().dtype(at::kFloat) : a.options());
+  VbEpiArgs e{};
+  e.mode = gelu ? VB_EPI_GELU : (out_f32 ? VB_EPI_STORE_F32 : VB_EPI_STORE);
+  e.D = d.data_ptr(); e.ldd = d.stride(0);
+  run_gemm(a, w, e);
+  return d;
+}
+
+std::tuple<Tensor, Tensor> linear_split(const Tensor& a, const Tensor& w, int64_t n0) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  const int64_t M = a.size(0), N = w.size(0);
+  TORCH_CHECK(n0 > 0 && n0 < N, "linear_split: 0 < n0 < N");
+  Tensor d = at::empty({M, n0}, a.options()), d2 = at::empty({M, N - n0}, a.options().dtype(at::kFloat));
+  VbEpiArgs e{};
+  e.mode = VB_EPI_SPLIT;
+  e.D = d.data_ptr(); e.ldd = n0; e.n0 = (int)n0; e.D2 = d2.data_ptr<float>(); e.ldd2 = N - n0;
+  run_gemm(a, w, e);
+  return {d, d2};
+}
+
+// x += a w^T (fp32 residual stream); returns tanh(alpha x) nw + nb in a's type, or an empty tensor without a norm.
+Tensor linear_residual_(const Tensor& a, const Tensor& w, Tensor x, const OptTensor& alpha, const OptTensor& nw, const OptTensor& nb) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  CHECK_F32(x);
+  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && x.size(0) == a.size(0) && x.size(1) == w.size(0), "linear_residual_: x [M, N]");
+  VbEpiArgs e{};
+  e.mode = VB_EPI_RESID;
+  e.X = x.data_ptr<float>(); e.ldx = x.stride(0);
+  Tensor h;
+  if (nw.has_value()) {
+    same(a, *nw, "linear_residual_");
+    same(a, *nb, "linear_residual_");
+    same(a, *alpha, "linear_residual_");
+    TORCH_CHECK(nw->numel() == w.size(0) && nb->numel() == w.size(0) && alpha->numel() == 1, "linear_residual_: norm sizes");
+    h = at::empty({a.size(0), w.size(0)}, a.options());
+    e.D = h.data_ptr(); e.ldd = h.stride(0); e.alpha = alpha->data_ptr(); e.nw = nw->data_ptr(); e.nb = nb->data_ptr();
+  } else {
+    h = at::empty({0}, a.options());
+  }
+  run_gemm(a, w, e);
+  return h;
+}
+
+std::tuple<Tensor, Tensor> embed_dyt(const Tensor& ids, const Tensor& w, double scale, const Tensor& alpha, const Tensor& nw, const Tensor& nb) {
+  const int dt = dtype_of(w);
+  const c10::cuda::CUDAGuard guard(w.device());
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && w.is_contiguous() && nw.numel() == w.size(1), "embed_dyt");
+  same(w, nw, "embed_dyt");
+  const int T = (int)ids.numel(), W = (int)w.size(1);
+  Tensor x = at::empty({T, W}, w.options().dtype(at::kFloat)), h = at::empty({T, W}, w.options());
+  vb_count_launches(1);
+  CHECK_RC(vb_embed_dyt(dt, lptr(ids), w.data_ptr(), (float)scale, x.data_ptr<float>(), h.data_ptr(), alpha.data_ptr(), nw.data_ptr(),
+                        nb.data_ptr(), T, W, (int)w.size(0), cur_stream()), "vb_embed_dyt");
+  return {x, h};
+}
+
+Tensor dynamic_tanh(const Tensor& x, const Tensor& alpha, const Tensor& nw, const Tensor& nb) {
+  CHECK_F32(x);
+  const int dt = dtype_of(nw);
+  const c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && nw.numel() == x.size(1) && nb.numel() == x.size(1) && alpha.numel() == 1, "dynamic_tanh");
+  Tensor h = at::empty(x.sizes(), nw.options());
+  vb_count_launches(1);
+  CHECK_RC(vb_dyt(dt, x.data_ptr<float>(), h.data_ptr(), alpha.data_ptr(), nw.data_ptr(), nb.data_ptr(), (int)x.size(0), (int)x.size(1), cur_stream()), "vb_dyt");
+  return h;
+}
+
+// In-place rotation of pairs (off + 2i, off + 2i + 1) of every head of x [T, heads, n] (a strided view), i < dims / 2.
+void rope_pairs_(Tensor x, const Tensor& pos, const Tensor& cs, const Tensor& sn, int64_t off, int64_t dims) {
+  const int dt = dtype_of(x);
+  CHECK_I32(pos);
+  CHECK_F32(cs);
+  CHECK_F32(sn);
+  TORCH_CHECK(x.dim() == 3 && x.stride(2) == 1 && off >= 0 && off + dims <= x.size(2) && dims % 2 == 0 && cs.size(1) == dims / 2 && cs.is_contiguous() &&
+              sn.is_contiguous() && pos.numel() == x.size(0), "rope_pairs_");
+  const c10::cuda::CUDAGuard guard(x.device());
+  vb_count_launches(1);
+  CHECK_RC(vb_rope_pairs(dt, x.data_ptr(), pos.data_ptr<int>(), cs.data_ptr<float>(), sn.data_ptr<float>(), (int)x.size(0), (int)x.size(1), x.stride(0),
+                         (int)x.stride(1), (int)off, (int)dims, (int)cs.size(0), cur_stream()), "vb_rope_pairs");
+}
+
+// p [T, q_rank + kv_rank + rot]; pages: view [blocks, block_size, kv_rank + rot] of the cache (or none), slot int64 [T] (negative: no append).
+std::tuple<Tensor, Tensor> latent_prep(const Tensor& p, const Tensor& qn, const Tensor& kn, double eps, const Tensor& pos, const Tensor& cs,
+                                       const Tensor& sn, const OptTensor& pages, const OptTensor& slot, bool want_rows) {
+  const int dt = dtype_of(p);
+  CHECK_I32(pos);
+  same(p, qn, "latent_prep");
+  same(p, kn, "latent_prep");
+  const int64_t T = p.size(0), qr = qn.numel(), kr = kn.numel(), rot = p.size(1) - qr - kr;
+  TORCH_CHECK(p.stride(1) == 1 && rot >= 0 && pos.numel() == T && cs.is_contiguous() && sn.is_contiguous() && 2 * cs.size(1) <= std::max<int64_t>(rot, 0), "latent_prep: sizes");
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor cq = at::empty({T, qr}, p.options());
+  Tensor lat = at::empty({want_rows ? T : 0, kr + rot}, p.options());
+  long long ps = 0, slots = 0;
+  int bs = 1;
+  if (pages.has_value()) {
+    same(p, *pages, "latent_prep");
+    TORCH_CHECK(pages->dim() == 3 && pages->size(2) == kr + rot && pages->stride(2) == 1 && pages->stride(1) == kr + rot && slot.has_value() &&
+                slot->scalar_type() == at::kLong && slot->is_contiguous() && slot->numel() == T, "latent_prep: pages [blocks, block_size, kv_rank + rot]");
+    ps = pages->stride(0); bs = (int)pages->size(1); slots = pages->size(0) * pages->size(1);
+  }
+  vb_count_launches(1);
+  CHECK_RC(vb_latent_prep(dt, p.data_ptr(), p.stride(0), qn.data_ptr(), kn.data_ptr(), (float)eps, pos.data_ptr<int>(), cs.data_ptr<float>(),
+                          sn.data_ptr<float>(), (int)(2 * cs.size(1)), (int)cs.size(0), cq.data_ptr(), want_rows ? lat.data_ptr() : nullptr, kr + rot, ptr(pages), ps, bs,
+                          slots, pages.has_value() ? lptr(*slot) : nullptr, (int)T, (int)qr, (int)kr, (int)rot, cur_stream()), "vb_latent_prep");
+  return {cq, lat};
+}
+
+Tensor gather_pages(const Tensor& pages, const Tensor& block_table, const Tensor& cu_k, const Tensor& k_start, int64_t total) {
+  const int dt = dtype_of(pages);
+  CHECK_I32(block_table);
+  CHECK_I32(cu_k);
+  CHECK_I32(k_start);
+  const c10::cuda::CUDAGuard guard(pages.device());
+  Tensor out = at::empty({total, pages.size(2)}, pages.options());
+  vb_count_launches(1);
+  CHECK_RC(vb_gather_pages(dt, pages.data_ptr(), pages.stride(0), (int)pages.size(1), block_table.data_ptr<int>(), (int)block_table.size(1), cu_k.data_ptr<int>(),
+                           k_start.data_ptr<int>(), (int)k_start.numel(), (int)pages.size(2), out.data_ptr(), (int)total, cur_stream()), "vb_gather_pages");
+  return out;
+}
+
+// out[m, h, :] = a[m, h, :] w[h] (b_mn: w [H, K, N]) or a[m, h, :] w[h]^T (w [H, N, K]), times sigmoid(gate[m, h]).
+Tensor headwise_linear(const Tensor& a, const Tensor& w, bool b_mn, const OptTensor& gate) {
+  const int dt = dtype_of(a);
+  same(a, w, "headwise_linear");
+  TORCH_CHECK(a.dim() == 3 && w.dim() == 3 && a.size(1) == w.size(0) && a.stride(2) == 1 && w.stride(2) == 1 && a.size(2) == (b_mn ? w.size(1) : w.size(2)), "headwise_linear");
+  const c10::cuda::CUDAGuard guard(a.device());
+  const int64_t M = a.size(0), H = a.size(1), K = a.size(2), N = b_mn ? w.size(2) : w.size(1);
+  Tensor d = at::empty({M, H, N}, a.options());
+  VbEpiArgs e{};
+  e.mode = VB_EPI_STORE;
+  e.D = d.data_ptr(); e.ldd = H * N;
+  if (gate.has_value()) {
+    CHECK_F32(*gate);
+    TORCH_CHECK(gate->size(0) == M && gate->size(1) >= H && gate->stride(1) == 1, "headwise_linear: gate [M, H]");
+    e.gate = gate->data_ptr<float>(); e.ldg = gate->stride(0);
+  }
+  vb_count_launches(1);
+  CHECK_RC(vb_gemm_simt(dt, a.data_ptr(), w.data_ptr(), (int)M, (int)N, (int)K, a.stride(0), w.stride(1), b_mn, (int)H, a.stride(1), w.stride(0), N, &e, cur_stream()),
+           "headwise_linear");
+  return d;
+}
+
+// Prompt attention: q [T, H, du + dr], ku [Tk, H, du], kr [Tk, dr], v [Tk, H, dv] (strided views), cu_q / cu_k int32 [B + 1].
+Tensor latent_attn_prefill(const Tensor& q, const Tensor& ku, const Tensor& kr, const Tensor& v, const Tensor& cu_q, const Tensor& cu_k,
+                           const OptTensor& sink, const OptTensor& gate, int64_t window, double scale) {
+  const int dt = dtype_of(q);
+  CHECK_I32(cu_q);
+  CHECK_I32(cu_k);
+  same(q, ku, "latent_attn_prefill");
+  TORCH_CHECK(q.dim() == 3 && ku.dim() == 3 && kr.dim() == 2 && v.dim() == 3 && q.stride(2) == 1 && ku.stride(2) == 1 && kr.stride(1) == 1 && v.stride(2) == 1 &&
+              q.size(2) == ku.size(2) + kr.size(1) && ku.size(1) == q.size(1) && v.size(1) == q.size(1) && cu_q.numel() == cu_k.numel(), "latent_attn_prefill");
+  const c10::cuda::CUDAGuard guard(q.device());
+  VbLatentAttn a{};
+  a.q = q.data_ptr(); a.ldq = q.stride(0); a.hq = (int)q.stride(1);
+  a.ku = ku.data_ptr(); a.ku_row = ku.stride(0); a.ku_head = (int)ku.stride(1);
+  a.kr = kr.data_ptr(); a.kr_row = kr.stride(0);
+  a.v = v.data_ptr(); a.v_row = v.stride(0); a.v_head = (int)v.stride(1);
+  a.cu_q = cu_q.data_ptr<int>(); a.cu_k = cu_k.data_ptr<int>();
+  a.T = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)ku.size(2); a.dr = (int)kr.size(1); a.dv = (int)v.size(2);
+  a.B = (int)cu_q.numel() - 1; a.window = (int)window; a.scale = (float)scale;
+  if (sink.has_value()) { same(q, *sink, "latent_attn_prefill"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
+  if (gate.has_value()) { CHECK_F32(*gate); TORCH_CHECK(gate->size(0) == a.T && gate->stride(1) == 1); a.gate = gate->data_ptr<float>(); a.ldg = gate->stride(0); }
+  Tensor out = at::empty({q.size(0), q.size(1), v.size(2)}, q.options());
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  vb_count_launches(1);
+  CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
+  return out;
+}
+
+// Decode attention in the latent space: q [S, H, kv_rank + rot] (absorbed query, rotated part last), pages [blocks, block_size, kv_rank + rot].
+Tensor latent_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& block_table, const Tensor& ctx_len, const OptTensor& sink,
+                          int64_t kv_rank, int64_t window, double scale) {
+  const int dt = dtype_of(q);
+  same(q, pages, "latent_attn_decode");
+  CHECK_I32(block_table);
+  CHECK_I32(ctx_len);
+  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && pages.dim() == 3 && pages.stride(2) == 1 && pages.size(2) == q.size(2) && kv_rank > 0 && kv_rank <= q.size(2) &&
+              block_table.size(0) == q.size(0) && ctx_len.numel() == q.size(0), "latent_attn_decode");
+  const c10::cuda::CUDAGuard guard(q.device());
+  VbLatentAttn a{};
+  a.q = q.data_ptr(); a.ldq = q.stride(0); a.hq = (int)q.stride(1);
+  char* base = reinterpret_cast<char*>(pages.data_ptr());
+  a.ku = base; a.ku_row = pages.stride(1);
+  a.kr = base + kv_rank * pages.element_size(); a.kr_row = pages.stride(1);
+  a.v = base; a.v_row = pages.stride(1);
+  a.block_table = block_table.data_ptr<int>(); a.max_blocks = (int)block_table.size(1); a.block_size = (int)pages.size(1); a.page_stride = pages.stride(0);
+  a.ctx_len = ctx_len.data_ptr<int>();
+  a.T = a.B = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)kv_rank; a.dr = (int)(q.size(2) - kv_rank); a.dv = (int)kv_rank;
+  a.window = (int)window; a.scale = (float)scale;
+  if (sink.has_value()) { same(q, *sink, "latent_attn_decode"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
+  Tensor out = at::empty({q.size(0), q.size(1), kv_rank}, q.options());
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  vb_count_launches(1);
+  CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
+  return out;
+}
+
+struct MlstmShape { int dt; int64_t T, H, d, e; };
+MlstmShape mlstm_check(const Tensor& p, const Tensor& gates, const Tensor& ib, const Tensor& fb, const Tensor& norm, int64_t d) {
+  MlstmShape s{dtype_of(p), p.size(0), ib.numel(), d, 0};
+  s.e = norm.numel() / s.H;
+  CHECK_F32(gates);
+  same(p, ib, "mlstm");
+  same(p, fb, "mlstm");
+  same(p, norm, "mlstm");
+  TORCH_CHECK(p.dim() == 2 && p.stride(1) == 1 && gates.dim() == 2 && gates.stride(1) == 1 && gates.size(0) == s.T && gates.size(1) >= 2 * s.H && fb.numel() == s.H &&
+              norm.numel() == s.H * s.e && p.size(1) >= 2 * s.H * d + 2 * s.H * s.e, "mlstm: [q | k | v | g] rows and [i | f] gates");
+  return s;
+}
+void mlstm_state_check(const Tensor& state, const MlstmShape& s) {
+  CHECK_F32(state);
+  TORCH_CHECK(state.dim() == 2 && state.stride(1) == 1 && state.size(1) == s.H * (s.d * s.e + s.d + 1), "mlstm: state [slots, H (d e + d + 1)]");
+}
+
+Tensor mlstm_decode(const Tensor& p, const Tensor& gates, const Tensor& ib, const Tensor& fb, double cap, Tensor state, const Tensor& active,
+                    const Tensor& norm, double eps, int64_t d) {
+  const MlstmShape s = mlstm_check(p, gates, ib, fb, norm, d);
+  mlstm_state_check(state, s);
+  TORCH_CHECK(active.is_cuda() && active.scalar_type() == at::kBool && active.is_contiguous() && active.numel() == s.T && state.size(0) >= s.T, "mlstm_decode: active [S]");
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor out = at::empty({s.T, s.H * s.e}, p.options());
+  vb_count_launches(1);
+  CHECK_RC(vb_mlstm_decode(s.dt, p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap, state.data_ptr<float>(),
+                           state.stride(0), reinterpret_cast<const uint8_t*>(active.data_ptr()), norm.data_ptr(), (float)eps, out.data_ptr(), out.stride(0), (int)s.T, (int)s.H,
+                           (int)s.d, (int)s.e, cur_stream()), "vb_mlstm_decode");
+  return out;
+}
+
+// Portion of one or more sequences (cu int32 [B + 1]); slots int32 [B] (or none: nothing is kept), fresh int32 [B]: start from zero.
+Tensor mlstm_prefill(const Tensor& p, const Tensor& gates, const Tensor& ib, const Tensor& fb, double cap, const OptTensor& state, const OptTensor& slots,
+                     const OptTensor& fresh, const Tensor& cu, const Tensor& norm, double eps, int64_t d) {
+  const MlstmShape s = mlstm_check(p, gates, ib, fb, norm, d);
+  CHECK_I32(cu);
+  const int64_t B = cu.numel() - 1;
+  if (slots.has_value()) {
+    TORCH_CHECK(state.has_value() && fresh.has_value(), "mlstm_prefill: slots need a state");
+    mlstm_state_check(*state, s);
+    CHECK_I32(*slots);
+    CHECK_I32(*fresh);
+    TORCH_CHECK(slots->numel() == B && fresh->numel() == B);
+  }
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor o = at::empty({s.T, s.H * s.e}, p.options().dtype(at::kFloat));
+  Tensor out = at::empty({s.T, s.H * s.e}, p.options());
+  vb_count_launches(slots.has_value() ? 3 : 2);
+  CHECK_RC(vb_mlstm_scan(s.dt, p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap,
+                         slots.has_value() ? state->data_ptr<float>() : nullptr, slots.has_value() ? state->stride(0) : 0, iptr(slots), iptr(fresh), cu.data_ptr<int>(), (int)B,
+                         o.data_ptr<float>(), (int)s.T, (int)s.H, (int)s.d, (int)s.e, cur_stream()), "vb_mlstm_scan");
+  const char* g = reinterpret_cast<const char*>(p.data_ptr()) + (2 * s.H * s.d + s.H * s.e) * p.element_size();
+  CHECK_RC(vb_mlstm_out(s.dt, o.data_ptr<float>(), g, p.stride(0), norm.data_ptr(), (float)eps, out.data_ptr(), out.stride(0), (int)s.T, (int)s.H, (int)s.e, cur_stream()),
+           "vb_mlstm_out");
+  return out;
+}
+
+}  // namespace
+
+TORCH_LIBRARY_FRAGMENT(verl_b200, m) {
+  m.def("linear_act", &linear_act);
+  m.def("linear_split", &linear_split);
+  m.def("linear_residual_", &linear_residual_);
+  m.def("embed_dyt", &embed_dyt);
+  m.def("dynamic_tanh", &dynamic_tanh);
+  m.def("rope_pairs_", &rope_pairs_);
+  m.def("latent_prep", &latent_prep);
+  m.def("gather_pages", &gather_pages);
+  m.def("headwise_linear", &headwise_linear);
+  m.def("latent_attn_prefill", &latent_attn_prefill);
+  m.def("latent_attn_decode", &latent_attn_decode);
+  m.def("mlstm_decode", &mlstm_decode);
+  m.def("mlstm_prefill", &mlstm_prefill);
+}

@@ -14,6 +14,7 @@
 // Warp roles (192 threads): warp 0 = TMA producer, warp 1 = MMA issuer (tcgen05.mma, accumulator in TMEM),
 // warps 2..5 = epilogue (tcgen05.ld: thread == weight row, registers == tokens) and fold.
 
+#include "mixer_epilogue.cuh"
 #include "tcgen05_common.cuh"
 
 #include <cuda_bf16.h>
@@ -60,6 +61,7 @@ struct SkinnyParams {
   unsigned int* done;    // per (token block, weight tile): split CTAs that have finished folding
   int* status;
   unsigned long long wait_ns;
+  VbEpiArgs mix;  // elementwise epilogue of the MIX variant (replaces D / bias)
 };
 
 __device__ int g_skinny_status[1];
@@ -93,6 +95,7 @@ __device__ __forceinline__ SkItem sk_item(const SkinnyParams& p, int it) {
   return r;
 }
 
+template <bool MIX>
 __global__ void __launch_bounds__(SK_THREADS, 1)
 gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_constant__ CUtensorMap tma_x,
                    const SkinnyParams p) {
@@ -214,6 +217,8 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
     const int q = warp & 3;  // TMEM lane quarter this warp may access
     const int et = threadIdx.x - 64;
     uint32_t acc_phase = 0;
+    float mix_alpha = 0.f;
+    if constexpr (MIX) mix_alpha = epi_alpha(p.mix);
     for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
       const SkItem w = sk_item(p, it);
       const int nl = q * 32 + lane;          // weight row within the tile
@@ -238,7 +243,13 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
         tmem_ld_wait();
         if (n_ok) {
           const int mrem = mvalid - c * 32;
-          if (direct) {
+          if (MIX && direct) {
+            const int col = w.out_col0 + nl;
+            const EpiColumn ec = epi_column(p.mix, col);
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              if (j < mrem) epi_store1(p.mix, tok0 + c * 32 + j, col, __uint_as_float(r[j]), mix_alpha, ec);
+          } else if (direct) {
 #pragma unroll
             for (int j = 0; j < 32; ++j)
               if (j < mrem) dp[static_cast<long long>(c * 32 + j) * p.ldd] = __float2bfloat16(__uint_as_float(r[j]) + bv);
@@ -309,7 +320,12 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
 #pragma unroll
             for (int u = 0; u < RB; ++u) {
               const int mm = m + 4 * u;
-              if (mm < r1) {
+              if (MIX) {
+                if (mm < r1) {
+                  const float v4[4] = {a[u].x, a[u].y, a[u].z, a[u].w};
+                  epi_store_row<4>(p.mix, mm, col, v4, mix_alpha);
+                }
+              } else if (mm < r1) {
                 uint2 o;
                 o.x = pack_bf16x2(a[u].x, a[u].y);
                 o.y = pack_bf16x2(a[u].z, a[u].w);
@@ -418,10 +434,9 @@ extern "C" int vb_gemm_skinny_status() {
 // floats when splits > 1 (ws_rows = 0 means M).
 // partials_only != 0: leave the partial sums in ws as [splits][ws_rows][N] and do not touch D (bias is ignored).
 // Returns 0 on success, a negative code for arguments the kernel does not serve, a positive cudaError_t otherwise.
-extern "C" int vb_gemm_skinny_seg(const void* X, const void* W, void* D, const void* bias, int M, int K, int w_rows,
-                                  long long ldx, long long ldw, long long ldd, int nseg, const int* seg_w0,
-                                  const int* seg_rows, int splits, float* ws, int ws_rows, int partials_only,
-                                  cudaStream_t stream) {
+static int sk_launch(const void* X, const void* W, void* D, const void* bias, int M, int K, int w_rows, long long ldx, long long ldw,
+                     long long ldd, int nseg, const int* seg_w0, const int* seg_rows, int splits, float* ws, int ws_rows,
+                     int partials_only, const VbEpiArgs* mix, cudaStream_t stream) {
   SkinnyParams p{};
   if (!sk_plan(M, K, nseg, seg_w0, seg_rows, splits, p)) return -1;
   if (splits > 0 && p.splits != splits) return -4;  // the caller sized ws for another split count
@@ -430,7 +445,8 @@ extern "C" int vb_gemm_skinny_seg(const void* X, const void* W, void* D, const v
   if ((ldx % 8) || (ldw % 8)) return -1;
   if ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) & 15) return -2;
   if (p.splits > 1 && ws == nullptr) return -5;
-  if (!partials_only && ((ldd % 4) || (reinterpret_cast<uintptr_t>(D) & 7))) return -2;
+  if (mix == nullptr && !partials_only && ((ldd % 4) || (reinterpret_cast<uintptr_t>(D) & 7))) return -2;
+  if (mix != nullptr) p.mix = *mix;
   const int sms = num_sms();
   const int work = p.num_tiles * p.tblocks;
   if (p.splits > 1 && !partials_only && (work * p.splits > sms || work > SK_SLOT)) return -6;
@@ -460,7 +476,8 @@ extern "C" int vb_gemm_skinny_seg(const void* X, const void* W, void* D, const v
   const int smem = p.stages * stage_bytes + 1024 + 256;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_skinny_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
+    cudaError_t e = cudaFuncSetAttribute(gemm_skinny_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_skinny_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
@@ -481,8 +498,25 @@ extern "C" int vb_gemm_skinny_seg(const void* X, const void* W, void* D, const v
     cfg.attrs = attr;
     cfg.numAttrs = 1;
   }
-  cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel, tw, tx, p);
+  cudaError_t e = mix != nullptr ? cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<true>, tw, tx, p)
+                                 : cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<false>, tw, tx, p);
   return static_cast<int>(e);
+}
+
+extern "C" int vb_gemm_skinny_seg(const void* X, const void* W, void* D, const void* bias, int M, int K, int w_rows,
+                                  long long ldx, long long ldw, long long ldd, int nseg, const int* seg_w0,
+                                  const int* seg_rows, int splits, float* ws, int ws_rows, int partials_only,
+                                  cudaStream_t stream) {
+  return sk_launch(X, W, D, bias, M, K, w_rows, ldx, ldw, ldd, nseg, seg_w0, seg_rows, splits, ws, ws_rows, partials_only, nullptr, stream);
+}
+
+// The same product through an elementwise epilogue of the mixer stack (all rows of W[N, K], one segment). Returns -1 for
+// sizes and alignments it does not serve.
+extern "C" int vb_gemm_skinny_epi(const void* X, const void* W, int M, int N, int K, long long ldx, long long ldw, const VbEpiArgs* e,
+                                  int splits, float* ws, cudaStream_t stream) {
+  if (!epi_aligned(*e, 4) || ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) & 15)) return -1;
+  const int w0 = 0;
+  return sk_launch(X, W, nullptr, nullptr, M, K, N, ldx, ldw, 0, 1, &w0, &N, splits, ws, 0, 0, e, stream);
 }
 
 // All rows of W[N, K]: one segment.

@@ -16,6 +16,7 @@
 //               TMEM accumulators; tcgen05.commit releases smem stages / publishes the accumulator
 //   warps 2..5  epilogue: tcgen05.ld (32 lanes x 32 columns per warp) -> bias -> bf16/fp32 -> global
 // The epilogue of tile i overlaps the main loop of tile i+1 through the double-buffered accumulator.
+#include "mixer_epilogue.cuh"
 #include "tcgen05_common.cuh"
 
 #include <math.h>
@@ -42,7 +43,9 @@ constexpr int GEMM_THREADS = 192;
 //               interleaves the two halves row by row (accumulator column 2j = gate_j, 2j+1 = up_j), so that a thread
 //               holds both members of a pair: D[M, I] = silu(gate) * up as bf16; optionally the pre-activation is
 //               also written in the stacked layout ([M, 2I], what the backward pass of a kept layer reads).
-enum { EPI_STORE = 0, EPI_LSE = 1, EPI_DLOGITS = 2, EPI_ALLREDUCE = 3, EPI_SWIGLU = 4 };
+//  EPI_MIXER    elementwise epilogues of the mixer stack (`mixer_epilogue.cuh`): erf-gelu, residual add with the next norm,
+//               or an output whose last columns stay fp32
+enum { EPI_STORE = 0, EPI_LSE = 1, EPI_DLOGITS = 2, EPI_ALLREDUCE = 3, EPI_SWIGLU = 4, EPI_MIXER = 5 };
 
 constexpr int AR_MAX_RANKS = 8;
 
@@ -107,6 +110,8 @@ struct GemmParams {
   // EPI_SWIGLU: N counts accumulator columns (2 * I); D is the activation [M, I]
   __nv_bfloat16* gu_out;  // pre-activation [M, 2I] (gate columns first), or null
   long long gu_ld;
+  // EPI_MIXER
+  VbEpiArgs mix;
 };
 
 constexpr int FIX_COUNTERS = 16384;
@@ -466,6 +471,8 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
     int acc = 0;
     uint32_t acc_phase = 0;
     bool ok = true;
+    float mix_alpha = 0.f;
+    if constexpr (EPI == EPI_MIXER) mix_alpha = epi_alpha(p.mix);
     for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x) {
       int m0, n0, kb0_, kb1_, b_off_;
       long long d_off;
@@ -483,7 +490,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
       float run_m = -INFINITY, run_l = 0.f, run_s = 0.f;
       long long label = -1;
       float r_lse = 0.f, r_ex = 0.f, r_glp = 0.f, r_gent = 0.f;
-      if constexpr (EPI != EPI_STORE) {
+      if constexpr (EPI != EPI_STORE && EPI != EPI_MIXER) {
         if (row_ok) {
           label = p.labels[row] - p.label_offset;
           if constexpr (EPI == EPI_DLOGITS) {
@@ -591,6 +598,18 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
                   *reinterpret_cast<uint2*>(go + j) = g4;
                   *reinterpret_cast<uint2*>(go + inter + j) = u4;
                 }
+              }
+            }
+          }
+        } else if constexpr (EPI == EPI_MIXER) {
+          if (row_ok) {
+#pragma unroll
+            for (int j = 0; j < 32; j += 8) {
+              if (j < ncols) {
+                float v[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(r[j + i]);
+                epi_store_row<8>(p.mix, row, col0 + j, v, mix_alpha);
               }
             }
           }
@@ -1105,6 +1124,21 @@ extern "C" int vb_gemm_bf16_swiglu(const void* A, const void* W, void* act, void
   p.M = M; p.N = 2 * I; p.K = K; p.D = act; p.ldd = ldd; p.status = status_ptr(); p.k_splits = 1;
   p.gu_out = reinterpret_cast<__nv_bfloat16*>(gu_out); p.gu_ld = gu_ld;
   return static_cast<int>(launch_variant<256, false, false, 4, EPI_SWIGLU>(ta, tb, p, num_sms(), stream));
+}
+
+// D = epilogue(A B^T) for the mixer-stack epilogues; A [M, K], B [N, K]. Returns -1 for sizes the TMA path does not serve.
+extern "C" int vb_gemm_bf16_epi(const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, const VbEpiArgs* e,
+                                cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((N % 8) || (lda % 8) || (ldb % 8) || ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B)) & 15) || !epi_aligned(*e, 8)) return -1;
+  const bool wide = N > 128;
+  CUtensorMap ta, tb;
+  if (!make_tmap_2d(&ta, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, K, lda, BK, BM, CU_TENSOR_MAP_SWIZZLE_128B)) return -3;
+  if (!make_tmap_2d(&tb, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, N, K, ldb, BK, wide ? 256 : 128, CU_TENSOR_MAP_SWIZZLE_128B)) return -3;
+  GemmParams p{};
+  p.M = M; p.N = N; p.K = K; p.status = status_ptr(); p.k_splits = 1; p.mix = *e;
+  return static_cast<int>(wide ? launch_variant<256, false, false, 4, EPI_MIXER>(ta, tb, p, num_sms(), stream)
+                               : launch_variant<128, false, false, 6, EPI_MIXER>(ta, tb, p, num_sms(), stream));
 }
 
 // Row-parallel linear of a tensor-parallel group with the all-reduce done inside the GEMM epilogue over peer memory:

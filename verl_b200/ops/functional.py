@@ -211,8 +211,7 @@ def rope_inv_freq(head_dim: int, theta: float, scaling: Optional[dict] = None, m
         if scaling.get("truncate", True):
             low, high = math.floor(low), math.ceil(high)
         low, high = max(low, 0), min(high, head_dim - 1)
-        if low == high:
-            high += 0.001
+        high = max(high, low + 0.001)
         ramp = ((torch.arange(head_dim // 2, dtype=torch.float64) - low) / (high - low)).clamp(0.0, 1.0)
         inv = inv / factor * ramp + inv * (1 - ramp)
         att = scaling.get("attention_factor")

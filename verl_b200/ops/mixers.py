@@ -1,0 +1,247 @@
+"""Operators of the mixer stacks (``models/mixer_stack.py``): Dynamic Tanh, GEMMs with fused epilogues, latent attention over
+expanded keys (prompts) and over the paged latents (decoding), and the mLSTM recurrence.
+
+As in ``functional``: CUDA tensors go to the hand-written kernels (bf16 or true fp32; nothing falls back silently), CPU
+tensors take a plain PyTorch path. The residual stream, gates, statistics and recurrent state are fp32 on every path.
+"""
+
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+import torch.nn.functional as TF
+
+from . import native
+
+__all__ = ["embed_dyt", "dynamic_tanh", "linear_act", "linear_split", "linear_residual_", "rope_pairs_", "latent_prep", "gather_pages",
+           "headwise_linear", "latent_attention_prefill", "latent_attention_decode", "mlstm_prefill", "mlstm_decode"]
+
+
+def _ops():
+    return native.ops()
+
+
+def _mm(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    return a.float() @ w.float().t()
+
+
+# ----------------------------------------------------------------------------------------------- norm, embedding, GEMMs
+def dynamic_tanh(x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """``tanh(alpha x) * weight + bias`` of the fp32 stream, in the weights' type (no statistics over the row)."""
+    if x.is_cuda:
+        return _ops().dynamic_tanh(x, alpha, weight, bias)
+    return (torch.tanh(alpha.float() * x) * weight.float() + bias.float()).to(weight.dtype)
+
+
+def embed_dyt(ids, weight, scale: float, alpha, nw, nb):
+    """(fp32 residual stream ``weight[ids] * scale``, its first Dynamic Tanh)."""
+    if weight.is_cuda:
+        return _ops().embed_dyt(ids.reshape(-1).contiguous(), weight, float(scale), alpha, nw, nb)
+    x = weight[ids.reshape(-1)].float() * scale
+    return x, dynamic_tanh(x, alpha, nw, nb)
+
+
+def linear_act(a: torch.Tensor, w: torch.Tensor, act: Optional[str] = None, out_f32: bool = False) -> torch.Tensor:
+    """``a w^T`` with an optional activation (``gelu_erf``) in the epilogue."""
+    assert act in (None, "gelu_erf")
+    if a.is_cuda:
+        return _ops().linear_act(a, w, act == "gelu_erf", bool(out_f32))
+    y = _mm(a, w)
+    y = TF.gelu(y) if act == "gelu_erf" else y
+    return y if out_f32 else y.to(a.dtype)
+
+
+def linear_split(a: torch.Tensor, w: torch.Tensor, n0: int):
+    """``a w^T`` whose first ``n0`` columns come in ``a``'s type and the rest as fp32 (gates that must not be rounded)."""
+    if a.is_cuda:
+        return _ops().linear_split(a, w, int(n0))
+    y = _mm(a, w)
+    return y[:, :n0].to(a.dtype).contiguous(), y[:, n0:].contiguous()
+
+
+def linear_residual_(a: torch.Tensor, w: torch.Tensor, x: torch.Tensor, norm=None) -> Optional[torch.Tensor]:
+    """``x += a w^T`` on the fp32 residual stream; with ``norm = (alpha, weight, bias)`` also returns the Dynamic Tanh of the
+    new stream, computed in the same epilogue."""
+    if a.is_cuda:
+        h = _ops().linear_residual_(a, w, x, *(norm if norm is not None else (None, None, None)))
+        return h if norm is not None else None
+    x += _mm(a, w)
+    return dynamic_tanh(x, *norm) if norm is not None else None
+
+
+# ----------------------------------------------------------------------------------------------- latent attention
+def _rotate(x: torch.Tensor, pos: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+    """``x`` [T, ..., n] fp32: pairs (2i, 2i + 1) of the first ``2 * cos.shape[1]`` dimensions are turned."""
+    half = cos.shape[1]
+    shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (half,)
+    c, s = cos[pos.long()].view(shape), sin[pos.long()].view(shape)
+    pairs = x[..., : 2 * half].unflatten(-1, (half, 2))
+    u, v = pairs[..., 0], pairs[..., 1]
+    return torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., 2 * half :]], -1)
+
+
+def rope_pairs_(x: torch.Tensor, positions: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, offset: int = 0) -> torch.Tensor:
+    """In-place interleaved rotation of ``x`` [T, heads, n] from dimension ``offset`` on (``2 * cos.shape[1]`` dimensions)."""
+    if x.is_cuda:
+        _ops().rope_pairs_(x, positions, cos, sin, int(offset), int(2 * cos.shape[1]))
+        return x
+    x[..., offset:] = _rotate(x[..., offset:].float(), positions, cos, sin).to(x.dtype)
+    return x
+
+
+def latent_prep(p, q_norm, kv_norm, eps: float, positions, cos, sin, pages=None, slots=None, want_rows: bool = False):
+    """``p`` [T, q_rank + kv_rank + rot]: RMS-normed query latent, and the row [normed latent | rotated shared key part], which
+    is appended to ``pages`` [blocks, block_size, kv_rank + rot] at ``slots`` (negative: skipped) and / or returned."""
+    if p.is_cuda:
+        return _ops().latent_prep(p, q_norm, kv_norm, float(eps), positions, cos, sin, pages, slots, bool(want_rows))
+    qr, kr = q_norm.numel(), kv_norm.numel()
+    rms = lambda z, w: z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    f = p.float()
+    cq = rms(f[:, :qr], q_norm).to(p.dtype)
+    row = torch.cat([rms(f[:, qr : qr + kr], kv_norm), _rotate(f[:, qr + kr :], positions, cos, sin)], -1).to(p.dtype)
+    if pages is not None:
+        ok = slots >= 0
+        at, bs = slots[ok], pages.shape[1]
+        pages[at // bs, at % bs] = row[ok]
+    return cq, (row if want_rows else row[:0])
+
+
+def gather_pages(pages, block_table, cu_k, k_start, total: int) -> torch.Tensor:
+    """[total, width]: for every sequence the cached rows ``k_start[b] .. k_start[b] + cu_k[b + 1] - cu_k[b]`` in order."""
+    if pages.is_cuda:
+        return _ops().gather_pages(pages, block_table, cu_k, k_start, int(total))
+    bs, out = pages.shape[1], []
+    for b in range(block_table.shape[0]):
+        at = int(k_start[b]) + torch.arange(int(cu_k[b + 1] - cu_k[b]))
+        out.append(pages[block_table[b, at // bs].long(), at % bs])
+    return torch.cat(out, 0)
+
+
+def headwise_linear(a: torch.Tensor, w: torch.Tensor, transposed: bool, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per-head product: ``a`` [M, H, K] with ``w`` [H, N, K], or ``w`` [H, K, N] when ``transposed``; head h of row m is multiplied
+    by ``sigmoid(gate[m, h])`` when a gate is given."""
+    if a.is_cuda:
+        return _ops().headwise_linear(a, w, bool(transposed), gate)
+    y = torch.einsum("mhk,hkn->mhn" if transposed else "mhk,hnk->mhn", a.float(), w.float())
+    if gate is not None:
+        y = y * torch.sigmoid(gate[:, : a.shape[1]]).unsqueeze(-1)
+    return y.to(a.dtype).contiguous()
+
+
+def _sink_softmax(s: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor:
+    """Softmax over the last dimension of ``s`` [H, ..., keys] with one extra score per head that has no value."""
+    if sink is None:
+        return torch.softmax(s, -1)
+    extra = sink.float().view(-1, *([1] * (s.dim() - 1))).expand(*s.shape[:-1], 1)
+    return torch.softmax(torch.cat([s, extra], -1), -1)[..., :-1]
+
+
+def latent_attention_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, window: int, scale: float, sink=None, gate=None) -> torch.Tensor:
+    """Causal windowed attention of packed prompts: ``q`` [T, H, du + dr] (rotated part last), ``k_unrot`` [Tk, H, du], ``k_rot``
+    [Tk, dr] shared by the heads, ``v`` [Tk, H, dv]; the last query of a sequence sits on its last key (``cu_k`` may hold earlier
+    keys). ``window`` > 0: a query sees that many keys, its own included. Output times ``sigmoid(gate[t, h])``."""
+    if q.is_cuda:
+        return _ops().latent_attn_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, sink, gate, int(window), float(scale))
+    out = torch.empty(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype)
+    du = k_unrot.shape[2]
+    cq, ck = cu_q.tolist(), cu_k.tolist()
+    for b in range(len(cq) - 1):
+        qs, ks = slice(cq[b], cq[b + 1]), slice(ck[b], ck[b + 1])
+        nq, nk = cq[b + 1] - cq[b], ck[b + 1] - ck[b]
+        qq = q[qs].float()
+        s = torch.einsum("qhd,khd->hqk", qq[..., :du], k_unrot[ks].float()) + torch.einsum("qhd,kd->hqk", qq[..., du:], k_rot[ks].float())
+        dist = torch.arange(nk - nq, nk)[:, None] - torch.arange(nk)[None, :]
+        hide = (dist < 0) | ((dist >= window) if window > 0 else torch.zeros_like(dist, dtype=torch.bool))
+        p = _sink_softmax((s * scale).masked_fill(hide, float("-inf")), sink)
+        o = torch.einsum("hqk,khd->qhd", p, v[ks].float())
+        if gate is not None:
+            o = o * torch.sigmoid(gate[qs, : q.shape[1]])[:, :, None]
+        out[qs] = o.to(q.dtype)
+    return out
+
+
+def latent_attention_decode(q, pages, block_table, ctx_len, kv_rank: int, window: int, scale: float, sink=None) -> torch.Tensor:
+    """One query per sequence in the latent space: ``q`` [S, H, kv_rank + rot] against the cached rows, which are key (whole row)
+    and value (first ``kv_rank``) of every head. Returns [S, H, kv_rank]; sequences with ``ctx_len`` 0 give zeros."""
+    if q.is_cuda:
+        return _ops().latent_attn_decode(q, pages, block_table, ctx_len, sink, int(kv_rank), int(window), float(scale))
+    out = torch.zeros(q.shape[0], q.shape[1], kv_rank, dtype=q.dtype)
+    bs = pages.shape[1]
+    for b, n in enumerate(ctx_len.tolist()):
+        if n <= 0:
+            continue
+        at = torch.arange(max(0, n - window) if window > 0 else 0, n)
+        rows = pages[block_table[b, at // bs].long(), at % bs].float()
+        p = _sink_softmax(q[b].float() @ rows.t() * scale, sink)
+        out[b] = (p @ rows[:, :kv_rank]).to(q.dtype)
+    return out
+
+
+# ----------------------------------------------------------------------------------------------- mLSTM
+def _mlstm_parts(p, gates, ib, fb, cap: float, d: int, e: int):
+    T, H = p.shape[0], ib.numel()
+    f = p.float()
+    q = f[:, : H * d].view(T, H, d) * d ** -0.5
+    k = f[:, H * d : 2 * H * d].view(T, H, d)
+    v = f[:, 2 * H * d : 2 * H * d + H * e].view(T, H, e)
+    g = f[:, 2 * H * d + H * e : 2 * H * (d + e)].view(T, H, e)
+    i_log = cap * torch.tanh((gates[:, :H] + ib.float()) / cap)
+    f_log = TF.logsigmoid(cap * torch.tanh((gates[:, H : 2 * H] + fb.float()) / cap))
+    return q, k, v, g, i_log, f_log
+
+
+def _mlstm_finish(o, g, norm, eps: float, dtype):
+    H, e = o.shape[1], o.shape[2]
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm.float().view(H, e) * torch.sigmoid(g)
+    return o.reshape(o.shape[0], H * e).to(dtype)
+
+
+def _state_views(row: torch.Tensor, H: int, d: int, e: int):
+    return row[: H * d * e].view(H, d, e), row[H * d * e : H * d * e + H * d].view(H, d), row[H * d * e + H * d : H * (d * e + d + 1)]
+
+
+def _mlstm_token(S, n, m, q, k, v, i_log, f_log):
+    """One token of one sequence, in place on the state views; returns o [H, e]."""
+    m_new = torch.maximum(f_log + m, i_log)
+    keep, add = torch.exp(f_log + m - m_new), torch.exp(i_log - m_new)
+    S.mul_(keep[:, None, None]).add_((add[:, None] * k)[:, :, None] * v[:, None, :])
+    n.mul_(keep[:, None]).add_(add[:, None] * k)
+    m.copy_(m_new)
+    den = torch.maximum((n * q).sum(-1).abs(), torch.exp(-m)) + 1e-6
+    return torch.einsum("hde,hd->he", S, q) / den[:, None]
+
+
+def mlstm_prefill(p, gates, ib, fb, cap: float, norm, eps: float, dim: int, cu, state=None, slots=None, fresh=None) -> torch.Tensor:
+    """Matrix-memory recurrence over packed portions. ``p`` [T, q | k | v | g] in the model's type, ``gates`` [T, i | f] fp32
+    pre-activations. Sequence b starts from zero when ``fresh[b]`` (else from ``state[slots[b]]``) and leaves its final state in
+    ``state[slots[b]]``; without ``slots`` every sequence starts from zero and nothing is kept."""
+    if p.is_cuda:
+        return _ops().mlstm_prefill(p, gates, ib, fb, float(cap), state, slots, fresh, cu, norm, float(eps), int(dim))
+    H = ib.numel()
+    e = norm.numel() // H
+    q, k, v, g, il, fl = _mlstm_parts(p, gates, ib, fb, cap, dim, e)
+    out = torch.empty(p.shape[0], H, e)
+    c = cu.tolist()
+    for b in range(len(c) - 1):
+        row = torch.zeros(H * (dim * e + dim + 1)) if slots is None else state[int(slots[b])]
+        if slots is not None and bool(fresh[b]):
+            row.zero_()
+        S, n, m = _state_views(row, H, dim, e)
+        for t in range(c[b], c[b + 1]):
+            out[t] = _mlstm_token(S, n, m, q[t], k[t], v[t], il[t], fl[t])
+    return _mlstm_finish(out, g, norm, eps, p.dtype)
+
+
+def mlstm_decode(p, gates, ib, fb, cap: float, norm, eps: float, dim: int, state, active) -> torch.Tensor:
+    """One token per slot: row s of ``p`` updates ``state[s]`` when ``active[s]`` (inactive slots keep theirs and give zeros)."""
+    if p.is_cuda:
+        return _ops().mlstm_decode(p, gates, ib, fb, float(cap), state, active, norm, float(eps), int(dim))
+    H = ib.numel()
+    e = norm.numel() // H
+    q, k, v, g, il, fl = _mlstm_parts(p, gates, ib, fb, cap, dim, e)
+    out = torch.zeros(p.shape[0], H, e)
+    for s in torch.nonzero(active).flatten().tolist():
+        S, n, m = _state_views(state[s], H, dim, e)
+        out[s] = _mlstm_token(S, n, m, q[s], k[s], v[s], il[s], fl[s])
+    return _mlstm_finish(out, g, norm, eps, p.dtype)

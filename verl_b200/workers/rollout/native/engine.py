@@ -16,6 +16,8 @@ Design (one engine per GPU, or per tensor-parallel group):
   head_dim]``; a sequence reserves the blocks for ``prompt + max_new_tokens`` at admission and returns
   them when it retires.  ``release_kv_cache`` / ``resume_kv_cache`` hand the pool's memory back to the
   trainer between rollout phases.
+* **Mixer stacks** (decoders whose layers differ, ``models/mixer_stack.py``) share the slots, blocks, scheduler, decode loop
+  and sampler; their cache (``cache.py``) is a page pool of latent rows plus one recurrent-state row per slot.
 * **Prefill** runs the packed varlen forward of the training model with a hook that scatters rotated
   K/V into the cache, in chunks of at most ``max_num_batched_tokens`` tokens.
 
@@ -37,10 +39,12 @@ from typing import Optional, Sequence
 import torch
 import torch.distributed as dist
 
+from ....models import build_decoder
 from ....models.config import ModelConfig
-from ....models.decoder import DecoderModel, PackedBatch, TensorParallelShard
+from ....models.decoder import PackedBatch, TensorParallelShard
 from ....models.weights import FlatParams
 from ....ops import functional as F
+from .cache import make_cache
 
 __all__ = ["SamplingParams", "RequestOutput", "RolloutEngine"]
 
@@ -81,6 +85,15 @@ class _Request:
     cached: int = 0                 # leading prompt tokens whose pages came from the prefix cache
 
 
+@dataclass
+class _Sequence:
+    """A sequence whose tokens are given from outside (``open_sequence``): its slot, pages and length so far."""
+
+    slot: int
+    blocks: list[int] = field(default_factory=list)
+    length: int = 0
+
+
 class RolloutEngine:
     def __init__(self, cfg: ModelConfig, params: FlatParams, *, max_num_seqs: int = 256,
                  max_num_batched_tokens: int = 8192, max_model_len: int = 4096, block_size: int = 64,
@@ -98,8 +111,10 @@ class RolloutEngine:
         # Prefix cache across requests: full pages stay indexed by a chain hash of their tokens after their last user has
         # finished (evicted least-recently-used when fresh pages run out); a new prompt that starts with cached pages (the
         # next turn of a conversation, a shared system prompt) points at them and is prefilled from the first uncached token.
-        # Emptied with every weight update. Off with routing recording (a cached page has no routing record).
-        self.enable_prefix_caching = bool(enable_prefix_caching) and not (bool(record_routing) and cfg.is_moe)
+        # Emptied with every weight update. Off with routing recording (a cached page has no routing record) and for models with
+        # recurrent layers (their state behind a page is not in the page).
+        self.enable_prefix_caching = (bool(enable_prefix_caching) and not (bool(record_routing) and cfg.is_moe)
+                                      and not (cfg.is_stack and cfg.stack.recurrent))
         self._page_of_hash: dict = {}      # chain hash -> page
         self._hash_of_page: dict = {}      # page -> chain hash
         self._idle_cached: "OrderedDict[int, None]" = OrderedDict()   # indexed pages without a user, oldest first
@@ -112,6 +127,8 @@ class RolloutEngine:
         self.tp_rank = dist.get_rank(tp_group) if tp_group is not None else 0
         assert cfg.num_key_value_heads % self.tp_size == 0 and (cfg.is_moe or cfg.intermediate_size % (8 * self.tp_size) == 0), \
             "tensor-parallel size must divide the KV heads and the MLP width"
+        assert not cfg.is_stack or (self.tp_size == 1 and self.quantization is None), \
+            f"{cfg.model_type}: served on one GPU per replica, without quantised weights"
         self.params = params
         self.device = params.flat.device
         self.is_cuda = self.device.type == "cuda"
@@ -122,12 +139,14 @@ class RolloutEngine:
         self.max_blocks_per_seq = (self.max_model_len + self.bs - 1) // self.bs
         self.eos = eos_token_id if eos_token_id is not None else cfg.eos_token_id
         self.valid_vocab = valid_vocab_size or cfg.vocab_size
-        self.use_graph = bool(use_cuda_graph) and self.is_cuda
+        self.use_graph = bool(use_cuda_graph) and self.is_cuda and params.flat.dtype == torch.bfloat16
         self.sync_interval = max(1, int(sync_interval))
         self.gpu_memory_utilization = gpu_memory_utilization
         self._num_blocks_req = num_blocks
-        self.model = DecoderModel(cfg, params, max_positions=self.max_model_len + 1)
+        self.model = build_decoder(cfg, params, max_positions=self.max_model_len + 1)
         self.model.kv_hook = self._prefill_kv_hook
+        self.cache = make_cache(cfg, params.flat.dtype, self.device, self.bs, self.S, self.tp_size)
+        self.sequences: dict[str, _Sequence] = {}
         self._tp_share = None
         if self.tp_size > 1:
             assert not cfg.is_moe, "tensor-parallel rollout of MoE models is not implemented (use expert parallelism)"
@@ -176,19 +195,19 @@ class RolloutEngine:
 
     # ------------------------------------------------------------------------------------ memory
     def kv_bytes_per_block(self) -> int:
-        c = self.cfg
-        return c.num_hidden_layers * 2 * self.bs * (c.kv_size // self.tp_size) * self.params.flat.element_size()
+        return self.cache.bytes_per_block()
 
     def resume_kv_cache(self) -> None:
         if self.kv is not None:
             return
-        c = self.cfg
         n = self._num_blocks_req
         if n is None:
             if self.is_cuda:
                 torch.cuda.empty_cache()  # cached-but-unused allocator blocks would otherwise count as occupied
                 free, total = torch.cuda.mem_get_info(self.device)
                 budget = min(free - (2 << 30), int(total * self.gpu_memory_utilization))
+                if self.cache.has_state:
+                    budget -= self.S * self.cache.state_elems * 4
                 n = max(self.max_blocks_per_seq, int(budget // self.kv_bytes_per_block()))
             else:
                 n = self.S * self.max_blocks_per_seq
@@ -198,8 +217,8 @@ class RolloutEngine:
             dist.all_reduce(t, op=dist.ReduceOp.MIN, group=self.tp_group)
             n = int(t.item())
         self.num_blocks = int(n)
-        self.kv = torch.zeros(c.num_hidden_layers, 2, self.num_blocks, self.bs, c.num_key_value_heads // self.tp_size, c.head_dim,
-                              dtype=self.params.flat.dtype, device=self.device)
+        self.cache.allocate(self.num_blocks)
+        self.kv = self.cache.kv
         self.free_blocks = list(range(self.num_blocks - 1, -1, -1))
         self._block_users = {}
         self._graph = None  # cache addresses changed
@@ -252,8 +271,9 @@ class RolloutEngine:
         self._idle_cached.clear()
 
     def release_kv_cache(self) -> None:
-        assert not self.running, "cannot release the KV cache with sequences in flight"
+        assert not self.running and not self.sequences, "cannot release the KV cache with sequences in flight"
         self.kv = None
+        self.cache.free()
         self._graph = None
         self.free_blocks = []
         self._block_users = {}
@@ -263,7 +283,7 @@ class RolloutEngine:
 
     def clear_kv_cache(self) -> None:
         """Forget all cached content (called after every weight update)."""
-        assert not self.running
+        assert not self.running and not self.sequences
         if self.quantization == "fp8":
             self.model.quantize_linear_weights_fp8()  # the bf16 weights changed: refresh the e4m3 copies
             self._graph = None
@@ -299,7 +319,7 @@ class RolloutEngine:
         nkv_l = self.cfg.num_key_value_heads // self.tp_size
         # VERL_B200_FUSED_ROPE_APPEND=0: rotate q, rotate k and append to the cache as three launches instead of one
         self.fused_rope_append = os.environ.get("VERL_B200_FUSED_ROPE_APPEND", "1") != "0"
-        self.grouped_decode = (self.is_cuda and self.share_prefill and self.bs == 64 and self.cfg.head_dim in (64, 128)
+        self.grouped_decode = (self.is_cuda and self.share_prefill and not self.cfg.is_stack and self.bs == 64 and self.cfg.head_dim in (64, 128)
                                and nh_l // max(1, nkv_l) <= 16 and os.environ.get("VERL_B200_GROUPED_DECODE", "0") == "1")
         self._groups: dict[int, list[int]] = {}
         self._slot_group: dict[int, int] = {}
@@ -466,7 +486,7 @@ class RolloutEngine:
             for r in reqs:
                 nb = (len(r.prompt) + self.bs - 1) // self.bs
                 blk = torch.tensor(r.blocks[:nb], dtype=torch.int64, device=self.device)
-                out[r.rid] = dict(prompt=list(r.prompt), kv=self.kv[:, :, blk].clone(), token=int(self.tok[r.slot]),
+                out[r.rid] = dict(prompt=list(r.prompt), **self.cache.export(blk, r.slot), token=int(self.tok[r.slot]),
                                   logprob=float(self.out_lp[r.slot, 0]), seed=int(self.seeds[r.slot]), block_size=self.bs,
                                   routed_prompt=getattr(r, "routed_prompt", None))
             idx = torch.tensor([r.slot for r in reqs], dtype=torch.int64, device=self.device)
@@ -495,7 +515,7 @@ class RolloutEngine:
             bt_rows[i, : len(r.blocks)] = torch.tensor(r.blocks, dtype=torch.int32)
             nb = (lens[i] + self.bs - 1) // self.bs
             dst = torch.tensor(r.blocks[:nb], dtype=torch.int64, device=dev)
-            self.kv[:, :, dst] = r.handoff["kv"].to(dev, dtype=self.kv.dtype)   # the KV transfer (a peer copy between GPUs)
+            self.cache.install(dst, r.slot, r.handoff)   # the KV transfer (a peer copy between GPUs)
             if self.record_routing:
                 r.routed_prompt = r.handoff.get("routed_prompt")
         slots = torch.tensor([r.slot for r in reqs], dtype=torch.int64, device=dev)
@@ -534,6 +554,47 @@ class RolloutEngine:
         self.active[slots] = ~done
         for r in reqs:
             self.running[r.slot] = r
+
+    @torch.no_grad()
+    def _run_portions(self, ids: torch.Tensor, starts: list[int], ends: list[int], bt_rows: torch.Tensor, slots: list[int]):
+        """Tokens ``starts[i] .. ends[i]`` of every sequence (packed in ``ids``, host) through the model in one batch, appended to
+        the cache behind the ``starts[i]`` tokens it already holds. ``bt_rows`` [B, blocks] (host): the sequences' block tables;
+        ``slots``: their slots. Returns (final hidden states [T, H], the packed batch)."""
+        dev = self.device
+        slot_rows = []
+        for i, (a, b) in enumerate(zip(starts, ends)):
+            p = torch.arange(a, b)
+            slot_rows.append(bt_rows[i, p // self.bs].long() * self.bs + p % self.bs)
+        slot_map = torch.cat(slot_rows)
+        if self.is_cuda:
+            ids, slot_map = ids.pin_memory().to(dev, non_blocking=True), slot_map.pin_memory().to(dev, non_blocking=True)
+        batch = PackedBatch.from_lengths(ids, [b - a for a, b in zip(starts, ends)], device=dev)
+        if any(starts):
+            batch.positions = torch.cat([torch.arange(a, b, dtype=torch.int32) for a, b in zip(starts, ends)]).to(dev)
+        if self.cfg.is_stack:
+            from ....models.mixer_stack import PortionCache
+
+            pc = PortionCache(self.cache, slot_map, torch.tensor(slots, dtype=torch.int32).to(dev), list(starts), bt_rows.to(dev))
+            return self.model.forward_hidden(batch, pc), batch
+        if any(starts):
+            rows = []
+            for i, a in enumerate(starts):
+                p = torch.arange(a)
+                rows.append(bt_rows[i, p // self.bs].long() * self.bs + p % self.bs)
+            cached_slots = torch.cat(rows).to(dev)
+            nkv_l, hd = self.kv.shape[-2], self.kv.shape[-1]
+            self.model.prefix_kv = lambda layer: (self.kv[layer, 0].view(-1, nkv_l, hd)[cached_slots],
+                                                  self.kv[layer, 1].view(-1, nkv_l, hd)[cached_slots], list(starts))
+            self.model._ensure_rope(max(ends) + 1)
+        self._prefill_slots = slot_map
+        try:
+            return self.model.forward_hidden(batch), batch
+        finally:
+            self._prefill_slots = None
+            self.model.prefix_kv = None
+
+    def _logits(self, h: torch.Tensor) -> torch.Tensor:
+        return self.model.logits(h) if self.cfg.is_stack else F.gemm(h, self.params.lm_head_weight)
 
     @torch.no_grad()
     def _prefill(self, reqs: list[_Request]) -> None:
@@ -575,34 +636,13 @@ class RolloutEngine:
             bt_rows[i, : len(r.blocks)] = torch.tensor(r.blocks, dtype=torch.int32)
         skip = [reqs[i].cached for i in leaders]        # tokens whose pages came from the prefix cache: not recomputed
         ids = torch.tensor([t for i in leaders for t in reqs[i].prompt[reqs[i].cached:]], dtype=torch.int64)
-        slot_rows = []
-        for i in leaders:
-            p = torch.arange(reqs[i].cached, lens[i])
-            slot_rows.append(bt_rows[i, p // self.bs].long() * self.bs + p % self.bs)
-        if self.is_cuda:
-            ids, slot_map = ids.pin_memory().to(dev, non_blocking=True), torch.cat(slot_rows).pin_memory().to(dev, non_blocking=True)
-        else:
-            slot_map = torch.cat(slot_rows)
-        batch = PackedBatch.from_lengths(ids, [lens[i] - c for i, c in zip(leaders, skip)], device=dev)
         if any(skip):
-            batch.positions = torch.cat([torch.arange(c, lens[i], dtype=torch.int32) for i, c in zip(leaders, skip)]).to(dev)
-            pages = torch.cat([bt_rows[i, : c // self.bs].long() for i, c in zip(leaders, skip)])
-            cached_slots = (pages.unsqueeze(1) * self.bs + torch.arange(self.bs).unsqueeze(0)).reshape(-1).to(dev)
-            nkv_l, hd = self.kv.shape[-2], self.kv.shape[-1]
-            self.model.prefix_kv = lambda layer: (self.kv[layer, 0].view(-1, nkv_l, hd)[cached_slots],
-                                                  self.kv[layer, 1].view(-1, nkv_l, hd)[cached_slots], skip)
-            self.model._ensure_rope(max(lens) + 1)
             self.stats["prefix_cache_hit_tokens"] = self.stats.get("prefix_cache_hit_tokens", 0) + sum(skip)
-        self._prefill_slots = slot_map
         if self.record_routing:
             from ....models.decoder import RouterReplay
 
             self.model.router_replay = RouterReplay("record")
-        try:
-            h = self.model.forward_hidden(batch)
-        finally:
-            self._prefill_slots = None
-            self.model.prefix_kv = None
+        h, batch = self._run_portions(ids, skip, [lens[i] for i in leaders], bt_rows[leaders], [reqs[i].slot for i in leaders])
         if self.enable_prefix_caching:
             for i in leaders:
                 self._index_pages(reqs[i].prompt, reqs[i].blocks, lens[i])
@@ -616,7 +656,7 @@ class RolloutEngine:
                 j = lead_idx[i]
                 r.routed_prompt = routed[cu[j] : cu[j + 1]]
         last = (batch.cu_seqlens[1:].long() - 1)
-        logits = F.gemm(h[last].contiguous(), self.params.lm_head_weight)
+        logits = self._logits(h[last].contiguous())
         if len(leaders) < len(reqs):
             logits = logits[torch.tensor(lead_idx, dtype=torch.int64, device=dev)]
             for i, r in enumerate(reqs):
@@ -627,7 +667,11 @@ class RolloutEngine:
                 if nb > nfull:  # the partially filled last page is private: copy it
                     src = torch.tensor(reqs[li].blocks[nfull:nb], dtype=torch.int64, device=dev)
                     dst = torch.tensor(r.blocks[nfull:nb], dtype=torch.int64, device=dev)
-                    self.kv[:, :, dst] = self.kv[:, :, src]
+                    self.cache.copy_blocks(dst, src)
+            if self.cache.has_state:
+                pairs = [(r.slot, reqs[leaders[lead_idx[i]]].slot) for i, r in enumerate(reqs) if leaders[lead_idx[i]] != i]
+                dst, src = (torch.tensor(c, dtype=torch.int64, device=dev) for c in zip(*pairs))
+                self.cache.copy_slots(dst, src)
             self.stats["prefill_tokens_shared"] = self.stats.get("prefill_tokens_shared", 0) + sum(lens) - sum(lens[i] for i in leaders)
         slots = torch.tensor([r.slot for r in reqs], dtype=torch.int64, device=dev)
         seeds = torch.tensor([(r.params.seed if r.params.seed is not None else self._seed * 1000003 + zlib.crc32(r.rid.encode()))
@@ -685,8 +729,8 @@ class RolloutEngine:
         return l.to(logits.dtype)
 
     # ------------------------------------------------------------------------------------ decode
-    def _decode_body(self) -> None:
-        """One decode step over all slots (static shapes; capturable)."""
+    def _decode_hidden(self) -> torch.Tensor:
+        """Every active slot's current token through the model (static shapes; capturable): final hidden states [S, H]."""
         cfg, P = self.cfg, self.params
         S = self.S
         act = self.active
@@ -695,6 +739,8 @@ class RolloutEngine:
         blk = torch.gather(self.block_table, 1, (pos_l // self.bs).unsqueeze(1)).squeeze(1).long()
         slot_map = torch.where(act, blk * self.bs + pos_l % self.bs, torch.full_like(pos_l, -1))
         ctx_eff = self.ctx * acti
+        if cfg.is_stack:
+            return self.model.decode_hidden(self.tok, self.pos, slot_map, ctx_eff, act, self.block_table, self.cache)
         tp = self.model.tp
         w_ = self.tp_size
         nh, nkv, hd, Q, KV = cfg.num_attention_heads // w_, cfg.num_key_value_heads // w_, cfg.head_dim, cfg.q_size // w_, cfg.kv_size // w_
@@ -736,7 +782,16 @@ class RolloutEngine:
             h2, x2, _ = F.rms_norm(o, W["post_attention_layernorm.weight"], cfg.rms_norm_eps, residual=x)
             a = self.model._mlp_fwd(W, h2, None)
             r = x2
-        hN = F.rms_norm(a, P["norm.weight"], cfg.rms_norm_eps, residual=r)[0]
+        return F.rms_norm(a, P["norm.weight"], cfg.rms_norm_eps, residual=r)[0]
+
+    def _decode_body(self) -> None:
+        """One decode step over all slots (static shapes; capturable)."""
+        cfg, P = self.cfg, self.params
+        S = self.S
+        act = self.active
+        acti = act.to(torch.int32)
+        tp = self.model.tp
+        hN = self._decode_hidden()
         if tp is not None and self._tp_share is not None and not self._use_penalty:
             sh = S // tp.size
             mine = slice(tp.rank * sh, (tp.rank + 1) * sh)
@@ -746,7 +801,7 @@ class RolloutEngine:
             tok = both[:, :sh].reshape(S).long()
             lp = both[:, sh:].reshape(S).view(torch.float32)
         else:
-            logits = F.gemm(hN, P.lm_head_weight)
+            logits = self._logits(hN)
             if self._use_penalty:
                 logits = self._penalise(logits)
             tok, lp = F.sample_tokens(logits, self.temperature, self.seeds, 0, self.valid_vocab, self.top_k, self.top_p)
@@ -790,6 +845,8 @@ class RolloutEngine:
                 snap = [t.clone() for t in (self.tok, self.pos, self.ctx, self.gen, self.active, self.seeds, self.out_tok, self.out_lp)]
                 side = torch.cuda.Stream(device=self.device)
                 side.wait_stream(torch.cuda.current_stream(self.device))
+                if self.cache.has_state:
+                    self.active.zero_()  # recurrent state is updated in place: the warm-up step must not touch it
                 with torch.cuda.stream(side):
                     self._decode_body()  # warm-up (allocator, lazy init) outside capture
                 torch.cuda.current_stream(self.device).wait_stream(side)
@@ -863,6 +920,70 @@ class RolloutEngine:
             self.free_slots.append(s)
         self.active[idx] = False
         self.ctx[idx] = 0
+
+    # ------------------------------------------------------------------------------------ given tokens (trace replay, scoring)
+    def open_sequence(self, key: str) -> None:
+        """Start a sequence whose tokens are given by ``feed`` instead of sampled; it takes a slot, and pages as it grows."""
+        assert key not in self.sequences, f"sequence {key!r} is open already"
+        assert self.free_slots, "no free sequence slot"
+        assert not self.running, "given-token sequences and sampled requests do not share the decode loop"
+        self.sequences[key] = _Sequence(self.free_slots.pop())
+
+    def close_sequence(self, key: str) -> None:
+        q = self.sequences.pop(key)
+        self._release_blocks(q.blocks)
+        self.free_slots.append(q.slot)
+
+    @torch.no_grad()
+    def feed(self, entries: Sequence[tuple[str, Sequence[int], Sequence[int]]]) -> list[torch.Tensor]:
+        """One step over open sequences: ``(key, next tokens, wanted places among them)`` per entry. Single tokens of running
+        sequences go through the decode step, everything else through the prompt path, each as one batch, exactly as in
+        generation. Returns per entry the fp32 logits [wanted, vocab]."""
+        out: list = [None] * len(entries)
+        V = self.cfg.vocab_size
+        prompts, singles = [], []
+        for j, (key, tokens, _) in enumerate(entries):
+            q = self.sequences[key]
+            assert len(tokens) > 0 and q.length + len(tokens) <= self.max_model_len, f"sequence {key!r} outgrows max_model_len"
+            need = -(-(q.length + len(tokens)) // self.bs) - len(q.blocks)
+            assert need <= len(self.free_blocks) + len(self._idle_cached), "the cache is full"
+            q.blocks += [self._take_block() for _ in range(need)]
+            (singles if len(tokens) == 1 and q.length > 0 else prompts).append(j)
+        table = lambda js: torch.stack([torch.nn.functional.pad(torch.tensor(self.sequences[entries[j][0]].blocks, dtype=torch.int32),
+                                                                (0, self.max_blocks_per_seq - len(self.sequences[entries[j][0]].blocks))) for j in js])
+        if prompts:
+            seqs = [self.sequences[entries[j][0]] for j in prompts]
+            n = [len(entries[j][1]) for j in prompts]
+            ids = torch.tensor([int(t) for j in prompts for t in entries[j][1]], dtype=torch.int64)
+            h, _ = self._run_portions(ids, [q.length for q in seqs], [q.length + c for q, c in zip(seqs, n)], table(prompts), [q.slot for q in seqs])
+            rows, row0 = [], 0
+            for j, c in zip(prompts, n):
+                rows += [row0 + int(w) for w in entries[j][2]]
+                row0 += c
+            logits = self._logits(h[torch.tensor(rows, dtype=torch.int64, device=self.device)].contiguous()).float() if rows else None
+            at = 0
+            for j in prompts:
+                k = len(entries[j][2])
+                out[j] = logits[at : at + k] if k else torch.empty(0, V)
+                at += k
+        if singles:
+            seqs = [self.sequences[entries[j][0]] for j in singles]
+            slots = torch.tensor([q.slot for q in seqs], dtype=torch.int64, device=self.device)
+            pos = torch.tensor([q.length for q in seqs], dtype=torch.int32, device=self.device)
+            self.block_table[slots] = table(singles).to(self.device)
+            self.tok[slots] = torch.tensor([int(entries[j][1][0]) for j in singles], dtype=torch.int64, device=self.device)
+            self.pos[slots] = pos
+            self.ctx[slots] = pos + 1
+            self.active.zero_()
+            self.active[slots] = True
+            logits = self._logits(self._decode_hidden())[slots].float()
+            self.active.zero_()
+            self.ctx[slots] = 0
+            for j, row in zip(singles, logits):
+                out[j] = row[None].expand(len(entries[j][2]), V)
+        for key, tokens, _ in entries:
+            self.sequences[key].length += len(tokens)
+        return out
 
     # ------------------------------------------------------------------------------------ driver loops
     def step(self) -> list[RequestOutput]:
