@@ -967,7 +967,7 @@ void gemm_grouped_wgrad_(const Tensor& dy, const Tensor& x, Tensor out, const Te
 
 }  // namespace
 
-extern "C" void vb_count_launches(long long n) { count(n); }
+extern "C" void verl_count_launches(long long n) { count(n); }
 
 TORCH_LIBRARY(verl_b200, m) {
   m.def("peer_barrier", &peer_barrier);

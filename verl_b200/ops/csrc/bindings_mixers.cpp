@@ -34,7 +34,7 @@ void run_gemm(const Tensor& a, const Tensor& w, const VbEpiArgs& e) {
   TORCH_CHECK(a.dim() == 2 && w.dim() == 2 && a.stride(1) == 1 && w.stride(1) == 1 && a.size(1) == w.size(1), "linear: a [M, K], w [N, K]");
   const int M = (int)a.size(0), K = (int)a.size(1), N = (int)w.size(0);
   if (M == 0 || N == 0) return;
-  vb_count_launches(1);
+  verl_count_launches(1);
   int rc = -1;
   if (dt == 1) {
     if (M <= 1024 && N % 8 == 0 && K % 8 == 0 && a.stride(0) % 8 == 0 && w.stride(0) % 8 == 0) {
@@ -103,7 +103,7 @@ std::tuple<Tensor, Tensor> embed_dyt(const Tensor& ids, const Tensor& w, double 
   same(w, nw, "embed_dyt");
   const int T = (int)ids.numel(), W = (int)w.size(1);
   Tensor x = at::empty({T, W}, w.options().dtype(at::kFloat)), h = at::empty({T, W}, w.options());
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_embed_dyt(dt, lptr(ids), w.data_ptr(), (float)scale, x.data_ptr<float>(), h.data_ptr(), alpha.data_ptr(), nw.data_ptr(),
                         nb.data_ptr(), T, W, (int)w.size(0), cur_stream()), "vb_embed_dyt");
   return {x, h};
@@ -115,7 +115,7 @@ Tensor dynamic_tanh(const Tensor& x, const Tensor& alpha, const Tensor& nw, cons
   const c10::cuda::CUDAGuard guard(x.device());
   TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && nw.numel() == x.size(1) && nb.numel() == x.size(1) && alpha.numel() == 1, "dynamic_tanh");
   Tensor h = at::empty(x.sizes(), nw.options());
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_dyt(dt, x.data_ptr<float>(), h.data_ptr(), alpha.data_ptr(), nw.data_ptr(), nb.data_ptr(), (int)x.size(0), (int)x.size(1), cur_stream()), "vb_dyt");
   return h;
 }
@@ -129,7 +129,7 @@ void rope_pairs_(Tensor x, const Tensor& pos, const Tensor& cs, const Tensor& sn
   TORCH_CHECK(x.dim() == 3 && x.stride(2) == 1 && off >= 0 && off + dims <= x.size(2) && dims % 2 == 0 && cs.size(1) == dims / 2 && cs.is_contiguous() &&
               sn.is_contiguous() && pos.numel() == x.size(0), "rope_pairs_");
   const c10::cuda::CUDAGuard guard(x.device());
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_rope_pairs(dt, x.data_ptr(), pos.data_ptr<int>(), cs.data_ptr<float>(), sn.data_ptr<float>(), (int)x.size(0), (int)x.size(1), x.stride(0),
                          (int)x.stride(1), (int)off, (int)dims, (int)cs.size(0), cur_stream()), "vb_rope_pairs");
 }
@@ -154,7 +154,7 @@ std::tuple<Tensor, Tensor> latent_prep(const Tensor& p, const Tensor& qn, const 
                 slot->scalar_type() == at::kLong && slot->is_contiguous() && slot->numel() == T, "latent_prep: pages [blocks, block_size, kv_rank + rot]");
     ps = pages->stride(0); bs = (int)pages->size(1); slots = pages->size(0) * pages->size(1);
   }
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_latent_prep(dt, p.data_ptr(), p.stride(0), qn.data_ptr(), kn.data_ptr(), (float)eps, pos.data_ptr<int>(), cs.data_ptr<float>(),
                           sn.data_ptr<float>(), (int)(2 * cs.size(1)), (int)cs.size(0), cq.data_ptr(), want_rows ? lat.data_ptr() : nullptr, kr + rot, ptr(pages), ps, bs,
                           slots, pages.has_value() ? lptr(*slot) : nullptr, (int)T, (int)qr, (int)kr, (int)rot, cur_stream()), "vb_latent_prep");
@@ -168,7 +168,7 @@ Tensor gather_pages(const Tensor& pages, const Tensor& block_table, const Tensor
   CHECK_I32(k_start);
   const c10::cuda::CUDAGuard guard(pages.device());
   Tensor out = at::empty({total, pages.size(2)}, pages.options());
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_gather_pages(dt, pages.data_ptr(), pages.stride(0), (int)pages.size(1), block_table.data_ptr<int>(), (int)block_table.size(1), cu_k.data_ptr<int>(),
                            k_start.data_ptr<int>(), (int)k_start.numel(), (int)pages.size(2), out.data_ptr(), (int)total, cur_stream()), "vb_gather_pages");
   return out;
@@ -190,7 +190,7 @@ Tensor headwise_linear(const Tensor& a, const Tensor& w, bool b_mn, const OptTen
     TORCH_CHECK(gate->size(0) == M && gate->size(1) >= H && gate->stride(1) == 1, "headwise_linear: gate [M, H]");
     e.gate = gate->data_ptr<float>(); e.ldg = gate->stride(0);
   }
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_gemm_simt(dt, a.data_ptr(), w.data_ptr(), (int)M, (int)N, (int)K, a.stride(0), w.stride(1), b_mn, (int)H, a.stride(1), w.stride(0), N, &e, cur_stream()),
            "headwise_linear");
   return d;
@@ -218,7 +218,7 @@ Tensor latent_attn_prefill(const Tensor& q, const Tensor& ku, const Tensor& kr, 
   if (gate.has_value()) { CHECK_F32(*gate); TORCH_CHECK(gate->size(0) == a.T && gate->stride(1) == 1); a.gate = gate->data_ptr<float>(); a.ldg = gate->stride(0); }
   Tensor out = at::empty({q.size(0), q.size(1), v.size(2)}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
   return out;
 }
@@ -246,7 +246,7 @@ Tensor latent_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& bl
   if (sink.has_value()) { same(q, *sink, "latent_attn_decode"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
   Tensor out = at::empty({q.size(0), q.size(1), kv_rank}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
   return out;
 }
@@ -275,7 +275,7 @@ Tensor mlstm_decode(const Tensor& p, const Tensor& gates, const Tensor& ib, cons
   TORCH_CHECK(active.is_cuda() && active.scalar_type() == at::kBool && active.is_contiguous() && active.numel() == s.T && state.size(0) >= s.T, "mlstm_decode: active [S]");
   const c10::cuda::CUDAGuard guard(p.device());
   Tensor out = at::empty({s.T, s.H * s.e}, p.options());
-  vb_count_launches(1);
+  verl_count_launches(1);
   CHECK_RC(vb_mlstm_decode(s.dt, p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap, state.data_ptr<float>(),
                            state.stride(0), reinterpret_cast<const uint8_t*>(active.data_ptr()), norm.data_ptr(), (float)eps, out.data_ptr(), out.stride(0), (int)s.T, (int)s.H,
                            (int)s.d, (int)s.e, cur_stream()), "vb_mlstm_decode");
@@ -298,7 +298,7 @@ Tensor mlstm_prefill(const Tensor& p, const Tensor& gates, const Tensor& ib, con
   const c10::cuda::CUDAGuard guard(p.device());
   Tensor o = at::empty({s.T, s.H * s.e}, p.options().dtype(at::kFloat));
   Tensor out = at::empty({s.T, s.H * s.e}, p.options());
-  vb_count_launches(slots.has_value() ? 3 : 2);
+  verl_count_launches(slots.has_value() ? 3 : 2);
   CHECK_RC(vb_mlstm_scan(s.dt, p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap,
                          slots.has_value() ? state->data_ptr<float>() : nullptr, slots.has_value() ? state->stride(0) : 0, iptr(slots), iptr(fresh), cu.data_ptr<int>(), (int)B,
                          o.data_ptr<float>(), (int)s.T, (int)s.H, (int)s.d, (int)s.e, cur_stream()), "vb_mlstm_scan");

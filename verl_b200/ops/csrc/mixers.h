@@ -49,7 +49,7 @@ struct VbLatentAttn {
 };
 
 extern "C" {
-void vb_count_launches(long long n);
+void verl_count_launches(long long n);
 // gemm_simt.cu
 int vb_gemm_simt(int dtype, const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, int b_mn, int batch,
                  long long sa, long long sb, long long sd, const VbEpiArgs* e, cudaStream_t s);
