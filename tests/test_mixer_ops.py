@@ -194,9 +194,9 @@ def test_decode_attention_over_pages(place, heads, rank, dr, bs, window):
     rows_of = lambda b, n: pages.cpu().float()[table[b].long()].reshape(per * bs, -1)[:n]
     for b, n in enumerate(ctx):
         if window and n > window:
-            q[b] = rows_of(b, n)[n - window - (b % 2)] * 3.0       # the key on the window's edge, inside or outside
+            q[b] = rows_of(b, n)[n - window - (b % 2)] * 2.0       # the key on the window's edge, inside or outside
         elif n > 1:
-            q[b] = rows_of(b, n)[0] * 3.0                          # the farthest key
+            q[b] = rows_of(b, n)[0] * 2.0                          # the farthest key
     got = X.latent_attention_decode(put(q, place), pages, table.to(place[0]), i32(ctx, place), rank, window, scale, put(sink, place))
     for b, n in enumerate(ctx):
         if n == 0:

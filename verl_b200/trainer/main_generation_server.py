@@ -67,11 +67,14 @@ def run_generation(config, tokenizer=None, engines: Optional[list] = None, promp
         path = os.path.expanduser(config.data.path)
         df = pd.read_json(path, lines=True) if path.endswith((".jsonl", ".json")) else pd.read_parquet(path)
         col = df[config.data.prompt_key].tolist()
-        if tokenizer is None:
+        as_ids = len(col) > 0 and all(not isinstance(c, str) and len(c) > 0 and isinstance(c[0], (int, np.integer)) for c in col)
+        if as_ids:      # prompts are token ids already: no tokenizer, the responses are written as token ids
+            prompts_ids = [[int(t) for t in c] for c in col]
+        elif tokenizer is None:
             from ..utils.tokenizer import hf_tokenizer
 
             tokenizer = hf_tokenizer(config.actor_rollout_ref.model.path)
-        prompts_ids = [tokenizer.apply_chat_template(list(c), add_generation_prompt=True, tokenize=True) if not isinstance(c, str)
+        prompts_ids = prompts_ids or [tokenizer.apply_chat_template(list(c), add_generation_prompt=True, tokenize=True) if not isinstance(c, str)
                        else tokenizer.encode(c) for c in col]
     sp = dict(temperature=float(rc.temperature), top_p=float(rc.top_p), top_k=int(rc.top_k), max_tokens=int(rc.response_length), logprobs=False)
 
@@ -81,7 +84,7 @@ def run_generation(config, tokenizer=None, engines: Optional[list] = None, promp
 
     outs = asyncio.run(go())
     if df is not None:
-        df["responses"] = [[tokenizer.decode(t, skip_special_tokens=True) for t in group] for group in outs]
+        df["responses"] = [[list(map(int, t)) if as_ids else tokenizer.decode(t, skip_special_tokens=True) for t in group] for group in outs]
         out_path = os.path.expanduser(config.data.output_path)
         os.makedirs(os.path.dirname(out_path) or ".", exist_ok=True)
         df.to_parquet(out_path)

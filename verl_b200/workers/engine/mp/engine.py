@@ -56,6 +56,8 @@ class ModelParallelEngine(NativeEngine):
         if g("context_parallel_size", 1) > 1 and self.pp_size > 1:
             raise NotImplementedError("context parallelism is combined with tensor and data parallelism; pipeline stages "
                                       "exchange whole token streams (use pipeline_model_parallel_size=1 with it)")
+        if self.arch.is_stack:
+            raise NotImplementedError(f"{self.arch.stack.design}: mixer stacks run in the data-parallel engine (strategy fsdp, forward only)")
         if self.arch.is_generic:
             raise NotImplementedError(f"model_type={self.arch.model_type!r} runs as a library module: tensor / pipeline / expert "
                                       f"parallel training covers the natively supported families; use the data-parallel engine "

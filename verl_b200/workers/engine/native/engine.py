@@ -33,7 +33,8 @@ import torch
 import torch.distributed as dist
 
 from ....models.config import ModelConfig
-from ....models.decoder import DecoderModel, PackedBatch
+from ....models import build_decoder
+from ....models.decoder import PackedBatch
 from ....models.weights import ALIGN, FlatParams
 from ....ops import functional as F
 from ....ops import native
@@ -248,6 +249,8 @@ class NativeEngine(BaseEngine):
             self.dtype = torch.float32
         ec = self.engine_config
         seed = int(getattr(ec, "seed", 42))
+        if self.arch.is_stack and not self.forward_only:
+            raise NotImplementedError(f"{self.arch.stack.design}: mixer stacks are served and scored (forward_only engines), not trained")
         self.fused_comm = False
         self.peer_barrier_timeout_s = float(getattr(ec, "peer_barrier_timeout_s", 120.0) or 120.0)
         self._sym_params = self._sym_grads = self._peer_barrier = None
@@ -295,7 +298,7 @@ class NativeEngine(BaseEngine):
                 "LoRA and sequence parallelism need one of the natively supported model families"
             self.model = GenericCausalLM(self.arch, self.params, recompute=recompute)
         else:
-            self.model = DecoderModel(self.arch, self.params, recompute=recompute)
+            self.model = build_decoder(self.arch, self.params, recompute=recompute)
         self.model.keep_layers_fn = self._layers_that_fit
         tm = getattr(self.model_config, "tiled_mlp", None) or {}
         if (tm.get("enabled") if hasattr(tm, "get") else getattr(tm, "enabled", False)):
@@ -372,7 +375,7 @@ class NativeEngine(BaseEngine):
         self._blk_size, self._blk_rank = self.sp_size, self.sp_rank
         # shared-prompt packing of GRPO groups (same results, fewer tokens through every projection and MLP)
         self._share_prefix = (bool(getattr(ec, "use_prefix_grouper", True)) and os.environ.get("VERL_B200_SHARE_PREFIX", "1") != "0"
-                              and self.sp_size == 1 and not self.arch.is_generic)
+                              and self.sp_size == 1 and not self.arch.is_generic and not self.arch.is_stack)
         if bool(getattr(ec, "enable_activation_offload", False)) and not self.forward_only:
             from ....utils.activation_offload import ActivationOffloader
 

@@ -371,7 +371,7 @@ class ActorRolloutRefWorker(Worker, DistProfilerExtension):
             pool_ranks = dist.get_process_group_ranks(pool if pool is not None else dist.group.WORLD) if ws > 1 else [0]
             n_pool, me = len(pool_ranks), (pool_ranks.index(dist.get_rank()) if ws > 1 else 0)
             tp = int(rc.tensor_model_parallel_size or 1)
-            tp = tp if (n_pool > 1 and tp > 1 and n_pool % tp == 0 and not arch.is_moe and not arch.is_generic
+            tp = tp if (n_pool > 1 and tp > 1 and n_pool % tp == 0 and not arch.is_moe and not arch.is_generic and not arch.is_stack
                         and arch.num_key_value_heads % tp == 0) else 1
             self.rollout_tp, self.rollout_tp_group = tp, None
             if tp > 1:  # only the members take part in creating their group

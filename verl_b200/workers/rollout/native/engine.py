@@ -125,7 +125,7 @@ class RolloutEngine:
         self.tp_group = tp_group
         self.tp_size = dist.get_world_size(tp_group) if tp_group is not None else 1
         self.tp_rank = dist.get_rank(tp_group) if tp_group is not None else 0
-        assert cfg.num_key_value_heads % self.tp_size == 0 and (cfg.is_moe or cfg.intermediate_size % (8 * self.tp_size) == 0), \
+        assert cfg.num_key_value_heads % self.tp_size == 0 and (cfg.is_moe or cfg.is_stack or cfg.intermediate_size % (8 * self.tp_size) == 0), \
             "tensor-parallel size must divide the KV heads and the MLP width"
         assert not cfg.is_stack or (self.tp_size == 1 and self.quantization is None), \
             f"{cfg.model_type}: served on one GPU per replica, without quantised weights"
