@@ -287,3 +287,14 @@ def test_mlstm_starts_from_zero_maximum(place):
     want = mlstm_want(p, g, ib, fb, norm, 10.0, 1e-2, H, d, e)
     got = X.mlstm_prefill(put(p, place), g.to(place[0]), put(ib, place), put(fb, place), 10.0, put(norm, place), 1e-2, d, i32([0, T], place))
     close(got, want, place)
+
+
+@pytest.mark.parametrize("m,h,dim,rank,rot_dim", [(3, 2, 24, 40, 8), (33, 5, 10, 14, 6), (70, 3, 128, 512, 64), (20, 17, 64, 136, 32)])
+def test_absorbed_query(place, m, h, dim, rank, rot_dim):
+    rot = dict(dims=rot_dim - 2, base=700.0)
+    spec = _rotary(rot)
+    cos, sin = F.rope_table(64, spec.dims, spec.base, place[0], spec.scaling)
+    q, uk, pos = rand(m, h, dim + rot_dim), rand(h, dim, rank, scale=dim ** -0.5), torch.randint(0, 64, (m,), generator=GEN)
+    got = X.latent_absorb(put(q, place), put(uk, place), pos.to(place[0], torch.int32), cos, sin)
+    close(got[..., :rank], torch.einsum("mhd,hdr->mhr", q[..., :dim].double(), uk.double()), place, rel16=4e-3)
+    close(got[..., rank:], plain.rotate_pairs(q[..., dim:].double(), pos, rot), place, rel16=4e-3)

@@ -114,8 +114,7 @@ class MixerStackModel:
     def _attention_decode(self, i, W, m, h, pos, slot_map, ctx_len, block_table, cache):
         S = h.shape[0]
         q, _, gate, cos, sin = self._attention_in(W, m, h, pos, cache.pages(i), slot_map, False)
-        X.rope_pairs_(q, pos, cos, sin, m.dim)
-        qa = torch.cat([X.headwise_linear(q[..., : m.dim], W["uk"], True), q[..., m.dim :]], -1)
+        qa = X.latent_absorb(q, W["uk"], pos, cos, sin)
         oc = X.latent_attention_decode(qa, cache.pages(i), block_table, ctx_len, m.kv_rank, m.window, m.scale, W["sink"])
         return X.headwise_linear(oc, W["uv"], False, gate).view(S, m.heads * m.vdim)
 
@@ -197,8 +196,8 @@ class MixerStackModel:
             if positions is not None:
                 h = h.index_select(0, positions)
                 labels = position_labels if position_labels is not None else labels.index_select(0, positions)
-            if h.is_cuda and h.dtype != torch.bfloat16:
-                logp = torch.log_softmax(self.logits(h) / max(temperature, 1e-8), -1)
+            if h.is_cuda and (h.dtype != torch.bfloat16 or h.shape[1] % 8 or self.cfg.vocab_size % 8):   # outside the fused head's sizes
+                logp = torch.log_softmax(X.linear_act(h, self.params.lm_head_weight, out_f32=True) / max(temperature, 1e-8), -1)
                 return logp.gather(-1, labels.unsqueeze(-1)).squeeze(-1), -(logp.exp() * logp).sum(-1)
             lp, ent, _ = F.lmhead_logprob_entropy(h, self.params.lm_head_weight, labels, temperature)
             return lp, ent

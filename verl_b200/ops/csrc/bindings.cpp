@@ -5,6 +5,7 @@
 #include <torch/library.h>
 
 #include "launchers.h"
+#include "mixers.h"
 
 #include <algorithm>
 #include <atomic>
@@ -154,6 +155,7 @@ int64_t gemm_status() {
   int b = vb_attn_status();
   if (b == 0) b = vb_attn_bwd_status();
   if (b == 0) b = vb_fp8_status();
+  if (b == 0) b = vb_latent_decode_status();
   const int c = vb_pd_status();
   return a != 0 ? a : (b != 0 ? 100 + b : (c != 0 ? 200 + c : 0));
 }

@@ -174,26 +174,59 @@ Tensor gather_pages(const Tensor& pages, const Tensor& block_table, const Tensor
   return out;
 }
 
-// out[m, h, :] = a[m, h, :] w[h] (b_mn: w [H, K, N]) or a[m, h, :] w[h]^T (w [H, N, K]), times sigmoid(gate[m, h]).
-Tensor headwise_linear(const Tensor& a, const Tensor& w, bool b_mn, const OptTensor& gate) {
+// out[m, h, :] = a[m, h, :] w[h] (b_mn: w [H, K, N]) or a[m, h, :] w[h]^T (w [H, N, K]), times sigmoid(gate[m, h]), into out with
+// the given strides; tensor cores where the sizes allow.
+void run_headwise(const Tensor& a, const Tensor& w, bool b_mn, const OptTensor& gate, VbHeadwise p) {
   const int dt = dtype_of(a);
   same(a, w, "headwise_linear");
-  TORCH_CHECK(a.dim() == 3 && w.dim() == 3 && a.size(1) == w.size(0) && a.stride(2) == 1 && w.stride(2) == 1 && a.size(2) == (b_mn ? w.size(1) : w.size(2)), "headwise_linear");
-  const c10::cuda::CUDAGuard guard(a.device());
-  const int64_t M = a.size(0), H = a.size(1), K = a.size(2), N = b_mn ? w.size(2) : w.size(1);
-  Tensor d = at::empty({M, H, N}, a.options());
-  VbEpiArgs e{};
-  e.mode = VB_EPI_STORE;
-  e.D = d.data_ptr(); e.ldd = H * N;
+  TORCH_CHECK(a.dim() == 3 && w.dim() == 3 && a.size(1) == w.size(0) && a.stride(2) == 1 && w.stride(2) == 1, "headwise_linear");
+  p.a = a.data_ptr(); p.lda = a.stride(0); p.a_head = a.stride(1);
+  p.w = w.data_ptr(); p.w_head = w.stride(0); p.ldw = w.stride(1); p.kn = b_mn;
+  p.M = (int)a.size(0); p.H = (int)a.size(1); p.K = (int)(b_mn ? w.size(1) : w.size(2)); p.N = (int)(b_mn ? w.size(2) : w.size(1));
   if (gate.has_value()) {
     CHECK_F32(*gate);
-    TORCH_CHECK(gate->size(0) == M && gate->size(1) >= H && gate->stride(1) == 1, "headwise_linear: gate [M, H]");
-    e.gate = gate->data_ptr<float>(); e.ldg = gate->stride(0);
+    TORCH_CHECK(gate->size(0) == p.M && gate->size(1) >= p.H && gate->stride(1) == 1, "headwise_linear: gate [M, H]");
+    p.gate = gate->data_ptr<float>(); p.ldg = gate->stride(0);
   }
   verl_count_launches(1);
-  CHECK_RC(vb_gemm_simt(dt, a.data_ptr(), w.data_ptr(), (int)M, (int)N, (int)K, a.stride(0), w.stride(1), b_mn, (int)H, a.stride(1), w.stride(0), N, &e, cur_stream()),
-           "headwise_linear");
+  int rc = dt == 1 ? vb_headwise(&p, cur_stream()) : -1;
+  if (rc < 0) {
+    VbEpiArgs e{};
+    e.mode = VB_EPI_STORE;
+    e.D = p.out; e.ldd = p.ldo; e.gate = p.gate; e.ldg = p.ldg;
+    rc = vb_gemm_simt(dt, p.a, p.w, p.M, p.N, p.K, p.lda, p.ldw, b_mn, p.H, p.a_head, p.w_head, p.o_head, &e, cur_stream());
+    if (rc == 0 && p.rot > 0) {
+      verl_count_launches(1);
+      rc = vb_rope_copy(dt, p.a, p.lda, (int)p.a_head, p.K, p.out, p.ldo, (int)p.o_head, p.N, p.pos, p.cos_t, p.sin_t, p.M, p.H, p.rot, p.half, p.max_pos, cur_stream());
+    }
+  }
+  CHECK_RC(rc, "headwise_linear");
+}
+
+Tensor headwise_linear(const Tensor& a, const Tensor& w, bool b_mn, const OptTensor& gate) {
+  TORCH_CHECK(a.dim() == 3 && w.dim() == 3 && a.size(2) == (b_mn ? w.size(1) : w.size(2)), "headwise_linear: sizes");
+  const c10::cuda::CUDAGuard guard(a.device());
+  const int64_t N = b_mn ? w.size(2) : w.size(1);
+  Tensor d = at::empty({a.size(0), a.size(1), N}, a.options());
+  VbHeadwise p{};
+  p.out = d.data_ptr(); p.ldo = d.stride(0); p.o_head = N;
+  run_headwise(a, w, b_mn, gate, p);
   return d;
+}
+
+// q [S, H, dim + rot], uk [H, dim, rank]: [q_unrotated uk | rotated part] as [S, H, rank + rot].
+Tensor latent_absorb(const Tensor& q, const Tensor& uk, const Tensor& pos, const Tensor& cs, const Tensor& sn) {
+  CHECK_I32(pos);
+  CHECK_F32(cs);
+  const int64_t rot = q.size(2) - uk.size(1), rank = uk.size(2);
+  TORCH_CHECK(q.dim() == 3 && rot >= 0 && 2 * cs.size(1) <= rot && cs.is_contiguous() && sn.is_contiguous() && pos.numel() == q.size(0), "latent_absorb: sizes");
+  const c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({q.size(0), q.size(1), rank + rot}, q.options());
+  VbHeadwise p{};
+  p.out = out.data_ptr(); p.ldo = out.stride(0); p.o_head = rank + rot;
+  p.rot = (int)rot; p.half = (int)cs.size(1); p.max_pos = (int)cs.size(0); p.pos = pos.data_ptr<int>(); p.cos_t = cs.data_ptr<float>(); p.sin_t = sn.data_ptr<float>();
+  run_headwise(q, uk, true, OptTensor(), p);
+  return out;
 }
 
 // Prompt attention: q [T, H, du + dr], ku [Tk, H, du], kr [Tk, dr], v [Tk, H, dv] (strided views), cu_q / cu_k int32 [B + 1].
@@ -246,6 +279,23 @@ Tensor latent_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& bl
   if (sink.has_value()) { same(q, *sink, "latent_attn_decode"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
   Tensor out = at::empty({q.size(0), q.size(1), kv_rank}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
+  if (dt == 1) {
+    const int64_t all = (int64_t)a.max_blocks * a.block_size;
+    const int ns = vb_latent_decode_splits(a.B, a.H, a.dv, a.du + a.dr, a.block_size, (int)(window > 0 ? std::min<int64_t>(window + 32, all) : all));
+    if (ns > 0) {
+      Tensor po, ml;
+      if (ns > 1) {
+        po = at::empty({a.B, a.H, ns, kv_rank}, q.options().dtype(at::kFloat));
+        ml = at::empty({a.B, a.H, ns, 2}, q.options().dtype(at::kFloat));
+      }
+      const int rc = vb_latent_decode(&a, pages.size(0), ns, ns > 1 ? po.data_ptr<float>() : nullptr, ns > 1 ? ml.data_ptr<float>() : nullptr, cur_stream());
+      if (rc >= 0) {
+        verl_count_launches(ns > 1 ? 2 : 1);
+        CHECK_RC(rc, "vb_latent_decode");
+        return out;
+      }
+    }
+  }
   verl_count_launches(1);
   CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
   return out;
@@ -320,6 +370,7 @@ TORCH_LIBRARY_FRAGMENT(verl_b200, m) {
   m.def("latent_prep", &latent_prep);
   m.def("gather_pages", &gather_pages);
   m.def("headwise_linear", &headwise_linear);
+  m.def("latent_absorb", &latent_absorb);
   m.def("latent_attn_prefill", &latent_attn_prefill);
   m.def("latent_attn_decode", &latent_attn_decode);
   m.def("mlstm_decode", &mlstm_decode);

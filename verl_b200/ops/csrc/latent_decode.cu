@@ -1,0 +1,307 @@
+// Decode-step attention in the latent space: one CTA = (sequence, group of 16 heads [, key split]).
+//
+// All heads read the same cached row, [latent (value and first key part) | rotated key part], so a row is streamed once per
+// head group: TMA brings 32-token tiles of the pages (128B swizzle, 64 columns per panel) into a shared-memory ring, and the
+// 16 heads are the M dimension of m16n8k16 MMAs (a 16-row sliver of work per byte: the kernel is bound by the stream, not by
+// the tensor pipe, as in paged_decode_tma.cu). Per tile
+//   scores   warp w takes tokens [8w, 8w + 8) over the whole row width, masked to the window
+//   softmax  running maximum shared by the four warps; it starts at the sink, which adds one unit of weight and no value
+//   values   warp w takes kv_rank / 4 latent columns over all 32 tokens
+// Tiles outside the window are never loaded. Compiled without fast math.
+#include "mixers.h"
+#include "mixer_common.cuh"
+#include "tcgen05_common.cuh"
+
+#include <math.h>
+
+namespace vb {
+
+constexpr int LD_TOK = 32, LD_THREADS = 128, LD_HEADS = 16, LD_MAX_STAGES = 4;
+
+struct LatentDecodeParams {
+  const __nv_bfloat16* q;   // [S, H, width]
+  long long ldq;
+  int hq;
+  const int* block_table;
+  int max_blocks, block_size, box_rows;
+  long long num_blocks;
+  const int* ctx_len;
+  const __nv_bfloat16* sink;
+  __nv_bfloat16* out;       // [S, H, rank]
+  float* part_o;            // [S, H, nsplit, rank] when nsplit > 1
+  float* part_ml;           // [S, H, nsplit, 2]
+  int H, width, rank, panels, window, nsplit, stages;
+  float scale_log2;
+  int* status;
+};
+
+__device__ int g_latent_decode_status[1];
+
+__device__ __forceinline__ void ld_ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ld_ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ld_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// NV: 8-column value blocks per warp (rank <= 32 NV)
+template <int NV>
+__global__ void __launch_bounds__(LD_THREADS, 2)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeParams p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int stage_bytes = p.panels * (LD_TOK * 128);
+  const int qpitch = p.panels * 128 + 16;                   // bytes of one query row (shifted banks per head)
+  uint8_t* sQ = smem + p.stages * stage_bytes;
+  uint8_t* sP = sQ + LD_HEADS * qpitch;                      // [16][40] bf16
+  float* sMax = reinterpret_cast<float*>(sP + LD_HEADS * 80);  // [4][16]
+  float* sSum = sMax + 64;                                   // [4][16]
+  uint64_t* full = reinterpret_cast<uint64_t*>(sSum + 64);   // [stages]
+
+  const int b = blockIdx.x, h0 = blockIdx.y * LD_HEADS, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int len = min(p.ctx_len[b], p.max_blocks * p.block_size);
+  const int nheads = min(LD_HEADS, p.H - h0);
+  const int first = (p.window > 0 && len > p.window) ? len - p.window : 0;
+  const int tile_a = first / LD_TOK, tile_b = (len + LD_TOK - 1) / LD_TOK;
+  const int per = (max(0, tile_b - tile_a) + p.nsplit - 1) / p.nsplit;
+  const int t0 = tile_a + split * per, n = max(0, min(tile_b, t0 + per) - t0);
+  const int* bt = p.block_table + static_cast<long long>(b) * p.max_blocks;
+
+  if (threadIdx.x == 0) {
+    tma_prefetch_desc(&tm);
+    for (int s = 0; s < p.stages; ++s) mbar_init(&full[s], 1);
+    mbar_fence_init();
+  }
+  for (int i = threadIdx.x; i < LD_HEADS * p.panels * 8; i += LD_THREADS) {
+    const int g = i / (p.panels * 8), c = i % (p.panels * 8);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (g < nheads && c * 8 < p.width) v = *reinterpret_cast<const uint4*>(p.q + b * p.ldq + static_cast<long long>(h0 + g) * p.hq + c * 8);
+    *reinterpret_cast<uint4*>(sQ + g * qpitch + c * 16) = v;
+  }
+  __syncthreads();
+
+  auto issue = [&](int i) {  // tile i of this CTA into stage i % stages (thread 0)
+    const int s = i % p.stages, tok = (t0 + i) * LD_TOK;
+    uint8_t* dst = smem + s * stage_bytes;
+    mbar_expect_tx(&full[s], static_cast<uint32_t>(stage_bytes));
+    for (int r = 0; r < LD_TOK; r += p.box_rows) {
+      // rows past the context re-read its last page: they are masked below
+      const int at = min(tok + r, (len - 1) / p.box_rows * p.box_rows);
+      const int blk = max(0, min(bt[at / p.block_size], static_cast<int>(p.num_blocks) - 1));
+      for (int c = 0; c < p.panels; ++c) tma_load_3d(dst + c * (LD_TOK * 128) + r * 128, &tm, &full[s], c * 64, at % p.block_size, blk);
+    }
+  };
+  if (threadIdx.x == 0)
+    for (int i = 0; i < min(n, p.stages - 1); ++i) issue(i);
+
+  float m_run[2], l_run[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int hd = (lane >> 2) + 8 * h;
+    const bool sk = p.sink != nullptr && split == 0 && hd < nheads;
+    m_run[h] = sk ? to_f(p.sink[h0 + hd]) * 1.4426950408889634f : -INFINITY;
+    l_run[h] = (sk && warp == 0 && (lane & 3) == 0) ? 1.f : 0.f;   // per-thread share of the denominator
+  }
+  float o[NV][4];
+#pragma unroll
+  for (int j = 0; j < NV; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+
+  const int mi = lane >> 3, r8 = lane & 7;
+  bool ok = true;
+  for (int i = 0; i < n; ++i) {
+    const int s = i % p.stages;
+    if (i > 0) __syncthreads();            // every warp is done with the tile before: its stage is free
+    if (threadIdx.x == 0 && i + p.stages - 1 < n) issue(i + p.stages - 1);
+    // a wait that runs out is recorded; the loop goes on so that every thread meets the same barriers
+    if (ok && !mbar_wait(&full[s], (i / p.stages) & 1)) ok = false;
+    const uint32_t kb = smem_u32(smem + s * stage_bytes);
+    // ---- scores of tokens [8 warp, 8 warp + 8)
+    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    {
+      const int tok = warp * 8 + r8;
+      const uint32_t qa = smem_u32(sQ) + ((mi & 1) * 8 + r8) * qpitch + (mi >> 1) * 16;
+#pragma unroll 4
+      for (int k2 = 0; k2 < p.panels * 2; ++k2) {
+        const int dc = k2 * 4 + mi;
+        uint32_t bf[4], a0[4], a1[4];
+        ld_ldsm_x4(bf, kb + (dc >> 3) * (LD_TOK * 128) + tok * 128 + (((dc & 7) ^ (tok & 7)) << 4));
+        ld_ldsm_x4(a0, qa + k2 * 64);
+        ld_ldsm_x4(a1, qa + k2 * 64 + 32);
+        ld_mma(s0, a0, bf[0], bf[1]);
+        ld_mma(s1, a1, bf[2], bf[3]);
+      }
+    }
+    const int tok0 = (t0 + i) * LD_TOK + warp * 8 + (lane & 3) * 2;
+    float v[2][2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = tok0 + e;
+        v[h][e] = (t >= first && t < len) ? (s0[h * 2 + e] + s1[h * 2 + e]) * p.scale_log2 : -INFINITY;
+      }
+      float mx = fmaxf(v[h][0], v[h][1]);
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      if ((lane & 3) == 0) sMax[warp * 16 + (lane >> 2) + 8 * h] = mx;
+    }
+    __syncthreads();
+    float alpha[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int hd = (lane >> 2) + 8 * h;
+      const float mn = fmaxf(fmaxf(fmaxf(sMax[hd], sMax[16 + hd]), fmaxf(sMax[32 + hd], sMax[48 + hd])), m_run[h]);
+      const float mu = mn == -INFINITY ? 0.f : mn;
+      alpha[h] = mn == -INFINITY ? 1.f : exp2f(m_run[h] - mn);
+      const float e0 = exp2f(v[h][0] - mu), e1 = exp2f(v[h][1] - mu);
+      l_run[h] = l_run[h] * alpha[h] + e0 + e1;
+      m_run[h] = mn;
+      *reinterpret_cast<uint32_t*>(sP + hd * 80 + (warp * 8 + (lane & 3) * 2) * 2) = pack_bf16x2(e0, e1);
+    }
+    __syncthreads();
+    // ---- values: this warp's columns over the 32 tokens
+    uint32_t pa[2][4];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) ld_ldsm_x4(pa[k], smem_u32(sP) + ((mi & 1) * 8 + r8) * 80 + k * 32 + (mi >> 1) * 16);
+    const bool resc = alpha[0] != 1.f || alpha[1] != 1.f;
+#pragma unroll
+    for (int j2 = 0; j2 < NV / 2; ++j2) {
+      const int dc = (warp * NV / 2 + j2) * 2 + (mi >> 1);
+      if (resc) {
+#pragma unroll
+        for (int q2 = 0; q2 < 2; ++q2) {
+          float* oo = o[2 * j2 + q2];
+          oo[0] *= alpha[0]; oo[1] *= alpha[0]; oo[2] *= alpha[1]; oo[3] *= alpha[1];
+        }
+      }
+      if ((warp * NV / 2 + j2) * 16 >= p.rank) continue;   // uniform over the warp
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int tok = k * 16 + (mi & 1) * 8 + r8;
+        uint32_t vb[4];
+        ld_ldsm_x4_t(vb, kb + (dc >> 3) * (LD_TOK * 128) + tok * 128 + (((dc & 7) ^ (tok & 7)) << 4));
+        ld_mma(o[2 * j2], pa[k], vb[0], vb[1]);
+        ld_mma(o[2 * j2 + 1], pa[k], vb[2], vb[3]);
+      }
+    }
+  }
+  if (!ok) atomicExch(p.status, 1);
+
+  // ---- denominators: every thread holds its own tokens' share
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    float l = l_run[h];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    if ((lane & 3) == 0) sSum[warp * 16 + (lane >> 2) + 8 * h] = l;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int hd = (lane >> 2) + 8 * h;
+    if (hd >= nheads) continue;
+    const float l = sSum[hd] + sSum[16 + hd] + sSum[32 + hd] + sSum[48 + hd];
+    const long long row = static_cast<long long>(b) * p.H + h0 + hd;
+    const float f = p.nsplit > 1 ? 1.f : (l > 0.f && len > 0 ? 1.f / l : 0.f);
+    float* po = p.nsplit > 1 ? p.part_o + (row * p.nsplit + split) * p.rank : nullptr;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int col = (warp * NV + j) * 8 + (lane & 3) * 2;
+      if (col >= p.rank) continue;
+      if (p.nsplit > 1) *reinterpret_cast<float2*>(po + col) = make_float2(o[j][2 * h], o[j][2 * h + 1]);
+      else *reinterpret_cast<uint32_t*>(p.out + row * p.rank + col) = pack_bf16x2(o[j][2 * h] * f, o[j][2 * h + 1] * f);
+    }
+    if (p.nsplit > 1 && warp == 0 && (lane & 3) == 0) {
+      p.part_ml[(row * p.nsplit + split) * 2] = m_run[h];
+      p.part_ml[(row * p.nsplit + split) * 2 + 1] = l;
+    }
+  }
+}
+
+// Joins the key splits of one (sequence, head).
+__global__ void latent_decode_merge_kernel(const float* __restrict__ po, const float* __restrict__ ml, const int* __restrict__ ctx_len,
+                                           __nv_bfloat16* __restrict__ out, int H, int nsplit, int rank) {
+  const long long row = blockIdx.x;
+  const float* m = ml + row * nsplit * 2;
+  float M = -INFINITY, L = 0.f;
+  for (int s = 0; s < nsplit; ++s) M = fmaxf(M, m[2 * s]);
+  for (int s = 0; s < nsplit; ++s) L += m[2 * s] == -INFINITY ? 0.f : exp2f(m[2 * s] - M) * m[2 * s + 1];
+  const float inv = (L > 0.f && ctx_len[row / H] > 0) ? 1.f / L : 0.f;
+  for (int c = threadIdx.x; c < rank; c += blockDim.x) {
+    float a = 0.f;
+    for (int s = 0; s < nsplit; ++s) a += m[2 * s] == -INFINITY ? 0.f : exp2f(m[2 * s] - M) * po[(row * nsplit + s) * rank + c];
+    out[row * rank + c] = __float2bfloat16(a * inv);
+  }
+}
+
+static int latent_decode_stages(int panels) {
+  const int fixed = LD_HEADS * (panels * 128 + 16) + LD_HEADS * 80 + 128 * 4 + 64 + 1024;
+  int s = (113 * 1024 - fixed) / (panels * LD_TOK * 128);     // two CTAs per SM
+  return s < 2 ? 0 : (s > LD_MAX_STAGES ? LD_MAX_STAGES : s);
+}
+static int latent_decode_smem(int panels, int stages) {
+  return stages * panels * LD_TOK * 128 + LD_HEADS * (panels * 128 + 16) + LD_HEADS * 80 + 128 * 4 + 64 + 1024;
+}
+
+}  // namespace vb
+
+using namespace vb;
+
+// Key splits for S sequences and H heads (0: the sizes are not served). max_keys: most keys a sequence can see.
+extern "C" int vb_latent_decode_splits(int S, int H, int rank, int width, int block_size, int max_keys) {
+  const int panels = (width + 63) / 64;
+  if (rank > 512 || rank % 8 || width % 8 || rank > width || block_size % 16 || latent_decode_stages(panels) == 0) return 0;
+  const int groups = S * ((H + LD_HEADS - 1) / LD_HEADS), tiles = (max_keys + LD_TOK - 1) / LD_TOK;
+  int s = (2 * num_sms() + groups - 1) / groups;
+  if (s > tiles / 4) s = tiles / 4;
+  return s < 1 ? 1 : (s > 16 ? 16 : s);
+}
+
+extern "C" int vb_latent_decode(const VbLatentAttn* a, long long num_blocks, int nsplit, float* part_o, float* part_ml, cudaStream_t stream) {
+  const int width = a->du + a->dr, panels = (width + 63) / 64;
+  if (a->hq % 8 || a->ldq % 8 || a->page_stride % 8) return -1;
+  if ((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->ku) | reinterpret_cast<uintptr_t>(a->out)) & 15) return -1;
+  LatentDecodeParams p{};
+  p.box_rows = a->block_size % LD_TOK == 0 ? LD_TOK : 16;
+  CUtensorMap tm;
+  if (!make_tmap_3d(&tm, a->ku, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, width, a->block_size, num_blocks, a->ku_row, a->page_stride, 64, p.box_rows, 1,
+                    CU_TENSOR_MAP_SWIZZLE_128B))
+    return -1;
+  static int* status = nullptr;
+  if (status == nullptr) cudaGetSymbolAddress(reinterpret_cast<void**>(&status), g_latent_decode_status);
+  p.q = reinterpret_cast<const __nv_bfloat16*>(a->q); p.ldq = a->ldq; p.hq = a->hq;
+  p.block_table = a->block_table; p.max_blocks = a->max_blocks; p.block_size = a->block_size; p.num_blocks = num_blocks;
+  p.ctx_len = a->ctx_len; p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink);
+  p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.part_o = part_o; p.part_ml = part_ml;
+  p.H = a->H; p.width = width; p.rank = a->dv; p.panels = panels; p.window = a->window; p.nsplit = nsplit;
+  p.stages = latent_decode_stages(panels); p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;
+  const int smem = latent_decode_smem(panels, p.stages);
+  const dim3 grid(a->B, (a->H + LD_HEADS - 1) / LD_HEADS, nsplit);
+  auto go = [&](auto kern) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 113 * 1024);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    kern<<<grid, LD_THREADS, smem, stream>>>(tm, p);
+    return static_cast<int>(cudaGetLastError());
+  };
+  int rc = a->dv <= 128 ? go(latent_decode_kernel<4>) : a->dv <= 256 ? go(latent_decode_kernel<8>) : go(latent_decode_kernel<16>);
+  if (rc == 0 && nsplit > 1) {
+    latent_decode_merge_kernel<<<a->B * a->H, 128, 0, stream>>>(part_o, part_ml, a->ctx_len, p.out, a->H, nsplit, p.rank);
+    rc = static_cast<int>(cudaGetLastError());
+  }
+  return rc;
+}
+
+extern "C" int vb_latent_decode_status() {
+  int h = 0;
+  if (cudaMemcpyFromSymbol(&h, g_latent_decode_status, sizeof(int)) != cudaSuccess) return -1;
+  if (h != 0) {
+    const int z = 0;
+    cudaMemcpyToSymbol(g_latent_decode_status, &z, sizeof(int));
+  }
+  return h;
+}

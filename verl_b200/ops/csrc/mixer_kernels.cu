@@ -70,6 +70,26 @@ __global__ void rope_pairs_kernel(T* __restrict__ x, const int* __restrict__ pos
   e[1] = from_f<T>(v * c + u * s);
 }
 
+// Out of place, between rows of different layout; dimensions behind the rotated ones are copied.
+template <typename T>
+__global__ void rope_copy_kernel(const T* __restrict__ a, long long lda, int a_head, int a_off, T* __restrict__ out, long long ldo, int o_head, int o_off,
+                                 const int* __restrict__ pos, const float* __restrict__ cs, const float* __restrict__ sn, int heads, int rot, int half,
+                                 int max_pos, long long total) {
+  const long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x;
+  if (i >= total) return;
+  const int c = static_cast<int>(i % rot);
+  const long long th = i / rot, t = th / heads;
+  const int hd = static_cast<int>(th % heads);
+  const T* src = a + t * lda + static_cast<long long>(hd) * a_head + a_off;
+  float o = to_f(src[c]);
+  if (c < 2 * half) {
+    const long long at = static_cast<long long>(min(max(pos[t], 0), max_pos - 1)) * half + (c >> 1);
+    const float w = to_f(src[c ^ 1]);
+    o = (c & 1) ? o * cs[at] + w * sn[at] : o * cs[at] - w * sn[at];
+  }
+  out[t * ldo + static_cast<long long>(hd) * o_head + o_off + c] = from_f<T>(o);
+}
+
 // --------------------------------------------------------------------------------------------- latent preparation
 // Row p[t] = [query latent (q_rank) | key/value latent (kv_rank) | shared key part (rot)]: RMS norms of the two latents,
 // rotation of the key part; the latent row (kv_rank + rot) goes to `lat` and / or to its place in the paged cache.
@@ -434,6 +454,18 @@ extern "C" int vb_rope_pairs(int dtype, void* x, const int* pos, const float* co
   const int grid = static_cast<int>((total + 255) / 256);
   if (dtype == 0) rope_pairs_kernel<float><<<grid, 256, 0, s>>>((float*)x, pos, cos_t, sin_t, heads, ld, hstride, off, half, max_pos, total);
   else rope_pairs_kernel<bf16><<<grid, 256, 0, s>>>((bf16*)x, pos, cos_t, sin_t, heads, ld, hstride, off, half, max_pos, total);
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int vb_rope_copy(int dtype, const void* a, long long lda, int a_head, int a_off, void* out, long long ldo, int o_head, int o_off,
+                            const int* pos, const float* cos_t, const float* sin_t, int T, int heads, int rot, int half, int max_pos, cudaStream_t s) {
+  const long long total = static_cast<long long>(T) * heads * rot;
+  if (total <= 0) return 0;
+  const int grid = static_cast<int>((total + 255) / 256);
+  if (dtype == 0)
+    rope_copy_kernel<float><<<grid, 256, 0, s>>>((const float*)a, lda, a_head, a_off, (float*)out, ldo, o_head, o_off, pos, cos_t, sin_t, heads, rot, half, max_pos, total);
+  else
+    rope_copy_kernel<bf16><<<grid, 256, 0, s>>>((const bf16*)a, lda, a_head, a_off, (bf16*)out, ldo, o_head, o_off, pos, cos_t, sin_t, heads, rot, half, max_pos, total);
   return static_cast<int>(cudaGetLastError());
 }
 

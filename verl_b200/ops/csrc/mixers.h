@@ -48,6 +48,19 @@ struct VbLatentAttn {
   float scale;
 };
 
+struct VbHeadwise {
+  const void* a; long long lda, a_head;   // a[m, h, k]
+  const void* w; long long w_head, ldw;   // w[h] as [N, K] (kn = 0) or [K, N] (kn = 1)
+  int kn;
+  void* out; long long ldo, o_head;
+  int M, N, K, H;
+  const float* gate; long long ldg;
+  // rot > 0: a[m, h, K .. K + rot) is rotated (pairs of the first 2 * half dimensions) and stored behind the product
+  int rot, half, max_pos;
+  const int* pos;
+  const float *cos_t, *sin_t;
+};
+
 extern "C" {
 void verl_count_launches(long long n);
 // gemm_simt.cu
@@ -63,6 +76,8 @@ int vb_embed_dyt(int dtype, const long long* ids, const void* w, float scale, fl
 int vb_dyt(int dtype, const float* x, void* h, const void* alpha, const void* nw, const void* nb, int T, int W, cudaStream_t s);
 int vb_rope_pairs(int dtype, void* x, const int* pos, const float* cos_t, const float* sin_t, int T, int heads, long long ld, int hstride,
                   int off, int dims, int max_pos, cudaStream_t s);
+int vb_rope_copy(int dtype, const void* a, long long lda, int a_head, int a_off, void* out, long long ldo, int o_head, int o_off, const int* pos,
+                 const float* cos_t, const float* sin_t, int T, int heads, int rot, int half, int max_pos, cudaStream_t s);
 int vb_latent_prep(int dtype, const void* p, long long ldp, const void* qn, const void* kn, float eps, const int* pos, const float* cos_t,
                    const float* sin_t, int dims, int max_pos, void* cq, void* lat, long long ldl, void* pages, long long page_stride,
                    int block_size, long long num_slots, const long long* slot, int T, int q_rank, int kv_rank, int rot, cudaStream_t s);
@@ -76,6 +91,12 @@ int vb_mlstm_scan(int dtype, const void* qkvg, long long ldp, const float* gates
                   int e, cudaStream_t s);
 int vb_mlstm_out(int dtype, const float* o, const void* g, long long ldg, const void* norm, float eps, void* out, long long ldo, int T, int H,
                  int e, cudaStream_t s);
+// headwise_mma.cu
+int vb_headwise(const VbHeadwise* p, cudaStream_t s);
+// latent_decode.cu
+int vb_latent_decode_splits(int S, int H, int rank, int width, int block_size, int max_keys);
+int vb_latent_decode(const VbLatentAttn* a, long long num_blocks, int nsplit, float* part_o, float* part_ml, cudaStream_t s);
+int vb_latent_decode_status();
 // latent_attention_simt.cu
 int vb_latent_attn_simt(int dtype, const VbLatentAttn* a, cudaStream_t s);
 }

@@ -15,7 +15,7 @@ import torch.nn.functional as TF
 from . import native
 
 __all__ = ["embed_dyt", "dynamic_tanh", "linear_act", "linear_split", "linear_residual_", "rope_pairs_", "latent_prep", "gather_pages",
-           "headwise_linear", "latent_attention_prefill", "latent_attention_decode", "mlstm_prefill", "mlstm_decode"]
+           "headwise_linear", "latent_absorb", "latent_attention_prefill", "latent_attention_decode", "mlstm_prefill", "mlstm_decode"]
 
 
 def _ops():
@@ -127,6 +127,15 @@ def headwise_linear(a: torch.Tensor, w: torch.Tensor, transposed: bool, gate: Op
     if gate is not None:
         y = y * torch.sigmoid(gate[:, : a.shape[1]]).unsqueeze(-1)
     return y.to(a.dtype).contiguous()
+
+
+def latent_absorb(q, uk, positions, cos, sin) -> torch.Tensor:
+    """Decode query in the latent space: ``q`` [S, H, dim + rot] -> [q_unrotated uk | rotated part] [S, H, kv_rank + rot] with ``uk``
+    [H, dim, kv_rank]."""
+    if q.is_cuda:
+        return _ops().latent_absorb(q, uk, positions, cos, sin)
+    dim = uk.shape[1]
+    return torch.cat([headwise_linear(q[..., :dim], uk, True), _rotate(q[..., dim:].float(), positions, cos, sin).to(q.dtype)], -1)
 
 
 def _sink_softmax(s: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor:
