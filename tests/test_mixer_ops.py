@@ -140,7 +140,7 @@ def attention_want(q, ku, kr, v, window, scale, sink, gate):
     return o * torch.sigmoid(gate)[:, :, None]
 
 
-ATT_SIZES = [(3, 16, 8, 24), (2, 128, 64, 128), (5, 40, 24, 48), (2, 10, 6, 12), (1, 64, 32, 64), (4, 48, 16, 128)]
+ATT_SIZES = [(3, 16, 8, 24), (2, 128, 64, 128), (5, 40, 24, 48), (2, 10, 6, 12), (1, 64, 32, 64), (4, 48, 16, 128), (2, 128, 128, 128), (2, 64, 16, 192)]
 
 
 @pytest.mark.parametrize("heads,du,dr,dv", ATT_SIZES)

@@ -36,7 +36,7 @@ NVCC_FLAGS = [
 ]
 
 # sources whose transcendental functions, divisions and square roots keep full fp32 accuracy
-PRECISE_MATH = ("gemm_simt", "mixer_kernels", "latent_attention_simt", "mlstm_chunk", "latent_decode", "headwise_mma", "latent_prefill_tcgen05")
+PRECISE_MATH = ("gemm_simt", "mixer_kernels", "latent_attention_simt", "mlstm_chunk", "latent_decode", "headwise_mma")
 
 
 def _nvcc_flags(stem: str) -> list:

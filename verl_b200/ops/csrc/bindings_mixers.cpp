@@ -252,7 +252,9 @@ Tensor latent_attn_prefill(const Tensor& q, const Tensor& ku, const Tensor& kr, 
   Tensor out = at::empty({q.size(0), q.size(1), v.size(2)}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   verl_count_launches(1);
-  CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
+  int rc = dt == 1 && a.T > 0 ? vb_latent_prefill(&a, (int)ku.size(0), cur_stream()) : -1;
+  if (rc < 0) rc = vb_latent_attn_simt(dt, &a, cur_stream());
+  CHECK_RC(rc, "latent_attn_prefill");
   return out;
 }
 

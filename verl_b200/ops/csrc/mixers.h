@@ -91,6 +91,9 @@ int vb_mlstm_scan(int dtype, const void* qkvg, long long ldp, const float* gates
                   int e, cudaStream_t s);
 int vb_mlstm_out(int dtype, const float* o, const void* g, long long ldg, const void* norm, float eps, void* out, long long ldo, int T, int H,
                  int e, cudaStream_t s);
+// latent_prefill_tcgen05.cu
+int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t s);
+int vb_latent_prefill_status();
 // headwise_mma.cu
 int vb_headwise(const VbHeadwise* p, cudaStream_t s);
 // latent_decode.cu
