@@ -67,6 +67,10 @@ def parse_args():
     p.add_argument("--offload", default="auto", choices=["auto", "on", "off"],
                    help="second Adam moment in pinned host memory (optimizer_offload), which leaves the GPU's memory to activations "
                         "instead of recomputation; auto = on one GPU, where the whole unsharded optimizer state would sit on it")
+    p.add_argument("--design", default=None, choices=["zorelorn"],
+                   help="instead of the GRPO step: prefill and decode throughput of this mixer-stack design at a few sizes, beside the uniform "
+                        "decoder of equal size (one JSON line per size and model)")
+    p.add_argument("--kernels", action="store_true", help="with --design: the kernels of both models, each against its roofline")
     p.add_argument("--critic", action="store_true", help="PPO with a critic of the same architecture and GAE instead of GRPO")
     return p.parse_args()
 
@@ -170,6 +174,10 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.design:
+        from verl_b200.workers.rollout.native.bench_stack import main as bench_stack
+
+        return bench_stack(args)
 
     import torch
     import torch.distributed as dist

@@ -225,16 +225,17 @@ def mlstm_want(p, gates, ib, fb, norm, cap, eps, H, d, e):
     return o * norm * torch.sigmoid(p[:, 2 * H * d + H * e :])
 
 
-MLSTM_SIZES = [(2, 16, 24), (3, 40, 16), (1, 128, 256), (2, 64, 64), (2, 10, 14), (1, 256, 96)]
+MLSTM_SIZES = [(2, 16, 24), (3, 40, 16), (1, 128, 256), (2, 64, 64), (2, 10, 14), (1, 256, 96), (2, 72, 320), (1, 64, 32)]
 
 
+@pytest.mark.parametrize("all_fresh", [False, True])
 @pytest.mark.parametrize("H,d,e", MLSTM_SIZES)
-def test_mlstm_prompts_and_steps(place, H, d, e):
+def test_mlstm_prompts_and_steps(place, H, d, e, all_fresh):
     """Prompts of unequal length, portions and single steps give what the token-by-token recurrence gives; slots are reused."""
     cap, eps, slots_n = 9.0, 1e-6, 6
     size = H * (d * e + d + 1)
     state = torch.full((slots_n, -(-size // 4) * 4 + 8), 3.0, device=place[0])[:, :size]       # stale content of an earlier user
-    lens = [1, 2, 63, 64, 65, 150]
+    lens = [1, 2, 63, 64, 65, 150 if not all_fresh else 900]
     parts = [mlstm_inputs(n + 12, H, d, e) for n in lens]
     want = [mlstm_want(p, g, parts[0][2], parts[0][3], parts[0][4], cap, eps, H, d, e) for p, g, *_ in parts]
     ib, fb, norm = (put(t, place) for t in parts[0][2:])
@@ -243,7 +244,7 @@ def test_mlstm_prompts_and_steps(place, H, d, e):
                           torch.cat([g[a:b] for (_, g, *_), a, b in zip(parts, lo, hi)]).to(place[0]))
     cu = lambda n: i32([0] + torch.tensor(n).cumsum(0).tolist(), place)
     p, g = cut([0] * 6, lens)
-    got = X.mlstm_prefill(p, g, ib, fb, cap, norm, eps, d, cu(lens), state, i32(slots, place), i32([1] * 6, place))
+    got = X.mlstm_prefill(p, g, ib, fb, cap, norm, eps, d, cu(lens), state, i32(slots, place), i32([1] * 6, place), all_fresh)
     row = 0
     for n, w in zip(lens, want):
         close(got[row : row + n], w[:n], place)

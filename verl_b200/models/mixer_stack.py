@@ -162,7 +162,7 @@ class MixerStackModel:
                 return self._attention_prefill(i, W, m, h, batch, pc, portion)
             p, gates = self._mlstm_in(W, m, h)
             return X.mlstm_prefill(p, gates, W["i.b"], W["f.b"], m.gate_cap, W["norm"], self.spec.norm_eps, m.dim, batch.cu_seqlens,
-                                   pc.cache.state(i) if pc is not None else None, pc.slots if pc is not None else None, fresh)
+                                   pc.cache.state(i) if pc is not None else None, pc.slots if pc is not None else None, fresh, not any(starts))
 
         return self._run(batch.input_ids, mix)
 

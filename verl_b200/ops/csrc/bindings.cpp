@@ -5,7 +5,6 @@
 #include <torch/library.h>
 
 #include "launchers.h"
-#include "mixers.h"
 
 #include <algorithm>
 #include <atomic>

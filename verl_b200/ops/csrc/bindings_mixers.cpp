@@ -336,7 +336,7 @@ Tensor mlstm_decode(const Tensor& p, const Tensor& gates, const Tensor& ib, cons
 
 // Portion of one or more sequences (cu int32 [B + 1]); slots int32 [B] (or none: nothing is kept), fresh int32 [B]: start from zero.
 Tensor mlstm_prefill(const Tensor& p, const Tensor& gates, const Tensor& ib, const Tensor& fb, double cap, const OptTensor& state, const OptTensor& slots,
-                     const OptTensor& fresh, const Tensor& cu, const Tensor& norm, double eps, int64_t d) {
+                     const OptTensor& fresh, const Tensor& cu, const Tensor& norm, double eps, int64_t d, bool all_fresh) {
   const MlstmShape s = mlstm_check(p, gates, ib, fb, norm, d);
   CHECK_I32(cu);
   const int64_t B = cu.numel() - 1;
@@ -348,13 +348,36 @@ Tensor mlstm_prefill(const Tensor& p, const Tensor& gates, const Tensor& ib, con
     TORCH_CHECK(slots->numel() == B && fresh->numel() == B);
   }
   const c10::cuda::CUDAGuard guard(p.device());
-  Tensor o = at::empty({s.T, s.H * s.e}, p.options().dtype(at::kFloat));
   Tensor out = at::empty({s.T, s.H * s.e}, p.options());
+  if (s.T == 0 || B == 0) return out;
+  const auto f32 = p.options().dtype(at::kFloat);
+  float* st = slots.has_value() ? state->data_ptr<float>() : nullptr;
+  const int64_t st_stride = slots.has_value() ? state->stride(0) : 0;
+  const char* g = reinterpret_cast<const char*>(p.data_ptr()) + (2 * s.H * s.d + s.H * s.e) * p.element_size();
+  if (s.dt == 1) {
+    int fused = 0;
+    const int nseg = vb_mlstm_chunk_segments((int)s.T, (int)B, (int)s.H, (int)s.d, (int)s.e, all_fresh || !slots.has_value(), &fused);
+    if (nseg > 0) {
+      Tensor local, raw;
+      if (nseg > 1) local = at::empty({B * (nseg - 1) * s.H * (s.d * s.e + s.d + 2)}, f32);
+      if (!fused) raw = at::empty({s.T, s.H * s.e}, f32);
+      int rc = vb_mlstm_chunk(p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap, st, st_stride, iptr(slots),
+                              iptr(fresh), cu.data_ptr<int>(), (int)B, nseg, nseg > 1 ? local.data_ptr<float>() : nullptr, norm.data_ptr(), (float)eps, out.data_ptr(),
+                              out.stride(0), fused ? nullptr : raw.data_ptr<float>(), (int)s.H, (int)s.d, (int)s.e, cur_stream());
+      if (rc >= 0) {
+        verl_count_launches((nseg > 1 ? 2 : 1) + (fused ? 0 : 1));
+        if (rc == 0 && !fused)
+          rc = vb_mlstm_out(s.dt, raw.data_ptr<float>(), g, p.stride(0), norm.data_ptr(), (float)eps, out.data_ptr(), out.stride(0), (int)s.T, (int)s.H, (int)s.e, cur_stream());
+        CHECK_RC(rc, "vb_mlstm_chunk");
+        return out;
+      }
+    }
+  }
+  Tensor o = at::empty({s.T, s.H * s.e}, f32);
   verl_count_launches(slots.has_value() ? 3 : 2);
   CHECK_RC(vb_mlstm_scan(s.dt, p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap,
-                         slots.has_value() ? state->data_ptr<float>() : nullptr, slots.has_value() ? state->stride(0) : 0, iptr(slots), iptr(fresh), cu.data_ptr<int>(), (int)B,
+                         st, st_stride, iptr(slots), iptr(fresh), cu.data_ptr<int>(), (int)B,
                          o.data_ptr<float>(), (int)s.T, (int)s.H, (int)s.d, (int)s.e, cur_stream()), "vb_mlstm_scan");
-  const char* g = reinterpret_cast<const char*>(p.data_ptr()) + (2 * s.H * s.d + s.H * s.e) * p.element_size();
   CHECK_RC(vb_mlstm_out(s.dt, o.data_ptr<float>(), g, p.stride(0), norm.data_ptr(), (float)eps, out.data_ptr(), out.stride(0), (int)s.T, (int)s.H, (int)s.e, cur_stream()),
            "vb_mlstm_out");
   return out;

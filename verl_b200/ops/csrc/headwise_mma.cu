@@ -35,19 +35,24 @@ headwise_kernel(const VbHeadwise p) {
   const bf16* B = reinterpret_cast<const bf16*>(p.w) + static_cast<long long>(h) * p.w_head;
   bf16* O = reinterpret_cast<bf16*>(p.out) + static_cast<long long>(h) * p.o_head;
   if (n0 >= p.N) {  // the positional part: pairs (2i, 2i + 1) of the first 2 * half dimensions turn, the rest is copied
-    const int half = p.half;
-    for (int i = tid; i < HW_T * p.rot; i += 128) {
-      const int m = m0 + i / p.rot, c = i % p.rot;
-      if (m >= p.M) continue;
-      const bf16* src = A + m * p.lda + p.K;
-      float o = to_f(src[c]);
-      if (c < 2 * half) {
-        const int at = min(max(p.pos[m], 0), p.max_pos - 1);
-        const float cc = p.cos_t[static_cast<long long>(at) * half + (c >> 1)], ss = p.sin_t[static_cast<long long>(at) * half + (c >> 1)];
-        const float w = to_f(src[c ^ 1]);
-        o = (c & 1) ? o * cc + w * ss : o * cc - w * ss;
+    const int hp = (p.rot + 1) / 2, per = hp < 128 ? 128 / hp : 1;   // pairs per row, rows per round
+    for (int c2 = tid % hp; c2 < hp && tid / hp < per; c2 += 128) {
+#pragma unroll 4
+      for (int r = tid / hp; r < HW_T; r += per) {
+        const int m = m0 + r, c = 2 * c2;
+        if (m >= p.M) continue;
+        const bf16* src = A + m * p.lda + p.K + c;
+        bf16* dst = O + m * p.ldo + p.N + c;
+        const float u = to_f(src[0]), v = c + 1 < p.rot ? to_f(src[1]) : 0.f;
+        float cc = 1.f, ss = 0.f;
+        if (c2 < p.half) {
+          const long long at = static_cast<long long>(min(max(p.pos[m], 0), p.max_pos - 1)) * p.half + c2;
+          cc = p.cos_t[at];
+          ss = p.sin_t[at];
+        }
+        dst[0] = from_f<bf16>(u * cc - v * ss);
+        if (c + 1 < p.rot) dst[1] = from_f<bf16>(v * cc + u * ss);
       }
-      O[m * p.ldo + p.N + c] = from_f<bf16>(o);
     }
     return;
   }

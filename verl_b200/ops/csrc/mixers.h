@@ -93,13 +93,16 @@ int vb_mlstm_out(int dtype, const float* o, const void* g, long long ldg, const 
                  int e, cudaStream_t s);
 // latent_prefill_tcgen05.cu
 int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t s);
-int vb_latent_prefill_status();
+// mlstm_chunk.cu
+int vb_mlstm_chunk_segments(int T, int B, int H, int d, int e, int all_fresh, int* fused);
+int vb_mlstm_chunk(const void* qkvg, long long ldp, const float* gates, long long ldg, const void* ib, const void* fb, float cap, float* state,
+                   long long slot_stride, const int* slots, const int* fresh, const int* cu, int B, int nseg, float* local, const void* norm,
+                   float eps, void* out, long long ldo, float* o, int H, int d, int e, cudaStream_t s);
 // headwise_mma.cu
 int vb_headwise(const VbHeadwise* p, cudaStream_t s);
 // latent_decode.cu
 int vb_latent_decode_splits(int S, int H, int rank, int width, int block_size, int max_keys);
 int vb_latent_decode(const VbLatentAttn* a, long long num_blocks, int nsplit, float* part_o, float* part_ml, cudaStream_t s);
-int vb_latent_decode_status();
 // latent_attention_simt.cu
 int vb_latent_attn_simt(int dtype, const VbLatentAttn* a, cudaStream_t s);
 }

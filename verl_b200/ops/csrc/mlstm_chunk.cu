@@ -1,0 +1,466 @@
+// mLSTM over prompts, 64 tokens at a time on m16n8k16 MMAs (bf16 projections, fp32 gates and state).
+//
+// With b_t the cumulative log forget gate inside a chunk, a_s = i_s - b_s and M_t = max(m_prev, max_{s <= t} a_s), the
+// recurrence's running maximum is m_t = b_t + M_t and
+//   o_t ~ exp(m_prev - M_t) q_t S_prev + sum_{s <= t} exp(a_s - M_t) (q_t . k_s) v_s
+//   S_C = exp(m_prev - M_C) S_prev + sum_s exp(a_s - M_C) k_s v_s^T
+// so a chunk is three small products. One CTA = (sequence segment, head, up to 256 columns of v); a warp owns 16 columns and
+// keeps their part of S^T in fp32 accumulators for the whole segment. The accumulator layout of S^T is the B-operand layout
+// of the read-out product, so S never leaves the registers; fp32 values that enter an MMA (S, the weighted scores, v weighted
+// by its gate) are split into two bf16 terms, which keeps 16 mantissa bits: the per-head norm behind the read-out magnifies
+// whatever is rounded where the terms of o cancel. Per-head RMS norm, weight and output gate close the chunk when one
+// CTA covers the head.
+//
+// Long sequences are cut into segments: a first launch (FULL = false) computes every segment's own contribution to the state
+// from nothing, the second starts each segment from the fold of those before it. Compiled without fast math.
+#include "mixers.h"
+#include "mixer_common.cuh"
+
+#include <math.h>
+
+namespace vb {
+
+typedef __nv_bfloat16 bf16;
+constexpr int MC_C = 64;          // tokens per chunk
+constexpr int MC_PP = MC_C + 8;   // row pitch of the weighted score tile
+
+struct MlstmChunkParams {
+  const bf16* p; long long ldp;      // [T, q | k | v | g]
+  const float* gates; long long ldg; // [T, i | f]
+  const bf16 *ib, *fb;
+  float cap;
+  float* state; long long slot_stride;
+  const int *slots, *fresh, *cu;
+  float* local;                      // [B, nseg - 1, H, d e + d + 2]: segment states from nothing
+  const bf16* norm;
+  float eps;
+  bf16* out; long long ldo;          // fused output, or
+  float* o;                          // raw read-out [T, H, e]
+  int H, d, e, nseg, cols;           // cols: columns of v per CTA
+};
+
+__device__ __forceinline__ uint32_t mc_smem(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
+__device__ __forceinline__ void mc_cp16(void* dst, const void* src, bool ok) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(mc_smem(dst)), "l"(src), "r"(ok ? 16 : 0));
+}
+__device__ __forceinline__ void mc_ldsm(uint32_t (&r)[4], uint32_t a) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mc_ldsm_t(uint32_t (&r)[4], uint32_t a) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mc_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// two floats as bf16 pair plus the pair of what rounding dropped
+__device__ __forceinline__ void mc_split(float x, float y, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+__device__ __forceinline__ float2 mc_unpack(uint32_t v) { return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u)); }
+
+template <int DP>
+struct McSmem {
+  static constexpr int QP = DP + 8, VP = (DP == 256 ? 128 : 256) + 8;    // row pitches
+  static constexpr int STAGE = (2 * MC_C * QP + MC_C * VP) * 2;
+  static constexpr int OFF_P = 2 * STAGE;
+  static constexpr int OFF_F = OFF_P + 2 * MC_C * MC_PP * 2;   // weighted scores in two bf16 terms
+  // floats: a, M, dec, eneg, w [64 each], den parts [4][64], qn [64], ss [2][16][64], n [DP], scalars [8]
+  static constexpr int FLOATS = 5 * MC_C + 4 * MC_C + MC_C + 2 * 16 * MC_C + DP + 8;
+  static constexpr int TOTAL = OFF_F + FLOATS * 4;
+};
+
+template <int DP, bool FULL>
+__global__ void __launch_bounds__(DP == 256 ? 256 : 512, 1)
+mlstm_chunk_kernel(const MlstmChunkParams P) {
+  using L = McSmem<DP>;
+  constexpr int KS = DP / 16, NT = DP / 8;
+  extern __shared__ __align__(16) uint8_t smem[];
+  float* fl = reinterpret_cast<float*>(smem + L::OFF_F);
+  float *sa = fl, *sM = sa + MC_C, *sdec = sM + MC_C, *sneg = sdec + MC_C, *sw = sneg + MC_C, *sden = sw + MC_C, *sqn = sden + 4 * MC_C,
+        *sss = sqn + MC_C, *sn = sss + 2 * 16 * MC_C, *sc = sn + DP;
+  bf16* sP = reinterpret_cast<bf16*>(smem + L::OFF_P);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nwarps = blockDim.x >> 5;
+  const int b = blockIdx.z / P.nseg, seg = blockIdx.z % P.nseg, h = blockIdx.y, c0 = blockIdx.x * P.cols;
+  const int H = P.H, d = P.d, e = P.e;
+  const int s0 = P.cu[b], len = P.cu[b + 1] - s0;
+  const int seg_len = ((len + P.nseg - 1) / P.nseg + MC_C - 1) / MC_C * MC_C;
+  const int t_lo = seg * seg_len, t_hi = min(len, t_lo + seg_len);
+  if (t_lo >= t_hi) return;
+  if (!FULL && t_hi == len) return;                  // nothing follows: the segment's own state is not needed
+  const int e0 = c0 + warp * 16;                     // first column of this warp
+  const bool e_ok = e0 < e && warp * 16 < P.cols;
+  const int er = lane >> 2, kc = (lane & 3) * 2, mi = lane >> 3, r8 = lane & 7;
+  const long long lsize = static_cast<long long>(d) * e + d + 2;
+  const bool have = P.slots != nullptr && P.slots[b] >= 0;
+  float* slot = have ? P.state + static_cast<long long>(P.slots[b]) * P.slot_stride : nullptr;
+  float* slot_S = have ? slot + static_cast<long long>(h) * d * e : nullptr;
+  float* slot_n = have ? slot + static_cast<long long>(H) * d * e + h * d : nullptr;
+  float* slot_m = have ? slot + static_cast<long long>(H) * d * e + H * d + h : nullptr;
+
+  // ---- S^T accumulators: tile j covers d columns [8j, 8j + 8); element (e0 + er (+ 8), 8j + kc (+ 1))
+  float S[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.f;
+  auto each = [&](auto fn) {                         // fn(tile, index, d row, e column) over this thread's valid elements
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int dd = j * 8 + kc + (i & 1), ee = e0 + er + (i >> 1) * 8;
+        if (e_ok && dd < d && ee < e) fn(S[j][i], dd, ee);
+      }
+  };
+  float m_prev = FULL ? 0.f : -INFINITY, f_total = 0.f;
+  for (int r = tid; r < DP; r += blockDim.x) sn[r] = 0.f;
+  if (FULL) {
+    if (have && P.fresh != nullptr && P.fresh[b] == 0) {
+      each([&](float& v, int dd, int ee) { v = slot_S[static_cast<long long>(dd) * e + ee]; });
+      for (int r = tid; r < d; r += blockDim.x) sn[r] = slot_n[r];
+      m_prev = *slot_m;
+    }
+    for (int g = 0; g < seg; ++g) {                  // fold of the segments before this one
+      const float* loc = P.local + ((static_cast<long long>(b) * (P.nseg - 1) + g) * H + h) * lsize;
+      const float m_loc = loc[lsize - 2], F = loc[lsize - 1];
+      const float m = fmaxf(F + m_prev, m_loc), keep = expf(F + m_prev - m), add = expf(m_loc - m);
+      each([&](float& v, int dd, int ee) { v = keep * v + add * loc[static_cast<long long>(dd) * e + ee]; });
+      for (int r = tid; r < d; r += blockDim.x) sn[r] = keep * sn[r] + add * loc[static_cast<long long>(d) * e + r];
+      m_prev = m;
+    }
+  }
+
+  const bf16* base = P.p + static_cast<long long>(s0) * P.ldp;
+  auto load = [&](int st, int t0) {
+    bf16* q = reinterpret_cast<bf16*>(smem + st * L::STAGE);
+    bf16* k = q + MC_C * L::QP;
+    bf16* v = k + MC_C * L::QP;
+    for (int i = tid; i < MC_C * (DP / 8); i += blockDim.x) {
+      const int r = i / (DP / 8), c = (i % (DP / 8)) * 8;
+      const bool ok = t0 + r < t_hi && c < d;
+      const bf16* row = base + static_cast<long long>(t0 + r) * P.ldp;
+      if (FULL) mc_cp16(q + r * L::QP + c, ok ? row + h * d + c : base, ok);
+      mc_cp16(k + r * L::QP + c, ok ? row + (H + h) * d + c : base, ok);
+    }
+    const int vc = (nwarps * 16) / 8;
+    for (int i = tid; i < MC_C * vc; i += blockDim.x) {
+      const int r = i / vc, c = (i % vc) * 8;
+      const bool ok = t0 + r < t_hi && c0 + c < e;
+      mc_cp16(v + r * L::VP + c, ok ? base + static_cast<long long>(t0 + r) * P.ldp + 2 * H * d + static_cast<long long>(h) * e + c0 + c : base, ok);
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+  const float ibv = to_f(P.ib[h]), fbv = to_f(P.fb[h]);
+  const float qs = 1.f / sqrtf(static_cast<float>(d));
+  load(0, t_lo);
+  int st = 0;
+  for (int t0 = t_lo; t0 < t_hi; t0 += MC_C, st ^= 1) {
+    // ---- gates of the chunk (warp 0, two neighbouring tokens per lane)
+    if (warp == 0) {
+      float il[2], ff[2];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int t = t0 + lane * 2 + u;
+        il[u] = -INFINITY;
+        ff[u] = 0.f;
+        if (t < t_hi) {
+          const float* g = P.gates + static_cast<long long>(s0 + t) * P.ldg;
+          il[u] = P.cap * tanhf((g[h] + ibv) / P.cap);
+          ff[u] = log_sigmoid(P.cap * tanhf((g[H + h] + fbv) / P.cap));
+        }
+      }
+      float run = ff[0] + ff[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float x = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += x;
+      }
+      const float b1 = run, b0 = run - ff[1];
+      const float a0 = il[0] - b0, a1 = il[1] - b1;
+      float mx = fmaxf(a0, a1);
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float x = __shfl_up_sync(0xffffffffu, mx, o);
+        if (lane >= o) mx = fmaxf(mx, x);
+      }
+      float before = __shfl_up_sync(0xffffffffu, mx, 1);
+      if (lane == 0) before = -INFINITY;
+      const float M0 = fmaxf(m_prev, fmaxf(before, a0)), M1 = fmaxf(m_prev, mx);
+      const float MC = __shfl_sync(0xffffffffu, M1, 31), bC = __shfl_sync(0xffffffffu, b1, 31);
+      const float aa[2] = {a0, a1}, MM[2] = {M0, M1}, bb[2] = {b0, b1};
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int t = lane * 2 + u;
+        sa[t] = aa[u];
+        sM[t] = MM[u];
+        sdec[t] = expf(m_prev - MM[u]);
+        sneg[t] = expf(-(bb[u] + MM[u]));
+        sw[t] = expf(aa[u] - MC);
+      }
+      if (lane == 0) {
+        sc[0] = expf(m_prev - MC);
+        sc[1] = bC + MC;
+        sc[2] = bC;
+      }
+    }
+    asm volatile("cp.async.wait_group 0;");
+    __syncthreads();                                  // A: chunk and gates are in shared memory, the other stage is free
+    if (t0 + MC_C < t_hi) load(st ^ 1, t0 + MC_C);
+    const bf16* q = reinterpret_cast<const bf16*>(smem + st * L::STAGE);
+    const bf16* k = q + MC_C * L::QP;
+    const bf16* v = k + MC_C * L::QP;
+    const uint32_t uq = mc_smem(q), uk = mc_smem(k), uv = mc_smem(v), uP = mc_smem(sP);
+    const float decC = sc[0], m_next = sc[1];
+    if (FULL) {
+      // ---- weighted scores P = exp(a_s - M_t) q_t . k_s, in 16 x 16 blocks; blocks above the diagonal are zero
+      for (int blk = warp; blk < 16; blk += nwarps) {
+        const int tb = (blk >> 2) * 16, sb = (blk & 3) * 16;
+        float acc[2][4] = {};
+        if (sb <= tb) {
+#pragma unroll
+          for (int kk = 0; kk < KS; ++kk) {
+            uint32_t fa[4], fb[4];
+            mc_ldsm(fa, uq + ((tb + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
+            mc_ldsm(fb, uk + ((sb + (mi >> 1) * 8 + r8) * L::QP + kk * 16 + (mi & 1) * 8) * 2);
+            mc_mma(acc[0], fa, fb[0], fb[1]);
+            mc_mma(acc[1], fa, fb[2], fb[3]);
+          }
+        }
+        float rs[2] = {0.f, 0.f};
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int t = tb + er + half * 8;
+          const float Mt = sM[t];
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            float x[2];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+              const int s = sb + j * 8 + kc + u;
+              x[u] = s <= t ? acc[j][half * 2 + u] * qs * expf(sa[s] - Mt) : 0.f;
+              rs[half] += x[u];
+            }
+            uint32_t hi, lo;
+            mc_split(x[0], x[1], hi, lo);
+            *reinterpret_cast<uint32_t*>(sP + t * MC_PP + sb + j * 8 + kc) = hi;
+            *reinterpret_cast<uint32_t*>(sP + (MC_C + t) * MC_PP + sb + j * 8 + kc) = lo;
+          }
+          rs[half] += __shfl_xor_sync(0xffffffffu, rs[half], 1);
+          rs[half] += __shfl_xor_sync(0xffffffffu, rs[half], 2);
+          if ((lane & 3) == 0) sden[(blk & 3) * MC_C + t] = rs[half];
+        }
+      }
+      // ---- q_t . n_prev
+      for (int t = warp; t < MC_C; t += nwarps) {
+        float x = 0.f;
+        for (int c = lane; c < DP; c += 32) x += to_f(q[t * L::QP + c]) * sn[c];
+        x = warp_sum(x);
+        if (lane == 0) sqn[t] = x * qs;
+      }
+      __syncthreads();                                // B: scores, row sums
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf) {                // 32 tokens at a time
+        float o[2][2][4] = {};
+        if (e_ok) {
+#pragma unroll
+          for (int kk = 0; kk < KS; ++kk) {           // read-out of the state
+            uint32_t h0, l0, h1, l1, h2, l2, h3, l3;
+            mc_split(S[2 * kk][0], S[2 * kk][1], h0, l0);
+            mc_split(S[2 * kk + 1][0], S[2 * kk + 1][1], h1, l1);
+            mc_split(S[2 * kk][2], S[2 * kk][3], h2, l2);
+            mc_split(S[2 * kk + 1][2], S[2 * kk + 1][3], h3, l3);
+#pragma unroll
+            for (int m = 0; m < 2; ++m) {
+              uint32_t fa[4];
+              mc_ldsm(fa, uq + ((hf * 32 + m * 16 + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
+              mc_mma(o[m][0], fa, h0, h1);
+              mc_mma(o[m][1], fa, h2, h3);
+              mc_mma(o[m][0], fa, l0, l1);
+              mc_mma(o[m][1], fa, l2, l3);
+            }
+          }
+#pragma unroll
+          for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+              const float f = sdec[hf * 32 + m * 16 + half * 8 + er] * qs;
+              o[m][0][half * 2] *= f; o[m][0][half * 2 + 1] *= f;
+              o[m][1][half * 2] *= f; o[m][1][half * 2 + 1] *= f;
+            }
+#pragma unroll
+          for (int kk = 0; kk < 2 + 2 * hf; ++kk) {   // the chunk's own tokens up to this half
+            uint32_t fv[4];
+            mc_ldsm_t(fv, uv + ((kk * 16 + (mi & 1) * 8 + r8) * L::VP + warp * 16 + (mi >> 1) * 8) * 2);
+#pragma unroll
+            for (int m = 0; m < 2; ++m) {
+              uint32_t fa[4];
+              mc_ldsm(fa, uP + ((hf * 32 + m * 16 + (mi & 1) * 8 + r8) * MC_PP + kk * 16 + (mi >> 1) * 8) * 2);
+              mc_mma(o[m][0], fa, fv[0], fv[1]);
+              mc_mma(o[m][1], fa, fv[2], fv[3]);
+              mc_ldsm(fa, uP + ((MC_C + hf * 32 + m * 16 + (mi & 1) * 8 + r8) * MC_PP + kk * 16 + (mi >> 1) * 8) * 2);
+              mc_mma(o[m][0], fa, fv[0], fv[1]);
+              mc_mma(o[m][1], fa, fv[2], fv[3]);
+            }
+          }
+        }
+        // ---- denominator; sum of squares over the head
+#pragma unroll
+        for (int m = 0; m < 2; ++m)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int t = hf * 32 + m * 16 + half * 8 + er;
+            const float den = sdec[t] * sqn[t] + ((sden[t] + sden[MC_C + t]) + (sden[2 * MC_C + t] + sden[3 * MC_C + t]));
+            const float inv = 1.f / (fmaxf(fabsf(den), sneg[t]) + 1e-6f);
+            float ss = 0.f;
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+              for (int u = 0; u < 2; ++u) {
+                float& x = o[m][n][half * 2 + u];
+                x *= inv;
+                ss += x * x;
+              }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            if ((lane & 3) == 0) sss[(hf * 16 + warp) * MC_C + t] = ss;
+          }
+        if (P.o == nullptr) __syncthreads();          // C
+        if (e_ok) {
+#pragma unroll
+          for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+              const int t = hf * 32 + m * 16 + half * 8 + er;
+              if (t0 + t >= t_hi) continue;
+              const long long tok = s0 + t0 + t;
+              if (P.o != nullptr) {
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                  const int ee = e0 + n * 8 + kc;
+                  if (ee < e) *reinterpret_cast<float2*>(P.o + (tok * H + h) * e + ee) = make_float2(o[m][n][half * 2], o[m][n][half * 2 + 1]);
+                }
+              } else {
+                float ss = 0.f;
+                for (int w = 0; w < nwarps; ++w) ss += sss[(hf * 16 + w) * MC_C + t];
+                const float rs = 1.f / sqrtf(ss / e + P.eps);
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                  const int ee = e0 + n * 8 + kc;
+                  if (ee >= e) continue;
+                  const float2 g = mc_unpack(*reinterpret_cast<const uint32_t*>(P.p + tok * P.ldp + 2 * H * d + static_cast<long long>(H + h) * e + ee));
+                  const float2 w = mc_unpack(*reinterpret_cast<const uint32_t*>(P.norm + h * e + ee));
+                  *reinterpret_cast<__nv_bfloat162*>(P.out + tok * P.ldo + h * e + ee) =
+                      __floats2bfloat162_rn(o[m][n][half * 2] * rs * w.x * sigmoid_f(g.x), o[m][n][half * 2 + 1] * rs * w.y * sigmoid_f(g.y));
+                }
+              }
+            }
+        }
+      }
+    }
+    // ---- state update: S^T = decC S^T + (w v)^T k
+    if (e_ok) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j) { S[j][0] *= decC; S[j][1] *= decC; S[j][2] *= decC; S[j][3] *= decC; }
+#pragma unroll
+      for (int kk = 0; kk < MC_C / 16; ++kk) {
+        uint32_t fv[4], hi[4], lo[4];
+        // (w v)^T as A: rows = v columns, k = tokens; registers {e0 s0, e8 s0, e0 s8, e8 s8}
+        mc_ldsm_t(fv, uv + ((kk * 16 + (mi >> 1) * 8 + r8) * L::VP + warp * 16 + (mi & 1) * 8) * 2);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int s = kk * 16 + (i >> 1) * 8 + kc;
+          const float2 x = mc_unpack(fv[i]);
+          mc_split(x.x * sw[s], x.y * sw[s + 1], hi[i], lo[i]);
+        }
+#pragma unroll
+        for (int j = 0; j < NT / 2; ++j) {
+          uint32_t fk[4];
+          mc_ldsm_t(fk, uk + ((kk * 16 + (mi & 1) * 8 + r8) * L::QP + j * 16 + (mi >> 1) * 8) * 2);
+          mc_mma(S[2 * j], hi, fk[0], fk[1]);
+          mc_mma(S[2 * j + 1], hi, fk[2], fk[3]);
+          mc_mma(S[2 * j], lo, fk[0], fk[1]);
+          mc_mma(S[2 * j + 1], lo, fk[2], fk[3]);
+        }
+      }
+    }
+    for (int r = tid; r < DP; r += blockDim.x) {
+      float x = decC * sn[r];
+#pragma unroll 8
+      for (int s = 0; s < MC_C; ++s) x += sw[s] * to_f(k[s * L::QP + r]);
+      sn[r] = x;
+    }
+    m_prev = m_next;
+    f_total += sc[2];
+    __syncthreads();                                  // D: gates and n may be replaced
+  }
+  // ---- final state of the sequence, or this segment's own state
+  if (!FULL) {
+    float* loc = P.local + ((static_cast<long long>(b) * (P.nseg - 1) + seg) * H + h) * lsize;
+    each([&](float& v, int dd, int ee) { loc[static_cast<long long>(dd) * e + ee] = v; });
+    if (blockIdx.x == 0) {
+      for (int r = tid; r < d; r += blockDim.x) loc[static_cast<long long>(d) * e + r] = sn[r];
+      if (tid == 0) { loc[lsize - 2] = m_prev; loc[lsize - 1] = f_total; }
+    }
+  } else if (have && t_hi == len) {
+    each([&](float& v, int dd, int ee) { slot_S[static_cast<long long>(dd) * e + ee] = v; });
+    if (blockIdx.x == 0) {
+      for (int r = tid; r < d; r += blockDim.x) slot_n[r] = sn[r];
+      if (tid == 0) *slot_m = m_prev;
+    }
+  }
+}
+
+static int mc_dp(int d) { return d <= 64 ? 64 : (d <= 128 ? 128 : 256); }
+static int mc_blocks(int d, int e) { const int mx = mc_dp(d) == 256 ? 128 : 256; return (e + mx - 1) / mx; }
+
+template <int DP>
+static int mc_launch(const MlstmChunkParams& p, int B, int blocks, int threads, cudaStream_t s) {
+  cudaError_t e = cudaFuncSetAttribute(mlstm_chunk_kernel<DP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, McSmem<DP>::TOTAL);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(mlstm_chunk_kernel<DP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, McSmem<DP>::TOTAL);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  const dim3 grid(blocks, p.H, B * p.nseg);
+  if (p.nseg > 1) mlstm_chunk_kernel<DP, false><<<grid, threads, McSmem<DP>::TOTAL, s>>>(p);
+  mlstm_chunk_kernel<DP, true><<<grid, threads, McSmem<DP>::TOTAL, s>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace vb
+
+using namespace vb;
+
+// Segments a sequence is cut into (1 = none; the workspace then needs B * (nseg - 1) * H * (d e + d + 2) floats), or 0 when the
+// sizes are not served. all_fresh: every sequence starts from zero.
+extern "C" int vb_mlstm_chunk_segments(int T, int B, int H, int d, int e, int all_fresh, int* fused) {
+  if (d % 8 || e % 8 || d > 256 || d < 8 || e < 8) return 0;
+  const int blocks = mc_blocks(d, e);
+  if (blocks > 1 && !all_fresh) return 0;   // column blocks would read n and m while the first one replaces them
+  *fused = blocks == 1;
+  if (!all_fresh) return 1;
+  int s = 148 / (B * H * blocks);
+  const int by_len = T / B / (4 * MC_C);
+  if (s > by_len) s = by_len;
+  if (s > 32) s = 32;
+  return (s < 1 || static_cast<long long>(B) * s > 65535) ? 1 : s;
+}
+
+extern "C" int vb_mlstm_chunk(const void* qkvg, long long ldp, const float* gates, long long ldg, const void* ib, const void* fb, float cap,
+                              float* state, long long slot_stride, const int* slots, const int* fresh, const int* cu, int B, int nseg, float* local,
+                              const void* norm, float eps, void* out, long long ldo, float* o, int H, int d, int e, cudaStream_t s) {
+  if (ldp % 8 || (reinterpret_cast<uintptr_t>(qkvg) & 15) || (ldo % 2) || (reinterpret_cast<uintptr_t>(norm) & 3) || static_cast<long long>(B) * nseg > 65535 || H > 65535) return -1;
+  MlstmChunkParams p{};
+  p.p = reinterpret_cast<const bf16*>(qkvg); p.ldp = ldp; p.gates = gates; p.ldg = ldg;
+  p.ib = reinterpret_cast<const bf16*>(ib); p.fb = reinterpret_cast<const bf16*>(fb); p.cap = cap;
+  p.state = state; p.slot_stride = slot_stride; p.slots = slots; p.fresh = fresh; p.cu = cu; p.local = local;
+  p.norm = reinterpret_cast<const bf16*>(norm); p.eps = eps; p.out = reinterpret_cast<bf16*>(out); p.ldo = ldo; p.o = o;
+  p.H = H; p.d = d; p.e = e; p.nseg = nseg;
+  const int blocks = mc_blocks(d, e);
+  p.cols = ((e + blocks - 1) / blocks + 15) / 16 * 16;
+  const int warps = p.cols / 16 < 4 ? 4 : p.cols / 16;
+  switch (mc_dp(d)) {
+    case 64: return mc_launch<64>(p, B, blocks, warps * 32, s);
+    case 128: return mc_launch<128>(p, B, blocks, warps * 32, s);
+    default: return mc_launch<256>(p, B, blocks, warps * 32, s);
+  }
+}

@@ -221,12 +221,14 @@ def _mlstm_token(S, n, m, q, k, v, i_log, f_log):
     return torch.einsum("hde,hd->he", S, q) / den[:, None]
 
 
-def mlstm_prefill(p, gates, ib, fb, cap: float, norm, eps: float, dim: int, cu, state=None, slots=None, fresh=None) -> torch.Tensor:
+def mlstm_prefill(p, gates, ib, fb, cap: float, norm, eps: float, dim: int, cu, state=None, slots=None, fresh=None,
+                  all_fresh: bool = False) -> torch.Tensor:
     """Matrix-memory recurrence over packed portions. ``p`` [T, q | k | v | g] in the model's type, ``gates`` [T, i | f] fp32
     pre-activations. Sequence b starts from zero when ``fresh[b]`` (else from ``state[slots[b]]``) and leaves its final state in
-    ``state[slots[b]]``; without ``slots`` every sequence starts from zero and nothing is kept."""
+    ``state[slots[b]]``; without ``slots`` every sequence starts from zero and nothing is kept. ``all_fresh``: the host knows that
+    every sequence is fresh (long prompts may then be cut into segments that run side by side)."""
     if p.is_cuda:
-        return _ops().mlstm_prefill(p, gates, ib, fb, float(cap), state, slots, fresh, cu, norm, float(eps), int(dim))
+        return _ops().mlstm_prefill(p, gates, ib, fb, float(cap), state, slots, fresh, cu, norm, float(eps), int(dim), bool(all_fresh))
     H = ib.numel()
     e = norm.numel() // H
     q, k, v, g, il, fl = _mlstm_parts(p, gates, ib, fb, cap, dim, e)

@@ -1,0 +1,207 @@
+"""Serving benchmark of a mixer-stack design beside the uniform decoder of equal size (same width, layers and parameters).
+
+    python bench.py --design zorelorn            # all sizes: prefill and decode throughput of both models
+    python bench.py --design zorelorn --kernels  # the kernels behind them, each against its roofline
+
+Random weights and tokens. Prefill runs packed prompts through the engine's prompt path into the cache, decode replays the
+captured decode step over all slots; CUDA events around every timed region, after warm-up, on inputs larger than L2. One
+JSON line per measurement.
+"""
+
+from __future__ import annotations
+
+import json
+
+import torch
+
+from ....models import FlatParams, ModelConfig
+from ....ops import functional as F
+from ....ops import mixers as X
+from ....ops import native
+from ....ops.bench_kernels import Timer, _peaks
+from ....utils.profiler.clocks import ClockSampler
+from .engine import RolloutEngine
+
+SIZES = {  # name -> (width, heads, q_rank, window, ff, layers, prompts, prompt length, decode slots, decode context)
+    "width2048": dict(width=2048, heads=16, q_rank=768, window=1024, ff=8192, layers=16, prompts=8, prompt_len=2048, slots=256, ctx=2048),
+    "width4096": dict(width=4096, heads=32, q_rank=1536, window=4096, ff=16384, layers=8, prompts=4, prompt_len=4096, slots=128, ctx=4096),
+}
+VOCAB = 32768
+
+
+def zorelorn_config(s: dict) -> ModelConfig:
+    attn = dict(type="latent_attention", mlp={"kind": "dense", "ff": s["ff"]},
+                mixer=dict(heads=s["heads"], dim=128, rot_dim=64, vdim=128, q_rank=s["q_rank"], kv_rank=512, mask={"size": s["window"]}, scale=192 ** -0.5,
+                           rot=dict(base=500000.0, dims=64, scaling=dict(factor=8.0, original=8192, fast=32.0, slow=1.0))))
+    mlstm = dict(type="mlstm", mlp=None, mixer=dict(heads=s["heads"] // 2, dim=128, vdim=256, gate_cap=15.0))
+    return ModelConfig.from_hf_dict({"architecture": "Zorelorn", "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "vocab": VOCAB, "width": s["width"],
+                                     "layers": [attn if i % 2 == 0 else mlstm for i in range(s["layers"])]})
+
+
+def uniform_config(s: dict, params: int) -> ModelConfig:
+    """Llama-type decoder of the same width and number of layers; its MLP is sized so that the parameters agree."""
+    mk = lambda ff: ModelConfig(model_type="llama", vocab_size=VOCAB, hidden_size=s["width"], intermediate_size=ff, num_hidden_layers=s["layers"],
+                                num_attention_heads=s["width"] // 128, num_key_value_heads=max(1, s["width"] // 512), head_dim=128, rope_theta=500000.0,
+                                max_position_embeddings=8192)
+    return mk(max(256, round((params - mk(0).num_parameters()) / (3 * s["width"] * s["layers"]) / 256) * 256))
+
+
+def _events(fn, steps: int) -> float:
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    a.record()
+    for _ in range(steps):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / steps
+
+
+def bench_model(cfg: ModelConfig, s: dict, steps: int, warmup: int) -> dict:
+    dev = torch.device("cuda", torch.cuda.current_device())
+    P = FlatParams(cfg, dtype=torch.bfloat16, device=dev)
+    P.init_weights(seed=1, std=0.02)
+    bs, S, n, L = 64, s["slots"], s["prompts"], s["prompt_len"]
+    per = -(-(s["ctx"] + 64) // bs)
+    eng = RolloutEngine(cfg, P, max_num_seqs=S, max_model_len=per * bs, block_size=bs, num_blocks=S * per, eos_token_id=-1)
+    ids = torch.randint(0, VOCAB, (n * L,))
+    table = torch.arange(S * per, dtype=torch.int32).view(S, per)
+
+    def prefill():
+        h, batch = eng._run_portions(ids, [0] * n, [L] * n, table[:n], list(range(n)))
+        return eng._logits(h[batch.cu_seqlens[1:].long() - 1])
+
+    for _ in range(warmup):
+        prefill()
+    sampler = ClockSampler(dev.index or 0, period_s=0.02).start()
+    ms_p = _events(prefill, steps)
+    eng.block_table.copy_(table)
+    for t, v in ((eng.tok, 5), (eng.pos, s["ctx"]), (eng.ctx, s["ctx"] + 1), (eng.gen, 1), (eng.max_new, 1 << 20)):
+        t.fill_(v)
+    eng.active.fill_(True)
+    eng.ignore_eos.fill_(True)
+    eng._ensure_out(64)
+    eng._decode_steps(warmup)
+    n0 = native.launch_count()
+    ms_d = _events(lambda: eng._decode_steps(1), 16)
+    launches = (native.launch_count() - n0) // 16
+    clocks = sampler.stop()
+    native.check_status()
+    out = {"parameters": cfg.num_parameters(), "prefill_tokens_per_s": round(n * L / ms_p * 1e3), "prefill_ms": round(ms_p, 3),
+           "decode_tokens_per_s": round(S / ms_d * 1e3), "decode_ms_per_step": round(ms_d, 3), "decode_kernels_per_step": launches, "clocks": clocks}
+    del eng, P
+    torch.cuda.empty_cache()
+    return out
+
+
+def run_models(steps: int, warmup: int, only=None) -> None:
+    for name, s in SIZES.items():
+        if only and name not in only:
+            continue
+        z = zorelorn_config(s)
+        for label, cfg in (("zorelorn", z), ("uniform decoder of equal size", uniform_config(s, z.num_parameters()))):
+            r = bench_model(cfg, s, steps, max(3, warmup))
+            print(json.dumps({"bench": "serving", "size": name, "model": label, "intermediate_size": cfg.intermediate_size, **s, **r, "dtype": "bf16",
+                              "data": "synthetic (random weights and tokens)"}), flush=True)
+
+
+# --------------------------------------------------------------------------------------------- kernels
+def run_kernels(iters: int = 20, only=None, sizes=None) -> None:
+    dev = torch.device("cuda", torch.cuda.current_device())
+    pk, timer = _peaks(), Timer(dev, iters, 3)
+    r = lambda *sh, sc=1.0, dt=torch.bfloat16: (torch.randn(*sh, device=dev) * sc).to(dt)
+
+    def case(size, phase, kernel, fn, flops, nbytes, new):
+        if only and kernel not in only:
+            return
+        ms = timer(fn)
+        floor = max(flops / (pk["bf16_tflops"] * 1e9), nbytes / (pk["hbm_gbs"] * 1e6))
+        print(json.dumps({"bench": "kernel", "size": size, "phase": phase, "kernel": kernel, "design": "zorelorn" if new else "uniform decoder", "us": round(ms * 1e3, 2),
+                          "roofline_us": round(floor * 1e3, 2), "fraction_of_measured": round(floor / ms, 3), "bound": "flops" if flops / pk["bf16_tflops"] > nbytes / pk["hbm_gbs"] * 1e3 else "bytes",
+                          "clocks": timer.clocks}), flush=True)
+
+    for name, s in SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        W, H, qr, ff, w = s["width"], s["heads"], s["q_rank"], s["ff"], s["window"]
+        Hm, d, e, kr, rot, dim, vd = H // 2, 128, 256, 512, 64, 128, 128
+        for phase, T in (("prefill", s["prompts"] * s["prompt_len"]), ("decode", s["slots"])):
+            h, x = r(T, W), torch.randn(T, W, device=dev)
+            norm = (r(1), r(W), r(W))
+            cut = qr + kr + rot
+            w_in, w_up, w_down, w_o = r(cut + H, W, sc=0.02), r(ff, W, sc=0.02), r(W, ff, sc=0.02), r(W, H * vd, sc=0.02)
+            act, att = r(T, ff), r(T, H * vd)
+            mm = lambda m, n, k: (2.0 * m * n * k, 2.0 * (m * k + n * k + m * n))
+            f, b = mm(T, cut + H, W)
+            case(name, phase, "linear_split (latent input projections)", lambda: X.linear_split(h, w_in, cut), f, b, True)
+            f, b = mm(T, ff, W)
+            case(name, phase, "linear_act (up projection + gelu)", lambda: X.linear_act(h, w_up, "gelu_erf"), f, b, True)
+            case(name, phase, "gemm (same product, no epilogue)", lambda: F.gemm(h, w_up), f, b, False)
+            f, b = mm(T, W, ff)
+            case(name, phase, "linear_residual (down projection + residual + norm)", lambda: X.linear_residual_(act, w_down, x, norm), f, b + 8.0 * T * W, True)
+            case(name, phase, "gemm (same product, no epilogue, K deep)", lambda: F.gemm(act, w_down), f, b, False)
+            f, b = mm(T, W, H * vd)
+            case(name, phase, "linear_residual (output projection + residual + norm)", lambda: X.linear_residual_(att, w_o, x, norm), f, b + 8.0 * T * W, True)
+            case(name, phase, "gemm (output projection)", lambda: F.gemm(att, w_o), f, b, False)
+            y = r(T, W)
+            case(name, phase, "rmsnorm with residual", lambda: F.rms_norm(h, norm[1], 1e-6, residual=y), 0, 8.0 * T * W, False)
+            cos, sin = F.rope_table(8192, rot, 5e5, dev)
+            pos = torch.arange(T, device=dev, dtype=torch.int32) % 4096
+            p, qn, kn = r(T, cut), r(qr), r(kr)
+            case(name, phase, "latent_prep (norms, rotation, rows)", lambda: X.latent_prep(p, qn, kn, 1e-6, pos, cos, sin, None, None, True), 0, 4.0 * T * cut, True)
+            q = r(T, H, dim + rot)
+            if phase == "prefill":
+                case(name, phase, "rope_pairs (query rotation)", lambda: X.rope_pairs_(q, pos, cos, sin, dim), 0, 4.0 * T * H * rot, True)
+                c = r(T, 128)
+                cs2, sn2 = F.rope_table(8192, 128, 5e5, dev)
+                qf = r(T, H, 128)
+                case(name, phase, "rope (query rotation, uniform)", lambda: F.apply_rope_(qf, pos, cs2, sn2), 0, 4.0 * T * H * 128, False)
+                n, L = s["prompts"], s["prompt_len"]
+                cu = (torch.arange(n + 1, device=dev, dtype=torch.int32) * L)
+                kv, rows, sink, gate = r(T, H * (dim + vd)), r(T, kr + rot), r(H), torch.randn(T, H, device=dev)
+                ku, v = kv[:, : H * dim].view(T, H, dim), kv[:, H * dim :].view(T, H, vd)
+                pairs = n * sum(min(i + 1, w) for i in range(L))
+                case(name, phase, "latent_attention_prefill", lambda: X.latent_attention_prefill(q, ku, rows[:, kr:], v, cu, cu, w, 192 ** -0.5, sink, gate),
+                     2.0 * pairs * H * (dim + rot + vd), 2.0 * T * (H * (dim + rot + dim + 2 * vd) + rot), True)
+                nkv = max(1, W // 512)
+                qq, kk, vv = r(T, W // 128, 128), r(T, nkv, 128), r(T, nkv, 128)
+                case(name, phase, "attention_varlen (uniform, causal)", lambda: F.attention_varlen(qq, kk, vv, cu, L), 4.0 * n * L * (L + 1) / 2 * (W // 128) * 128,
+                     2.0 * T * (2 * W + 2 * nkv * 128), False)
+            else:
+                S, ctx, bs = s["slots"], s["ctx"], 64
+                per = -(-(ctx + 64) // bs)
+                pages = r(S * per, bs, kr + rot, sc=0.5)
+                table = torch.arange(S * per, device=dev, dtype=torch.int32).view(S, per)
+                cl = torch.full((S,), ctx, device=dev, dtype=torch.int32)
+                qa, sink, uk, uv, oc, gate = r(S, H, kr + rot), r(H), r(H, dim, kr), r(H, vd, kr), r(S, H, kr), torch.randn(S, H, device=dev)
+                seen = min(ctx, w)
+                case(name, phase, "latent_attention_decode", lambda: X.latent_attention_decode(qa, pages, table, cl, kr, w, 192 ** -0.5, sink),
+                     2.0 * S * seen * H * (2 * kr + rot), 2.0 * S * seen * (kr + rot) + 2.0 * S * H * (2 * kr + rot), True)
+                nkv = max(1, W // 512)
+                kc, vc = r(S * per, bs, nkv, 128, sc=0.5), r(S * per, bs, nkv, 128, sc=0.5)
+                qd = r(S, W // 128, 128)
+                case(name, phase, "paged_decode_attention (uniform)", lambda: F.paged_decode_attention(qd, kc, vc, table, cl), 4.0 * S * ctx * W, 4.0 * S * ctx * nkv * 128, False)
+                case(name, phase, "latent_absorb (query into latent space)", lambda: X.latent_absorb(q, uk, pos, cos, sin), 2.0 * S * H * dim * kr,
+                     2.0 * (S * H * (dim + rot) + H * dim * kr + S * H * (kr + rot)), True)
+                case(name, phase, "headwise_linear (values out of latent space + gate)", lambda: X.headwise_linear(oc, uv, False, gate), 2.0 * S * H * vd * kr,
+                     2.0 * (S * H * kr + H * vd * kr + S * H * vd), True)
+                del pages, kc, vc
+            pm, gates, bias, nm = r(T, 2 * Hm * (d + e)), torch.randn(T, 2 * Hm, device=dev), r(Hm), r(Hm * e)
+            io = 2.0 * T * (2 * Hm * (d + e) + Hm * e) + 8.0 * T * Hm
+            if phase == "prefill":
+                C = 64
+                case(name, phase, "mlstm_prefill", lambda: X.mlstm_prefill(pm, gates, bias, bias, 15.0, nm, 1e-6, d, cu), 2.0 * T * Hm * (C / 2 * (d + e) + 2 * d * e), io, True)
+            else:
+                st = torch.zeros(T, Hm * (d * e + d + 1), device=dev)
+                act_ = torch.ones(T, dtype=torch.bool, device=dev)
+                case(name, phase, "mlstm_decode (step, norm, gate)", lambda: X.mlstm_decode(pm, gates, bias, bias, 15.0, nm, 1e-6, d, st, act_), 0, io + 8.0 * T * Hm * d * e, True)
+            torch.cuda.empty_cache()
+    native.check_status()
+
+
+def main(args) -> None:
+    native.load()
+    if args.kernels:
+        run_kernels()
+    else:
+        run_models(args.steps if args.steps > 2 else 5, args.warmup)
