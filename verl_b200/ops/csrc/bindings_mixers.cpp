@@ -355,19 +355,15 @@ Tensor mlstm_prefill(const Tensor& p, const Tensor& gates, const Tensor& ib, con
   const int64_t st_stride = slots.has_value() ? state->stride(0) : 0;
   const char* g = reinterpret_cast<const char*>(p.data_ptr()) + (2 * s.H * s.d + s.H * s.e) * p.element_size();
   if (s.dt == 1) {
-    int fused = 0;
-    const int nseg = vb_mlstm_chunk_segments((int)s.T, (int)B, (int)s.H, (int)s.d, (int)s.e, all_fresh || !slots.has_value(), &fused);
+    const int nseg = vb_mlstm_chunk_segments((int)s.T, (int)B, (int)s.H, (int)s.d, (int)s.e, all_fresh || !slots.has_value());
     if (nseg > 0) {
-      Tensor local, raw;
+      Tensor local;
       if (nseg > 1) local = at::empty({B * (nseg - 1) * s.H * (s.d * s.e + s.d + 2)}, f32);
-      if (!fused) raw = at::empty({s.T, s.H * s.e}, f32);
-      int rc = vb_mlstm_chunk(p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap, st, st_stride, iptr(slots),
-                              iptr(fresh), cu.data_ptr<int>(), (int)B, nseg, nseg > 1 ? local.data_ptr<float>() : nullptr, norm.data_ptr(), (float)eps, out.data_ptr(),
-                              out.stride(0), fused ? nullptr : raw.data_ptr<float>(), (int)s.H, (int)s.d, (int)s.e, cur_stream());
+      const int rc = vb_mlstm_chunk(p.data_ptr(), p.stride(0), gates.data_ptr<float>(), gates.stride(0), ib.data_ptr(), fb.data_ptr(), (float)cap, st, st_stride,
+                                    iptr(slots), iptr(fresh), cu.data_ptr<int>(), (int)B, nseg, nseg > 1 ? local.data_ptr<float>() : nullptr, norm.data_ptr(), (float)eps,
+                                    out.data_ptr(), out.stride(0), (int)s.H, (int)s.d, (int)s.e, cur_stream());
       if (rc >= 0) {
-        verl_count_launches((nseg > 1 ? 2 : 1) + (fused ? 0 : 1));
-        if (rc == 0 && !fused)
-          rc = vb_mlstm_out(s.dt, raw.data_ptr<float>(), g, p.stride(0), norm.data_ptr(), (float)eps, out.data_ptr(), out.stride(0), (int)s.T, (int)s.H, (int)s.e, cur_stream());
+        verl_count_launches(nseg > 1 ? 2 : 1);
         CHECK_RC(rc, "vb_mlstm_chunk");
         return out;
       }

@@ -94,10 +94,10 @@ int vb_mlstm_out(int dtype, const float* o, const void* g, long long ldg, const 
 // latent_prefill_tcgen05.cu
 int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t s);
 // mlstm_chunk.cu
-int vb_mlstm_chunk_segments(int T, int B, int H, int d, int e, int all_fresh, int* fused);
+int vb_mlstm_chunk_segments(int T, int B, int H, int d, int e, int all_fresh);
 int vb_mlstm_chunk(const void* qkvg, long long ldp, const float* gates, long long ldg, const void* ib, const void* fb, float cap, float* state,
                    long long slot_stride, const int* slots, const int* fresh, const int* cu, int B, int nseg, float* local, const void* norm,
-                   float eps, void* out, long long ldo, float* o, int H, int d, int e, cudaStream_t s);
+                   float eps, void* out, long long ldo, int H, int d, int e, cudaStream_t s);
 // headwise_mma.cu
 int vb_headwise(const VbHeadwise* p, cudaStream_t s);
 // latent_decode.cu

@@ -4,18 +4,19 @@
 // recurrence's running maximum is m_t = b_t + M_t and
 //   o_t ~ exp(m_prev - M_t) q_t S_prev + sum_{s <= t} exp(a_s - M_t) (q_t . k_s) v_s
 //   S_C = exp(m_prev - M_C) S_prev + sum_s exp(a_s - M_C) k_s v_s^T
-// so a chunk is three small products. One CTA = (sequence segment, head, up to 256 columns of v); a warp owns 16 columns and
-// keeps their part of S^T in fp32 accumulators for the whole segment. The accumulator layout of S^T is the B-operand layout
+// so a chunk is three small products. One CTA = (sequence segment, head, up to 128 columns of v), the CTAs of a head form a
+// cluster; a warp owns 16 columns and keeps their part of S^T in fp32 accumulators for the whole segment. The accumulator layout of S^T is the B-operand layout
 // of the read-out product, so S never leaves the registers; fp32 values that enter an MMA (S, the weighted scores, v weighted
 // by its gate) are split into two bf16 terms, which keeps 16 mantissa bits: the per-head norm behind the read-out magnifies
-// whatever is rounded where the terms of o cancel. Per-head RMS norm, weight and output gate close the chunk when one
-// CTA covers the head.
+// whatever is rounded where the terms of o cancel. Per-head RMS norm, weight and output gate close the chunk; the
+// CTAs of a head exchange their sums of squares through distributed shared memory.
 //
 // Long sequences are cut into segments: a first launch (FULL = false) computes every segment's own contribution to the state
 // from nothing, the second starts each segment from the fold of those before it. Compiled without fast math.
 #include "mixers.h"
 #include "mixer_common.cuh"
 
+#include <cooperative_groups.h>
 #include <math.h>
 
 namespace vb {
@@ -34,8 +35,7 @@ struct MlstmChunkParams {
   float* local;                      // [B, nseg - 1, H, d e + d + 2]: segment states from nothing
   const bf16* norm;
   float eps;
-  bf16* out; long long ldo;          // fused output, or
-  float* o;                          // raw read-out [T, H, e]
+  bf16* out; long long ldo;
   int H, d, e, nseg, cols;           // cols: columns of v per CTA
 };
 
@@ -62,34 +62,40 @@ __device__ __forceinline__ void mc_split(float x, float y, uint32_t& hi, uint32_
 }
 __device__ __forceinline__ float2 mc_unpack(uint32_t v) { return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u)); }
 
+constexpr int MC_THREADS = 256, MC_COLS = 128, MC_VP = MC_COLS + 8, MC_MAX_BLOCKS = 8;
+
 template <int DP>
 struct McSmem {
-  static constexpr int QP = DP + 8, VP = (DP == 256 ? 128 : 256) + 8;    // row pitches
-  static constexpr int STAGE = (2 * MC_C * QP + MC_C * VP) * 2;
-  static constexpr int OFF_P = 2 * STAGE;
-  static constexpr int OFF_F = OFF_P + 2 * MC_C * MC_PP * 2;   // weighted scores in two bf16 terms
-  // floats: a, M, dec, eneg, w [64 each], den parts [4][64], qn [64], ss [2][16][64], n [DP], scalars [8]
-  static constexpr int FLOATS = 5 * MC_C + 4 * MC_C + MC_C + 2 * 16 * MC_C + DP + 8;
+  static constexpr int QP = DP + 8;
+  static constexpr int STAGE = (2 * MC_C * QP + MC_C * MC_VP) * 2;      // q, k, v of a chunk
+  static constexpr int OFF_G = 2 * STAGE;                               // output gates
+  static constexpr int OFF_P = OFF_G + MC_C * MC_VP * 2;                // weighted scores in two bf16 terms
+  static constexpr int OFF_F = OFF_P + 2 * MC_C * MC_PP * 2;
+  // floats: a, M, dec, eneg, w [64 each], row sums [4][64], q.n [64], squares [8][64], peers [2][8][64], n [DP], n parts [3][DP], scalars [8]
+  static constexpr int FLOATS = 5 * MC_C + 4 * MC_C + MC_C + 8 * MC_C + 2 * MC_MAX_BLOCKS * MC_C + 4 * DP + 8;
   static constexpr int TOTAL = OFF_F + FLOATS * 4;
 };
 
 template <int DP, bool FULL>
-__global__ void __launch_bounds__(DP == 256 ? 256 : 512, 1)
+__global__ void __launch_bounds__(MC_THREADS, 1)
 mlstm_chunk_kernel(const MlstmChunkParams P) {
   using L = McSmem<DP>;
+  namespace cg = cooperative_groups;
   constexpr int KS = DP / 16, NT = DP / 8;
+  constexpr int PARTS = DP >= MC_THREADS ? 1 : (MC_THREADS / DP < 4 ? MC_THREADS / DP : 4);   // token parts of the n update
   extern __shared__ __align__(16) uint8_t smem[];
   float* fl = reinterpret_cast<float*>(smem + L::OFF_F);
   float *sa = fl, *sM = sa + MC_C, *sdec = sM + MC_C, *sneg = sdec + MC_C, *sw = sneg + MC_C, *sden = sw + MC_C, *sqn = sden + 4 * MC_C,
-        *sss = sqn + MC_C, *sn = sss + 2 * 16 * MC_C, *sc = sn + DP;
+        *sss = sqn + MC_C, *speer = sss + 8 * MC_C, *sn = speer + 2 * MC_MAX_BLOCKS * MC_C, *snp = sn + DP, *sc = snp + 3 * DP;
   bf16* sP = reinterpret_cast<bf16*>(smem + L::OFF_P);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nwarps = blockDim.x >> 5;
+  bf16* sG = reinterpret_cast<bf16*>(smem + L::OFF_G);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int b = blockIdx.z / P.nseg, seg = blockIdx.z % P.nseg, h = blockIdx.y, c0 = blockIdx.x * P.cols;
   const int H = P.H, d = P.d, e = P.e;
   const int s0 = P.cu[b], len = P.cu[b + 1] - s0;
   const int seg_len = ((len + P.nseg - 1) / P.nseg + MC_C - 1) / MC_C * MC_C;
   const int t_lo = seg * seg_len, t_hi = min(len, t_lo + seg_len);
-  if (t_lo >= t_hi) return;
+  if (t_lo >= t_hi) return;                          // the same for every CTA of a cluster
   if (!FULL && t_hi == len) return;                  // nothing follows: the segment's own state is not needed
   const int e0 = c0 + warp * 16;                     // first column of this warp
   const bool e_ok = e0 < e && warp * 16 < P.cols;
@@ -105,7 +111,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
   float S[NT][4];
 #pragma unroll
   for (int j = 0; j < NT; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.f;
-  auto each = [&](auto fn) {                         // fn(tile, index, d row, e column) over this thread's valid elements
+  auto each = [&](auto fn) {                         // fn(element, d row, e column) over this thread's valid elements
 #pragma unroll
     for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -115,11 +121,12 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       }
   };
   float m_prev = FULL ? 0.f : -INFINITY, f_total = 0.f;
-  for (int r = tid; r < DP; r += blockDim.x) sn[r] = 0.f;
+  for (int r = tid; r < DP; r += MC_THREADS) sn[r] = 0.f;
+  for (int r = tid; r < 3 * DP; r += MC_THREADS) snp[r] = 0.f;
   if (FULL) {
     if (have && P.fresh != nullptr && P.fresh[b] == 0) {
       each([&](float& v, int dd, int ee) { v = slot_S[static_cast<long long>(dd) * e + ee]; });
-      for (int r = tid; r < d; r += blockDim.x) sn[r] = slot_n[r];
+      for (int r = tid; r < d; r += MC_THREADS) sn[r] = slot_n[r];
       m_prev = *slot_m;
     }
     for (int g = 0; g < seg; ++g) {                  // fold of the segments before this one
@@ -127,50 +134,70 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       const float m_loc = loc[lsize - 2], F = loc[lsize - 1];
       const float m = fmaxf(F + m_prev, m_loc), keep = expf(F + m_prev - m), add = expf(m_loc - m);
       each([&](float& v, int dd, int ee) { v = keep * v + add * loc[static_cast<long long>(dd) * e + ee]; });
-      for (int r = tid; r < d; r += blockDim.x) sn[r] = keep * sn[r] + add * loc[static_cast<long long>(d) * e + r];
+      for (int r = tid; r < d; r += MC_THREADS) sn[r] = keep * sn[r] + add * loc[static_cast<long long>(d) * e + r];
       m_prev = m;
     }
   }
+  float wn[2][2] = {};                               // norm weights of this thread's columns
+  if (FULL && e_ok)
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+        if (e0 + n * 8 + kc + u < e) wn[n][u] = to_f(P.norm[h * e + e0 + n * 8 + kc + u]);
 
   const bf16* base = P.p + static_cast<long long>(s0) * P.ldp;
+  const int vw = min(P.cols, e - c0) / 8;            // 16-byte pieces of a v or g row
+  auto load_v = [&](bf16* dst, int t0, long long off) {
+    for (int i = tid; i < MC_C * (MC_COLS / 8); i += MC_THREADS) {
+      const int r = i / (MC_COLS / 8), c = i % (MC_COLS / 8);
+      const bool ok = t0 + r < t_hi && c < vw;
+      mc_cp16(dst + r * MC_VP + c * 8, ok ? base + static_cast<long long>(t0 + r) * P.ldp + off + c * 8 : base, ok);
+    }
+  };
   auto load = [&](int st, int t0) {
     bf16* q = reinterpret_cast<bf16*>(smem + st * L::STAGE);
     bf16* k = q + MC_C * L::QP;
-    bf16* v = k + MC_C * L::QP;
-    for (int i = tid; i < MC_C * (DP / 8); i += blockDim.x) {
+    for (int i = tid; i < MC_C * (DP / 8); i += MC_THREADS) {
       const int r = i / (DP / 8), c = (i % (DP / 8)) * 8;
       const bool ok = t0 + r < t_hi && c < d;
       const bf16* row = base + static_cast<long long>(t0 + r) * P.ldp;
       if (FULL) mc_cp16(q + r * L::QP + c, ok ? row + h * d + c : base, ok);
       mc_cp16(k + r * L::QP + c, ok ? row + (H + h) * d + c : base, ok);
     }
-    const int vc = (nwarps * 16) / 8;
-    for (int i = tid; i < MC_C * vc; i += blockDim.x) {
-      const int r = i / vc, c = (i % vc) * 8;
-      const bool ok = t0 + r < t_hi && c0 + c < e;
-      mc_cp16(v + r * L::VP + c, ok ? base + static_cast<long long>(t0 + r) * P.ldp + 2 * H * d + static_cast<long long>(h) * e + c0 + c : base, ok);
-    }
+    load_v(k + MC_C * L::QP, t0, 2 * H * d + static_cast<long long>(h) * e + c0);
     asm volatile("cp.async.commit_group;");
   };
   const float ibv = to_f(P.ib[h]), fbv = to_f(P.fb[h]);
   const float qs = 1.f / sqrtf(static_cast<float>(d));
+  float gi[2], gf[2];                                // gate pre-activations of the next chunk (warp 0, two tokens per lane)
+  auto fetch_gates = [&](int t0) {
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int t = t0 + lane * 2 + u;
+      const float* g = P.gates + static_cast<long long>(s0 + t) * P.ldg;
+      gi[u] = t < t_hi ? g[h] : 0.f;
+      gf[u] = t < t_hi ? g[H + h] : 0.f;
+    }
+  };
+  if (warp == 0) fetch_gates(t_lo);
   load(0, t_lo);
+  cg::cluster_group cluster = cg::this_cluster();
+  const int nblk = gridDim.x;
+  if (nblk > 1) cluster.sync();                      // peers run, and have read the stored state, before anything is replaced
+  __syncthreads();
   int st = 0;
   for (int t0 = t_lo; t0 < t_hi; t0 += MC_C, st ^= 1) {
-    // ---- gates of the chunk (warp 0, two neighbouring tokens per lane)
+    // ---- gates of the chunk
     if (warp == 0) {
       float il[2], ff[2];
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
-        const int t = t0 + lane * 2 + u;
-        il[u] = -INFINITY;
-        ff[u] = 0.f;
-        if (t < t_hi) {
-          const float* g = P.gates + static_cast<long long>(s0 + t) * P.ldg;
-          il[u] = P.cap * tanhf((g[h] + ibv) / P.cap);
-          ff[u] = log_sigmoid(P.cap * tanhf((g[H + h] + fbv) / P.cap));
-        }
+        const bool ok = t0 + lane * 2 + u < t_hi;
+        il[u] = ok ? P.cap * tanhf((gi[u] + ibv) / P.cap) : -INFINITY;
+        ff[u] = ok ? log_sigmoid(P.cap * tanhf((gf[u] + fbv) / P.cap)) : 0.f;
       }
+      fetch_gates(t0 + MC_C);
       float run = ff[0] + ff[1];
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
@@ -205,158 +232,158 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
         sc[2] = bC;
       }
     }
+    for (int r = tid; r < DP; r += MC_THREADS) {      // the parts of the last chunk's n update
+#pragma unroll
+      for (int u = 0; u < PARTS - 1; ++u) sn[r] += snp[u * DP + r];
+    }
     asm volatile("cp.async.wait_group 0;");
     __syncthreads();                                  // A: chunk and gates are in shared memory, the other stage is free
-    if (t0 + MC_C < t_hi) load(st ^ 1, t0 + MC_C);
+    const bool more = t0 + MC_C < t_hi;
+    if (FULL) {
+      load_v(sG, t0, 2 * H * d + static_cast<long long>(H + h) * e + c0);
+      asm volatile("cp.async.commit_group;");
+    }
+    if (more) load(st ^ 1, t0 + MC_C);
     const bf16* q = reinterpret_cast<const bf16*>(smem + st * L::STAGE);
     const bf16* k = q + MC_C * L::QP;
-    const bf16* v = k + MC_C * L::QP;
-    const uint32_t uq = mc_smem(q), uk = mc_smem(k), uv = mc_smem(v), uP = mc_smem(sP);
+    const uint32_t uq = mc_smem(q), uk = mc_smem(k), uv = mc_smem(k + MC_C * L::QP), uP = mc_smem(sP);
     const float decC = sc[0], m_next = sc[1];
+    float o[4][2][4] = {};
+    const int par = ((t0 - t_lo) / MC_C) & 1;
     if (FULL) {
-      // ---- weighted scores P = exp(a_s - M_t) q_t . k_s, in 16 x 16 blocks; blocks above the diagonal are zero
-      for (int blk = warp; blk < 16; blk += nwarps) {
-        const int tb = (blk >> 2) * 16, sb = (blk & 3) * 16;
-        float acc[2][4] = {};
-        if (sb <= tb) {
+      // ---- weighted scores P = exp(a_s - M_t) q_t . k_s: a warp owns 16 rows and 32 columns, zero above the diagonal
+      {
+        const int tb = (warp >> 1) * 16;
+        float rs[2][2] = {};
 #pragma unroll
-          for (int kk = 0; kk < KS; ++kk) {
-            uint32_t fa[4], fb[4];
-            mc_ldsm(fa, uq + ((tb + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
-            mc_ldsm(fb, uk + ((sb + (mi >> 1) * 8 + r8) * L::QP + kk * 16 + (mi & 1) * 8) * 2);
-            mc_mma(acc[0], fa, fb[0], fb[1]);
-            mc_mma(acc[1], fa, fb[2], fb[3]);
-          }
-        }
-        float rs[2] = {0.f, 0.f};
+        for (int j2 = 0; j2 < 2; ++j2) {
+          const int sb = ((warp & 1) * 2 + j2) * 16;
+          float acc[2][4] = {};
+          if (sb <= tb) {
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int t = tb + er + half * 8;
-          const float Mt = sM[t];
-#pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            float x[2];
-#pragma unroll
-            for (int u = 0; u < 2; ++u) {
-              const int s = sb + j * 8 + kc + u;
-              x[u] = s <= t ? acc[j][half * 2 + u] * qs * expf(sa[s] - Mt) : 0.f;
-              rs[half] += x[u];
-            }
-            uint32_t hi, lo;
-            mc_split(x[0], x[1], hi, lo);
-            *reinterpret_cast<uint32_t*>(sP + t * MC_PP + sb + j * 8 + kc) = hi;
-            *reinterpret_cast<uint32_t*>(sP + (MC_C + t) * MC_PP + sb + j * 8 + kc) = lo;
-          }
-          rs[half] += __shfl_xor_sync(0xffffffffu, rs[half], 1);
-          rs[half] += __shfl_xor_sync(0xffffffffu, rs[half], 2);
-          if ((lane & 3) == 0) sden[(blk & 3) * MC_C + t] = rs[half];
-        }
-      }
-      // ---- q_t . n_prev
-      for (int t = warp; t < MC_C; t += nwarps) {
-        float x = 0.f;
-        for (int c = lane; c < DP; c += 32) x += to_f(q[t * L::QP + c]) * sn[c];
-        x = warp_sum(x);
-        if (lane == 0) sqn[t] = x * qs;
-      }
-      __syncthreads();                                // B: scores, row sums
-#pragma unroll
-      for (int hf = 0; hf < 2; ++hf) {                // 32 tokens at a time
-        float o[2][2][4] = {};
-        if (e_ok) {
-#pragma unroll
-          for (int kk = 0; kk < KS; ++kk) {           // read-out of the state
-            uint32_t h0, l0, h1, l1, h2, l2, h3, l3;
-            mc_split(S[2 * kk][0], S[2 * kk][1], h0, l0);
-            mc_split(S[2 * kk + 1][0], S[2 * kk + 1][1], h1, l1);
-            mc_split(S[2 * kk][2], S[2 * kk][3], h2, l2);
-            mc_split(S[2 * kk + 1][2], S[2 * kk + 1][3], h3, l3);
-#pragma unroll
-            for (int m = 0; m < 2; ++m) {
-              uint32_t fa[4];
-              mc_ldsm(fa, uq + ((hf * 32 + m * 16 + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
-              mc_mma(o[m][0], fa, h0, h1);
-              mc_mma(o[m][1], fa, h2, h3);
-              mc_mma(o[m][0], fa, l0, l1);
-              mc_mma(o[m][1], fa, l2, l3);
+            for (int kk = 0; kk < KS; ++kk) {
+              uint32_t fa[4], fb[4];
+              mc_ldsm(fa, uq + ((tb + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
+              mc_ldsm(fb, uk + ((sb + (mi >> 1) * 8 + r8) * L::QP + kk * 16 + (mi & 1) * 8) * 2);
+              mc_mma(acc[0], fa, fb[0], fb[1]);
+              mc_mma(acc[1], fa, fb[2], fb[3]);
             }
           }
-#pragma unroll
-          for (int m = 0; m < 2; ++m)
-#pragma unroll
-            for (int half = 0; half < 2; ++half) {
-              const float f = sdec[hf * 32 + m * 16 + half * 8 + er] * qs;
-              o[m][0][half * 2] *= f; o[m][0][half * 2 + 1] *= f;
-              o[m][1][half * 2] *= f; o[m][1][half * 2 + 1] *= f;
-            }
-#pragma unroll
-          for (int kk = 0; kk < 2 + 2 * hf; ++kk) {   // the chunk's own tokens up to this half
-            uint32_t fv[4];
-            mc_ldsm_t(fv, uv + ((kk * 16 + (mi & 1) * 8 + r8) * L::VP + warp * 16 + (mi >> 1) * 8) * 2);
-#pragma unroll
-            for (int m = 0; m < 2; ++m) {
-              uint32_t fa[4];
-              mc_ldsm(fa, uP + ((hf * 32 + m * 16 + (mi & 1) * 8 + r8) * MC_PP + kk * 16 + (mi >> 1) * 8) * 2);
-              mc_mma(o[m][0], fa, fv[0], fv[1]);
-              mc_mma(o[m][1], fa, fv[2], fv[3]);
-              mc_ldsm(fa, uP + ((MC_C + hf * 32 + m * 16 + (mi & 1) * 8 + r8) * MC_PP + kk * 16 + (mi >> 1) * 8) * 2);
-              mc_mma(o[m][0], fa, fv[0], fv[1]);
-              mc_mma(o[m][1], fa, fv[2], fv[3]);
-            }
-          }
-        }
-        // ---- denominator; sum of squares over the head
-#pragma unroll
-        for (int m = 0; m < 2; ++m)
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
-            const int t = hf * 32 + m * 16 + half * 8 + er;
-            const float den = sdec[t] * sqn[t] + ((sden[t] + sden[MC_C + t]) + (sden[2 * MC_C + t] + sden[3 * MC_C + t]));
-            const float inv = 1.f / (fmaxf(fabsf(den), sneg[t]) + 1e-6f);
-            float ss = 0.f;
+            const int t = tb + er + half * 8;
+            const float Mt = sM[t];
 #pragma unroll
-            for (int n = 0; n < 2; ++n)
+            for (int j = 0; j < 2; ++j) {
+              float x[2];
 #pragma unroll
               for (int u = 0; u < 2; ++u) {
-                float& x = o[m][n][half * 2 + u];
-                x *= inv;
-                ss += x * x;
+                const int s = sb + j * 8 + kc + u;
+                x[u] = s <= t ? acc[j][half * 2 + u] * qs * __expf(sa[s] - Mt) : 0.f;
+                rs[j2][half] += x[u];
               }
-            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
-            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-            if ((lane & 3) == 0) sss[(hf * 16 + warp) * MC_C + t] = ss;
+              uint32_t hi, lo;
+              mc_split(x[0], x[1], hi, lo);
+              *reinterpret_cast<uint32_t*>(sP + t * MC_PP + sb + j * 8 + kc) = hi;
+              *reinterpret_cast<uint32_t*>(sP + (MC_C + t) * MC_PP + sb + j * 8 + kc) = lo;
+            }
           }
-        if (P.o == nullptr) __syncthreads();          // C
-        if (e_ok) {
+        }
 #pragma unroll
-          for (int m = 0; m < 2; ++m)
+        for (int half = 0; half < 2; ++half) {
+          float r = rs[0][half] + rs[1][half];
+          r += __shfl_xor_sync(0xffffffffu, r, 1);
+          r += __shfl_xor_sync(0xffffffffu, r, 2);
+          if ((lane & 3) == 0) sden[(warp & 1) * MC_C + tb + er + half * 8] = r;
+        }
+      }
+      // ---- q_t . n_prev: four lanes per token
+      {
+        const int t = tid >> 2;
+        float x = 0.f;
+#pragma unroll 8
+        for (int c = (tid & 3) * 2; c < DP; c += 8) {
+          const float2 qq = mc_unpack(*reinterpret_cast<const uint32_t*>(q + t * L::QP + c));
+          x += qq.x * sn[c] + qq.y * sn[c + 1];
+        }
+        x += __shfl_xor_sync(0xffffffffu, x, 1);
+        x += __shfl_xor_sync(0xffffffffu, x, 2);
+        if ((tid & 3) == 0) sqn[t] = x * qs;
+      }
+      __syncthreads();                                // B: scores, row sums
+      if (e_ok) {
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-              const int t = hf * 32 + m * 16 + half * 8 + er;
-              if (t0 + t >= t_hi) continue;
-              const long long tok = s0 + t0 + t;
-              if (P.o != nullptr) {
+        for (int kk = 0; kk < KS; ++kk) {             // read-out of the state
+          uint32_t h0, l0, h1, l1, h2, l2, h3, l3;
+          mc_split(S[2 * kk][0], S[2 * kk][1], h0, l0);
+          mc_split(S[2 * kk + 1][0], S[2 * kk + 1][1], h1, l1);
+          mc_split(S[2 * kk][2], S[2 * kk][3], h2, l2);
+          mc_split(S[2 * kk + 1][2], S[2 * kk + 1][3], h3, l3);
 #pragma unroll
-                for (int n = 0; n < 2; ++n) {
-                  const int ee = e0 + n * 8 + kc;
-                  if (ee < e) *reinterpret_cast<float2*>(P.o + (tok * H + h) * e + ee) = make_float2(o[m][n][half * 2], o[m][n][half * 2 + 1]);
-                }
-              } else {
-                float ss = 0.f;
-                for (int w = 0; w < nwarps; ++w) ss += sss[(hf * 16 + w) * MC_C + t];
-                const float rs = 1.f / sqrtf(ss / e + P.eps);
+          for (int m = 0; m < 4; ++m) {
+            uint32_t fa[4];
+            mc_ldsm(fa, uq + ((m * 16 + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
+            mc_mma(o[m][0], fa, h0, h1);
+            mc_mma(o[m][1], fa, h2, h3);
+            mc_mma(o[m][0], fa, l0, l1);
+            mc_mma(o[m][1], fa, l2, l3);
+          }
+        }
 #pragma unroll
-                for (int n = 0; n < 2; ++n) {
-                  const int ee = e0 + n * 8 + kc;
-                  if (ee >= e) continue;
-                  const float2 g = mc_unpack(*reinterpret_cast<const uint32_t*>(P.p + tok * P.ldp + 2 * H * d + static_cast<long long>(H + h) * e + ee));
-                  const float2 w = mc_unpack(*reinterpret_cast<const uint32_t*>(P.norm + h * e + ee));
-                  *reinterpret_cast<__nv_bfloat162*>(P.out + tok * P.ldo + h * e + ee) =
-                      __floats2bfloat162_rn(o[m][n][half * 2] * rs * w.x * sigmoid_f(g.x), o[m][n][half * 2 + 1] * rs * w.y * sigmoid_f(g.y));
-                }
-              }
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const float f = sdec[m * 16 + half * 8 + er] * qs;
+            o[m][0][half * 2] *= f; o[m][0][half * 2 + 1] *= f;
+            o[m][1][half * 2] *= f; o[m][1][half * 2 + 1] *= f;
+          }
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {              // the chunk's own tokens
+          uint32_t fv[4];
+          mc_ldsm_t(fv, uv + ((kk * 16 + (mi & 1) * 8 + r8) * MC_VP + warp * 16 + (mi >> 1) * 8) * 2);
+#pragma unroll
+          for (int m = kk; m < 4; ++m)
+#pragma unroll
+            for (int term = 0; term < 2; ++term) {
+              uint32_t fa[4];
+              mc_ldsm(fa, uP + ((term * MC_C + m * 16 + (mi & 1) * 8 + r8) * MC_PP + kk * 16 + (mi >> 1) * 8) * 2);
+              mc_mma(o[m][0], fa, fv[0], fv[1]);
+              mc_mma(o[m][1], fa, fv[2], fv[3]);
             }
         }
+      }
+      // ---- denominator; sum of squares over the head
+#pragma unroll
+      for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int t = m * 16 + half * 8 + er;
+          const float den = sdec[t] * sqn[t] + (sden[t] + sden[MC_C + t]);
+          const float inv = __frcp_rn(fmaxf(fabsf(den), sneg[t]) + 1e-6f);
+          float ss = 0.f;
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+              float& x = o[m][n][half * 2 + u];
+              x *= inv;
+              ss += x * x;
+            }
+          ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+          ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+          if ((lane & 3) == 0) sss[warp * MC_C + t] = ss;
+        }
+      if (more) asm volatile("cp.async.wait_group 1;");
+      else asm volatile("cp.async.wait_group 0;");
+      __syncthreads();                                // C: sums of squares, output gates
+      if (nblk > 1) {
+        if (tid < MC_C) {
+          float ss = 0.f;
+#pragma unroll
+          for (int w = 0; w < 8; ++w) ss += sss[w * MC_C + tid];
+          for (int r = 0; r < nblk; ++r) cluster.map_shared_rank(speer, r)[(par * MC_MAX_BLOCKS + blockIdx.x) * MC_C + tid] = ss;
+        }
+        asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
       }
     }
     // ---- state update: S^T = decC S^T + (w v)^T k
@@ -367,7 +394,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       for (int kk = 0; kk < MC_C / 16; ++kk) {
         uint32_t fv[4], hi[4], lo[4];
         // (w v)^T as A: rows = v columns, k = tokens; registers {e0 s0, e8 s0, e0 s8, e8 s8}
-        mc_ldsm_t(fv, uv + ((kk * 16 + (mi >> 1) * 8 + r8) * L::VP + warp * 16 + (mi & 1) * 8) * 2);
+        mc_ldsm_t(fv, uv + ((kk * 16 + (mi >> 1) * 8 + r8) * MC_VP + warp * 16 + (mi & 1) * 8) * 2);
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int s = kk * 16 + (i >> 1) * 8 + kc;
@@ -385,45 +412,89 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
         }
       }
     }
-    for (int r = tid; r < DP; r += blockDim.x) {
-      float x = decC * sn[r];
+    for (int i = tid; i < DP * PARTS; i += MC_THREADS) {
+      const int r = i % DP, part = i / DP;
+      float x = part == 0 ? decC * sn[r] : 0.f;
 #pragma unroll 8
-      for (int s = 0; s < MC_C; ++s) x += sw[s] * to_f(k[s * L::QP + r]);
-      sn[r] = x;
+      for (int s = part * (MC_C / PARTS); s < (part + 1) * (MC_C / PARTS); ++s) x += sw[s] * to_f(k[s * L::QP + r]);
+      if (part == 0) sn[r] = x;
+      else snp[(part - 1) * DP + r] = x;
+    }
+    if (FULL) {
+      // ---- norm over the head, weight, output gate
+      if (nblk > 1) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+      if (e_ok) {
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int t = m * 16 + half * 8 + er;
+            float ss = 0.f;
+            if (nblk > 1) {
+              for (int r = 0; r < nblk; ++r) ss += speer[(par * MC_MAX_BLOCKS + r) * MC_C + t];
+            } else {
+#pragma unroll
+              for (int w = 0; w < 8; ++w) ss += sss[w * MC_C + t];
+            }
+            const float rs = rsqrtf(ss / e + P.eps);
+            bf16* dst = P.out + static_cast<long long>(s0 + t0 + t) * P.ldo + h * e + e0 + kc;
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+              const float2 g = mc_unpack(*reinterpret_cast<const uint32_t*>(sG + t * MC_VP + warp * 16 + n * 8 + kc));
+              const float y0 = __fdividef(o[m][n][half * 2] * rs * wn[n][0], 1.f + __expf(-g.x));
+              const float y1 = __fdividef(o[m][n][half * 2 + 1] * rs * wn[n][1], 1.f + __expf(-g.y));
+              if (t0 + t < t_hi && e0 + n * 8 + kc < e) *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) = __floats2bfloat162_rn(y0, y1);
+            }
+          }
+      }
     }
     m_prev = m_next;
     f_total += sc[2];
-    __syncthreads();                                  // D: gates and n may be replaced
+    __syncthreads();                                  // D: gates, n and the chunk may be replaced
   }
+  for (int r = tid; r < DP; r += MC_THREADS)
+#pragma unroll
+    for (int u = 0; u < PARTS - 1; ++u) sn[r] += snp[u * DP + r];
   // ---- final state of the sequence, or this segment's own state
   if (!FULL) {
     float* loc = P.local + ((static_cast<long long>(b) * (P.nseg - 1) + seg) * H + h) * lsize;
     each([&](float& v, int dd, int ee) { loc[static_cast<long long>(dd) * e + ee] = v; });
     if (blockIdx.x == 0) {
-      for (int r = tid; r < d; r += blockDim.x) loc[static_cast<long long>(d) * e + r] = sn[r];
+      for (int r = tid; r < d; r += MC_THREADS) loc[static_cast<long long>(d) * e + r] = sn[r];
       if (tid == 0) { loc[lsize - 2] = m_prev; loc[lsize - 1] = f_total; }
     }
   } else if (have && t_hi == len) {
     each([&](float& v, int dd, int ee) { slot_S[static_cast<long long>(dd) * e + ee] = v; });
     if (blockIdx.x == 0) {
-      for (int r = tid; r < d; r += blockDim.x) slot_n[r] = sn[r];
+      for (int r = tid; r < d; r += MC_THREADS) slot_n[r] = sn[r];
       if (tid == 0) *slot_m = m_prev;
     }
   }
 }
 
 static int mc_dp(int d) { return d <= 64 ? 64 : (d <= 128 ? 128 : 256); }
-static int mc_blocks(int d, int e) { const int mx = mc_dp(d) == 256 ? 128 : 256; return (e + mx - 1) / mx; }
 
 template <int DP>
-static int mc_launch(const MlstmChunkParams& p, int B, int blocks, int threads, cudaStream_t s) {
-  cudaError_t e = cudaFuncSetAttribute(mlstm_chunk_kernel<DP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, McSmem<DP>::TOTAL);
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(mlstm_chunk_kernel<DP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, McSmem<DP>::TOTAL);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  const dim3 grid(blocks, p.H, B * p.nseg);
-  if (p.nseg > 1) mlstm_chunk_kernel<DP, false><<<grid, threads, McSmem<DP>::TOTAL, s>>>(p);
-  mlstm_chunk_kernel<DP, true><<<grid, threads, McSmem<DP>::TOTAL, s>>>(p);
-  return static_cast<int>(cudaGetLastError());
+static int mc_launch(const MlstmChunkParams& p, int B, int blocks, cudaStream_t s) {
+  auto go = [&](auto kern) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, McSmem<DP>::TOTAL);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3(blocks, p.H, B * p.nseg);
+    cfg.blockDim = dim3(MC_THREADS);
+    cfg.dynamicSmemBytes = McSmem<DP>::TOTAL;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = blocks;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    return static_cast<int>(cudaLaunchKernelEx(&cfg, kern, p));
+  };
+  int rc = p.nseg > 1 ? go(mlstm_chunk_kernel<DP, false>) : 0;
+  if (rc == 0) rc = go(mlstm_chunk_kernel<DP, true>);
+  return rc;
 }
 
 }  // namespace vb
@@ -432,11 +503,9 @@ using namespace vb;
 
 // Segments a sequence is cut into (1 = none; the workspace then needs B * (nseg - 1) * H * (d e + d + 2) floats), or 0 when the
 // sizes are not served. all_fresh: every sequence starts from zero.
-extern "C" int vb_mlstm_chunk_segments(int T, int B, int H, int d, int e, int all_fresh, int* fused) {
-  if (d % 8 || e % 8 || d > 256 || d < 8 || e < 8) return 0;
-  const int blocks = mc_blocks(d, e);
-  if (blocks > 1 && !all_fresh) return 0;   // column blocks would read n and m while the first one replaces them
-  *fused = blocks == 1;
+extern "C" int vb_mlstm_chunk_segments(int T, int B, int H, int d, int e, int all_fresh) {
+  const int blocks = (e + MC_COLS - 1) / MC_COLS;
+  if (d % 8 || e % 8 || d > 256 || d < 8 || e < 8 || blocks > MC_MAX_BLOCKS || B > 65535 || H > 65535) return 0;
   if (!all_fresh) return 1;
   int s = 148 / (B * H * blocks);
   const int by_len = T / B / (4 * MC_C);
@@ -447,20 +516,20 @@ extern "C" int vb_mlstm_chunk_segments(int T, int B, int H, int d, int e, int al
 
 extern "C" int vb_mlstm_chunk(const void* qkvg, long long ldp, const float* gates, long long ldg, const void* ib, const void* fb, float cap,
                               float* state, long long slot_stride, const int* slots, const int* fresh, const int* cu, int B, int nseg, float* local,
-                              const void* norm, float eps, void* out, long long ldo, float* o, int H, int d, int e, cudaStream_t s) {
-  if (ldp % 8 || (reinterpret_cast<uintptr_t>(qkvg) & 15) || (ldo % 2) || (reinterpret_cast<uintptr_t>(norm) & 3) || static_cast<long long>(B) * nseg > 65535 || H > 65535) return -1;
+                              const void* norm, float eps, void* out, long long ldo, int H, int d, int e, cudaStream_t s) {
+  if (ldp % 8 || (reinterpret_cast<uintptr_t>(qkvg) & 15) || (ldo % 2) || (reinterpret_cast<uintptr_t>(out) & 3)) return -1;
   MlstmChunkParams p{};
   p.p = reinterpret_cast<const bf16*>(qkvg); p.ldp = ldp; p.gates = gates; p.ldg = ldg;
   p.ib = reinterpret_cast<const bf16*>(ib); p.fb = reinterpret_cast<const bf16*>(fb); p.cap = cap;
   p.state = state; p.slot_stride = slot_stride; p.slots = slots; p.fresh = fresh; p.cu = cu; p.local = local;
-  p.norm = reinterpret_cast<const bf16*>(norm); p.eps = eps; p.out = reinterpret_cast<bf16*>(out); p.ldo = ldo; p.o = o;
+  p.norm = reinterpret_cast<const bf16*>(norm); p.eps = eps; p.out = reinterpret_cast<bf16*>(out); p.ldo = ldo;
   p.H = H; p.d = d; p.e = e; p.nseg = nseg;
-  const int blocks = mc_blocks(d, e);
+  int blocks = (e + MC_COLS - 1) / MC_COLS;
   p.cols = ((e + blocks - 1) / blocks + 15) / 16 * 16;
-  const int warps = p.cols / 16 < 4 ? 4 : p.cols / 16;
+  blocks = (e + p.cols - 1) / p.cols;
   switch (mc_dp(d)) {
-    case 64: return mc_launch<64>(p, B, blocks, warps * 32, s);
-    case 128: return mc_launch<128>(p, B, blocks, warps * 32, s);
-    default: return mc_launch<256>(p, B, blocks, warps * 32, s);
+    case 64: return mc_launch<64>(p, B, blocks, s);
+    case 128: return mc_launch<128>(p, B, blocks, s);
+    default: return mc_launch<256>(p, B, blocks, s);
   }
 }
