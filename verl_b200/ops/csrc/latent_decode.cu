@@ -1,8 +1,8 @@
-// Decode-step attention in the latent space: one CTA = (sequence, group of 16 heads [, key split]).
+// Decode-step attention in the latent space: one CTA = (sequence, one or two groups of 16 heads [, key split]).
 //
 // All heads read the same cached row, [latent (value and first key part) | rotated key part], so a row is streamed once per
-// head group: TMA brings 32-token tiles of the pages (128B swizzle, 64 columns per panel) into a shared-memory ring, and the
-// 16 heads are the M dimension of m16n8k16 MMAs (a 16-row sliver of work per byte: the kernel is bound by the stream, not by
+// CTA: a producer warp brings 32-token tiles of the pages by TMA (128B swizzle, 64 columns per panel) into a shared-memory ring, and the
+// 16 heads of a group of four warps are the M dimension of m16n8k16 MMAs (a 16-row sliver of work per byte: the kernel is bound by the stream, not by
 // the tensor pipe, as in paged_decode_tma.cu). Per tile
 //   scores   warp w takes tokens [8w, 8w + 8) over the whole row width, masked to the window
 //   softmax  running maximum shared by the four warps; it starts at the sink, which adds one unit of weight and no value
@@ -16,7 +16,7 @@
 
 namespace vb {
 
-constexpr int LD_TOK = 32, LD_THREADS = 128, LD_HEADS = 16, LD_MAX_STAGES = 4;
+constexpr int LD_TOK = 32, LD_HEADS = 16, LD_MAX_STAGES = 4;
 
 struct LatentDecodeParams {
   const __nv_bfloat16* q;   // [S, H, width]
@@ -48,24 +48,28 @@ __device__ __forceinline__ void ld_mma(float (&d)[4], const uint32_t (&a)[4], ui
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// NV: 8-column value blocks per warp (rank <= 32 NV)
-template <int NV>
-__global__ void __launch_bounds__(LD_THREADS, 2)
+// NV: 8-column value blocks per warp (rank <= 32 NV); NG: groups of 16 heads per CTA
+template <int NV, int NG>
+__global__ void __launch_bounds__(128 * NG + 32, NG == 1 ? 2 : 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int stage_bytes = p.panels * (LD_TOK * 128);
   const int qpitch = p.panels * 128 + 16;                   // bytes of one query row (shifted banks per head)
   uint8_t* sQ = smem + p.stages * stage_bytes;
-  uint8_t* sP = sQ + LD_HEADS * qpitch;                      // [16][40] bf16
-  float* sMax = reinterpret_cast<float*>(sP + LD_HEADS * 80);  // [4][16]
+  const int group = NG == 1 ? 0 : min(static_cast<int>(threadIdx.x >> 7), NG - 1);
+  uint8_t* sP = sQ + NG * LD_HEADS * qpitch + group * (LD_HEADS * 80);  // [16][40] bf16
+  float* sMax = reinterpret_cast<float*>(sQ + NG * LD_HEADS * (qpitch + 80)) + group * 128;  // [4][16]
   float* sSum = sMax + 64;                                   // [4][16]
-  uint64_t* full = reinterpret_cast<uint64_t*>(sSum + 64);   // [stages]
+  uint64_t* full = reinterpret_cast<uint64_t*>(sQ + NG * (LD_HEADS * (qpitch + 80) + 512));  // [stages]
+  uint64_t* empty = full + LD_MAX_STAGES;
 
-  const int b = blockIdx.x, h0 = blockIdx.y * LD_HEADS, split = blockIdx.z;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = blockIdx.x, h0 = (blockIdx.y * NG + group) * LD_HEADS, split = blockIdx.z;
+  const int wall = threadIdx.x >> 5, warp = wall & 3, lane = threadIdx.x & 31;
+  const bool producer = wall == 4 * NG;
+  sQ += group * LD_HEADS * qpitch;
   const int len = min(p.ctx_len[b], p.max_blocks * p.block_size);
-  const int nheads = min(LD_HEADS, p.H - h0);
+  const int nheads = max(0, min(LD_HEADS, p.H - h0));
   const int first = (p.window > 0 && len > p.window) ? len - p.window : 0;
   const int tile_a = first / LD_TOK, tile_b = (len + LD_TOK - 1) / LD_TOK;
   const int per = (max(0, tile_b - tile_a) + p.nsplit - 1) / p.nsplit;
@@ -74,10 +78,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
 
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&tm);
-    for (int s = 0; s < p.stages; ++s) mbar_init(&full[s], 1);
+    for (int s = 0; s < p.stages; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 4 * NG);
+    }
     mbar_fence_init();
   }
-  for (int i = threadIdx.x; i < LD_HEADS * p.panels * 8; i += LD_THREADS) {
+  for (int i = threadIdx.x & 127; i < LD_HEADS * p.panels * 8 && !producer; i += 128) {
     const int g = i / (p.panels * 8), c = i % (p.panels * 8);
     uint4 v = make_uint4(0, 0, 0, 0);
     if (g < nheads && c * 8 < p.width) v = *reinterpret_cast<const uint4*>(p.q + b * p.ldq + static_cast<long long>(h0 + g) * p.hq + c * 8);
@@ -85,19 +92,27 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
   }
   __syncthreads();
 
-  auto issue = [&](int i) {  // tile i of this CTA into stage i % stages (thread 0)
-    const int s = i % p.stages, tok = (t0 + i) * LD_TOK;
-    uint8_t* dst = smem + s * stage_bytes;
-    mbar_expect_tx(&full[s], static_cast<uint32_t>(stage_bytes));
-    for (int r = 0; r < LD_TOK; r += p.box_rows) {
-      // rows past the context re-read its last page: they are masked below
-      const int at = min(tok + r, (len - 1) / p.box_rows * p.box_rows);
-      const int blk = max(0, min(bt[at / p.block_size], static_cast<int>(p.num_blocks) - 1));
-      for (int c = 0; c < p.panels; ++c) tma_load_3d(dst + c * (LD_TOK * 128) + r * 128, &tm, &full[s], c * 64, at % p.block_size, blk);
+  if (producer) {
+    if (lane == 0) {
+      for (int i = 0; i < n; ++i) {
+        const int s = i % p.stages, tok = (t0 + i) * LD_TOK;
+        if (i >= p.stages && !mbar_wait(&empty[s], ((i / p.stages) & 1) ^ 1)) {
+          atomicExch(p.status, 2);
+          break;
+        }
+        uint8_t* dst = smem + s * stage_bytes;
+        mbar_expect_tx(&full[s], static_cast<uint32_t>(stage_bytes));
+        for (int r = 0; r < LD_TOK; r += p.box_rows) {
+          // rows past the context re-read its last page: they are masked below
+          const int at = min(tok + r, (len - 1) / p.box_rows * p.box_rows);
+          const int blk = max(0, min(bt[at / p.block_size], static_cast<int>(p.num_blocks) - 1));
+          for (int c = 0; c < p.panels; ++c) tma_load_3d(dst + c * (LD_TOK * 128) + r * 128, &tm, &full[s], c * 64, at % p.block_size, blk);
+        }
+      }
     }
-  };
-  if (threadIdx.x == 0)
-    for (int i = 0; i < min(n, p.stages - 1); ++i) issue(i);
+    return;   // the consumers wait for every copy before they leave
+  }
+  auto sync_group = [&]() { asm volatile("bar.sync %0, 128;" ::"r"(1 + group) : "memory"); };
 
   float m_run[2], l_run[2];
 #pragma unroll
@@ -115,8 +130,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
   bool ok = true;
   for (int i = 0; i < n; ++i) {
     const int s = i % p.stages;
-    if (i > 0) __syncthreads();            // every warp is done with the tile before: its stage is free
-    if (threadIdx.x == 0 && i + p.stages - 1 < n) issue(i + p.stages - 1);
     // a wait that runs out is recorded; the loop goes on so that every thread meets the same barriers
     if (ok && !mbar_wait(&full[s], (i / p.stages) & 1)) ok = false;
     const uint32_t kb = smem_u32(smem + s * stage_bytes);
@@ -150,7 +163,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
       if ((lane & 3) == 0) sMax[warp * 16 + (lane >> 2) + 8 * h] = mx;
     }
-    __syncthreads();
+    sync_group();
     float alpha[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -163,7 +176,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
       m_run[h] = mn;
       *reinterpret_cast<uint32_t*>(sP + hd * 80 + (warp * 8 + (lane & 3) * 2) * 2) = pack_bf16x2(e0, e1);
     }
-    __syncthreads();
+    sync_group();
     // ---- values: this warp's columns over the 32 tokens
     uint32_t pa[2][4];
 #pragma unroll
@@ -189,6 +202,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
         ld_mma(o[2 * j2 + 1], pa[k], vb[2], vb[3]);
       }
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[s]);
   }
   if (!ok) atomicExch(p.status, 1);
 
@@ -200,7 +215,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
     l += __shfl_xor_sync(0xffffffffu, l, 2);
     if ((lane & 3) == 0) sSum[warp * 16 + (lane >> 2) + 8 * h] = l;
   }
-  __syncthreads();
+  sync_group();
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int hd = (lane >> 2) + 8 * h;
@@ -239,13 +254,11 @@ __global__ void latent_decode_merge_kernel(const float* __restrict__ po, const f
   }
 }
 
-static int latent_decode_stages(int panels) {
-  const int fixed = LD_HEADS * (panels * 128 + 16) + LD_HEADS * 80 + 128 * 4 + 64 + 1024;
-  int s = (113 * 1024 - fixed) / (panels * LD_TOK * 128);     // two CTAs per SM
+static int latent_decode_groups(int H) { return H > LD_HEADS ? 2 : 1; }
+static int latent_decode_fixed(int panels, int ng) { return ng * (LD_HEADS * (panels * 128 + 16 + 80) + 512) + 2 * LD_MAX_STAGES * 8 + 1024; }
+static int latent_decode_stages(int panels, int ng) {
+  const int s = ((ng == 1 ? 113 * 1024 : 227 * 1024) - latent_decode_fixed(panels, ng)) / (panels * LD_TOK * 128);  // two CTAs per SM / one
   return s < 2 ? 0 : (s > LD_MAX_STAGES ? LD_MAX_STAGES : s);
-}
-static int latent_decode_smem(int panels, int stages) {
-  return stages * panels * LD_TOK * 128 + LD_HEADS * (panels * 128 + 16) + LD_HEADS * 80 + 128 * 4 + 64 + 1024;
 }
 
 }  // namespace vb
@@ -255,9 +268,9 @@ using namespace vb;
 // Key splits for S sequences and H heads (0: the sizes are not served). max_keys: most keys a sequence can see.
 extern "C" int vb_latent_decode_splits(int S, int H, int rank, int width, int block_size, int max_keys) {
   const int panels = (width + 63) / 64;
-  if (rank > 512 || rank % 8 || width % 8 || rank > width || block_size % 16 || latent_decode_stages(panels) == 0) return 0;
-  const int groups = S * ((H + LD_HEADS - 1) / LD_HEADS), tiles = (max_keys + LD_TOK - 1) / LD_TOK;
-  int s = (2 * num_sms() + groups - 1) / groups;
+  if (rank > 512 || rank % 8 || width % 8 || rank > width || block_size % 16 || latent_decode_stages(panels, latent_decode_groups(H)) == 0) return 0;
+  const int ng = latent_decode_groups(H), groups = S * ((H + ng * LD_HEADS - 1) / (ng * LD_HEADS)), tiles = (max_keys + LD_TOK - 1) / LD_TOK;
+  int s = ((ng == 1 ? 2 : 1) * num_sms() + groups - 1) / groups;
   if (s > tiles / 4) s = tiles / 4;
   return s < 1 ? 1 : (s > 16 ? 16 : s);
 }
@@ -279,16 +292,19 @@ extern "C" int vb_latent_decode(const VbLatentAttn* a, long long num_blocks, int
   p.ctx_len = a->ctx_len; p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink);
   p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.part_o = part_o; p.part_ml = part_ml;
   p.H = a->H; p.width = width; p.rank = a->dv; p.panels = panels; p.window = a->window; p.nsplit = nsplit;
-  p.stages = latent_decode_stages(panels); p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;
-  const int smem = latent_decode_smem(panels, p.stages);
-  const dim3 grid(a->B, (a->H + LD_HEADS - 1) / LD_HEADS, nsplit);
+  const int ng = latent_decode_groups(a->H);
+  p.stages = latent_decode_stages(panels, ng); p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;
+  const int smem = latent_decode_fixed(panels, ng) + p.stages * panels * LD_TOK * 128;
+  const dim3 grid(a->B, (a->H + ng * LD_HEADS - 1) / (ng * LD_HEADS), nsplit);
   auto go = [&](auto kern) {
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 113 * 1024);
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
-    kern<<<grid, LD_THREADS, smem, stream>>>(tm, p);
+    kern<<<grid, 128 * ng + 32, smem, stream>>>(tm, p);
     return static_cast<int>(cudaGetLastError());
   };
-  int rc = a->dv <= 128 ? go(latent_decode_kernel<4>) : a->dv <= 256 ? go(latent_decode_kernel<8>) : go(latent_decode_kernel<16>);
+  int rc;
+  if (ng == 1) rc = a->dv <= 128 ? go(latent_decode_kernel<4, 1>) : a->dv <= 256 ? go(latent_decode_kernel<8, 1>) : go(latent_decode_kernel<16, 1>);
+  else rc = a->dv <= 128 ? go(latent_decode_kernel<4, 2>) : a->dv <= 256 ? go(latent_decode_kernel<8, 2>) : go(latent_decode_kernel<16, 2>);
   if (rc == 0 && nsplit > 1) {
     latent_decode_merge_kernel<<<a->B * a->H, 128, 0, stream>>>(part_o, part_ml, a->ctx_len, p.out, a->H, nsplit, p.rank);
     rc = static_cast<int>(cudaGetLastError());

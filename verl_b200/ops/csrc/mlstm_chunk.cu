@@ -169,7 +169,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
     asm volatile("cp.async.commit_group;");
   };
   const float ibv = to_f(P.ib[h]), fbv = to_f(P.fb[h]);
-  const float qs = 1.f / sqrtf(static_cast<float>(d));
+  const float qs = 1.f / sqrtf(static_cast<float>(d)), inv_e = 1.f / e;
   float gi[2], gf[2];                                // gate pre-activations of the next chunk (warp 0, two tokens per lane)
   auto fetch_gates = [&](int t0) {
 #pragma unroll
@@ -359,7 +359,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
         for (int half = 0; half < 2; ++half) {
           const int t = m * 16 + half * 8 + er;
           const float den = sdec[t] * sqn[t] + (sden[t] + sden[MC_C + t]);
-          const float inv = __frcp_rn(fmaxf(fabsf(den), sneg[t]) + 1e-6f);
+          const float inv = __fdividef(1.f, fmaxf(fabsf(den), sneg[t]) + 1e-6f);
           float ss = 0.f;
 #pragma unroll
           for (int n = 0; n < 2; ++n)
@@ -436,7 +436,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
 #pragma unroll
               for (int w = 0; w < 8; ++w) ss += sss[w * MC_C + t];
             }
-            const float rs = rsqrtf(ss / e + P.eps);
+            const float rs = rsqrtf(ss * inv_e + P.eps);
             bf16* dst = P.out + static_cast<long long>(s0 + t0 + t) * P.ldo + h * e + e0 + kc;
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
