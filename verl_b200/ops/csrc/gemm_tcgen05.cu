@@ -148,6 +148,8 @@ struct GemmSmem {
   static constexpr int B_BYTES = BN * BK * 2;
   static constexpr int RING = STAGES * (A_BYTES + B_BYTES);
   static constexpr int TOTAL = RING + 256 + 1024;  // barriers + alignment slack
+  static constexpr int STAGE_LD = 36;              // EPI_MIXER: row pitch (floats) of a warp's 32 x 32 transposition tile
+  static constexpr int TOTAL_MIXER = TOTAL + 4 * 32 * STAGE_LD * 4;
 };
 
 // Pass B of the all-reduce epilogue for one warp's slab (32 rows x BN columns): sum the bf16 partials of all ranks in rank
@@ -472,7 +474,22 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
     uint32_t acc_phase = 0;
     bool ok = true;
     float mix_alpha = 0.f;
-    if constexpr (EPI == EPI_MIXER) mix_alpha = epi_alpha(p.mix);
+    // residual stream of the 32 x 32 block at (row0, col): lanes sweep the columns, four rows per round, so that reads and
+    // writes are whole 128-byte lines
+    float4 mix_x[8];
+    float* mix_tile = nullptr;
+    const bool mix_resid = EPI == EPI_MIXER && p.mix.mode == VB_EPI_RESID;
+    auto mix_fetch = [&](int row0, int col) {
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        const int rr = row0 + u * 4 + (lane >> 3), cc = col + (lane & 7) * 4;
+        if (rr < p.M && cc < p.N) mix_x[u] = *reinterpret_cast<const float4*>(p.mix.X + static_cast<long long>(rr) * p.mix.ldx + cc);
+      }
+    };
+    if constexpr (EPI == EPI_MIXER) {
+      mix_alpha = epi_alpha(p.mix);
+      mix_tile = reinterpret_cast<float*>(smem + GemmSmem<BN, STAGES>::RING + 256) + q * 32 * GemmSmem<BN, STAGES>::STAGE_LD;
+    }
     for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x) {
       int m0, n0, kb0_, kb1_, b_off_;
       long long d_off;
@@ -504,6 +521,9 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
         }
       }
       constexpr float LOG2E = 1.4426950408889634f;
+      if constexpr (EPI == EPI_MIXER) {
+        if (mix_resid) mix_fetch(m0 + q * 32, n0);
+      }
 #pragma unroll 1
       for (int c = 0; c < BN / 32; ++c) {
         const int col0 = n0 + c * 32;
@@ -602,7 +622,44 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
             }
           }
         } else if constexpr (EPI == EPI_MIXER) {
-          if (row_ok) {
+          if (mix_resid) {
+            constexpr int LD = GemmSmem<BN, STAGES>::STAGE_LD;
+#pragma unroll
+            for (int j = 0; j < 32; j += 4)
+              *reinterpret_cast<uint4*>(mix_tile + lane * LD + j) = make_uint4(r[j], r[j + 1], r[j + 2], r[j + 3]);
+            __syncwarp();
+            float4 xs[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u) xs[u] = mix_x[u];
+            if (col0 + 32 < p.N && c + 1 < BN / 32) mix_fetch(m0 + q * 32, col0 + 32);
+            const int cc = col0 + (lane & 7) * 4;
+            if (cc < p.N) {
+              float w4[4], b4[4];
+              if (p.mix.D != nullptr) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  w4[i] = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.mix.nw)[cc + i]);
+                  b4[i] = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.mix.nb)[cc + i]);
+                }
+              }
+#pragma unroll
+              for (int u = 0; u < 8; ++u) {
+                const int rl = u * 4 + (lane >> 3), rr = m0 + q * 32 + rl;
+                if (rr < p.M) {
+                  float4 a = *reinterpret_cast<const float4*>(mix_tile + rl * LD + (lane & 7) * 4);
+                  a.x += xs[u].x; a.y += xs[u].y; a.z += xs[u].z; a.w += xs[u].w;
+                  *reinterpret_cast<float4*>(p.mix.X + static_cast<long long>(rr) * p.mix.ldx + cc) = a;
+                  if (p.mix.D != nullptr) {
+                    const float y0 = tanh_full(mix_alpha * a.x) * w4[0] + b4[0], y1 = tanh_full(mix_alpha * a.y) * w4[1] + b4[1];
+                    const float y2 = tanh_full(mix_alpha * a.z) * w4[2] + b4[2], y3 = tanh_full(mix_alpha * a.w) * w4[3] + b4[3];
+                    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.mix.D) + static_cast<long long>(rr) * p.mix.ldd + cc) =
+                        make_uint2(pack_bf16x2(y0, y1), pack_bf16x2(y2, y3));
+                  }
+                }
+              }
+            }
+            __syncwarp();
+          } else if (row_ok) {
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
               if (j < ncols) {
@@ -851,7 +908,7 @@ template <int BN, bool A_MN, bool B_MN, int STAGES, int EPI = EPI_STORE>
 static cudaError_t launch_variant(const CUtensorMap& ta, const CUtensorMap& tb, const GemmParams& p, int sms,
                                   cudaStream_t stream) {
   auto kern = gemm_bf16_kernel<BN, A_MN, B_MN, STAGES, EPI>;
-  constexpr int smem = GemmSmem<BN, STAGES>::TOTAL;
+  constexpr int smem = EPI == EPI_MIXER ? GemmSmem<BN, STAGES>::TOTAL_MIXER : GemmSmem<BN, STAGES>::TOTAL;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
