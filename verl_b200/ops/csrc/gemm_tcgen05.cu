@@ -637,9 +637,10 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
               float w4[4], b4[4];
               if (p.mix.D != nullptr) {
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                  w4[i] = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.mix.nw)[cc + i]);
-                  b4[i] = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.mix.nb)[cc + i]);
+                for (int i = 0; i < 2; ++i) {
+                  const float2 a = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(p.mix.nw)[cc / 2 + i]);
+                  const float2 b = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(p.mix.nb)[cc / 2 + i]);
+                  w4[2 * i] = a.x; w4[2 * i + 1] = a.y; b4[2 * i] = b.x; b4[2 * i + 1] = b.y;
                 }
               }
 #pragma unroll

@@ -7,15 +7,13 @@
 
 namespace vb {
 
-// tanh that keeps fp32 accuracy in files compiled with fast math: Maclaurin series near zero, exponential form elsewhere.
+// tanh with fp32 accuracy in files compiled with fast math, without branches: the exponential form, and the first terms of
+// the Maclaurin series near zero, where the former cancels.
 __device__ __forceinline__ float tanh_full(float x) {
-  const float ax = fabsf(x);
-  if (ax < 0.25f) {
-    const float s = x * x;
-    return x * (1.f + s * (-1.f / 3.f + s * (2.f / 15.f + s * (-17.f / 315.f + s * (62.f / 2835.f)))));
-  }
-  const float t = 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(ax, 20.f)));
-  return copysignf(t, x);
+  const float ax = fabsf(x), s = x * x;
+  const float small = x * (1.f + s * (-1.f / 3.f + s * (2.f / 15.f)));
+  const float large = copysignf(1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(ax, 20.f))), x);
+  return ax < 0.1f ? small : large;
 }
 __device__ __forceinline__ float gelu_erf_full(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
@@ -103,7 +101,7 @@ inline bool epi_aligned(const VbEpiArgs& e, int nv) {
   const bool f32 = e.mode == VB_EPI_STORE_F32;
   if (e.D != nullptr && ((e.ldd % (f32 ? 4 : nv)) || bad(e.D, f32 ? 16 : 2 * nv))) return false;
   if (e.mode == VB_EPI_SPLIT && ((e.n0 % 8) || (e.ldd2 % 4) || bad(e.D2, 16))) return false;
-  if (e.mode == VB_EPI_RESID && ((e.ldx % 4) || bad(e.X, 16))) return false;
+  if (e.mode == VB_EPI_RESID && ((e.ldx % 4) || bad(e.X, 16) || (e.D != nullptr && (bad(e.nw, 4) || bad(e.nb, 4))))) return false;
   return true;
 }
 
