@@ -5,7 +5,7 @@
 //   o_t ~ exp(m_prev - M_t) q_t S_prev + sum_{s <= t} exp(a_s - M_t) (q_t . k_s) v_s
 //   S_C = exp(m_prev - M_C) S_prev + sum_s exp(a_s - M_C) k_s v_s^T
 // so a chunk is three small products. One CTA = (sequence segment, head, up to 128 columns of v), the CTAs of a head form a
-// cluster; a warp owns 16 columns and keeps their part of S^T in fp32 accumulators for the whole segment. The accumulator layout of S^T is the B-operand layout
+// cluster; a pair of warps owns 16 columns and keeps their part of S^T in fp32 accumulators for the whole segment. The accumulator layout of S^T is the B-operand layout
 // of the read-out product, so S never leaves the registers; fp32 values that enter an MMA (S, the weighted scores, v weighted
 // by its gate) are split into two bf16 terms, which keeps 16 mantissa bits: the per-head norm behind the read-out magnifies
 // whatever is rounded where the terms of o cancel. Per-head RMS norm, weight and output gate close the chunk; the
@@ -62,15 +62,17 @@ __device__ __forceinline__ void mc_split(float x, float y, uint32_t& hi, uint32_
 }
 __device__ __forceinline__ float2 mc_unpack(uint32_t v) { return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u)); }
 
-constexpr int MC_THREADS = 256, MC_COLS = 128, MC_VP = MC_COLS + 8, MC_MAX_BLOCKS = 8;
+constexpr int MC_THREADS = 512, MC_COLS = 128, MC_VP = MC_COLS + 8, MC_MAX_BLOCKS = 8;
 
 template <int DP>
 struct McSmem {
   static constexpr int QP = DP + 8;
   static constexpr int STAGE = (2 * MC_C * QP + MC_C * MC_VP) * 2;      // q, k, v of a chunk
-  static constexpr int OFF_G = 2 * STAGE;                               // output gates
+  static constexpr int BUFS = DP == 256 ? 1 : 2;
+  static constexpr int OFF_G = BUFS * STAGE;                            // output gates
   static constexpr int OFF_P = OFF_G + MC_C * MC_VP * 2;                // weighted scores in two bf16 terms
-  static constexpr int OFF_F = OFF_P + 2 * MC_C * MC_PP * 2;
+  static constexpr int OFF_X = OFF_P + 2 * MC_C * MC_PP * 2;            // partial read-outs exchanged by the warps of a pair
+  static constexpr int OFF_F = OFF_X + 16 * 16 * 32 * 4;
   // floats: a, M, dec, eneg, w [64 each], row sums [4][64], q.n [64], squares [8][64], peers [2][8][64], n [DP], n parts [3][DP], scalars [8]
   static constexpr int FLOATS = 5 * MC_C + 4 * MC_C + MC_C + 8 * MC_C + 2 * MC_MAX_BLOCKS * MC_C + 4 * DP + 8;
   static constexpr int TOTAL = OFF_F + FLOATS * 4;
@@ -81,7 +83,7 @@ __global__ void __launch_bounds__(MC_THREADS, 1)
 mlstm_chunk_kernel(const MlstmChunkParams P) {
   using L = McSmem<DP>;
   namespace cg = cooperative_groups;
-  constexpr int KS = DP / 16, NT = DP / 8;
+  constexpr int KS = DP / 16, NT = DP / 16;          // k steps of q k; 8-column tiles of S^T per warp
   constexpr int PARTS = DP >= MC_THREADS ? 1 : (MC_THREADS / DP < 4 ? MC_THREADS / DP : 4);   // token parts of the n update
   extern __shared__ __align__(16) uint8_t smem[];
   float* fl = reinterpret_cast<float*>(smem + L::OFF_F);
@@ -89,7 +91,9 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
         *sss = sqn + MC_C, *speer = sss + 8 * MC_C, *sn = speer + 2 * MC_MAX_BLOCKS * MC_C, *snp = sn + DP, *sc = snp + 3 * DP;
   bf16* sP = reinterpret_cast<bf16*>(smem + L::OFF_P);
   bf16* sG = reinterpret_cast<bf16*>(smem + L::OFF_G);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* sX = reinterpret_cast<float*>(smem + L::OFF_X);
+  // two warps share 16 columns of v (wg): each holds half of the d columns of S^T and finishes half of the tokens (hw)
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wg = warp & 7, hw = warp >> 3;
   const int b = blockIdx.z / P.nseg, seg = blockIdx.z % P.nseg, h = blockIdx.y, c0 = blockIdx.x * P.cols;
   const int H = P.H, d = P.d, e = P.e;
   const int s0 = P.cu[b], len = P.cu[b + 1] - s0;
@@ -97,8 +101,8 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
   const int t_lo = seg * seg_len, t_hi = min(len, t_lo + seg_len);
   if (t_lo >= t_hi) return;                          // the same for every CTA of a cluster
   if (!FULL && t_hi == len) return;                  // nothing follows: the segment's own state is not needed
-  const int e0 = c0 + warp * 16;                     // first column of this warp
-  const bool e_ok = e0 < e && warp * 16 < P.cols;
+  const int e0 = c0 + wg * 16, d0 = hw * (DP / 2);   // first column and first d of this warp
+  const bool e_ok = e0 < e && wg * 16 < P.cols;
   const int er = lane >> 2, kc = (lane & 3) * 2, mi = lane >> 3, r8 = lane & 7;
   const long long lsize = static_cast<long long>(d) * e + d + 2;
   const bool have = P.slots != nullptr && P.slots[b] >= 0;
@@ -107,7 +111,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
   float* slot_n = have ? slot + static_cast<long long>(H) * d * e + h * d : nullptr;
   float* slot_m = have ? slot + static_cast<long long>(H) * d * e + H * d + h : nullptr;
 
-  // ---- S^T accumulators: tile j covers d columns [8j, 8j + 8); element (e0 + er (+ 8), 8j + kc (+ 1))
+  // ---- S^T accumulators: tile j covers d columns [d0 + 8j, + 8); element (e0 + er (+ 8), d0 + 8j + kc (+ 1))
   float S[NT][4];
 #pragma unroll
   for (int j = 0; j < NT; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.f;
@@ -116,7 +120,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
     for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int dd = j * 8 + kc + (i & 1), ee = e0 + er + (i >> 1) * 8;
+        const int dd = d0 + j * 8 + kc + (i & 1), ee = e0 + er + (i >> 1) * 8;
         if (e_ok && dd < d && ee < e) fn(S[j][i], dd, ee);
       }
   };
@@ -187,7 +191,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
   if (nblk > 1) cluster.sync();                      // peers run, and have read the stored state, before anything is replaced
   __syncthreads();
   int st = 0;
-  for (int t0 = t_lo; t0 < t_hi; t0 += MC_C, st ^= 1) {
+  for (int t0 = t_lo; t0 < t_hi; t0 += MC_C, st ^= L::BUFS - 1) {
     // ---- gates of the chunk
     if (warp == 0) {
       float il[2], ff[2];
@@ -243,110 +247,118 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       load_v(sG, t0, 2 * H * d + static_cast<long long>(H + h) * e + c0);
       asm volatile("cp.async.commit_group;");
     }
-    if (more) load(st ^ 1, t0 + MC_C);
+    if (L::BUFS == 2 && more) load(st ^ 1, t0 + MC_C);
     const bf16* q = reinterpret_cast<const bf16*>(smem + st * L::STAGE);
     const bf16* k = q + MC_C * L::QP;
     const uint32_t uq = mc_smem(q), uk = mc_smem(k), uv = mc_smem(k + MC_C * L::QP), uP = mc_smem(sP);
     const float decC = sc[0], m_next = sc[1];
-    float o[4][2][4] = {};
+    float o[2][2][4] = {};
     const int par = ((t0 - t_lo) / MC_C) & 1;
     if (FULL) {
-      // ---- weighted scores P = exp(a_s - M_t) q_t . k_s: a warp owns 16 rows and 32 columns, zero above the diagonal
+      // ---- weighted scores P = exp(a_s - M_t) q_t . k_s: a warp owns a 16 x 16 block, zero above the diagonal
       {
-        const int tb = (warp >> 1) * 16;
-        float rs[2][2] = {};
+        const int tb = (warp >> 2) * 16, sb = (warp & 3) * 16;
+        float acc[2][4] = {};
+        if (sb <= tb) {
 #pragma unroll
-        for (int j2 = 0; j2 < 2; ++j2) {
-          const int sb = ((warp & 1) * 2 + j2) * 16;
-          float acc[2][4] = {};
-          if (sb <= tb) {
-#pragma unroll
-            for (int kk = 0; kk < KS; ++kk) {
-              uint32_t fa[4], fb[4];
-              mc_ldsm(fa, uq + ((tb + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
-              mc_ldsm(fb, uk + ((sb + (mi >> 1) * 8 + r8) * L::QP + kk * 16 + (mi & 1) * 8) * 2);
-              mc_mma(acc[0], fa, fb[0], fb[1]);
-              mc_mma(acc[1], fa, fb[2], fb[3]);
-            }
-          }
-#pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int t = tb + er + half * 8;
-            const float Mt = sM[t];
-#pragma unroll
-            for (int j = 0; j < 2; ++j) {
-              float x[2];
-#pragma unroll
-              for (int u = 0; u < 2; ++u) {
-                const int s = sb + j * 8 + kc + u;
-                x[u] = s <= t ? acc[j][half * 2 + u] * qs * __expf(sa[s] - Mt) : 0.f;
-                rs[j2][half] += x[u];
-              }
-              uint32_t hi, lo;
-              mc_split(x[0], x[1], hi, lo);
-              *reinterpret_cast<uint32_t*>(sP + t * MC_PP + sb + j * 8 + kc) = hi;
-              *reinterpret_cast<uint32_t*>(sP + (MC_C + t) * MC_PP + sb + j * 8 + kc) = lo;
-            }
+          for (int kk = 0; kk < KS; ++kk) {
+            uint32_t fa[4], fb[4];
+            mc_ldsm(fa, uq + ((tb + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
+            mc_ldsm(fb, uk + ((sb + (mi >> 1) * 8 + r8) * L::QP + kk * 16 + (mi & 1) * 8) * 2);
+            mc_mma(acc[0], fa, fb[0], fb[1]);
+            mc_mma(acc[1], fa, fb[2], fb[3]);
           }
         }
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          float r = rs[0][half] + rs[1][half];
-          r += __shfl_xor_sync(0xffffffffu, r, 1);
-          r += __shfl_xor_sync(0xffffffffu, r, 2);
-          if ((lane & 3) == 0) sden[(warp & 1) * MC_C + tb + er + half * 8] = r;
+          const int t = tb + er + half * 8;
+          const float Mt = sM[t];
+          float rs = 0.f;
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            float x[2];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+              const int s = sb + j * 8 + kc + u;
+              x[u] = s <= t ? acc[j][half * 2 + u] * qs * __expf(sa[s] - Mt) : 0.f;
+              rs += x[u];
+            }
+            uint32_t hi, lo;
+            mc_split(x[0], x[1], hi, lo);
+            *reinterpret_cast<uint32_t*>(sP + t * MC_PP + sb + j * 8 + kc) = hi;
+            *reinterpret_cast<uint32_t*>(sP + (MC_C + t) * MC_PP + sb + j * 8 + kc) = lo;
+          }
+          rs += __shfl_xor_sync(0xffffffffu, rs, 1);
+          rs += __shfl_xor_sync(0xffffffffu, rs, 2);
+          if ((lane & 3) == 0) sden[(warp & 3) * MC_C + t] = rs;
         }
       }
-      // ---- q_t . n_prev: four lanes per token
+      // ---- q_t . n_prev: eight lanes per token
       {
-        const int t = tid >> 2;
+        const int t = tid >> 3;
         float x = 0.f;
-#pragma unroll 8
-        for (int c = (tid & 3) * 2; c < DP; c += 8) {
+#pragma unroll 4
+        for (int c = (tid & 7) * 2; c < DP; c += 16) {
           const float2 qq = mc_unpack(*reinterpret_cast<const uint32_t*>(q + t * L::QP + c));
           x += qq.x * sn[c] + qq.y * sn[c + 1];
         }
         x += __shfl_xor_sync(0xffffffffu, x, 1);
         x += __shfl_xor_sync(0xffffffffu, x, 2);
-        if ((tid & 3) == 0) sqn[t] = x * qs;
+        x += __shfl_xor_sync(0xffffffffu, x, 4);
+        if ((tid & 7) == 0) sqn[t] = x * qs;
       }
-      __syncthreads();                                // B: scores, row sums
-      if (e_ok) {
+      // ---- read-out of this warp's half of the state for all tokens; the pair swaps the halves it does not finish
+      {
+        float r[4][2][4] = {};
+        if (e_ok) {
 #pragma unroll
-        for (int kk = 0; kk < KS; ++kk) {             // read-out of the state
-          uint32_t h0, l0, h1, l1, h2, l2, h3, l3;
-          mc_split(S[2 * kk][0], S[2 * kk][1], h0, l0);
-          mc_split(S[2 * kk + 1][0], S[2 * kk + 1][1], h1, l1);
-          mc_split(S[2 * kk][2], S[2 * kk][3], h2, l2);
-          mc_split(S[2 * kk + 1][2], S[2 * kk + 1][3], h3, l3);
+          for (int kk = 0; kk < KS / 2; ++kk) {
+            uint32_t h0, l0, h1, l1, h2, l2, h3, l3;
+            mc_split(S[2 * kk][0], S[2 * kk][1], h0, l0);
+            mc_split(S[2 * kk + 1][0], S[2 * kk + 1][1], h1, l1);
+            mc_split(S[2 * kk][2], S[2 * kk][3], h2, l2);
+            mc_split(S[2 * kk + 1][2], S[2 * kk + 1][3], h3, l3);
 #pragma unroll
-          for (int m = 0; m < 4; ++m) {
-            uint32_t fa[4];
-            mc_ldsm(fa, uq + ((m * 16 + (mi & 1) * 8 + r8) * L::QP + kk * 16 + (mi >> 1) * 8) * 2);
-            mc_mma(o[m][0], fa, h0, h1);
-            mc_mma(o[m][1], fa, h2, h3);
-            mc_mma(o[m][0], fa, l0, l1);
-            mc_mma(o[m][1], fa, l2, l3);
+            for (int m = 0; m < 4; ++m) {
+              uint32_t fa[4];
+              mc_ldsm(fa, uq + ((m * 16 + (mi & 1) * 8 + r8) * L::QP + d0 + kk * 16 + (mi >> 1) * 8) * 2);
+              mc_mma(r[m][0], fa, h0, h1);
+              mc_mma(r[m][1], fa, h2, h3);
+              mc_mma(r[m][0], fa, l0, l1);
+              mc_mma(r[m][1], fa, l2, l3);
+            }
           }
         }
 #pragma unroll
-        for (int m = 0; m < 4; ++m)
+        for (int m = 0; m < 2; ++m)
 #pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const float f = sdec[m * 16 + half * 8 + er] * qs;
-            o[m][0][half * 2] *= f; o[m][0][half * 2 + 1] *= f;
-            o[m][1][half * 2] *= f; o[m][1][half * 2 + 1] *= f;
-          }
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              sX[((warp * 2 + m) * 8 + n * 4 + i) * 32 + lane] = hw ? r[m][n][i] : r[2 + m][n][i];
+              o[m][n][i] = hw ? r[2 + m][n][i] : r[m][n][i];
+            }
+      }
+      __syncthreads();                                // B: scores, row sums, partial read-outs
+      if (e_ok) {
+#pragma unroll
+        for (int m = 0; m < 2; ++m)
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+              o[m][n][i] = (o[m][n][i] + sX[(((warp ^ 8) * 2 + m) * 8 + n * 4 + i) * 32 + lane]) * (sdec[hw * 32 + m * 16 + (i >> 1) * 8 + er] * qs);
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk) {              // the chunk's own tokens
+          if (kk >= 2 + 2 * hw) continue;
           uint32_t fv[4];
-          mc_ldsm_t(fv, uv + ((kk * 16 + (mi & 1) * 8 + r8) * MC_VP + warp * 16 + (mi >> 1) * 8) * 2);
+          mc_ldsm_t(fv, uv + ((kk * 16 + (mi & 1) * 8 + r8) * MC_VP + wg * 16 + (mi >> 1) * 8) * 2);
 #pragma unroll
-          for (int m = kk; m < 4; ++m)
+          for (int m = 0; m < 2; ++m)
 #pragma unroll
             for (int term = 0; term < 2; ++term) {
               uint32_t fa[4];
-              mc_ldsm(fa, uP + ((term * MC_C + m * 16 + (mi & 1) * 8 + r8) * MC_PP + kk * 16 + (mi >> 1) * 8) * 2);
+              mc_ldsm(fa, uP + ((term * MC_C + hw * 32 + m * 16 + (mi & 1) * 8 + r8) * MC_PP + kk * 16 + (mi >> 1) * 8) * 2);
               mc_mma(o[m][0], fa, fv[0], fv[1]);
               mc_mma(o[m][1], fa, fv[2], fv[3]);
             }
@@ -354,11 +366,11 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       }
       // ---- denominator; sum of squares over the head
 #pragma unroll
-      for (int m = 0; m < 4; ++m)
+      for (int m = 0; m < 2; ++m)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          const int t = m * 16 + half * 8 + er;
-          const float den = sdec[t] * sqn[t] + (sden[t] + sden[MC_C + t]);
+          const int t = hw * 32 + m * 16 + half * 8 + er;
+          const float den = sdec[t] * sqn[t] + ((sden[t] + sden[MC_C + t]) + (sden[2 * MC_C + t] + sden[3 * MC_C + t]));
           const float inv = __fdividef(1.f, fmaxf(fabsf(den), sneg[t]) + 1e-6f);
           float ss = 0.f;
 #pragma unroll
@@ -371,9 +383,9 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
             }
           ss += __shfl_xor_sync(0xffffffffu, ss, 1);
           ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-          if ((lane & 3) == 0) sss[warp * MC_C + t] = ss;
+          if ((lane & 3) == 0) sss[wg * MC_C + t] = ss;
         }
-      if (more) asm volatile("cp.async.wait_group 1;");
+      if (L::BUFS == 2 && more) asm volatile("cp.async.wait_group 1;");
       else asm volatile("cp.async.wait_group 0;");
       __syncthreads();                                // C: sums of squares, output gates
       if (nblk > 1) {
@@ -394,7 +406,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       for (int kk = 0; kk < MC_C / 16; ++kk) {
         uint32_t fv[4], hi[4], lo[4];
         // (w v)^T as A: rows = v columns, k = tokens; registers {e0 s0, e8 s0, e0 s8, e8 s8}
-        mc_ldsm_t(fv, uv + ((kk * 16 + (mi >> 1) * 8 + r8) * MC_VP + warp * 16 + (mi & 1) * 8) * 2);
+        mc_ldsm_t(fv, uv + ((kk * 16 + (mi >> 1) * 8 + r8) * MC_VP + wg * 16 + (mi & 1) * 8) * 2);
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int s = kk * 16 + (i >> 1) * 8 + kc;
@@ -404,7 +416,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
 #pragma unroll
         for (int j = 0; j < NT / 2; ++j) {
           uint32_t fk[4];
-          mc_ldsm_t(fk, uk + ((kk * 16 + (mi & 1) * 8 + r8) * L::QP + j * 16 + (mi >> 1) * 8) * 2);
+          mc_ldsm_t(fk, uk + ((kk * 16 + (mi & 1) * 8 + r8) * L::QP + d0 + j * 16 + (mi >> 1) * 8) * 2);
           mc_mma(S[2 * j], hi, fk[0], fk[1]);
           mc_mma(S[2 * j + 1], hi, fk[2], fk[3]);
           mc_mma(S[2 * j], lo, fk[0], fk[1]);
@@ -425,10 +437,10 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       if (nblk > 1) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
       if (e_ok) {
 #pragma unroll
-        for (int m = 0; m < 4; ++m)
+        for (int m = 0; m < 2; ++m)
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
-            const int t = m * 16 + half * 8 + er;
+            const int t = hw * 32 + m * 16 + half * 8 + er;
             float ss = 0.f;
             if (nblk > 1) {
               for (int r = 0; r < nblk; ++r) ss += speer[(par * MC_MAX_BLOCKS + r) * MC_C + t];
@@ -440,7 +452,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
             bf16* dst = P.out + static_cast<long long>(s0 + t0 + t) * P.ldo + h * e + e0 + kc;
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-              const float2 g = mc_unpack(*reinterpret_cast<const uint32_t*>(sG + t * MC_VP + warp * 16 + n * 8 + kc));
+              const float2 g = mc_unpack(*reinterpret_cast<const uint32_t*>(sG + t * MC_VP + wg * 16 + n * 8 + kc));
               const float y0 = __fdividef(o[m][n][half * 2] * rs * wn[n][0], 1.f + __expf(-g.x));
               const float y1 = __fdividef(o[m][n][half * 2 + 1] * rs * wn[n][1], 1.f + __expf(-g.y));
               if (t0 + t < t_hi && e0 + n * 8 + kc < e) *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) = __floats2bfloat162_rn(y0, y1);
@@ -451,6 +463,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
     m_prev = m_next;
     f_total += sc[2];
     __syncthreads();                                  // D: gates, n and the chunk may be replaced
+    if (L::BUFS == 1 && more) load(0, t0 + MC_C);
   }
   for (int r = tid; r < DP; r += MC_THREADS)
 #pragma unroll
