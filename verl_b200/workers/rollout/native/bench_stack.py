@@ -10,6 +10,7 @@ JSON line per measurement.
 
 from __future__ import annotations
 
+import gc
 import json
 
 import torch
@@ -90,6 +91,7 @@ def bench_model(cfg: ModelConfig, s: dict, steps: int, warmup: int) -> dict:
     out = {"parameters": cfg.num_parameters(), "prefill_tokens_per_s": round(n * L / ms_p * 1e3), "prefill_ms": round(ms_p, 3),
            "decode_tokens_per_s": round(S / ms_d * 1e3), "decode_ms_per_step": round(ms_d, 3), "decode_kernels_per_step": launches, "clocks": clocks}
     del eng, P
+    gc.collect()
     torch.cuda.empty_cache()
     return out
 

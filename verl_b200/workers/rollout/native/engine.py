@@ -28,6 +28,7 @@ max_num_seqs / max_num_batched_tokens, dummy-weight start, KV release/resume, ab
 
 from __future__ import annotations
 
+import gc
 import math
 import os
 import time
@@ -854,6 +855,7 @@ class RolloutEngine:
                     dst.copy_(src)
                 from ....ops import native
 
+                gc.collect()  # a dropped engine's graph that is destroyed during this capture would invalidate it
                 g = torch.cuda.CUDAGraph()
                 n0 = native.launch_count()
                 with torch.cuda.graph(g):
