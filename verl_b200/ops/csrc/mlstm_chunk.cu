@@ -311,6 +311,11 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       {
         float r[4][2][4] = {};
         if (e_ok) {
+          uint32_t fa[2][4];                          // query fragments, one product ahead
+          auto fetch = [&](int i) {
+            mc_ldsm(fa[i & 1], uq + (((i & 3) * 16 + (mi & 1) * 8 + r8) * L::QP + d0 + (i >> 2) * 16 + (mi >> 1) * 8) * 2);
+          };
+          fetch(0);
 #pragma unroll
           for (int kk = 0; kk < KS / 2; ++kk) {
             uint32_t h0, l0, h1, l1, h2, l2, h3, l3;
@@ -320,12 +325,11 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
             mc_split(S[2 * kk + 1][2], S[2 * kk + 1][3], h3, l3);
 #pragma unroll
             for (int m = 0; m < 4; ++m) {
-              uint32_t fa[4];
-              mc_ldsm(fa, uq + ((m * 16 + (mi & 1) * 8 + r8) * L::QP + d0 + kk * 16 + (mi >> 1) * 8) * 2);
-              mc_mma(r[m][0], fa, h0, h1);
-              mc_mma(r[m][1], fa, h2, h3);
-              mc_mma(r[m][0], fa, l0, l1);
-              mc_mma(r[m][1], fa, l2, l3);
+              if (kk * 4 + m + 1 < KS * 2) fetch(kk * 4 + m + 1);
+              mc_mma(r[m][0], fa[m & 1], h0, h1);
+              mc_mma(r[m][1], fa[m & 1], h2, h3);
+              mc_mma(r[m][0], fa[m & 1], l0, l1);
+              mc_mma(r[m][1], fa[m & 1], l2, l3);
             }
           }
         }
@@ -413,14 +417,16 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
           const float2 x = mc_unpack(fv[i]);
           mc_split(x.x * sw[s], x.y * sw[s + 1], hi[i], lo[i]);
         }
+        uint32_t fk[2][4];                            // key fragments, one product ahead
+        auto fetch = [&](int j) { mc_ldsm_t(fk[j & 1], uk + ((kk * 16 + (mi & 1) * 8 + r8) * L::QP + d0 + j * 16 + (mi >> 1) * 8) * 2); };
+        fetch(0);
 #pragma unroll
         for (int j = 0; j < NT / 2; ++j) {
-          uint32_t fk[4];
-          mc_ldsm_t(fk, uk + ((kk * 16 + (mi & 1) * 8 + r8) * L::QP + d0 + j * 16 + (mi >> 1) * 8) * 2);
-          mc_mma(S[2 * j], hi, fk[0], fk[1]);
-          mc_mma(S[2 * j + 1], hi, fk[2], fk[3]);
-          mc_mma(S[2 * j], lo, fk[0], fk[1]);
-          mc_mma(S[2 * j + 1], lo, fk[2], fk[3]);
+          if (j + 1 < NT / 2) fetch(j + 1);
+          mc_mma(S[2 * j], hi, fk[j & 1][0], fk[j & 1][1]);
+          mc_mma(S[2 * j + 1], hi, fk[j & 1][2], fk[j & 1][3]);
+          mc_mma(S[2 * j], lo, fk[j & 1][0], fk[j & 1][1]);
+          mc_mma(S[2 * j + 1], lo, fk[j & 1][2], fk[j & 1][3]);
         }
       }
     }
