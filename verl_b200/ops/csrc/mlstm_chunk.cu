@@ -73,8 +73,10 @@ struct McSmem {
   static constexpr int OFF_P = OFF_G + MC_C * MC_VP * 2;                // weighted scores in two bf16 terms
   static constexpr int OFF_X = OFF_P + 2 * MC_C * MC_PP * 2;            // partial read-outs exchanged by the warps of a pair
   static constexpr int OFF_F = OFF_X + 16 * 16 * 32 * 4;
-  // floats: a, M, dec, eneg, w [64 each], row sums [4][64], q.n [64], squares [8][64], peers [2][8][64], n [DP], n parts [3][DP], scalars [8]
-  static constexpr int FLOATS = 5 * MC_C + 4 * MC_C + MC_C + 8 * MC_C + 2 * MC_MAX_BLOCKS * MC_C + 4 * DP + 8;
+  // floats: two gate buffers {a, M, dec, eneg, w [64 each], scalars [8]}, row sums [4][64], q.n [64], squares [8][64], peers [2][8][64],
+  // n [DP], n parts [7][DP]
+  static constexpr int GATES = 5 * MC_C + 8;
+  static constexpr int FLOATS = 2 * GATES + 4 * MC_C + MC_C + 8 * MC_C + 2 * MC_MAX_BLOCKS * MC_C + 8 * DP;
   static constexpr int TOTAL = OFF_F + FLOATS * 4;
 };
 
@@ -84,11 +86,11 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
   using L = McSmem<DP>;
   namespace cg = cooperative_groups;
   constexpr int KS = DP / 16, NT = DP / 16;          // k steps of q k; 8-column tiles of S^T per warp
-  constexpr int PARTS = DP >= MC_THREADS ? 1 : (MC_THREADS / DP < 4 ? MC_THREADS / DP : 4);   // token parts of the n update
+  constexpr int PARTS = MC_THREADS / (DP / 2) < 8 ? MC_THREADS / (DP / 2) : 8;   // token parts of the n update (two columns a thread)
   extern __shared__ __align__(16) uint8_t smem[];
   float* fl = reinterpret_cast<float*>(smem + L::OFF_F);
-  float *sa = fl, *sM = sa + MC_C, *sdec = sM + MC_C, *sneg = sdec + MC_C, *sw = sneg + MC_C, *sden = sw + MC_C, *sqn = sden + 4 * MC_C,
-        *sss = sqn + MC_C, *speer = sss + 8 * MC_C, *sn = speer + 2 * MC_MAX_BLOCKS * MC_C, *snp = sn + DP, *sc = snp + 3 * DP;
+  float *sden = fl + 2 * L::GATES, *sqn = sden + 4 * MC_C, *sss = sqn + MC_C, *speer = sss + 8 * MC_C, *sn = speer + 2 * MC_MAX_BLOCKS * MC_C,
+        *snp = sn + DP;
   bf16* sP = reinterpret_cast<bf16*>(smem + L::OFF_P);
   bf16* sG = reinterpret_cast<bf16*>(smem + L::OFF_G);
   float* sX = reinterpret_cast<float*>(smem + L::OFF_X);
@@ -126,7 +128,7 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
   };
   float m_prev = FULL ? 0.f : -INFINITY, f_total = 0.f;
   for (int r = tid; r < DP; r += MC_THREADS) sn[r] = 0.f;
-  for (int r = tid; r < 3 * DP; r += MC_THREADS) snp[r] = 0.f;
+  for (int r = tid; r < 7 * DP; r += MC_THREADS) snp[r] = 0.f;
   if (FULL) {
     if (have && P.fresh != nullptr && P.fresh[b] == 0) {
       each([&](float& v, int dd, int ee) { v = slot_S[static_cast<long long>(dd) * e + ee]; });
@@ -184,58 +186,65 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
       gf[u] = t < t_hi ? g[H + h] : 0.f;
     }
   };
-  if (warp == 0) fetch_gates(t_lo);
+  // Gates of the chunk at t0 into buffer `buf` (one warp; its score block lies above the diagonal, so it has the time), and the
+  // request for those of the chunk after it.
+  float m_run = m_prev;
+  auto gates = [&](int t0, int buf) {
+    float *sa = fl + buf * L::GATES, *sM = sa + MC_C, *sdec = sM + MC_C, *sneg = sdec + MC_C, *sw = sneg + MC_C, *sc = sw + MC_C;
+    float il[2], ff[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const bool ok = t0 + lane * 2 + u < t_hi;
+      il[u] = ok ? P.cap * tanhf((gi[u] + ibv) / P.cap) : -INFINITY;
+      ff[u] = ok ? log_sigmoid(P.cap * tanhf((gf[u] + fbv) / P.cap)) : 0.f;
+    }
+    fetch_gates(t0 + MC_C);
+    float run = ff[0] + ff[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += x;
+    }
+    const float b1 = run, b0 = run - ff[1];
+    const float a0 = il[0] - b0, a1 = il[1] - b1;
+    float mx = fmaxf(a0, a1);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, mx, o);
+      if (lane >= o) mx = fmaxf(mx, x);
+    }
+    float before = __shfl_up_sync(0xffffffffu, mx, 1);
+    if (lane == 0) before = -INFINITY;
+    const float M0 = fmaxf(m_run, fmaxf(before, a0)), M1 = fmaxf(m_run, mx);
+    const float MC = __shfl_sync(0xffffffffu, M1, 31), bC = __shfl_sync(0xffffffffu, b1, 31);
+    const float aa[2] = {a0, a1}, MM[2] = {M0, M1}, bb[2] = {b0, b1};
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int t = lane * 2 + u;
+      sa[t] = aa[u];
+      sM[t] = MM[u];
+      sdec[t] = expf(m_run - MM[u]);
+      sneg[t] = expf(-(bb[u] + MM[u]));
+      sw[t] = expf(aa[u] - MC);
+    }
+    if (lane == 0) {
+      sc[0] = expf(m_run - MC);
+      sc[1] = bC + MC;
+      sc[2] = bC;
+    }
+    m_run = bC + MC;
+  };
   load(0, t_lo);
+  if (warp == 1) {
+    fetch_gates(t_lo);
+    gates(t_lo, 0);
+  }
   cg::cluster_group cluster = cg::this_cluster();
   const int nblk = gridDim.x;
   if (nblk > 1) cluster.sync();                      // peers run, and have read the stored state, before anything is replaced
   __syncthreads();
   int st = 0;
   for (int t0 = t_lo; t0 < t_hi; t0 += MC_C, st ^= L::BUFS - 1) {
-    // ---- gates of the chunk
-    if (warp == 0) {
-      float il[2], ff[2];
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const bool ok = t0 + lane * 2 + u < t_hi;
-        il[u] = ok ? P.cap * tanhf((gi[u] + ibv) / P.cap) : -INFINITY;
-        ff[u] = ok ? log_sigmoid(P.cap * tanhf((gf[u] + fbv) / P.cap)) : 0.f;
-      }
-      fetch_gates(t0 + MC_C);
-      float run = ff[0] + ff[1];
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float x = __shfl_up_sync(0xffffffffu, run, o);
-        if (lane >= o) run += x;
-      }
-      const float b1 = run, b0 = run - ff[1];
-      const float a0 = il[0] - b0, a1 = il[1] - b1;
-      float mx = fmaxf(a0, a1);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float x = __shfl_up_sync(0xffffffffu, mx, o);
-        if (lane >= o) mx = fmaxf(mx, x);
-      }
-      float before = __shfl_up_sync(0xffffffffu, mx, 1);
-      if (lane == 0) before = -INFINITY;
-      const float M0 = fmaxf(m_prev, fmaxf(before, a0)), M1 = fmaxf(m_prev, mx);
-      const float MC = __shfl_sync(0xffffffffu, M1, 31), bC = __shfl_sync(0xffffffffu, b1, 31);
-      const float aa[2] = {a0, a1}, MM[2] = {M0, M1}, bb[2] = {b0, b1};
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int t = lane * 2 + u;
-        sa[t] = aa[u];
-        sM[t] = MM[u];
-        sdec[t] = expf(m_prev - MM[u]);
-        sneg[t] = expf(-(bb[u] + MM[u]));
-        sw[t] = expf(aa[u] - MC);
-      }
-      if (lane == 0) {
-        sc[0] = expf(m_prev - MC);
-        sc[1] = bC + MC;
-        sc[2] = bC;
-      }
-    }
     for (int r = tid; r < DP; r += MC_THREADS) {      // the parts of the last chunk's n update
 #pragma unroll
       for (int u = 0; u < PARTS - 1; ++u) sn[r] += snp[u * DP + r];
@@ -251,9 +260,11 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
     const bf16* q = reinterpret_cast<const bf16*>(smem + st * L::STAGE);
     const bf16* k = q + MC_C * L::QP;
     const uint32_t uq = mc_smem(q), uk = mc_smem(k), uv = mc_smem(k + MC_C * L::QP), uP = mc_smem(sP);
-    const float decC = sc[0], m_next = sc[1];
-    float o[2][2][4] = {};
     const int par = ((t0 - t_lo) / MC_C) & 1;
+    const float *sa = fl + par * L::GATES, *sM = sa + MC_C, *sdec = sM + MC_C, *sneg = sdec + MC_C, *sw = sneg + MC_C, *sc = sw + MC_C;
+    const float decC = sc[0], m_next = sc[1];
+    if (warp == 1 && more) gates(t0 + MC_C, par ^ 1);
+    float o[2][2][4] = {};
     if (FULL) {
       // ---- weighted scores P = exp(a_s - M_t) q_t . k_s: a warp owns a 16 x 16 block, zero above the diagonal
       {
@@ -430,13 +441,23 @@ mlstm_chunk_kernel(const MlstmChunkParams P) {
         }
       }
     }
-    for (int i = tid; i < DP * PARTS; i += MC_THREADS) {
-      const int r = i % DP, part = i / DP;
-      float x = part == 0 ? decC * sn[r] : 0.f;
-#pragma unroll 8
-      for (int s = part * (MC_C / PARTS); s < (part + 1) * (MC_C / PARTS); ++s) x += sw[s] * to_f(k[s * L::QP + r]);
-      if (part == 0) sn[r] = x;
-      else snp[(part - 1) * DP + r] = x;
+    if (tid < DP / 2 * PARTS) {
+      const int r = tid % (DP / 2) * 2, part = tid / (DP / 2);
+      float x0 = part == 0 ? decC * sn[r] : 0.f, x1 = part == 0 ? decC * sn[r + 1] : 0.f;
+#pragma unroll
+      for (int s = part * (MC_C / PARTS); s < (part + 1) * (MC_C / PARTS); s += 4) {
+        const float4 w = *reinterpret_cast<const float4*>(sw + s);
+        const float ww[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const float2 kk = mc_unpack(*reinterpret_cast<const uint32_t*>(k + (s + u) * L::QP + r));
+          x0 += ww[u] * kk.x;
+          x1 += ww[u] * kk.y;
+        }
+      }
+      float* dst = part == 0 ? sn + r : snp + (part - 1) * DP + r;
+      dst[0] = x0;
+      dst[1] = x1;
     }
     if (FULL) {
       // ---- norm over the head, weight, output gate
