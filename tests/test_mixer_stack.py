@@ -48,7 +48,7 @@ CONFIGS = {
     "odd": config([mlstm(heads=1, dim=10, vdim=14), attn(22, heads=3, dim=10, rot_dim=6, vdim=14, q_rank=18, kv_rank=20, window=5, scaling=None), attn(30, window=1)],
                   width=42, vocab=61, scale=0.8),
     # recurrent layers share weights with a later owner; the window passes a page and a chunk
-    "wide": config([mlstm(64, heads=2, dim=64, vdim=128, weights_of=2), attn(136, heads=8, dim=64, rot_dim=32, vdim=64, q_rank=96, kv_rank=128, window=65, scale=0.1),
+    "wide": config([mlstm(64, heads=2, dim=64, vdim=128, weights_of=2), attn(136, heads=6, dim=72, rot_dim=40, vdim=80, q_rank=88, kv_rank=136, window=65, scale=0.1),
                     mlstm(64, heads=2, dim=64, vdim=128)], width=128, vocab=200),
     # no window limit and partly rotated keys
     "full": config([attn(48, window=None, rot_dim=16, rot_dims=12), mlstm(48)]),
