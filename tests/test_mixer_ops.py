@@ -1,6 +1,7 @@
 """Operators of the mixer stacks, one mechanism at a time, against the plain restatement (``oracles/mixer_stack_plain.py``)."""
 
 import math
+import zlib
 
 import pytest
 import torch
@@ -18,6 +19,7 @@ GEN = torch.Generator().manual_seed(7)
 
 @pytest.fixture(params=PLACES)
 def place(request):
+    GEN.manual_seed(zlib.crc32(request.node.name.split("[")[0].encode()))     # the same inputs whatever ran before
     return request.param
 
 
@@ -212,7 +214,7 @@ def test_decode_attention_over_pages(place, heads, rank, dr, bs, window):
 def mlstm_inputs(T, H, d, e, gate_scale=2.0, f_bias=1.0):
     p = rand(T, 2 * H * (d + e))
     gates = torch.randn(T, 2 * H + 5, generator=GEN) * gate_scale
-    return p, gates, rand(H), rand(H) + f_bias, rand(H * e)
+    return p, gates, rand(H), (rand(H) + f_bias).bfloat16().float(), rand(H * e)
 
 
 def mlstm_want(p, gates, ib, fb, norm, cap, eps, H, d, e):
