@@ -211,10 +211,11 @@ class ModelConfig:
         """A mixer stack: the layer list in typed form; the framework-wide sizes summarise it (planning, reports)."""
         spec = parse_stack(d)
         heads = max(l.mixer.heads for l in spec.layers)
+        kv_heads = max(getattr(l.mixer, "kv_heads", l.mixer.heads) for l in spec.layers)
         return cls(model_type=spec.design.lower(), vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
                    intermediate_size=max((l.mlp.ff for l in spec.layers if l.mlp is not None), default=0), num_hidden_layers=len(spec.layers),
-                   num_attention_heads=heads, num_key_value_heads=heads, head_dim=max(l.mixer.vdim for l in spec.layers),
-                   rms_norm_eps=spec.norm_eps, bos_token_id=d.get("bos_token_id"), eos_token_id=d.get("eos_token_id"),
+                   num_attention_heads=heads, num_key_value_heads=kv_heads, head_dim=max(l.mixer.vdim for l in spec.layers),
+                   rms_norm_eps=spec.norm_eps, tie_word_embeddings=spec.tied_head, bos_token_id=d.get("bos_token_id"), eos_token_id=d.get("eos_token_id"),
                    pad_token_id=d.get("pad_token_id"), max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)), stack=spec,
                    extra={"hf_config": dict(d), "_explicit": ("attention_bias",)})
 

@@ -42,15 +42,15 @@ class ParamSpec:
 
 def _stack_param_specs(cfg: ModelConfig) -> list[ParamSpec]:
     """Mixer stacks: checkpoint names throughout, projections of the same input fused (``mixer_stack_config.fused_rows``)."""
-    from .mixer_stack_config import layer_tensors
+    from .mixer_stack_config import layer_tensors, model_tensors
 
     h, L = cfg.hidden_size, cfg.num_hidden_layers
-    specs = [ParamSpec("embed", (cfg.vocab_size, h), "normal", True, -1)]
+    first, last = model_tensors(cfg.stack, h, cfg.vocab_size)
+    specs = [ParamSpec(*t, -1) for t in first]
     for i, l in enumerate(cfg.stack.layers):
         if l.owner == i:
-            specs += [ParamSpec(n, shape, init, decay, i) for n, shape, init, decay in layer_tensors(cfg.stack, h, i)]
-    return specs + [ParamSpec("final.norm", (h,), "ones", False, L), ParamSpec("final.norm.b", (h,), "zeros", False, L),
-                    ParamSpec("final.norm.alpha", (1,), "fill:0.5", False, L), ParamSpec("head", (cfg.vocab_size, h), "normal", True, L)]
+            specs += [ParamSpec(*t, i) for t in layer_tensors(cfg.stack, h, i)]
+    return specs + [ParamSpec(*t, L) for t in last]
 
 
 def build_param_specs(cfg: ModelConfig, value_head: bool = False) -> list[ParamSpec]:
@@ -187,7 +187,7 @@ class FlatParams:
     @property
     def lm_head_weight(self) -> torch.Tensor:
         if self.cfg.is_stack:
-            return self.views["head"]
+            return self.views["embed" if self.cfg.stack.tied_head else "head"]
         return self.views["embed_tokens.weight"] if "lm_head.weight" not in self.views else self.views["lm_head.weight"]
 
     # ------------------------------------------------------------------ init
@@ -216,16 +216,16 @@ class FlatParams:
         """HF-named tensors as zero-copy views of the fused storage."""
         cfg = self.cfg
         if cfg.is_stack:
-            from .mixer_stack_config import checkpoint_parts
+            from .mixer_stack_config import checkpoint_parts, is_scalar
 
-            parts = checkpoint_parts(cfg.stack)
+            parts = checkpoint_parts(cfg.stack, cfg.hidden_size)
             for s in self.specs:
                 v = self.views[s.name]
                 if s.name in parts:
                     for name, r0, rows in parts[s.name]:
                         yield name, v[r0 : r0 + rows]
                 else:
-                    yield s.name, (v.view(()) if s.name.endswith(".alpha") else v)
+                    yield s.name, (v.view(()) if is_scalar(s.name) else v)
             return
         q, kv = cfg.q_size, cfg.kv_size
         mixtral, phi3 = cfg.model_type == "mixtral", cfg.model_type == "phi3"

@@ -1,5 +1,6 @@
-"""Operators of the mixer stacks (``models/mixer_stack.py``): Dynamic Tanh, GEMMs with fused epilogues, latent attention over
-expanded keys (prompts) and over the paged latents (decoding), and the mLSTM recurrence.
+"""Operators of the mixer stacks (``models/mixer_stack.py``): norms, GEMMs with fused epilogues, latent attention over expanded
+keys (prompts) and over the paged latents (decoding), grouped-query attention with capped scores over cached keys and values,
+mixtures of experts, and the mLSTM recurrence.
 
 As in ``functional``: CUDA tensors go to the hand-written kernels (bf16 or true fp32; nothing falls back silently), CPU
 tensors take a plain PyTorch path. The residual stream, gates, statistics and recurrent state are fp32 on every path.
@@ -7,6 +8,7 @@ tensors take a plain PyTorch path. The residual stream, gates, statistics and re
 
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -15,7 +17,9 @@ import torch.nn.functional as TF
 from . import native
 
 __all__ = ["embed_dyt", "dynamic_tanh", "linear_act", "linear_split", "linear_residual_", "rope_pairs_", "latent_prep", "gather_pages",
-           "headwise_linear", "latent_absorb", "latent_attention_prefill", "latent_attention_decode", "mlstm_prefill", "mlstm_decode"]
+           "headwise_linear", "latent_absorb", "latent_attention_prefill", "latent_attention_decode", "mlstm_prefill", "mlstm_decode",
+           "embed_rms", "linear_partial", "linear_softcap", "residual_rms_", "gated_silu", "gated_up", "gated_up_split", "ExpertPlan", "expert_dispatch",
+           "expert_up", "expert_down", "qkv_prep", "grouped_attention_prefill", "grouped_attention_decode"]
 
 
 def _ops():
@@ -68,6 +72,134 @@ def linear_residual_(a: torch.Tensor, w: torch.Tensor, x: torch.Tensor, norm=Non
         return h if norm is not None else None
     x += _mm(a, w)
     return dynamic_tanh(x, *norm) if norm is not None else None
+
+
+# ----------------------------------------------------------------------------------------------- RMS norms on sublayer outputs
+def _rms(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+
+def embed_rms(ids, weight, scale: float, nw, eps: float):
+    """(fp32 residual stream ``rms_norm(weight[ids] * scale) * nw``, the same in the weights' type)."""
+    if weight.is_cuda:
+        return _ops().embed_rms(ids.reshape(-1).contiguous(), weight, float(scale), nw, float(eps))
+    x = _rms(weight[ids.reshape(-1)].float() * scale, nw, eps)
+    return x, x.to(weight.dtype)
+
+
+def linear_partial(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``a w^T`` for a consumer that reads whole rows (``residual_rms_``): [M, N] in ``a``'s type, or, where few tokens make the
+    GEMM split its depth, the fp32 partial products [splits, M, N] for the consumer to add up."""
+    if a.is_cuda:
+        return _ops().linear_partial(a, w)
+    return _mm(a, w).to(a.dtype)
+
+
+def residual_rms_(x, y: Optional[torch.Tensor], nw, eps: float, mult: float, next_nw=None, experts=None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``x += mult * rms_norm(Y) * nw`` on the fp32 residual stream. ``Y`` is ``y`` ([T, W], or partial products [splits, T, W];
+    multiplied by ``sigmoid(gate[t])`` when a gate is given) plus, with ``experts = (rows, slot)``, the rows ``slot[t, j]`` of the
+    expert outputs. Returns the new stream in the weights' type, or its RMS norm with ``next_nw``."""
+    rows, slot = experts if experts is not None else (None, None)
+    if x.is_cuda:
+        return _ops().residual_rms_(x, y, nw, float(eps), float(mult), next_nw, rows, slot, gate)
+    total = torch.zeros_like(x)
+    if y is not None:
+        total = y.float().sum(0) if y.dim() == 3 else y.float()
+        if gate is not None:
+            total = total * torch.sigmoid(gate)[:, None]
+    if rows is not None:
+        total = total + rows[slot.long()].float().sum(1)
+    x += mult * _rms(total, nw, eps)
+    return (x if next_nw is None else _rms(x, next_nw, eps)).to(nw.dtype)
+
+
+def linear_softcap(a: torch.Tensor, w: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap * tanh(a w^T / cap)`` in ``a``'s type (``cap`` 0: the plain product)."""
+    if cap <= 0:
+        return linear_act(a, w)
+    if a.is_cuda:
+        return _ops().linear_softcap(a, w, float(cap))
+    return (cap * torch.tanh(_mm(a, w) / cap)).to(a.dtype)
+
+
+# ----------------------------------------------------------------------------------------------- gated feed-forward, experts
+def gated_silu(gu: torch.Tensor) -> torch.Tensor:
+    """``silu(g) * u`` of rows [g | u]."""
+    if gu.is_cuda:
+        return _ops().gated_silu(gu)
+    g, u = gu.float().chunk(2, -1)
+    return (TF.silu(g) * u).to(gu.dtype)
+
+
+def gated_up(h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``silu(h W_g^T) * (h W_u^T)`` for the stacked rows ``w = [W_g; W_u]``: in the GEMM's epilogue for prompts."""
+    if h.is_cuda and h.dtype == torch.bfloat16 and h.shape[0] > 1024 and w.shape[0] % 16 == 0 and w.shape[1] % 8 == 0 and w.data_ptr() % 16 == 0:
+        return _ops().gemm_swiglu(h, w, False)[0]
+    return gated_silu(linear_act(h, w))
+
+
+def gated_up_split(h: torch.Tensor, w: torch.Tensor, n0: int):
+    """(``gated_up`` of the first ``n0`` rows of ``w``, fp32 product with the rest); None in the first place when ``n0`` is 0."""
+    if n0 == 0:
+        return None, linear_act(h, w, out_f32=True)
+    if h.shape[0] > 1024:
+        return gated_up(h, w[:n0]), linear_act(h, w[n0:], out_f32=True)
+    gu, tail = linear_split(h, w, n0)
+    return gated_silu(gu), tail
+
+
+@dataclass
+class ExpertPlan:
+    """Tokens grouped by expert: ``x`` [rows, width] copies of the tokens (every expert's rows start at a multiple of 128 on the
+    GPU), ``slot`` [T, top] row of every copy, ``scale`` [rows] score of the copy's expert, and which expert owns which rows."""
+
+    x: torch.Tensor
+    slot: torch.Tensor
+    scale: torch.Tensor
+    tile_expert: torch.Tensor     # GPU: expert of every 128-row tile; CPU: first row of every expert [E + 1]
+    num_tiles: torch.Tensor
+
+
+def expert_dispatch(h: torch.Tensor, logits: torch.Tensor, experts: int, top: int, renormalize: bool = False) -> ExpertPlan:
+    """Router: the ``top`` experts with the largest ``sigmoid(logits)`` of every token (``logits`` fp32, columns past ``experts``
+    ignored), and the tokens' copies in expert order. No host synchronisation."""
+    if h.is_cuda:
+        return ExpertPlan(*_ops().expert_dispatch(h, logits, int(experts), int(top), bool(renormalize)))
+    s, e = torch.topk(torch.sigmoid(logits[:, :experts].float()), top, dim=-1)
+    if renormalize:
+        s = s / s.sum(-1, keepdim=True)
+    order = torch.argsort(e.reshape(-1), stable=True)
+    slot = torch.empty_like(order)
+    slot[order] = torch.arange(order.numel())
+    first = torch.zeros(experts + 1, dtype=torch.int64)
+    first[1:] = torch.bincount(e.reshape(-1), minlength=experts).cumsum(0)
+    return ExpertPlan(h[order // top], slot.view(-1, top), s.reshape(-1)[order], first, first[-1:])
+
+
+def expert_up(plan: ExpertPlan, w: torch.Tensor, ff: int) -> torch.Tensor:
+    """Per copy ``silu(s g) * (s u)`` with [g | u] = ``x w_e^T`` and the copy's score s (a factor on the expert's input); ``w``
+    [E * 2 ff, width]."""
+    w3 = w.view(-1, 2 * ff, w.shape[1])
+    if w.is_cuda:
+        return _ops().expert_up(plan.x, w3, plan.scale, plan.tile_expert, plan.num_tiles)
+    out = torch.empty(plan.x.shape[0], ff, dtype=plan.x.dtype)
+    for e in range(w3.shape[0]):
+        at = slice(int(plan.tile_expert[e]), int(plan.tile_expert[e + 1]))
+        g, u = (_mm(plan.x[at], w3[e]) * plan.scale[at, None]).chunk(2, -1)
+        out[at] = (TF.silu(g) * u).to(out.dtype)
+    return out
+
+
+def expert_down(act: torch.Tensor, w: torch.Tensor, plan: ExpertPlan) -> torch.Tensor:
+    """Per copy ``act w_e^T``; ``w`` [E * width, ff]. Rows without a copy hold anything."""
+    w3 = w.view(-1, plan.x.shape[1], w.shape[1])
+    if w.is_cuda:
+        return _ops().expert_linear(act, w3, plan.tile_expert, plan.num_tiles)
+    out = torch.empty(act.shape[0], w3.shape[1], dtype=act.dtype)
+    for e in range(w3.shape[0]):
+        at = slice(int(plan.tile_expert[e]), int(plan.tile_expert[e + 1]))
+        out[at] = _mm(act[at], w3[e]).to(out.dtype)
+    return out
 
 
 # ----------------------------------------------------------------------------------------------- latent attention

@@ -107,7 +107,11 @@ class FlopsCounter:
         if getattr(c, "is_stack", False):   # every matrix of every layer run once per token (the embedding gather is free)
             from ..models.mixer_stack_config import layer_tensors
 
-            mats = lambda i: sum(s[0] * s[1] for _, s, *_ in layer_tensors(c.stack, c.hidden_size, i) if len(s) == 2)
+            def mats(i):
+                f = c.stack.layers[i].mlp
+                used = f.top / f.experts if f is not None and f.kind == "moe" else 1.0
+                return sum(s[0] * s[1] * (used if ".experts." in n else 1.0) for n, s, *_ in layer_tensors(c.stack, c.hidden_size, i) if len(s) == 2)
+
             return float(sum(mats(l.owner) for l in c.stack.layers) + c.vocab_size * c.hidden_size)
         h = c.hidden_size
         attn_lin = h * (c.q_size + 2 * c.kv_size) + c.q_size * h
