@@ -1,13 +1,17 @@
-"""Decoder whose layers differ: latent attention and matrix-memory recurrences on one fp32 residual stream.
+"""Decoder whose layers differ: attention and recurrent mixers, dense and mixture-of-experts feed-forwards on one fp32 residual
+stream.
 
 The model runs packed prompt portions (``forward_hidden``) and one-token steps over all slots (``decode_hidden``) against the
-same cache object: a page pool for the latent rows of the attention layers and one fp32 state row per slot for the recurrent
+same cache object: a page pool for the rows of the attention layers and one fp32 state row per slot for the recurrent
 layers (``workers/rollout/native/cache.py::StackCache``). Layers that share weights still have their own pages and state.
 
-Step layout: every projection that reads a layer's input is one GEMM; norms are elementwise, so the GEMM that ends a sublayer
-adds to the residual stream and applies the next norm in its epilogue, and the feed-forward activation runs in the epilogue
-of its up-projection. Prompts expand keys and values from the latents; decoding absorbs the key expansion into the query and
-applies the value expansion to the attention output, so only latent rows are read.
+Step layout: every projection that reads a layer's input is one GEMM. Stacks with elementwise norms in front of the sublayers:
+the GEMM that ends a sublayer adds to the residual stream and applies the next norm in its epilogue. Stacks with RMS norms on
+the sublayers' outputs: one row kernel behind that GEMM adds up its partial products (and the experts' rows), norms them, adds
+to the stream and writes the next sublayer's input. Feed-forward activations run in the epilogue of the up-projection. Latent
+attention: prompts expand keys and values from the latents; decoding absorbs the key expansion into the query and applies the
+value expansion to the attention output, so only latent rows are read. Grouped-query attention caches normed, rotated keys and
+mixed values; experts run on tokens grouped by expert without a host synchronisation.
 
 Forward only: the stacks are served (rollout, log-probs), not trained.
 """
@@ -54,13 +58,15 @@ class MixerStackModel:
         self._rope_len = 0
         self._rope: dict = {}
         self._ensure_rope(max_positions or 2048)
+        self._zero_sinks: dict = {}
         self._weights = [self._layer_weights(i) for i in range(len(self.spec.layers))]
         self._final_norm = self._norm("final.norm")
+        self._embed_norm = self._norm("embed.norm") if self.spec.embedding_norm else None
 
     # ------------------------------------------------------------------------------------ weights and tables
-    def _norm(self, name: str) -> tuple:
+    def _norm(self, name: str):
         P = self.params
-        return (P[name + ".alpha"], P[name], P[name + ".b"])
+        return P[name] if self.spec.norm == "rms" else (P[name + ".alpha"], P[name], P[name + ".b"])
 
     def _layer_weights(self, i: int) -> dict:
         layer = self.spec.layers[i]
@@ -71,8 +77,12 @@ class MixerStackModel:
         if m.kind == "latent_attention":
             out["uk"] = out["ukv"][: m.heads * m.dim].view(m.heads, m.dim, m.kv_rank)
             out["uv"] = out["ukv"][m.heads * m.dim :].view(m.heads, m.vdim, m.kv_rank)
+        elif m.kind == "attention":
+            if m.heads not in self._zero_sinks:
+                self._zero_sinks[m.heads] = torch.zeros(m.heads, dtype=self.params.flat.dtype, device=self.device)
+            out["sink"] = self._zero_sinks[m.heads] if m.zero_sink else None
         if layer.mlp is not None:
-            out.update(norm2=self._norm(p + "norm2"), up=W["mlp.up"], down=W["mlp.down"])
+            out.update(norm2=self._norm(p + "norm2"), **{k: v for k, v in W.items() if k.startswith("mlp.")})
         return out
 
     def _ensure_rope(self, n: int) -> None:
@@ -118,12 +128,47 @@ class MixerStackModel:
         oc = X.latent_attention_decode(qa, cache.pages(i), block_table, ctx_len, m.kv_rank, m.window, m.scale, W["sink"])
         return X.headwise_linear(oc, W["uv"], False, gate).view(S, m.heads * m.vdim)
 
+    def _grouped_in(self, i, W, m, h, pos, pages, slot_map, want_rows: bool, first: dict):
+        """Queries and the row [keys | values]; ``first`` carries the values of the stack's first value-mixing layer."""
+        p = X.linear_act(h, W["in"])
+        cos, sin = self._rope[m.rot.key()]
+        v_first = None
+        if m.v_mix:
+            if i == self.spec.value_source:
+                a = (m.heads + m.kv_heads) * m.dim
+                first["values"] = p[:, a : a + m.kv_heads * m.vdim]
+            else:
+                v_first = first["values"]
+        return X.qkv_prep(p, W["q.norm"], W["k.norm"], self.spec.norm_eps, pos, cos, sin, m.heads, m.kv_heads, m.vdim, v_first,
+                          W["vmix"] if v_first is not None else None, pages, slot_map, want_rows)
+
+    def _grouped_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict], first: dict):
+        pages = pc.cache.pages(i) if pc is not None else None
+        q, rows = self._grouped_in(i, W, m, h, batch.positions, pages, pc.slot_map if pc is not None else None, portion is None, first)
+        cu_k = batch.cu_seqlens
+        if portion is not None:
+            lo, cu_k, total = portion[m.window]
+            rows = X.gather_pages(pages, pc.block_table, cu_k, lo, total)
+        k, v = rows[:, : m.kv_heads * m.dim].unflatten(1, (m.kv_heads, m.dim)), rows[:, m.kv_heads * m.dim :].unflatten(1, (m.kv_heads, m.vdim))
+        return X.grouped_attention_prefill(q, k, v, batch.cu_seqlens, cu_k, m.window, m.scale, m.softcap, W["sink"]).flatten(1)
+
+    def _grouped_decode(self, i, W, m, h, pos, slot_map, ctx_len, block_table, cache, first: dict):
+        q, _ = self._grouped_in(i, W, m, h, pos, cache.pages(i), slot_map, False, first)
+        return X.grouped_attention_decode(q, cache.pages(i), block_table, ctx_len, m.kv_heads, m.vdim, m.window, m.scale, m.softcap, W["sink"]).flatten(1)
+
     def _mlstm_in(self, W, m, h):
         return X.linear_split(h, W["in"], 2 * m.heads * (m.dim + m.vdim))
 
     # ------------------------------------------------------------------------------------ layer loop
     def _run(self, ids: torch.Tensor, mix: Callable) -> torch.Tensor:
         """Embedding, layers, final norm; ``mix(i, weights, mixer, h)`` is the layer's mixer up to its output projection."""
+        return (self._run_output_norms if self.spec.norm_on == "output" else self._run_input_norms)(ids, mix)
+
+    def _layer_done(self, i: int, x: torch.Tensor) -> None:
+        if self.stats_hook is not None:
+            self.stats_hook(f"layers.{i}.residual", x)
+
+    def _run_input_norms(self, ids: torch.Tensor, mix: Callable) -> torch.Tensor:
         layers, Ws = self.spec.layers, self._weights
         x, h = X.embed_dyt(ids, self.params["embed"], self.spec.embedding_scale, *Ws[0]["norm1"])
         for i, layer in enumerate(layers):
@@ -134,9 +179,27 @@ class MixerStackModel:
                 h = X.linear_residual_(o, W["o"], x, nxt)
             else:
                 h = X.linear_residual_(o, W["o"], x, W["norm2"])
-                h = X.linear_residual_(X.linear_act(h, W["up"], layer.mlp.act), W["down"], x, nxt)
-            if self.stats_hook is not None:
-                self.stats_hook(f"layers.{i}.residual", x)
+                h = X.linear_residual_(X.linear_act(h, W["mlp.up"], layer.mlp.act), W["mlp.down"], x, nxt)
+            self._layer_done(i, x)
+        return h
+
+    def _run_output_norms(self, ids: torch.Tensor, mix: Callable) -> torch.Tensor:
+        spec, layers = self.spec, self.spec.layers
+        eps, mult = spec.norm_eps, spec.residual_mult
+        x, h = X.embed_rms(ids, self.params["embed"], spec.embedding_scale, self._embed_norm, eps)
+        for i, layer in enumerate(layers):
+            W, f = self._weights[i], layer.mlp
+            nxt = self._final_norm if i + 1 == len(layers) else None   # the last sublayer's kernel applies the final norm
+            h = X.residual_rms_(x, X.linear_partial(mix(i, W, layer.mixer, h), W["o"]), W["norm1"], eps, mult, nxt if f is None else None)
+            if f is not None and f.kind == "moe":
+                act, tail = X.gated_up_split(h, W["mlp.in"], 2 * f.shared_ff)     # tail: router logits, then the shared expert's gate
+                plan = X.expert_dispatch(h, tail, f.experts, f.top, f.renormalize)
+                rows = X.expert_down(X.expert_up(plan, W["mlp.experts.in"], f.ff), W["mlp.experts.down"], plan)
+                y, gate = (X.linear_partial(act, W["mlp.shared.down"]), tail[:, f.experts]) if f.shared_ff else (None, None)
+                h = X.residual_rms_(x, y, W["norm2"], eps, mult, nxt, (rows, plan.slot), gate)
+            elif f is not None:
+                h = X.residual_rms_(x, X.linear_partial(X.gated_up(h, W["mlp.in"]), W["mlp.down"]), W["norm2"], eps, mult, nxt)
+            self._layer_done(i, x)
         return h
 
     @torch.no_grad()
@@ -150,16 +213,19 @@ class MixerStackModel:
         portion = None
         if any(starts):
             portion = {}
-            for w in {l.mixer.window for l in self.spec.layers if l.mixer.kind == "latent_attention"}:
+            for w in {l.mixer.window for l in self.spec.layers if l.mixer.page_width}:
                 lo = [max(0, s - w + 1) if w > 0 else 0 for s in starts]
                 cu = torch.zeros(len(lens) + 1, dtype=torch.int32)
                 cu[1:] = torch.cumsum(torch.tensor([s + n - a for s, n, a in zip(starts, lens, lo)], dtype=torch.int32), 0)
                 portion[w] = (torch.tensor(lo, dtype=torch.int32).to(self.device), cu.to(self.device), int(cu[-1]))
-        fresh = torch.tensor([int(s == 0) for s in starts], dtype=torch.int32).to(self.device) if pc is not None else None
+        fresh = torch.tensor([int(s == 0) for s in starts], dtype=torch.int32).to(self.device) if pc is not None and self.spec.recurrent else None
+        first: dict = {}
 
         def mix(i, W, m, h):
             if m.kind == "latent_attention":
                 return self._attention_prefill(i, W, m, h, batch, pc, portion)
+            if m.kind == "attention":
+                return self._grouped_prefill(i, W, m, h, batch, pc, portion, first)
             p, gates = self._mlstm_in(W, m, h)
             return X.mlstm_prefill(p, gates, W["i.b"], W["f.b"], m.gate_cap, W["norm"], self.spec.norm_eps, m.dim, batch.cu_seqlens,
                                    pc.cache.state(i) if pc is not None else None, pc.slots if pc is not None else None, fresh, not any(starts))
@@ -169,10 +235,13 @@ class MixerStackModel:
     @torch.no_grad()
     def decode_hidden(self, tok, pos, slot_map, ctx_len, active, block_table, cache) -> torch.Tensor:
         """One token for every slot (static shapes, capturable); inactive slots leave cache and state untouched."""
+        first: dict = {}
 
         def mix(i, W, m, h):
             if m.kind == "latent_attention":
                 return self._attention_decode(i, W, m, h, pos, slot_map, ctx_len, block_table, cache)
+            if m.kind == "attention":
+                return self._grouped_decode(i, W, m, h, pos, slot_map, ctx_len, block_table, cache, first)
             p, gates = self._mlstm_in(W, m, h)
             return X.mlstm_decode(p, gates, W["i.b"], W["f.b"], m.gate_cap, W["norm"], self.spec.norm_eps, m.dim, cache.state(i), active)
 
@@ -180,7 +249,7 @@ class MixerStackModel:
 
     # ------------------------------------------------------------------------------------ heads
     def logits(self, h: torch.Tensor) -> torch.Tensor:
-        return X.linear_act(h, self.params.lm_head_weight)
+        return X.linear_softcap(h, self.params.lm_head_weight, self.spec.logit_softcap)
 
     def forward_logits(self, batch: PackedBatch) -> torch.Tensor:
         return self.logits(self.forward_hidden(batch))
@@ -196,8 +265,18 @@ class MixerStackModel:
             if positions is not None:
                 h = h.index_select(0, positions)
                 labels = position_labels if position_labels is not None else labels.index_select(0, positions)
-            if h.is_cuda and (h.dtype != torch.bfloat16 or h.shape[1] % 8 or self.cfg.vocab_size % 8):   # outside the fused head's sizes
-                logp = torch.log_softmax(X.linear_act(h, self.params.lm_head_weight, out_f32=True) / max(temperature, 1e-8), -1)
-                return logp.gather(-1, labels.unsqueeze(-1)).squeeze(-1), -(logp.exp() * logp).sum(-1)
-            lp, ent, _ = F.lmhead_logprob_entropy(h, self.params.lm_head_weight, labels, temperature)
+            cap, w = self.spec.logit_softcap, self.params.lm_head_weight
+            # the fused head has no soft cap and serves bf16 sizes that are multiples of 8
+            if cap > 0 or (h.is_cuda and (h.dtype != torch.bfloat16 or h.shape[1] % 8 or self.cfg.vocab_size % 8)):
+                rows = max(256, (1 << 28) // self.cfg.vocab_size)
+                parts = [self._row_logprobs(h[a : a + rows], w, labels[a : a + rows], cap, temperature) for a in range(0, h.shape[0], rows)]
+                return torch.cat([p[0] for p in parts]), torch.cat([p[1] for p in parts])
+            lp, ent, _ = F.lmhead_logprob_entropy(h, w, labels, temperature)
             return lp, ent
+
+    @staticmethod
+    def _row_logprobs(h, w, labels, cap: float, temperature: float):
+        z = X.linear_act(h, w, out_f32=True)
+        z = cap * torch.tanh(z / cap) if cap > 0 else z
+        logp = torch.log_softmax(z / max(temperature, 1e-8), -1)
+        return logp.gather(-1, labels.unsqueeze(-1)).squeeze(-1), -(logp.exp() * logp).sum(-1)

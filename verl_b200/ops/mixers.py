@@ -319,6 +319,75 @@ def latent_attention_decode(q, pages, block_table, ctx_len, kv_rank: int, window
     return out
 
 
+# ----------------------------------------------------------------------------------------------- grouped-query attention
+def qkv_prep(p, q_norm, k_norm, eps: float, positions, cos, sin, heads: int, kv_heads: int, vdim: int, v_first=None, vmix=None, pages=None, slots=None,
+             want_rows: bool = False):
+    """``p`` [T, q | k | v]: RMS norm per query and key head, rotation of their first ``2 * cos.shape[1]`` dimensions (pairs 2i,
+    2i + 1), and values mixed as ``(1 - vmix) v + vmix v_first`` when ``v_first`` [T, kv_heads * vdim] is given. Returns the queries
+    [T, heads, dim]; the row [keys | values] is appended to ``pages`` [blocks, block_size, kv_heads * (dim + vdim)] at ``slots``
+    (negative: skipped) and / or returned."""
+    dim = q_norm.numel()
+    if p.is_cuda:
+        return _ops().qkv_prep(p, q_norm, k_norm, float(eps), positions, cos, sin, int(heads), int(kv_heads), int(vdim), v_first, vmix, pages, slots,
+                               bool(want_rows))
+    T, a, b = p.shape[0], heads * dim, (heads + kv_heads) * dim
+    f = p.float()
+    q = _rotate(_rms(f[:, :a].view(T, heads, dim), q_norm, eps), positions, cos, sin).to(p.dtype)
+    k = _rotate(_rms(f[:, a:b].view(T, kv_heads, dim), k_norm, eps), positions, cos, sin)
+    v = f[:, b : b + kv_heads * vdim]
+    if v_first is not None:
+        v = (1.0 - vmix.float()) * v + vmix.float() * v_first.float()
+    row = torch.cat([k.flatten(1), v], -1).to(p.dtype)
+    if pages is not None:
+        ok = slots >= 0
+        at, bs = slots[ok], pages.shape[1]
+        pages[at // bs, at % bs] = row[ok]
+    return q, (row if want_rows else row[:0])
+
+
+def _soft_cap(s: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(s / cap) if cap > 0 else s
+
+
+def grouped_attention_prefill(q, k, v, cu_q, cu_k, window: int, scale: float, softcap: float = 0.0, sink=None) -> torch.Tensor:
+    """Causal attention of packed prompts: ``q`` [T, H, d], ``k`` [Tk, G, d], ``v`` [Tk, G, e] (query head h reads key head h // (H / G));
+    scores ``softcap * tanh(q k scale / softcap)``; ``cu_q`` / ``cu_k`` / ``window`` / ``sink`` as in ``latent_attention_prefill``."""
+    if q.is_cuda:
+        return _ops().grouped_attn_prefill(q, k, v, cu_q, cu_k, sink, int(window), float(scale), float(softcap))
+    out = torch.empty(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype)
+    n = q.shape[1] // k.shape[1]
+    cq, ck = cu_q.tolist(), cu_k.tolist()
+    for b in range(len(cq) - 1):
+        qs, ks = slice(cq[b], cq[b + 1]), slice(ck[b], ck[b + 1])
+        nq, nk = cq[b + 1] - cq[b], ck[b + 1] - ck[b]
+        s = _soft_cap(torch.einsum("qhd,khd->hqk", q[qs].float(), k[ks].float().repeat_interleave(n, 1)) * scale, softcap)
+        dist = torch.arange(nk - nq, nk)[:, None] - torch.arange(nk)[None, :]
+        hide = (dist < 0) | ((dist >= window) if window > 0 else torch.zeros_like(dist, dtype=torch.bool))
+        w = _sink_softmax(s.masked_fill(hide, float("-inf")), sink)
+        out[qs] = torch.einsum("hqk,khd->qhd", w, v[ks].float().repeat_interleave(n, 1)).to(q.dtype)
+    return out
+
+
+def grouped_attention_decode(q, pages, block_table, ctx_len, kv_heads: int, vdim: int, window: int, scale: float, softcap: float = 0.0,
+                             sink=None) -> torch.Tensor:
+    """One query per sequence, ``q`` [S, H, d], against cached rows [keys | values] (``qkv_prep``). Returns [S, H, vdim]; sequences
+    with ``ctx_len`` 0 give zeros."""
+    if q.is_cuda:
+        return _ops().grouped_attn_decode(q, pages, block_table, ctx_len, sink, int(kv_heads), int(vdim), int(window), float(scale), float(softcap))
+    out = torch.zeros(q.shape[0], q.shape[1], vdim, dtype=q.dtype)
+    bs, G, d = pages.shape[1], kv_heads, q.shape[2]
+    for b, n in enumerate(ctx_len.tolist()):
+        if n <= 0:
+            continue
+        at = torch.arange(max(0, n - window) if window > 0 else 0, n)
+        rows = pages[block_table[b, at // bs].long(), at % bs].float()
+        k, v = rows[:, : G * d].view(-1, G, d), rows[:, G * d :].view(-1, G, vdim)
+        s = _soft_cap(torch.einsum("gnd,kgd->gnk", q[b].float().view(G, -1, d), k).flatten(0, 1) * scale, softcap)
+        w = _sink_softmax(s, sink)
+        out[b] = torch.einsum("gnk,kge->gne", w.view(G, -1, len(at)), v).flatten(0, 1).to(q.dtype)
+    return out
+
+
 # ----------------------------------------------------------------------------------------------- mLSTM
 def _mlstm_parts(p, gates, ib, fb, cap: float, d: int, e: int):
     T, H = p.shape[0], ib.numel()
