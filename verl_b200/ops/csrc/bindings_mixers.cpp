@@ -303,6 +303,286 @@ Tensor latent_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& bl
   return out;
 }
 
+// ---- stacks with RMS norms on the sublayer outputs
+std::tuple<Tensor, Tensor> embed_rms(const Tensor& ids, const Tensor& w, double scale, const Tensor& nw, double eps) {
+  const int dt = dtype_of(w);
+  const c10::cuda::CUDAGuard guard(w.device());
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && w.dim() == 2 && w.is_contiguous() && nw.numel() == w.size(1), "embed_rms");
+  same(w, nw, "embed_rms");
+  const int T = (int)ids.numel(), W = (int)w.size(1);
+  Tensor x = at::empty({T, W}, w.options().dtype(at::kFloat)), h = at::empty({T, W}, w.options());
+  verl_count_launches(1);
+  CHECK_RC(vb_embed_rms(dt, lptr(ids), w.data_ptr(), (float)scale, nw.data_ptr(), (float)eps, x.data_ptr<float>(), h.data_ptr(), T, W, (int)w.size(0), cur_stream()),
+           "vb_embed_rms");
+  return {x, h};
+}
+
+// a w^T for a row kernel: fp32 partial products [splits, M, N] where the GEMM splits K, else [M, N] in a's type.
+Tensor linear_partial(const Tensor& a, const Tensor& w) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  const int dt = dtype_of(a);
+  same(a, w, "linear_partial");
+  TORCH_CHECK(a.dim() == 2 && w.dim() == 2 && a.stride(1) == 1 && w.stride(1) == 1 && a.size(1) == w.size(1), "linear_partial: a [M, K], w [N, K]");
+  const int M = (int)a.size(0), K = (int)a.size(1), N = (int)w.size(0);
+  if (dt == 1 && M > 0 && M <= 1024 && N % 8 == 0 && K % 8 == 0 && a.stride(0) % 8 == 0 && w.stride(0) % 8 == 0) {
+    const int s = vb_gemm_skinny_splits(M, N, K);
+    if (s > 1) {
+      Tensor ws = at::empty({s, M, N}, a.options().dtype(at::kFloat));
+      const int rc = vb_gemm_skinny(a.data_ptr(), w.data_ptr(), nullptr, nullptr, M, N, K, a.stride(0), w.stride(0), 0, s, ws.data_ptr<float>(), 0, 1, cur_stream());
+      if (rc == 0) {
+        verl_count_launches(1);
+        return ws;
+      }
+      TORCH_CHECK(rc < 0, "linear_partial failed with code ", rc);
+    }
+  }
+  return linear_act(a, w, false, false);
+}
+
+Tensor linear_softcap(const Tensor& a, const Tensor& w, double cap) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  TORCH_CHECK(cap > 0, "linear_softcap: cap > 0");
+  Tensor d = at::empty({a.size(0), w.size(0)}, a.options());
+  VbEpiArgs e{};
+  e.mode = VB_EPI_SOFTCAP;
+  e.cap = (float)cap;
+  e.D = d.data_ptr(); e.ldd = d.stride(0);
+  run_gemm(a, w, e);
+  return d;
+}
+
+// x += mult * rms_norm(Y) nw (see VbResidRms); returns the new stream, or its norm with `next`, in nw's type.
+Tensor residual_rms_(Tensor x, const OptTensor& y, const Tensor& nw, double eps, double mult, const OptTensor& next, const OptTensor& rows, const OptTensor& slot,
+                     const OptTensor& gate) {
+  CHECK_F32(x);
+  const int dt = dtype_of(nw);
+  const c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && nw.numel() == x.size(1) && (y.has_value() || rows.has_value()), "residual_rms_: x [T, W]");
+  VbResidRms p{};
+  p.T = (int)x.size(0); p.W = (int)x.size(1);
+  p.x = x.data_ptr<float>(); p.nw = nw.data_ptr(); p.eps = (float)eps; p.mult = (float)mult;
+  if (y.has_value()) {
+    const bool parts = y->dim() == 3;
+    TORCH_CHECK(y->is_cuda() && y->size(-1) == p.W && y->size(-2) == p.T && y->stride(-1) == 1, "residual_rms_: y");
+    if (parts) CHECK_F32(*y); else same(nw, *y, "residual_rms_");
+    p.y = y->data_ptr(); p.y_f32 = parts; p.splits = parts ? (int)y->size(0) : 1; p.split_stride = parts ? y->stride(0) : 0; p.ldy = y->stride(-2);
+  }
+  if (rows.has_value()) {
+    same(nw, *rows, "residual_rms_");
+    TORCH_CHECK(slot.has_value() && rows->dim() == 2 && rows->size(1) == p.W && rows->stride(1) == 1 && slot->dim() == 2 && slot->size(0) == p.T, "residual_rms_: rows");
+    CHECK_I32(*slot);
+    p.rows = rows->data_ptr(); p.ldr = rows->stride(0); p.slot = slot->data_ptr<int>(); p.top = (int)slot->size(1);
+  }
+  if (gate.has_value()) {
+    CHECK_F32(*gate);
+    TORCH_CHECK(gate->dim() == 1 && gate->numel() == p.T, "residual_rms_: gate [T]");
+    p.gate = gate->data_ptr<float>(); p.ldgate = gate->stride(0);
+  }
+  if (next.has_value()) { same(nw, *next, "residual_rms_"); TORCH_CHECK(next->numel() == p.W); p.next = next->data_ptr(); }
+  Tensor h = at::empty({p.T, p.W}, nw.options());
+  p.h = h.data_ptr();
+  verl_count_launches(1);
+  CHECK_RC(vb_residual_rms(dt, &p, cur_stream()), "vb_residual_rms");
+  return h;
+}
+
+Tensor gated_silu_rows(const Tensor& gu, const float* row_scale) {
+  const int dt = dtype_of(gu);
+  TORCH_CHECK(gu.dim() == 2 && gu.stride(1) == 1 && gu.size(1) % 2 == 0, "gated_silu: [T, 2 I]");
+  Tensor out = at::empty({gu.size(0), gu.size(1) / 2}, gu.options());
+  verl_count_launches(1);
+  CHECK_RC(vb_gated_silu(dt, gu.data_ptr(), gu.stride(0), row_scale, out.data_ptr(), (int)out.size(0), (int)out.size(1), cur_stream()), "vb_gated_silu");
+  return out;
+}
+Tensor gated_silu(const Tensor& gu) {
+  const c10::cuda::CUDAGuard guard(gu.device());
+  return gated_silu_rows(gu, nullptr);
+}
+
+// Router and expert-grouped copies of the tokens: (x [rows, W], slot [T, k], score per row, expert per 128-row tile, number of tiles).
+std::tuple<Tensor, Tensor, Tensor, Tensor, Tensor> expert_dispatch(const Tensor& h, const Tensor& z, int64_t E, int64_t k, bool renorm) {
+  const int dt = dtype_of(h);
+  CHECK_F32(z);
+  const c10::cuda::CUDAGuard guard(h.device());
+  const int64_t T = h.size(0), W = h.size(1);
+  TORCH_CHECK(h.dim() == 2 && h.stride(1) == 1 && z.dim() == 2 && z.stride(1) == 1 && z.size(0) == T && z.size(1) >= E && k >= 1 && k <= E, "expert_dispatch");
+  const int64_t tiles = std::max<int64_t>(1, (T * k + 127) / 128 + std::min<int64_t>(E, T * k));
+  const auto i32 = h.options().dtype(at::kInt), f32 = h.options().dtype(at::kFloat);
+  Tensor counts = at::zeros({E}, i32), expert = at::empty({T, k}, i32), rank = at::empty({T, k}, i32), slot = at::empty({T, k}, i32);
+  Tensor score = at::empty({T, k}, f32), row_scale = at::empty({tiles * 128}, f32), tile_expert = at::empty({tiles}, i32), num_tiles = at::empty({1}, i32);
+  Tensor x = at::empty({tiles * 128, W}, h.options());
+  if (T == 0) { num_tiles.zero_(); return {x, slot, row_scale, tile_expert, num_tiles}; }
+  verl_count_launches(2);
+  CHECK_RC(vb_expert_route(z.data_ptr<float>(), z.stride(0), (int)T, (int)E, (int)k, renorm, score.data_ptr<float>(), expert.data_ptr<int>(), rank.data_ptr<int>(),
+                           counts.data_ptr<int>(), cur_stream()), "vb_expert_route");
+  CHECK_RC(vb_expert_place(dt, h.data_ptr(), h.stride(0), score.data_ptr<float>(), expert.data_ptr<int>(), rank.data_ptr<int>(), counts.data_ptr<int>(), (int)T, (int)E,
+                           (int)k, (int)W, x.data_ptr(), row_scale.data_ptr<float>(), slot.data_ptr<int>(), tile_expert.data_ptr<int>(), num_tiles.data_ptr<int>(),
+                           (int)tiles, cur_stream()), "vb_expert_place");
+  return {x, slot, row_scale, tile_expert, num_tiles};
+}
+
+// out[rows, N] = a w_e^T per 128-row tile, w [E, N, K]: tensor cores where the sizes allow.
+Tensor expert_linear(const Tensor& a, const Tensor& w, const Tensor& tile_expert, const Tensor& num_tiles) {
+  const int dt = dtype_of(a);
+  same(a, w, "expert_linear");
+  CHECK_I32(tile_expert);
+  CHECK_I32(num_tiles);
+  TORCH_CHECK(a.dim() == 2 && a.stride(1) == 1 && a.size(0) == tile_expert.numel() * 128 && w.dim() == 3 && w.is_contiguous() && w.size(2) == a.size(1), "expert_linear");
+  const c10::cuda::CUDAGuard guard(a.device());
+  const int rows = (int)a.size(0), N = (int)w.size(1), K = (int)w.size(2), E = (int)w.size(0);
+  Tensor d = at::empty({rows, N}, a.options());
+  verl_count_launches(1);
+  int rc = -1;
+  if (dt == 1 && K % 8 == 0)
+    rc = vb_gemm_grouped(1, a.data_ptr(), w.data_ptr(), d.data_ptr(), rows, rows, N, K, a.stride(0), K, N, 0, 0, E, tile_expert.data_ptr<int>(),
+                         num_tiles.data_ptr<int>(), nullptr, cur_stream());
+  if (rc < 0) {
+    VbEpiArgs e{};
+    e.mode = VB_EPI_STORE;
+    e.D = d.data_ptr(); e.ldd = N;
+    rc = vb_gemm_simt_grouped(dt, a.data_ptr(), w.data_ptr(), rows, N, K, a.stride(0), tile_expert.data_ptr<int>(), num_tiles.data_ptr<int>(), &e, cur_stream());
+  }
+  CHECK_RC(rc, "expert_linear");
+  return d;
+}
+
+// act[rows, I] = silu(s g) * (s u), [g | u] = x w_e^T, w [E, 2 I, K], s = scale[row].
+Tensor expert_up(const Tensor& x, const Tensor& w, const Tensor& scale, const Tensor& tile_expert, const Tensor& num_tiles) {
+  CHECK_F32(scale);
+  CHECK_I32(tile_expert);
+  CHECK_I32(num_tiles);
+  same(x, w, "expert_up");
+  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && scale.numel() == x.size(0) && x.size(0) == tile_expert.numel() * 128 && w.dim() == 3 && w.is_contiguous() &&
+              w.size(2) == x.size(1) && w.size(1) % 2 == 0, "expert_up");
+  const c10::cuda::CUDAGuard guard(x.device());
+  const int rows = (int)x.size(0), I = (int)w.size(1) / 2, K = (int)w.size(2);
+  if (dtype_of(x) == 1) {
+    Tensor act = at::empty({rows, I}, x.options());
+    const int rc = vb_gemm_grouped_swiglu(x.data_ptr(), w.data_ptr(), act.data_ptr(), rows, I, K, x.stride(0), I, scale.data_ptr<float>(), (int)w.size(0),
+                                          tile_expert.data_ptr<int>(), num_tiles.data_ptr<int>(), cur_stream());
+    if (rc >= 0) {
+      verl_count_launches(1);
+      CHECK_RC(rc, "expert_up");
+      return act;
+    }
+  }
+  return gated_silu_rows(expert_linear(x, w, tile_expert, num_tiles), scale.data_ptr<float>());
+}
+
+// p [T, q | k | v]; see VbQkvPrep. Returns (queries [T, H, dim], rows [T or 0, G (dim + vdim)]).
+std::tuple<Tensor, Tensor> qkv_prep(const Tensor& p, const Tensor& qn, const Tensor& kn, double eps, const Tensor& pos, const Tensor& cs, const Tensor& sn, int64_t H,
+                                    int64_t G, int64_t vdim, const OptTensor& vfirst, const OptTensor& vmix, const OptTensor& pages, const OptTensor& slot,
+                                    bool want_rows) {
+  const int dt = dtype_of(p);
+  CHECK_I32(pos);
+  CHECK_F32(cs);
+  CHECK_F32(sn);
+  same(p, qn, "qkv_prep");
+  same(p, kn, "qkv_prep");
+  const int64_t T = p.size(0), dim = qn.numel(), width = G * (dim + vdim);
+  TORCH_CHECK(p.dim() == 2 && p.stride(1) == 1 && p.size(1) >= (H + G) * dim + G * vdim && kn.numel() == dim && pos.numel() == T && cs.is_contiguous() &&
+              sn.is_contiguous() && cs.dim() == 2 && 2 * cs.size(1) <= dim, "qkv_prep: sizes");
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor q = at::empty({T, H, dim}, p.options()), rows = at::empty({want_rows ? T : 0, width}, p.options());
+  VbQkvPrep a{};
+  a.p = p.data_ptr(); a.ldp = p.stride(0); a.qn = qn.data_ptr(); a.kn = kn.data_ptr(); a.pos = pos.data_ptr<int>();
+  a.cos_t = cs.data_ptr<float>(); a.sin_t = sn.data_ptr<float>(); a.half = (int)cs.size(1); a.max_pos = (int)cs.size(0);
+  if (vfirst.has_value()) {
+    same(p, *vfirst, "qkv_prep");
+    TORCH_CHECK(vmix.has_value() && vmix->numel() == 1 && vfirst->dim() == 2 && vfirst->size(0) == T && vfirst->size(1) == G * vdim && vfirst->stride(1) == 1, "qkv_prep: v_first");
+    same(p, *vmix, "qkv_prep");
+    a.vfirst = vfirst->data_ptr(); a.ldvf = vfirst->stride(0); a.vmix = vmix->data_ptr();
+  }
+  a.q = q.data_ptr();
+  a.ldr = width;
+  if (want_rows) a.rows = rows.data_ptr();
+  a.block_size = 1;
+  if (pages.has_value()) {
+    same(p, *pages, "qkv_prep");
+    TORCH_CHECK(pages->dim() == 3 && pages->size(2) == width && pages->stride(2) == 1 && pages->stride(1) == width && slot.has_value() && slot->is_cuda() &&
+                slot->scalar_type() == at::kLong && slot->is_contiguous() && slot->numel() == T, "qkv_prep: pages [blocks, block_size, kv_heads (dim + vdim)]");
+    a.pages = pages->data_ptr(); a.page_stride = pages->stride(0); a.block_size = (int)pages->size(1); a.num_slots = pages->size(0) * pages->size(1); a.slot = lptr(*slot);
+  }
+  a.T = (int)T; a.H = (int)H; a.G = (int)G; a.dim = (int)dim; a.vdim = (int)vdim; a.eps = (float)eps;
+  verl_count_launches(1);
+  CHECK_RC(vb_qkv_prep(dt, &a, cur_stream()), "vb_qkv_prep");
+  return {q, rows};
+}
+
+// Prompt attention: q [T, H, d], k [Tk, G, d], v [Tk, G, e] (strided views), cu_q / cu_k int32 [B + 1].
+Tensor grouped_attn_prefill(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& cu_q, const Tensor& cu_k, const OptTensor& sink, int64_t window,
+                            double scale, double softcap) {
+  const int dt = dtype_of(q);
+  CHECK_I32(cu_q);
+  CHECK_I32(cu_k);
+  same(q, k, "grouped_attn_prefill");
+  same(q, v, "grouped_attn_prefill");
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.stride(2) == 1 && k.stride(2) == 1 && v.stride(2) == 1 && q.size(2) == k.size(2) && k.size(1) > 0 &&
+              q.size(1) % k.size(1) == 0 && v.size(1) == k.size(1) && v.size(0) == k.size(0) && cu_q.numel() == cu_k.numel(), "grouped_attn_prefill");
+  const c10::cuda::CUDAGuard guard(q.device());
+  VbLatentAttn a{};
+  a.q = q.data_ptr(); a.ldq = q.stride(0); a.hq = (int)q.stride(1);
+  a.ku = k.data_ptr(); a.ku_row = k.stride(0); a.ku_head = (int)k.stride(1);
+  a.v = v.data_ptr(); a.v_row = v.stride(0); a.v_head = (int)v.stride(1);
+  a.cu_q = cu_q.data_ptr<int>(); a.cu_k = cu_k.data_ptr<int>();
+  a.T = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)q.size(2); a.dv = (int)v.size(2); a.B = (int)cu_q.numel() - 1;
+  a.window = (int)window; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / k.size(1));
+  if (sink.has_value()) { same(q, *sink, "grouped_attn_prefill"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
+  Tensor out = at::empty({q.size(0), q.size(1), v.size(2)}, q.options());
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  verl_count_launches(1);
+  int rc = dt == 1 && a.T > 0 ? vb_latent_prefill(&a, (int)k.size(0), cur_stream()) : -1;
+  if (rc < 0) rc = vb_latent_attn_simt(dt, &a, cur_stream());
+  CHECK_RC(rc, "grouped_attn_prefill");
+  return out;
+}
+
+// Decode attention: q [S, H, d], pages [blocks, block_size, G (d + vdim)] with rows [keys | values].
+Tensor grouped_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& block_table, const Tensor& ctx_len, const OptTensor& sink, int64_t G, int64_t vdim,
+                           int64_t window, double scale, double softcap) {
+  const int dt = dtype_of(q);
+  same(q, pages, "grouped_attn_decode");
+  CHECK_I32(block_table);
+  CHECK_I32(ctx_len);
+  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && pages.dim() == 3 && pages.stride(2) == 1 && G > 0 && q.size(1) % G == 0 && pages.size(2) == G * (q.size(2) + vdim) &&
+              block_table.size(0) == q.size(0) && ctx_len.numel() == q.size(0), "grouped_attn_decode");
+  const c10::cuda::CUDAGuard guard(q.device());
+  VbLatentAttn a{};
+  const int64_t d = q.size(2);
+  a.q = q.data_ptr(); a.ldq = q.stride(0); a.hq = (int)q.stride(1);
+  char* base = reinterpret_cast<char*>(pages.data_ptr());
+  a.ku = base; a.ku_row = pages.stride(1); a.ku_head = (int)d;
+  a.kr = base;
+  a.v = base + G * d * pages.element_size(); a.v_row = pages.stride(1); a.v_head = (int)vdim;
+  a.block_table = block_table.data_ptr<int>(); a.max_blocks = (int)block_table.size(1); a.block_size = (int)pages.size(1); a.page_stride = pages.stride(0);
+  a.ctx_len = ctx_len.data_ptr<int>();
+  a.T = a.B = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)d; a.dv = (int)vdim;
+  a.window = (int)window; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / G);
+  if (sink.has_value()) { same(q, *sink, "grouped_attn_decode"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
+  Tensor out = at::empty({q.size(0), q.size(1), vdim}, q.options());
+  a.out = out.data_ptr(); a.ldo = out.stride(0);
+  if (dt == 1) {
+    const int64_t all = (int64_t)a.max_blocks * a.block_size;
+    const int ns = vb_grouped_decode_splits(&a, (int)(window > 0 ? std::min<int64_t>(window + 64, all) : all));
+    if (ns > 0) {
+      Tensor po, ml;
+      if (ns > 1) {
+        po = at::empty({a.B, a.H, ns, vdim}, q.options().dtype(at::kFloat));
+        ml = at::empty({a.B, a.H, ns, 2}, q.options().dtype(at::kFloat));
+      }
+      const int rc = vb_grouped_decode(&a, pages.size(0), ns, ns > 1 ? po.data_ptr<float>() : nullptr, ns > 1 ? ml.data_ptr<float>() : nullptr, cur_stream());
+      if (rc >= 0) {
+        verl_count_launches(ns > 1 ? 2 : 1);
+        CHECK_RC(rc, "vb_grouped_decode");
+        return out;
+      }
+    }
+  }
+  verl_count_launches(1);
+  CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
+  return out;
+}
+
 struct MlstmShape { int dt; int64_t T, H, d, e; };
 MlstmShape mlstm_check(const Tensor& p, const Tensor& gates, const Tensor& ib, const Tensor& fb, const Tensor& norm, int64_t d) {
   MlstmShape s{dtype_of(p), p.size(0), ib.numel(), d, 0};
@@ -394,6 +674,17 @@ TORCH_LIBRARY_FRAGMENT(verl_b200, m) {
   m.def("latent_absorb", &latent_absorb);
   m.def("latent_attn_prefill", &latent_attn_prefill);
   m.def("latent_attn_decode", &latent_attn_decode);
+  m.def("embed_rms", &embed_rms);
+  m.def("linear_partial", &linear_partial);
+  m.def("linear_softcap", &linear_softcap);
+  m.def("residual_rms_", &residual_rms_);
+  m.def("gated_silu", &gated_silu);
+  m.def("expert_dispatch", &expert_dispatch);
+  m.def("expert_linear", &expert_linear);
+  m.def("expert_up", &expert_up);
+  m.def("qkv_prep", &qkv_prep);
+  m.def("grouped_attn_prefill", &grouped_attn_prefill);
+  m.def("grouped_attn_decode", &grouped_attn_decode);
   m.def("mlstm_decode", &mlstm_decode);
   m.def("mlstm_prefill", &mlstm_prefill);
 }

@@ -11,7 +11,12 @@ constexpr int SG_T = 64, SG_K = 16;
 template <typename T>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, int M, int N, int K, long long lda, long long ldb, int b_mn,
-                 long long sa, long long sb, long long sd, VbEpiArgs e) {
+                 long long sa, long long sb, long long sd, VbEpiArgs e, const int* __restrict__ tile_expert, const int* __restrict__ num_tiles) {
+  if (tile_expert != nullptr) {            // rows grouped by expert, 128 to a tile
+    const int tile = blockIdx.y * SG_T / 128;
+    if (tile >= *num_tiles) return;
+    B += static_cast<long long>(tile_expert[tile]) * N * K;
+  }
   __shared__ float As[SG_K][SG_T + 4], Bs[SG_K][SG_T + 4];
   A += blockIdx.z * sa;
   B += blockIdx.z * sb;
@@ -60,6 +65,7 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, int M, int N,
           if (e.gate != nullptr) v *= sigmoid_f(e.gate[m * e.ldg + blockIdx.z]);
           D[m * e.ldd + n] = from_f<T>(v); break;
         case VB_EPI_STORE_F32: (reinterpret_cast<float*>(e.D) + blockIdx.z * sd)[m * e.ldd + n] = v; break;
+        case VB_EPI_SOFTCAP: D[m * e.ldd + n] = from_f<T>(e.cap * tanhf(v / e.cap)); break;
         case VB_EPI_GELU: D[m * e.ldd + n] = from_f<T>(gelu_erf(v)); break;
         case VB_EPI_SPLIT:
           if (n < e.n0) D[m * e.ldd + n] = from_f<T>(v);
@@ -80,14 +86,24 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, int M, int N,
 
 using namespace vb;
 
-extern "C" int vb_gemm_simt(int dtype, const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, int b_mn, int batch,
-                            long long sa, long long sb, long long sd, const VbEpiArgs* e, cudaStream_t s) {
+static int simt_launch(int dtype, const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, int b_mn, int batch,
+                       long long sa, long long sb, long long sd, const VbEpiArgs* e, const int* tile_expert, const int* num_tiles, cudaStream_t s) {
   if (M <= 0 || N <= 0 || batch <= 0) return 0;
   dim3 grid((N + SG_T - 1) / SG_T, (M + SG_T - 1) / SG_T, batch);
   if (grid.y > 65535 || grid.z > 65535) return -1;
   if (dtype == 0)
-    gemm_simt_kernel<float><<<grid, 256, 0, s>>>((const float*)A, (const float*)B, M, N, K, lda, ldb, b_mn, sa, sb, sd, *e);
+    gemm_simt_kernel<float><<<grid, 256, 0, s>>>((const float*)A, (const float*)B, M, N, K, lda, ldb, b_mn, sa, sb, sd, *e, tile_expert, num_tiles);
   else
-    gemm_simt_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>((const __nv_bfloat16*)A, (const __nv_bfloat16*)B, M, N, K, lda, ldb, b_mn, sa, sb, sd, *e);
+    gemm_simt_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>((const __nv_bfloat16*)A, (const __nv_bfloat16*)B, M, N, K, lda, ldb, b_mn, sa, sb, sd, *e, tile_expert, num_tiles);
   return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int vb_gemm_simt(int dtype, const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, int b_mn, int batch,
+                            long long sa, long long sb, long long sd, const VbEpiArgs* e, cudaStream_t s) {
+  return simt_launch(dtype, A, B, M, N, K, lda, ldb, b_mn, batch, sa, sb, sd, e, nullptr, nullptr, s);
+}
+
+extern "C" int vb_gemm_simt_grouped(int dtype, const void* A, const void* B, int M, int N, int K, long long lda, const int* tile_expert, const int* num_tiles,
+                                    const VbEpiArgs* e, cudaStream_t s) {
+  return simt_launch(dtype, A, B, M, N, K, lda, K, 0, 1, 0, 0, 0, e, tile_expert, num_tiles, s);
 }

@@ -108,6 +108,7 @@ struct GemmParams {
   const __nv_bfloat16* fix_bias;
   int fix_out_f32, fix_accumulate;
   // EPI_SWIGLU: N counts accumulator columns (2 * I); D is the activation [M, I]
+  const float* row_scale;  // [M] factor on both halves of a row (a score that scales an expert's input), or null
   __nv_bfloat16* gu_out;  // pre-activation [M, 2I] (gate columns first), or null
   long long gu_ld;
   // EPI_MIXER
@@ -360,7 +361,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
           }
           if constexpr (EPI == EPI_SWIGLU) {
             // (k, half, row) box of 64 x 2 x BN/2: shared-memory row 2j holds gate row n0/2 + j, row 2j + 1 its up row
-            tma_load_3d(sb, &tma_b, &full_bar[stage], k0, 0, n0 >> 1);
+            tma_load_3d(sb, &tma_b, &full_bar[stage], k0, 0, b_off + (n0 >> 1));
           } else if constexpr (!B_MN) {
             tma_load_2d(sb, &tma_b, &full_bar[stage], k0, b_off + n0);
           } else {
@@ -507,7 +508,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
       float run_m = -INFINITY, run_l = 0.f, run_s = 0.f;
       long long label = -1;
       float r_lse = 0.f, r_ex = 0.f, r_glp = 0.f, r_gent = 0.f;
-      if constexpr (EPI != EPI_STORE && EPI != EPI_MIXER) {
+      if constexpr (EPI == EPI_LSE || EPI == EPI_DLOGITS) {
         if (row_ok) {
           label = p.labels[row] - p.label_offset;
           if constexpr (EPI == EPI_DLOGITS) {
@@ -586,13 +587,14 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
           }
         } else if constexpr (EPI == EPI_SWIGLU) {
           if (row_ok) {
+            const float rs = p.row_scale != nullptr ? p.row_scale[row] : 1.f;
             const int ac0 = col0 >> 1;        // first activation column of this chunk
             const int npairs = ncols >> 1;    // multiple of 4
             const int inter = p.N >> 1;
             float act[16];
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
-              const float g = __uint_as_float(r[2 * j]), u = __uint_as_float(r[2 * j + 1]);
+              const float g = __uint_as_float(r[2 * j]) * rs, u = __uint_as_float(r[2 * j + 1]) * rs;
               act[j] = g / (1.f + __expf(-g)) * u;
             }
             __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.D) + static_cast<long long>(row) * p.ldd + ac0;
@@ -1181,6 +1183,25 @@ extern "C" int vb_gemm_bf16_swiglu(const void* A, const void* W, void* act, void
   GemmParams p{};
   p.M = M; p.N = 2 * I; p.K = K; p.D = act; p.ldd = ldd; p.status = status_ptr(); p.k_splits = 1;
   p.gu_out = reinterpret_cast<__nv_bfloat16*>(gu_out); p.gu_ld = gu_ld;
+  return static_cast<int>(launch_variant<256, false, false, 4, EPI_SWIGLU>(ta, tb, p, num_sms(), stream));
+}
+
+// Gated up-projection of rows grouped by expert (128 rows to a tile, padding rows included): act[rows_cap, I] from the experts'
+// stacked [gate; up] weights W [E, 2I, K]; row_scale [rows_cap] multiplies both halves before the activation.
+extern "C" int vb_gemm_grouped_swiglu(const void* A, const void* W, void* act, int rows_cap, int I, int K, long long lda, long long ldd,
+                                      const float* row_scale, int E, const int* tile_expert, const int* num_tiles, cudaStream_t stream) {
+  if (rows_cap <= 0 || I <= 0 || K <= 0 || E <= 0) return 0;
+  if ((I % 4) || (K % 8) || (lda % 8) || (ldd % 4) || (rows_cap % 128)) return -1;
+  if (((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) || (reinterpret_cast<uintptr_t>(act) & 7)) return -1;
+  CUtensorMap ta, tb;
+  if (!make_tmap_2d(&ta, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows_cap, K, lda, BK, BM, CU_TENSOR_MAP_SWIZZLE_128B)) return -3;
+  // (k, half, row): expert e's gate row j is (., 0, 2 I e + j), its up row (., 1, 2 I e + j)
+  const uint64_t rows = static_cast<uint64_t>(2 * E - 1) * I;
+  if (!make_tmap_3d(&tb, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, 2, rows, static_cast<uint64_t>(I) * K, K, BK, 2, 128, CU_TENSOR_MAP_SWIZZLE_128B))
+    return -3;
+  GemmParams p{};
+  p.M = rows_cap; p.N = 2 * I; p.K = K; p.D = act; p.ldd = ldd; p.status = status_ptr(); p.k_splits = 1;
+  p.grp_mode = 1; p.grp_E = E; p.grp_tile_expert = tile_expert; p.grp_num_mtiles = num_tiles; p.grp_b_rows = 2 * I; p.row_scale = row_scale;
   return static_cast<int>(launch_variant<256, false, false, 4, EPI_SWIGLU>(ta, tb, p, num_sms(), stream));
 }
 

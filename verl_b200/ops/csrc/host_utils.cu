@@ -46,6 +46,19 @@ bool make_tmap_3d(CUtensorMap* out, const void* base, CUtensorMapDataType dt, in
   return r == CUDA_SUCCESS;
 }
 
+bool make_tmap_4d(CUtensorMap* out, const void* base, CUtensorMapDataType dt, int elem_bytes, const uint64_t (&dims)[4], const uint64_t (&strides)[3],
+                  const uint32_t (&boxes)[4], CUtensorMapSwizzle sw) {
+  PFN_encodeTiled enc = get_encode_tiled();
+  if (!enc) return false;
+  cuuint64_t gdim[4], gstride[3];
+  cuuint32_t box[4], estr[4] = {1, 1, 1, 1};
+  for (int i = 0; i < 4; ++i) { gdim[i] = dims[i]; box[i] = boxes[i]; }
+  for (int i = 0; i < 3; ++i) gstride[i] = strides[i] * static_cast<uint64_t>(elem_bytes);
+  CUresult r = enc(out, dt, 4, const_cast<void*>(base), gdim, gstride, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, sw,
+                   CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS;
+}
+
 int num_sms() {
   static int sms = 0;
   if (sms == 0) {

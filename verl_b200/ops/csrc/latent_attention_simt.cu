@@ -1,7 +1,8 @@
 // Windowed attention with a sink over latent or expanded keys, one warp per (query, head), on the fp32 pipeline.
 //
 // One kernel covers both uses of latent attention: prompts (per-head keys and values expanded from the latents, contiguous
-// rows) and decoding (all heads share the latent row as key and value, rows found through the page table). It serves fp32
+// rows) and decoding (all heads share the latent row as key and value, rows found through the page table), and grouped-query
+// attention in both forms (key / value heads shared by groups of query heads, capped scores). It serves fp32
 // tensors and bf16 sizes outside the tensor-core kernels. Keys are taken 32 at a time: a lane owns a key for the scores, the
 // lanes then share the value columns. Compiled without fast math.
 #include "mixers.h"
@@ -21,7 +22,7 @@ latent_attn_simt_kernel(const VbLatentAttn a) {
   float* so = sq + dq;
   const long long i = blockIdx.x * 4ll + warp;
   if (i >= static_cast<long long>(a.T) * a.H) return;
-  const int h = static_cast<int>(i % a.H);
+  const int h = static_cast<int>(i % a.H), kvh = a.kv_group > 1 ? h / a.kv_group : h;
   const long long t = i / a.H;
   // which sequence, which key rows
   int b = static_cast<int>(t), last;         // index of the query's own key inside its sequence
@@ -65,16 +66,17 @@ latent_attn_simt_kernel(const VbLatentAttn a) {
       const T *ku, *kr;
       if (a.block_table != nullptr) {
         row += static_cast<long long>(j % a.block_size) * a.ku_row;
-        ku = reinterpret_cast<const T*>(a.ku) + row;
+        ku = reinterpret_cast<const T*>(a.ku) + row + static_cast<long long>(kvh) * a.ku_head;
         kr = reinterpret_cast<const T*>(a.kr) + row;
       } else {
-        ku = reinterpret_cast<const T*>(a.ku) + row * a.ku_row + static_cast<long long>(h) * a.ku_head;
+        ku = reinterpret_cast<const T*>(a.ku) + row * a.ku_row + static_cast<long long>(kvh) * a.ku_head;
         kr = reinterpret_cast<const T*>(a.kr) + row * a.kr_row;
       }
       float acc = 0.f;
       for (int c = 0; c < a.du; ++c) acc = fmaf(sq[c], to_f(ku[c]), acc);
       for (int c = 0; c < a.dr; ++c) acc = fmaf(sq[a.du + c], to_f(kr[c]), acc);
       s = acc * a.scale;
+      if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float alpha = expf(m - m_new);
@@ -86,8 +88,7 @@ latent_attn_simt_kernel(const VbLatentAttn a) {
     for (int jj = 0; jj < n; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const long long rj = __shfl_sync(0xffffffffu, row, jj);
-      const T* v = a.block_table != nullptr ? reinterpret_cast<const T*>(a.v) + rj
-                                            : reinterpret_cast<const T*>(a.v) + rj * a.v_row + static_cast<long long>(h) * a.v_head;
+      const T* v = reinterpret_cast<const T*>(a.v) + (a.block_table != nullptr ? rj : rj * a.v_row) + static_cast<long long>(kvh) * a.v_head;
       for (int c = lane; c < a.dv; c += 32) so[c] = fmaf(pj, to_f(v[c]), so[c]);
     }
   }

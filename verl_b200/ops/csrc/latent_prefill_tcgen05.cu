@@ -1,4 +1,6 @@
-// Prompt attention of latent-attention layers on tcgen05 tensor cores: causal, windowed, with a sink and an output gate.
+// Prompt attention of the mixer stacks on tcgen05 tensor cores: causal, windowed, with a sink, capped scores and an output gate.
+// Latent attention, or grouped-query attention with query / key and value sizes of its own (no rotated part, kv_group query
+// heads per key head).
 //
 // One CTA = (sequence, NT query tiles of 128 rows, head). The score product runs over two operand groups, the head's
 // unrotated key part and the rotated part shared by all heads, accumulated in the same TMEM tile, so keys are never
@@ -23,20 +25,26 @@ constexpr int LP_BQ = 128, LP_BK = 64;
 struct LatentPrefillParams {
   const int* cu_q;
   const int* cu_k;
-  int num_seqs, dv, window, pu, pr, pv, su, sr;  // panels of 64 columns (unrotated, rotated, value), k steps of 16
+  int num_seqs, dv, window, kv_group, pu, pr, pv, su, sr;  // panels of 64 columns (unrotated, rotated, value), k steps of 16
   const __nv_bfloat16* sink;
   const float* gate;
   long long ldg;
   __nv_bfloat16* out;
   long long ldo;
   float scale_log2;
+  float cap_z, cap_log2;   // CAP: score = cap_log2 * tanh(product * cap_z), in powers of two
   int tmem_cols;
   int* status;
 };
 
 __device__ int g_latent_prefill_status[1];
 
-template <int NT>
+// tanh(z) / z over s = z^2 <= 1/4: interpolation at the five Chebyshev nodes of [0, 1/4], error 1.4e-8
+__device__ __forceinline__ float tanh_ratio(float s) {
+  return fmaf(s, fmaf(s, fmaf(s, fmaf(s, 0.01713134443f, -0.05298423883f), 0.13324750505f), -0.33333067944f), 0.99999998676f);
+}
+
+template <int NT, bool CAP>
 __global__ void __launch_bounds__(64 + 128 * NT, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_constant__ CUtensorMap tm_qr, const __grid_constant__ CUtensorMap tm_ku,
                       const __grid_constant__ CUtensorMap tm_kr, const __grid_constant__ CUtensorMap tm_v, const LatentPrefillParams p) {
@@ -54,7 +62,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
   uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bar_o + NT);
   int* s_tile = reinterpret_cast<int*>(tmem_holder + 2);  // query start, first row, queries, key start, keys, found
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y, kvh = head / p.kv_group;
   if (threadIdx.x == 0) {
     int t = blockIdx.x, found = 0, qs = 0, q0 = 0, nq = 0, ks = 0, nk = 0;
     for (int s = 0; s < p.num_seqs; ++s) {
@@ -118,11 +126,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         const uint32_t ph = ((j >> 1) & 1) ^ 1;
         if (!mbar_wait(&k_empty[st], ph)) { atomicExch(p.status, ST_TIMEOUT_PRODUCER); break; }
         mbar_expect_tx(&k_full[st], static_cast<uint32_t>(k_bytes));
-        for (int c = 0; c < p.pu; ++c) tma_load_3d(sK + st * k_bytes + c * (LP_BK * 128), &tm_ku, &k_full[st], 64 * c, head, row);
+        for (int c = 0; c < p.pu; ++c) tma_load_3d(sK + st * k_bytes + c * (LP_BK * 128), &tm_ku, &k_full[st], 64 * c, kvh, row);
         for (int c = 0; c < p.pr; ++c) tma_load_2d(sK + st * k_bytes + (p.pu + c) * (LP_BK * 128), &tm_kr, &k_full[st], 64 * c, row);
         if (!mbar_wait(&v_empty[st], ph)) { atomicExch(p.status, ST_TIMEOUT_PRODUCER); break; }
         mbar_expect_tx(&v_full[st], static_cast<uint32_t>(v_bytes));
-        for (int c = 0; c < p.pv; ++c) tma_load_3d(sV + st * v_bytes + c * (LP_BK * 128), &tm_v, &v_full[st], 64 * c, head, row);
+        for (int c = 0; c < p.pv; ++c) tma_load_3d(sV + st * v_bytes + c * (LP_BK * 128), &tm_v, &v_full[st], 64 * c, kvh, row);
       }
     }
   } else if (warp == 1) {
@@ -204,9 +212,34 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         // visible: first_c <= c <= last_c
         const int last_c = pos - col0, first_c = p.window > 0 ? pos - p.window + 1 - col0 : -1;
         float mx = -INFINITY;
+        if constexpr (CAP) {
+          float most = 0.f;
+#pragma unroll
+          for (int c = 0; c < 32; ++c) {
+            const float u = __uint_as_float(x0[c]) * p.cap_z, v = __uint_as_float(x1[c]) * p.cap_z;
+            x0[c] = __float_as_uint(u);
+            x1[c] = __float_as_uint(v);
+            most = fmaxf(most, fmaxf(fabsf(u), fabsf(v)));
+          }
+          if (__any_sync(0xffffffffu, most > 0.5f)) {   // beyond the polynomial: the exponential form
+            auto cap = [&](uint32_t& x) {
+              x = __float_as_uint(p.cap_log2 * (1.f - __fdividef(2.f, 1.f + exp2f(fminf(__uint_as_float(x), 20.f) * 2.8853900817779268f))));
+            };
+#pragma unroll
+            for (int c = 0; c < 32; ++c) { cap(x0[c]); cap(x1[c]); }
+          } else {
+            auto cap = [&](uint32_t& x) {
+              const float z = __uint_as_float(x);
+              x = __float_as_uint(z * p.cap_log2 * tanh_ratio(z * z));
+            };
+#pragma unroll
+            for (int c = 0; c < 32; ++c) { cap(x0[c]); cap(x1[c]); }
+          }
+        }
 #pragma unroll
         for (int c = 0; c < 32; ++c) {
-          float u = __uint_as_float(x0[c]) * p.scale_log2, v = __uint_as_float(x1[c]) * p.scale_log2;
+          float u = __uint_as_float(x0[c]), v = __uint_as_float(x1[c]);
+          if constexpr (!CAP) { u *= p.scale_log2; v *= p.scale_log2; }
           if (need_mask) {
             if (c > last_c || c < first_c) u = -INFINITY;
             if (c + 32 > last_c || c + 32 < first_c) v = -INFINITY;
@@ -310,8 +343,8 @@ using namespace vb;
 extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t stream) {
   const int pu = (a->du + 63) / 64, pr = (a->dr + 63) / 64, pv = (a->dv + 63) / 64;
   auto mis = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) != 0; };
-  if (a->du < 8 || a->dr < 8 || a->du % 8 || a->dr % 8 || a->dv % 8 || a->hq % 8 || a->ldq % 8 || a->ku_head % 8 || a->ku_row % 8 || a->kr_row % 8 ||
-      a->v_head % 8 || a->v_row % 8 || a->ldo % 8 || mis(a->q) || mis(a->ku) || mis(a->kr) || mis(a->v) || mis(a->out) || pv > 4)
+  if (a->du < 8 || a->dr < 0 || a->du % 8 || a->dr % 8 || a->dv % 8 || a->hq % 8 || a->ldq % 8 || a->ku_head % 8 || a->ku_row % 8 || a->kr_row % 8 ||
+      a->v_head % 8 || a->v_row % 8 || a->ldo % 8 || mis(a->q) || mis(a->ku) || (a->dr > 0 && mis(a->kr)) || mis(a->v) || mis(a->out) || pv > 4)
     return -1;
   const int limit = 232448, qp = pu + pr;
   const int nt = (pv <= 2 && latent_prefill_smem(2, qp, pv) <= limit) ? 2 : 1;
@@ -321,20 +354,28 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
   const auto sw = CU_TENSOR_MAP_SWIZZLE_128B;
   CUtensorMap tqu, tqr, tku, tkr, tv;
   const char* qr = reinterpret_cast<const char*>(a->q) + 2 * a->du;
-  if (mis(qr)) return -1;
+  if (a->dr > 0 && mis(qr)) return -1;
+  const int kv_group = a->kv_group > 1 ? a->kv_group : 1, kv_heads = a->H / kv_group;
   if (!make_tmap_3d(&tqu, a->q, bf, 2, a->du, a->H, a->T, a->hq, a->ldq, 64, 1, LP_BQ, sw) ||
-      !make_tmap_3d(&tqr, qr, bf, 2, a->dr, a->H, a->T, a->hq, a->ldq, 64, 1, LP_BQ, sw) ||
-      !make_tmap_3d(&tku, a->ku, bf, 2, a->du, a->H, Tk, a->ku_head, a->ku_row, 64, 1, LP_BK, sw) ||
-      !make_tmap_2d(&tkr, a->kr, bf, 2, Tk, a->dr, a->kr_row, 64, LP_BK, sw) ||
-      !make_tmap_3d(&tv, a->v, bf, 2, a->dv, a->H, Tk, a->v_head, a->v_row, 64, 1, LP_BK, sw))
+      !make_tmap_3d(&tku, a->ku, bf, 2, a->du, kv_heads, Tk, a->ku_head, a->ku_row, 64, 1, LP_BK, sw) ||
+      !make_tmap_3d(&tv, a->v, bf, 2, a->dv, kv_heads, Tk, a->v_head, a->v_row, 64, 1, LP_BK, sw))
     return -1;
+  if (a->dr > 0) {
+    if (!make_tmap_3d(&tqr, qr, bf, 2, a->dr, a->H, a->T, a->hq, a->ldq, 64, 1, LP_BQ, sw) ||
+        !make_tmap_2d(&tkr, a->kr, bf, 2, Tk, a->dr, a->kr_row, 64, LP_BK, sw))
+      return -1;
+  } else {          // never used
+    tqr = tqu;
+    tkr = tku;
+  }
   static int* status = nullptr;
   if (status == nullptr) cudaGetSymbolAddress(reinterpret_cast<void**>(&status), g_latent_prefill_status);
   LatentPrefillParams p{};
-  p.cu_q = a->cu_q; p.cu_k = a->cu_k; p.num_seqs = a->B; p.dv = a->dv; p.window = a->window; p.pu = pu; p.pr = pr; p.pv = pv;
+  p.cu_q = a->cu_q; p.cu_k = a->cu_k; p.num_seqs = a->B; p.dv = a->dv; p.window = a->window; p.kv_group = kv_group; p.pu = pu; p.pr = pr; p.pv = pv;
   p.su = (a->du + 15) / 16; p.sr = (a->dr + 15) / 16;
   p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink); p.gate = a->gate; p.ldg = a->ldg;
   p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo; p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;
+  if (a->softcap > 0.f) { p.cap_z = a->scale / a->softcap; p.cap_log2 = a->softcap * 1.4426950408889634f; }
   p.tmem_cols = 128;
   while (p.tmem_cols < nt * (2 * LP_BK + pv * 64)) p.tmem_cols *= 2;
   const dim3 grid((a->T + nt * LP_BQ - 1) / (nt * LP_BQ) + a->B, a->H);
@@ -344,7 +385,8 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
     kern<<<grid, 64 + 128 * nt, smem, stream>>>(tqu, tqr, tku, tkr, tv, p);
     return static_cast<int>(cudaGetLastError());
   };
-  return nt == 2 ? go(latent_prefill_kernel<2>) : go(latent_prefill_kernel<1>);
+  if (a->softcap > 0.f) return nt == 2 ? go(latent_prefill_kernel<2, true>) : go(latent_prefill_kernel<1, true>);
+  return nt == 2 ? go(latent_prefill_kernel<2, false>) : go(latent_prefill_kernel<1, false>);
 }
 
 extern "C" int vb_latent_prefill_status() {

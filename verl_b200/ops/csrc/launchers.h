@@ -127,6 +127,7 @@ int vb_gemm_fp8_blockscale_grouped(const void* Aq, const float* sa, const void* 
 int vb_fp8_quant_128x128(const void* w, long long ldw, void* q, long long ldq, float* scale_inv, int R, int C, cudaStream_t s);
 int vb_fp8_status();
 int vb_latent_decode_status();
+int vb_grouped_decode_status();
 int vb_latent_prefill_status();
 // moe_kernels.cu
 int vb_moe_route_topk(const void* logits, long long ld, int T, int E, int k, int renorm, float* weights, int* experts, int* counts,

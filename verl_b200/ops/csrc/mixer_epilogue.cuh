@@ -35,6 +35,8 @@ __device__ __forceinline__ void epi_store1(const VbEpiArgs& e, long long row, in
   __nv_bfloat16* D = reinterpret_cast<__nv_bfloat16*>(e.D);
   if (e.mode == VB_EPI_GELU) {
     D[row * e.ldd + col] = __float2bfloat16(gelu_erf_full(v));
+  } else if (e.mode == VB_EPI_SOFTCAP) {
+    D[row * e.ldd + col] = __float2bfloat16(e.cap * tanh_full(v / e.cap));
   } else if (e.mode == VB_EPI_STORE_F32) {
     reinterpret_cast<float*>(e.D)[row * e.ldd + col] = v;
   } else if (e.mode == VB_EPI_SPLIT) {
@@ -68,6 +70,11 @@ __device__ __forceinline__ void epi_store_row(const VbEpiArgs& e, long long row,
     float o[NV];
 #pragma unroll
     for (int i = 0; i < NV; ++i) o[i] = gelu_erf_full(v[i]);
+    put16(o);
+  } else if (e.mode == VB_EPI_SOFTCAP) {
+    float o[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] = e.cap * tanh_full(v[i] / e.cap);
     put16(o);
   } else if (e.mode == VB_EPI_STORE_F32) {
     put32(reinterpret_cast<float*>(e.D) + row * e.ldd + col, v);

@@ -1,4 +1,4 @@
-// C launchers of the mixer-stack kernels (latent attention, mLSTM, Dynamic Tanh, GEMMs with their epilogues).
+// C launchers of the mixer-stack kernels (latent and grouped-query attention, mLSTM, norms, experts, GEMMs with their epilogues).
 // dtype: 0 = fp32 tensors, 1 = bf16 tensors (weights and activations; statistics, states and residual are always fp32).
 #pragma once
 #include <cuda_runtime.h>
@@ -11,6 +11,7 @@ enum VbEpi : int {
   VB_EPI_GELU = 2,      // D = erf-gelu(acc) in the operands' type
   VB_EPI_SPLIT = 3,     // columns [0, n0) -> D in the operands' type, columns [n0, N) -> D2 as fp32
   VB_EPI_RESID = 4,     // X += acc (fp32 residual stream); D = tanh(alpha X) w + b in the operands' type when D is given
+  VB_EPI_SOFTCAP = 5,   // D = cap * tanh(acc / cap) in the operands' type
 };
 
 struct VbEpiArgs {
@@ -25,10 +26,13 @@ struct VbEpiArgs {
   const void* alpha;  // scalar, operands' type
   const void* nw;     // [N]
   const void* nb;     // [N]
+  float cap;
   const float* gate;  // batched products: batch z of row m is multiplied by sigmoid(gate[m * ldg + z]) when given
   long long ldg;
 };
 
+// Attention with per-head or shared keys and values. Latent attention: du unrotated and dr rotated key dimensions (the latter
+// shared by the heads); grouped-query attention: dr = 0, query head h reads key / value head h / kv_group.
 struct VbLatentAttn {
   // queries [T, H, du + dr]: row stride ldq, head stride hq; unrotated part first
   const void* q; long long ldq; int hq;
@@ -46,6 +50,41 @@ struct VbLatentAttn {
   void* out; long long ldo; // [T, H, dv]
   int B, T, H, du, dr, dv, window;
   float scale;
+  int kv_group;             // query heads per key / value head (0 or 1: one)
+  float softcap;            // score = softcap * tanh(score / softcap); 0: off
+};
+
+// x += mult * rms_norm(Y) * nw;  Y = [sigmoid(gate)] sum of `splits` planes of y + sum_j rows[slot[t, j]]
+struct VbResidRms {
+  float* x;                 // [T, W] fp32 residual stream
+  const void* y;            // null: none
+  int y_f32, splits;        // y in fp32 (partial products) or in the weights' type (one plane)
+  long long split_stride, ldy;
+  const void* rows;         // expert outputs, or null
+  long long ldr;
+  const int* slot;          // [T, top]
+  int top;
+  const float* gate;        // gate[t * ldgate], or null
+  long long ldgate;
+  const void *nw, *next;    // norm of the sublayer; next: norm of the new stream, or null (h is the stream itself)
+  void* h;                  // [T, W]
+  float eps, mult;
+  int T, W;
+};
+
+struct VbQkvPrep {
+  const void* p; long long ldp;       // [T, q | k | v]
+  const void *qn, *kn;                // [dim]
+  const int* pos;
+  const float *cos_t, *sin_t;         // [max_pos, half]
+  int half, max_pos;
+  const void* vfirst; long long ldvf; // values of the first mixing layer (or null)
+  const void* vmix;                   // scalar
+  void* q;                            // [T, H, dim]
+  void* rows; long long ldr;          // [T, G (dim + vdim)] or null
+  void* pages; long long page_stride; int block_size; long long num_slots; const long long* slot;
+  int T, H, G, dim, vdim;
+  float eps;
 };
 
 struct VbHeadwise {
@@ -66,10 +105,29 @@ void verl_count_launches(long long n);
 // gemm_simt.cu
 int vb_gemm_simt(int dtype, const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, int b_mn, int batch,
                  long long sa, long long sb, long long sd, const VbEpiArgs* e, cudaStream_t s);
+// rows grouped by expert: 128-row tile i of A meets B[tile_expert[i]] ([N, K] matrices, back to back); tiles past *num_tiles are skipped
+int vb_gemm_simt_grouped(int dtype, const void* A, const void* B, int M, int N, int K, long long lda, const int* tile_expert, const int* num_tiles,
+                         const VbEpiArgs* e, cudaStream_t s);
 // gemm_tcgen05.cu / gemm_skinny_tcgen05.cu: same epilogues on the tensor cores (bf16). Return -1 for shapes they do not serve.
 int vb_gemm_bf16_epi(const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, const VbEpiArgs* e, cudaStream_t s);
 int vb_gemm_skinny_epi(const void* X, const void* W, int M, int N, int K, long long ldx, long long ldw, const VbEpiArgs* e, int splits,
                        float* ws, cudaStream_t s);
+// act[rows, I] = silu(r g) * (r u), [g | u] = A W_e^T with W_e = [gate; up] ([2I, K]) of the tile's expert and r = row_scale[row]
+int vb_gemm_grouped_swiglu(const void* A, const void* W, void* act, int rows_cap, int I, int K, long long lda, long long ldd, const float* row_scale,
+                           int E, const int* tile_expert, const int* num_tiles, cudaStream_t s);
+// stack_rows.cu
+int vb_embed_rms(int dtype, const long long* ids, const void* w, float scale, const void* nw, float eps, float* x, void* h, int T, int W, int V,
+                 cudaStream_t s);
+int vb_residual_rms(int dtype, const VbResidRms* p, cudaStream_t s);
+int vb_gated_silu(int dtype, const void* gu, long long ldg, const float* row_scale, void* out, int T, int I, cudaStream_t s);
+int vb_qkv_prep(int dtype, const VbQkvPrep* p, cudaStream_t s);
+// experts.cu
+int vb_expert_route(const float* z, long long ldz, int T, int E, int k, int renorm, float* score, int* expert, int* rank, int* counts, cudaStream_t s);
+int vb_expert_place(int dtype, const void* h, long long ldh, const float* score, const int* expert, const int* rank, const int* counts, int T, int E, int k,
+                    int W, void* x, float* row_scale, int* slot, int* tile_expert, int* num_tiles, int max_tiles, cudaStream_t s);
+// grouped_decode.cu
+int vb_grouped_decode_splits(const VbLatentAttn* a, int max_keys);
+int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, int nsplit, float* part_o, float* part_ml, cudaStream_t s);
 // mixer_kernels.cu
 int vb_embed_dyt(int dtype, const long long* ids, const void* w, float scale, float* x, void* h, const void* alpha, const void* nw,
                  const void* nb, int T, int W, int V, cudaStream_t s);
