@@ -9,15 +9,13 @@ import pytest
 import torch
 
 from oracles import mixer_stack_plain as plain
+from stack_testing import PLACES, close, feed_all, tokens
 from verl_b200.models import FlatParams, ModelConfig, PackedBatch, build_decoder
 from verl_b200.utils.model import load_hf_weights_into, save_hf_weights
 from verl_b200.workers.rollout.native.engine import RolloutEngine, SamplingParams
 
 torch.set_num_threads(min(4, torch.get_num_threads()))
 REPO = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-PLACES = [pytest.param(("cpu", torch.float32), id="cpu-fp32"),
-          pytest.param(("cuda", torch.float32), id="cuda-fp32", marks=pytest.mark.gpu),
-          pytest.param(("cuda", torch.bfloat16), id="cuda-bf16", marks=pytest.mark.gpu)]
 
 
 @pytest.fixture(params=PLACES)
@@ -136,39 +134,6 @@ def engine(models, name, place, **kw):
     args = dict(max_num_seqs=5, max_model_len=400, block_size=16, num_blocks=100, sync_interval=3, eos_token_id=-1)
     args.update(kw)
     return RolloutEngine(arch, P, **args)
-
-
-def tokens(n, seed, vocab):
-    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def close(got, want, place, what=""):
-    """Root-mean-square error over the vocabulary, relative to the logits' spread, at every position."""
-    got, want = got.detach().cpu().double(), want.double()
-    spread = (want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt()
-    d = got - want
-    err = (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / spread
-    limit = 1e-4 if place[1] == torch.float32 else 0.06
-    assert float(err.max()) < limit, (what, float(err.max()), int(err.argmax()))
-
-
-def feed_all(eng, seqs, cuts, keep_open=False):
-    """Feed the token lists in portions of the given sizes (last size repeats); logits of every position per sequence."""
-    for k in seqs:
-        eng.open_sequence(k)
-    at, out = {k: 0 for k in seqs}, {k: [] for k in seqs}
-    step = 0
-    while any(at[k] < len(t) for k, t in seqs.items()):
-        n = cuts[min(step, len(cuts) - 1)]
-        entries = [(k, t[at[k] : at[k] + n], list(range(min(n, len(t) - at[k])))) for k, t in seqs.items() if at[k] < len(t)]
-        for (k, part, _), l in zip(entries, eng.feed(entries)):
-            out[k].append(l.cpu())
-            at[k] += len(part)
-        step += 1
-    if not keep_open:
-        for k in seqs:
-            eng.close_sequence(k)
-    return {k: torch.cat(v) for k, v in out.items()}
 
 
 # ---------------------------------------------------------------------------------------------- configuration and weights

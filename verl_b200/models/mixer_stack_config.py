@@ -232,7 +232,7 @@ def parse_tofinex(d: dict) -> StackSpec:
     spec = StackSpec(design="Tofinex", embedding_scale=1.0, norm="rms", norm_eps=float(d["norm"]["eps"]), layers=_layers(d, ("attention",), gated=True),
                      norm_on="output", residual_mult=float(d["residual_mult"]), embedding_norm=True, tied_head=True,
                      logit_softcap=float(d.get("logit_softcap") or 0.0))
-    if len({l.mixer.kv_heads * l.mixer.vdim for l in spec.layers if l.mixer.v_mix}) > 1:
+    if len({(l.mixer.kv_heads, l.mixer.vdim) for l in spec.layers if l.mixer.v_mix}) > 1:
         raise ValueError("value-mixing layers need one number of value heads and one value size")
     return spec
 

@@ -364,7 +364,7 @@ Tensor residual_rms_(Tensor x, const OptTensor& y, const Tensor& nw, double eps,
   if (y.has_value()) {
     const bool parts = y->dim() == 3;
     TORCH_CHECK(y->is_cuda() && y->size(-1) == p.W && y->size(-2) == p.T && y->stride(-1) == 1, "residual_rms_: y");
-    if (parts) CHECK_F32(*y); else same(nw, *y, "residual_rms_");
+    if (parts) { CHECK_F32(*y); } else { same(nw, *y, "residual_rms_"); }
     p.y = y->data_ptr(); p.y_f32 = parts; p.splits = parts ? (int)y->size(0) : 1; p.split_stride = parts ? y->stride(0) : 0; p.ldy = y->stride(-2);
   }
   if (rows.has_value()) {
