@@ -61,7 +61,8 @@ struct SkinnyParams {
   unsigned int* done;    // per (token block, weight tile): split CTAs that have finished folding
   int* status;
   unsigned long long wait_ns;
-  VbEpiArgs mix;  // elementwise epilogue of the MIX variant (replaces D / bias)
+  float cap, inv_cap;  // SK_CAP: output cap * tanh(value / cap)
+  VbEpiArgs mix;  // elementwise epilogue of the SK_MIX variant (replaces D / bias)
 };
 
 __device__ int g_skinny_status[1];
@@ -95,7 +96,9 @@ __device__ __forceinline__ SkItem sk_item(const SkinnyParams& p, int it) {
   return r;
 }
 
-template <bool MIX>
+enum SkinnyEpi : int { SK_PLAIN = 0, SK_CAP = 1, SK_MIX = 2 };
+
+template <int EPI>
 __global__ void __launch_bounds__(SK_THREADS, 1)
 gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_constant__ CUtensorMap tma_x,
                    const SkinnyParams p) {
@@ -218,7 +221,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
     const int et = threadIdx.x - 64;
     uint32_t acc_phase = 0;
     float mix_alpha = 0.f;
-    if constexpr (MIX) mix_alpha = epi_alpha(p.mix);
+    if constexpr (EPI == SK_MIX) mix_alpha = epi_alpha(p.mix);
     for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
       const SkItem w = sk_item(p, it);
       const int nl = q * 32 + lane;          // weight row within the tile
@@ -243,7 +246,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
         tmem_ld_wait();
         if (n_ok) {
           const int mrem = mvalid - c * 32;
-          if (MIX && direct) {
+          if (EPI == SK_MIX && direct) {
             const int col = w.out_col0 + nl;
             const EpiColumn ec = epi_column(p.mix, col);
 #pragma unroll
@@ -252,7 +255,11 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
           } else if (direct) {
 #pragma unroll
             for (int j = 0; j < 32; ++j)
-              if (j < mrem) dp[static_cast<long long>(c * 32 + j) * p.ldd] = __float2bfloat16(__uint_as_float(r[j]) + bv);
+              if (j < mrem) {
+                float v = __uint_as_float(r[j]) + bv;
+                if constexpr (EPI == SK_CAP) v = p.cap * tanh_full(v * p.inv_cap);
+                dp[static_cast<long long>(c * 32 + j) * p.ldd] = __float2bfloat16(v);
+              }
           } else {
 #pragma unroll
             for (int j = 0; j < 32; ++j)
@@ -320,12 +327,16 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
 #pragma unroll
             for (int u = 0; u < RB; ++u) {
               const int mm = m + 4 * u;
-              if (MIX) {
+              if (EPI == SK_MIX) {
                 if (mm < r1) {
                   const float v4[4] = {a[u].x, a[u].y, a[u].z, a[u].w};
                   epi_store_row<4>(p.mix, mm, col, v4, mix_alpha);
                 }
               } else if (mm < r1) {
+                if constexpr (EPI == SK_CAP) {
+                  a[u].x = p.cap * tanh_full(a[u].x * p.inv_cap); a[u].y = p.cap * tanh_full(a[u].y * p.inv_cap);
+                  a[u].z = p.cap * tanh_full(a[u].z * p.inv_cap); a[u].w = p.cap * tanh_full(a[u].w * p.inv_cap);
+                }
                 uint2 o;
                 o.x = pack_bf16x2(a[u].x, a[u].y);
                 o.y = pack_bf16x2(a[u].z, a[u].w);
@@ -436,8 +447,9 @@ extern "C" int vb_gemm_skinny_status() {
 // Returns 0 on success, a negative code for arguments the kernel does not serve, a positive cudaError_t otherwise.
 static int sk_launch(const void* X, const void* W, void* D, const void* bias, int M, int K, int w_rows, long long ldx, long long ldw,
                      long long ldd, int nseg, const int* seg_w0, const int* seg_rows, int splits, float* ws, int ws_rows,
-                     int partials_only, const VbEpiArgs* mix, cudaStream_t stream) {
+                     int partials_only, const VbEpiArgs* mix, cudaStream_t stream, float cap = 0.f) {
   SkinnyParams p{};
+  if (cap > 0.f) { p.cap = cap; p.inv_cap = 1.f / cap; }
   if (!sk_plan(M, K, nseg, seg_w0, seg_rows, splits, p)) return -1;
   if (splits > 0 && p.splits != splits) return -4;  // the caller sized ws for another split count
   for (int s = 0; s < nseg; ++s)
@@ -476,8 +488,9 @@ static int sk_launch(const void* X, const void* W, void* D, const void* bias, in
   const int smem = p.stages * stage_bytes + 1024 + 256;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_skinny_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_skinny_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
+    cudaError_t e = cudaFuncSetAttribute(gemm_skinny_kernel<SK_PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_skinny_kernel<SK_CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_skinny_kernel<SK_MIX>, cudaFuncAttributeMaxDynamicSharedMemorySize, SK_SMEM_LIMIT);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
@@ -498,8 +511,9 @@ static int sk_launch(const void* X, const void* W, void* D, const void* bias, in
     cfg.attrs = attr;
     cfg.numAttrs = 1;
   }
-  cudaError_t e = mix != nullptr ? cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<true>, tw, tx, p)
-                                 : cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<false>, tw, tx, p);
+  cudaError_t e = mix != nullptr ? cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<SK_MIX>, tw, tx, p)
+                  : cap > 0.f    ? cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<SK_CAP>, tw, tx, p)
+                                 : cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<SK_PLAIN>, tw, tx, p);
   return static_cast<int>(e);
 }
 
@@ -516,6 +530,8 @@ extern "C" int vb_gemm_skinny_epi(const void* X, const void* W, int M, int N, in
                                   int splits, float* ws, cudaStream_t stream) {
   if (!epi_aligned(*e, 4) || ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) & 15)) return -1;
   const int w0 = 0;
+  if (e->mode == VB_EPI_STORE || e->mode == VB_EPI_SOFTCAP)   // the plain kernel: its stores have no switch over the modes
+    return sk_launch(X, W, e->D, nullptr, M, K, N, ldx, ldw, e->ldd, 1, &w0, &N, splits, ws, 0, 0, nullptr, stream, e->mode == VB_EPI_SOFTCAP ? e->cap : 0.f);
   return sk_launch(X, W, nullptr, nullptr, M, K, N, ldx, ldw, 0, 1, &w0, &N, splits, ws, 0, 0, e, stream);
 }
 

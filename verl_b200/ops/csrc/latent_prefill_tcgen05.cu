@@ -2,7 +2,8 @@
 // Latent attention, or grouped-query attention with query / key and value sizes of its own (no rotated part, kv_group query
 // heads per key head).
 //
-// One CTA = (sequence, NT query tiles of 128 rows, head). The score product runs over two operand groups, the head's
+// One CTA = (sequence, NT query tiles of 128 rows, head): one tile where two such CTAs fit an SM (the softmax, start and end of
+// one run under the products of the other), else two tiles that share the key blocks, else one. The score product runs over two operand groups, the head's
 // unrotated key part and the rotated part shared by all heads, accumulated in the same TMEM tile, so keys are never
 // concatenated in memory. Only key blocks that some row of a tile can see are loaded and multiplied.
 //
@@ -32,24 +33,49 @@ struct LatentPrefillParams {
   __nv_bfloat16* out;
   long long ldo;
   float scale_log2;
-  float cap_z, cap_log2;   // CAP: score = cap_log2 * tanh(product * cap_z), in powers of two
+  // CAP: score = cap_log2 * tanh(x * cap_z) of the product x, in powers of two. Where |x| <= cap_near: x times a polynomial in
+  // x^2 with coefficients cap_poly
+  float cap_z, cap_log2, cap_near, cap_poly[5];
   int tmem_cols;
   int* status;
 };
 
 __device__ int g_latent_prefill_status[1];
 
-// tanh(z) / z over s = z^2 <= 1/4: interpolation at the five Chebyshev nodes of [0, 1/4], error 1.4e-8
-__device__ __forceinline__ float tanh_ratio(float s) {
-  return fmaf(s, fmaf(s, fmaf(s, fmaf(s, 0.01713134443f, -0.05298423883f), 0.13324750505f), -0.33333067944f), 0.99999998676f);
+// two fp32 values in a 64-bit register pair: one instruction for both
+__device__ __forceinline__ uint64_t pack2(uint32_t a, uint32_t b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "r"(a), "r"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t both2(float v) { return pack2(__float_as_uint(v), __float_as_uint(v)); }
+__device__ __forceinline__ void unpack2(uint64_t v, uint32_t& a, uint32_t& b) { asm("mov.b64 {%0, %1}, %2;" : "=r"(a), "=r"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.ftz.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.ftz.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.ftz.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
 }
 
 template <int NT, bool CAP>
-__global__ void __launch_bounds__(64 + 128 * NT, 1)
+__global__ void __launch_bounds__(64 + 128 * NT, 3 - NT)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_constant__ CUtensorMap tm_qr, const __grid_constant__ CUtensorMap tm_ku,
                       const __grid_constant__ CUtensorMap tm_kr, const __grid_constant__ CUtensorMap tm_v, const LatentPrefillParams p) {
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  uint8_t* smem = smem_raw;
+  if ((smem_u32(smem) & 1023u) != 0u) {  // the swizzled layouts need 1024-byte aligned tiles; there is no slack for rounding up
+    if (threadIdx.x == 0) atomicExch(p.status, 9);
+    return;
+  }
   const int qp = p.pu + p.pr;
   const int q_bytes = qp * (LP_BQ * 128), k_bytes = qp * (LP_BK * 128), v_bytes = p.pv * (LP_BK * 128);
   uint8_t* sQ = smem;
@@ -215,39 +241,40 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         if constexpr (CAP) {
           float most = 0.f;
 #pragma unroll
-          for (int c = 0; c < 32; ++c) {
-            const float u = __uint_as_float(x0[c]) * p.cap_z, v = __uint_as_float(x1[c]) * p.cap_z;
-            x0[c] = __float_as_uint(u);
-            x1[c] = __float_as_uint(v);
-            most = fmaxf(most, fmaxf(fabsf(u), fabsf(v)));
-          }
-          if (__any_sync(0xffffffffu, most > 0.5f)) {   // beyond the polynomial: the exponential form
+          for (int c = 0; c < 32; ++c) most = fmaxf(most, fmaxf(fabsf(__uint_as_float(x0[c])), fabsf(__uint_as_float(x1[c]))));
+          if (__any_sync(0xffffffffu, most > p.cap_near)) {   // beyond the polynomial: the exponential form
             auto cap = [&](uint32_t& x) {
-              x = __float_as_uint(p.cap_log2 * (1.f - __fdividef(2.f, 1.f + exp2f(fminf(__uint_as_float(x), 20.f) * 2.8853900817779268f))));
+              const float z = fminf(__uint_as_float(x) * p.cap_z, 20.f);
+              x = __float_as_uint(p.cap_log2 * (1.f - __fdividef(2.f, 1.f + exp2f(z * 2.8853900817779268f))));
             };
 #pragma unroll
             for (int c = 0; c < 32; ++c) { cap(x0[c]); cap(x1[c]); }
           } else {
-            auto cap = [&](uint32_t& x) {
-              const float z = __uint_as_float(x);
-              x = __float_as_uint(z * p.cap_log2 * tanh_ratio(z * z));
+            const uint64_t a0 = both2(p.cap_poly[0]), a1 = both2(p.cap_poly[1]), a2 = both2(p.cap_poly[2]), a3 = both2(p.cap_poly[3]), a4 = both2(p.cap_poly[4]);
+            auto cap = [&](uint32_t& x, uint32_t& y) {
+              const uint64_t z = pack2(x, y), s = mul2(z, z);
+              unpack2(mul2(z, fma2(s, fma2(s, fma2(s, fma2(s, a4, a3), a2), a1), a0)), x, y);
             };
 #pragma unroll
-            for (int c = 0; c < 32; ++c) { cap(x0[c]); cap(x1[c]); }
+            for (int c = 0; c < 32; c += 2) { cap(x0[c], x0[c + 1]); cap(x1[c], x1[c + 1]); }
+          }
+        } else {
+          const uint64_t f = both2(p.scale_log2);
+#pragma unroll
+          for (int c = 0; c < 32; c += 2) {
+            unpack2(mul2(pack2(x0[c], x0[c + 1]), f), x0[c], x0[c + 1]);
+            unpack2(mul2(pack2(x1[c], x1[c + 1]), f), x1[c], x1[c + 1]);
+          }
+        }
+        if (need_mask) {
+#pragma unroll
+          for (int c = 0; c < 32; ++c) {
+            if (c > last_c || c < first_c) x0[c] = 0xff800000u;
+            if (c + 32 > last_c || c + 32 < first_c) x1[c] = 0xff800000u;
           }
         }
 #pragma unroll
-        for (int c = 0; c < 32; ++c) {
-          float u = __uint_as_float(x0[c]), v = __uint_as_float(x1[c]);
-          if constexpr (!CAP) { u *= p.scale_log2; v *= p.scale_log2; }
-          if (need_mask) {
-            if (c > last_c || c < first_c) u = -INFINITY;
-            if (c + 32 > last_c || c + 32 < first_c) v = -INFINITY;
-          }
-          x0[c] = __float_as_uint(u);
-          x1[c] = __float_as_uint(v);
-          mx = fmaxf(mx, fmaxf(u, v));
-        }
+        for (int c = 0; c < 32; ++c) mx = fmaxf(mx, fmaxf(__uint_as_float(x0[c]), __uint_as_float(x1[c])));
         float alpha = 1.f;
         const bool grow = mx > m_run + 8.f;   // also the first visible key of a row without a sink
         if (grow) {
@@ -255,18 +282,24 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
           m_run = mx;
           l_run *= alpha;
         }
-        const float m_use = m_run == -INFINITY ? 0.f : m_run;
-        float sum = 0.f;
+        const uint64_t minus_m = both2(m_run == -INFINITY ? 0.f : -m_run);
+        uint64_t sum = 0;
         uint32_t pk[32];
+        auto weight = [&](uint32_t a, uint32_t b) {
+          uint32_t u, v;
+          unpack2(add2(pack2(a, b), minus_m), u, v);
+          const float e0 = exp2f(__uint_as_float(u)), e1 = exp2f(__uint_as_float(v));
+          sum = add2(sum, pack2(__float_as_uint(e0), __float_as_uint(e1)));
+          return pack_bf16x2(e0, e1);
+        };
 #pragma unroll
         for (int c = 0; c < 32; c += 2) {
-          const float a0 = exp2f(__uint_as_float(x0[c]) - m_use), a1 = exp2f(__uint_as_float(x0[c + 1]) - m_use);
-          const float b0 = exp2f(__uint_as_float(x1[c]) - m_use), b1 = exp2f(__uint_as_float(x1[c + 1]) - m_use);
-          sum += (a0 + a1) + (b0 + b1);
-          pk[c >> 1] = pack_bf16x2(a0, a1);
-          pk[16 + (c >> 1)] = pack_bf16x2(b0, b1);
+          pk[c >> 1] = weight(x0[c], x0[c + 1]);
+          pk[16 + (c >> 1)] = weight(x1[c], x1[c + 1]);
         }
-        l_run += sum;
+        uint32_t s_lo, s_hi;
+        unpack2(sum, s_lo, s_hi);
+        l_run += __uint_as_float(s_lo) + __uint_as_float(s_hi);
         if (jj > 0) {
           // P and O are in use by the previous block's product until bar_o
           if (!mbar_wait(&bar_o[t], (jj - 1) & 1)) { ok = false; break; }
@@ -332,7 +365,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
 }
 
 static int latent_prefill_smem(int nt, int qp, int pv) {
-  return nt * qp * LP_BQ * 128 + 2 * qp * LP_BK * 128 + 2 * pv * LP_BK * 128 + nt * LP_BQ * LP_BK * 2 + 256 + 1024;
+  return nt * qp * LP_BQ * 128 + 2 * qp * LP_BK * 128 + 2 * pv * LP_BK * 128 + nt * LP_BQ * LP_BK * 2 + 192;
 }
 
 }  // namespace vb
@@ -347,7 +380,8 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
       a->v_head % 8 || a->v_row % 8 || a->ldo % 8 || mis(a->q) || mis(a->ku) || (a->dr > 0 && mis(a->kr)) || mis(a->v) || mis(a->out) || pv > 4)
     return -1;
   const int limit = 232448, qp = pu + pr;
-  const int nt = (pv <= 2 && latent_prefill_smem(2, qp, pv) <= limit) ? 2 : 1;
+  const bool pair = pv <= 2 && 2 * (latent_prefill_smem(1, qp, pv) + 1024) <= 228 * 1024;   // two CTAs of one tile (and 256 TMEM columns each)
+  const int nt = (!pair && pv <= 2 && latent_prefill_smem(2, qp, pv) <= limit) ? 2 : 1;
   const int smem = latent_prefill_smem(nt, qp, pv);
   if (smem > limit) return -1;
   const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
@@ -375,7 +409,16 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
   p.su = (a->du + 15) / 16; p.sr = (a->dr + 15) / 16;
   p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink); p.gate = a->gate; p.ldg = a->ldg;
   p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo; p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;
-  if (a->softcap > 0.f) { p.cap_z = a->scale / a->softcap; p.cap_log2 = a->softcap * 1.4426950408889634f; }
+  if (a->softcap > 0.f) {
+    // tanh(z) = z (c0 + c1 z^2 + ...) for |z| <= 1/2: interpolated at the five Chebyshev nodes of z^2 in [0, 1/4], relative error 1.4e-8
+    const double c[5] = {0.9999999867573895, -0.3333306794442257, 0.13324750504795058, -0.05298423882896009, 0.01713134443244478};
+    const double z = static_cast<double>(a->scale) / a->softcap;
+    p.cap_z = static_cast<float>(z);
+    p.cap_log2 = a->softcap * 1.4426950408889634f;
+    p.cap_near = static_cast<float>(0.5 / (z > 0 ? z : -z));
+    double f = a->softcap * 1.4426950408889634 * z;
+    for (int i = 0; i < 5; ++i, f *= z * z) p.cap_poly[i] = static_cast<float>(c[i] * f);
+  }
   p.tmem_cols = 128;
   while (p.tmem_cols < nt * (2 * LP_BK + pv * 64)) p.tmem_cols *= 2;
   const dim3 grid((a->T + nt * LP_BQ - 1) / (nt * LP_BQ) + a->B, a->H);

@@ -1,7 +1,8 @@
-"""Serving benchmark of a mixer-stack design beside the uniform decoder of equal size (same width, layers and parameters).
+"""Serving benchmark of a mixer-stack design beside the closest uniform decoder of equal size (same width, layers and parameters).
 
     python bench.py --design zorelorn            # all sizes: prefill and decode throughput of both models
     python bench.py --design zorelorn --kernels  # the kernels behind them, each against its roofline
+    python bench.py --design tofinex [--kernels]
 
 Random weights and tokens. Prefill runs packed prompts through the engine's prompt path into the cache, decode replays the
 captured decode step over all slots; CUDA events around every timed region, after warm-up, on inputs larger than L2. One
@@ -15,7 +16,7 @@ import json
 
 import torch
 
-from ....models import FlatParams, ModelConfig
+from ....models import DecoderModel, FlatParams, ModelConfig
 from ....ops import functional as F
 from ....ops import mixers as X
 from ....ops import native
@@ -28,6 +29,12 @@ SIZES = {  # name -> (width, heads, q_rank, window, ff, layers, prompts, prompt 
     "width4096": dict(width=4096, heads=32, q_rank=1536, window=4096, ff=16384, layers=8, prompts=4, prompt_len=4096, slots=128, ctx=4096),
 }
 VOCAB = 32768
+# experts = 0: dense feed-forwards of size ff; else every layer has ``experts`` of size ff, ``top`` per token, and a shared one
+TOFINEX_SIZES = {
+    "dense2048": dict(width=2048, heads=16, kv_heads=4, ff=8192, experts=0, top=0, shared_ff=0, layers=12, prompts=8, prompt_len=2048, slots=256, ctx=2048),
+    "moe2048": dict(width=2048, heads=16, kv_heads=4, ff=768, experts=64, top=6, shared_ff=1536, layers=8, prompts=8, prompt_len=2048, slots=256, ctx=2048),
+    "moe4096": dict(width=4096, heads=32, kv_heads=8, ff=1536, experts=32, top=2, shared_ff=3072, layers=4, prompts=4, prompt_len=4096, slots=128, ctx=4096),
+}
 
 
 def zorelorn_config(s: dict) -> ModelConfig:
@@ -45,6 +52,29 @@ def uniform_config(s: dict, params: int) -> ModelConfig:
                                 num_attention_heads=s["width"] // 128, num_key_value_heads=max(1, s["width"] // 512), head_dim=128, rope_theta=500000.0,
                                 max_position_embeddings=8192)
     return mk(max(256, round((params - mk(0).num_parameters()) / (3 * s["width"] * s["layers"]) / 256) * 256))
+
+
+def tofinex_config(s: dict) -> ModelConfig:
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    if s["experts"]:
+        mlp = {"kind": "moe", "expert": {"ff": s["ff"]}, "router": {"experts": s["experts"], "top": s["top"]}, "shared": {"ff": s["shared_ff"]}}
+    mixer = dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, v_mix=True, rot=dict(base=500000.0, dims=128))
+    return ModelConfig.from_hf_dict({"architecture": "Tofinex", "logit_softcap": 20.0, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "vocab": VOCAB, "width": s["width"],
+                                     "layers": [{"type": "attention", "mixer": mixer, "mlp": mlp}] * s["layers"]})
+
+
+def closest_to_tofinex(s: dict, params: int) -> ModelConfig:
+    """Qwen-type decoder with the same attention sizes, query / key norms and feed-forwards (softmax router, shared expert)."""
+    moe = s["experts"] > 0
+    kw = dict(num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"], shared_expert_intermediate_size=s["shared_ff"]) if moe else {}
+    return ModelConfig(model_type="qwen2_moe" if moe else "qwen3", vocab_size=VOCAB, hidden_size=s["width"], intermediate_size=s["ff"], num_hidden_layers=s["layers"],
+                       num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"], head_dim=128, rope_theta=500000.0, max_position_embeddings=8192,
+                       qk_norm=True, attention_bias=False, tie_word_embeddings=True, **kw)
+
+
+# design -> (sizes, its configuration, label and configuration of the closest existing model)
+DESIGNS = {"zorelorn": (SIZES, zorelorn_config, "uniform decoder of equal size", uniform_config),
+           "tofinex": (TOFINEX_SIZES, tofinex_config, "closest existing decoder", closest_to_tofinex)}
 
 
 def _events(fn, steps: int) -> float:
@@ -70,7 +100,7 @@ def bench_model(cfg: ModelConfig, s: dict, steps: int, warmup: int) -> dict:
 
     def prefill():
         h, batch = eng._run_portions(ids, [0] * n, [L] * n, table[:n], list(range(n)))
-        return eng._logits(h[batch.cu_seqlens[1:].long() - 1])
+        return eng._logits(h[batch.cu_seqlens[1:].long() - 1].contiguous())
 
     for _ in range(warmup):
         prefill()
@@ -96,31 +126,39 @@ def bench_model(cfg: ModelConfig, s: dict, steps: int, warmup: int) -> dict:
     return out
 
 
-def run_models(steps: int, warmup: int, only=None) -> None:
-    for name, s in SIZES.items():
+def run_models(design: str, steps: int, warmup: int, only=None) -> None:
+    sizes, make, other, make_other = DESIGNS[design]
+    for name, s in sizes.items():
         if only and name not in only:
             continue
-        z = zorelorn_config(s)
-        for label, cfg in (("zorelorn", z), ("uniform decoder of equal size", uniform_config(s, z.num_parameters()))):
+        z = make(s)
+        for label, cfg in ((design, z), (other, make_other(s, z.num_parameters()))):
             r = bench_model(cfg, s, steps, max(3, warmup))
             print(json.dumps({"bench": "serving", "size": name, "model": label, "intermediate_size": cfg.intermediate_size, **s, **r, "dtype": "bf16",
                               "data": "synthetic (random weights and tokens)"}), flush=True)
 
 
 # --------------------------------------------------------------------------------------------- kernels
-def run_kernels(iters: int = 20, only=None, sizes=None) -> None:
-    dev = torch.device("cuda", torch.cuda.current_device())
-    pk, timer = _peaks(), Timer(dev, iters, 3)
-    r = lambda *sh, sc=1.0, dt=torch.bfloat16: (torch.randn(*sh, device=dev) * sc).to(dt)
+def _kernel_reporter(design: str, other: str, timer, only):
+    pk = _peaks()
 
     def case(size, phase, kernel, fn, flops, nbytes, new):
         if only and kernel not in only:
             return
         ms = timer(fn)
         floor = max(flops / (pk["bf16_tflops"] * 1e9), nbytes / (pk["hbm_gbs"] * 1e6))
-        print(json.dumps({"bench": "kernel", "size": size, "phase": phase, "kernel": kernel, "design": "zorelorn" if new else "uniform decoder", "us": round(ms * 1e3, 2),
+        print(json.dumps({"bench": "kernel", "size": size, "phase": phase, "kernel": kernel, "design": design if new else other, "us": round(ms * 1e3, 2),
                           "roofline_us": round(floor * 1e3, 2), "fraction_of_measured": round(floor / ms, 3), "bound": "flops" if flops / pk["bf16_tflops"] > nbytes / pk["hbm_gbs"] * 1e3 else "bytes",
                           "clocks": timer.clocks}), flush=True)
+
+    return case
+
+
+def run_kernels(iters: int = 20, only=None, sizes=None) -> None:
+    dev = torch.device("cuda", torch.cuda.current_device())
+    timer = Timer(dev, iters, 3)
+    r = lambda *sh, sc=1.0, dt=torch.bfloat16: (torch.randn(*sh, device=dev) * sc).to(dt)
+    case = _kernel_reporter("zorelorn", "uniform decoder", timer, only)
 
     for name, s in SIZES.items():
         if sizes and name not in sizes:
@@ -201,9 +239,117 @@ def run_kernels(iters: int = 20, only=None, sizes=None) -> None:
     native.check_status()
 
 
+def run_tofinex_kernels(iters: int = 20, only=None, sizes=None) -> None:
+    dev = torch.device("cuda", torch.cuda.current_device())
+    timer = Timer(dev, iters, 3)
+    r = lambda *sh, sc=1.0, dt=torch.bfloat16: (torch.randn(*sh, device=dev) * sc).to(dt)
+    case = _kernel_reporter("tofinex", "closest decoder", timer, only)
+    mm = lambda m, n, k: (2.0 * m * n * k, 2.0 * (m * k + n * k + m * n))
+    for name, s in TOFINEX_SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        W, H, G, ff, E, top, sff, d = s["width"], s["heads"], s["kv_heads"], s["ff"], s["experts"], s["top"], s["shared_ff"], 128
+        qkv, Q, scale, cap = (H + 2 * G) * d, H * d, d ** -0.5, 30.0
+        cos, sin = F.rope_table(8192, d, 5e5, dev)
+        nw, qn, kn, lam = r(W), r(d), r(d), r(1)
+        for phase, T in (("prefill", s["prompts"] * s["prompt_len"]), ("decode", s["slots"])):
+            h, x, att, res = r(T, W), torch.randn(T, W, device=dev), r(T, Q), r(T, W)
+            w_in, w_o = r(qkv, W, sc=0.02), r(W, Q, sc=0.02)
+            pos = torch.arange(T, device=dev, dtype=torch.int32) % 4096
+            f, b = mm(T, qkv, W)
+            case(name, phase, "linear_act (query, key and value projection)", lambda: X.linear_act(h, w_in), f, b, True)
+            case(name, phase, "gemm (same product)", lambda: F.gemm(h, w_in), f, b, False)
+            f, b = mm(T, W, Q)
+            case(name, phase, "linear_partial (output projection)", lambda: X.linear_partial(att, w_o), f, b, True)
+            case(name, phase, "gemm (output projection)", lambda: F.gemm(att, w_o), f, b, False)
+            y = X.linear_partial(att, w_o)
+            case(name, phase, "residual_rms (partial products, norm, residual, next input)", lambda: X.residual_rms_(x, y, nw, 1e-6, 0.5), 0,
+                 y.numel() * y.element_size() + 10.0 * T * W, True)
+            case(name, phase, "rmsnorm with residual", lambda: F.rms_norm(h, nw, 1e-6, residual=res), 0, 8.0 * T * W, False)
+            p, first = r(T, qkv), r(T, G * d)
+            case(name, phase, "qkv_prep (norms, rotation, value mix, rows)", lambda: X.qkv_prep(p, qn, kn, 1e-6, pos, cos, sin, H, G, d, first, lam, None, None, True), 0,
+                 4.0 * T * qkv + 2.0 * T * G * d, True)
+            q, k, v = r(T, H, d), r(T, G, d), r(T, G, d)
+            case(name, phase, "rope (query rotation)", lambda: F.apply_rope_(q, pos, cos, sin), 0, 4.0 * T * Q, False)
+            if phase == "prefill":
+                n, L = s["prompts"], s["prompt_len"]
+                cu = torch.arange(n + 1, device=dev, dtype=torch.int32) * L
+                sink = torch.zeros(H, device=dev, dtype=torch.bfloat16)
+                fl, by = 4.0 * n * L * (L + 1) / 2 * Q, 2.0 * T * (2 * Q + 2 * G * d)
+                case(name, phase, "grouped_attention_prefill (capped scores, sink)", lambda: X.grouped_attention_prefill(q, k, v, cu, cu, 0, scale, cap, sink), fl, by, True)
+                case(name, phase, "attention_varlen", lambda: F.attention_varlen(q, k, v, cu, L), fl, by, False)
+            else:
+                S, ctx, bs = s["slots"], s["ctx"], 64
+                per = -(-(ctx + 64) // bs)
+                pages, kc, vc = r(S * per, bs, 2 * G * d, sc=0.5), r(S * per, bs, G, d, sc=0.5), r(S * per, bs, G, d, sc=0.5)
+                table = torch.arange(S * per, device=dev, dtype=torch.int32).view(S, per)
+                cl = torch.full((S,), ctx, device=dev, dtype=torch.int32)
+                sink = torch.zeros(H, device=dev, dtype=torch.bfloat16)
+                fl, by = 4.0 * S * ctx * Q, 4.0 * S * ctx * G * d
+                case(name, phase, "grouped_attention_decode (capped scores, sink)", lambda: X.grouped_attention_decode(q, pages, table, cl, G, d, 0, scale, cap, sink), fl, by, True)
+                case(name, phase, "paged_decode_attention", lambda: F.paged_decode_attention(q, kc, vc, table, cl), fl, by, False)
+                del pages, kc, vc
+            if not E:
+                w_gu, w_d, a = r(2 * ff, W, sc=0.02), r(W, ff, sc=0.02), r(T, ff)
+                f, b = mm(T, 2 * ff, W)
+                case(name, phase, "gated_up (gate, up, activation)", lambda: X.gated_up(h, w_gu), f, b - 2.0 * T * ff, True)
+                case(name, phase, "gemm_swiglu", lambda: F.gemm_swiglu(h, w_gu)[0], f, b - 2.0 * T * ff, False)
+                f, b = mm(T, W, ff)
+                case(name, phase, "linear_partial (down projection)", lambda: X.linear_partial(a, w_d), f, b, True)
+                case(name, phase, "gemm (down projection)", lambda: F.gemm(a, w_d), f, b, False)
+                del w_gu, w_d, a
+            else:
+                w_m = r(2 * sff + -(-(E + 1) // 8) * 8, W, sc=0.02)
+                w_u, w_dn = r(E * 2 * ff, W, sc=0.02), r(E * W, ff, sc=0.02)
+                f, b = mm(T, w_m.shape[0], W)
+                case(name, phase, "gated_up_split (shared expert, router, gate)", lambda: X.gated_up_split(h, w_m, 2 * sff), f, b - 2.0 * T * sff, True)
+                w_gu, w_r = w_m[: 2 * sff].contiguous(), w_m[2 * sff :].contiguous()
+                case(name, phase, "gemm_swiglu + router gemm", lambda: (F.gemm_swiglu(h, w_gu)[0], F.gemm(h, w_r)), f, b - 2.0 * T * sff, False)
+                z = torch.randn(T, E + 8, device=dev)
+                zb = z[:, :E].to(torch.bfloat16).contiguous()
+                rows, used = T * top, min(E, T * top)
+                by = 4.0 * T * E + 2.0 * T * W + 2.0 * rows * W
+                case(name, phase, "expert_dispatch (route, place, copy)", lambda: X.expert_dispatch(h, z, E, top), 0, by, True)
+                ops = native.ops()
+
+                def route_other():
+                    wts, idx, counts = ops.moe_route_topk(zb, top, False)
+                    plan = DecoderModel._moe_plan(idx.long(), counts, T, top, E)
+                    return plan, ops.moe_gather_rows(h, plan["src"], None), wts
+
+                case(name, phase, "moe_route_topk + plan + gather_rows", route_other, 0, by, False)
+                plan = X.expert_dispatch(h, z, E, top)
+                act = X.expert_up(plan, w_u, ff)
+                oplan, xp, wts = route_other()
+                w3, d3 = w_u.view(E, 2 * ff, W), w_dn.view(E, W, ff)
+                fl, by = 2.0 * rows * 2 * ff * W, 2.0 * (used * 2 * ff * W + rows * (W + ff))
+                case(name, phase, "expert_up (gate, up, score, activation)", lambda: X.expert_up(plan, w_u, ff), fl, by, True)
+                case(name, phase, "gemm_grouped_rows + swiglu", lambda: F.swiglu(ops.gemm_grouped_rows(xp, w3, False, oplan["tile_expert"], oplan["num_mtiles"])), fl, by, False)
+                a2 = r(xp.shape[0], ff)
+                fl, by = 2.0 * rows * ff * W, 2.0 * (used * ff * W + rows * (W + ff))
+                case(name, phase, "expert_down", lambda: X.expert_down(act, w_dn, plan), fl, by, True)
+                case(name, phase, "gemm_grouped_rows (down)", lambda: ops.gemm_grouped_rows(a2, d3, False, oplan["tile_expert"], oplan["num_mtiles"]), fl, by, False)
+                out = X.expert_down(act, w_dn, plan)
+                case(name, phase, "residual_rms (experts, gated shared part, norm, residual)", lambda: X.residual_rms_(x, h, nw, 1e-6, 0.5, None, (out, plan.slot), z[:, E]), 0,
+                     2.0 * rows * W + 12.0 * T * W, True)
+                yo = ops.gemm_grouped_rows(a2, d3, False, oplan["tile_expert"], oplan["num_mtiles"])
+                case(name, phase, "moe_combine", lambda: ops.moe_combine(yo, oplan["slot"], wts), 0, 2.0 * rows * W + 2.0 * T * W, False)
+                del w_m, w_u, w_dn, plan, act, xp, a2, out, yo
+            ids, emb = torch.randint(0, VOCAB, (T,), device=dev), r(VOCAB, W)
+            case(name, phase, "embed_rms", lambda: X.embed_rms(ids, emb, 1.0, nw, 1e-6), 0, 8.0 * T * W, True)
+            case(name, phase, "embedding", lambda: F.embedding(ids, emb), 0, 4.0 * T * W, False)
+            if phase == "decode":
+                f, b = mm(T, VOCAB, W)
+                case(name, phase, "linear_softcap (logits)", lambda: X.linear_softcap(h, emb, 20.0), f, b, True)
+                case(name, phase, "gemm (logits)", lambda: F.gemm(h, emb), f, b, False)
+            del emb
+            torch.cuda.empty_cache()
+    native.check_status()
+
+
 def main(args) -> None:
     native.load()
     if args.kernels:
-        run_kernels()
+        {"zorelorn": run_kernels, "tofinex": run_tofinex_kernels}[args.design]()
     else:
-        run_models(args.steps if args.steps > 2 else 5, args.warmup)
+        run_models(args.design, args.steps if args.steps > 2 else 5, args.warmup)
