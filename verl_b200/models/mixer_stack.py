@@ -6,12 +6,14 @@ same cache object: a page pool for the rows of the attention layers and one fp32
 layers (``workers/rollout/native/cache.py::StackCache``). Layers that share weights still have their own pages and state.
 
 Step layout: every projection that reads a layer's input is one GEMM. Stacks with elementwise norms in front of the sublayers:
-the GEMM that ends a sublayer adds to the residual stream and applies the next norm in its epilogue. Stacks with RMS norms on
+the GEMM that ends a sublayer adds to the residual stream and applies the next norm in its epilogue (with norms on both sides
+also the one on the sublayer's output). Stacks with RMS norms on
 the sublayers' outputs: one row kernel behind that GEMM adds up its partial products (and the experts' rows), norms them, adds
 to the stream and writes the next sublayer's input. Feed-forward activations run in the epilogue of the up-projection. Latent
 attention: prompts expand keys and values from the latents; decoding absorbs the key expansion into the query and applies the
-value expansion to the attention output, so only latent rows are read. Grouped-query attention caches normed, rotated keys and
-mixed values; experts run on tokens grouped by expert without a host synchronisation.
+value expansion to the attention output, so only latent rows are read; a layer may read another layer's rows. Grouped-query
+attention caches normed, rotated keys and mixed or convolved values, the convolution's last inputs are state; experts run on
+tokens grouped by expert without a host synchronisation.
 
 Forward only: the stacks are served (rollout, log-probs), not trained.
 """
@@ -59,6 +61,7 @@ class MixerStackModel:
         self._rope: dict = {}
         self._ensure_rope(max_positions or 2048)
         self._zero_sinks: dict = {}
+        self._row_readers = {l.mixer.kv_from for l in self.spec.layers if getattr(l.mixer, "kv_from", -1) >= 0}   # layers whose rows others use
         self._weights = [self._layer_weights(i) for i in range(len(self.spec.layers))]
         self._final_norm = self._norm("final.norm")
         self._embed_norm = self._norm("embed.norm") if self.spec.embedding_norm else None
@@ -72,17 +75,22 @@ class MixerStackModel:
         layer = self.spec.layers[i]
         p = f"l{layer.owner}."
         W = {k[len(p):]: v for k, v in self.params.views.items() if k.startswith(p)}
-        out = {"norm1": self._norm(p + "norm1"), **{k[4:]: v for k, v in W.items() if k.startswith("mix.")}}
+        both = self.spec.norm_on == "both"
+        out = {"norm1": self._norm(p + "norm1"), "norm1b": self._norm(p + "norm1b") if both else None,
+               **{k[4:]: v for k, v in W.items() if k.startswith("mix.")}}
         m = layer.mixer
         if m.kind == "latent_attention":
             out["uk"] = out["ukv"][: m.heads * m.dim].view(m.heads, m.dim, m.kv_rank)
             out["uv"] = out["ukv"][m.heads * m.dim :].view(m.heads, m.vdim, m.kv_rank)
+        elif m.kind == "lightning":
+            out["decay"] = torch.tensor(m.decay, dtype=torch.float32, device=self.device)
         elif m.kind == "attention":
             if m.heads not in self._zero_sinks:
                 self._zero_sinks[m.heads] = torch.zeros(m.heads, dtype=self.params.flat.dtype, device=self.device)
             out["sink"] = self._zero_sinks[m.heads] if m.zero_sink else None
         if layer.mlp is not None:
-            out.update(norm2=self._norm(p + "norm2"), **{k: v for k, v in W.items() if k.startswith("mlp.")})
+            out.update(norm2=self._norm(p + "norm2"), norm2b=self._norm(p + "norm2b") if both else None,
+                       **{k: v for k, v in W.items() if k.startswith("mlp.")})
         return out
 
     def _ensure_rope(self, n: int) -> None:
@@ -100,38 +108,56 @@ class MixerStackModel:
 
     # ------------------------------------------------------------------------------------ mixers
     def _attention_in(self, W, m, h, pos, pages, slot_map, want_rows: bool):
-        cut = m.q_rank + m.kv_rank + m.rot_dim
-        p, gate = X.linear_split(h, W["in"], cut)
+        """Queries [T, heads, dim + rot_dim] (not rotated), the layer's own latent rows (None: it reads another layer's), gates."""
         cos, sin = self._rope[m.rot.key()]
-        cq, rows = X.latent_prep(p, W["dq.norm"], W["dkv.norm"], self.spec.norm_eps, pos, cos, sin, pages, slot_map, want_rows)
-        q = X.linear_act(cq, W["uq"]).view(h.shape[0], m.heads, m.dim + m.rot_dim)
-        return q, rows, gate, cos, sin
+        q_cols = m.heads * (m.dim + m.rot_dim)
+        p, gate = X.linear_split(h, W["in"], m.q_rank + m.kv_rank + m.rot_dim) if m.gate else (X.linear_act(h, W["in"]), None)
+        cq, rows = None, None
+        if m.kv_from < 0:
+            at = 0 if m.q_rank else -(-q_cols // 8) * 8
+            cq, rows = X.latent_prep(p[:, at : at + m.q_rank + m.kv_rank + m.rot_dim], W["dq.norm"] if m.q_rank else None, W["dkv.norm"], self.spec.norm_eps,
+                                     pos, cos, sin, pages, slot_map, want_rows)
+        q = X.linear_act(cq, W["uq"]) if m.q_rank else p[:, :q_cols]
+        return q.unflatten(1, (m.heads, m.dim + m.rot_dim)), rows, gate, cos, sin
 
-    def _attention_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict]):
-        pages = pc.cache.pages(i) if pc is not None else None
+    def _attention_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict], shared: dict):
+        """``shared``: rows that other layers of this pass may use."""
+        src = m.kv_from if m.kv_from >= 0 else i
+        pages = pc.cache.pages(src) if pc is not None else None
         q, rows, gate, cos, sin = self._attention_in(W, m, h, batch.positions, pages, pc.slot_map if pc is not None else None, portion is None)
         X.rope_pairs_(q, batch.positions, cos, sin, m.dim)
-        cu_k = batch.cu_seqlens
+        cu_k, key = batch.cu_seqlens, (src, m.window, m.keep_first)
         if portion is not None:      # earlier tokens of some sequence are in the cache: take the keys from the pages
-            lo, cu_k, total = portion[m.window]
-            rows = X.gather_pages(pages, pc.block_table, cu_k, lo, total)
+            lo, cu_k, total = portion[key[1:]]
+        else:
+            key = (src,)
+        if key in shared:
+            rows = shared[key]
+        else:
+            rows = X.gather_pages(pages, pc.block_table, cu_k, lo, total) if portion is not None else rows
+            if src in self._row_readers:
+                shared[key] = rows
         kv = X.linear_act(rows[:, : m.kv_rank], W["ukv"])
         ku = kv[:, : m.heads * m.dim].view(-1, m.heads, m.dim)
         v = kv[:, m.heads * m.dim :].view(-1, m.heads, m.vdim)
-        o = X.latent_attention_prefill(q, ku, rows[:, m.kv_rank :], v, batch.cu_seqlens, cu_k, m.window, m.scale, W["sink"], gate)
+        o = X.latent_attention_prefill(q, ku, rows[:, m.kv_rank :], v, batch.cu_seqlens, cu_k, m.window, m.scale, W.get("sink"), gate, m.keep_first)
         return o.view(h.shape[0], m.heads * m.vdim)
 
     def _attention_decode(self, i, W, m, h, pos, slot_map, ctx_len, block_table, cache):
-        S = h.shape[0]
-        q, _, gate, cos, sin = self._attention_in(W, m, h, pos, cache.pages(i), slot_map, False)
+        S, pages = h.shape[0], cache.pages(m.kv_from if m.kv_from >= 0 else i)
+        q, _, gate, cos, sin = self._attention_in(W, m, h, pos, pages, slot_map, False)
         qa = X.latent_absorb(q, W["uk"], pos, cos, sin)
-        oc = X.latent_attention_decode(qa, cache.pages(i), block_table, ctx_len, m.kv_rank, m.window, m.scale, W["sink"])
+        oc = X.latent_attention_decode(qa, pages, block_table, ctx_len, m.kv_rank, m.window, m.scale, W.get("sink"), m.keep_first)
         return X.headwise_linear(oc, W["uv"], False, gate).view(S, m.heads * m.vdim)
 
-    def _grouped_in(self, i, W, m, h, pos, pages, slot_map, want_rows: bool, first: dict):
-        """Queries and the row [keys | values]; ``first`` carries the values of the stack's first value-mixing layer."""
-        p = X.linear_act(h, W["in"])
+    def _grouped_in(self, i, W, m, h, pos, pages, slot_map, want_rows: bool, first: dict, past: dict):
+        """Queries and the row [keys | values]; ``first`` carries the values of the stack's first value-mixing layer, ``past`` says
+        where the inputs of a convolution go on from."""
+        p = X.linear_bias(h, W["in"], W["in.b"]) if m.bias else X.linear_act(h, W["in"])
         cos, sin = self._rope[m.rot.key()]
+        if m.norm_after_rot:
+            return X.conv_qkv_prep(p, W.get("in.conv"), self.spec.norm_eps, pos, cos, sin, m.heads, m.kv_heads, m.dim, m.vdim, m.rot.pairing == "halves",
+                                   **past, pages=pages, page_slots=slot_map, want_rows=want_rows)
         v_first = None
         if m.v_mix:
             if i == self.spec.value_source:
@@ -142,19 +168,27 @@ class MixerStackModel:
         return X.qkv_prep(p, W["q.norm"], W["k.norm"], self.spec.norm_eps, pos, cos, sin, m.heads, m.kv_heads, m.vdim, v_first,
                           W["vmix"] if v_first is not None else None, pages, slot_map, want_rows)
 
-    def _grouped_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict], first: dict):
+    def _grouped_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict], first: dict, fresh):
         pages = pc.cache.pages(i) if pc is not None else None
-        q, rows = self._grouped_in(i, W, m, h, batch.positions, pages, pc.slot_map if pc is not None else None, portion is None, first)
+        past = {"cu": batch.cu_seqlens, "state": pc.cache.state(i), "slots": pc.slots, "fresh": fresh} if pc is not None and m.state_size else {"cu": batch.cu_seqlens}
+        q, rows = self._grouped_in(i, W, m, h, batch.positions, pages, pc.slot_map if pc is not None else None, portion is None, first, past)
         cu_k = batch.cu_seqlens
         if portion is not None:
-            lo, cu_k, total = portion[m.window]
+            lo, cu_k, total = portion[(m.window, m.keep_first)]
             rows = X.gather_pages(pages, pc.block_table, cu_k, lo, total)
         k, v = rows[:, : m.kv_heads * m.dim].unflatten(1, (m.kv_heads, m.dim)), rows[:, m.kv_heads * m.dim :].unflatten(1, (m.kv_heads, m.vdim))
-        return X.grouped_attention_prefill(q, k, v, batch.cu_seqlens, cu_k, m.window, m.scale, m.softcap, W["sink"]).flatten(1)
+        return X.grouped_attention_prefill(q, k, v, batch.cu_seqlens, cu_k, m.window, m.scale, m.softcap, W["sink"], m.keep_first).flatten(1)
 
-    def _grouped_decode(self, i, W, m, h, pos, slot_map, ctx_len, block_table, cache, first: dict):
-        q, _ = self._grouped_in(i, W, m, h, pos, cache.pages(i), slot_map, False, first)
-        return X.grouped_attention_decode(q, cache.pages(i), block_table, ctx_len, m.kv_heads, m.vdim, m.window, m.scale, m.softcap, W["sink"]).flatten(1)
+    def _grouped_decode(self, i, W, m, h, pos, slot_map, ctx_len, active, block_table, cache, first: dict):
+        past = {"state": cache.state(i), "active": active} if m.state_size else {"active": active}
+        q, _ = self._grouped_in(i, W, m, h, pos, cache.pages(i), slot_map, False, first, past)
+        return X.grouped_attention_decode(q, cache.pages(i), block_table, ctx_len, m.kv_heads, m.vdim, m.window, m.scale, m.softcap, W["sink"],
+                                          m.keep_first).flatten(1)
+
+    def _lightning(self, W, m, h, recur: Callable) -> torch.Tensor:
+        n = m.heads * (2 * m.dim + m.vdim)
+        p = X.linear_silu(h, W["in"], n)
+        return X.gated_rms(recur(p, W["decay"], m.dim, m.vdim), p[:, n : n + m.heads * m.vdim], W["norm"], self.spec.norm_eps)
 
     def _mlstm_in(self, W, m, h):
         return X.linear_split(h, W["in"], 2 * m.heads * (m.dim + m.vdim))
@@ -169,17 +203,23 @@ class MixerStackModel:
             self.stats_hook(f"layers.{i}.residual", x)
 
     def _run_input_norms(self, ids: torch.Tensor, mix: Callable) -> torch.Tensor:
+        """Dynamic Tanh in front of the sublayers, with ``norm_on`` "both" also on their outputs."""
         layers, Ws = self.spec.layers, self._weights
-        x, h = X.embed_dyt(ids, self.params["embed"], self.spec.embedding_scale, *Ws[0]["norm1"])
+        if self._embed_norm is not None:
+            x, h = X.embed_dyt2(ids, self.params["embed"], self._embed_norm, Ws[0]["norm1"])
+        else:
+            x, h = X.embed_dyt(ids, self.params["embed"], self.spec.embedding_scale, *Ws[0]["norm1"])
         for i, layer in enumerate(layers):
-            W = Ws[i]
+            W, f = Ws[i], layer.mlp
             nxt = Ws[i + 1]["norm1"] if i + 1 < len(layers) else self._final_norm
             o = mix(i, W, layer.mixer, h)
-            if layer.mlp is None:
-                h = X.linear_residual_(o, W["o"], x, nxt)
-            else:
-                h = X.linear_residual_(o, W["o"], x, W["norm2"])
-                h = X.linear_residual_(X.linear_act(h, W["mlp.up"], layer.mlp.act), W["mlp.down"], x, nxt)
+            h = X.linear_residual_(o, W["o"], x, nxt if f is None else W["norm2"], W["norm1b"])
+            if f is not None and f.kind == "moe":
+                plan = X.expert_dispatch(h, X.linear_act(h, W["mlp.in"], out_f32=True), f.experts, f.top, f.renormalize, W.get("mlp.correction"), f.groups, f.keep)
+                rows = X.expert_down(X.expert_up(plan, W["mlp.experts.in"], f.ff, f.act, f.limit), W["mlp.experts.down"], plan)
+                h = X.residual_dyt_(x, rows, plan.slot, W["norm2b"], nxt)
+            elif f is not None:
+                h = X.linear_residual_(X.linear_act(h, W["mlp.up"], f.act), W["mlp.down"], x, nxt, W["norm2b"])
             self._layer_done(i, x)
         return h
 
@@ -213,19 +253,24 @@ class MixerStackModel:
         portion = None
         if any(starts):
             portion = {}
-            for w in {l.mixer.window for l in self.spec.layers if l.mixer.page_width}:
-                lo = [max(0, s - w + 1) if w > 0 else 0 for s in starts]
+            for w in {(l.mixer.window, l.mixer.keep_first) for l in self.spec.layers if hasattr(l.mixer, "window")}:
+                # rows a layer reads: from the window's start, or all where the first tokens stay visible
+                lo = [max(0, s - w[0] + 1) if w[0] > 0 and w[1] == 0 else 0 for s in starts]
                 cu = torch.zeros(len(lens) + 1, dtype=torch.int32)
                 cu[1:] = torch.cumsum(torch.tensor([s + n - a for s, n, a in zip(starts, lens, lo)], dtype=torch.int32), 0)
                 portion[w] = (torch.tensor(lo, dtype=torch.int32).to(self.device), cu.to(self.device), int(cu[-1]))
         fresh = torch.tensor([int(s == 0) for s in starts], dtype=torch.int32).to(self.device) if pc is not None and self.spec.recurrent else None
         first: dict = {}
+        shared: dict = {}
 
         def mix(i, W, m, h):
             if m.kind == "latent_attention":
-                return self._attention_prefill(i, W, m, h, batch, pc, portion)
+                return self._attention_prefill(i, W, m, h, batch, pc, portion, shared)
             if m.kind == "attention":
-                return self._grouped_prefill(i, W, m, h, batch, pc, portion, first)
+                return self._grouped_prefill(i, W, m, h, batch, pc, portion, first, fresh)
+            if m.kind == "lightning":
+                kept = (pc.cache.state(i), pc.slots, fresh) if pc is not None else (None, None, None)
+                return self._lightning(W, m, h, lambda *a: X.lightning_prefill(*a, batch.cu_seqlens, *kept, not any(starts)))
             p, gates = self._mlstm_in(W, m, h)
             return X.mlstm_prefill(p, gates, W["i.b"], W["f.b"], m.gate_cap, W["norm"], self.spec.norm_eps, m.dim, batch.cu_seqlens,
                                    pc.cache.state(i) if pc is not None else None, pc.slots if pc is not None else None, fresh, not any(starts))
@@ -241,7 +286,9 @@ class MixerStackModel:
             if m.kind == "latent_attention":
                 return self._attention_decode(i, W, m, h, pos, slot_map, ctx_len, block_table, cache)
             if m.kind == "attention":
-                return self._grouped_decode(i, W, m, h, pos, slot_map, ctx_len, block_table, cache, first)
+                return self._grouped_decode(i, W, m, h, pos, slot_map, ctx_len, active, block_table, cache, first)
+            if m.kind == "lightning":
+                return self._lightning(W, m, h, lambda *a: X.lightning_decode(*a, cache.state(i), active))
             p, gates = self._mlstm_in(W, m, h)
             return X.mlstm_decode(p, gates, W["i.b"], W["f.b"], m.gate_cap, W["norm"], self.spec.norm_eps, m.dim, cache.state(i), active)
 

@@ -1,8 +1,8 @@
 """Description of decoders whose layers differ: a list of token mixers and feed-forwards with their own sizes.
 
 A *mixer stack* is a residual decoder in which every layer names its mixer (a kind of attention, a recurrent layer, ...), the
-mixer's sizes, and its feed-forward or none; a layer may reuse another layer's weights. Norms sit in front of the sublayers or
-on their outputs. The specs below are the typed form of such a configuration; ``DESIGNS`` maps the ``architecture`` of a
+mixer's sizes, and its feed-forward or none; a layer may reuse another layer's weights or its cached latents. Norms sit in front
+of the sublayers, on their outputs, or on both sides. The specs below are the typed form of such a configuration; ``DESIGNS`` maps the ``architecture`` of a
 ``config.json`` to the reader of its keys and is the place to register another design. Sizes and constants all come from the
 configuration.
 """
@@ -12,14 +12,14 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Callable, Optional, Union
 
-__all__ = ["RotarySpec", "LatentAttentionSpec", "GroupedAttentionSpec", "MLstmSpec", "DenseMlpSpec", "GatedMlpSpec", "MoeSpec", "LayerSpec",
+__all__ = ["RotarySpec", "LatentAttentionSpec", "GroupedAttentionSpec", "MLstmSpec", "LightningSpec", "DenseMlpSpec", "GatedMlpSpec", "MoeSpec", "LayerSpec",
            "StackSpec", "DESIGNS", "is_stack_config", "parse_stack"]
 
 
 @dataclass(frozen=True)
 class RotarySpec:
     """Rotary positions: frequencies of ``dims`` dimensions at ``base``, ``pairing`` of the dimensions ("interleaved": 2i with
-    2i + 1), and a context extension in the form ``ops.functional.rope_inv_freq`` reads."""
+    2i + 1; "halves": i with i + dims / 2), and a context extension in the form ``ops.functional.rope_inv_freq`` reads."""
 
     dims: int
     base: float
@@ -33,7 +33,8 @@ class RotarySpec:
 @dataclass(frozen=True)
 class LatentAttentionSpec:
     """Attention whose keys and values are expanded from one cached latent row per token (``kv_rank`` normed dimensions and
-    ``rot_dim`` rotated ones shared by all heads); queries go through a latent of ``q_rank``."""
+    ``rot_dim`` rotated ones shared by all heads). Queries go through a latent of ``q_rank`` (0: projected directly). A layer with
+    ``kv_from`` reads the rows that layer ``kv_from`` cached and has none of its own."""
 
     heads: int
     dim: int          # unrotated query / key size per head
@@ -44,11 +45,15 @@ class LatentAttentionSpec:
     scale: float
     rot: RotarySpec
     window: int = 0   # tokens a query sees, itself included; 0 = all
+    sink: bool = True         # one more score per head that has no value
+    gate: bool = True         # output times the sigmoid of one gate per head
+    kv_from: int = -1         # layer whose cached rows are used; -1: own rows
+    keep_first: int = 0
     kind: str = "latent_attention"
 
     @property
     def page_width(self) -> int:
-        return self.kv_rank + self.rot_dim
+        return self.kv_rank + self.rot_dim if self.kv_from < 0 else 0
 
     @property
     def state_size(self) -> int:
@@ -59,7 +64,9 @@ class LatentAttentionSpec:
 class GroupedAttentionSpec:
     """Grouped-query attention over cached keys and values: RMS norm per query / key head, rotation of the first ``rot.dims``
     dimensions, optional soft cap of the scores, an optional key of score 0 that has no value, and values mixed with those of
-    the stack's first value-mixing layer."""
+    the stack's first value-mixing layer. The norms carry weights and come before the rotation, or are plain and come after it
+    (``norm_after_rot``). The projections may have biases and pass a causal convolution of ``conv`` taps over time per channel,
+    whose last ``conv`` - 1 inputs are part of a sequence's state."""
 
     heads: int
     kv_heads: int
@@ -71,7 +78,15 @@ class GroupedAttentionSpec:
     zero_sink: bool = True    # one is added to the softmax denominator
     v_mix: bool = False
     window: int = 0
+    keep_first: int = 0       # first tokens of a sequence that every query sees besides its window
+    norm_after_rot: bool = False
+    bias: bool = False
+    conv: int = 1             # taps; 1 = no convolution
     kind: str = "attention"
+
+    @property
+    def channels(self) -> int:
+        return (self.heads + self.kv_heads) * self.dim + self.kv_heads * self.vdim
 
     @property
     def page_width(self) -> int:
@@ -79,7 +94,7 @@ class GroupedAttentionSpec:
 
     @property
     def state_size(self) -> int:
-        return 0
+        return (self.conv - 1) * self.channels
 
 
 @dataclass(frozen=True)
@@ -102,6 +117,26 @@ class MLstmSpec:
 
 
 @dataclass(frozen=True)
+class LightningSpec:
+    """Linear recurrence with one fixed decay per head: S = decay S + k v^T, read with q; q, k and v pass a silu. The heads' outputs
+    are normed together and gated."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    kind: str = "lightning"
+
+    @property
+    def page_width(self) -> int:
+        return 0
+
+    @property
+    def state_size(self) -> int:
+        return self.heads * self.dim * self.vdim
+
+
+@dataclass(frozen=True)
 class DenseMlpSpec:
     ff: int
     act: str = "gelu_erf"
@@ -118,21 +153,28 @@ class GatedMlpSpec:
 
 @dataclass(frozen=True)
 class MoeSpec:
-    """Gated experts of which every token uses ``top``: sigmoid scores, the score of a chosen expert scales the expert's input
-    (``renormalize``: scores divided by their sum first); a shared expert of ``shared_ff`` (0 = none) is added, multiplied by the
-    sigmoid of its own gate."""
+    """Gated experts of which every token uses ``top``: sigmoid scores, the score of a chosen expert scales the expert's input or
+    output (``renormalize``: scores divided by their sum first); a shared expert of ``shared_ff`` (0 = none) is added, multiplied by
+    the sigmoid of its own gate. Experts may be chosen by corrected scores (``correction``: one addend per expert) and from the
+    ``keep`` best of ``groups`` groups of neighbours (a group's score: the sum of its two largest). ``act``: "silu", or "clipped":
+    ``g sigmoid(1.702 g) (u + 1)`` with g <= ``limit`` and ``|u| <= limit``."""
 
     experts: int
     top: int
     ff: int
     shared_ff: int = 0
     renormalize: bool = False
+    correction: bool = False
+    groups: int = 1
+    keep: int = 1
+    act: str = "silu"         # "silu" scales the expert's input by the score, "clipped" its output
+    limit: float = 0.0
     kind: str = "moe"
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[LatentAttentionSpec, GroupedAttentionSpec, MLstmSpec]
+    mixer: Union[LatentAttentionSpec, GroupedAttentionSpec, MLstmSpec, LightningSpec]
     mlp: Union[DenseMlpSpec, GatedMlpSpec, MoeSpec, None]
     owner: int        # layer whose tensors this one uses (itself, or an earlier one with shared weights)
 
@@ -144,7 +186,7 @@ class StackSpec:
     norm: str         # "dynamic_tanh" | "rms"
     norm_eps: float   # eps of the RMS norms
     layers: tuple
-    norm_on: str = "input"        # where a sublayer's norm sits: on its "input" or on its "output"
+    norm_on: str = "input"        # where a sublayer's norm sits: on its "input", on its "output", or on "both" sides
     residual_mult: float = 1.0    # factor on what a sublayer adds to the stream
     embedding_norm: bool = False  # the embedding passes the stack's norm
     tied_head: bool = False       # the output matrix is the embedding table
@@ -161,7 +203,7 @@ class StackSpec:
 
 
 # --------------------------------------------------------------------------------------------- readers of config.json
-def _rotary(d: dict) -> RotarySpec:
+def _rotary(d: dict, pairing: str = "interleaved") -> RotarySpec:
     scaling = None
     s = d.get("scaling")
     if s:
@@ -169,7 +211,7 @@ def _rotary(d: dict) -> RotarySpec:
 
         scaling = {"rope_type": "yarn", "factor": float(s["factor"]), "original_max_position_embeddings": s["original"],
                    "beta_fast": float(s["fast"]), "beta_slow": float(s["slow"]), "attention_factor": 0.1 * math.log(float(s["factor"])) + 1.0}
-    return RotarySpec(dims=int(d["dims"]), base=float(d["base"]), scaling=scaling)
+    return RotarySpec(dims=int(d["dims"]), base=float(d["base"]), pairing=pairing, scaling=scaling)
 
 
 def _latent_attention(m: dict) -> LatentAttentionSpec:
@@ -190,6 +232,32 @@ def _grouped_attention(m: dict) -> GroupedAttentionSpec:
     return spec
 
 
+def _shared_latent_attention(m: dict) -> LatentAttentionSpec:
+    """Queries projected directly, no sink, no gate; the rows may be another layer's."""
+    mask = m.get("mask") or {}
+    return LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), q_rank=0, kv_rank=int(m["kv_rank"]),
+                               scale=float(m["scale"]), rot=_rotary(m["rot"]), window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
+                               sink=False, gate=False, kv_from=int(m["kv_from"]) if m.get("kv_from") is not None else -1)
+
+
+def _convolved_attention(m: dict) -> GroupedAttentionSpec:
+    """Biased, convolved projections; plain norms behind the rotation; a window that keeps the first tokens."""
+    mask = m.get("mask") or {}
+    spec = GroupedAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                                rot=_rotary(m["rot"], "halves"), zero_sink=False, window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
+                                norm_after_rot=True, bias=True, conv=int(m.get("conv") or 1))
+    if spec.heads % spec.kv_heads or spec.rot.dims % 2 or spec.rot.dims > spec.dim or spec.conv < 1:
+        raise ValueError(f"attention sizes: {spec}")
+    return spec
+
+
+def _lightning(m: dict) -> LightningSpec:
+    spec = LightningSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), decay=tuple(float(x) for x in m["decay"]))
+    if len(spec.decay) != spec.heads:
+        raise ValueError(f"one decay per head: {spec}")
+    return spec
+
+
 MIXER_READERS: dict[str, Callable[[dict], Any]] = {"latent_attention": _latent_attention, "mlstm": _mlstm, "attention": _grouped_attention}
 
 
@@ -200,6 +268,13 @@ def _mlp(d: Optional[dict], gated: bool = False) -> Union[DenseMlpSpec, GatedMlp
         return GatedMlpSpec(ff=int(d["ff"])) if gated else DenseMlpSpec(ff=int(d["ff"]))
     if d.get("kind") == "moe" and gated:
         r = d["router"]
+        if "limit" in d["expert"]:
+            g = r.get("groups") or {}
+            spec = MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(d["expert"]["ff"]), renormalize=True, correction=True,
+                           groups=int(g.get("count", 1)), keep=int(g.get("keep", g.get("count", 1))), act="clipped", limit=float(d["expert"]["limit"]))
+            if spec.experts % spec.groups or not 1 <= spec.keep <= spec.groups or not 1 <= spec.top <= spec.keep * (spec.experts // spec.groups):
+                raise ValueError(f"expert groups: {spec}")
+            return spec
         return MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(d["expert"]["ff"]), shared_ff=int((d.get("shared") or {}).get("ff", 0)))
     raise NotImplementedError(f"feed-forward kind {d.get('kind')!r}")
 
@@ -215,11 +290,13 @@ def _owner(layers: list, i: int) -> int:
 
 
 def _layers(d: dict, mixers: tuple, gated: bool = False) -> tuple:
+    """``mixers``: the design's mixer types, or a type -> reader mapping where they differ from ``MIXER_READERS``."""
+    readers = mixers if isinstance(mixers, dict) else {t: MIXER_READERS[t] for t in mixers}
     layers = []
     for i, l in enumerate(d["layers"]):
-        if l["type"] not in mixers:
+        if l["type"] not in readers:
             raise NotImplementedError(f"mixer type {l['type']!r}")
-        layers.append(LayerSpec(mixer=MIXER_READERS[l["type"]](l["mixer"]), mlp=_mlp(l.get("mlp"), gated), owner=_owner(d["layers"], i)))
+        layers.append(LayerSpec(mixer=readers[l["type"]](l["mixer"]), mlp=_mlp(l.get("mlp"), gated), owner=_owner(d["layers"], i)))
     return tuple(layers)
 
 
@@ -237,7 +314,21 @@ def parse_tofinex(d: dict) -> StackSpec:
     return spec
 
 
-DESIGNS: dict[str, Callable[[dict], StackSpec]] = {"Zorelorn": parse_zorelorn, "Tofinex": parse_tofinex}
+def parse_luzitar(d: dict) -> StackSpec:
+    readers = {"lightning": _lightning, "attention": _convolved_attention, "latent_attention": _shared_latent_attention}
+    spec = StackSpec(design="Luzitar", embedding_scale=1.0, norm="dynamic_tanh", norm_eps=float(d["norm"]["eps"]), layers=_layers(d, readers, gated=True),
+                     norm_on="both", embedding_norm=True, logit_softcap=float(d.get("logit_softcap") or 0.0))
+    for i, l in enumerate(spec.layers):
+        j = getattr(l.mixer, "kv_from", -1)
+        if j < 0:
+            continue
+        m, src = l.mixer, spec.layers[j].mixer if j < i else None
+        if src is None or src.kind != "latent_attention" or src.kv_from >= 0 or (src.kv_rank, src.rot_dim, src.rot) != (m.kv_rank, m.rot_dim, m.rot):
+            raise ValueError(f"layer {i}: kv_from {j} must be an earlier latent layer with rows of its own, of the same sizes and rotation")
+    return spec
+
+
+DESIGNS: dict[str, Callable[[dict], StackSpec]] = {"Zorelorn": parse_zorelorn, "Tofinex": parse_tofinex, "Luzitar": parse_luzitar}
 
 
 def is_stack_config(d: dict) -> bool:
@@ -271,26 +362,37 @@ def layer_tensors(spec: StackSpec, width: int, i: int) -> list:
     """Stored tensors of layer ``i`` (a weight owner): ``(name, shape, initialisation, weight decay)``. Projections of the same
     input are one matrix; its rows are padded to a multiple of 8."""
     l, p = spec.layers[i], f"l{i}."
-    out = norm_tensors(spec, p + "norm1", width)
+    sides = lambda name: norm_tensors(spec, p + name, width) + (norm_tensors(spec, p + name + "b", width) if spec.norm_on == "both" else [])
+    out = sides("norm1")
     m, f = l.mixer, l.mlp
     if m.kind == "latent_attention":
-        out += [(p + "mix.in", (m.q_rank + m.kv_rank + m.rot_dim + _up8(m.heads), width), "normal", True),
-                (p + "mix.dq.norm", (m.q_rank,), "ones", False), (p + "mix.dkv.norm", (m.kv_rank,), "ones", False),
-                (p + "mix.uq", (m.heads * (m.dim + m.rot_dim), m.q_rank), "normal", True),
-                (p + "mix.ukv", (m.heads * (m.dim + m.vdim), m.kv_rank), "normal", True),
-                (p + "mix.sink", (m.heads,), "zeros", False), (p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
+        # queries (or their latent), key / value latent with the rotated key part, gates
+        rows = m.kv_rank + m.rot_dim if m.kv_from < 0 else 0
+        n = (m.q_rank or _up8(m.heads * (m.dim + m.rot_dim))) + rows
+        out += [(p + "mix.in", (n + _up8(m.heads) if m.gate else _up8(n), width), "normal", True)]
+        out += [(p + "mix.dq.norm", (m.q_rank,), "ones", False)] if m.q_rank else []
+        out += [(p + "mix.dkv.norm", (m.kv_rank,), "ones", False)] if rows else []
+        out += [(p + "mix.uq", (m.heads * (m.dim + m.rot_dim), m.q_rank), "normal", True)] if m.q_rank else []
+        out += [(p + "mix.ukv", (m.heads * (m.dim + m.vdim), m.kv_rank), "normal", True)]
+        out += [(p + "mix.sink", (m.heads,), "zeros", False)] if m.sink else []
+        out += [(p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
     elif m.kind == "attention":
-        out += [(p + "mix.in", (_up8((m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim), width), "normal", True),
-                (p + "mix.q.norm", (m.dim,), "ones", False), (p + "mix.k.norm", (m.dim,), "ones", False)]
+        out += [(p + "mix.in", (_up8(m.channels), width), "normal", True)]
+        out += [(p + "mix.in.b", (_up8(m.channels),), "zeros", False)] if m.bias else []
+        out += [(p + "mix.in.conv", (m.channels, m.conv), "normal", False)] if m.conv > 1 else []
+        out += [] if m.norm_after_rot else [(p + "mix.q.norm", (m.dim,), "ones", False), (p + "mix.k.norm", (m.dim,), "ones", False)]
         out += [(p + "mix.vmix", (1,), "fill:0.5", False)] if m.v_mix else []
         out += [(p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
+    elif m.kind == "lightning":
+        out += [(p + "mix.in", (_up8(2 * m.heads * (m.dim + m.vdim)), width), "normal", True), (p + "mix.norm", (m.heads * m.vdim,), "ones", False),
+                (p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
     else:
         out += [(p + "mix.in", (2 * m.heads * (m.dim + m.vdim) + _up8(2 * m.heads), width), "normal", True),
                 (p + "mix.i.b", (m.heads,), "zeros", False), (p + "mix.f.b", (m.heads,), "fill:4.0", False),
                 (p + "mix.norm", (m.heads * m.vdim,), "ones", False), (p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
     if f is None:
         return out
-    out += norm_tensors(spec, p + "norm2", width)
+    out += sides("norm2")
     if f.kind == "dense":
         out += [(p + "mlp.up", (f.ff, width), "normal", True), (p + "mlp.down", (width, f.ff), "normal", True)]
     elif f.kind == "gated":
@@ -298,6 +400,7 @@ def layer_tensors(spec: StackSpec, width: int, i: int) -> list:
     else:
         # one matrix for everything that reads every token (shared expert, router, shared gate); the experts' are stacked
         out += [(p + "mlp.in", (2 * f.shared_ff + _up8(f.experts + (1 if f.shared_ff else 0)), width), "normal", True)]
+        out += [(p + "mlp.correction", (f.experts,), "zeros", False)] if f.correction else []
         out += [(p + "mlp.shared.down", (width, f.shared_ff), "normal", True)] if f.shared_ff else []
         out += [(p + "mlp.experts.in", (f.experts * 2 * f.ff, width), "normal", True), (p + "mlp.experts.down", (f.experts * width, f.ff), "normal", True)]
     return out
@@ -316,10 +419,20 @@ def fused_rows(spec: StackSpec, width: int, i: int) -> dict:
     """Fused tensor of layer ``i`` -> [(checkpoint name, first row, rows)]."""
     m, f, p = spec.layers[i].mixer, spec.layers[i].mlp, f"l{i}.mix."
     if m.kind == "latent_attention":
-        out = {p + "in": _consecutive((p + "dq", m.q_rank), (p + "dkv", m.kv_rank + m.rot_dim), (p + "g", m.heads)),
-               p + "ukv": _consecutive((p + "uk", m.heads * m.dim), (p + "uv", m.heads * m.vdim))}
+        q = m.heads * (m.dim + m.rot_dim)
+        rows = [("dq", 0, m.q_rank)] if m.q_rank else [("q", 0, q)]
+        at = m.q_rank or _up8(q)
+        if m.kv_from < 0:
+            rows += [("dkv", at, m.kv_rank + m.rot_dim)]
+            at += m.kv_rank + m.rot_dim
+        rows += [("g", at, m.heads)] if m.gate else []
+        out = {p + "in": [(p + name, r0, n) for name, r0, n in rows], p + "ukv": _consecutive((p + "uk", m.heads * m.dim), (p + "uv", m.heads * m.vdim))}
     elif m.kind == "attention":
-        out = {p + "in": _consecutive((p + "q", m.heads * m.dim), (p + "k", m.kv_heads * m.dim), (p + "v", m.kv_heads * m.vdim))}
+        sizes = (("q", m.heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim))
+        out = {p + "in" + what: _consecutive(*((p + name + what, n) for name, n in sizes)) for what in ("", *([".b"] if m.bias else []), *([".conv"] if m.conv > 1 else []))}
+    elif m.kind == "lightning":
+        qk, v = m.heads * m.dim, m.heads * m.vdim
+        out = {p + "in": _consecutive((p + "q", qk), (p + "k", qk), (p + "v", v), (p + "g", v))}
     else:
         qk, v = m.heads * m.dim, m.heads * m.vdim
         out = {p + "in": _consecutive((p + "q", qk), (p + "k", qk), (p + "v", v), (p + "g", v), (p + "i", m.heads), (p + "f", m.heads))}

@@ -1,6 +1,6 @@
 """Operators of the mixer stacks (``models/mixer_stack.py``): norms, GEMMs with fused epilogues, latent attention over expanded
 keys (prompts) and over the paged latents (decoding), grouped-query attention with capped scores over cached keys and values,
-mixtures of experts, and the mLSTM recurrence.
+mixtures of experts, short convolutions, and the mLSTM and lightning recurrences.
 
 As in ``functional``: CUDA tensors go to the hand-written kernels (bf16 or true fp32; nothing falls back silently), CPU
 tensors take a plain PyTorch path. The residual stream, gates, statistics and recurrent state are fp32 on every path.
@@ -19,7 +19,8 @@ from . import native
 __all__ = ["embed_dyt", "dynamic_tanh", "linear_act", "linear_split", "linear_residual_", "rope_pairs_", "latent_prep", "gather_pages",
            "headwise_linear", "latent_absorb", "latent_attention_prefill", "latent_attention_decode", "mlstm_prefill", "mlstm_decode",
            "embed_rms", "linear_partial", "linear_softcap", "residual_rms_", "gated_silu", "gated_up", "gated_up_split", "ExpertPlan", "expert_dispatch",
-           "expert_up", "expert_down", "qkv_prep", "grouped_attention_prefill", "grouped_attention_decode"]
+           "expert_up", "expert_down", "qkv_prep", "grouped_attention_prefill", "grouped_attention_decode", "embed_dyt2", "linear_bias",
+           "linear_silu", "residual_dyt_", "conv_qkv_prep", "lightning_prefill", "lightning_decode", "gated_rms"]
 
 
 def _ops():
@@ -46,6 +47,18 @@ def embed_dyt(ids, weight, scale: float, alpha, nw, nb):
     return x, dynamic_tanh(x, alpha, nw, nb)
 
 
+def embed_dyt2(ids, weight, embed_norm, first_norm):
+    """(fp32 residual stream: the Dynamic Tanh ``embed_norm`` of ``weight[ids]``, the Dynamic Tanh ``first_norm`` of that stream)."""
+    if weight.is_cuda:
+        return _ops().embed_dyt2(ids.reshape(-1).contiguous(), weight, *embed_norm, *first_norm)
+    x = dynamic_tanh_f32(weight[ids.reshape(-1)].float(), *embed_norm)
+    return x, dynamic_tanh(x, *first_norm)
+
+
+def dynamic_tanh_f32(x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    return torch.tanh(alpha.float() * x) * weight.float() + bias.float()
+
+
 def linear_act(a: torch.Tensor, w: torch.Tensor, act: Optional[str] = None, out_f32: bool = False) -> torch.Tensor:
     """``a w^T`` with an optional activation (``gelu_erf``) in the epilogue."""
     assert act in (None, "gelu_erf")
@@ -64,14 +77,40 @@ def linear_split(a: torch.Tensor, w: torch.Tensor, n0: int):
     return y[:, :n0].to(a.dtype).contiguous(), y[:, n0:].contiguous()
 
 
-def linear_residual_(a: torch.Tensor, w: torch.Tensor, x: torch.Tensor, norm=None) -> Optional[torch.Tensor]:
-    """``x += a w^T`` on the fp32 residual stream; with ``norm = (alpha, weight, bias)`` also returns the Dynamic Tanh of the
-    new stream, computed in the same epilogue."""
+def linear_bias(a: torch.Tensor, w: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
+    """``a w^T + b``."""
     if a.is_cuda:
-        h = _ops().linear_residual_(a, w, x, *(norm if norm is not None else (None, None, None)))
+        return _ops().linear_bias(a, w, b)
+    return (_mm(a, w) + b.float()).to(a.dtype)
+
+
+def linear_silu(a: torch.Tensor, w: torch.Tensor, n0: int) -> torch.Tensor:
+    """``a w^T`` with a silu on the first ``n0`` columns."""
+    if a.is_cuda:
+        return _ops().linear_silu(a, w, int(n0))
+    y = _mm(a, w)
+    return torch.cat([TF.silu(y[:, :n0]), y[:, n0:]], -1).to(a.dtype)
+
+
+def linear_residual_(a: torch.Tensor, w: torch.Tensor, x: torch.Tensor, norm=None, post=None) -> Optional[torch.Tensor]:
+    """``x += a w^T`` on the fp32 residual stream, or with ``post = (alpha, weight, bias)`` the Dynamic Tanh of that product; with
+    ``norm`` (likewise) also returns the Dynamic Tanh of the new stream, computed in the same epilogue."""
+    none = (None, None, None)
+    if a.is_cuda:
+        h = _ops().linear_residual_(a, w, x, *(norm if norm is not None else none), *(post if post is not None else none))
         return h if norm is not None else None
-    x += _mm(a, w)
+    y = _mm(a, w)
+    x += y if post is None else dynamic_tanh_f32(y, *post)
     return dynamic_tanh(x, *norm) if norm is not None else None
+
+
+def residual_dyt_(x, rows, slot, post, norm) -> torch.Tensor:
+    """``x += post(Y)`` on the fp32 residual stream with Y[t] the sum of the expert rows ``rows[slot[t, j]]``; returns ``norm`` of the
+    new stream (both Dynamic Tanh ``(alpha, weight, bias)``)."""
+    if x.is_cuda:
+        return _ops().residual_dyt_(x, rows, slot, *post, *norm)
+    x += dynamic_tanh_f32(rows[slot.long()].float().sum(1), *post)
+    return dynamic_tanh(x, *norm)
 
 
 # ----------------------------------------------------------------------------------------------- RMS norms on sublayer outputs
@@ -160,14 +199,25 @@ class ExpertPlan:
     num_tiles: torch.Tensor
 
 
-def expert_dispatch(h: torch.Tensor, logits: torch.Tensor, experts: int, top: int, renormalize: bool = False) -> ExpertPlan:
+def expert_dispatch(h: torch.Tensor, logits: torch.Tensor, experts: int, top: int, renormalize: bool = False, correction: Optional[torch.Tensor] = None,
+                    groups: int = 1, keep: int = 1) -> ExpertPlan:
     """Router: the ``top`` experts with the largest ``sigmoid(logits)`` of every token (``logits`` fp32, columns past ``experts``
-    ignored), and the tokens' copies in expert order. No host synchronisation."""
+    ignored), and the tokens' copies in expert order. ``correction`` [experts] is added for the choice only. With ``groups`` > 1 only
+    experts of the ``keep`` best groups of neighbours can be chosen; a group counts the sum of its two largest choice scores. No
+    host synchronisation."""
     if h.is_cuda:
-        return ExpertPlan(*_ops().expert_dispatch(h, logits, int(experts), int(top), bool(renormalize)))
-    s, e = torch.topk(torch.sigmoid(logits[:, :experts].float()), top, dim=-1)
+        return ExpertPlan(*_ops().expert_dispatch(h, logits, int(experts), int(top), bool(renormalize), correction, int(groups), int(keep)))
+    score = torch.sigmoid(logits[:, :experts].float())
+    choice = score if correction is None else score + correction.float()
+    if groups > 1:
+        g = choice.view(-1, groups, experts // groups)
+        best = torch.topk(torch.topk(g, min(2, g.shape[2]), dim=-1).values.sum(-1), keep, dim=-1).indices
+        hidden = torch.ones(g.shape[:2], dtype=torch.bool).scatter_(1, best, False)
+        choice = g.masked_fill(hidden.unsqueeze(-1), float("-inf")).flatten(1)
+    e = torch.topk(choice, top, dim=-1).indices
+    s = score.gather(1, e)
     if renormalize:
-        s = s / s.sum(-1, keepdim=True)
+        s = s / (s.sum(-1, keepdim=True) + 1e-20)
     order = torch.argsort(e.reshape(-1), stable=True)
     slot = torch.empty_like(order)
     slot[order] = torch.arange(order.numel())
@@ -176,15 +226,21 @@ def expert_dispatch(h: torch.Tensor, logits: torch.Tensor, experts: int, top: in
     return ExpertPlan(h[order // top], slot.view(-1, top), s.reshape(-1)[order], first, first[-1:])
 
 
-def expert_up(plan: ExpertPlan, w: torch.Tensor, ff: int) -> torch.Tensor:
-    """Per copy ``silu(s g) * (s u)`` with [g | u] = ``x w_e^T`` and the copy's score s (a factor on the expert's input); ``w``
-    [E * 2 ff, width]."""
+def expert_up(plan: ExpertPlan, w: torch.Tensor, ff: int, act: str = "silu", limit: float = 0.0) -> torch.Tensor:
+    """Per copy ``silu(s g) * (s u)`` with [g | u] = ``x w_e^T`` and the copy's score s (a factor on the expert's input), or with
+    ``act`` "clipped" ``s g sigmoid(1.702 g) (u + 1)`` with g <= limit and -limit <= u <= limit; ``w`` [E * 2 ff, width]."""
+    assert act in ("silu", "clipped") and (act == "silu" or limit > 0)
     w3 = w.view(-1, 2 * ff, w.shape[1])
     if w.is_cuda:
-        return _ops().expert_up(plan.x, w3, plan.scale, plan.tile_expert, plan.num_tiles)
+        return _ops().expert_up(plan.x, w3, plan.scale, plan.tile_expert, plan.num_tiles, float(limit) if act == "clipped" else 0.0)
     out = torch.empty(plan.x.shape[0], ff, dtype=plan.x.dtype)
     for e in range(w3.shape[0]):
         at = slice(int(plan.tile_expert[e]), int(plan.tile_expert[e + 1]))
+        if act == "clipped":
+            g, u = _mm(plan.x[at], w3[e]).chunk(2, -1)
+            g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+            out[at] = (g * torch.sigmoid(1.702 * g) * (u + 1.0) * plan.scale[at, None]).to(out.dtype)
+            continue
         g, u = (_mm(plan.x[at], w3[e]) * plan.scale[at, None]).chunk(2, -1)
         out[at] = (TF.silu(g) * u).to(out.dtype)
     return out
@@ -223,14 +279,14 @@ def rope_pairs_(x: torch.Tensor, positions: torch.Tensor, cos: torch.Tensor, sin
 
 
 def latent_prep(p, q_norm, kv_norm, eps: float, positions, cos, sin, pages=None, slots=None, want_rows: bool = False):
-    """``p`` [T, q_rank + kv_rank + rot]: RMS-normed query latent, and the row [normed latent | rotated shared key part], which
-    is appended to ``pages`` [blocks, block_size, kv_rank + rot] at ``slots`` (negative: skipped) and / or returned."""
+    """``p`` [T, q_rank + kv_rank + rot]: RMS-normed query latent (``q_norm`` None: there is none), and the row [normed latent |
+    rotated shared key part], which is appended to ``pages`` [blocks, block_size, kv_rank + rot] at ``slots`` (negative: skipped) and / or returned."""
     if p.is_cuda:
         return _ops().latent_prep(p, q_norm, kv_norm, float(eps), positions, cos, sin, pages, slots, bool(want_rows))
-    qr, kr = q_norm.numel(), kv_norm.numel()
+    qr, kr = q_norm.numel() if q_norm is not None else 0, kv_norm.numel()
     rms = lambda z, w: z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) * w.float()
     f = p.float()
-    cq = rms(f[:, :qr], q_norm).to(p.dtype)
+    cq = rms(f[:, :qr], q_norm).to(p.dtype) if qr else p[:, :0]
     row = torch.cat([rms(f[:, qr : qr + kr], kv_norm), _rotate(f[:, qr + kr :], positions, cos, sin)], -1).to(p.dtype)
     if pages is not None:
         ok = slots >= 0
@@ -278,12 +334,25 @@ def _sink_softmax(s: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor
     return torch.softmax(torch.cat([s, extra], -1), -1)[..., :-1]
 
 
-def latent_attention_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, window: int, scale: float, sink=None, gate=None) -> torch.Tensor:
+def _hidden_keys(nq: int, nk: int, window: int, keep_first: int) -> torch.Tensor:
+    """[nq, nk]: keys a query does not see; the last query sits on the last key."""
+    dist, key = torch.arange(nk - nq, nk)[:, None] - torch.arange(nk)[None, :], torch.arange(nk)[None, :]
+    return (dist < 0) | ((dist >= window) & (key >= keep_first) if window > 0 else torch.zeros_like(dist, dtype=torch.bool))
+
+
+def _seen_keys(n: int, window: int, keep_first: int) -> torch.Tensor:
+    """Positions the last of ``n`` tokens sees."""
+    key = torch.arange(n)
+    return key[(key >= n - window) | (key < keep_first)] if window > 0 else key
+
+
+def latent_attention_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, window: int, scale: float, sink=None, gate=None, keep_first: int = 0) -> torch.Tensor:
     """Causal windowed attention of packed prompts: ``q`` [T, H, du + dr] (rotated part last), ``k_unrot`` [Tk, H, du], ``k_rot``
     [Tk, dr] shared by the heads, ``v`` [Tk, H, dv]; the last query of a sequence sits on its last key (``cu_k`` may hold earlier
-    keys). ``window`` > 0: a query sees that many keys, its own included. Output times ``sigmoid(gate[t, h])``."""
+    keys). ``window`` > 0: a query sees that many keys, its own included, and the first ``keep_first`` keys of the sequence. Output
+    times ``sigmoid(gate[t, h])``."""
     if q.is_cuda:
-        return _ops().latent_attn_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, sink, gate, int(window), float(scale))
+        return _ops().latent_attn_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, sink, gate, int(window), float(scale), int(keep_first))
     out = torch.empty(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype)
     du = k_unrot.shape[2]
     cq, ck = cu_q.tolist(), cu_k.tolist()
@@ -292,8 +361,7 @@ def latent_attention_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, window: int, scal
         nq, nk = cq[b + 1] - cq[b], ck[b + 1] - ck[b]
         qq = q[qs].float()
         s = torch.einsum("qhd,khd->hqk", qq[..., :du], k_unrot[ks].float()) + torch.einsum("qhd,kd->hqk", qq[..., du:], k_rot[ks].float())
-        dist = torch.arange(nk - nq, nk)[:, None] - torch.arange(nk)[None, :]
-        hide = (dist < 0) | ((dist >= window) if window > 0 else torch.zeros_like(dist, dtype=torch.bool))
+        hide = _hidden_keys(nq, nk, window, keep_first)
         p = _sink_softmax((s * scale).masked_fill(hide, float("-inf")), sink)
         o = torch.einsum("hqk,khd->qhd", p, v[ks].float())
         if gate is not None:
@@ -302,17 +370,17 @@ def latent_attention_prefill(q, k_unrot, k_rot, v, cu_q, cu_k, window: int, scal
     return out
 
 
-def latent_attention_decode(q, pages, block_table, ctx_len, kv_rank: int, window: int, scale: float, sink=None) -> torch.Tensor:
+def latent_attention_decode(q, pages, block_table, ctx_len, kv_rank: int, window: int, scale: float, sink=None, keep_first: int = 0) -> torch.Tensor:
     """One query per sequence in the latent space: ``q`` [S, H, kv_rank + rot] against the cached rows, which are key (whole row)
     and value (first ``kv_rank``) of every head. Returns [S, H, kv_rank]; sequences with ``ctx_len`` 0 give zeros."""
     if q.is_cuda:
-        return _ops().latent_attn_decode(q, pages, block_table, ctx_len, sink, int(kv_rank), int(window), float(scale))
+        return _ops().latent_attn_decode(q, pages, block_table, ctx_len, sink, int(kv_rank), int(window), float(scale), int(keep_first))
     out = torch.zeros(q.shape[0], q.shape[1], kv_rank, dtype=q.dtype)
     bs = pages.shape[1]
     for b, n in enumerate(ctx_len.tolist()):
         if n <= 0:
             continue
-        at = torch.arange(max(0, n - window) if window > 0 else 0, n)
+        at = _seen_keys(n, window, keep_first)
         rows = pages[block_table[b, at // bs].long(), at % bs].float()
         p = _sink_softmax(q[b].float() @ rows.t() * scale, sink)
         out[b] = (p @ rows[:, :kv_rank]).to(q.dtype)
@@ -349,11 +417,12 @@ def _soft_cap(s: torch.Tensor, cap: float) -> torch.Tensor:
     return cap * torch.tanh(s / cap) if cap > 0 else s
 
 
-def grouped_attention_prefill(q, k, v, cu_q, cu_k, window: int, scale: float, softcap: float = 0.0, sink=None) -> torch.Tensor:
+def grouped_attention_prefill(q, k, v, cu_q, cu_k, window: int, scale: float, softcap: float = 0.0, sink=None,
+                              keep_first: int = 0) -> torch.Tensor:
     """Causal attention of packed prompts: ``q`` [T, H, d], ``k`` [Tk, G, d], ``v`` [Tk, G, e] (query head h reads key head h // (H / G));
-    scores ``softcap * tanh(q k scale / softcap)``; ``cu_q`` / ``cu_k`` / ``window`` / ``sink`` as in ``latent_attention_prefill``."""
+    scores ``softcap * tanh(q k scale / softcap)``; ``cu_q`` / ``cu_k`` / ``window`` / ``keep_first`` / ``sink`` as in ``latent_attention_prefill``."""
     if q.is_cuda:
-        return _ops().grouped_attn_prefill(q, k, v, cu_q, cu_k, sink, int(window), float(scale), float(softcap))
+        return _ops().grouped_attn_prefill(q, k, v, cu_q, cu_k, sink, int(window), float(scale), float(softcap), int(keep_first))
     out = torch.empty(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype)
     n = q.shape[1] // k.shape[1]
     cq, ck = cu_q.tolist(), cu_k.tolist()
@@ -361,31 +430,138 @@ def grouped_attention_prefill(q, k, v, cu_q, cu_k, window: int, scale: float, so
         qs, ks = slice(cq[b], cq[b + 1]), slice(ck[b], ck[b + 1])
         nq, nk = cq[b + 1] - cq[b], ck[b + 1] - ck[b]
         s = _soft_cap(torch.einsum("qhd,khd->hqk", q[qs].float(), k[ks].float().repeat_interleave(n, 1)) * scale, softcap)
-        dist = torch.arange(nk - nq, nk)[:, None] - torch.arange(nk)[None, :]
-        hide = (dist < 0) | ((dist >= window) if window > 0 else torch.zeros_like(dist, dtype=torch.bool))
+        hide = _hidden_keys(nq, nk, window, keep_first)
         w = _sink_softmax(s.masked_fill(hide, float("-inf")), sink)
         out[qs] = torch.einsum("hqk,khd->qhd", w, v[ks].float().repeat_interleave(n, 1)).to(q.dtype)
     return out
 
 
 def grouped_attention_decode(q, pages, block_table, ctx_len, kv_heads: int, vdim: int, window: int, scale: float, softcap: float = 0.0,
-                             sink=None) -> torch.Tensor:
+                             sink=None, keep_first: int = 0) -> torch.Tensor:
     """One query per sequence, ``q`` [S, H, d], against cached rows [keys | values] (``qkv_prep``). Returns [S, H, vdim]; sequences
     with ``ctx_len`` 0 give zeros."""
     if q.is_cuda:
-        return _ops().grouped_attn_decode(q, pages, block_table, ctx_len, sink, int(kv_heads), int(vdim), int(window), float(scale), float(softcap))
+        return _ops().grouped_attn_decode(q, pages, block_table, ctx_len, sink, int(kv_heads), int(vdim), int(window), float(scale), float(softcap),
+                                          int(keep_first))
     out = torch.zeros(q.shape[0], q.shape[1], vdim, dtype=q.dtype)
     bs, G, d = pages.shape[1], kv_heads, q.shape[2]
     for b, n in enumerate(ctx_len.tolist()):
         if n <= 0:
             continue
-        at = torch.arange(max(0, n - window) if window > 0 else 0, n)
+        at = _seen_keys(n, window, keep_first)
         rows = pages[block_table[b, at // bs].long(), at % bs].float()
         k, v = rows[:, : G * d].view(-1, G, d), rows[:, G * d :].view(-1, G, vdim)
         s = _soft_cap(torch.einsum("gnd,kgd->gnk", q[b].float().view(G, -1, d), k).flatten(0, 1) * scale, softcap)
         w = _sink_softmax(s, sink)
         out[b] = torch.einsum("gnk,kge->gne", w.view(G, -1, len(at)), v).flatten(0, 1).to(q.dtype)
     return out
+
+
+# ----------------------------------------------------------------------------------------------- short convolution in front of attention
+def _rotate_halves(x: torch.Tensor, pos: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+    """``x`` [T, heads, n] fp32: pairs (i, i + half) of the first ``2 * half`` dimensions are turned."""
+    half = cos.shape[1]
+    c, s = cos[pos.long()][:, None], sin[pos.long()][:, None]
+    u, v = x[..., :half], x[..., half : 2 * half]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half :]], -1)
+
+
+def _conv_portion(u: torch.Tensor, w: torch.Tensor, past: torch.Tensor):
+    """``u`` [n, C] behind ``past`` [taps - 1, C]: (outputs [n, C], the last taps - 1 inputs)."""
+    taps = w.shape[1]
+    row = torch.cat([past, u], 0)
+    return sum(row[j : j + u.shape[0]] * w[:, j].float() for j in range(taps)), row[row.shape[0] - taps + 1 :]
+
+
+def conv_qkv_prep(p, conv, eps: float, positions, cos, sin, heads: int, kv_heads: int, dim: int, vdim: int, halves: bool = True, cu=None, state=None, slots=None,
+                  fresh=None, active=None, pages=None, page_slots=None, want_rows: bool = False):
+    """``p`` [T, q | k | v]: causal convolution over time (``conv`` [channels, taps], None: none; zeros before a sequence's first
+    token), rotation of the first ``2 * cos.shape[1]`` dimensions of every query and key head (pairs (i, i + half), or (2i, 2i + 1)
+    without ``halves``), then an RMS norm without weight over the head. Portions (``cu`` given): sequence b goes on from the inputs in
+    ``state[slots[b]]`` unless ``fresh[b]``, and leaves its last ones there; without ``slots`` every sequence starts from zeros and
+    nothing is kept. Steps (``cu`` None): row s is the next token of ``state[s]`` where ``active[s]``. ``state`` rows: [taps - 1, channels]
+    fp32, oldest first. Returns (queries [T, heads, dim], rows [keys | values]) as ``qkv_prep``."""
+    if p.is_cuda:
+        return _ops().conv_qkv_prep(p, conv, float(eps), positions, cos, sin, int(heads), int(kv_heads), int(dim), int(vdim), bool(halves), cu, state, slots,
+                                    fresh, active, pages, page_slots, bool(want_rows))
+    T, C = p.shape[0], (heads + kv_heads) * dim + kv_heads * vdim
+    f = p[:, :C].float()
+    if conv is not None and conv.shape[1] > 1:
+        n, u, f = conv.shape[1] - 1, f, torch.zeros(T, C)
+        if cu is None:
+            for s in torch.nonzero(active).flatten().tolist():
+                past = state[s].view(n, C)
+                f[s : s + 1], last = _conv_portion(u[s : s + 1], conv, past.clone())
+                past.copy_(last)
+        else:
+            c = cu.tolist()
+            for b in range(len(c) - 1):
+                past = state[int(slots[b])].view(n, C) if slots is not None else None
+                f[c[b] : c[b + 1]], last = _conv_portion(u[c[b] : c[b + 1]], conv, torch.zeros(n, C) if past is None or bool(fresh[b]) else past.clone())
+                if past is not None:
+                    past.copy_(last)
+    elif conv is not None:
+        f = f * conv[:, 0].float()
+    a, b = heads * dim, (heads + kv_heads) * dim
+    turn = _rotate_halves if halves else _rotate
+    unit = lambda z: z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps)
+    q = unit(turn(f[:, :a].view(T, heads, dim), positions, cos, sin)).to(p.dtype)
+    k = unit(turn(f[:, a:b].view(T, kv_heads, dim), positions, cos, sin))
+    row = torch.cat([k.flatten(1), f[:, b:]], -1).to(p.dtype)
+    if pages is not None:
+        ok = page_slots >= 0
+        at, bs = page_slots[ok], pages.shape[1]
+        pages[at // bs, at % bs] = row[ok]
+    return q, (row if want_rows else row[:0])
+
+
+# ----------------------------------------------------------------------------------------------- lightning recurrence
+def _lightning_token(S, decay, q, k, v):
+    """One token of one sequence, in place on S [H, d, e]; returns o [H, e]."""
+    S.mul_(decay[:, None, None]).add_(k[:, :, None] * v[:, None, :])
+    return torch.einsum("hde,hd->he", S, q)
+
+
+def _lightning_parts(p, decay, dim: int, vdim: int):
+    H, T, f = decay.numel(), p.shape[0], p.float()
+    return f[:, : H * dim].view(T, H, dim), f[:, H * dim : 2 * H * dim].view(T, H, dim), f[:, 2 * H * dim : 2 * H * dim + H * vdim].view(T, H, vdim)
+
+
+def lightning_prefill(p, decay, dim: int, vdim: int, cu, state=None, slots=None, fresh=None, all_fresh: bool = False) -> torch.Tensor:
+    """``S = decay S + k v^T``, ``o = S^T q`` per head over packed portions; ``p`` [T, q | k | v | ...] (activated), ``decay`` [H] fp32.
+    ``cu`` / ``state`` / ``slots`` / ``fresh`` / ``all_fresh`` as in ``mlstm_prefill`` with state rows [H, dim, vdim]. Returns [T, H vdim]."""
+    if p.is_cuda:
+        return _ops().lightning_prefill(p, decay, int(dim), int(vdim), cu, state, slots, fresh, bool(all_fresh))
+    H = decay.numel()
+    q, k, v = _lightning_parts(p, decay, dim, vdim)
+    out = torch.empty(p.shape[0], H, vdim)
+    c = cu.tolist()
+    for b in range(len(c) - 1):
+        S = torch.zeros(H, dim, vdim) if slots is None else state[int(slots[b])].view(H, dim, vdim)
+        if slots is not None and bool(fresh[b]):
+            S.zero_()
+        for t in range(c[b], c[b + 1]):
+            out[t] = _lightning_token(S, decay, q[t], k[t], v[t])
+    return out.flatten(1).to(p.dtype)
+
+
+def lightning_decode(p, decay, dim: int, vdim: int, state, active) -> torch.Tensor:
+    """One token per slot: row s of ``p`` updates ``state[s]`` when ``active[s]`` (inactive slots keep theirs and give zeros)."""
+    if p.is_cuda:
+        return _ops().lightning_decode(p, decay, int(dim), int(vdim), state, active)
+    H = decay.numel()
+    q, k, v = _lightning_parts(p, decay, dim, vdim)
+    out = torch.zeros(p.shape[0], H, vdim)
+    for s in torch.nonzero(active).flatten().tolist():
+        out[s] = _lightning_token(state[s].view(H, dim, vdim), decay, q[s], k[s], v[s])
+    return out.flatten(1).to(p.dtype)
+
+
+def gated_rms(o: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, eps: float) -> torch.Tensor:
+    """``rms_norm(o) * norm * sigmoid(gate)`` over whole rows."""
+    if o.is_cuda:
+        return _ops().gated_rms(o, gate, norm, float(eps))
+    return (_rms(o.float(), norm, eps) * torch.sigmoid(gate.float())).to(norm.dtype)
 
 
 # ----------------------------------------------------------------------------------------------- mLSTM
