@@ -73,8 +73,32 @@ std::tuple<Tensor, Tensor> linear_split(const Tensor& a, const Tensor& w, int64_
   return {d, d2};
 }
 
-// x += a w^T (fp32 residual stream); returns tanh(alpha x) nw + nb in a's type, or an empty tensor without a norm.
-Tensor linear_residual_(const Tensor& a, const Tensor& w, Tensor x, const OptTensor& alpha, const OptTensor& nw, const OptTensor& nb) {
+Tensor linear_bias(const Tensor& a, const Tensor& w, const Tensor& b) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  same(a, b, "linear_bias");
+  TORCH_CHECK(b.numel() == w.size(0) && b.is_contiguous(), "linear_bias: bias [N]");
+  Tensor d = at::empty({a.size(0), w.size(0)}, a.options());
+  VbEpiArgs e{};
+  e.mode = VB_EPI_BIAS;
+  e.D = d.data_ptr(); e.ldd = d.stride(0); e.nb = b.data_ptr();
+  run_gemm(a, w, e);
+  return d;
+}
+
+Tensor linear_silu(const Tensor& a, const Tensor& w, int64_t n0) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  Tensor d = at::empty({a.size(0), w.size(0)}, a.options());
+  VbEpiArgs e{};
+  e.mode = VB_EPI_SILU;
+  e.D = d.data_ptr(); e.ldd = d.stride(0); e.n0 = (int)n0;
+  run_gemm(a, w, e);
+  return d;
+}
+
+// x += a w^T, or x += tanh(palpha a w^T) pw + pb (fp32 residual stream); returns tanh(alpha x) nw + nb in a's type, or an empty tensor
+// without a norm.
+Tensor linear_residual_(const Tensor& a, const Tensor& w, Tensor x, const OptTensor& alpha, const OptTensor& nw, const OptTensor& nb, const OptTensor& palpha,
+                        const OptTensor& pw, const OptTensor& pb) {
   const c10::cuda::CUDAGuard guard(a.device());
   CHECK_F32(x);
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && x.size(0) == a.size(0) && x.size(1) == w.size(0), "linear_residual_: x [M, N]");
@@ -92,6 +116,13 @@ Tensor linear_residual_(const Tensor& a, const Tensor& w, Tensor x, const OptTen
   } else {
     h = at::empty({0}, a.options());
   }
+  if (pw.has_value()) {
+    same(a, *pw, "linear_residual_");
+    same(a, *pb, "linear_residual_");
+    same(a, *palpha, "linear_residual_");
+    TORCH_CHECK(pw->numel() == w.size(0) && pb->numel() == w.size(0) && palpha->numel() == 1, "linear_residual_: norm sizes");
+    e.palpha = palpha->data_ptr(); e.pw = pw->data_ptr(); e.pb = pb->data_ptr();
+  }
   run_gemm(a, w, e);
   return h;
 }
@@ -107,6 +138,57 @@ std::tuple<Tensor, Tensor> embed_dyt(const Tensor& ids, const Tensor& w, double 
   CHECK_RC(vb_embed_dyt(dt, lptr(ids), w.data_ptr(), (float)scale, x.data_ptr<float>(), h.data_ptr(), alpha.data_ptr(), nw.data_ptr(),
                         nb.data_ptr(), T, W, (int)w.size(0), cur_stream()), "vb_embed_dyt");
   return {x, h};
+}
+
+std::tuple<Tensor, Tensor> embed_dyt2(const Tensor& ids, const Tensor& w, const Tensor& ealpha, const Tensor& ew, const Tensor& eb, const Tensor& alpha,
+                                      const Tensor& nw, const Tensor& nb) {
+  const int dt = dtype_of(w);
+  const c10::cuda::CUDAGuard guard(w.device());
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && w.is_contiguous() && nw.numel() == w.size(1) && nb.numel() == w.size(1) &&
+              ew.numel() == w.size(1) && eb.numel() == w.size(1) && ealpha.numel() == 1 && alpha.numel() == 1, "embed_dyt2");
+  for (const Tensor* t : {&nw, &nb, &alpha, &ew, &eb, &ealpha}) same(w, *t, "embed_dyt2");
+  const int T = (int)ids.numel(), W = (int)w.size(1);
+  Tensor x = at::empty({T, W}, w.options().dtype(at::kFloat)), h = at::empty({T, W}, w.options());
+  verl_count_launches(1);
+  CHECK_RC(vb_embed_dyt2(dt, lptr(ids), w.data_ptr(), x.data_ptr<float>(), h.data_ptr(), ealpha.data_ptr(), ew.data_ptr(), eb.data_ptr(), alpha.data_ptr(),
+                         nw.data_ptr(), nb.data_ptr(), T, W, (int)w.size(0), cur_stream()), "vb_embed_dyt2");
+  return {x, h};
+}
+
+// x += post(sum_j rows[slot[t, j]]); returns norm(x) in the norm's type (both Dynamic Tanh).
+Tensor residual_dyt_(Tensor x, const Tensor& rows, const Tensor& slot, const Tensor& palpha, const Tensor& pw, const Tensor& pb, const Tensor& alpha, const Tensor& nw,
+                     const Tensor& nb) {
+  CHECK_F32(x);
+  CHECK_I32(slot);
+  const int dt = dtype_of(nw);
+  const c10::cuda::CUDAGuard guard(x.device());
+  for (const Tensor* t : {&rows, &palpha, &pw, &pb, &alpha, &nb}) same(nw, *t, "residual_dyt_");
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && rows.dim() == 2 && rows.stride(1) == 1 && rows.size(1) == x.size(1) && slot.dim() == 2 && slot.size(0) == x.size(0) &&
+              nw.numel() == x.size(1) && nb.numel() == x.size(1) && pw.numel() == x.size(1) && pb.numel() == x.size(1) && alpha.numel() == 1 && palpha.numel() == 1,
+              "residual_dyt_: sizes");
+  VbResidDyt p{};
+  p.x = x.data_ptr<float>(); p.rows = rows.data_ptr(); p.ldr = rows.stride(0); p.slot = slot.data_ptr<int>(); p.top = (int)slot.size(1);
+  p.palpha = palpha.data_ptr(); p.pw = pw.data_ptr(); p.pb = pb.data_ptr(); p.alpha = alpha.data_ptr(); p.nw = nw.data_ptr(); p.nb = nb.data_ptr();
+  p.T = (int)x.size(0); p.W = (int)x.size(1);
+  Tensor h = at::empty({p.T, p.W}, nw.options());
+  p.h = h.data_ptr();
+  verl_count_launches(1);
+  CHECK_RC(vb_residual_dyt(dt, &p, cur_stream()), "vb_residual_dyt");
+  return h;
+}
+
+// rms_norm(o) norm sigmoid(g) over whole rows (strided views).
+Tensor gated_rms(const Tensor& o, const Tensor& g, const Tensor& norm, double eps) {
+  const int dt = dtype_of(o);
+  same(o, g, "gated_rms");
+  same(o, norm, "gated_rms");
+  TORCH_CHECK(o.dim() == 2 && g.sizes() == o.sizes() && o.stride(1) == 1 && g.stride(1) == 1 && norm.numel() == o.size(1), "gated_rms: [T, W]");
+  const c10::cuda::CUDAGuard guard(o.device());
+  Tensor out = at::empty(o.sizes(), o.options());
+  verl_count_launches(1);
+  CHECK_RC(vb_gated_rms(dt, o.data_ptr(), o.stride(0), g.data_ptr(), g.stride(0), norm.data_ptr(), (float)eps, out.data_ptr(), (int)o.size(0), (int)o.size(1),
+                        cur_stream()), "vb_gated_rms");
+  return out;
 }
 
 Tensor dynamic_tanh(const Tensor& x, const Tensor& alpha, const Tensor& nw, const Tensor& nb) {
@@ -135,13 +217,13 @@ void rope_pairs_(Tensor x, const Tensor& pos, const Tensor& cs, const Tensor& sn
 }
 
 // p [T, q_rank + kv_rank + rot]; pages: view [blocks, block_size, kv_rank + rot] of the cache (or none), slot int64 [T] (negative: no append).
-std::tuple<Tensor, Tensor> latent_prep(const Tensor& p, const Tensor& qn, const Tensor& kn, double eps, const Tensor& pos, const Tensor& cs,
+std::tuple<Tensor, Tensor> latent_prep(const Tensor& p, const OptTensor& qn, const Tensor& kn, double eps, const Tensor& pos, const Tensor& cs,
                                        const Tensor& sn, const OptTensor& pages, const OptTensor& slot, bool want_rows) {
   const int dt = dtype_of(p);
   CHECK_I32(pos);
-  same(p, qn, "latent_prep");
+  if (qn.has_value()) same(p, *qn, "latent_prep");
   same(p, kn, "latent_prep");
-  const int64_t T = p.size(0), qr = qn.numel(), kr = kn.numel(), rot = p.size(1) - qr - kr;
+  const int64_t T = p.size(0), qr = qn.has_value() ? qn->numel() : 0, kr = kn.numel(), rot = p.size(1) - qr - kr;
   TORCH_CHECK(p.stride(1) == 1 && rot >= 0 && pos.numel() == T && cs.is_contiguous() && sn.is_contiguous() && 2 * cs.size(1) <= std::max<int64_t>(rot, 0), "latent_prep: sizes");
   const c10::cuda::CUDAGuard guard(p.device());
   Tensor cq = at::empty({T, qr}, p.options());
@@ -155,7 +237,7 @@ std::tuple<Tensor, Tensor> latent_prep(const Tensor& p, const Tensor& qn, const 
     ps = pages->stride(0); bs = (int)pages->size(1); slots = pages->size(0) * pages->size(1);
   }
   verl_count_launches(1);
-  CHECK_RC(vb_latent_prep(dt, p.data_ptr(), p.stride(0), qn.data_ptr(), kn.data_ptr(), (float)eps, pos.data_ptr<int>(), cs.data_ptr<float>(),
+  CHECK_RC(vb_latent_prep(dt, p.data_ptr(), p.stride(0), ptr(qn), kn.data_ptr(), (float)eps, pos.data_ptr<int>(), cs.data_ptr<float>(),
                           sn.data_ptr<float>(), (int)(2 * cs.size(1)), (int)cs.size(0), cq.data_ptr(), want_rows ? lat.data_ptr() : nullptr, kr + rot, ptr(pages), ps, bs,
                           slots, pages.has_value() ? lptr(*slot) : nullptr, (int)T, (int)qr, (int)kr, (int)rot, cur_stream()), "vb_latent_prep");
   return {cq, lat};
@@ -231,7 +313,7 @@ Tensor latent_absorb(const Tensor& q, const Tensor& uk, const Tensor& pos, const
 
 // Prompt attention: q [T, H, du + dr], ku [Tk, H, du], kr [Tk, dr], v [Tk, H, dv] (strided views), cu_q / cu_k int32 [B + 1].
 Tensor latent_attn_prefill(const Tensor& q, const Tensor& ku, const Tensor& kr, const Tensor& v, const Tensor& cu_q, const Tensor& cu_k,
-                           const OptTensor& sink, const OptTensor& gate, int64_t window, double scale) {
+                           const OptTensor& sink, const OptTensor& gate, int64_t window, double scale, int64_t keep_first) {
   const int dt = dtype_of(q);
   CHECK_I32(cu_q);
   CHECK_I32(cu_k);
@@ -246,7 +328,7 @@ Tensor latent_attn_prefill(const Tensor& q, const Tensor& ku, const Tensor& kr, 
   a.v = v.data_ptr(); a.v_row = v.stride(0); a.v_head = (int)v.stride(1);
   a.cu_q = cu_q.data_ptr<int>(); a.cu_k = cu_k.data_ptr<int>();
   a.T = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)ku.size(2); a.dr = (int)kr.size(1); a.dv = (int)v.size(2);
-  a.B = (int)cu_q.numel() - 1; a.window = (int)window; a.scale = (float)scale;
+  a.B = (int)cu_q.numel() - 1; a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale;
   if (sink.has_value()) { same(q, *sink, "latent_attn_prefill"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
   if (gate.has_value()) { CHECK_F32(*gate); TORCH_CHECK(gate->size(0) == a.T && gate->stride(1) == 1); a.gate = gate->data_ptr<float>(); a.ldg = gate->stride(0); }
   Tensor out = at::empty({q.size(0), q.size(1), v.size(2)}, q.options());
@@ -260,7 +342,7 @@ Tensor latent_attn_prefill(const Tensor& q, const Tensor& ku, const Tensor& kr, 
 
 // Decode attention in the latent space: q [S, H, kv_rank + rot] (absorbed query, rotated part last), pages [blocks, block_size, kv_rank + rot].
 Tensor latent_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& block_table, const Tensor& ctx_len, const OptTensor& sink,
-                          int64_t kv_rank, int64_t window, double scale) {
+                          int64_t kv_rank, int64_t window, double scale, int64_t keep_first) {
   const int dt = dtype_of(q);
   same(q, pages, "latent_attn_decode");
   CHECK_I32(block_table);
@@ -277,13 +359,13 @@ Tensor latent_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& bl
   a.block_table = block_table.data_ptr<int>(); a.max_blocks = (int)block_table.size(1); a.block_size = (int)pages.size(1); a.page_stride = pages.stride(0);
   a.ctx_len = ctx_len.data_ptr<int>();
   a.T = a.B = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)kv_rank; a.dr = (int)(q.size(2) - kv_rank); a.dv = (int)kv_rank;
-  a.window = (int)window; a.scale = (float)scale;
+  a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale;
   if (sink.has_value()) { same(q, *sink, "latent_attn_decode"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
   Tensor out = at::empty({q.size(0), q.size(1), kv_rank}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   if (dt == 1) {
     const int64_t all = (int64_t)a.max_blocks * a.block_size;
-    const int ns = vb_latent_decode_splits(a.B, a.H, a.dv, a.du + a.dr, a.block_size, (int)(window > 0 ? std::min<int64_t>(window + 32, all) : all));
+    const int ns = vb_latent_decode_splits(a.B, a.H, a.dv, a.du + a.dr, a.block_size, (int)(window > 0 ? std::min<int64_t>(window + keep_first + 64, all) : all));
     if (ns > 0) {
       Tensor po, ml;
       if (ns > 1) {
@@ -386,26 +468,29 @@ Tensor residual_rms_(Tensor x, const OptTensor& y, const Tensor& nw, double eps,
   return h;
 }
 
-Tensor gated_silu_rows(const Tensor& gu, const float* row_scale) {
+Tensor gated_silu_rows(const Tensor& gu, const float* row_scale, float clip) {
   const int dt = dtype_of(gu);
   TORCH_CHECK(gu.dim() == 2 && gu.stride(1) == 1 && gu.size(1) % 2 == 0, "gated_silu: [T, 2 I]");
   Tensor out = at::empty({gu.size(0), gu.size(1) / 2}, gu.options());
   verl_count_launches(1);
-  CHECK_RC(vb_gated_silu(dt, gu.data_ptr(), gu.stride(0), row_scale, out.data_ptr(), (int)out.size(0), (int)out.size(1), cur_stream()), "vb_gated_silu");
+  CHECK_RC(vb_gated_silu(dt, gu.data_ptr(), gu.stride(0), row_scale, clip, out.data_ptr(), (int)out.size(0), (int)out.size(1), cur_stream()), "vb_gated_silu");
   return out;
 }
 Tensor gated_silu(const Tensor& gu) {
   const c10::cuda::CUDAGuard guard(gu.device());
-  return gated_silu_rows(gu, nullptr);
+  return gated_silu_rows(gu, nullptr, 0.f);
 }
 
 // Router and expert-grouped copies of the tokens: (x [rows, W], slot [T, k], score per row, expert per 128-row tile, number of tiles).
-std::tuple<Tensor, Tensor, Tensor, Tensor, Tensor> expert_dispatch(const Tensor& h, const Tensor& z, int64_t E, int64_t k, bool renorm) {
+std::tuple<Tensor, Tensor, Tensor, Tensor, Tensor> expert_dispatch(const Tensor& h, const Tensor& z, int64_t E, int64_t k, bool renorm,
+                                                                   const OptTensor& corr, int64_t groups, int64_t keep) {
   const int dt = dtype_of(h);
   CHECK_F32(z);
   const c10::cuda::CUDAGuard guard(h.device());
   const int64_t T = h.size(0), W = h.size(1);
   TORCH_CHECK(h.dim() == 2 && h.stride(1) == 1 && z.dim() == 2 && z.stride(1) == 1 && z.size(0) == T && z.size(1) >= E && k >= 1 && k <= E, "expert_dispatch");
+  TORCH_CHECK(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && k <= keep * (E / groups), "expert_dispatch: groups");
+  if (corr.has_value()) { same(h, *corr, "expert_dispatch"); TORCH_CHECK(corr->numel() == E && corr->is_contiguous(), "expert_dispatch: correction [E]"); }
   const int64_t tiles = std::max<int64_t>(1, (T * k + 127) / 128 + std::min<int64_t>(E, T * k));
   const auto i32 = h.options().dtype(at::kInt), f32 = h.options().dtype(at::kFloat);
   Tensor counts = at::zeros({E}, i32), expert = at::empty({T, k}, i32), rank = at::empty({T, k}, i32), slot = at::empty({T, k}, i32);
@@ -413,7 +498,7 @@ std::tuple<Tensor, Tensor, Tensor, Tensor, Tensor> expert_dispatch(const Tensor&
   Tensor x = at::empty({tiles * 128, W}, h.options());
   if (T == 0) { num_tiles.zero_(); return {x, slot, row_scale, tile_expert, num_tiles}; }
   verl_count_launches(2);
-  CHECK_RC(vb_expert_route(z.data_ptr<float>(), z.stride(0), (int)T, (int)E, (int)k, renorm, score.data_ptr<float>(), expert.data_ptr<int>(), rank.data_ptr<int>(),
+  CHECK_RC(vb_expert_route(dt, z.data_ptr<float>(), z.stride(0), ptr(corr), (int)groups, (int)keep, (int)T, (int)E, (int)k, renorm, score.data_ptr<float>(), expert.data_ptr<int>(), rank.data_ptr<int>(),
                            counts.data_ptr<int>(), cur_stream()), "vb_expert_route");
   CHECK_RC(vb_expert_place(dt, h.data_ptr(), h.stride(0), score.data_ptr<float>(), expert.data_ptr<int>(), rank.data_ptr<int>(), counts.data_ptr<int>(), (int)T, (int)E,
                            (int)k, (int)W, x.data_ptr(), row_scale.data_ptr<float>(), slot.data_ptr<int>(), tile_expert.data_ptr<int>(), num_tiles.data_ptr<int>(),
@@ -446,8 +531,8 @@ Tensor expert_linear(const Tensor& a, const Tensor& w, const Tensor& tile_expert
   return d;
 }
 
-// act[rows, I] = silu(s g) * (s u), [g | u] = x w_e^T, w [E, 2 I, K], s = scale[row].
-Tensor expert_up(const Tensor& x, const Tensor& w, const Tensor& scale, const Tensor& tile_expert, const Tensor& num_tiles) {
+// act[rows, I] = silu(s g) * (s u), [g | u] = x w_e^T, w [E, 2 I, K], s = scale[row]; clip > 0: s g sigmoid(1.702 g) (u + 1), g <= clip, |u| <= clip.
+Tensor expert_up(const Tensor& x, const Tensor& w, const Tensor& scale, const Tensor& tile_expert, const Tensor& num_tiles, double clip) {
   CHECK_F32(scale);
   CHECK_I32(tile_expert);
   CHECK_I32(num_tiles);
@@ -459,14 +544,14 @@ Tensor expert_up(const Tensor& x, const Tensor& w, const Tensor& scale, const Te
   if (dtype_of(x) == 1) {
     Tensor act = at::empty({rows, I}, x.options());
     const int rc = vb_gemm_grouped_swiglu(x.data_ptr(), w.data_ptr(), act.data_ptr(), rows, I, K, x.stride(0), I, scale.data_ptr<float>(), (int)w.size(0),
-                                          tile_expert.data_ptr<int>(), num_tiles.data_ptr<int>(), cur_stream());
+                                          tile_expert.data_ptr<int>(), num_tiles.data_ptr<int>(), (float)clip, cur_stream());
     if (rc >= 0) {
       verl_count_launches(1);
       CHECK_RC(rc, "expert_up");
       return act;
     }
   }
-  return gated_silu_rows(expert_linear(x, w, tile_expert, num_tiles), scale.data_ptr<float>());
+  return gated_silu_rows(expert_linear(x, w, tile_expert, num_tiles), scale.data_ptr<float>(), (float)clip);
 }
 
 // p [T, q | k | v]; see VbQkvPrep. Returns (queries [T, H, dim], rows [T or 0, G (dim + vdim)]).
@@ -511,7 +596,7 @@ std::tuple<Tensor, Tensor> qkv_prep(const Tensor& p, const Tensor& qn, const Ten
 
 // Prompt attention: q [T, H, d], k [Tk, G, d], v [Tk, G, e] (strided views), cu_q / cu_k int32 [B + 1].
 Tensor grouped_attn_prefill(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& cu_q, const Tensor& cu_k, const OptTensor& sink, int64_t window,
-                            double scale, double softcap) {
+                            double scale, double softcap, int64_t keep_first) {
   const int dt = dtype_of(q);
   CHECK_I32(cu_q);
   CHECK_I32(cu_k);
@@ -526,7 +611,7 @@ Tensor grouped_attn_prefill(const Tensor& q, const Tensor& k, const Tensor& v, c
   a.v = v.data_ptr(); a.v_row = v.stride(0); a.v_head = (int)v.stride(1);
   a.cu_q = cu_q.data_ptr<int>(); a.cu_k = cu_k.data_ptr<int>();
   a.T = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)q.size(2); a.dv = (int)v.size(2); a.B = (int)cu_q.numel() - 1;
-  a.window = (int)window; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / k.size(1));
+  a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / k.size(1));
   if (sink.has_value()) { same(q, *sink, "grouped_attn_prefill"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
   Tensor out = at::empty({q.size(0), q.size(1), v.size(2)}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
@@ -539,7 +624,7 @@ Tensor grouped_attn_prefill(const Tensor& q, const Tensor& k, const Tensor& v, c
 
 // Decode attention: q [S, H, d], pages [blocks, block_size, G (d + vdim)] with rows [keys | values].
 Tensor grouped_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& block_table, const Tensor& ctx_len, const OptTensor& sink, int64_t G, int64_t vdim,
-                           int64_t window, double scale, double softcap) {
+                           int64_t window, double scale, double softcap, int64_t keep_first) {
   const int dt = dtype_of(q);
   same(q, pages, "grouped_attn_decode");
   CHECK_I32(block_table);
@@ -557,13 +642,13 @@ Tensor grouped_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& b
   a.block_table = block_table.data_ptr<int>(); a.max_blocks = (int)block_table.size(1); a.block_size = (int)pages.size(1); a.page_stride = pages.stride(0);
   a.ctx_len = ctx_len.data_ptr<int>();
   a.T = a.B = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)d; a.dv = (int)vdim;
-  a.window = (int)window; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / G);
+  a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / G);
   if (sink.has_value()) { same(q, *sink, "grouped_attn_decode"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
   Tensor out = at::empty({q.size(0), q.size(1), vdim}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   if (dt == 1) {
     const int64_t all = (int64_t)a.max_blocks * a.block_size;
-    const int ns = vb_grouped_decode_splits(&a, (int)(window > 0 ? std::min<int64_t>(window + 64, all) : all));
+    const int ns = vb_grouped_decode_splits(&a, (int)(window > 0 ? std::min<int64_t>(window + keep_first + 128, all) : all));
     if (ns > 0) {
       Tensor po, ml;
       if (ns > 1) {
@@ -580,6 +665,128 @@ Tensor grouped_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& b
   }
   verl_count_launches(1);
   CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
+  return out;
+}
+
+// p [T, q | k | v]; see VbConvPrep. cu given: portions, else one token per slot. Returns (queries [T, H, dim], rows [T or 0, G (dim + vdim)]).
+std::tuple<Tensor, Tensor> conv_qkv_prep(const Tensor& p, const OptTensor& conv, double eps, const Tensor& pos, const Tensor& cs, const Tensor& sn, int64_t H, int64_t G,
+                                         int64_t dim, int64_t vdim, bool halves, const OptTensor& cu, const OptTensor& state, const OptTensor& slots,
+                                         const OptTensor& fresh, const OptTensor& active, const OptTensor& pages, const OptTensor& page_slot, bool want_rows) {
+  const int dt = dtype_of(p);
+  CHECK_I32(pos);
+  CHECK_F32(cs);
+  CHECK_F32(sn);
+  const int64_t T = p.size(0), C = (H + G) * dim + G * vdim, width = G * (dim + vdim);
+  TORCH_CHECK(p.dim() == 2 && p.stride(1) == 1 && p.size(1) >= C && H > 0 && G > 0 && pos.numel() == T && cs.dim() == 2 && cs.is_contiguous() && sn.is_contiguous() &&
+              sn.sizes() == cs.sizes() && 2 * cs.size(1) <= dim, "conv_qkv_prep: sizes");
+  const c10::cuda::CUDAGuard guard(p.device());
+  VbConvPrep a{};
+  a.taps = 1;
+  if (conv.has_value()) {
+    same(p, *conv, "conv_qkv_prep");
+    TORCH_CHECK(conv->dim() == 2 && conv->size(0) == C && conv->size(1) >= 1 && conv->is_contiguous(), "conv_qkv_prep: conv [channels, taps]");
+    a.conv = conv->data_ptr(); a.taps = (int)conv->size(1);
+  }
+  if (cu.has_value()) {
+    CHECK_I32(*cu);
+    a.cu = cu->data_ptr<int>(); a.B = (int)cu->numel() - 1;
+  }
+  if (state.has_value() && a.taps > 1) {
+    CHECK_F32(*state);
+    TORCH_CHECK(state->dim() == 2 && state->stride(1) == 1 && state->size(1) == (a.taps - 1) * C, "conv_qkv_prep: state [slots, (taps - 1) channels]");
+    a.state = state->data_ptr<float>(); a.slot_stride = state->stride(0);
+    if (cu.has_value()) {
+      TORCH_CHECK(slots.has_value() && fresh.has_value() && slots->numel() == a.B && fresh->numel() == a.B, "conv_qkv_prep: slots and fresh [B]");
+      CHECK_I32(*slots);
+      CHECK_I32(*fresh);
+      a.slots = slots->data_ptr<int>(); a.fresh = fresh->data_ptr<int>();
+    } else {
+      TORCH_CHECK(state->size(0) >= T, "conv_qkv_prep: one state row per token of a step");
+    }
+  }
+  if (!cu.has_value()) {
+    TORCH_CHECK(active.has_value() && active->is_cuda() && active->scalar_type() == at::kBool && active->is_contiguous() && active->numel() == T, "conv_qkv_prep: active [S]");
+    TORCH_CHECK(a.taps == 1 || a.state != nullptr, "conv_qkv_prep: steps need a state");
+    a.active = reinterpret_cast<const uint8_t*>(active->data_ptr());
+  }
+  Tensor q = at::empty({T, H, dim}, p.options()), rows = at::empty({want_rows ? T : 0, width}, p.options());
+  a.p = p.data_ptr(); a.ldp = p.stride(0); a.pos = pos.data_ptr<int>(); a.cos_t = cs.data_ptr<float>(); a.sin_t = sn.data_ptr<float>();
+  a.half = (int)cs.size(1); a.max_pos = (int)cs.size(0); a.halves = halves;
+  a.q = q.data_ptr(); a.ldr = width; a.block_size = 1;
+  if (want_rows) a.rows = rows.data_ptr();
+  if (pages.has_value()) {
+    same(p, *pages, "conv_qkv_prep");
+    TORCH_CHECK(pages->dim() == 3 && pages->size(2) == width && pages->stride(2) == 1 && pages->stride(1) == width && page_slot.has_value() && page_slot->is_cuda() &&
+                page_slot->scalar_type() == at::kLong && page_slot->is_contiguous() && page_slot->numel() == T, "conv_qkv_prep: pages [blocks, block_size, kv_heads (dim + vdim)]");
+    a.pages = pages->data_ptr(); a.page_stride = pages->stride(0); a.block_size = (int)pages->size(1); a.num_slots = pages->size(0) * pages->size(1);
+    a.page_slot = lptr(*page_slot);
+  }
+  a.T = (int)T; a.H = (int)H; a.G = (int)G; a.dim = (int)dim; a.vdim = (int)vdim; a.eps = (float)eps;
+  verl_count_launches(a.cu != nullptr && a.state != nullptr ? 2 : 1);
+  CHECK_RC(vb_conv_prep(dt, &a, cur_stream()), "vb_conv_prep");
+  return {q, rows};
+}
+
+// p [T, q | k | v | ...], decay fp32 [H]
+VbLightning lightning_args(const Tensor& p, const Tensor& decay, int64_t d, int64_t e, const OptTensor& state, Tensor& out) {
+  CHECK_F32(decay);
+  const int64_t H = decay.numel();
+  TORCH_CHECK(p.dim() == 2 && p.stride(1) == 1 && d > 0 && e > 0 && p.size(1) >= H * (2 * d + e) && decay.is_contiguous(), "lightning: rows [q | k | v]");
+  VbLightning a{};
+  if (state.has_value()) {
+    CHECK_F32(*state);
+    TORCH_CHECK(state->dim() == 2 && state->stride(1) == 1 && state->size(1) == H * d * e, "lightning: state [slots, H d e]");
+    a.state = state->data_ptr<float>(); a.slot_stride = state->stride(0);
+  }
+  out = at::empty({p.size(0), H * e}, p.options());
+  a.p = p.data_ptr(); a.ldp = p.stride(0); a.decay = decay.data_ptr<float>(); a.out = out.data_ptr(); a.ldo = out.stride(0);
+  a.T = (int)p.size(0); a.H = (int)H; a.d = (int)d; a.e = (int)e;
+  return a;
+}
+
+Tensor lightning_decode(const Tensor& p, const Tensor& decay, int64_t d, int64_t e, Tensor state, const Tensor& active) {
+  const int dt = dtype_of(p);
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor out;
+  VbLightning a = lightning_args(p, decay, d, e, state, out);
+  TORCH_CHECK(active.is_cuda() && active.scalar_type() == at::kBool && active.is_contiguous() && active.numel() == a.T && state.size(0) >= a.T, "lightning_decode: active [S]");
+  a.active = reinterpret_cast<const uint8_t*>(active.data_ptr());
+  verl_count_launches(1);
+  CHECK_RC(vb_lightning_decode(dt, &a, cur_stream()), "vb_lightning_decode");
+  return out;
+}
+
+Tensor lightning_prefill(const Tensor& p, const Tensor& decay, int64_t d, int64_t e, const Tensor& cu, const OptTensor& state, const OptTensor& slots, const OptTensor& fresh,
+                         bool all_fresh) {
+  const int dt = dtype_of(p);
+  CHECK_I32(cu);
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor out;
+  VbLightning a = lightning_args(p, decay, d, e, state, out);
+  a.B = (int)cu.numel() - 1;
+  a.cu = cu.data_ptr<int>();
+  if (slots.has_value()) {
+    TORCH_CHECK(state.has_value() && fresh.has_value() && slots->numel() == a.B && fresh->numel() == a.B, "lightning_prefill: slots need a state");
+    CHECK_I32(*slots);
+    CHECK_I32(*fresh);
+    a.slots = slots->data_ptr<int>(); a.fresh = fresh->data_ptr<int>();
+  }
+  if (a.T == 0 || a.B == 0) return out;
+  if (dt == 1) {
+    const int nseg = vb_lightning_chunk_segments(a.T, a.B, a.H, a.d, a.e, all_fresh || !slots.has_value());
+    if (nseg > 0) {
+      Tensor local;
+      if (nseg > 1) local = at::empty({(int64_t)a.B * (nseg - 1) * a.H * d * e}, p.options().dtype(at::kFloat));
+      const int rc = vb_lightning_chunk(&a, nseg, nseg > 1 ? local.data_ptr<float>() : nullptr, cur_stream());
+      if (rc >= 0) {
+        verl_count_launches(nseg > 1 ? 2 : 1);
+        CHECK_RC(rc, "vb_lightning_chunk");
+        return out;
+      }
+    }
+  }
+  verl_count_launches(1);
+  CHECK_RC(vb_lightning_scan(dt, &a, cur_stream()), "vb_lightning_scan");
   return out;
 }
 
@@ -685,6 +892,14 @@ TORCH_LIBRARY_FRAGMENT(verl_b200, m) {
   m.def("qkv_prep", &qkv_prep);
   m.def("grouped_attn_prefill", &grouped_attn_prefill);
   m.def("grouped_attn_decode", &grouped_attn_decode);
+  m.def("linear_bias", &linear_bias);
+  m.def("linear_silu", &linear_silu);
+  m.def("embed_dyt2", &embed_dyt2);
+  m.def("residual_dyt_", &residual_dyt_);
+  m.def("gated_rms", &gated_rms);
+  m.def("conv_qkv_prep", &conv_qkv_prep);
+  m.def("lightning_decode", &lightning_decode);
+  m.def("lightning_prefill", &lightning_prefill);
   m.def("mlstm_decode", &mlstm_decode);
   m.def("mlstm_prefill", &mlstm_prefill);
 }

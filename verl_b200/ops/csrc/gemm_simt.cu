@@ -50,6 +50,7 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, int M, int N,
     __syncthreads();
   }
   const float alpha = (e.mode == VB_EPI_RESID && e.D != nullptr) ? to_f(*reinterpret_cast<const T*>(e.alpha)) : 0.f;
+  const float palpha = (e.mode == VB_EPI_RESID && e.pw != nullptr) ? to_f(*reinterpret_cast<const T*>(e.palpha)) : 0.f;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
@@ -67,11 +68,14 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, int M, int N,
         case VB_EPI_STORE_F32: (reinterpret_cast<float*>(e.D) + blockIdx.z * sd)[m * e.ldd + n] = v; break;
         case VB_EPI_SOFTCAP: D[m * e.ldd + n] = from_f<T>(e.cap * tanhf(v / e.cap)); break;
         case VB_EPI_GELU: D[m * e.ldd + n] = from_f<T>(gelu_erf(v)); break;
+        case VB_EPI_BIAS: D[m * e.ldd + n] = from_f<T>(v + to_f(reinterpret_cast<const T*>(e.nb)[n])); break;
+        case VB_EPI_SILU: D[m * e.ldd + n] = from_f<T>(n < e.n0 ? v * sigmoid_f(v) : v); break;
         case VB_EPI_SPLIT:
           if (n < e.n0) D[m * e.ldd + n] = from_f<T>(v);
           else e.D2[m * e.ldd2 + n - e.n0] = v;
           break;
         default: {
+          if (e.pw != nullptr) v = tanhf(palpha * v) * to_f(reinterpret_cast<const T*>(e.pw)[n]) + to_f(reinterpret_cast<const T*>(e.pb)[n]);
           const float x = e.X[m * e.ldx + n] + v;
           e.X[m * e.ldx + n] = x;
           if (e.D != nullptr)

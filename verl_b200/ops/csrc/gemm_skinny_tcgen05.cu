@@ -220,8 +220,11 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
     const int q = warp & 3;  // TMEM lane quarter this warp may access
     const int et = threadIdx.x - 64;
     uint32_t acc_phase = 0;
-    float mix_alpha = 0.f;
-    if constexpr (EPI == SK_MIX) mix_alpha = epi_alpha(p.mix);
+    float mix_alpha = 0.f, mix_palpha = 0.f;
+    if constexpr (EPI == SK_MIX) {
+      mix_alpha = epi_alpha(p.mix);
+      mix_palpha = epi_palpha(p.mix);
+    }
     for (int it = blockIdx.x; it < num_items; it += gridDim.x) {
       const SkItem w = sk_item(p, it);
       const int nl = q * 32 + lane;          // weight row within the tile
@@ -251,7 +254,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
             const EpiColumn ec = epi_column(p.mix, col);
 #pragma unroll
             for (int j = 0; j < 32; ++j)
-              if (j < mrem) epi_store1(p.mix, tok0 + c * 32 + j, col, __uint_as_float(r[j]), mix_alpha, ec);
+              if (j < mrem) epi_store1(p.mix, tok0 + c * 32 + j, col, __uint_as_float(r[j]), mix_alpha, mix_palpha, ec);
           } else if (direct) {
 #pragma unroll
             for (int j = 0; j < 32; ++j)
@@ -330,7 +333,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
               if (EPI == SK_MIX) {
                 if (mm < r1) {
                   const float v4[4] = {a[u].x, a[u].y, a[u].z, a[u].w};
-                  epi_store_row<4>(p.mix, mm, col, v4, mix_alpha);
+                  epi_store_row<4>(p.mix, mm, col, v4, mix_alpha, mix_palpha);
                 }
               } else if (mm < r1) {
                 if constexpr (EPI == SK_CAP) {

@@ -109,6 +109,7 @@ struct GemmParams {
   int fix_out_f32, fix_accumulate;
   // EPI_SWIGLU: N counts accumulator columns (2 * I); D is the activation [M, I]
   const float* row_scale;  // [M] factor on both halves of a row (a score that scales an expert's input), or null
+  float glu_clip;          // > 0: row_scale g sigmoid(1.702 g) (u + 1) with g <= glu_clip and |u| <= glu_clip
   __nv_bfloat16* gu_out;  // pre-activation [M, 2I] (gate columns first), or null
   long long gu_ld;
   // EPI_MIXER
@@ -474,7 +475,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
     int acc = 0;
     uint32_t acc_phase = 0;
     bool ok = true;
-    float mix_alpha = 0.f;
+    float mix_alpha = 0.f, mix_palpha = 0.f;
     // residual stream of the 32 x 32 block at (row0, col): lanes sweep the columns, four rows per round, so that reads and
     // writes are whole 128-byte lines
     float4 mix_x[8];
@@ -489,6 +490,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
     };
     if constexpr (EPI == EPI_MIXER) {
       mix_alpha = epi_alpha(p.mix);
+      mix_palpha = epi_palpha(p.mix);
       mix_tile = reinterpret_cast<float*>(smem + GemmSmem<BN, STAGES>::RING + 256) + q * 32 * GemmSmem<BN, STAGES>::STAGE_LD;
     }
     for (int t = blockIdx.x; t < num_tiles && ok; t += gridDim.x) {
@@ -594,8 +596,13 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
             float act[16];
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
-              const float g = __uint_as_float(r[2 * j]) * rs, u = __uint_as_float(r[2 * j + 1]) * rs;
-              act[j] = g / (1.f + __expf(-g)) * u;
+              if (p.glu_clip > 0.f) {
+                const float g = fminf(__uint_as_float(r[2 * j]), p.glu_clip), u = fminf(fmaxf(__uint_as_float(r[2 * j + 1]), -p.glu_clip), p.glu_clip);
+                act[j] = g / (1.f + __expf(-1.702f * g)) * (u + 1.f) * rs;
+              } else {
+                const float g = __uint_as_float(r[2 * j]) * rs, u = __uint_as_float(r[2 * j + 1]) * rs;
+                act[j] = g / (1.f + __expf(-g)) * u;
+              }
             }
             __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.D) + static_cast<long long>(row) * p.ldd + ac0;
 #pragma unroll
@@ -636,7 +643,16 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
             if (col0 + 32 < p.N && c + 1 < BN / 32) mix_fetch(m0 + q * 32, col0 + 32);
             const int cc = col0 + (lane & 7) * 4;
             if (cc < p.N) {
-              float w4[4], b4[4];
+              float w4[4], b4[4], pw4[4], pb4[4];
+              const bool post = p.mix.pw != nullptr;
+              if (post) {
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                  const float2 a = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(p.mix.pw)[cc / 2 + i]);
+                  const float2 b = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(p.mix.pb)[cc / 2 + i]);
+                  pw4[2 * i] = a.x; pw4[2 * i + 1] = a.y; pb4[2 * i] = b.x; pb4[2 * i + 1] = b.y;
+                }
+              }
               if (p.mix.D != nullptr) {
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
@@ -650,6 +666,12 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
                 const int rl = u * 4 + (lane >> 3), rr = m0 + q * 32 + rl;
                 if (rr < p.M) {
                   float4 a = *reinterpret_cast<const float4*>(mix_tile + rl * LD + (lane & 7) * 4);
+                  if (post) {
+                    a.x = tanh_full(mix_palpha * a.x) * pw4[0] + pb4[0];
+                    a.y = tanh_full(mix_palpha * a.y) * pw4[1] + pb4[1];
+                    a.z = tanh_full(mix_palpha * a.z) * pw4[2] + pb4[2];
+                    a.w = tanh_full(mix_palpha * a.w) * pw4[3] + pb4[3];
+                  }
                   a.x += xs[u].x; a.y += xs[u].y; a.z += xs[u].z; a.w += xs[u].w;
                   *reinterpret_cast<float4*>(p.mix.X + static_cast<long long>(rr) * p.mix.ldx + cc) = a;
                   if (p.mix.D != nullptr) {
@@ -669,7 +691,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
                 float v[8];
 #pragma unroll
                 for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(r[j + i]);
-                epi_store_row<8>(p.mix, row, col0 + j, v, mix_alpha);
+                epi_store_row<8>(p.mix, row, col0 + j, v, mix_alpha, mix_palpha);
               }
             }
           }
@@ -1189,7 +1211,7 @@ extern "C" int vb_gemm_bf16_swiglu(const void* A, const void* W, void* act, void
 // Gated up-projection of rows grouped by expert (128 rows to a tile, padding rows included): act[rows_cap, I] from the experts'
 // stacked [gate; up] weights W [E, 2I, K]; row_scale [rows_cap] multiplies both halves before the activation.
 extern "C" int vb_gemm_grouped_swiglu(const void* A, const void* W, void* act, int rows_cap, int I, int K, long long lda, long long ldd,
-                                      const float* row_scale, int E, const int* tile_expert, const int* num_tiles, cudaStream_t stream) {
+                                      const float* row_scale, int E, const int* tile_expert, const int* num_tiles, float clip, cudaStream_t stream) {
   if (rows_cap <= 0 || I <= 0 || K <= 0 || E <= 0) return 0;
   if ((I % 4) || (K % 8) || (lda % 8) || (ldd % 4) || (rows_cap % 128)) return -1;
   if (((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) || (reinterpret_cast<uintptr_t>(act) & 7)) return -1;
@@ -1201,7 +1223,7 @@ extern "C" int vb_gemm_grouped_swiglu(const void* A, const void* W, void* act, i
     return -3;
   GemmParams p{};
   p.M = rows_cap; p.N = 2 * I; p.K = K; p.D = act; p.ldd = ldd; p.status = status_ptr(); p.k_splits = 1;
-  p.grp_mode = 1; p.grp_E = E; p.grp_tile_expert = tile_expert; p.grp_num_mtiles = num_tiles; p.grp_b_rows = 2 * I; p.row_scale = row_scale;
+  p.grp_mode = 1; p.grp_E = E; p.grp_tile_expert = tile_expert; p.grp_num_mtiles = num_tiles; p.grp_b_rows = 2 * I; p.row_scale = row_scale; p.glu_clip = clip;
   return static_cast<int>(launch_variant<256, false, false, 4, EPI_SWIGLU>(ta, tb, p, num_sms(), stream));
 }
 

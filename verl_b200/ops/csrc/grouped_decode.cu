@@ -6,7 +6,7 @@
 // heads are the M dimension of m16n8k16 MMAs: like every decode attention the kernel is bound by the stream, not by the
 // tensor pipe. Each of four warps owns 16 of a tile's tokens and keeps its own online softmax; warps and key splits are merged
 // at the end, where the sink (one more score without a value) joins the denominator. Scores may be capped
-// (cap * tanh(score / cap)). Tiles outside the window are never loaded. Compiled without fast math.
+// (cap * tanh(score / cap)). Only the tiles of the window and of the kept first tokens are loaded. Compiled without fast math.
 #include "mixer_epilogue.cuh"
 #include "mixers.h"
 #include "mixer_common.cuh"
@@ -30,7 +30,7 @@ struct GroupedDecodeParams {
   __nv_bfloat16* out;       // [S, H, vdim]
   float* part_o;            // [S, H, nsplit, vdim] when nsplit > 1
   float* part_ml;           // [S, H, nsplit, 2]
-  int H, share, chunks, dim, vdim, window, nsplit;   // chunks: groups of 16 query heads per key head
+  int H, share, chunks, dim, vdim, window, keep, nsplit;   // chunks: groups of 16 query heads per key head
   float scale_log2, cap_z, cap_log2;
   int* status;
 };
@@ -77,8 +77,11 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_con
   const int len = min(p.ctx_len[b], p.max_blocks * p.block_size);
   const int first = (p.window > 0 && len > p.window) ? len - p.window : 0;
   const int tile_a = first / GD_TOK, tile_b = (len + GD_TOK - 1) / GD_TOK;
-  const int per = (max(0, tile_b - tile_a) + p.nsplit - 1) / p.nsplit;
-  const int t0 = tile_a + split * per, n = max(0, min(tile_b, t0 + per) - t0);
+  // the list of tiles: those of the kept tokens that lie in front of the window's, then the window's
+  const int nkeep = min((p.keep + GD_TOK - 1) / GD_TOK, tile_a), listed = nkeep + max(0, tile_b - tile_a);
+  const int per = (listed + p.nsplit - 1) / p.nsplit;
+  const int t0 = split * per, n = max(0, min(listed, t0 + per) - t0);
+  auto tile_at = [&](int i) { return t0 + i < nkeep ? t0 + i : tile_a + t0 + i - nkeep; };
   const int* bt = p.block_table + static_cast<long long>(b) * p.max_blocks;
 
   if (threadIdx.x == 0) {
@@ -99,7 +102,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_con
   __syncthreads();
 
   auto issue = [&](int i) {   // tile t0 + i into stage i % GD_STAGES (thread 0 only)
-    const int s = i % GD_STAGES, tok = (t0 + i) * GD_TOK;
+    const int s = i % GD_STAGES, tok = tile_at(i) * GD_TOK;
     uint8_t* dst = smem + s * L::STAGE;
     mbar_expect_tx(&full[s], L::STAGE);
     for (int r = 0; r < GD_TOK; r += p.box_rows) {
@@ -143,7 +146,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_con
       }
     }
     // rows: heads lane / 4 and + 8; columns: tokens 8 nb + 2 (lane % 4) and + 1
-    const int tok_base = (t0 + i) * GD_TOK + tw + (lane & 3) * 2;
+    const int tok_base = tile_at(i) * GD_TOK + tw + (lane & 3) * 2;
     float alpha[2];
     uint32_t pa[4];
 #pragma unroll
@@ -156,7 +159,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_con
           const int t = tok_base + nb * 8 + e;
           const float x = sc[nb][h * 2 + e];
           const float y = p.cap_log2 > 0.f ? p.cap_log2 * tanh_full(x * p.cap_z) : x * p.scale_log2;
-          v[nb * 2 + e] = (t >= first && t < len) ? y : -INFINITY;
+          v[nb * 2 + e] = ((t >= first || t < p.keep) && t < len) ? y : -INFINITY;
         }
       float mx = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -296,7 +299,7 @@ extern "C" int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, in
   p.q = reinterpret_cast<const __nv_bfloat16*>(a->q); p.ldq = a->ldq; p.hq = a->hq;
   p.block_table = a->block_table; p.max_blocks = a->max_blocks; p.block_size = a->block_size; p.num_blocks = num_blocks; p.ctx_len = a->ctx_len;
   p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink); p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.part_o = part_o; p.part_ml = part_ml;
-  p.H = a->H; p.dim = a->du; p.vdim = a->dv; p.window = a->window; p.nsplit = nsplit; p.status = status;
+  p.H = a->H; p.dim = a->du; p.vdim = a->dv; p.window = a->window; p.keep = a->window > 0 ? a->keep_first : 0; p.nsplit = nsplit; p.status = status;
   p.scale_log2 = a->scale * 1.4426950408889634f;
   if (a->softcap > 0.f) { p.cap_z = a->scale / a->softcap; p.cap_log2 = a->softcap * 1.4426950408889634f; }
   const dim3 grid(a->B, kv_heads * p.chunks, nsplit);

@@ -1,4 +1,4 @@
-// Windowed attention with a sink over latent or expanded keys, one warp per (query, head), on the fp32 pipeline.
+// Windowed attention (kept first keys, a sink) over latent or expanded keys, one warp per (query, head), on the fp32 pipeline.
 //
 // One kernel covers both uses of latent attention: prompts (per-head keys and values expanded from the latents, contiguous
 // rows) and decoding (all heads share the latent row as key and value, rows found through the page table), and grouped-query
@@ -52,12 +52,13 @@ latent_attn_simt_kernel(const VbLatentAttn a) {
   __syncwarp();
   const float sink = a.sink != nullptr ? to_f(reinterpret_cast<const T*>(a.sink)[h]) : -INFINITY;
   float m = sink, l = a.sink != nullptr ? 1.f : 0.f;
-  const int first = a.window > 0 ? max(0, last - a.window + 1) : 0;
-  for (int j0 = first; j0 <= last; j0 += 32) {
-    const int j = j0 + lane;
+  const int first = a.window > 0 ? max(0, last - a.window + 1) : 0, kept = min(a.keep_first, first);
+  // the kept keys [0, kept) in front of the window's [first, last]
+  for (int j0 = kept > 0 ? 0 : first; j0 <= last; j0 = j0 + 32 < kept || j0 >= first ? j0 + 32 : first) {
+    const int j = j0 + lane, end = j0 < first ? kept - 1 : last;
     long long row = 0;
     float s = -INFINITY;
-    if (j <= last) {
+    if (j <= end) {
       if (a.block_table != nullptr)
         row = a.block_table[static_cast<long long>(b) * a.max_blocks + j / a.block_size] * a.page_stride;
       else
@@ -80,11 +81,11 @@ latent_attn_simt_kernel(const VbLatentAttn a) {
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float alpha = expf(m - m_new);
-    const float p = j <= last ? expf(s - m_new) : 0.f;
+    const float p = j <= end ? expf(s - m_new) : 0.f;
     l = l * alpha + warp_sum(p);
     m = m_new;
     for (int c = lane; c < a.dv; c += 32) so[c] *= alpha;
-    const int n = min(32, last - j0 + 1);
+    const int n = min(32, end - j0 + 1);
     for (int jj = 0; jj < n; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const long long rj = __shfl_sync(0xffffffffu, row, jj);

@@ -9,7 +9,7 @@
 //   softmax  running maximum starts at the sink, which adds one unit of weight and no value
 //   values   warp w takes kv_rank / 4 latent columns over all 32 tokens
 // so that one barrier per tile is enough.
-// Tiles outside the window are never loaded. Compiled without fast math.
+// Only the tiles of the window and of the kept first tokens are loaded. Compiled without fast math.
 #include "mixers.h"
 #include "mixer_common.cuh"
 #include "tcgen05_common.cuh"
@@ -32,7 +32,7 @@ struct LatentDecodeParams {
   __nv_bfloat16* out;       // [S, H, rank]
   float* part_o;            // [S, H, nsplit, rank] when nsplit > 1
   float* part_ml;           // [S, H, nsplit, 2]
-  int H, width, rank, panels, window, nsplit, stages;
+  int H, width, rank, panels, window, keep, nsplit, stages;
   float scale_log2;
   int* status;
 };
@@ -74,8 +74,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
   const int nheads = max(0, min(LD_HEADS, p.H - h0));
   const int first = (p.window > 0 && len > p.window) ? len - p.window : 0;
   const int tile_a = first / LD_TOK, tile_b = (len + LD_TOK - 1) / LD_TOK;
-  const int per = (max(0, tile_b - tile_a) + p.nsplit - 1) / p.nsplit;
-  const int t0 = tile_a + split * per, n = max(0, min(tile_b, t0 + per) - t0);
+  // the list of tiles: those of the kept tokens that lie in front of the window's, then the window's
+  const int nkeep = min((p.keep + LD_TOK - 1) / LD_TOK, tile_a), listed = nkeep + max(0, tile_b - tile_a);
+  const int per = (listed + p.nsplit - 1) / p.nsplit;
+  const int t0 = split * per, n = max(0, min(listed, t0 + per) - t0);
+  auto tile_at = [&](int i) { return t0 + i < nkeep ? t0 + i : tile_a + t0 + i - nkeep; };
   const int* bt = p.block_table + static_cast<long long>(b) * p.max_blocks;
 
   if (threadIdx.x == 0) {
@@ -97,7 +100,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
   if (producer) {
     if (lane == 0) {
       for (int i = 0; i < n; ++i) {
-        const int s = i % p.stages, tok = (t0 + i) * LD_TOK;
+        const int s = i % p.stages, tok = tile_at(i) * LD_TOK;
         if (i >= p.stages && !mbar_wait(&empty[s], ((i / p.stages) & 1) ^ 1)) {
           atomicExch(p.status, 2);
           break;
@@ -173,7 +176,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
     sync_group();
     // ---- weights: rows lane / 4 and + 8, columns 8 nb + 2 (lane % 4) and + 1
     const float* all = sS + (i & 1) * 4 * (LD_HEADS * LD_SP) + (lane >> 2) * LD_SP + (lane & 3) * 2;
-    const int tok0 = (t0 + i) * LD_TOK + (lane & 3) * 2;
+    const int tok0 = tile_at(i) * LD_TOK + (lane & 3) * 2;
     float alpha[2];
     uint32_t pa[2][4];
 #pragma unroll
@@ -189,8 +192,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm, const LatentDecodeP
           x.y += y.y;
         }
         const int t = tok0 + nb * 8;
-        v[nb][0] = (t >= first && t < len) ? x.x * p.scale_log2 : -INFINITY;
-        v[nb][1] = (t + 1 >= first && t + 1 < len) ? x.y * p.scale_log2 : -INFINITY;
+        v[nb][0] = ((t >= first || t < p.keep) && t < len) ? x.x * p.scale_log2 : -INFINITY;
+        v[nb][1] = ((t + 1 >= first || t + 1 < p.keep) && t + 1 < len) ? x.y * p.scale_log2 : -INFINITY;
         mx = fmaxf(mx, fmaxf(v[nb][0], v[nb][1]));
       }
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -321,7 +324,7 @@ extern "C" int vb_latent_decode(const VbLatentAttn* a, long long num_blocks, int
   p.block_table = a->block_table; p.max_blocks = a->max_blocks; p.block_size = a->block_size; p.num_blocks = num_blocks;
   p.ctx_len = a->ctx_len; p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink);
   p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.part_o = part_o; p.part_ml = part_ml;
-  p.H = a->H; p.width = width; p.rank = a->dv; p.panels = panels; p.window = a->window; p.nsplit = nsplit;
+  p.H = a->H; p.width = width; p.rank = a->dv; p.panels = panels; p.window = a->window; p.keep = a->window > 0 ? a->keep_first : 0; p.nsplit = nsplit;
   const int ng = latent_decode_groups(a->H);
   p.stages = latent_decode_stages(panels, ng); p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;
   const int smem = latent_decode_fixed(panels, ng) + p.stages * panels * LD_TOK * 128;

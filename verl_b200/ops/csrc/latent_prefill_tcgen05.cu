@@ -1,4 +1,5 @@
-// Prompt attention of the mixer stacks on tcgen05 tensor cores: causal, windowed, with a sink, capped scores and an output gate.
+// Prompt attention of the mixer stacks on tcgen05 tensor cores: causal, windowed (with kept first keys), with a sink, capped scores
+// and an output gate.
 // Latent attention, or grouped-query attention with query / key and value sizes of its own (no rotated part, kv_group query
 // heads per key head).
 //
@@ -26,7 +27,7 @@ constexpr int LP_BQ = 128, LP_BK = 64;
 struct LatentPrefillParams {
   const int* cu_q;
   const int* cu_k;
-  int num_seqs, dv, window, kv_group, pu, pr, pv, su, sr;  // panels of 64 columns (unrotated, rotated, value), k steps of 16
+  int num_seqs, dv, window, keep, kv_group, pu, pr, pv, su, sr;  // panels of 64 columns (unrotated, rotated, value), k steps of 16
   const __nv_bfloat16* sink;
   const float* gate;
   long long ldg;
@@ -125,18 +126,23 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
   const int seq_q = s_tile[0], q0 = s_tile[1], nq = s_tile[2], seq_k = s_tile[3], nk = s_tile[4];
   const bool valid = s_tile[5] != 0;
   const int off = nk - nq;  // position of query row 0 among the sequence's keys
-  // key blocks: block j holds keys [(jb0 + j) * 64, + 64); tile t uses j in [ja[t], jz[t])
-  int jb0 = 0, ja[NT], jz[NT], nblk = 0;
+  // key blocks: entry j of the list holds keys [block_at(j) * 64, + 64); tile t uses j in [ja[t], jz[t]). Blocks of kept keys in front
+  // of the window's come first; every tile walks the list from its start then.
+  int jb0 = 0, nkeep = 0, ja[NT], jz[NT], nblk = 0;
 #pragma unroll
   for (int t = 0; t < NT; ++t) {
     const int r0 = q0 + t * LP_BQ;
     const int lo = p.window > 0 ? max(0, r0 + off - p.window + 1) : 0;
-    if (t == 0) jb0 = lo / LP_BK;
+    if (t == 0) {
+      jb0 = lo / LP_BK;
+      nkeep = min((p.keep + LP_BK - 1) / LP_BK, jb0);
+    }
     const bool act = valid && r0 < nq;
-    ja[t] = act ? lo / LP_BK - jb0 : 0;
-    jz[t] = act ? min(min(r0 + LP_BQ, nq) - 1 + off, nk - 1) / LP_BK - jb0 + 1 : 0;
+    ja[t] = act && p.keep == 0 ? lo / LP_BK - jb0 : 0;
+    jz[t] = act ? min(min(r0 + LP_BQ, nq) - 1 + off, nk - 1) / LP_BK - jb0 + 1 + nkeep : 0;
     nblk = max(nblk, jz[t]);
   }
+  auto block_at = [&](int j) { return j < nkeep ? j : jb0 + j - nkeep; };
   const uint32_t tm_o = NT * 2 * LP_BK;
 
   if (warp == 0) {
@@ -148,7 +154,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         for (int c = 0; c < p.pr; ++c) tma_load_3d(sQ + t * q_bytes + (p.pu + c) * (LP_BQ * 128), &tm_qr, q_full, 64 * c, head, row);
       }
       for (int j = 0; j < nblk; ++j) {
-        const int st = j & 1, row = seq_k + (jb0 + j) * LP_BK;
+        const int st = j & 1, row = seq_k + block_at(j) * LP_BK;
         const uint32_t ph = ((j >> 1) & 1) ^ 1;
         if (!mbar_wait(&k_empty[st], ph)) { atomicExch(p.status, ST_TIMEOUT_PRODUCER); break; }
         mbar_expect_tx(&k_full[st], static_cast<uint32_t>(k_bytes));
@@ -233,10 +239,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         tmem_ld_32x32(tmem_base + (t * 2 + (jj & 1)) * LP_BK + lane_off, x0);
         tmem_ld_32x32(tmem_base + (t * 2 + (jj & 1)) * LP_BK + 32 + lane_off, x1);
         tmem_ld_wait();
-        const int col0 = (jb0 + a + jj) * LP_BK;
+        const int col0 = block_at(a + jj) * LP_BK;
         const bool need_mask = col0 + LP_BK - 1 > tile_lo || (p.window > 0 && tile_hi - col0 >= p.window);
-        // visible: first_c <= c <= last_c
-        const int last_c = pos - col0, first_c = p.window > 0 ? pos - p.window + 1 - col0 : -1;
+        // visible: first_c <= c <= last_c, or c < keep_c and c <= last_c
+        const int last_c = pos - col0, first_c = p.window > 0 ? pos - p.window + 1 - col0 : -1, keep_c = p.keep - col0;
         float mx = -INFINITY;
         if constexpr (CAP) {
           float most = 0.f;
@@ -269,8 +275,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         if (need_mask) {
 #pragma unroll
           for (int c = 0; c < 32; ++c) {
-            if (c > last_c || c < first_c) x0[c] = 0xff800000u;
-            if (c + 32 > last_c || c + 32 < first_c) x1[c] = 0xff800000u;
+            if (c > last_c || (c < first_c && c >= keep_c)) x0[c] = 0xff800000u;
+            if (c + 32 > last_c || (c + 32 < first_c && c + 32 >= keep_c)) x1[c] = 0xff800000u;
           }
         }
 #pragma unroll
@@ -405,7 +411,7 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
   static int* status = nullptr;
   if (status == nullptr) cudaGetSymbolAddress(reinterpret_cast<void**>(&status), g_latent_prefill_status);
   LatentPrefillParams p{};
-  p.cu_q = a->cu_q; p.cu_k = a->cu_k; p.num_seqs = a->B; p.dv = a->dv; p.window = a->window; p.kv_group = kv_group; p.pu = pu; p.pr = pr; p.pv = pv;
+  p.cu_q = a->cu_q; p.cu_k = a->cu_k; p.num_seqs = a->B; p.dv = a->dv; p.window = a->window; p.keep = a->window > 0 ? a->keep_first : 0; p.kv_group = kv_group; p.pu = pu; p.pr = pr; p.pv = pv;
   p.su = (a->du + 15) / 16; p.sr = (a->dr + 15) / 16;
   p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink); p.gate = a->gate; p.ldg = a->ldg;
   p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo; p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;

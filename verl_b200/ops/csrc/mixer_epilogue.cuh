@@ -17,21 +17,31 @@ __device__ __forceinline__ float tanh_full(float x) {
 }
 __device__ __forceinline__ float gelu_erf_full(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
-struct EpiColumn { float w, b; };  // norm weight and bias of an output column
+__device__ __forceinline__ float silu_full(float z) { return z / (1.f + __expf(-z)); }
+
+struct EpiColumn { float w, b, pw, pb; };  // weight and bias of an output column: of the norm of the stream, of the norm of the product
 __device__ __forceinline__ EpiColumn epi_column(const VbEpiArgs& e, int col) {
-  EpiColumn c{0.f, 0.f};
+  EpiColumn c{0.f, 0.f, 0.f, 0.f};
   if (e.mode == VB_EPI_RESID && e.D != nullptr) {
     c.w = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.nw)[col]);
     c.b = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.nb)[col]);
   }
+  if (e.mode == VB_EPI_RESID && e.pw != nullptr) {
+    c.pw = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.pw)[col]);
+    c.pb = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.pb)[col]);
+  }
+  if (e.mode == VB_EPI_BIAS) c.b = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.nb)[col]);
   return c;
+}
+__device__ __forceinline__ float epi_palpha(const VbEpiArgs& e) {
+  return (e.mode == VB_EPI_RESID && e.pw != nullptr) ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(e.palpha)) : 0.f;
 }
 __device__ __forceinline__ float epi_alpha(const VbEpiArgs& e) {
   return (e.mode == VB_EPI_RESID && e.D != nullptr) ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(e.alpha)) : 0.f;
 }
 
 // One element.
-__device__ __forceinline__ void epi_store1(const VbEpiArgs& e, long long row, int col, float v, float alpha, const EpiColumn& c) {
+__device__ __forceinline__ void epi_store1(const VbEpiArgs& e, long long row, int col, float v, float alpha, float palpha, const EpiColumn& c) {
   __nv_bfloat16* D = reinterpret_cast<__nv_bfloat16*>(e.D);
   if (e.mode == VB_EPI_GELU) {
     D[row * e.ldd + col] = __float2bfloat16(gelu_erf_full(v));
@@ -43,9 +53,13 @@ __device__ __forceinline__ void epi_store1(const VbEpiArgs& e, long long row, in
     if (col < e.n0) D[row * e.ldd + col] = __float2bfloat16(v);
     else e.D2[row * e.ldd2 + col - e.n0] = v;
   } else if (e.mode == VB_EPI_RESID) {
-    const float x = e.X[row * e.ldx + col] + v;
+    const float x = e.X[row * e.ldx + col] + (e.pw != nullptr ? tanh_full(palpha * v) * c.pw + c.pb : v);
     e.X[row * e.ldx + col] = x;
     if (D != nullptr) D[row * e.ldd + col] = __float2bfloat16(tanh_full(alpha * x) * c.w + c.b);
+  } else if (e.mode == VB_EPI_BIAS) {
+    D[row * e.ldd + col] = __float2bfloat16(v + c.b);
+  } else if (e.mode == VB_EPI_SILU) {
+    D[row * e.ldd + col] = __float2bfloat16(col < e.n0 ? silu_full(v) : v);
   } else {
     D[row * e.ldd + col] = __float2bfloat16(v);
   }
@@ -53,7 +67,7 @@ __device__ __forceinline__ void epi_store1(const VbEpiArgs& e, long long row, in
 
 // NV consecutive columns of one row (NV = 4 or 8, col a multiple of NV, split point a multiple of NV).
 template <int NV>
-__device__ __forceinline__ void epi_store_row(const VbEpiArgs& e, long long row, int col, const float (&v)[NV], float alpha) {
+__device__ __forceinline__ void epi_store_row(const VbEpiArgs& e, long long row, int col, const float (&v)[NV], float alpha, float palpha) {
   __nv_bfloat16* D = reinterpret_cast<__nv_bfloat16*>(e.D);
   auto put16 = [&](const float (&o)[NV]) {
     __nv_bfloat16* dst = D + row * e.ldd + col;
@@ -85,9 +99,17 @@ __device__ __forceinline__ void epi_store_row(const VbEpiArgs& e, long long row,
     float* xp = e.X + row * e.ldx + col;
     float o[NV];
 #pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] = v[i];
+    if (e.pw != nullptr) {
+      const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(e.pw) + col;
+      const __nv_bfloat16* b = reinterpret_cast<const __nv_bfloat16*>(e.pb) + col;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) o[i] = tanh_full(palpha * v[i]) * __bfloat162float(w[i]) + __bfloat162float(b[i]);
+    }
+#pragma unroll
     for (int i = 0; i < NV; i += 4) {
       const float4 a = *reinterpret_cast<const float4*>(xp + i);
-      o[i] = v[i] + a.x; o[i + 1] = v[i + 1] + a.y; o[i + 2] = v[i + 2] + a.z; o[i + 3] = v[i + 3] + a.w;
+      o[i] += a.x; o[i + 1] += a.y; o[i + 2] += a.z; o[i + 3] += a.w;
     }
     put32(xp, o);
     if (D != nullptr) {
@@ -97,6 +119,17 @@ __device__ __forceinline__ void epi_store_row(const VbEpiArgs& e, long long row,
       for (int i = 0; i < NV; ++i) o[i] = tanh_full(alpha * o[i]) * __bfloat162float(w[i]) + __bfloat162float(b[i]);
       put16(o);
     }
+  } else if (e.mode == VB_EPI_BIAS) {
+    const __nv_bfloat16* b = reinterpret_cast<const __nv_bfloat16*>(e.nb) + col;
+    float o[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] = v[i] + __bfloat162float(b[i]);
+    put16(o);
+  } else if (e.mode == VB_EPI_SILU) {
+    float o[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] = col + i < e.n0 ? silu_full(v[i]) : v[i];
+    put16(o);
   } else {
     put16(v);
   }
@@ -108,7 +141,7 @@ inline bool epi_aligned(const VbEpiArgs& e, int nv) {
   const bool f32 = e.mode == VB_EPI_STORE_F32;
   if (e.D != nullptr && ((e.ldd % (f32 ? 4 : nv)) || bad(e.D, f32 ? 16 : 2 * nv))) return false;
   if (e.mode == VB_EPI_SPLIT && ((e.n0 % 8) || (e.ldd2 % 4) || bad(e.D2, 16))) return false;
-  if (e.mode == VB_EPI_RESID && ((e.ldx % 4) || bad(e.X, 16) || (e.D != nullptr && (bad(e.nw, 4) || bad(e.nb, 4))))) return false;
+  if (e.mode == VB_EPI_RESID && ((e.ldx % 4) || bad(e.X, 16) || bad(e.pw, 4) || bad(e.pb, 4) || (e.D != nullptr && (bad(e.nw, 4) || bad(e.nb, 4))))) return false;
   return true;
 }
 

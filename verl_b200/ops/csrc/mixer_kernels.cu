@@ -15,7 +15,7 @@ typedef __nv_bfloat16 bf16;
 template <typename T, int VEC>
 __global__ void embed_dyt_kernel(const long long* __restrict__ ids, const T* __restrict__ w, float scale, float* __restrict__ x,
                                  T* __restrict__ h, const T* __restrict__ alpha, const T* __restrict__ nw, const T* __restrict__ nb,
-                                 int W, int V) {
+                                 const T* __restrict__ ealpha, const T* __restrict__ ew, const T* __restrict__ eb, int W, int V) {
   const long long t = blockIdx.x;
   const long long id = ids == nullptr ? 0 : ids[t];
   const bool ok = ids == nullptr || (id >= 0 && id < V);
@@ -28,6 +28,13 @@ __global__ void embed_dyt_kernel(const long long* __restrict__ ids, const T* __r
       if (ok) Vec<T, VEC>::load(w + id * W + c, v);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) v[i] = ok ? v[i] * scale : 0.f;
+      if (ew != nullptr) {               // the embedding passes a norm of its own
+        const float ea = to_f(*ealpha);
+        Vec<T, VEC>::load(ew + c, g);
+        Vec<T, VEC>::load(eb + c, b);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = tanhf(ea * v[i]) * g[i] + b[i];
+      }
       Vec<float, VEC>::store(x + t * W + c, v);
     }
     if (h != nullptr) {
@@ -42,12 +49,14 @@ __global__ void embed_dyt_kernel(const long long* __restrict__ ids, const T* __r
 
 template <typename T>
 static int embed_dyt(const long long* ids, const void* w, float scale, float* x, void* h, const void* alpha, const void* nw, const void* nb,
-                     int T_, int W, int V, cudaStream_t s) {
+                     const void* ea, const void* ew, const void* eb, int T_, int W, int V, cudaStream_t s) {
   const int thr = W >= 1024 ? 256 : 128;
   if (W % 8 == 0)
-    embed_dyt_kernel<T, 8><<<T_, thr, 0, s>>>(ids, (const T*)w, scale, x, (T*)h, (const T*)alpha, (const T*)nw, (const T*)nb, W, V);
+    embed_dyt_kernel<T, 8><<<T_, thr, 0, s>>>(ids, (const T*)w, scale, x, (T*)h, (const T*)alpha, (const T*)nw, (const T*)nb, (const T*)ea, (const T*)ew,
+                                               (const T*)eb, W, V);
   else
-    embed_dyt_kernel<T, 1><<<T_, thr, 0, s>>>(ids, (const T*)w, scale, x, (T*)h, (const T*)alpha, (const T*)nw, (const T*)nb, W, V);
+    embed_dyt_kernel<T, 1><<<T_, thr, 0, s>>>(ids, (const T*)w, scale, x, (T*)h, (const T*)alpha, (const T*)nw, (const T*)nb, (const T*)ea, (const T*)ew,
+                                               (const T*)eb, W, V);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -440,7 +449,14 @@ using namespace vb;
 extern "C" int vb_embed_dyt(int dtype, const long long* ids, const void* w, float scale, float* x, void* h, const void* alpha, const void* nw,
                             const void* nb, int T, int W, int V, cudaStream_t s) {
   if (T <= 0) return 0;
-  return dtype == 0 ? embed_dyt<float>(ids, w, scale, x, h, alpha, nw, nb, T, W, V, s) : embed_dyt<bf16>(ids, w, scale, x, h, alpha, nw, nb, T, W, V, s);
+  return dtype == 0 ? embed_dyt<float>(ids, w, scale, x, h, alpha, nw, nb, nullptr, nullptr, nullptr, T, W, V, s)
+                    : embed_dyt<bf16>(ids, w, scale, x, h, alpha, nw, nb, nullptr, nullptr, nullptr, T, W, V, s);
+}
+extern "C" int vb_embed_dyt2(int dtype, const long long* ids, const void* w, float* x, void* h, const void* ealpha, const void* ew, const void* eb,
+                             const void* alpha, const void* nw, const void* nb, int T, int W, int V, cudaStream_t s) {
+  if (T <= 0) return 0;
+  return dtype == 0 ? embed_dyt<float>(ids, w, 1.f, x, h, alpha, nw, nb, ealpha, ew, eb, T, W, V, s)
+                    : embed_dyt<bf16>(ids, w, 1.f, x, h, alpha, nw, nb, ealpha, ew, eb, T, W, V, s);
 }
 extern "C" int vb_dyt(int dtype, const float* x, void* h, const void* alpha, const void* nw, const void* nb, int T, int W, cudaStream_t s) {
   return vb_embed_dyt(dtype, nullptr, nullptr, 1.f, const_cast<float*>(x), h, alpha, nw, nb, T, W, 0, s);

@@ -1,4 +1,5 @@
-// C launchers of the mixer-stack kernels (latent and grouped-query attention, mLSTM, norms, experts, GEMMs with their epilogues).
+// C launchers of the mixer-stack kernels (latent and grouped-query attention, mLSTM and lightning recurrences, short convolutions,
+// norms, experts, GEMMs with their epilogues).
 // dtype: 0 = fp32 tensors, 1 = bf16 tensors (weights and activations; statistics, states and residual are always fp32).
 #pragma once
 #include <cuda_runtime.h>
@@ -10,8 +11,11 @@ enum VbEpi : int {
   VB_EPI_STORE_F32 = 1, // D = acc as fp32
   VB_EPI_GELU = 2,      // D = erf-gelu(acc) in the operands' type
   VB_EPI_SPLIT = 3,     // columns [0, n0) -> D in the operands' type, columns [n0, N) -> D2 as fp32
-  VB_EPI_RESID = 4,     // X += acc (fp32 residual stream); D = tanh(alpha X) w + b in the operands' type when D is given
+  VB_EPI_RESID = 4,     // X += acc, or tanh(palpha acc) pw + pb when pw is given (fp32 residual stream); D = tanh(alpha X) nw + nb in the
+                        // operands' type when D is given
   VB_EPI_SOFTCAP = 5,   // D = cap * tanh(acc / cap) in the operands' type
+  VB_EPI_BIAS = 6,      // D = acc + nb in the operands' type
+  VB_EPI_SILU = 7,      // D = silu(acc) in columns [0, n0), acc in the others, in the operands' type
 };
 
 struct VbEpiArgs {
@@ -29,6 +33,9 @@ struct VbEpiArgs {
   float cap;
   const float* gate;  // batched products: batch z of row m is multiplied by sigmoid(gate[m * ldg + z]) when given
   long long ldg;
+  const void* palpha; // VB_EPI_RESID: norm of the product (scalar, [N], [N]), or null
+  const void* pw;
+  const void* pb;
 };
 
 // Attention with per-head or shared keys and values. Latent attention: du unrotated and dr rotated key dimensions (the latter
@@ -52,6 +59,7 @@ struct VbLatentAttn {
   float scale;
   int kv_group;             // query heads per key / value head (0 or 1: one)
   float softcap;            // score = softcap * tanh(score / softcap); 0: off
+  int keep_first;           // with a window: the sequence's first keys that every query sees besides
 };
 
 // x += mult * rms_norm(Y) * nw;  Y = [sigmoid(gate)] sum of `splits` planes of y + sum_j rows[slot[t, j]]
@@ -87,6 +95,43 @@ struct VbQkvPrep {
   float eps;
 };
 
+// x += post(sum_j rows[slot[t, j]]), h = next(x); both norms Dynamic Tanh
+struct VbResidDyt {
+  float* x;                 // [T, W]
+  const void* rows; long long ldr;
+  const int* slot; int top; // [T, top]
+  const void *palpha, *pw, *pb, *alpha, *nw, *nb;
+  void* h;                  // [T, W]
+  int T, W;
+};
+
+// Row p[t] = [q of H heads | k of G heads | v of G heads]: causal convolution per channel, rotation of q and k, norm without weight.
+struct VbConvPrep {
+  const void* p; long long ldp;
+  const void* conv; int taps;         // [channels, taps], last tap = the token itself (null: no convolution, taps = 1)
+  const int* cu; int B;               // portions: sequence b = tokens cu[b] .. cu[b + 1]; null: one token per sequence
+  float* state; long long slot_stride;// last taps - 1 inputs per slot, [taps - 1, channels], oldest first (null: zeros, nothing kept)
+  const int *slots, *fresh;           // portions
+  const uint8_t* active;              // steps: row t is slot t
+  const int* pos; const float *cos_t, *sin_t; int half, max_pos, halves;
+  void* q;                            // [T, H, dim]
+  void* rows; long long ldr;          // [T, G (dim + vdim)] or null
+  void* pages; long long page_stride; int block_size; long long num_slots; const long long* page_slot;
+  int T, H, G, dim, vdim;
+  float eps;
+};
+
+// Recurrence S = decay S + k v^T, o = S^T q per head over rows p[t] = [q | k | v | ...].
+struct VbLightning {
+  const void* p; long long ldp;
+  const float* decay;                 // [H]
+  float* state; long long slot_stride;// [slots, H, d, e] or null
+  const int *slots, *fresh, *cu;      // portions
+  const uint8_t* active;              // steps: row t is slot t
+  void* out; long long ldo;           // [T, H e]
+  int T, B, H, d, e;
+};
+
 struct VbHeadwise {
   const void* a; long long lda, a_head;   // a[m, h, k]
   const void* w; long long w_head, ldw;   // w[h] as [N, K] (kn = 0) or [K, N] (kn = 1)
@@ -112,17 +157,28 @@ int vb_gemm_simt_grouped(int dtype, const void* A, const void* B, int M, int N, 
 int vb_gemm_bf16_epi(const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, const VbEpiArgs* e, cudaStream_t s);
 int vb_gemm_skinny_epi(const void* X, const void* W, int M, int N, int K, long long ldx, long long ldw, const VbEpiArgs* e, int splits,
                        float* ws, cudaStream_t s);
-// act[rows, I] = silu(r g) * (r u), [g | u] = A W_e^T with W_e = [gate; up] ([2I, K]) of the tile's expert and r = row_scale[row]
+// act[rows, I] = silu(r g) * (r u), [g | u] = A W_e^T with W_e = [gate; up] ([2I, K]) of the tile's expert and r = row_scale[row];
+// clip > 0: r g sigmoid(1.702 g) (u + 1) with g <= clip and |u| <= clip
 int vb_gemm_grouped_swiglu(const void* A, const void* W, void* act, int rows_cap, int I, int K, long long lda, long long ldd, const float* row_scale,
-                           int E, const int* tile_expert, const int* num_tiles, cudaStream_t s);
+                           int E, const int* tile_expert, const int* num_tiles, float clip, cudaStream_t s);
 // stack_rows.cu
 int vb_embed_rms(int dtype, const long long* ids, const void* w, float scale, const void* nw, float eps, float* x, void* h, int T, int W, int V,
                  cudaStream_t s);
 int vb_residual_rms(int dtype, const VbResidRms* p, cudaStream_t s);
-int vb_gated_silu(int dtype, const void* gu, long long ldg, const float* row_scale, void* out, int T, int I, cudaStream_t s);
+int vb_gated_silu(int dtype, const void* gu, long long ldg, const float* row_scale, float clip, void* out, int T, int I, cudaStream_t s);
+int vb_residual_dyt(int dtype, const VbResidDyt* p, cudaStream_t s);
+int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W, cudaStream_t s);
+// conv_prep.cu
+int vb_conv_prep(int dtype, const VbConvPrep* p, cudaStream_t s);
+// lightning.cu / lightning_chunk.cu
+int vb_lightning_decode(int dtype, const VbLightning* p, cudaStream_t s);
+int vb_lightning_scan(int dtype, const VbLightning* p, cudaStream_t s);
+int vb_lightning_chunk_segments(int T, int B, int H, int d, int e, int all_fresh);
+int vb_lightning_chunk(const VbLightning* p, int nseg, float* local, cudaStream_t s);
 int vb_qkv_prep(int dtype, const VbQkvPrep* p, cudaStream_t s);
 // experts.cu
-int vb_expert_route(const float* z, long long ldz, int T, int E, int k, int renorm, float* score, int* expert, int* rank, int* counts, cudaStream_t s);
+// corr (null: none) is added to the scores for the choice; groups > 1: only experts of the `keep` best groups can be chosen
+int vb_expert_route(int dtype, const float* z, long long ldz, const void* corr, int groups, int keep, int T, int E, int k, int renorm, float* score, int* expert, int* rank, int* counts, cudaStream_t s);
 int vb_expert_place(int dtype, const void* h, long long ldh, const float* score, const int* expert, const int* rank, const int* counts, int T, int E, int k,
                     int W, void* x, float* row_scale, int* slot, int* tile_expert, int* num_tiles, int max_tiles, cudaStream_t s);
 // grouped_decode.cu
@@ -131,6 +187,9 @@ int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, int nsplit, f
 // mixer_kernels.cu
 int vb_embed_dyt(int dtype, const long long* ids, const void* w, float scale, float* x, void* h, const void* alpha, const void* nw,
                  const void* nb, int T, int W, int V, cudaStream_t s);
+// x = tanh(ealpha w[id]) ew + eb, h = tanh(alpha x) nw + nb
+int vb_embed_dyt2(int dtype, const long long* ids, const void* w, float* x, void* h, const void* ealpha, const void* ew, const void* eb, const void* alpha,
+                  const void* nw, const void* nb, int T, int W, int V, cudaStream_t s);
 int vb_dyt(int dtype, const float* x, void* h, const void* alpha, const void* nw, const void* nb, int T, int W, cudaStream_t s);
 int vb_rope_pairs(int dtype, void* x, const int* pos, const float* cos_t, const float* sin_t, int T, int heads, long long ld, int hstride,
                   int off, int dims, int max_pos, cudaStream_t s);

@@ -1,6 +1,7 @@
-// Row kernels of stacks whose RMS norms sit on the sublayers' outputs: normed embedding, residual add of a normed sublayer
-// output (which also adds up split-K partial products and the rows of chosen experts), gated activation, and the preparation
-// of grouped-query attention (norm and rotation of query and key heads, value mixing, append to the paged cache).
+// Row kernels of stacks with norms on the sublayers' outputs: normed embedding, residual add of a normed sublayer output (which
+// also adds up split-K partial products and the rows of chosen experts; RMS or Dynamic Tanh), gated activations, gated RMS norm
+// of a row, and the preparation of grouped-query attention (norm and rotation of query and key heads, value mixing, append to
+// the paged cache).
 // Statistics, angles and the residual stream are fp32; compiled without fast math.
 #include "mixers.h"
 #include "mixer_common.cuh"
@@ -130,9 +131,94 @@ static int residual_rms(const VbResidRms* p, cudaStream_t s) {
   return -1;
 }
 
-// --------------------------------------------------------------------------------------------- silu(r g) * (r u)
+// --------------------------------------------------------------------------------------------- residual + Dynamic Tanh of experts' rows
+// Elementwise: a thread owns VEC columns of one token, requests all its rows before it uses the first.
 template <typename T, int VEC>
-__global__ void gated_silu_kernel(const T* __restrict__ gu, long long ldg, const float* __restrict__ row_scale, T* __restrict__ out, int I, long long total) {
+__global__ void __launch_bounds__(256) residual_dyt_kernel(const VbResidDyt p, long long total) {
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= total) return;
+  const int per = p.W / VEC, c = static_cast<int>(i % per) * VEC;
+  const long long t = i / per;
+  const T* rows = reinterpret_cast<const T*>(p.rows);
+  const int* slot = p.slot + t * p.top;
+  float x[VEC], y[VEC], v[4][VEC], w[VEC], b[VEC];
+  Vec<float, VEC>::load(p.x + t * p.W + c, x);
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) y[k] = 0.f;
+  for (int j = 0; j < p.top; j += 4) {
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+      if (j + u < p.top) Vec<T, VEC>::load(rows + static_cast<long long>(slot[j + u]) * p.ldr + c, v[u]);
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+      if (j + u < p.top) {
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) y[k] += v[u][k];
+      }
+  }
+  const float pa = to_f(*reinterpret_cast<const T*>(p.palpha)), na = to_f(*reinterpret_cast<const T*>(p.alpha));
+  Vec<T, VEC>::load(reinterpret_cast<const T*>(p.pw) + c, w);
+  Vec<T, VEC>::load(reinterpret_cast<const T*>(p.pb) + c, b);
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) x[k] += tanhf(pa * y[k]) * w[k] + b[k];
+  Vec<float, VEC>::store(p.x + t * p.W + c, x);
+  Vec<T, VEC>::load(reinterpret_cast<const T*>(p.nw) + c, w);
+  Vec<T, VEC>::load(reinterpret_cast<const T*>(p.nb) + c, b);
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) x[k] = tanhf(na * x[k]) * w[k] + b[k];
+  Vec<T, VEC>::store(reinterpret_cast<T*>(p.h) + t * p.W + c, x);
+}
+
+// --------------------------------------------------------------------------------------------- rms_norm(o) * w * sigmoid(g) over whole rows
+template <typename T, int VEC, int ITEMS>
+__global__ void gated_rms_kernel(const T* __restrict__ o, long long ldo, const T* __restrict__ g, long long ldg, const T* __restrict__ norm, float eps,
+                                 T* __restrict__ out, int W) {
+  __shared__ float red[33];
+  const long long t = blockIdx.x;
+  float v[ITEMS][VEC], z[ITEMS][VEC], w[VEC], ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int c = (it * blockDim.x + threadIdx.x) * VEC;
+    if (c >= W) continue;
+    Vec<T, VEC>::load(o + t * ldo + c, v[it]);
+    Vec<T, VEC>::load(g + t * ldg + c, z[it]);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) ss += v[it][k] * v[it][k];
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, red) / W + eps);
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int c = (it * blockDim.x + threadIdx.x) * VEC;
+    if (c >= W) continue;
+    Vec<T, VEC>::load(norm + c, w);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[it][k] = v[it][k] * r * w[k] * sigmoid_f(z[it][k]);
+    Vec<T, VEC>::store(out + t * W + c, v[it]);
+  }
+}
+
+template <typename T, int VEC>
+static int gated_rms(const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T_, int W, cudaStream_t s) {
+  const int nvec = (W + VEC - 1) / VEC;
+  int thr = nvec >= 256 ? 256 : (nvec + 31) / 32 * 32;
+  if (nvec > 8 * thr) thr = 1024;
+  const int items = (nvec + thr - 1) / thr;
+  auto go = [&](auto kern) {
+    kern<<<T_, thr, 0, s>>>((const T*)o, ldo, (const T*)g, ldg, (const T*)norm, eps, (T*)out, W);
+    return static_cast<int>(cudaGetLastError());
+  };
+  if (items == 1) return go(gated_rms_kernel<T, VEC, 1>);
+  if (items == 2) return go(gated_rms_kernel<T, VEC, 2>);
+  if (items <= 4) return go(gated_rms_kernel<T, VEC, 4>);
+  if (items <= 8) return go(gated_rms_kernel<T, VEC, 8>);
+  if (VEC == 1 && items <= 32) return go(gated_rms_kernel<T, VEC, 32>);
+  return -1;
+}
+
+// --------------------------------------------------------------------------------------------- silu(r g) * (r u), or the clipped form
+template <typename T, int VEC>
+__global__ void gated_silu_kernel(const T* __restrict__ gu, long long ldg, const float* __restrict__ row_scale, float clip, T* __restrict__ out, int I,
+                                  long long total) {
   const long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x;
   if (i >= total) return;
   const int per = I / VEC, c = static_cast<int>(i % per) * VEC;
@@ -143,8 +229,13 @@ __global__ void gated_silu_kernel(const T* __restrict__ gu, long long ldg, const
   Vec<T, VEC>::load(gu + t * ldg + I + c, u);
 #pragma unroll
   for (int k = 0; k < VEC; ++k) {
-    const float z = g[k] * r;
-    g[k] = z * sigmoid_f(z) * (u[k] * r);
+    if (clip > 0.f) {
+      const float z = fminf(g[k], clip);
+      g[k] = z * sigmoid_f(1.702f * z) * (fminf(fmaxf(u[k], -clip), clip) + 1.f) * r;
+    } else {
+      const float z = g[k] * r;
+      g[k] = z * sigmoid_f(z) * (u[k] * r);
+    }
   }
   Vec<T, VEC>::store(out + t * I + c, g);
 }
@@ -261,19 +352,43 @@ extern "C" int vb_residual_rms(int dtype, const VbResidRms* p, cudaStream_t s) {
   return vec ? residual_rms<bf16, 8>(p, s) : residual_rms<bf16, 1>(p, s);
 }
 
-extern "C" int vb_gated_silu(int dtype, const void* gu, long long ldg, const float* row_scale, void* out, int T, int I, cudaStream_t s) {
+extern "C" int vb_gated_silu(int dtype, const void* gu, long long ldg, const float* row_scale, float clip, void* out, int T, int I, cudaStream_t s) {
   if (T <= 0 || I <= 0) return 0;
   const bool vec = I % 8 == 0 && ldg % 8 == 0 && !mis16(gu) && !mis16(out);
   const long long total = static_cast<long long>(T) * (vec ? I / 8 : I);
   const unsigned grid = static_cast<unsigned>((total + 255) / 256);
   if (dtype == 0) {
-    if (vec) gated_silu_kernel<float, 8><<<grid, 256, 0, s>>>((const float*)gu, ldg, row_scale, (float*)out, I, total);
-    else gated_silu_kernel<float, 1><<<grid, 256, 0, s>>>((const float*)gu, ldg, row_scale, (float*)out, I, total);
+    if (vec) gated_silu_kernel<float, 8><<<grid, 256, 0, s>>>((const float*)gu, ldg, row_scale, clip, (float*)out, I, total);
+    else gated_silu_kernel<float, 1><<<grid, 256, 0, s>>>((const float*)gu, ldg, row_scale, clip, (float*)out, I, total);
   } else {
-    if (vec) gated_silu_kernel<bf16, 8><<<grid, 256, 0, s>>>((const bf16*)gu, ldg, row_scale, (bf16*)out, I, total);
-    else gated_silu_kernel<bf16, 1><<<grid, 256, 0, s>>>((const bf16*)gu, ldg, row_scale, (bf16*)out, I, total);
+    if (vec) gated_silu_kernel<bf16, 8><<<grid, 256, 0, s>>>((const bf16*)gu, ldg, row_scale, clip, (bf16*)out, I, total);
+    else gated_silu_kernel<bf16, 1><<<grid, 256, 0, s>>>((const bf16*)gu, ldg, row_scale, clip, (bf16*)out, I, total);
   }
   return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int vb_residual_dyt(int dtype, const VbResidDyt* p, cudaStream_t s) {
+  if (p->T <= 0) return 0;
+  const bool vec = p->W % 8 == 0 && p->ldr % 8 == 0 && !mis16(p->x) && !mis16(p->rows) && !mis16(p->pw) && !mis16(p->pb) && !mis16(p->nw) && !mis16(p->nb) &&
+                   !mis16(p->h);
+  const long long total = static_cast<long long>(p->T) * (vec ? p->W / 8 : p->W);
+  const unsigned grid = static_cast<unsigned>((total + 255) / 256);
+  if (dtype == 0) {
+    if (vec) residual_dyt_kernel<float, 8><<<grid, 256, 0, s>>>(*p, total);
+    else residual_dyt_kernel<float, 1><<<grid, 256, 0, s>>>(*p, total);
+  } else {
+    if (vec) residual_dyt_kernel<bf16, 8><<<grid, 256, 0, s>>>(*p, total);
+    else residual_dyt_kernel<bf16, 1><<<grid, 256, 0, s>>>(*p, total);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W,
+                            cudaStream_t s) {
+  if (T <= 0 || W <= 0) return 0;
+  const bool vec = W % 8 == 0 && ldo % 8 == 0 && ldg % 8 == 0 && !mis16(o) && !mis16(g) && !mis16(norm) && !mis16(out);
+  if (dtype == 0) return vec ? gated_rms<float, 8>(o, ldo, g, ldg, norm, eps, out, T, W, s) : gated_rms<float, 1>(o, ldo, g, ldg, norm, eps, out, T, W, s);
+  return vec ? gated_rms<bf16, 8>(o, ldo, g, ldg, norm, eps, out, T, W, s) : gated_rms<bf16, 1>(o, ldo, g, ldg, norm, eps, out, T, W, s);
 }
 
 extern "C" int vb_qkv_prep(int dtype, const VbQkvPrep* p, cudaStream_t s) {
