@@ -98,7 +98,9 @@ def lightning(h, w, m, eps):
 
 def attention(h, w, m, eps):
     T, H, G, pos = h.shape[0], m["heads"], m["kv_heads"], torch.arange(h.shape[0])
-    part = {n: short_conv(h @ w[n].t() + w[n + ".b"], w[n + ".conv"]) for n in "qkv"}
+    part = {n: h @ w[n].t() + w[n + ".b"] for n in "qkv"}
+    if m.get("conv"):
+        part = {n: short_conv(u, w[n + ".conv"]) for n, u in part.items()}
     q = unit_rms(rotate(part["q"].view(T, H, m["dim"]), pos, m["rot"], True), eps)
     k = unit_rms(rotate(part["k"].view(T, G, m["dim"]), pos, m["rot"], True), eps)
     v, visible = part["v"].view(T, G, m["vdim"]), sees(T, m.get("mask"))

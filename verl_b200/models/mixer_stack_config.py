@@ -81,7 +81,7 @@ class GroupedAttentionSpec:
     keep_first: int = 0       # first tokens of a sequence that every query sees besides its window
     norm_after_rot: bool = False
     bias: bool = False
-    conv: int = 1             # taps; 1 = no convolution
+    conv: int = 0             # taps; 0 = no convolution
     kind: str = "attention"
 
     @property
@@ -94,7 +94,7 @@ class GroupedAttentionSpec:
 
     @property
     def state_size(self) -> int:
-        return (self.conv - 1) * self.channels
+        return max(self.conv - 1, 0) * self.channels
 
 
 @dataclass(frozen=True)
@@ -245,8 +245,8 @@ def _convolved_attention(m: dict) -> GroupedAttentionSpec:
     mask = m.get("mask") or {}
     spec = GroupedAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
                                 rot=_rotary(m["rot"], "halves"), zero_sink=False, window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
-                                norm_after_rot=True, bias=True, conv=int(m.get("conv") or 1))
-    if spec.heads % spec.kv_heads or spec.rot.dims % 2 or spec.rot.dims > spec.dim or spec.conv < 1:
+                                norm_after_rot=True, bias=True, conv=int(m.get("conv") or 0))
+    if spec.heads % spec.kv_heads or spec.rot.dims % 2 or spec.rot.dims > spec.dim or spec.conv < 0:
         raise ValueError(f"attention sizes: {spec}")
     return spec
 
@@ -379,7 +379,7 @@ def layer_tensors(spec: StackSpec, width: int, i: int) -> list:
     elif m.kind == "attention":
         out += [(p + "mix.in", (_up8(m.channels), width), "normal", True)]
         out += [(p + "mix.in.b", (_up8(m.channels),), "zeros", False)] if m.bias else []
-        out += [(p + "mix.in.conv", (m.channels, m.conv), "normal", False)] if m.conv > 1 else []
+        out += [(p + "mix.in.conv", (m.channels, m.conv), "normal", False)] if m.conv else []
         out += [] if m.norm_after_rot else [(p + "mix.q.norm", (m.dim,), "ones", False), (p + "mix.k.norm", (m.dim,), "ones", False)]
         out += [(p + "mix.vmix", (1,), "fill:0.5", False)] if m.v_mix else []
         out += [(p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
@@ -429,7 +429,7 @@ def fused_rows(spec: StackSpec, width: int, i: int) -> dict:
         out = {p + "in": [(p + name, r0, n) for name, r0, n in rows], p + "ukv": _consecutive((p + "uk", m.heads * m.dim), (p + "uv", m.heads * m.vdim))}
     elif m.kind == "attention":
         sizes = (("q", m.heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim))
-        out = {p + "in" + what: _consecutive(*((p + name + what, n) for name, n in sizes)) for what in ("", *([".b"] if m.bias else []), *([".conv"] if m.conv > 1 else []))}
+        out = {p + "in" + what: _consecutive(*((p + name + what, n) for name, n in sizes)) for what in ("", *([".b"] if m.bias else []), *([".conv"] if m.conv else []))}
     elif m.kind == "lightning":
         qk, v = m.heads * m.dim, m.heads * m.vdim
         out = {p + "in": _consecutive((p + "q", qk), (p + "k", qk), (p + "v", v), (p + "g", v))}
