@@ -43,7 +43,7 @@ def i32(v, place):
 
 
 def norm_of(width, alpha):
-    return {"n.alpha": torch.tensor(alpha), "n": 1 + rand(width, scale=0.3), "n.b": rand(width, scale=0.2)}
+    return {"n.alpha": torch.tensor(alpha), "n": rand(width), "n.b": rand(width, scale=0.2)}
 
 
 def norm_args(n, place):
@@ -107,7 +107,7 @@ def test_residual_add_of_normed_expert_rows(place, t, width, top):
 
 @pytest.mark.parametrize("t,width", [(1, 16), (5, 35), (40, 264), (3, 4096), (2, 9000)])
 def test_gated_norm_of_whole_rows(place, t, width):
-    both, w = rand(t, 2 * width + 8), 1 + rand(width, scale=0.3)
+    both, w = rand(t, 2 * width + 8), rand(width)
     view = put(both, place)
     got = X.gated_rms(put(both[:, :width].contiguous(), place), view[:, width + 8 :], put(w, place), 3e-2)
     o, g = both[:, :width].double(), both[:, width + 8 :].double()
@@ -293,7 +293,7 @@ def test_latent_attention_without_sink_and_gate(place, H, du, dr, rank, e, windo
 
 def test_latent_rows_without_a_query_latent(place):
     rank, dr, T = 40, 8, 30
-    p, w, tab = rand(T, 16 + rank + dr), 1 + rand(rank, scale=0.2), F.rope_table(64, dr, 300.0, place[0])
+    p, w, tab = rand(T, 16 + rank + dr), rand(rank), F.rope_table(64, dr, 300.0, place[0])
     pos = torch.arange(T, dtype=torch.int32, device=place[0])
     cq, rows = X.latent_prep(put(p, place)[:, 16:], None, put(w, place), 1e-3, pos, *tab, None, None, True)
     z = p[:, 16:].double()
@@ -388,7 +388,7 @@ def test_grouped_routing_and_clipped_experts(place, E, top, groups, keep, t):
     """Router, copies in expert order, both products and the sum of the rows, against the token-by-token mixture."""
     W, ff, limit = 24, 16, 0.8
     h, z = rand(t, W), torch.randn(t, -(-E // 8) * 8, generator=GEN)
-    corr = rand(E, scale=0.7) - 0.6              # many choice scores are negative
+    corr = (rand(E, scale=0.7) - 0.6).bfloat16().float()     # many choice scores are negative
     gate, up, down = rand(E, ff, W, scale=0.4), rand(E, ff, W, scale=0.4), rand(E, W, ff, scale=0.3)
     s = plain.sigmoid(z[:, :E].double())
     want = torch.zeros(t, W).double()
