@@ -3,6 +3,7 @@
     python bench.py --design zorelorn            # all sizes: prefill and decode throughput of both models
     python bench.py --design zorelorn --kernels  # the kernels behind them, each against its roofline
     python bench.py --design tofinex [--kernels]
+    python bench.py --design luzitar [--kernels]
 
 Random weights and tokens. Prefill runs packed prompts through the engine's prompt path into the cache, decode replays the
 captured decode step over all slots; CUDA events around every timed region, after warm-up, on inputs larger than L2. One
@@ -34,6 +35,15 @@ TOFINEX_SIZES = {
     "dense2048": dict(width=2048, heads=16, kv_heads=4, ff=8192, experts=0, top=0, shared_ff=0, layers=12, prompts=8, prompt_len=2048, slots=256, ctx=2048),
     "moe2048": dict(width=2048, heads=16, kv_heads=4, ff=768, experts=64, top=6, shared_ff=1536, layers=8, prompts=8, prompt_len=2048, slots=256, ctx=2048),
     "moe4096": dict(width=4096, heads=32, kv_heads=8, ff=1536, experts=32, top=2, shared_ff=3072, layers=4, prompts=4, prompt_len=4096, slots=128, ctx=4096),
+}
+# layers in turn: lightning, windowed attention, latent attention, latent attention over the rows of the one before; experts everywhere
+LUZITAR_SIZES = {
+    "moe2048": dict(width=2048, heads=16, kv_heads=4, window=1024, keep=64, ff=768, experts=64, top=6, groups=8, group_keep=4, layers=8, prompts=8, prompt_len=2048, slots=256,
+                    ctx=2048),
+    "moe2048-long": dict(width=2048, heads=16, kv_heads=4, window=1024, keep=64, ff=768, experts=64, top=6, groups=8, group_keep=4, layers=8, prompts=1, prompt_len=16384, slots=32,
+                         ctx=16384),
+    "moe4096": dict(width=4096, heads=32, kv_heads=8, window=2048, keep=64, ff=1536, experts=32, top=2, groups=4, group_keep=2, layers=4, prompts=4, prompt_len=4096, slots=128,
+                    ctx=4096),
 }
 
 
@@ -72,9 +82,31 @@ def closest_to_tofinex(s: dict, params: int) -> ModelConfig:
                        qk_norm=True, attention_bias=False, tie_word_embeddings=True, **kw)
 
 
+def luzitar_config(s: dict) -> ModelConfig:
+    H, layers = s["heads"], []
+    mlp = {"kind": "moe", "expert": {"ff": s["ff"], "limit": 7.0},
+           "router": {"experts": s["experts"], "top": s["top"], "groups": {"count": s["groups"], "keep": s["group_keep"]}}}
+    latent = dict(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=dict(base=500000.0, dims=64))
+    for i in range(0, s["layers"], 4):
+        layers += [("lightning", dict(heads=H, dim=128, vdim=128, decay=[1.0 - 2.0 ** (-2.0 - 6.0 * h / H) for h in range(H)])),
+                   ("attention", dict(heads=H, kv_heads=s["kv_heads"], dim=128, vdim=128, conv=4, scale=128 ** 0.5, mask={"size": s["window"], "keep_first": s["keep"]},
+                                      rot=dict(base=500000.0, dims=64, scaling=dict(factor=8.0, original=8192, fast=32.0, slow=1.0)))),
+                   ("latent_attention", latent), ("latent_attention", {**latent, "kv_from": i + 2})]
+    return ModelConfig.from_hf_dict({"architecture": "Luzitar", "logit_softcap": 20.0, "norm": {"eps": 1e-6}, "vocab": VOCAB, "width": s["width"],
+                                     "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in layers[: s["layers"]]]})
+
+
+def closest_to_luzitar(s: dict, params: int) -> ModelConfig:
+    """Qwen3-MoE-type decoder: full attention of the same head sizes in every layer, the same experts (softmax router)."""
+    return ModelConfig(model_type="qwen3_moe", vocab_size=VOCAB, hidden_size=s["width"], intermediate_size=s["ff"], num_hidden_layers=s["layers"],
+                       num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"], head_dim=128, rope_theta=500000.0, max_position_embeddings=1 << 15, qk_norm=True,
+                       attention_bias=False, tie_word_embeddings=False, num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"])
+
+
 # design -> (sizes, its configuration, label and configuration of the closest existing model)
 DESIGNS = {"zorelorn": (SIZES, zorelorn_config, "uniform decoder of equal size", uniform_config),
-           "tofinex": (TOFINEX_SIZES, tofinex_config, "closest existing decoder", closest_to_tofinex)}
+           "tofinex": (TOFINEX_SIZES, tofinex_config, "closest existing decoder", closest_to_tofinex),
+           "luzitar": (LUZITAR_SIZES, luzitar_config, "closest existing decoder", closest_to_luzitar)}
 
 
 def _events(fn, steps: int) -> float:
@@ -347,9 +379,163 @@ def run_tofinex_kernels(iters: int = 20, only=None, sizes=None) -> None:
     native.check_status()
 
 
+def run_luzitar_kernels(iters: int = 20, only=None, sizes=None) -> None:
+    dev = torch.device("cuda", torch.cuda.current_device())
+    timer = Timer(dev, iters, 3)
+    r = lambda *sh, sc=1.0, dt=torch.bfloat16: (torch.randn(*sh, device=dev) * sc).to(dt)
+    case = _kernel_reporter("luzitar", "closest decoder", timer, only)
+    mm = lambda m, n, k: (2.0 * m * n * k, 2.0 * (m * k + n * k + m * n))
+    ops = native.ops()
+    for name, s in LUZITAR_SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        W, H, G, E, top, ff, win, keep, d = s["width"], s["heads"], s["kv_heads"], s["experts"], s["top"], s["ff"], s["window"], s["keep"], 128
+        Q, qkv, kr, rot, scale = H * d, (H + 2 * G) * d, 512, 64, 192 ** -0.5
+        cos, sin = F.rope_table(1 << 15, d, 5e5, dev)
+        cos2, sin2 = F.rope_table(1 << 15, rot, 5e5, dev)
+        norm, post, nw = (r(1), r(W), r(W)), (r(1), r(W), r(W)), r(W)
+        for phase, T in (("prefill", s["prompts"] * s["prompt_len"]), ("decode", s["slots"])):
+            h, x, att = r(T, W), torch.randn(T, W, device=dev), r(T, Q)
+            n, L, S, ctx, bs = s["prompts"], s["prompt_len"], s["slots"], s["ctx"], 64
+            pos = torch.arange(T, device=dev, dtype=torch.int32) % L if phase == "prefill" else torch.full((T,), ctx, device=dev, dtype=torch.int32)
+            cu = torch.arange(n + 1, device=dev, dtype=torch.int32) * L
+            active = torch.ones(S, dtype=torch.bool, device=dev)
+            table, cl = None, None
+            if phase == "decode":
+                per = -(-(ctx + 64) // bs)
+                table = torch.arange(S * per, device=dev, dtype=torch.int32).view(S, per)
+                cl = torch.full((S,), ctx, device=dev, dtype=torch.int32)
+            # ---- attention of the closest model, the like kernel of every mixer
+            q, k, v = r(T, H, d), r(T, G, d), r(T, G, d)
+            if phase == "prefill":
+                case(name, phase, "attention_varlen", lambda: F.attention_varlen(q, k, v, cu, L), 4.0 * n * L * (L + 1) / 2 * Q, 2.0 * T * (2 * Q + 2 * G * d), False)
+            else:
+                kc, vc = r(S * per, bs, G, d, sc=0.5), r(S * per, bs, G, d, sc=0.5)
+                case(name, phase, "paged_decode_attention", lambda: F.paged_decode_attention(q, kc, vc, table, cl), 4.0 * S * ctx * Q, 4.0 * S * ctx * G * d, False)
+                del kc, vc
+            case(name, phase, "rope (query rotation)", lambda: F.apply_rope_(q, pos, cos, sin), 0, 4.0 * T * Q, False)
+            case(name, phase, "rmsnorm with residual", lambda: F.rms_norm(h, nw, 1e-6, residual=att[:, :W].contiguous() if Q != W else att), 0, 8.0 * T * W, False)
+            # ---- lightning
+            w = r(4 * Q, W, sc=0.02)
+            f, b = mm(T, 4 * Q, W)
+            case(name, phase, "linear_silu (q, k, v with silu, g)", lambda: X.linear_silu(h, w, 3 * Q), f, b, True)
+            case(name, phase, "gemm (q, k, v, g)", lambda: F.gemm(h, w), f, b, False)
+            p, nm = r(T, 4 * Q, sc=0.5), r(Q)
+            decay = torch.tensor([1.0 - 2.0 ** (-2.0 - 6.0 * i / H) for i in range(H)], device=dev)
+            state = torch.zeros(max(n, S), H * d * d, device=dev)
+            if phase == "prefill":
+                slots, fresh = torch.arange(n, device=dev, dtype=torch.int32), torch.ones(n, device=dev, dtype=torch.int32)
+                case(name, phase, "lightning_prefill", lambda: X.lightning_prefill(p, decay, d, d, cu, state, slots, fresh, True), 2.0 * T * H * (64 / 2 * 2 * d + 2 * d * d),
+                     8.0 * T * Q + 4.0 * n * H * d * d, True)
+            else:
+                case(name, phase, "lightning_decode", lambda: X.lightning_decode(p, decay, d, d, state, active), 0, 8.0 * T * Q + 8.0 * T * H * d * d, True)
+            case(name, phase, "gated_rms (norm of all heads, gate)", lambda: X.gated_rms(att, p[:, 3 * Q :], nm, 1e-6), 0, 6.0 * T * Q, True)
+            del w, p, state
+            # ---- windowed attention with convolved projections
+            w, bias = r(qkv, W, sc=0.02), r(qkv)
+            f, b = mm(T, qkv, W)
+            case(name, phase, "linear_bias (q, k, v)", lambda: X.linear_bias(h, w, bias), f, b, True)
+            case(name, phase, "gemm (q, k, v)", lambda: F.gemm(h, w), f, b, False)
+            p, conv, state = r(T, qkv), r(qkv, 4, sc=0.5), torch.zeros(max(n, S), 3 * qkv, device=dev)
+            if phase == "prefill":
+                kw = dict(cu=cu, state=state, slots=slots, fresh=fresh, want_rows=True)
+                by = 4.0 * T * qkv + 12.0 * n * qkv
+            else:
+                kw, by = dict(active=active, state=state, want_rows=True), 4.0 * T * qkv + 24.0 * T * qkv
+            case(name, phase, "conv_qkv_prep (convolution, rotation, norms, rows)", lambda: X.conv_qkv_prep(p, conv, 1e-6, pos, cos2, sin2, H, G, d, d, True, **kw), 0, by, True)
+            if phase == "prefill":
+                pairs = n * sum(min(i + 1, win) + max(0, min(keep, i + 1 - win)) for i in range(L))
+                case(name, phase, "grouped_attention_prefill (window, kept tokens)", lambda: X.grouped_attention_prefill(q, k, v, cu, cu, win, scale, 0.0, None, keep), 4.0 * pairs * Q,
+                     2.0 * T * (2 * Q + 2 * G * d), True)
+            else:
+                pages, seen = r(S * per, bs, 2 * G * d, sc=0.5), min(ctx, win + keep)
+                case(name, phase, "grouped_attention_decode (window, kept tokens)", lambda: X.grouped_attention_decode(q, pages, table, cl, G, d, win, scale, 0.0, None, keep),
+                     4.0 * S * seen * Q, 4.0 * S * seen * G * d, True)
+                del pages
+            del w, p, state
+            # ---- latent attention
+            cut = H * (d + rot)
+            w = r(cut + kr + rot, W, sc=0.02)
+            f, b = mm(T, cut + kr + rot, W)
+            case(name, phase, "linear_act (queries, latents)", lambda: X.linear_act(h, w), f, b, True)
+            case(name, phase, "gemm (queries, latents)", lambda: F.gemm(h, w), f, b, False)
+            p, kn = r(T, cut + kr + rot), r(kr)
+            case(name, phase, "latent_prep (norm, rotation, rows)", lambda: X.latent_prep(p[:, cut:], None, kn, 1e-6, pos, cos2, sin2, None, None, True), 0, 4.0 * T * (kr + rot), True)
+            ql = p[:, :cut].unflatten(1, (H, d + rot))
+            if phase == "prefill":
+                case(name, phase, "rope_pairs (query rotation)", lambda: X.rope_pairs_(ql, pos, cos2, sin2, d), 0, 4.0 * T * H * rot, True)
+                rows, wkv = r(T, kr + rot), r(2 * Q, kr, sc=0.05)
+                f, b = mm(T, 2 * Q, kr)
+                case(name, phase, "linear_act (keys and values of the latents)", lambda: X.linear_act(rows[:, :kr], wkv), f, b, True)
+                rc = rows[:, :kr].contiguous()
+                case(name, phase, "gemm (keys and values of the latents)", lambda: F.gemm(rc, wkv), f, b, False)
+                kv = r(T, 2 * Q)
+                ku, vl = kv[:, :Q].view(T, H, d), kv[:, Q:].view(T, H, d)
+                case(name, phase, "latent_attention_prefill", lambda: X.latent_attention_prefill(ql, ku, rows[:, kr:], vl, cu, cu, 0, scale), 2.0 * n * L * (L + 1) / 2 * H * (2 * d + rot),
+                     2.0 * T * (H * (2 * d + rot + 2 * d) + rot), True)
+                del rows, kv, ku, vl, wkv, rc
+            else:
+                pages, qa, uk, uv, oc = r(S * per, bs, kr + rot, sc=0.5), r(S, H, kr + rot), r(H, d, kr), r(H, d, kr), r(S, H, kr)
+                case(name, phase, "latent_attention_decode", lambda: X.latent_attention_decode(qa, pages, table, cl, kr, 0, scale), 2.0 * S * ctx * H * (2 * kr + rot),
+                     2.0 * S * ctx * (kr + rot) + 2.0 * S * H * (2 * kr + rot), True)
+                case(name, phase, "latent_absorb (query into latent space)", lambda: X.latent_absorb(ql, uk, pos, cos2, sin2), 2.0 * S * H * d * kr,
+                     2.0 * (S * H * (d + rot) + H * d * kr + S * H * (kr + rot)), True)
+                case(name, phase, "headwise_linear (values out of latent space)", lambda: X.headwise_linear(oc, uv, False), 2.0 * S * H * d * kr,
+                     2.0 * (S * H * kr + H * d * kr + S * H * d), True)
+                del pages, qa, uk, uv, oc
+            del w, p, ql
+            # ---- output projection, experts
+            w = r(W, Q, sc=0.02)
+            f, b = mm(T, W, Q)
+            case(name, phase, "linear_residual (output projection, both norms, residual)", lambda: X.linear_residual_(att, w, x, norm, post), f, b + 8.0 * T * W, True)
+            case(name, phase, "gemm (output projection)", lambda: F.gemm(att, w), f, b, False)
+            w, corr = r(E, W, sc=0.02), r(E)
+            f, b = mm(T, E, W)
+            case(name, phase, "linear_act (router, fp32)", lambda: X.linear_act(h, w, out_f32=True), f, b + 2.0 * T * E, True)
+            case(name, phase, "gemm (router)", lambda: F.gemm(h, w), f, b, False)
+            z = torch.randn(T, E, device=dev)
+            zb, rows = z.to(torch.bfloat16), T * top
+            used, by = min(E, rows), 4.0 * T * E + 2.0 * T * W + 2.0 * rows * W
+            case(name, phase, "expert_dispatch (groups, route, place, copy)", lambda: X.expert_dispatch(h, z, E, top, True, corr, s["groups"], s["group_keep"]), 0, by, True)
+
+            def route_other():
+                wts, idx, counts = ops.moe_route_topk(zb, top, False)
+                plan = DecoderModel._moe_plan(idx.long(), counts, T, top, E)
+                return plan, ops.moe_gather_rows(h, plan["src"], None), wts
+
+            case(name, phase, "moe_route_topk + plan + gather_rows", route_other, 0, by, False)
+            w_u, w_d = r(E * 2 * ff, W, sc=0.02), r(E * W, ff, sc=0.02)
+            plan = X.expert_dispatch(h, z, E, top, True, None, 1, 1)      # the same choices as the other router's
+            oplan, xp, wts = route_other()
+            w3, d3 = w_u.view(E, 2 * ff, W), w_d.view(E, W, ff)
+            fl, by = 2.0 * rows * 2 * ff * W, 2.0 * (used * 2 * ff * W + rows * (W + ff))
+            case(name, phase, "expert_up (gate, up, clipped activation, score)", lambda: X.expert_up(plan, w_u, ff, "clipped", 7.0), fl, by, True)
+            case(name, phase, "gemm_grouped_rows + swiglu", lambda: F.swiglu(ops.gemm_grouped_rows(xp, w3, False, oplan["tile_expert"], oplan["num_mtiles"])), fl, by, False)
+            act = X.expert_up(plan, w_u, ff, "clipped", 7.0)
+            a2 = r(xp.shape[0], ff)
+            fl, by = 2.0 * rows * ff * W, 2.0 * (used * ff * W + rows * (W + ff))
+            case(name, phase, "expert_down", lambda: X.expert_down(act, w_d, plan), fl, by, True)
+            case(name, phase, "gemm_grouped_rows (down)", lambda: ops.gemm_grouped_rows(a2, d3, False, oplan["tile_expert"], oplan["num_mtiles"]), fl, by, False)
+            out = X.expert_down(act, w_d, plan)
+            case(name, phase, "residual_dyt (experts, both norms, residual)", lambda: X.residual_dyt_(x, out, plan.slot, post, norm), 0, 2.0 * rows * W + 10.0 * T * W, True)
+            yo = ops.gemm_grouped_rows(a2, d3, False, oplan["tile_expert"], oplan["num_mtiles"])
+            case(name, phase, "moe_combine", lambda: ops.moe_combine(yo, oplan["slot"], wts), 0, 2.0 * rows * W + 2.0 * T * W, False)
+            del w, w_u, w_d, plan, act, xp, a2, out, yo
+            ids, emb = torch.randint(0, VOCAB, (T,), device=dev), r(VOCAB, W)
+            case(name, phase, "embed_dyt2 (embedding, its norm, first norm)", lambda: X.embed_dyt2(ids, emb, post, norm), 0, 8.0 * T * W, True)
+            case(name, phase, "embedding", lambda: F.embedding(ids, emb), 0, 4.0 * T * W, False)
+            if phase == "decode":
+                f, b = mm(T, VOCAB, W)
+                case(name, phase, "linear_softcap (logits)", lambda: X.linear_softcap(h, emb, 20.0), f, b, True)
+                case(name, phase, "gemm (logits)", lambda: F.gemm(h, emb), f, b, False)
+            del emb, h, x, att, q, k, v
+            torch.cuda.empty_cache()
+    native.check_status()
+
+
 def main(args) -> None:
     native.load()
     if args.kernels:
-        {"zorelorn": run_kernels, "tofinex": run_tofinex_kernels}[args.design]()
+        {"zorelorn": run_kernels, "tofinex": run_tofinex_kernels, "luzitar": run_luzitar_kernels}[args.design]()
     else:
         run_models(args.design, args.steps if args.steps > 2 else 5, args.warmup)
