@@ -192,6 +192,34 @@ def test_convolved_preparation(place, H, G, d, e, rot, taps, halves):
         close(flat, want[b][1][:n], place)
 
 
+@pytest.mark.parametrize("taps", [2, 3, 4])
+def test_convolution_of_many_portions_at_once(place, taps):
+    """Thousands of tokens in portions of one to a few hundred, some behind kept inputs."""
+    H, G, d, e, eps, rot = 6, 2, 32, 24, 1e-3, {"dims": 16, "base": 500.0}
+    C = (H + G) * d + G * e
+    lens = [1, 2, 3, 4, 5, 7, 1, 1, 300, 2, 259, 3] * 11 + [1900]
+    starts = [i % 3 * 2 for i in range(len(lens))]            # 0, 2 or 4 tokens came before
+    conv, tab = rand(C, taps, scale=taps ** -0.5), F.rope_table(2048, rot["dims"], rot["base"], place[0])
+    ps = [rand(n + a, C) for n, a in zip(lens, starts)]
+    state = torch.zeros(len(lens), (taps - 1) * C)
+    for b, (p, a) in enumerate(zip(ps, starts)):
+        before = torch.cat([torch.zeros(taps - 1, C), p[:a]])[-(taps - 1):]
+        state[b] = before.flatten() if a else 9.0
+    state = state.to(place[0])
+    part = torch.cat([p[a:] for p, a in zip(ps, starts)])
+    pos = torch.cat([torch.arange(a, a + n, dtype=torch.int32) for n, a in zip(lens, starts)]).to(place[0])
+    cu = i32([sum(lens[:i]) for i in range(len(lens) + 1)], place)
+    q, rows = X.conv_qkv_prep(put(part, place), put(conv, place), eps, pos, *tab, H, G, d, e, True, cu, state, i32(range(len(lens)), place),
+                              i32([int(a == 0) for a in starts], place), want_rows=True)
+    want = [prepared(p, conv, H, G, d, e, rot, True, eps) for p in ps]
+    at = 0
+    for n, a, (wq, wr), p, st in zip(lens, starts, want, ps, state.cpu()):
+        close(q[at : at + n], wq[a:], place)
+        close(rows[at : at + n], wr[a:], place)
+        assert torch.equal(st.view(taps - 1, C), torch.cat([torch.zeros(taps - 1, C), p])[-(taps - 1):])
+        at += n
+
+
 def test_convolution_reaches_over_every_portion_edge(place):
     """One loud input: the outputs of the next taps - 1 tokens show it wherever the portions are cut."""
     taps, H, d = 4, 1, 8

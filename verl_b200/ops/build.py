@@ -37,7 +37,7 @@ NVCC_FLAGS = [
 
 # sources whose transcendental functions, divisions and square roots keep full fp32 accuracy
 PRECISE_MATH = ("gemm_simt", "mixer_kernels", "latent_attention_simt", "mlstm_chunk", "latent_decode", "headwise_mma",
-                "stack_rows", "experts", "grouped_decode", "conv_prep", "lightning", "lightning_chunk")
+                "stack_rows", "experts", "grouped_decode", "conv_prep", "lightning", "lightning_chunk", "lightning_tcgen05")
 
 
 def _nvcc_flags(stem: str) -> list:

@@ -777,9 +777,10 @@ Tensor lightning_prefill(const Tensor& p, const Tensor& decay, int64_t d, int64_
     if (nseg > 0) {
       Tensor local;
       if (nseg > 1) local = at::empty({(int64_t)a.B * (nseg - 1) * a.H * d * e}, p.options().dtype(at::kFloat));
-      const int rc = vb_lightning_chunk(&a, nseg, nseg > 1 ? local.data_ptr<float>() : nullptr, cur_stream());
+      float* ws = nseg > 1 ? local.data_ptr<float>() : nullptr;
+      const int rc = d <= 128 ? vb_lightning_tc(&a, nseg, ws, cur_stream()) : vb_lightning_chunk(&a, nseg, ws, cur_stream());
       if (rc >= 0) {
-        verl_count_launches(nseg > 1 ? 2 : 1);
+        verl_count_launches(nseg == 1 ? 1 : d <= 128 ? 3 : 2);
         CHECK_RC(rc, "vb_lightning_chunk");
         return out;
       }

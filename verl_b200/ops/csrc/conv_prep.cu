@@ -34,71 +34,110 @@ __device__ __forceinline__ float* conv_past(const VbConvPrep& a, int b) {
   return a.state + static_cast<long long>(a.slots[b]) * a.slot_stride;
 }
 
-// A unit is one head row over a run of R tokens; L lanes share it, a lane holds eight consecutive channels of the unit (n <= 8 L)
-// with their taps and the last inputs in registers.
-template <typename T, int TAPS>
-__global__ void __launch_bounds__(256)
-conv_prep_kernel(const VbConvPrep a, int L, int R, long long units) {
-  constexpr int VEC = 8, PAST = TAPS - 1;
-  const long long u = (blockIdx.x * 256ll + threadIdx.x) / L;
-  const int lane = threadIdx.x & (L - 1), per = a.H + 2 * a.G, C = (a.H + a.G) * a.dim + a.G * a.vdim;
-  const bool live = u < units;
-  const ConvUnit un = conv_unit(a, live ? static_cast<int>(u % per) : 0);
-  const long long t0 = live ? u / per * R : 0;
-  const int c = lane * VEC, k = live ? static_cast<int>(u % per) : 0;
-  const bool in = live && c < un.n;
-  const T* p = reinterpret_cast<const T*>(a.p);
-  const int width = a.G * (a.dim + a.vdim);
-  float w[VEC][TAPS], past[PAST > 0 ? PAST : 1][VEC];
+// Eight consecutive elements as loaded; unpacking is left to the place of use, so that all loads go out first.
+template <typename T> struct Raw8;
+template <> struct Raw8<bf16> {
+  uint4 a;
+  __device__ __forceinline__ void load(const bf16* p) { a = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void zero() { a = make_uint4(0, 0, 0, 0); }
+  __device__ __forceinline__ void get(float (&v)[8]) const {
+    const uint32_t u[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
-  for (int i = 0; i < VEC; ++i)
+    for (int i = 0; i < 4; ++i) {
+      v[2 * i] = __uint_as_float(u[i] << 16);
+      v[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+    }
+  }
+};
+template <> struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
+  __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
+  __device__ __forceinline__ void get(float (&v)[8]) const {
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+};
+
+// L lanes share a head row, a lane holds eight consecutive channels (n <= 8 L) of N consecutive tokens: taps and the window of inputs
+// stay in registers. A block takes one head.
+template <typename T, int TAPS, int N>
+__global__ void __launch_bounds__(256, 2)
+conv_prep_kernel(const VbConvPrep a, int L) {
+  constexpr int VEC = 8, PAST = TAPS - 1;
+  const int lane = threadIdx.x & (L - 1), k = blockIdx.y, C = (a.H + a.G) * a.dim + a.G * a.vdim, c = lane * VEC;
+  const int t0 = (blockIdx.x * (256 / L) + threadIdx.x / L) * N;
+  const ConvUnit un = conv_unit(a, k);
+  const bool mine = c < un.n && t0 < a.T, rot = !un.is_v && c < 2 * a.half;
+  const T* p = reinterpret_cast<const T*>(a.p) + static_cast<long long>(t0) * a.ldp + un.col + c;
+  Raw8<T> raw[N];
+  int where[N];
+#pragma unroll
+  for (int u = 0; u < N; ++u) {
+    if (mine && t0 + u < a.T) raw[u].load(p + u * a.ldp);
+    else raw[u].zero();
+    where[u] = rot && t0 + u < a.T ? min(max(a.pos[t0 + u], 0), a.max_pos - 1) : 0;
+  }
+  float w[VEC * TAPS], past[PAST > 0 ? PAST : 1][VEC];
+  if (a.conv != nullptr && mine) {       // the lane's taps are consecutive: [channel, tap]
 #pragma unroll
     for (int j = 0; j < TAPS; ++j)
-      w[i][j] = in && a.conv != nullptr ? to_f(reinterpret_cast<const T*>(a.conv)[static_cast<long long>(un.col + c + i) * TAPS + j]) : (j == TAPS - 1 ? 1.f : 0.f);
-  int b = 0;
-  long long s0 = 0, s1 = 0;
-  // inputs of local tokens i - PAST .. i - 1
-  auto refill = [&](long long t) {
-    if constexpr (PAST > 0) {
-      const float* st = nullptr;
-      if (a.cu != nullptr) st = conv_past(a, b);
-      else if (a.state != nullptr && a.active[t]) st = a.state + t * a.slot_stride;
-      const long long i = a.cu != nullptr ? t - s0 : 0;
+      Vec<T, VEC>::load(reinterpret_cast<const T*>(a.conv) + static_cast<long long>(un.col + c) * TAPS + j * VEC, *reinterpret_cast<float(*)[VEC]>(w + j * VEC));
+  } else {
 #pragma unroll
-      for (int h = 0; h < PAST; ++h) {
-        const long long at = i - PAST + h;
+    for (int i = 0; i < VEC * TAPS; ++i) w[i] = i % TAPS == PAST ? 1.f : 0.f;
+  }
+  // the inputs in front of token t: rows of its portion, then what the sequence kept, then zeros
+  int s1 = 0;                            // end of the portion
+  float* st = nullptr;
+  auto refill = [&](int t) {
+    int back = 0;
+    if (a.cu != nullptr) {
+      const int b = conv_sequence(a, t);
+      back = t - a.cu[b];
+      s1 = a.cu[b + 1];
+      st = back < PAST ? conv_past(a, b) : nullptr;
+    } else {
+      s1 = t + 1;
+      st = a.state != nullptr && a.active[t] ? a.state + static_cast<long long>(t) * a.slot_stride : nullptr;
+    }
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) past[h][e] = 0.f;
-        if (!in) continue;
-        if (at >= 0) Vec<T, VEC>::load(p + (s0 + at) * a.ldp + un.col + c, past[h]);
-        else if (st != nullptr) Vec<float, VEC>::load(st + (at + PAST) * C + un.col + c, past[h]);
-      }
+    for (int h = 0; h < PAST; ++h) {
+      const int at = back - PAST + h;    // index inside the portion
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) past[h][i] = 0.f;
+      if (at >= 0) Vec<T, VEC>::load(p + static_cast<long long>(t - t0 - PAST + h) * a.ldp, past[h]);
+      else if (st != nullptr) Vec<float, VEC>::load(st + static_cast<long long>(at + PAST) * C + un.col + c, past[h]);
     }
   };
-  if (a.cu != nullptr && live) {
-    b = conv_sequence(a, t0);
-    s0 = a.cu[b];
-    s1 = a.cu[b + 1];
-  }
-  if (live) refill(t0);
-  for (int r = 0; r < R; ++r) {
-    const long long t = t0 + r;
-    const bool ok = live && t < a.T;
-    float v[VEC], x[VEC];
+  if (PAST > 0 && mine) refill(t0);
+  const bool first = c < a.half;         // of a pair of halves
+  const int src = a.halves && c < 2 * a.half ? (first ? lane + a.half / VEC : lane - a.half / VEC) : lane;
+  const float inv_n = 1.f / un.n;
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) x[i] = 0.f;
-    if (ok && a.cu != nullptr && t >= s1) {
-      while (b + 1 < a.B && t >= a.cu[b + 1]) ++b;
-      s0 = a.cu[b];
-      s1 = a.cu[b + 1];
-      refill(t);
+  for (int u = 0; u < N; ++u) {
+    const int t = t0 + u;
+    const bool ok = mine && t < a.T;
+    float cs[VEC], sn[VEC], x[VEC], v[VEC];
+    if (rot && ok) {
+      const long long tab = static_cast<long long>(where[u]) * a.half;
+      if (a.halves) {
+        Vec<float, VEC>::load(a.cos_t + tab + (first ? c : c - a.half), cs);
+        Vec<float, VEC>::load(a.sin_t + tab + (first ? c : c - a.half), sn);
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; i += 2) {
+          cs[i] = c + i < 2 * a.half ? a.cos_t[tab + ((c + i) >> 1)] : 1.f;
+          sn[i] = c + i < 2 * a.half ? a.sin_t[tab + ((c + i) >> 1)] : 0.f;
+        }
+      }
     }
-    if (ok && in) Vec<T, VEC>::load(p + t * a.ldp + un.col + c, x);
+    raw[u].get(x);
+    if (PAST > 0 && u > 0 && ok && t >= s1) refill(t);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) {
-      v[i] = w[i][TAPS - 1] * x[i];
+      v[i] = w[i * TAPS + PAST] * x[i];
 #pragma unroll
-      for (int h = 0; h < PAST; ++h) v[i] += w[i][h] * past[h][i];
+      for (int h = 0; h < PAST; ++h) v[i] += w[i * TAPS + h] * past[h][i];
     }
     if constexpr (PAST > 0) {
 #pragma unroll
@@ -107,55 +146,47 @@ conv_prep_kernel(const VbConvPrep a, int L, int R, long long units) {
         for (int i = 0; i < VEC; ++i) past[h][i] = past[h + 1][i];
 #pragma unroll
       for (int i = 0; i < VEC; ++i) past[PAST - 1][i] = x[i];
-      if (ok && in && a.cu == nullptr && a.state != nullptr && a.active[t]) {
+      if (N == 1 && ok && a.cu == nullptr && st != nullptr) {   // a step keeps its inputs itself
 #pragma unroll
-        for (int h = 0; h < PAST; ++h) Vec<float, VEC>::store(a.state + t * a.slot_stride + h * C + un.col + c, past[h]);
+        for (int h = 0; h < PAST; ++h) Vec<float, VEC>::store(st + static_cast<long long>(h) * C + un.col + c, past[h]);
       }
     }
-    // rotation; the partner of (i, i + half) sits half / 8 lanes away
-    const bool turn = ok && in && !un.is_v && c < 2 * a.half;
-    const long long tab = turn ? static_cast<long long>(min(max(a.pos[t], 0), a.max_pos - 1)) * a.half : 0;
-    if (a.halves) {
-      const int off = a.half / VEC, first = c < a.half;
-      const int src = c < 2 * a.half ? (first ? lane + off : lane - off) : lane;
+    if (!un.is_v) {                      // the same for the whole block
+      // rotation; the partner of (i, i + half) sits half / 8 lanes away
+      if (a.halves) {
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        const float o = __shfl_sync(0xffffffffu, v[i], src, L);
-        if (turn) {
-          const int f = (first ? c : c - a.half) + i;
-          const float cs = a.cos_t[tab + f], sn = a.sin_t[tab + f];
-          v[i] = first ? v[i] * cs - o * sn : v[i] * cs + o * sn;
+        for (int i = 0; i < VEC; ++i) {
+          const float o = __shfl_sync(0xffffffffu, v[i], src, L);
+          if (rot && ok) v[i] = v[i] * cs[i] + (first ? -o : o) * sn[i];
+        }
+      } else if (rot && ok) {
+#pragma unroll
+        for (int i = 0; i < VEC; i += 2) {
+          const float y = v[i], z = v[i + 1];
+          v[i] = y * cs[i] - z * sn[i];
+          v[i + 1] = z * cs[i] + y * sn[i];
         }
       }
-    } else if (turn) {
-#pragma unroll
-      for (int i = 0; i < VEC; i += 2)
-        if (c + i < 2 * a.half) {
-          const float cs = a.cos_t[tab + ((c + i) >> 1)], sn = a.sin_t[tab + ((c + i) >> 1)], y = v[i], z = v[i + 1];
-          v[i] = y * cs - z * sn;
-          v[i + 1] = z * cs + y * sn;
-        }
-    }
-    float ss = 0.f;
-    if (!un.is_v) {
+      float ss = 0.f;
 #pragma unroll
       for (int i = 0; i < VEC; ++i) ss += v[i] * v[i];
-    }
-    for (int s = L >> 1; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
-    if (!ok || !in) continue;
-    if (!un.is_v) {
-      const float f = 1.f / sqrtf(ss / un.n + a.eps);
+      if (c >= un.n) ss = 0.f;
+      for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+      const float f = rsqrtf(ss * inv_n + a.eps);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) v[i] *= f;
     }
+    if (!ok) continue;
     if (un.is_q) {
-      Vec<T, VEC>::store(reinterpret_cast<T*>(a.q) + (t * a.H + k) * a.dim + c, v);
+      Vec<T, VEC>::store(reinterpret_cast<T*>(a.q) + (static_cast<long long>(t) * a.H + k) * a.dim + c, v);
     } else {
       if (a.rows != nullptr) Vec<T, VEC>::store(reinterpret_cast<T*>(a.rows) + t * a.ldr + un.channel_row + c, v);
       if (a.pages != nullptr) {
         const long long sl = a.page_slot[t];
-        if (sl >= 0 && sl < a.num_slots)
-          Vec<T, VEC>::store(reinterpret_cast<T*>(a.pages) + (sl / a.block_size) * a.page_stride + (sl % a.block_size) * width + un.channel_row + c, v);
+        if (sl >= 0 && sl < a.num_slots) {
+          const unsigned blk = static_cast<unsigned>(sl) / static_cast<unsigned>(a.block_size), at = static_cast<unsigned>(sl) - blk * a.block_size;
+          Vec<T, VEC>::store(reinterpret_cast<T*>(a.pages) + blk * a.page_stride + static_cast<long long>(at) * (a.G * (a.dim + a.vdim)) + un.channel_row + c, v);
+        }
       }
     }
   }
@@ -256,28 +287,22 @@ extern "C" int vb_conv_prep(int dtype, const VbConvPrep* p, cudaStream_t s) {
   if (p->T <= 0) return 0;
   auto mis = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) != 0; };
   const int C = (p->H + p->G) * p->dim + p->G * p->vdim, per = p->H + 2 * p->G, most = p->dim > p->vdim ? p->dim : p->vdim;
-  const bool vec = p->dim % 8 == 0 && p->vdim % 8 == 0 && most <= 256 && p->taps <= 4 && p->ldp % 8 == 0 && p->ldr % 8 == 0 && p->page_stride % 8 == 0 &&
-                   p->slot_stride % 4 == 0 && (!p->halves || p->half % 8 == 0) && !mis(p->p) && !mis(p->q) && !mis(p->rows) && !mis(p->pages) && !mis(p->state);
+  const bool vec = p->num_slots < (1ll << 31) && per <= 65535 && p->dim % 8 == 0 && p->vdim % 8 == 0 && most <= 256 && p->taps <= 4 && p->ldp % 8 == 0 && p->ldr % 8 == 0 && p->page_stride % 8 == 0 &&
+                   p->slot_stride % 4 == 0 && (!p->halves || p->half % 8 == 0) && !mis(p->p) && !mis(p->q) && !mis(p->rows) && !mis(p->pages) && !mis(p->state) &&
+                   !mis(p->cos_t) && !mis(p->sin_t) && !mis(p->conv);
   if (p->B > 65535) return -1;
   if (vec) {
     int L = 1;
     while (L < 32 && L * 8 < most) L *= 2;
-    // long runs reuse the inputs, short ones fill the GPU
-    const int R = p->cu == nullptr ? 1 : (static_cast<long long>(p->T) * per * L > 148ll * 2048 * 32 ? 16 : 4);
-    const long long units = (p->T + R - 1ll) / R * per;
-    const unsigned grid = static_cast<unsigned>((units * L + 255) / 256);
-    auto go = [&](auto kern) { kern<<<grid, 256, 0, s>>>(*p, L, R, units); };
-    if (dtype == 0) {
-      if (p->taps == 1) go(conv_prep_kernel<float, 1>);
-      else if (p->taps == 2) go(conv_prep_kernel<float, 2>);
-      else if (p->taps == 3) go(conv_prep_kernel<float, 3>);
-      else go(conv_prep_kernel<float, 4>);
-    } else {
-      if (p->taps == 1) go(conv_prep_kernel<bf16, 1>);
-      else if (p->taps == 2) go(conv_prep_kernel<bf16, 2>);
-      else if (p->taps == 3) go(conv_prep_kernel<bf16, 3>);
-      else go(conv_prep_kernel<bf16, 4>);
-    }
+    const int n = p->cu != nullptr && static_cast<long long>(p->T) * per * L >= 148ll * 512 * 4 ? 4 : 1;     // tokens per thread
+    const dim3 grid((p->T + 256 / L * n - 1) / (256 / L * n), per);
+    auto go = [&](auto kern) { kern<<<grid, 256, 0, s>>>(*p, L); };
+#define VB_CONV(T_, N_)                                                                              \
+  (p->taps == 1 ? go(conv_prep_kernel<T_, 1, N_>) : p->taps == 2 ? go(conv_prep_kernel<T_, 2, N_>)   \
+   : p->taps == 3 ? go(conv_prep_kernel<T_, 3, N_>) : go(conv_prep_kernel<T_, 4, N_>))
+    if (n == 4) dtype == 0 ? VB_CONV(float, 4) : VB_CONV(bf16, 4);
+    else dtype == 0 ? VB_CONV(float, 1) : VB_CONV(bf16, 1);
+#undef VB_CONV
   } else {
     const long long units = static_cast<long long>(p->T) * per;
     const unsigned grid = static_cast<unsigned>((units + 3) / 4);

@@ -1,4 +1,5 @@
-// Lightning recurrence over prompts, 64 tokens at a time on m16n8k16 MMAs (bf16 q, k, v; fp32 state).
+// Lightning recurrence over prompts for query / key sizes of 129 to 256 (lightning_tcgen05.cu serves the others), 64 tokens at a time on
+// m16n8k16 MMAs (bf16 q, k, v; fp32 state).
 //
 // With the head's fixed decay l, inside a chunk
 //   o_t = l^(t + 1) q_t S_prev + sum_{s <= t} l^(t - s) (q_t . k_s) v_s
@@ -56,7 +57,7 @@ struct LcSmem {
 };
 
 template <int DP, int EW, bool FULL>
-__global__ void __launch_bounds__(32 * EW, DP == 256 ? 1 : 2)
+__global__ void __launch_bounds__(32 * EW, 1)
 lightning_chunk_kernel(const VbLightning P, int nseg, float* __restrict__ local) {
   using L = LcSmem<DP, EW>;
   constexpr int THREADS = 32 * EW, NT = DP / 8, KS = DP / 16, QROW = DP * 2, VROW = EW * 32, PROW = LC_C * 2;
@@ -266,8 +267,8 @@ using namespace vb;
 extern "C" int vb_lightning_chunk_segments(int T, int B, int H, int d, int e, int all_fresh) {
   if (d % 8 || e % 8 || d > 256 || d < 8 || e < 8 || B > 65535 || H > 65535) return 0;
   if (!all_fresh) return 1;
-  const int cols = e <= 64 ? 64 : 128, ctas = B * H * ((e + cols - 1) / cols);
-  int s = (d > 128 ? 1 : 2) * 148 / ctas;
+  const int cols = d > 128 && e <= 64 ? 64 : 128, ctas = B * H * ((e + cols - 1) / cols);
+  int s = 148 / ctas;
   const int by_len = T / B / (4 * LC_C);
   if (s > by_len) s = by_len;
   if (s > 32) s = 32;
@@ -276,7 +277,5 @@ extern "C" int vb_lightning_chunk_segments(int T, int B, int H, int d, int e, in
 
 extern "C" int vb_lightning_chunk(const VbLightning* p, int nseg, float* local, cudaStream_t s) {
   if (p->ldp % 8 || (reinterpret_cast<uintptr_t>(p->p) & 15) || (p->ldo % 2) || (reinterpret_cast<uintptr_t>(p->out) & 3)) return -1;
-  const int dp = p->d <= 64 ? 64 : p->d <= 128 ? 128 : 256;
-  if (p->e <= 64) return dp == 64 ? lc_launch<64, 4>(*p, nseg, local, s) : dp == 128 ? lc_launch<128, 4>(*p, nseg, local, s) : lc_launch<256, 4>(*p, nseg, local, s);
-  return dp == 64 ? lc_launch<64, 8>(*p, nseg, local, s) : dp == 128 ? lc_launch<128, 8>(*p, nseg, local, s) : lc_launch<256, 8>(*p, nseg, local, s);
+  return p->e <= 64 ? lc_launch<256, 4>(*p, nseg, local, s) : lc_launch<256, 8>(*p, nseg, local, s);
 }

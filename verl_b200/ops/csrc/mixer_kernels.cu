@@ -161,6 +161,60 @@ latent_prep_kernel(const T* __restrict__ p, long long ldp, const T* __restrict__
   }
 }
 
+// The same without a query latent: one warp per token, the row in registers (kv_rank <= 1024, sizes multiples of 8).
+template <int ITEMS>
+__global__ void __launch_bounds__(256)
+latent_row_kernel(const bf16* __restrict__ p, long long ldp, const bf16* __restrict__ kn, float eps, const int* __restrict__ pos, const float* __restrict__ cs,
+                  const float* __restrict__ sn, int half, int max_pos, bf16* __restrict__ lat, long long ldl, bf16* __restrict__ pages, long long page_stride,
+                  int block_size, long long num_slots, const long long* __restrict__ slot, int T, int kv_rank, int rot) {
+  const long long t = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (t >= T) return;
+  const bf16* row = p + t * ldp;
+  float v[ITEMS][8], r8[8], g[8], sum = 0.f;
+  const int rc = lane * 8;                                   // this lane's part of the shared key part
+  if (rc < rot) Vec<bf16, 8>::load(row + kv_rank + rc, r8);
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    if (c >= kv_rank) continue;
+    Vec<bf16, 8>::load(row + c, v[i]);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) sum += v[i][k] * v[i][k];
+  }
+  bf16 *d0 = lat != nullptr ? lat + t * ldl : nullptr, *d1 = nullptr;
+  if (pages != nullptr) {
+    const long long sl = slot[t];
+    if (sl >= 0 && sl < num_slots) {
+      const unsigned blk = static_cast<unsigned>(sl) / static_cast<unsigned>(block_size);
+      d1 = pages + blk * page_stride + static_cast<long long>(static_cast<unsigned>(sl) - blk * block_size) * (kv_rank + rot);
+    }
+  }
+  const float r = 1.f / sqrtf(warp_sum(sum) / kv_rank + eps);
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    if (c >= kv_rank) continue;
+    Vec<bf16, 8>::load(kn + c, g);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v[i][k] *= r * g[k];
+    if (d0 != nullptr) Vec<bf16, 8>::store(d0 + c, v[i]);
+    if (d1 != nullptr) Vec<bf16, 8>::store(d1 + c, v[i]);
+  }
+  if (rc < rot) {
+    const long long tab = static_cast<long long>(min(max(pos[t], 0), max_pos - 1)) * half;
+#pragma unroll
+    for (int k = 0; k < 8; k += 2)
+      if (rc + k < 2 * half) {
+        const float c = cs[tab + ((rc + k) >> 1)], s = sn[tab + ((rc + k) >> 1)], x = r8[k], y = r8[k + 1];
+        r8[k] = x * c - y * s;
+        r8[k + 1] = y * c + x * s;
+      }
+    if (d0 != nullptr) Vec<bf16, 8>::store(d0 + kv_rank + rc, r8);
+    if (d1 != nullptr) Vec<bf16, 8>::store(d1 + kv_rank + rc, r8);
+  }
+}
+
 // Rows of the paged cache laid out contiguously: sequence b contributes the tokens k_start[b] .. of its block table.
 template <typename T>
 __global__ void gather_pages_kernel(const T* __restrict__ pages, long long page_stride, int block_size, const int* __restrict__ bt,
@@ -492,6 +546,15 @@ extern "C" int vb_latent_prep(int dtype, const void* p, long long ldp, const voi
   if (T <= 0) return 0;
   const bool v8 = dtype == 1 && q_rank % 8 == 0 && kv_rank % 8 == 0 && rot % 8 == 0 && ldp % 8 == 0 && ldl % 8 == 0 && page_stride % 8 == 0 &&
                   !((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(pages) | reinterpret_cast<uintptr_t>(lat)) & 15);
+  if (v8 && q_rank == 0 && kv_rank <= 1024 && rot <= 256 && num_slots < (1ll << 31) && !(reinterpret_cast<uintptr_t>(kn) & 15)) {
+    const int grid = (T + 7) / 8;
+    auto go = [&](auto kern) {
+      kern<<<grid, 256, 0, s>>>((const bf16*)p, ldp, (const bf16*)kn, eps, pos, cos_t, sin_t, dims / 2, max_pos, (bf16*)lat, ldl, (bf16*)pages, page_stride, block_size,
+                                num_slots, slot, T, kv_rank, rot);
+      return static_cast<int>(cudaGetLastError());
+    };
+    return kv_rank <= 256 ? go(latent_row_kernel<1>) : kv_rank <= 512 ? go(latent_row_kernel<2>) : go(latent_row_kernel<4>);
+  }
 #define VB_PREP(T_, V_)                                                                                                                     \
   latent_prep_kernel<T_, V_><<<T, 128, 0, s>>>((const T_*)p, ldp, (const T_*)qn, (const T_*)kn, eps, pos, cos_t, sin_t, dims, max_pos, (T_*)cq, \
                                                (T_*)lat, ldl, (T_*)pages, page_stride, block_size, num_slots, slot, q_rank, kv_rank, rot)

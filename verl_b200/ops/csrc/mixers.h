@@ -170,10 +170,11 @@ int vb_residual_dyt(int dtype, const VbResidDyt* p, cudaStream_t s);
 int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W, cudaStream_t s);
 // conv_prep.cu
 int vb_conv_prep(int dtype, const VbConvPrep* p, cudaStream_t s);
-// lightning.cu / lightning_chunk.cu
+// lightning.cu / lightning_tcgen05.cu (d <= 128) / lightning_chunk.cu; nseg > 1: workspace of B (nseg - 1) H d e floats
 int vb_lightning_decode(int dtype, const VbLightning* p, cudaStream_t s);
 int vb_lightning_scan(int dtype, const VbLightning* p, cudaStream_t s);
 int vb_lightning_chunk_segments(int T, int B, int H, int d, int e, int all_fresh);
+int vb_lightning_tc(const VbLightning* p, int nseg, float* local, cudaStream_t s);
 int vb_lightning_chunk(const VbLightning* p, int nseg, float* local, cudaStream_t s);
 int vb_qkv_prep(int dtype, const VbQkvPrep* p, cudaStream_t s);
 // experts.cu

@@ -452,6 +452,11 @@ def run_luzitar_kernels(iters: int = 20, only=None, sizes=None) -> None:
                 case(name, phase, "grouped_attention_decode (window, kept tokens)", lambda: X.grouped_attention_decode(q, pages, table, cl, G, d, win, scale, 0.0, None, keep),
                      4.0 * S * seen * Q, 4.0 * S * seen * G * d, True)
                 del pages
+                few = -(-seen // bs)
+                kc, vc, ct = r(S * few, bs, G, d, sc=0.5), r(S * few, bs, G, d, sc=0.5), torch.arange(S * few, device=dev, dtype=torch.int32).view(S, few)
+                case(name, phase, "paged_decode_attention (as many keys)", lambda: F.paged_decode_attention(q, kc, vc, ct, cl.clamp(max=seen)), 4.0 * S * seen * Q, 4.0 * S * seen * G * d,
+                     False)
+                del kc, vc, ct
             del w, p, state
             # ---- latent attention
             cut = H * (d + rot)
