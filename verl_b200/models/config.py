@@ -12,7 +12,7 @@ import os
 from dataclasses import asdict, dataclass, field
 from typing import Any, Optional
 
-from .mixer_stack_config import StackSpec, is_stack_config, parse_stack
+from .mixer_stack_config import StackSpec, is_stack_config, parse_stack, sizes_from_tensors
 
 __all__ = ["ModelConfig", "PRESETS", "get_preset", "NATIVE_FAMILIES"]
 
@@ -241,7 +241,12 @@ class ModelConfig:
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
         with open(os.path.join(path, "config.json")) as f:
-            return cls.from_hf_dict(json.load(f))
+            d = json.load(f)
+        if is_stack_config(d):
+            from ..utils.model import tensor_shape
+
+            d = sizes_from_tensors(d, lambda name: tensor_shape(path, name))
+        return cls.from_hf_dict(d)
 
     def to_hf_dict(self) -> dict[str, Any]:
         if self.is_generic or self.is_stack:

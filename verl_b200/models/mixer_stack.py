@@ -9,7 +9,8 @@ Step layout: every projection that reads a layer's input is one GEMM. Stacks wit
 the GEMM that ends a sublayer adds to the residual stream and applies the next norm in its epilogue (with norms on both sides
 also the one on the sublayer's output). Stacks with RMS norms on
 the sublayers' outputs: one row kernel behind that GEMM adds up its partial products (and the experts' rows), norms them, adds
-to the stream and writes the next sublayer's input. Feed-forward activations run in the epilogue of the up-projection. Latent
+to the stream and writes the next sublayer's input. Stacks with RMS norms in front of the sublayers: the GEMM adds to the stream
+(in decode steps the row kernel adds its partial products), one row kernel norms the stream and applies the input convolution. Feed-forward activations run in the epilogue of the up-projection. Latent
 attention: prompts expand keys and values from the latents; decoding absorbs the key expansion into the query and applies the
 value expansion to the attention output, so only latent rows are read; a layer may read another layer's rows. Grouped-query
 attention caches normed, rotated keys and mixed or convolved values, the convolution's last inputs are state; experts run on
@@ -62,6 +63,7 @@ class MixerStackModel:
         self._ensure_rope(max_positions or 2048)
         self._zero_sinks: dict = {}
         self._row_readers = {l.mixer.kv_from for l in self.spec.layers if getattr(l.mixer, "kv_from", -1) >= 0}   # layers whose rows others use
+        self._no_rotation = (torch.ones(1, 0, device=self.device), torch.zeros(1, 0, device=self.device))
         self._weights = [self._layer_weights(i) for i in range(len(self.spec.layers))]
         self._final_norm = self._norm("final.norm")
         self._embed_norm = self._norm("embed.norm") if self.spec.embedding_norm else None
@@ -77,7 +79,7 @@ class MixerStackModel:
         W = {k[len(p):]: v for k, v in self.params.views.items() if k.startswith(p)}
         both = self.spec.norm_on == "both"
         out = {"norm1": self._norm(p + "norm1"), "norm1b": self._norm(p + "norm1b") if both else None,
-               **{k[4:]: v for k, v in W.items() if k.startswith("mix.")}}
+               "canon1": W.get("canon1"), **{k[4:]: v for k, v in W.items() if k.startswith("mix.")}}
         m = layer.mixer
         if m.kind == "latent_attention":
             out["uk"] = out["ukv"][: m.heads * m.dim].view(m.heads, m.dim, m.kv_rank)
@@ -120,23 +122,26 @@ class MixerStackModel:
         q = X.linear_act(cq, W["uq"]) if m.q_rank else p[:, :q_cols]
         return q.unflatten(1, (m.heads, m.dim + m.rot_dim)), rows, gate, cos, sin
 
+    def _key_rows(self, src: int, m, rows, batch: PackedBatch, pages, pc: Optional[PortionCache], portion: Optional[dict], shared: dict):
+        """(rows of the keys and values that layer ``src`` owns, their offsets per sequence); ``rows``: those of this pass when ``src`` is the
+        running layer. ``shared``: rows that other layers of this pass may use."""
+        key, cu_k = (src,), batch.cu_seqlens
+        if portion is not None:      # earlier tokens of some sequence are in the cache: take the keys from the pages
+            key = (src, m.span)
+            lo, cu_k, total = portion[m.span]
+        if key not in shared:
+            rows = X.gather_pages(pages, pc.block_table, cu_k, lo, total) if portion is not None else rows
+            if src not in self._row_readers:
+                return rows, cu_k
+            shared[key] = rows
+        return shared[key], cu_k
+
     def _attention_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict], shared: dict):
-        """``shared``: rows that other layers of this pass may use."""
         src = m.kv_from if m.kv_from >= 0 else i
         pages = pc.cache.pages(src) if pc is not None else None
         q, rows, gate, cos, sin = self._attention_in(W, m, h, batch.positions, pages, pc.slot_map if pc is not None else None, portion is None)
         X.rope_pairs_(q, batch.positions, cos, sin, m.dim)
-        cu_k, key = batch.cu_seqlens, (src, m.window, m.keep_first)
-        if portion is not None:      # earlier tokens of some sequence are in the cache: take the keys from the pages
-            lo, cu_k, total = portion[key[1:]]
-        else:
-            key = (src,)
-        if key in shared:
-            rows = shared[key]
-        else:
-            rows = X.gather_pages(pages, pc.block_table, cu_k, lo, total) if portion is not None else rows
-            if src in self._row_readers:
-                shared[key] = rows
+        rows, cu_k = self._key_rows(src, m, rows, batch, pages, pc, portion, shared)
         kv = X.linear_act(rows[:, : m.kv_rank], W["ukv"])
         ku = kv[:, : m.heads * m.dim].view(-1, m.heads, m.dim)
         v = kv[:, m.heads * m.dim :].view(-1, m.heads, m.vdim)
@@ -151,13 +156,17 @@ class MixerStackModel:
         return X.headwise_linear(oc, W["uv"], False, gate).view(S, m.heads * m.vdim)
 
     def _grouped_in(self, i, W, m, h, pos, pages, slot_map, want_rows: bool, first: dict, past: dict):
-        """Queries and the row [keys | values]; ``first`` carries the values of the stack's first value-mixing layer, ``past`` says
-        where the inputs of a convolution go on from."""
+        """Queries and the row [keys | values] (none for a layer that reads another's); ``first`` carries the values of the stack's first
+        value-mixing layer, ``past`` says where the inputs of a convolution go on from."""
         p = X.linear_bias(h, W["in"], W["in.b"]) if m.bias else X.linear_act(h, W["in"])
-        cos, sin = self._rope[m.rot.key()]
-        if m.norm_after_rot:
-            return X.conv_qkv_prep(p, W.get("in.conv"), self.spec.norm_eps, pos, cos, sin, m.heads, m.kv_heads, m.dim, m.vdim, m.rot.pairing == "halves",
-                                   **past, pages=pages, page_slots=slot_map, want_rows=want_rows)
+        if m.norm_over == "all":
+            return X.whole_norm_prep(p, W["q.norm"], W["k.norm"], W["temp"], self.spec.norm_eps, m.heads, m.kv_heads, m.vdim, pages, slot_map, want_rows)
+        cos, sin = self._rope[m.rot.key()] if m.rot is not None else self._no_rotation
+        if m.norm_after_rot or m.norm_over == "none":
+            own = m.kv_from < 0
+            return X.conv_qkv_prep(p, W.get("in.conv"), self.spec.norm_eps, pos, cos, sin, m.heads * m.maps, m.kv_heads * m.maps if own else 0, m.dim, m.vdim,
+                                   m.rot.pairing == "halves", **past, pages=pages if own else None, page_slots=slot_map, want_rows=want_rows and own,
+                                   norm=m.norm_after_rot, v_heads=m.kv_heads if own else 0)
         v_first = None
         if m.v_mix:
             if i == self.spec.value_source:
@@ -168,22 +177,30 @@ class MixerStackModel:
         return X.qkv_prep(p, W["q.norm"], W["k.norm"], self.spec.norm_eps, pos, cos, sin, m.heads, m.kv_heads, m.vdim, v_first,
                           W["vmix"] if v_first is not None else None, pages, slot_map, want_rows)
 
-    def _grouped_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict], first: dict, fresh):
-        pages = pc.cache.pages(i) if pc is not None else None
+    def _difference(self, W, m):
+        return (W["lambda"], m.diff, self.spec.norm_eps) if m.maps == 2 else None
+
+    def _grouped_prefill(self, i, W, m, h, batch: PackedBatch, pc: Optional[PortionCache], portion: Optional[dict], first: dict, fresh, shared: dict):
+        src = m.kv_from if m.kv_from >= 0 else i
+        pages = pc.cache.pages(src) if pc is not None else None
         past = {"cu": batch.cu_seqlens, "state": pc.cache.state(i), "slots": pc.slots, "fresh": fresh} if pc is not None and m.state_size else {"cu": batch.cu_seqlens}
         q, rows = self._grouped_in(i, W, m, h, batch.positions, pages, pc.slot_map if pc is not None else None, portion is None, first, past)
-        cu_k = batch.cu_seqlens
-        if portion is not None:
-            lo, cu_k, total = portion[(m.window, m.keep_first)]
-            rows = X.gather_pages(pages, pc.block_table, cu_k, lo, total)
-        k, v = rows[:, : m.kv_heads * m.dim].unflatten(1, (m.kv_heads, m.dim)), rows[:, m.kv_heads * m.dim :].unflatten(1, (m.kv_heads, m.vdim))
-        return X.grouped_attention_prefill(q, k, v, batch.cu_seqlens, cu_k, m.window, m.scale, m.softcap, W["sink"], m.keep_first).flatten(1)
+        rows, cu_k = self._key_rows(src, m, rows, batch, pages, pc, portion, shared)
+        k, v = rows[:, : m.k_cols].unflatten(1, (m.kv_heads * m.maps, m.dim)), rows[:, m.k_cols :].unflatten(1, (m.kv_heads, m.vdim))
+        return X.grouped_attention_prefill(q, k, v, batch.cu_seqlens, cu_k, m.window, m.scale, m.softcap, W["sink"], m.keep_first, m.chunk,
+                                           self._difference(W, m)).flatten(1)
 
     def _grouped_decode(self, i, W, m, h, pos, slot_map, ctx_len, active, block_table, cache, first: dict):
         past = {"state": cache.state(i), "active": active} if m.state_size else {"active": active}
-        q, _ = self._grouped_in(i, W, m, h, pos, cache.pages(i), slot_map, False, first, past)
-        return X.grouped_attention_decode(q, cache.pages(i), block_table, ctx_len, m.kv_heads, m.vdim, m.window, m.scale, m.softcap, W["sink"],
-                                          m.keep_first).flatten(1)
+        pages = cache.pages(m.kv_from if m.kv_from >= 0 else i)
+        q, _ = self._grouped_in(i, W, m, h, pos, pages, slot_map, False, first, past)
+        return X.grouped_attention_decode(q, pages, block_table, ctx_len, m.kv_heads, m.vdim, m.window, m.scale, m.softcap, W["sink"],
+                                          m.keep_first, m.chunk, self._difference(W, m)).flatten(1)
+
+    def _delta_in(self, W, m, h):
+        """The fused projection [r | k | v | a | g | ...] and the decay's pre-activation."""
+        p = X.linear_tanh(h, W["in"], m.low)
+        return p, X.linear_act(p[:, m.low : m.low + m.rank], W["w2"])
 
     def _lightning(self, W, m, h, recur: Callable) -> torch.Tensor:
         n = m.heads * (2 * m.dim + m.vdim)
@@ -194,9 +211,12 @@ class MixerStackModel:
         return X.linear_split(h, W["in"], 2 * m.heads * (m.dim + m.vdim))
 
     # ------------------------------------------------------------------------------------ layer loop
-    def _run(self, ids: torch.Tensor, mix: Callable) -> torch.Tensor:
-        """Embedding, layers, final norm; ``mix(i, weights, mixer, h)`` is the layer's mixer up to its output projection."""
-        return (self._run_output_norms if self.spec.norm_on == "output" else self._run_input_norms)(ids, mix)
+    def _run(self, ids: torch.Tensor, mix: Callable, past: Callable) -> torch.Tensor:
+        """Embedding, layers, final norm; ``mix(i, weights, mixer, h)`` is the layer's mixer up to its output projection, ``past(i)`` says where
+        the convolution of a layer's input goes on from."""
+        if self.spec.norm_on == "output":
+            return self._run_output_norms(ids, mix)
+        return self._run_input_norms(ids, mix) if self.spec.norm == "dynamic_tanh" else self._run_input_rms(ids, mix, past)
 
     def _layer_done(self, i: int, x: torch.Tensor) -> None:
         if self.stats_hook is not None:
@@ -222,6 +242,32 @@ class MixerStackModel:
                 h = X.linear_residual_(X.linear_act(h, W["mlp.up"], f.act), W["mlp.down"], x, nxt, W["norm2b"])
             self._layer_done(i, x)
         return h
+
+    def _run_input_rms(self, ids: torch.Tensor, mix: Callable, past: Callable) -> torch.Tensor:
+        """RMS norms in front of the sublayers, with ``input_conv`` a convolution of the mixers' inputs."""
+        layers, Ws, eps = self.spec.layers, self._weights, self.spec.norm_eps
+        x = X.embed_rows(ids, self.params["embed"], self.spec.embedding_scale)
+        y = bias = None        # what the row kernel still has to add to the stream
+        steps = "active" in past(0)
+
+        def add(a, w, b=None):
+            if steps:
+                return X.linear_partial(a, w), b
+            X.linear_residual_(a, w, x, bias=b)
+            return None, None
+
+        for i, layer in enumerate(layers):
+            W, f = Ws[i], layer.mlp
+            h = X.rms_conv(x, W["norm1"], eps, y, bias, W["canon1"], **(past(i) if W["canon1"] is not None else {}))
+            y, bias = add(mix(i, W, layer.mixer, h), W["o"])
+            if f is not None:
+                h = X.rms_conv(x, W["norm2"], eps, y, bias)
+                up = X.linear_bias(h, W["mlp.up"], W["mlp.up.b"], f.act) if f.bias else X.linear_act(h, W["mlp.up"], f.act)
+                y, bias = add(up, W["mlp.down"], W.get("mlp.down.b"))
+            if self.stats_hook is not None:
+                total = x if y is None else x + (y.float().sum(0) if y.dim() == 3 else y.float())
+                self._layer_done(i, total if bias is None else total + bias.float())
+        return X.rms_conv(x, self._final_norm, eps, y, bias)
 
     def _run_output_norms(self, ids: torch.Tensor, mix: Callable) -> torch.Tensor:
         spec, layers = self.spec, self.spec.layers
@@ -253,9 +299,10 @@ class MixerStackModel:
         portion = None
         if any(starts):
             portion = {}
-            for w in {(l.mixer.window, l.mixer.keep_first) for l in self.spec.layers if hasattr(l.mixer, "window")}:
-                # rows a layer reads: from the window's start, or all where the first tokens stay visible
-                lo = [max(0, s - w[0] + 1) if w[0] > 0 and w[1] == 0 else 0 for s in starts]
+            for w in {l.mixer.span for l in self.spec.layers if hasattr(l.mixer, "span")}:
+                # rows a layer reads: from the window's or the chunk's start, or all where the first tokens stay visible
+                window, keep, chunk = w
+                lo = [s // chunk * chunk if chunk > 0 else max(0, s - window + 1) if window > 0 and keep == 0 else 0 for s in starts]
                 cu = torch.zeros(len(lens) + 1, dtype=torch.int32)
                 cu[1:] = torch.cumsum(torch.tensor([s + n - a for s, n, a in zip(starts, lens, lo)], dtype=torch.int32), 0)
                 portion[w] = (torch.tensor(lo, dtype=torch.int32).to(self.device), cu.to(self.device), int(cu[-1]))
@@ -267,7 +314,12 @@ class MixerStackModel:
             if m.kind == "latent_attention":
                 return self._attention_prefill(i, W, m, h, batch, pc, portion, shared)
             if m.kind == "attention":
-                return self._grouped_prefill(i, W, m, h, batch, pc, portion, first, fresh)
+                return self._grouped_prefill(i, W, m, h, batch, pc, portion, first, fresh, shared)
+            if m.kind == "general_delta":
+                kept = (pc.cache.state(i), pc.slots, fresh) if pc is not None else (None, None, None)
+                p, zw = self._delta_in(W, m, h)
+                o = X.delta_prefill(p, zw, W["a.b"], W["w0"], m.heads, batch.cu_seqlens, *kept)
+                return X.gated_rms(o, p[:, 4 * m.width : 5 * m.width], W["norm"], self.spec.norm_eps, m.heads)
             if m.kind == "lightning":
                 kept = (pc.cache.state(i), pc.slots, fresh) if pc is not None else (None, None, None)
                 return self._lightning(W, m, h, lambda *a: X.lightning_prefill(*a, batch.cu_seqlens, *kept, not any(starts)))
@@ -275,7 +327,11 @@ class MixerStackModel:
             return X.mlstm_prefill(p, gates, W["i.b"], W["f.b"], m.gate_cap, W["norm"], self.spec.norm_eps, m.dim, batch.cu_seqlens,
                                    pc.cache.state(i) if pc is not None else None, pc.slots if pc is not None else None, fresh, not any(starts))
 
-        return self._run(batch.input_ids, mix)
+        def past(i):
+            kept = {"state": pc.cache.input_state(i), "slots": pc.slots, "fresh": fresh} if pc is not None and self.spec.input_conv > 1 else {}
+            return {"cu": batch.cu_seqlens, **kept}
+
+        return self._run(batch.input_ids, mix, past)
 
     @torch.no_grad()
     def decode_hidden(self, tok, pos, slot_map, ctx_len, active, block_table, cache) -> torch.Tensor:
@@ -287,12 +343,15 @@ class MixerStackModel:
                 return self._attention_decode(i, W, m, h, pos, slot_map, ctx_len, block_table, cache)
             if m.kind == "attention":
                 return self._grouped_decode(i, W, m, h, pos, slot_map, ctx_len, active, block_table, cache, first)
+            if m.kind == "general_delta":
+                p, zw = self._delta_in(W, m, h)
+                return X.delta_decode(p, zw, W["a.b"], W["w0"], m.heads, W["norm"], self.spec.norm_eps, cache.state(i), active)
             if m.kind == "lightning":
                 return self._lightning(W, m, h, lambda *a: X.lightning_decode(*a, cache.state(i), active))
             p, gates = self._mlstm_in(W, m, h)
             return X.mlstm_decode(p, gates, W["i.b"], W["f.b"], m.gate_cap, W["norm"], self.spec.norm_eps, m.dim, cache.state(i), active)
 
-        return self._run(tok, mix)
+        return self._run(tok, mix, lambda i: {"state": cache.input_state(i) if self.spec.input_conv > 1 else None, "active": active})
 
     # ------------------------------------------------------------------------------------ heads
     def logits(self, h: torch.Tensor) -> torch.Tensor:

@@ -9,11 +9,11 @@ configuration.
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Any, Callable, Optional, Union
 
-__all__ = ["RotarySpec", "LatentAttentionSpec", "GroupedAttentionSpec", "MLstmSpec", "LightningSpec", "DenseMlpSpec", "GatedMlpSpec", "MoeSpec", "LayerSpec",
-           "StackSpec", "DESIGNS", "is_stack_config", "parse_stack"]
+__all__ = ["RotarySpec", "LatentAttentionSpec", "GroupedAttentionSpec", "MLstmSpec", "LightningSpec", "DeltaSpec", "DenseMlpSpec", "GatedMlpSpec", "MoeSpec",
+           "LayerSpec", "StackSpec", "DESIGNS", "is_stack_config", "sizes_from_tensors", "parse_stack"]
 
 
 @dataclass(frozen=True)
@@ -52,6 +52,10 @@ class LatentAttentionSpec:
     kind: str = "latent_attention"
 
     @property
+    def span(self) -> tuple:
+        return (self.window, self.keep_first, 0)
+
+    @property
     def page_width(self) -> int:
         return self.kv_rank + self.rot_dim if self.kv_from < 0 else 0
 
@@ -65,15 +69,17 @@ class GroupedAttentionSpec:
     """Grouped-query attention over cached keys and values: RMS norm per query / key head, rotation of the first ``rot.dims``
     dimensions, optional soft cap of the scores, an optional key of score 0 that has no value, and values mixed with those of
     the stack's first value-mixing layer. The norms carry weights and come before the rotation, or are plain and come after it
-    (``norm_after_rot``). The projections may have biases and pass a causal convolution of ``conv`` taps over time per channel,
-    whose last ``conv`` - 1 inputs are part of a sequence's state."""
+    (``norm_after_rot``), or span all heads (``norm_over`` "all"), or there are none. The projections may have biases and pass a
+    causal convolution of ``conv`` taps over time per channel, whose last ``conv`` - 1 inputs are part of a sequence's state. With
+    ``maps`` 2 (differential attention) every head has two query / key maps of ``dim`` over the same values; the head's output is the
+    first map's minus lambda times the second's, normed, times 1 - ``diff``. A layer with ``kv_from`` reads the rows that layer cached."""
 
     heads: int
     kv_heads: int
     dim: int          # query / key size per head
     vdim: int
     scale: float
-    rot: RotarySpec
+    rot: Optional[RotarySpec]
     softcap: float = 0.0      # score = softcap * tanh(score / softcap); 0 = off
     zero_sink: bool = True    # one is added to the softmax denominator
     v_mix: bool = False
@@ -82,15 +88,40 @@ class GroupedAttentionSpec:
     norm_after_rot: bool = False
     bias: bool = False
     conv: int = 0             # taps; 0 = no convolution
+    chunk: int = 0            # a query sees the keys of its own chunk of this many positions; 0 = all
+    maps: int = 1             # 2: differential attention
+    diff: float = 0.0
+    norm_over: str = "head"   # what a query / key norm spans: "head" | "all" heads | "none"
+    temp: bool = False        # scores times one number per head
+    kv_from: int = -1         # layer whose cached rows are used; -1: own rows
     kind: str = "attention"
 
     @property
+    def q_cols(self) -> int:
+        return self.heads * self.maps * self.dim
+
+    @property
+    def k_cols(self) -> int:
+        return self.kv_heads * self.maps * self.dim
+
+    @property
+    def row_width(self) -> int:
+        """Cached row [keys | values]."""
+        return self.k_cols + self.kv_heads * self.vdim
+
+    @property
     def channels(self) -> int:
-        return (self.heads + self.kv_heads) * self.dim + self.kv_heads * self.vdim
+        """Projected columns."""
+        return self.q_cols + (self.row_width if self.kv_from < 0 else 0)
 
     @property
     def page_width(self) -> int:
-        return self.kv_heads * (self.dim + self.vdim)
+        return self.row_width if self.kv_from < 0 else 0
+
+    @property
+    def span(self) -> tuple:
+        """What decides which cached rows a prompt portion reads."""
+        return (self.window, self.keep_first, self.chunk)
 
     @property
     def state_size(self) -> int:
@@ -137,9 +168,43 @@ class LightningSpec:
 
 
 @dataclass(frozen=True)
+class DeltaSpec:
+    """Generalized delta rule on a matrix memory: per head S = diag(w) S - (a u) (u^T S) + k v^T, read with r; u is the unit key, the
+    decay w and the removal rate a are numbers per head and key channel. The decay's pre-activation comes through ``rank`` channels
+    with a tanh. Every head's output is normed, the heads are gated together."""
+
+    heads: int
+    dim: int
+    rank: int
+    kind: str = "general_delta"
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @property
+    def width(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def low(self) -> int:
+        """First column of the decay's channels in the fused projection [r | k | v | a | g | decay]."""
+        return _up8(5 * self.width)
+
+    @property
+    def page_width(self) -> int:
+        return 0
+
+    @property
+    def state_size(self) -> int:
+        return self.heads * self.dim * self.dim
+
+
+@dataclass(frozen=True)
 class DenseMlpSpec:
     ff: int
-    act: str = "gelu_erf"
+    act: str = "gelu_erf"     # "gelu_erf" | "relu2" (the square of relu)
+    bias: bool = False
     kind: str = "dense"
 
 
@@ -174,7 +239,7 @@ class MoeSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[LatentAttentionSpec, GroupedAttentionSpec, MLstmSpec, LightningSpec]
+    mixer: Union[LatentAttentionSpec, GroupedAttentionSpec, MLstmSpec, LightningSpec, DeltaSpec]
     mlp: Union[DenseMlpSpec, GatedMlpSpec, MoeSpec, None]
     owner: int        # layer whose tensors this one uses (itself, or an earlier one with shared weights)
 
@@ -191,10 +256,11 @@ class StackSpec:
     embedding_norm: bool = False  # the embedding passes the stack's norm
     tied_head: bool = False       # the output matrix is the embedding table
     logit_softcap: float = 0.0    # 0 = off
+    input_conv: int = 0           # taps of the causal convolution that every mixer's input h passes, h + conv(h); the last taps - 1 h are state
 
     @property
     def recurrent(self) -> bool:
-        return any(l.mixer.state_size for l in self.layers)
+        return self.input_conv > 1 or any(l.mixer.state_size for l in self.layers)
 
     @property
     def value_source(self) -> int:
@@ -256,6 +322,29 @@ def _lightning(m: dict) -> LightningSpec:
     if len(spec.decay) != spec.heads:
         raise ValueError(f"one decay per head: {spec}")
     return spec
+
+
+def _chunk(m: dict) -> int:
+    return int((m.get("mask") or {}).get("size") or 0)
+
+
+def _differential_attention(m: dict) -> GroupedAttentionSpec:
+    """Two rotated query / key maps per head, no norms; keys and values may be another layer's."""
+    return GroupedAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                                rot=_rotary(m["rot"], "halves"), zero_sink=False, chunk=_chunk(m), maps=2, diff=float(m["diff"]), norm_over="none",
+                                kv_from=int(m["kv_from"]) if m.get("kv_from") is not None else -1)
+
+
+def _whole_norm_attention(m: dict) -> GroupedAttentionSpec:
+    """Norms over the whole query and key projections, one temperature per head, no rotation."""
+    return GroupedAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]), rot=None,
+                                zero_sink=False, chunk=_chunk(m), norm_over="all", temp=True)
+
+
+def _general_delta(m: dict) -> DeltaSpec:
+    if "decay_rank" not in m:
+        raise ValueError("a general_delta mixer needs decay_rank (read from the weights with sizes_from_tensors)")
+    return DeltaSpec(heads=int(m["heads"]), dim=int(m["dim"]), rank=int(m["decay_rank"]))
 
 
 MIXER_READERS: dict[str, Callable[[dict], Any]] = {"latent_attention": _latent_attention, "mlstm": _mlstm, "attention": _grouped_attention}
@@ -328,11 +417,44 @@ def parse_luzitar(d: dict) -> StackSpec:
     return spec
 
 
-DESIGNS: dict[str, Callable[[dict], StackSpec]] = {"Zorelorn": parse_zorelorn, "Tofinex": parse_tofinex, "Luzitar": parse_luzitar}
+def parse_fusazen(d: dict) -> StackSpec:
+    readers = {"general_delta": _general_delta, "attention": _differential_attention, "attention_2": _whole_norm_attention}
+    layers = tuple(replace(l, mlp=DenseMlpSpec(ff=l.mlp.ff, act="relu2", bias=True)) if l.mlp is not None else l for l in _layers(d, readers))
+    spec = StackSpec(design="Fusazen", embedding_scale=float(d["embedding"]["scale"]), norm="rms", norm_eps=float(d["norm"]["eps"]), layers=layers,
+                     input_conv=int(d["canon"]["taps"]))
+    if spec.input_conv < 1:
+        raise ValueError(f"taps of the input convolution: {spec.input_conv}")
+    for i, l in enumerate(spec.layers):
+        m = l.mixer
+        if m.kind != "attention":
+            continue
+        if m.heads % m.kv_heads or m.chunk < 0 or (m.rot is not None and (m.rot.dims % 2 or m.rot.dims > m.dim)):
+            raise ValueError(f"attention sizes: {m}")
+        if m.kv_from >= 0:
+            src = spec.layers[m.kv_from].mixer if m.kv_from < i else None
+            same = lambda a: (a.kind, a.maps, a.kv_heads, a.dim, a.vdim, a.rot)
+            if src is None or src.kind != "attention" or src.kv_from >= 0 or same(src) != same(m):
+                raise ValueError(f"layer {i}: kv_from {m.kv_from} must be an earlier layer of the same kind with rows of its own, of the same sizes and rotation")
+    return spec
+
+
+DESIGNS: dict[str, Callable[[dict], StackSpec]] = {"Zorelorn": parse_zorelorn, "Tofinex": parse_tofinex, "Luzitar": parse_luzitar, "Fusazen": parse_fusazen}
 
 
 def is_stack_config(d: dict) -> bool:
     return d.get("architecture") in DESIGNS
+
+
+def sizes_from_tensors(d: dict, shape_of: Callable[[str], tuple]) -> dict:
+    """The configuration with the sizes that only the weights tell; ``shape_of`` gives the shape of a stored tensor."""
+    if d.get("architecture") != "Fusazen":
+        return d
+    layers = []
+    for i, l in enumerate(d["layers"]):
+        if l["type"] == "general_delta" and "decay_rank" not in l["mixer"]:
+            l = {**l, "mixer": {**l["mixer"], "decay_rank": int(shape_of(f"l{i}.mix.w1")[0])}}
+        layers.append(l)
+    return {**d, "layers": layers}
 
 
 def parse_stack(d: dict) -> StackSpec:
@@ -364,6 +486,7 @@ def layer_tensors(spec: StackSpec, width: int, i: int) -> list:
     l, p = spec.layers[i], f"l{i}."
     sides = lambda name: norm_tensors(spec, p + name, width) + (norm_tensors(spec, p + name + "b", width) if spec.norm_on == "both" else [])
     out = sides("norm1")
+    out += [(p + "canon1", (width, spec.input_conv), "normal", False)] if spec.input_conv else []
     m, f = l.mixer, l.mlp
     if m.kind == "latent_attention":
         # queries (or their latent), key / value latent with the rotated key part, gates
@@ -380,9 +503,17 @@ def layer_tensors(spec: StackSpec, width: int, i: int) -> list:
         out += [(p + "mix.in", (_up8(m.channels), width), "normal", True)]
         out += [(p + "mix.in.b", (_up8(m.channels),), "zeros", False)] if m.bias else []
         out += [(p + "mix.in.conv", (m.channels, m.conv), "normal", False)] if m.conv else []
-        out += [] if m.norm_after_rot else [(p + "mix.q.norm", (m.dim,), "ones", False), (p + "mix.k.norm", (m.dim,), "ones", False)]
+        if not m.norm_after_rot and m.norm_over != "none":
+            out += [(p + "mix.q.norm", (m.dim if m.norm_over == "head" else m.q_cols,), "ones", False),
+                    (p + "mix.k.norm", (m.dim if m.norm_over == "head" else m.k_cols,), "ones", False)]
+        out += [(p + "mix.temp", (m.heads,), "ones", False)] if m.temp else []
+        out += [(p + "mix.lambda", (4 * m.dim,), "zeros", False)] if m.maps == 2 else []
         out += [(p + "mix.vmix", (1,), "fill:0.5", False)] if m.v_mix else []
         out += [(p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
+    elif m.kind == "general_delta":
+        n = m.width
+        out += [(p + "mix.in", (m.low + _up8(m.rank), width), "normal", True), (p + "mix.a.b", (n,), "zeros", False), (p + "mix.w2", (n, m.rank), "normal", True),
+                (p + "mix.w0", (n,), "zeros", False), (p + "mix.norm", (n,), "ones", False), (p + "mix.o", (width, n), "normal", True)]
     elif m.kind == "lightning":
         out += [(p + "mix.in", (_up8(2 * m.heads * (m.dim + m.vdim)), width), "normal", True), (p + "mix.norm", (m.heads * m.vdim,), "ones", False),
                 (p + "mix.o", (width, m.heads * m.vdim), "normal", True)]
@@ -395,6 +526,7 @@ def layer_tensors(spec: StackSpec, width: int, i: int) -> list:
     out += sides("norm2")
     if f.kind == "dense":
         out += [(p + "mlp.up", (f.ff, width), "normal", True), (p + "mlp.down", (width, f.ff), "normal", True)]
+        out += [(p + "mlp.up.b", (f.ff,), "zeros", False), (p + "mlp.down.b", (width,), "zeros", False)] if f.bias else []
     elif f.kind == "gated":
         out += [(p + "mlp.in", (2 * f.ff, width), "normal", True), (p + "mlp.down", (width, f.ff), "normal", True)]
     else:
@@ -428,8 +560,12 @@ def fused_rows(spec: StackSpec, width: int, i: int) -> dict:
         rows += [("g", at, m.heads)] if m.gate else []
         out = {p + "in": [(p + name, r0, n) for name, r0, n in rows], p + "ukv": _consecutive((p + "uk", m.heads * m.dim), (p + "uv", m.heads * m.vdim))}
     elif m.kind == "attention":
-        sizes = (("q", m.heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim))
+        sizes = (("q", m.q_cols), *((("k", m.k_cols), ("v", m.kv_heads * m.vdim)) if m.kv_from < 0 else ()))
         out = {p + "in" + what: _consecutive(*((p + name + what, n) for name, n in sizes)) for what in ("", *([".b"] if m.bias else []), *([".conv"] if m.conv else []))}
+        if m.maps == 2:
+            out[p + "lambda"] = _consecutive(*((p + name, m.dim) for name in ("lq1", "lk1", "lq2", "lk2")))
+    elif m.kind == "general_delta":
+        out = {p + "in": _consecutive(*((p + name, m.width) for name in "rkvag")) + [(p + "w1", m.low, m.rank)]}
     elif m.kind == "lightning":
         qk, v = m.heads * m.dim, m.heads * m.vdim
         out = {p + "in": _consecutive((p + "q", qk), (p + "k", qk), (p + "v", v), (p + "g", v))}

@@ -1,6 +1,6 @@
 """Operators of the mixer stacks (``models/mixer_stack.py``): norms, GEMMs with fused epilogues, latent attention over expanded
 keys (prompts) and over the paged latents (decoding), grouped-query attention with capped scores over cached keys and values,
-mixtures of experts, short convolutions, and the mLSTM and lightning recurrences.
+differential attention, mixtures of experts, short convolutions, and the mLSTM, lightning and delta-rule recurrences.
 
 As in ``functional``: CUDA tensors go to the hand-written kernels (bf16 or true fp32; nothing falls back silently), CPU
 tensors take a plain PyTorch path. The residual stream, gates, statistics and recurrent state are fp32 on every path.
@@ -8,6 +8,7 @@ tensors take a plain PyTorch path. The residual stream, gates, statistics and re
 
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Optional
 
@@ -20,7 +21,8 @@ __all__ = ["embed_dyt", "dynamic_tanh", "linear_act", "linear_split", "linear_re
            "headwise_linear", "latent_absorb", "latent_attention_prefill", "latent_attention_decode", "mlstm_prefill", "mlstm_decode",
            "embed_rms", "linear_partial", "linear_softcap", "residual_rms_", "gated_silu", "gated_up", "gated_up_split", "ExpertPlan", "expert_dispatch",
            "expert_up", "expert_down", "qkv_prep", "grouped_attention_prefill", "grouped_attention_decode", "embed_dyt2", "linear_bias",
-           "linear_silu", "residual_dyt_", "conv_qkv_prep", "lightning_prefill", "lightning_decode", "gated_rms"]
+           "linear_silu", "residual_dyt_", "conv_qkv_prep", "lightning_prefill", "lightning_decode", "gated_rms",
+           "embed_rows", "rms_conv", "linear_tanh", "whole_norm_prep", "delta_prefill", "delta_decode"]
 
 
 def _ops():
@@ -77,11 +79,21 @@ def linear_split(a: torch.Tensor, w: torch.Tensor, n0: int):
     return y[:, :n0].to(a.dtype).contiguous(), y[:, n0:].contiguous()
 
 
-def linear_bias(a: torch.Tensor, w: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
-    """``a w^T + b``."""
+def linear_bias(a: torch.Tensor, w: torch.Tensor, b: torch.Tensor, act: Optional[str] = None) -> torch.Tensor:
+    """``a w^T + b`` with an optional activation (``relu2``: the square of relu) in the epilogue."""
+    assert act in (None, "relu2")
     if a.is_cuda:
-        return _ops().linear_bias(a, w, b)
-    return (_mm(a, w) + b.float()).to(a.dtype)
+        return _ops().linear_bias(a, w, b, act == "relu2")
+    y = _mm(a, w) + b.float()
+    return (y if act is None else y.clamp(min=0).square()).to(a.dtype)
+
+
+def linear_tanh(a: torch.Tensor, w: torch.Tensor, n0: int) -> torch.Tensor:
+    """``a w^T`` with a tanh on the columns from ``n0`` on."""
+    if a.is_cuda:
+        return _ops().linear_tanh(a, w, int(n0))
+    y = _mm(a, w)
+    return torch.cat([y[:, :n0], torch.tanh(y[:, n0:])], -1).to(a.dtype)
 
 
 def linear_silu(a: torch.Tensor, w: torch.Tensor, n0: int) -> torch.Tensor:
@@ -92,14 +104,14 @@ def linear_silu(a: torch.Tensor, w: torch.Tensor, n0: int) -> torch.Tensor:
     return torch.cat([TF.silu(y[:, :n0]), y[:, n0:]], -1).to(a.dtype)
 
 
-def linear_residual_(a: torch.Tensor, w: torch.Tensor, x: torch.Tensor, norm=None, post=None) -> Optional[torch.Tensor]:
-    """``x += a w^T`` on the fp32 residual stream, or with ``post = (alpha, weight, bias)`` the Dynamic Tanh of that product; with
+def linear_residual_(a: torch.Tensor, w: torch.Tensor, x: torch.Tensor, norm=None, post=None, bias=None) -> Optional[torch.Tensor]:
+    """``x += a w^T (+ bias)`` on the fp32 residual stream, or with ``post = (alpha, weight, bias)`` the Dynamic Tanh of that product; with
     ``norm`` (likewise) also returns the Dynamic Tanh of the new stream, computed in the same epilogue."""
     none = (None, None, None)
     if a.is_cuda:
-        h = _ops().linear_residual_(a, w, x, *(norm if norm is not None else none), *(post if post is not None else none))
+        h = _ops().linear_residual_(a, w, x, *(norm if norm is not None else none), *(post if post is not None else none), bias)
         return h if norm is not None else None
-    y = _mm(a, w)
+    y = _mm(a, w) if bias is None else _mm(a, w) + bias.float()
     x += y if post is None else dynamic_tanh_f32(y, *post)
     return dynamic_tanh(x, *norm) if norm is not None else None
 
@@ -124,6 +136,31 @@ def embed_rms(ids, weight, scale: float, nw, eps: float):
         return _ops().embed_rms(ids.reshape(-1).contiguous(), weight, float(scale), nw, float(eps))
     x = _rms(weight[ids.reshape(-1)].float() * scale, nw, eps)
     return x, x.to(weight.dtype)
+
+
+def embed_rows(ids, weight, scale: float) -> torch.Tensor:
+    """fp32 residual stream ``weight[ids] * scale``."""
+    if weight.is_cuda:
+        return _ops().embed_rows(ids.reshape(-1).contiguous(), weight, float(scale))
+    return weight[ids.reshape(-1)].float() * scale
+
+
+def rms_conv(x: torch.Tensor, nw: torch.Tensor, eps: float, y=None, bias=None, conv=None, cu=None, state=None, slots=None, fresh=None, active=None) -> torch.Tensor:
+    """``h = rms_norm(x) * nw`` of the fp32 residual stream in the weights' type, or with ``conv`` [width, taps] ``h`` plus its causal
+    convolution over time (last tap: the token itself, zeros before a sequence's first token). ``y`` ([T, W], or partial products
+    [splits, T, W]) and ``bias`` are added to ``x`` first (not with ``cu``). Portions (``cu``), steps (``active``) and ``state`` as in
+    ``conv_qkv_prep``: what is kept are the last taps - 1 rows ``h`` (fp32) of a sequence."""
+    assert y is None or cu is None, "rms_conv: portions take the stream as it is"
+    if x.is_cuda:
+        return _ops().rms_conv(x, y, bias, nw, float(eps), conv, cu, state, slots, fresh, active)
+    if y is not None:
+        x += y.float().sum(0) if y.dim() == 3 else y.float()
+    if bias is not None:
+        x += bias.float()
+    h = _rms(x, nw, eps)
+    if conv is not None:
+        h = h + _conv_rows(h, conv, cu, state, slots, fresh, active)
+    return h.to(nw.dtype)
 
 
 def linear_partial(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -334,15 +371,19 @@ def _sink_softmax(s: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor
     return torch.softmax(torch.cat([s, extra], -1), -1)[..., :-1]
 
 
-def _hidden_keys(nq: int, nk: int, window: int, keep_first: int) -> torch.Tensor:
+def _hidden_keys(nq: int, nk: int, window: int, keep_first: int, chunk: int = 0) -> torch.Tensor:
     """[nq, nk]: keys a query does not see; the last query sits on the last key."""
     dist, key = torch.arange(nk - nq, nk)[:, None] - torch.arange(nk)[None, :], torch.arange(nk)[None, :]
+    if chunk > 0:
+        return (dist < 0) | ((dist + key) // chunk != key // chunk)
     return (dist < 0) | ((dist >= window) & (key >= keep_first) if window > 0 else torch.zeros_like(dist, dtype=torch.bool))
 
 
-def _seen_keys(n: int, window: int, keep_first: int) -> torch.Tensor:
+def _seen_keys(n: int, window: int, keep_first: int, chunk: int = 0) -> torch.Tensor:
     """Positions the last of ``n`` tokens sees."""
     key = torch.arange(n)
+    if chunk > 0:
+        return key[(n - 1) // chunk * chunk :]
     return key[(key >= n - window) | (key < keep_first)] if window > 0 else key
 
 
@@ -417,43 +458,69 @@ def _soft_cap(s: torch.Tensor, cap: float) -> torch.Tensor:
     return cap * torch.tanh(s / cap) if cap > 0 else s
 
 
+def _difference(o: torch.Tensor, diff) -> torch.Tensor:
+    """``o`` [..., 2 H, e] fp32, the two maps of a head behind each other -> [..., H, e]."""
+    vectors, const, eps = diff
+    q1, k1, q2, k2 = vectors.float().chunk(4)
+    lam = torch.exp((q1 * k1).sum()) - torch.exp((q2 * k2).sum()) + const
+    o = o.unflatten(-2, (-1, 2))
+    o = o[..., 0, :] - lam * o[..., 1, :]
+    return o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * (1.0 - const)
+
+
+def _key_heads(heads: int, kv_heads: int, maps: int) -> torch.Tensor:
+    """Key head of every query head; the maps of a head are neighbours."""
+    h = torch.arange(heads)
+    return h // maps // (heads // maps // kv_heads) * maps + h % maps
+
+
 def grouped_attention_prefill(q, k, v, cu_q, cu_k, window: int, scale: float, softcap: float = 0.0, sink=None,
-                              keep_first: int = 0) -> torch.Tensor:
+                              keep_first: int = 0, chunk: int = 0, diff=None) -> torch.Tensor:
     """Causal attention of packed prompts: ``q`` [T, H, d], ``k`` [Tk, G, d], ``v`` [Tk, G, e] (query head h reads key head h // (H / G));
-    scores ``softcap * tanh(q k scale / softcap)``; ``cu_q`` / ``cu_k`` / ``window`` / ``keep_first`` / ``sink`` as in ``latent_attention_prefill``."""
+    scores ``softcap * tanh(q k scale / softcap)``; ``cu_q`` / ``cu_k`` / ``window`` / ``keep_first`` / ``sink`` as in ``latent_attention_prefill``.
+    ``chunk`` > 0: a query sees the keys of its own chunk of that many positions (the first key of every sequence starts a chunk).
+    ``diff = (vectors, const, eps)``: differential attention, ``q`` [T, 2 H, d] and ``k`` [Tk, 2 G, d] hold the two maps of a head behind
+    each other; the outputs a1, a2 become ``(1 - const) rms_norm(a1 - lambda a2)`` without weight, lambda = exp(x1 . x2) - exp(x3 . x4) +
+    const with ``vectors`` = x1 | x2 | x3 | x4."""
     if q.is_cuda:
-        return _ops().grouped_attn_prefill(q, k, v, cu_q, cu_k, sink, int(window), float(scale), float(softcap), int(keep_first))
-    out = torch.empty(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype)
-    n = q.shape[1] // k.shape[1]
+        return _ops().grouped_attn_prefill(q, k, v, cu_q, cu_k, sink, int(window), float(scale), float(softcap), int(keep_first), int(chunk),
+                                           *(diff if diff is not None else (None, 0.0, 0.0)))
+    maps = 1 if diff is None else 2
+    H, G = q.shape[1], v.shape[1]
+    out = torch.empty(q.shape[0], H // maps, v.shape[2], dtype=q.dtype)
+    kh = _key_heads(H, G, maps)
     cq, ck = cu_q.tolist(), cu_k.tolist()
     for b in range(len(cq) - 1):
         qs, ks = slice(cq[b], cq[b + 1]), slice(ck[b], ck[b + 1])
         nq, nk = cq[b + 1] - cq[b], ck[b + 1] - ck[b]
-        s = _soft_cap(torch.einsum("qhd,khd->hqk", q[qs].float(), k[ks].float().repeat_interleave(n, 1)) * scale, softcap)
-        hide = _hidden_keys(nq, nk, window, keep_first)
+        s = _soft_cap(torch.einsum("qhd,khd->hqk", q[qs].float(), k[ks].float()[:, kh]) * scale, softcap)
+        hide = _hidden_keys(nq, nk, window, keep_first, chunk)
         w = _sink_softmax(s.masked_fill(hide, float("-inf")), sink)
-        out[qs] = torch.einsum("hqk,khd->qhd", w, v[ks].float().repeat_interleave(n, 1)).to(q.dtype)
+        o = torch.einsum("hqk,khd->qhd", w, v[ks].float()[:, kh // maps])
+        out[qs] = (o if diff is None else _difference(o, diff)).to(q.dtype)
     return out
 
 
 def grouped_attention_decode(q, pages, block_table, ctx_len, kv_heads: int, vdim: int, window: int, scale: float, softcap: float = 0.0,
-                             sink=None, keep_first: int = 0) -> torch.Tensor:
+                             sink=None, keep_first: int = 0, chunk: int = 0, diff=None) -> torch.Tensor:
     """One query per sequence, ``q`` [S, H, d], against cached rows [keys | values] (``qkv_prep``). Returns [S, H, vdim]; sequences
-    with ``ctx_len`` 0 give zeros."""
+    with ``ctx_len`` 0 give zeros. ``chunk`` and ``diff`` as in ``grouped_attention_prefill``."""
     if q.is_cuda:
         return _ops().grouped_attn_decode(q, pages, block_table, ctx_len, sink, int(kv_heads), int(vdim), int(window), float(scale), float(softcap),
-                                          int(keep_first))
-    out = torch.zeros(q.shape[0], q.shape[1], vdim, dtype=q.dtype)
-    bs, G, d = pages.shape[1], kv_heads, q.shape[2]
+                                          int(keep_first), int(chunk), *(diff if diff is not None else (None, 0.0, 0.0)))
+    maps = 1 if diff is None else 2
+    bs, G, d, H = pages.shape[1], kv_heads, q.shape[2], q.shape[1]
+    out = torch.zeros(q.shape[0], H // maps, vdim, dtype=q.dtype)
+    kh = _key_heads(H, G, maps)
     for b, n in enumerate(ctx_len.tolist()):
         if n <= 0:
             continue
-        at = _seen_keys(n, window, keep_first)
+        at = _seen_keys(n, window, keep_first, chunk)
         rows = pages[block_table[b, at // bs].long(), at % bs].float()
-        k, v = rows[:, : G * d].view(-1, G, d), rows[:, G * d :].view(-1, G, vdim)
-        s = _soft_cap(torch.einsum("gnd,kgd->gnk", q[b].float().view(G, -1, d), k).flatten(0, 1) * scale, softcap)
-        w = _sink_softmax(s, sink)
-        out[b] = torch.einsum("gnk,kge->gne", w.view(G, -1, len(at)), v).flatten(0, 1).to(q.dtype)
+        k, v = rows[:, : G * maps * d].view(-1, G * maps, d), rows[:, G * maps * d :].view(-1, G, vdim)
+        s = _soft_cap(torch.einsum("hd,khd->hk", q[b].float(), k[:, kh]) * scale, softcap)
+        o = torch.einsum("hk,khe->he", _sink_softmax(s, sink), v[:, kh // maps])
+        out[b] = (o if diff is None else _difference(o, diff)).to(q.dtype)
     return out
 
 
@@ -473,46 +540,72 @@ def _conv_portion(u: torch.Tensor, w: torch.Tensor, past: torch.Tensor):
     return sum(row[j : j + u.shape[0]] * w[:, j].float() for j in range(taps)), row[row.shape[0] - taps + 1 :]
 
 
+def _conv_rows(u: torch.Tensor, conv: torch.Tensor, cu, state, slots, fresh, active) -> torch.Tensor:
+    """Causal convolution of the rows ``u`` [T, C] of portions or steps (see ``conv_qkv_prep``); moves the kept inputs on."""
+    (T, C), n = u.shape, conv.shape[1] - 1
+    if n == 0:
+        return u * conv[:, 0].float()
+    f = torch.zeros(T, C)
+    if cu is None:
+        for s in torch.nonzero(active).flatten().tolist():
+            past = state[s].view(n, C)
+            f[s : s + 1], last = _conv_portion(u[s : s + 1], conv, past.clone())
+            past.copy_(last)
+        return f
+    c = cu.tolist()
+    for b in range(len(c) - 1):
+        past = state[int(slots[b])].view(n, C) if slots is not None else None
+        f[c[b] : c[b + 1]], last = _conv_portion(u[c[b] : c[b + 1]], conv, torch.zeros(n, C) if past is None or bool(fresh[b]) else past.clone())
+        if past is not None:
+            past.copy_(last)
+    return f
+
+
 def conv_qkv_prep(p, conv, eps: float, positions, cos, sin, heads: int, kv_heads: int, dim: int, vdim: int, halves: bool = True, cu=None, state=None, slots=None,
-                  fresh=None, active=None, pages=None, page_slots=None, want_rows: bool = False):
+                  fresh=None, active=None, pages=None, page_slots=None, want_rows: bool = False, norm: bool = True, v_heads: Optional[int] = None):
     """``p`` [T, q | k | v]: causal convolution over time (``conv`` [channels, taps], None: none; zeros before a sequence's first
     token), rotation of the first ``2 * cos.shape[1]`` dimensions of every query and key head (pairs (i, i + half), or (2i, 2i + 1)
-    without ``halves``), then an RMS norm without weight over the head. Portions (``cu`` given): sequence b goes on from the inputs in
+    without ``halves``), then with ``norm`` an RMS norm without weight over the head. There are ``kv_heads`` key heads (0: queries only) and
+    ``v_heads`` value heads (default: as many). Portions (``cu`` given): sequence b goes on from the inputs in
     ``state[slots[b]]`` unless ``fresh[b]``, and leaves its last ones there; without ``slots`` every sequence starts from zeros and
     nothing is kept. Steps (``cu`` None): row s is the next token of ``state[s]`` where ``active[s]``. ``state`` rows: [taps - 1, channels]
     fp32, oldest first. Returns (queries [T, heads, dim], rows [keys | values]) as ``qkv_prep``."""
+    v_heads = kv_heads if v_heads is None else v_heads
     if p.is_cuda:
-        return _ops().conv_qkv_prep(p, conv, float(eps), positions, cos, sin, int(heads), int(kv_heads), int(dim), int(vdim), bool(halves), cu, state, slots,
-                                    fresh, active, pages, page_slots, bool(want_rows))
-    T, C = p.shape[0], (heads + kv_heads) * dim + kv_heads * vdim
+        return _ops().conv_qkv_prep(p, conv, float(eps), positions, cos, sin, int(heads), int(kv_heads), int(v_heads), int(dim), int(vdim), bool(halves), bool(norm),
+                                    cu, state, slots, fresh, active, pages, page_slots, bool(want_rows))
+    T, C = p.shape[0], (heads + kv_heads) * dim + v_heads * vdim
     f = p[:, :C].float()
-    if conv is not None and conv.shape[1] > 1:
-        n, u, f = conv.shape[1] - 1, f, torch.zeros(T, C)
-        if cu is None:
-            for s in torch.nonzero(active).flatten().tolist():
-                past = state[s].view(n, C)
-                f[s : s + 1], last = _conv_portion(u[s : s + 1], conv, past.clone())
-                past.copy_(last)
-        else:
-            c = cu.tolist()
-            for b in range(len(c) - 1):
-                past = state[int(slots[b])].view(n, C) if slots is not None else None
-                f[c[b] : c[b + 1]], last = _conv_portion(u[c[b] : c[b + 1]], conv, torch.zeros(n, C) if past is None or bool(fresh[b]) else past.clone())
-                if past is not None:
-                    past.copy_(last)
-    elif conv is not None:
-        f = f * conv[:, 0].float()
+    if conv is not None:
+        f = _conv_rows(f, conv, cu, state, slots, fresh, active)
     a, b = heads * dim, (heads + kv_heads) * dim
     turn = _rotate_halves if halves else _rotate
-    unit = lambda z: z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps)
+    unit = lambda z: z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) if norm else z
     q = unit(turn(f[:, :a].view(T, heads, dim), positions, cos, sin)).to(p.dtype)
     k = unit(turn(f[:, a:b].view(T, kv_heads, dim), positions, cos, sin))
     row = torch.cat([k.flatten(1), f[:, b:]], -1).to(p.dtype)
-    if pages is not None:
-        ok = page_slots >= 0
-        at, bs = page_slots[ok], pages.shape[1]
-        pages[at // bs, at % bs] = row[ok]
+    _append(pages, page_slots, row)
     return q, (row if want_rows else row[:0])
+
+
+def _append(pages, slots, row) -> None:
+    if pages is not None:
+        ok = slots >= 0
+        at, bs = slots[ok], pages.shape[1]
+        pages[at // bs, at % bs] = row[ok]
+
+
+def whole_norm_prep(p, q_norm, k_norm, temp, eps: float, heads: int, kv_heads: int, vdim: int, pages=None, slots=None, want_rows: bool = False):
+    """``p`` [T, q | k | v]: weighted RMS norms over all query and over all key columns, queries times their head's ``temp``. Returns
+    (queries [T, heads, dim], rows [keys | values]) and appends the rows as ``qkv_prep`` does."""
+    if p.is_cuda:
+        return _ops().whole_norm_prep(p, q_norm, k_norm, temp, float(eps), int(heads), int(kv_heads), int(vdim), pages, slots, bool(want_rows))
+    a, b = q_norm.numel(), q_norm.numel() + k_norm.numel()
+    f = p.float()
+    q = _rms(f[:, :a], q_norm, eps).view(-1, heads, a // heads) * temp.float()[:, None]
+    row = torch.cat([_rms(f[:, a:b], k_norm, eps), f[:, b : b + kv_heads * vdim]], -1).to(p.dtype)
+    _append(pages, slots, row)
+    return q.to(p.dtype), (row if want_rows else row[:0])
 
 
 # ----------------------------------------------------------------------------------------------- lightning recurrence
@@ -557,11 +650,65 @@ def lightning_decode(p, decay, dim: int, vdim: int, state, active) -> torch.Tens
     return out.flatten(1).to(p.dtype)
 
 
-def gated_rms(o: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, eps: float) -> torch.Tensor:
-    """``rms_norm(o) * norm * sigmoid(gate)`` over whole rows."""
+def gated_rms(o: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, eps: float, heads: int = 1) -> torch.Tensor:
+    """``rms_norm(o) * norm * sigmoid(gate)``; the norm's statistics span whole rows, or each of ``heads`` equal parts."""
     if o.is_cuda:
-        return _ops().gated_rms(o, gate, norm, float(eps))
-    return (_rms(o.float(), norm, eps) * torch.sigmoid(gate.float())).to(norm.dtype)
+        return _ops().gated_rms(o, gate, norm, float(eps), int(heads))
+    n = o.float().unflatten(-1, (heads, -1))
+    n = (n * torch.rsqrt(n.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2)
+    return (n * norm.float() * torch.sigmoid(gate.float())).to(norm.dtype)
+
+
+# ----------------------------------------------------------------------------------------------- generalized delta rule
+def _delta_parts(p, zw, ab, w0, heads: int):
+    """(r, k, v, decay, removal rate) [T, heads, dim] and the unit keys, fp32."""
+    n = ab.numel()
+    f = lambda z: z.float().view(-1, heads, n // heads)
+    r, k, v, za = (f(p[:, i * n : (i + 1) * n]) for i in range(4))
+    w = torch.exp(-math.exp(-0.5) * torch.sigmoid(f(zw[:, :n]) + f(w0)))
+    return r, k, v, w, torch.sigmoid(za + f(ab)), k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+
+
+def _delta_token(S, r, k, v, w, a, u):
+    """One token of one sequence, in place on S [H, d, d]; returns o [H, d]."""
+    held = torch.einsum("hd,hde->he", u, S)
+    S.mul_(w[:, :, None]).sub_((a * u)[:, :, None] * held[:, None, :]).add_(k[:, :, None] * v[:, None, :])
+    return torch.einsum("hde,hd->he", S, r)
+
+
+def delta_prefill(p, zw, ab, w0, heads: int, cu, state=None, slots=None, fresh=None) -> torch.Tensor:
+    """Generalized delta rule over packed portions: ``p`` [T, r | k | v | za | ...], ``zw`` [T, heads * dim], per head and key channel the decay
+    ``w = exp(-exp(-1/2) sigmoid(zw + w0))`` and the removal rate ``a = sigmoid(za + ab)``; with the unit key u, ``S = diag(w) S - (a u)
+    (u^T S) + k v^T``, ``o = S^T r``. ``cu`` / ``state`` / ``slots`` / ``fresh`` as in ``mlstm_prefill`` with state rows [heads, dim, dim]. Returns
+    [T, heads * dim]."""
+    if p.is_cuda:
+        return _ops().delta_prefill(p, zw, ab, w0, int(heads), cu, state, slots, fresh)
+    n = ab.numel()
+    d = n // heads
+    parts = _delta_parts(p, zw, ab, w0, heads)
+    out = torch.empty(p.shape[0], heads, d)
+    c = cu.tolist()
+    for b in range(len(c) - 1):
+        S = torch.zeros(heads, d, d) if slots is None else state[int(slots[b])].view(heads, d, d)
+        if slots is not None and bool(fresh[b]):
+            S.zero_()
+        for t in range(c[b], c[b + 1]):
+            out[t] = _delta_token(S, *(z[t] for z in parts))
+    return out.flatten(1).to(p.dtype)
+
+
+def delta_decode(p, zw, ab, w0, heads: int, norm, eps: float, state, active) -> torch.Tensor:
+    """One token per slot: row s of ``p`` [S, r | k | v | za | g | ...] updates ``state[s]`` when ``active[s]`` (inactive slots keep theirs and give
+    zeros). Returns the finished rows: per head ``rms_norm(o)``, times ``norm``, times ``sigmoid(g)``."""
+    if p.is_cuda:
+        return _ops().delta_decode(p, zw, ab, w0, int(heads), norm, float(eps), state, active)
+    n = ab.numel()
+    d = n // heads
+    parts = _delta_parts(p, zw, ab, w0, heads)
+    out = torch.zeros(p.shape[0], heads, d)
+    for s in torch.nonzero(active).flatten().tolist():
+        out[s] = _delta_token(state[s].view(heads, d, d), *(z[s] for z in parts))
+    return gated_rms(out.flatten(1), p[:, 4 * n : 5 * n], norm, eps, heads)
 
 
 # ----------------------------------------------------------------------------------------------- mLSTM

@@ -13,7 +13,7 @@ from typing import Iterable
 
 import torch
 
-__all__ = ["load_hf_weights_into", "save_hf_weights", "compute_position_id_with_mask", "print_model_size",
+__all__ = ["load_hf_weights_into", "tensor_shape", "save_hf_weights", "compute_position_id_with_mask", "print_model_size",
            "get_model_size", "update_model_config", "load_valuehead_model"]
 
 
@@ -34,6 +34,20 @@ def _iter_hf_tensors(path: str) -> Iterable[tuple[str, torch.Tensor]]:
     for f in sorted(glob.glob(os.path.join(path, "pytorch_model*.bin"))) + sorted(glob.glob(os.path.join(path, "*.pt"))):
         sd = torch.load(f, map_location="cpu", weights_only=True)
         yield from sd.items()
+
+
+def tensor_shape(path: str, name: str) -> tuple:
+    """Shape of a stored tensor (safetensors: from the header alone)."""
+    from safetensors import safe_open
+
+    for f in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(f, framework="pt", device="cpu") as sf:
+            if name in sf.keys():
+                return tuple(sf.get_slice(name).get_shape())
+    for k, t in _iter_hf_tensors(path):
+        if k == name:
+            return tuple(t.shape)
+    raise KeyError(f"no tensor {name} in {path}")
 
 
 def load_hf_weights_into(params, path: str, strict: bool = False) -> list[str]:

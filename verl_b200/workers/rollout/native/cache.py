@@ -2,13 +2,15 @@
 
 * :class:`DenseKVCache`: keys and values of a uniform decoder, one pool ``[layers, 2, blocks, block_size, kv_heads, head_dim]``.
 * :class:`StackCache`: mixer stacks. Attention layers that cache a row per token share a page pool (a block holds the rows of
-  all such layers for ``block_size`` tokens); recurrent layers own a part of one fp32 state row per sequence slot.
+  all such layers for ``block_size`` tokens); recurrent layers and convolutions own parts of one fp32 state row per sequence slot.
 
 A sequence is its block list plus its slot; ``copy_blocks`` / ``copy_slots`` duplicate them (samples of one prompt) and
 ``export`` / ``install`` move them between engines (prefill / decode disaggregation).
 """
 
 from __future__ import annotations
+
+from typing import Optional
 
 import torch
 
@@ -53,15 +55,17 @@ class StackCache:
         self.dtype, self.device, self.bs = dtype, device, block_size
         # element offsets of every layer inside a block (rows of the layer's tokens are contiguous) and inside a state row
         self._page_off, self._page_w, self._state_off, self._state_n = {}, {}, {}, {}
+        past = max(cfg.stack.input_conv - 1, 0) * cfg.hidden_size
         off = st = 0
         for i, l in enumerate(cfg.stack.layers):
             w, n = l.mixer.page_width, l.mixer.state_size
             if w:
                 self._page_off[i], self._page_w[i] = off, w
                 off += -(-block_size * w // 8) * 8      # 16-byte aligned starts
-            if n:
-                self._state_off[i], self._state_n[i] = st, n
-                st += -(-n // 4) * 4
+            for key, n in ((i, n), ((i, "input"), past)):
+                if n:
+                    self._state_off[key], self._state_n[key] = st, n
+                    st += -(-n // 4) * 4
         self.block_elems, self.state_elems = max(off, 8), st
         self.has_state = st > 0
         self.num_slots = num_slots
@@ -85,8 +89,15 @@ class StackCache:
 
     def state(self, layer: int) -> torch.Tensor:
         """[slots, size] view of a recurrent layer's state."""
-        o = self._state_off[layer]
-        return self.states[:, o : o + self._state_n[layer]]
+        return self._state_view(layer)
+
+    def input_state(self, layer: int) -> Optional[torch.Tensor]:
+        """[slots, (taps - 1) width] view of what the convolution of a layer's input keeps (None: it keeps nothing)."""
+        return self._state_view((layer, "input")) if (layer, "input") in self._state_off else None
+
+    def _state_view(self, key) -> torch.Tensor:
+        o = self._state_off[key]
+        return self.states[:, o : o + self._state_n[key]]
 
     def copy_blocks(self, dst: torch.Tensor, src: torch.Tensor) -> None:
         self.kv[dst] = self.kv[src]
