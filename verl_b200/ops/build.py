@@ -37,7 +37,8 @@ NVCC_FLAGS = [
 
 # sources whose transcendental functions, divisions and square roots keep full fp32 accuracy
 PRECISE_MATH = ("gemm_simt", "mixer_kernels", "latent_attention_simt", "mlstm_chunk", "latent_decode", "headwise_mma",
-                "stack_rows", "experts", "grouped_decode", "conv_prep", "lightning", "lightning_chunk", "lightning_tcgen05")
+                "stack_rows", "experts", "grouped_decode", "conv_prep", "lightning", "lightning_chunk", "lightning_tcgen05",
+                "rms_conv", "delta_rule", "delta_chunk")
 
 
 def _nvcc_flags(stem: str) -> list:

@@ -73,14 +73,24 @@ std::tuple<Tensor, Tensor> linear_split(const Tensor& a, const Tensor& w, int64_
   return {d, d2};
 }
 
-Tensor linear_bias(const Tensor& a, const Tensor& w, const Tensor& b) {
+Tensor linear_bias(const Tensor& a, const Tensor& w, const Tensor& b, bool relu2) {
   const c10::cuda::CUDAGuard guard(a.device());
   same(a, b, "linear_bias");
   TORCH_CHECK(b.numel() == w.size(0) && b.is_contiguous(), "linear_bias: bias [N]");
   Tensor d = at::empty({a.size(0), w.size(0)}, a.options());
   VbEpiArgs e{};
-  e.mode = VB_EPI_BIAS;
+  e.mode = relu2 ? VB_EPI_BIAS_RELU2 : VB_EPI_BIAS;
   e.D = d.data_ptr(); e.ldd = d.stride(0); e.nb = b.data_ptr();
+  run_gemm(a, w, e);
+  return d;
+}
+
+Tensor linear_tanh(const Tensor& a, const Tensor& w, int64_t n0) {
+  const c10::cuda::CUDAGuard guard(a.device());
+  Tensor d = at::empty({a.size(0), w.size(0)}, a.options());
+  VbEpiArgs e{};
+  e.mode = VB_EPI_TANH;
+  e.D = d.data_ptr(); e.ldd = d.stride(0); e.n0 = (int)n0;
   run_gemm(a, w, e);
   return d;
 }
@@ -95,10 +105,10 @@ Tensor linear_silu(const Tensor& a, const Tensor& w, int64_t n0) {
   return d;
 }
 
-// x += a w^T, or x += tanh(palpha a w^T) pw + pb (fp32 residual stream); returns tanh(alpha x) nw + nb in a's type, or an empty tensor
+// x += a w^T (+ bias), or x += tanh(palpha a w^T) pw + pb (fp32 residual stream); returns tanh(alpha x) nw + nb in a's type, or an empty tensor
 // without a norm.
 Tensor linear_residual_(const Tensor& a, const Tensor& w, Tensor x, const OptTensor& alpha, const OptTensor& nw, const OptTensor& nb, const OptTensor& palpha,
-                        const OptTensor& pw, const OptTensor& pb) {
+                        const OptTensor& pw, const OptTensor& pb, const OptTensor& bias) {
   const c10::cuda::CUDAGuard guard(a.device());
   CHECK_F32(x);
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && x.size(0) == a.size(0) && x.size(1) == w.size(0), "linear_residual_: x [M, N]");
@@ -122,6 +132,11 @@ Tensor linear_residual_(const Tensor& a, const Tensor& w, Tensor x, const OptTen
     same(a, *palpha, "linear_residual_");
     TORCH_CHECK(pw->numel() == w.size(0) && pb->numel() == w.size(0) && palpha->numel() == 1, "linear_residual_: norm sizes");
     e.palpha = palpha->data_ptr(); e.pw = pw->data_ptr(); e.pb = pb->data_ptr();
+  }
+  if (bias.has_value()) {
+    same(a, *bias, "linear_residual_");
+    TORCH_CHECK(!pw.has_value() && bias->numel() == w.size(0) && bias->is_contiguous(), "linear_residual_: bias [N]");
+    e.pb = bias->data_ptr();
   }
   run_gemm(a, w, e);
   return h;
@@ -177,17 +192,18 @@ Tensor residual_dyt_(Tensor x, const Tensor& rows, const Tensor& slot, const Ten
   return h;
 }
 
-// rms_norm(o) norm sigmoid(g) over whole rows (strided views).
-Tensor gated_rms(const Tensor& o, const Tensor& g, const Tensor& norm, double eps) {
+// rms_norm(o) norm sigmoid(g) over whole rows or each of `heads` parts (strided views).
+Tensor gated_rms(const Tensor& o, const Tensor& g, const Tensor& norm, double eps, int64_t heads) {
   const int dt = dtype_of(o);
   same(o, g, "gated_rms");
   same(o, norm, "gated_rms");
-  TORCH_CHECK(o.dim() == 2 && g.sizes() == o.sizes() && o.stride(1) == 1 && g.stride(1) == 1 && norm.numel() == o.size(1), "gated_rms: [T, W]");
+  TORCH_CHECK(o.dim() == 2 && g.sizes() == o.sizes() && o.stride(1) == 1 && g.stride(1) == 1 && norm.numel() == o.size(1) && heads >= 1 &&
+              o.size(1) % heads == 0, "gated_rms: [T, W]");
   const c10::cuda::CUDAGuard guard(o.device());
   Tensor out = at::empty(o.sizes(), o.options());
   verl_count_launches(1);
   CHECK_RC(vb_gated_rms(dt, o.data_ptr(), o.stride(0), g.data_ptr(), g.stride(0), norm.data_ptr(), (float)eps, out.data_ptr(), (int)o.size(0), (int)o.size(1),
-                        cur_stream()), "vb_gated_rms");
+                        (int)heads, cur_stream()), "vb_gated_rms");
   return out;
 }
 
@@ -335,7 +351,7 @@ Tensor latent_attn_prefill(const Tensor& q, const Tensor& ku, const Tensor& kr, 
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   verl_count_launches(1);
   int rc = dt == 1 && a.T > 0 ? vb_latent_prefill(&a, (int)ku.size(0), cur_stream()) : -1;
-  if (rc < 0) rc = vb_latent_attn_simt(dt, &a, cur_stream());
+  if (rc < 0) rc = vb_latent_attn_simt(dt, &a, 0, cur_stream());
   CHECK_RC(rc, "latent_attn_prefill");
   return out;
 }
@@ -381,7 +397,7 @@ Tensor latent_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& bl
     }
   }
   verl_count_launches(1);
-  CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
+  CHECK_RC(vb_latent_attn_simt(dt, &a, 0, cur_stream()), "vb_latent_attn_simt");
   return out;
 }
 
@@ -594,61 +610,103 @@ std::tuple<Tensor, Tensor> qkv_prep(const Tensor& p, const Tensor& qn, const Ten
   return {q, rows};
 }
 
-// Prompt attention: q [T, H, d], k [Tk, G, d], v [Tk, G, e] (strided views), cu_q / cu_k int32 [B + 1].
+// Differential attention over q [*, 2 H, d]: arguments of the difference; `out` [T, H, e].
+void diff_args(VbLatentAttn& a, const Tensor& q, const OptTensor& vec, double diff, double eps) {
+  a.maps = vec.has_value() ? 2 : 1;
+  if (!vec.has_value()) return;
+  same(q, *vec, "differential attention");
+  TORCH_CHECK(q.size(1) % 2 == 0 && vec->is_contiguous() && vec->numel() == 4 * q.size(2), "differential attention: four vectors of a map's size");
+  a.diff_vec = vec->data_ptr(); a.diff = (float)diff; a.eps = (float)eps;
+}
+// The difference behind an attention kernel that leaves the maps apart.
+void diff_simt(int dt, VbLatentAttn a, const Tensor& q, const Tensor& out) {
+  Tensor maps = at::empty({a.T, a.H, a.dv}, q.options().dtype(at::kFloat));
+  a.out = maps.data_ptr(); a.ldo = maps.stride(0);
+  verl_count_launches(2);
+  CHECK_RC(vb_latent_attn_simt(dt, &a, 1, cur_stream()), "vb_latent_attn_simt");
+  CHECK_RC(vb_diff_combine(dt, maps.data_ptr(), 1, a.diff_vec, a.du, a.diff, a.eps, out.data_ptr(), a.T, a.H / 2, a.dv, cur_stream()), "vb_diff_combine");
+}
+
+// Prompt attention: q [T, H, d], k [Tk, G, d], v [Tk, G, e] (strided views), cu_q / cu_k int32 [B + 1]; with `vec` q [T, 2 H, d], k [Tk, 2 G, d].
 Tensor grouped_attn_prefill(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& cu_q, const Tensor& cu_k, const OptTensor& sink, int64_t window,
-                            double scale, double softcap, int64_t keep_first) {
+                            double scale, double softcap, int64_t keep_first, int64_t chunk, const OptTensor& vec, double diff, double eps) {
   const int dt = dtype_of(q);
   CHECK_I32(cu_q);
   CHECK_I32(cu_k);
   same(q, k, "grouped_attn_prefill");
   same(q, v, "grouped_attn_prefill");
   TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.stride(2) == 1 && k.stride(2) == 1 && v.stride(2) == 1 && q.size(2) == k.size(2) && k.size(1) > 0 &&
-              q.size(1) % k.size(1) == 0 && v.size(1) == k.size(1) && v.size(0) == k.size(0) && cu_q.numel() == cu_k.numel(), "grouped_attn_prefill");
+              q.size(1) % k.size(1) == 0 && v.size(1) * (vec.has_value() ? 2 : 1) == k.size(1) && v.size(0) == k.size(0) && cu_q.numel() == cu_k.numel() &&
+              !(chunk > 0 && window > 0), "grouped_attn_prefill");
   const c10::cuda::CUDAGuard guard(q.device());
   VbLatentAttn a{};
+  diff_args(a, q, vec, diff, eps);
+  a.chunk = (int)chunk;
   a.q = q.data_ptr(); a.ldq = q.stride(0); a.hq = (int)q.stride(1);
   a.ku = k.data_ptr(); a.ku_row = k.stride(0); a.ku_head = (int)k.stride(1);
   a.v = v.data_ptr(); a.v_row = v.stride(0); a.v_head = (int)v.stride(1);
   a.cu_q = cu_q.data_ptr<int>(); a.cu_k = cu_k.data_ptr<int>();
   a.T = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)q.size(2); a.dv = (int)v.size(2); a.B = (int)cu_q.numel() - 1;
-  a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / k.size(1));
+  a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / k.size(1));   // query heads per key / value head, maps not counted
   if (sink.has_value()) { same(q, *sink, "grouped_attn_prefill"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
-  Tensor out = at::empty({q.size(0), q.size(1), v.size(2)}, q.options());
+  Tensor out = at::empty({q.size(0), q.size(1) / a.maps, v.size(2)}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
-  verl_count_launches(1);
   int rc = dt == 1 && a.T > 0 ? vb_latent_prefill(&a, (int)k.size(0), cur_stream()) : -1;
-  if (rc < 0) rc = vb_latent_attn_simt(dt, &a, cur_stream());
+  if (rc >= 0) verl_count_launches(1);
+  if (rc < 0 && a.maps > 1) {
+    // values too wide for both maps' products at once: the maps as heads of their own over the values of their pair
+    if (dt == 1 && a.T > 0) {
+      VbLatentAttn m = a;
+      Tensor both = at::empty({a.T, a.H, a.dv}, q.options());
+      m.maps = 1; m.kv_group = a.kv_group; m.split_maps = 1; m.out = both.data_ptr(); m.ldo = both.stride(0);
+      rc = vb_latent_prefill(&m, (int)k.size(0), cur_stream());
+      if (rc == 0) {
+        verl_count_launches(2);
+        CHECK_RC(vb_diff_combine(dt, both.data_ptr(), 0, a.diff_vec, a.du, a.diff, a.eps, out.data_ptr(), a.T, a.H / 2, a.dv, cur_stream()), "vb_diff_combine");
+        return out;
+      }
+    }
+    if (rc < 0) {
+      diff_simt(dt, a, q, out);
+      return out;
+    }
+  }
+  if (rc < 0) verl_count_launches(1);
+  if (rc < 0) rc = vb_latent_attn_simt(dt, &a, 0, cur_stream());
   CHECK_RC(rc, "grouped_attn_prefill");
   return out;
 }
 
 // Decode attention: q [S, H, d], pages [blocks, block_size, G (d + vdim)] with rows [keys | values].
 Tensor grouped_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& block_table, const Tensor& ctx_len, const OptTensor& sink, int64_t G, int64_t vdim,
-                           int64_t window, double scale, double softcap, int64_t keep_first) {
+                           int64_t window, double scale, double softcap, int64_t keep_first, int64_t chunk, const OptTensor& vec, double diff, double eps) {
   const int dt = dtype_of(q);
+  const int64_t maps = vec.has_value() ? 2 : 1;
   same(q, pages, "grouped_attn_decode");
   CHECK_I32(block_table);
   CHECK_I32(ctx_len);
-  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && pages.dim() == 3 && pages.stride(2) == 1 && G > 0 && q.size(1) % G == 0 && pages.size(2) == G * (q.size(2) + vdim) &&
-              block_table.size(0) == q.size(0) && ctx_len.numel() == q.size(0), "grouped_attn_decode");
+  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && pages.dim() == 3 && pages.stride(2) == 1 && G > 0 && q.size(1) % (G * maps) == 0 &&
+              pages.size(2) == G * (maps * q.size(2) + vdim) && block_table.size(0) == q.size(0) && ctx_len.numel() == q.size(0) && !(chunk > 0 && window > 0), "grouped_attn_decode");
   const c10::cuda::CUDAGuard guard(q.device());
   VbLatentAttn a{};
+  diff_args(a, q, vec, diff, eps);
+  a.chunk = (int)chunk;
   const int64_t d = q.size(2);
   a.q = q.data_ptr(); a.ldq = q.stride(0); a.hq = (int)q.stride(1);
   char* base = reinterpret_cast<char*>(pages.data_ptr());
   a.ku = base; a.ku_row = pages.stride(1); a.ku_head = (int)d;
   a.kr = base;
-  a.v = base + G * d * pages.element_size(); a.v_row = pages.stride(1); a.v_head = (int)vdim;
+  a.v = base + G * maps * d * pages.element_size(); a.v_row = pages.stride(1); a.v_head = (int)vdim;
   a.block_table = block_table.data_ptr<int>(); a.max_blocks = (int)block_table.size(1); a.block_size = (int)pages.size(1); a.page_stride = pages.stride(0);
   a.ctx_len = ctx_len.data_ptr<int>();
   a.T = a.B = (int)q.size(0); a.H = (int)q.size(1); a.du = (int)d; a.dv = (int)vdim;
-  a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / G);
+  a.window = (int)window; a.keep_first = (int)keep_first; a.scale = (float)scale; a.softcap = (float)softcap; a.kv_group = (int)(q.size(1) / (G * maps));
   if (sink.has_value()) { same(q, *sink, "grouped_attn_decode"); TORCH_CHECK(sink->numel() == a.H); a.sink = sink->data_ptr(); }
-  Tensor out = at::empty({q.size(0), q.size(1), vdim}, q.options());
+  Tensor out = at::empty({q.size(0), q.size(1) / maps, vdim}, q.options());
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   if (dt == 1) {
     const int64_t all = (int64_t)a.max_blocks * a.block_size;
-    const int ns = vb_grouped_decode_splits(&a, (int)(window > 0 ? std::min<int64_t>(window + keep_first + 128, all) : all));
+    const int ns = vb_grouped_decode_splits(&a, (int)(window > 0 ? std::min<int64_t>(window + keep_first + 128, all) : chunk > 0 ? std::min<int64_t>(chunk + 64, all) : all));
     if (ns > 0) {
       Tensor po, ml;
       if (ns > 1) {
@@ -663,21 +721,163 @@ Tensor grouped_attn_decode(const Tensor& q, const Tensor& pages, const Tensor& b
       }
     }
   }
+  if (maps > 1) {
+    diff_simt(dt, a, q, out);
+    return out;
+  }
   verl_count_launches(1);
-  CHECK_RC(vb_latent_attn_simt(dt, &a, cur_stream()), "vb_latent_attn_simt");
+  CHECK_RC(vb_latent_attn_simt(dt, &a, 0, cur_stream()), "vb_latent_attn_simt");
   return out;
 }
 
-// p [T, q | k | v]; see VbConvPrep. cu given: portions, else one token per slot. Returns (queries [T, H, dim], rows [T or 0, G (dim + vdim)]).
+// p [T, q | k | v]; see VbWholeNorm. Returns (queries [T, H, dim], rows [T or 0, G (dim + vdim)]).
+std::tuple<Tensor, Tensor> whole_norm_prep(const Tensor& p, const Tensor& qn, const Tensor& kn, const Tensor& temp, double eps, int64_t H, int64_t G, int64_t vdim,
+                                           const OptTensor& pages, const OptTensor& slot, bool want_rows) {
+  const int dt = dtype_of(p);
+  for (const Tensor* t : {&qn, &kn, &temp}) same(p, *t, "whole_norm_prep");
+  const int64_t T = p.size(0), dim = qn.numel() / H, width = G * (dim + vdim);
+  TORCH_CHECK(p.dim() == 2 && p.stride(1) == 1 && qn.numel() == H * dim && kn.numel() == G * dim && temp.numel() == H && p.size(1) >= (H + G) * dim + G * vdim, "whole_norm_prep: sizes");
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor q = at::empty({T, H, dim}, p.options()), rows = at::empty({want_rows ? T : 0, width}, p.options());
+  VbWholeNorm a{};
+  a.p = p.data_ptr(); a.ldp = p.stride(0); a.qn = qn.data_ptr(); a.kn = kn.data_ptr(); a.temp = temp.data_ptr(); a.q = q.data_ptr(); a.ldr = width;
+  if (want_rows) a.rows = rows.data_ptr();
+  a.block_size = 1;
+  if (pages.has_value()) {
+    same(p, *pages, "whole_norm_prep");
+    TORCH_CHECK(pages->dim() == 3 && pages->size(2) == width && pages->stride(2) == 1 && pages->stride(1) == width && slot.has_value() && slot->is_cuda() &&
+                slot->scalar_type() == at::kLong && slot->is_contiguous() && slot->numel() == T, "whole_norm_prep: pages [blocks, block_size, kv_heads (dim + vdim)]");
+    a.pages = pages->data_ptr(); a.page_stride = pages->stride(0); a.block_size = (int)pages->size(1); a.num_slots = pages->size(0) * pages->size(1); a.page_slot = lptr(*slot);
+  }
+  a.T = (int)T; a.H = (int)H; a.G = (int)G; a.dim = (int)dim; a.vdim = (int)vdim; a.eps = (float)eps;
+  verl_count_launches(1);
+  CHECK_RC(vb_whole_norm(dt, &a, cur_stream()), "vb_whole_norm");
+  return {q, rows};
+}
+
+Tensor embed_rows(const Tensor& ids, const Tensor& w, double scale) {
+  const int dt = dtype_of(w);
+  const c10::cuda::CUDAGuard guard(w.device());
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && w.dim() == 2 && w.is_contiguous(), "embed_rows");
+  Tensor x = at::empty({ids.numel(), w.size(1)}, w.options().dtype(at::kFloat));
+  verl_count_launches(1);
+  CHECK_RC(vb_embed_rows(dt, lptr(ids), w.data_ptr(), (float)scale, x.data_ptr<float>(), (int)ids.numel(), (int)w.size(1), (int)w.size(0), cur_stream()), "vb_embed_rows");
+  return x;
+}
+
+// See VbRmsConv: cu given: portions, else one token per row.
+Tensor rms_conv(Tensor x, const OptTensor& y, const OptTensor& bias, const Tensor& nw, double eps, const OptTensor& conv, const OptTensor& cu, const OptTensor& state,
+                const OptTensor& slots, const OptTensor& fresh, const OptTensor& active) {
+  CHECK_F32(x);
+  const int dt = dtype_of(nw);
+  const c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && nw.numel() == x.size(1) && nw.is_contiguous(), "rms_conv: x [T, W]");
+  VbRmsConv a{};
+  a.T = (int)x.size(0); a.W = (int)x.size(1); a.x = x.data_ptr<float>(); a.nw = nw.data_ptr(); a.eps = (float)eps; a.taps = 1;
+  if (y.has_value()) {
+    const bool parts = y->dim() == 3;
+    TORCH_CHECK(y->is_cuda() && y->size(-1) == a.W && y->size(-2) == a.T && y->stride(-1) == 1, "rms_conv: y");
+    if (parts) { CHECK_F32(*y); } else { same(nw, *y, "rms_conv"); }
+    a.y = y->data_ptr(); a.y_f32 = parts; a.splits = parts ? (int)y->size(0) : 1; a.split_stride = parts ? y->stride(0) : 0; a.ldy = y->stride(-2);
+  }
+  if (bias.has_value()) { same(nw, *bias, "rms_conv"); TORCH_CHECK(bias->numel() == a.W && bias->is_contiguous(), "rms_conv: bias [W]"); a.bias = bias->data_ptr(); }
+  if (conv.has_value()) {
+    same(nw, *conv, "rms_conv");
+    TORCH_CHECK(conv->dim() == 2 && conv->size(0) == a.W && conv->size(1) >= 1 && conv->is_contiguous(), "rms_conv: conv [W, taps]");
+    a.conv = conv->data_ptr(); a.taps = (int)conv->size(1);
+    if (state.has_value() && a.taps > 1) {
+      CHECK_F32(*state);
+      TORCH_CHECK(state->dim() == 2 && state->stride(1) == 1 && state->size(1) == (int64_t)(a.taps - 1) * a.W, "rms_conv: state [slots, (taps - 1) W]");
+      a.state = state->data_ptr<float>(); a.slot_stride = state->stride(0);
+    }
+    if (cu.has_value()) {
+      CHECK_I32(*cu);
+      TORCH_CHECK(!y.has_value() && !bias.has_value(), "rms_conv: portions take the stream as it is");
+      a.cu = cu->data_ptr<int>(); a.B = (int)cu->numel() - 1;
+      if (a.state != nullptr) {
+        TORCH_CHECK(slots.has_value() && fresh.has_value() && slots->numel() == a.B && fresh->numel() == a.B, "rms_conv: slots and fresh [B]");
+        CHECK_I32(*slots);
+        CHECK_I32(*fresh);
+        a.slots = slots->data_ptr<int>(); a.fresh = fresh->data_ptr<int>();
+      }
+    } else {
+      TORCH_CHECK(active.has_value() && active->is_cuda() && active->scalar_type() == at::kBool && active->is_contiguous() && active->numel() == a.T, "rms_conv: active [S]");
+      TORCH_CHECK(a.taps == 1 || (a.state != nullptr && state->size(0) >= a.T), "rms_conv: steps need a state");
+      a.active = reinterpret_cast<const uint8_t*>(active->data_ptr());
+    }
+  }
+  Tensor h = at::empty({a.T, a.W}, nw.options());
+  a.h = h.data_ptr();
+  verl_count_launches(a.cu != nullptr && a.state != nullptr ? 2 : 1);
+  CHECK_RC(vb_rms_conv(dt, &a, cur_stream()), "vb_rms_conv");
+  return h;
+}
+
+// p [T, r | k | v | za | g | ...], zw [T, H d]
+VbDelta delta_args(const Tensor& p, const Tensor& zw, const Tensor& ab, const Tensor& w0, int64_t H, const OptTensor& state, Tensor& out) {
+  for (const Tensor* t : {&zw, &ab, &w0}) same(p, *t, "delta");
+  const int64_t W = ab.numel(), d = W / H;
+  TORCH_CHECK(H > 0 && W == H * d && w0.numel() == W && ab.is_contiguous() && w0.is_contiguous() && p.dim() == 2 && p.stride(1) == 1 && p.size(1) >= 5 * W && zw.dim() == 2 &&
+              zw.stride(1) == 1 && zw.size(0) == p.size(0) && zw.size(1) >= W, "delta: rows [r | k | v | a | g]");
+  VbDelta a{};
+  if (state.has_value()) {
+    CHECK_F32(*state);
+    TORCH_CHECK(state->dim() == 2 && state->stride(1) == 1 && state->size(1) == W * d, "delta: state [slots, H d d]");
+    a.state = state->data_ptr<float>(); a.slot_stride = state->stride(0);
+  }
+  out = at::empty({p.size(0), W}, p.options());
+  a.p = p.data_ptr(); a.ldp = p.stride(0); a.zw = zw.data_ptr(); a.ldz = zw.stride(0); a.ab = ab.data_ptr(); a.w0 = w0.data_ptr(); a.out = out.data_ptr(); a.ldo = out.stride(0);
+  a.T = (int)p.size(0); a.H = (int)H; a.d = (int)d;
+  return a;
+}
+
+Tensor delta_decode(const Tensor& p, const Tensor& zw, const Tensor& ab, const Tensor& w0, int64_t H, const Tensor& norm, double eps, Tensor state, const Tensor& active) {
+  const int dt = dtype_of(p);
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor out;
+  VbDelta a = delta_args(p, zw, ab, w0, H, state, out);
+  same(p, norm, "delta_decode");
+  TORCH_CHECK(norm.numel() == ab.numel() && norm.is_contiguous() && active.is_cuda() && active.scalar_type() == at::kBool && active.is_contiguous() && active.numel() == a.T &&
+              state.size(0) >= a.T, "delta_decode: active [S]");
+  a.active = reinterpret_cast<const uint8_t*>(active.data_ptr()); a.norm = norm.data_ptr(); a.eps = (float)eps;
+  verl_count_launches(1);
+  CHECK_RC(vb_delta_decode(dt, &a, cur_stream()), "vb_delta_decode");
+  return out;
+}
+
+Tensor delta_prefill(const Tensor& p, const Tensor& zw, const Tensor& ab, const Tensor& w0, int64_t H, const Tensor& cu, const OptTensor& state, const OptTensor& slots,
+                     const OptTensor& fresh) {
+  const int dt = dtype_of(p);
+  CHECK_I32(cu);
+  const c10::cuda::CUDAGuard guard(p.device());
+  Tensor out;
+  VbDelta a = delta_args(p, zw, ab, w0, H, state, out);
+  a.B = (int)cu.numel() - 1;
+  a.cu = cu.data_ptr<int>();
+  if (slots.has_value()) {
+    TORCH_CHECK(state.has_value() && fresh.has_value() && slots->numel() == a.B && fresh->numel() == a.B, "delta_prefill: slots need a state");
+    CHECK_I32(*slots);
+    CHECK_I32(*fresh);
+    a.slots = slots->data_ptr<int>(); a.fresh = fresh->data_ptr<int>();
+  }
+  if (a.T == 0 || a.B == 0) return out;
+  verl_count_launches(1);
+  int rc = dt == 1 ? vb_delta_chunk(&a, cur_stream()) : -1;
+  if (rc < 0) rc = vb_delta_scan(dt, &a, cur_stream());
+  CHECK_RC(rc, "delta_prefill");
+  return out;
+}
+
+// p [T, q | k | v]; see VbConvPrep. cu given: portions, else one token per slot. Returns (queries [T, H, dim], rows [T or 0, G dim + GV vdim]).
 std::tuple<Tensor, Tensor> conv_qkv_prep(const Tensor& p, const OptTensor& conv, double eps, const Tensor& pos, const Tensor& cs, const Tensor& sn, int64_t H, int64_t G,
-                                         int64_t dim, int64_t vdim, bool halves, const OptTensor& cu, const OptTensor& state, const OptTensor& slots,
+                                         int64_t GV, int64_t dim, int64_t vdim, bool halves, bool norm, const OptTensor& cu, const OptTensor& state, const OptTensor& slots,
                                          const OptTensor& fresh, const OptTensor& active, const OptTensor& pages, const OptTensor& page_slot, bool want_rows) {
   const int dt = dtype_of(p);
   CHECK_I32(pos);
   CHECK_F32(cs);
   CHECK_F32(sn);
-  const int64_t T = p.size(0), C = (H + G) * dim + G * vdim, width = G * (dim + vdim);
-  TORCH_CHECK(p.dim() == 2 && p.stride(1) == 1 && p.size(1) >= C && H > 0 && G > 0 && pos.numel() == T && cs.dim() == 2 && cs.is_contiguous() && sn.is_contiguous() &&
+  const int64_t T = p.size(0), C = (H + G) * dim + GV * vdim, width = G * dim + GV * vdim;
+  TORCH_CHECK(p.dim() == 2 && p.stride(1) == 1 && p.size(1) >= C && H > 0 && G >= 0 && GV >= 0 && pos.numel() == T && cs.dim() == 2 && cs.is_contiguous() && sn.is_contiguous() &&
               sn.sizes() == cs.sizes() && 2 * cs.size(1) <= dim, "conv_qkv_prep: sizes");
   const c10::cuda::CUDAGuard guard(p.device());
   VbConvPrep a{};
@@ -721,7 +921,7 @@ std::tuple<Tensor, Tensor> conv_qkv_prep(const Tensor& p, const OptTensor& conv,
     a.pages = pages->data_ptr(); a.page_stride = pages->stride(0); a.block_size = (int)pages->size(1); a.num_slots = pages->size(0) * pages->size(1);
     a.page_slot = lptr(*page_slot);
   }
-  a.T = (int)T; a.H = (int)H; a.G = (int)G; a.dim = (int)dim; a.vdim = (int)vdim; a.eps = (float)eps;
+  a.T = (int)T; a.H = (int)H; a.G = (int)G; a.GV = (int)GV; a.dim = (int)dim; a.vdim = (int)vdim; a.norm = norm; a.eps = (float)eps;
   verl_count_launches(a.cu != nullptr && a.state != nullptr ? 2 : 1);
   CHECK_RC(vb_conv_prep(dt, &a, cur_stream()), "vb_conv_prep");
   return {q, rows};
@@ -903,4 +1103,10 @@ TORCH_LIBRARY_FRAGMENT(verl_b200, m) {
   m.def("lightning_prefill", &lightning_prefill);
   m.def("mlstm_decode", &mlstm_decode);
   m.def("mlstm_prefill", &mlstm_prefill);
+  m.def("linear_tanh", &linear_tanh);
+  m.def("whole_norm_prep", &whole_norm_prep);
+  m.def("embed_rows", &embed_rows);
+  m.def("rms_conv", &rms_conv);
+  m.def("delta_prefill", &delta_prefill);
+  m.def("delta_decode", &delta_decode);
 }

@@ -14,7 +14,7 @@ struct ConvUnit { int n, col, channel_row; bool is_q, is_v; };
 __device__ __forceinline__ ConvUnit conv_unit(const VbConvPrep& a, int k) {
   ConvUnit u;
   u.is_q = k < a.H;
-  u.is_v = k >= a.H + a.G;
+  u.is_v = k >= a.H + a.G;       // a.GV heads
   u.n = u.is_v ? a.vdim : a.dim;
   u.col = u.is_v ? (a.H + a.G) * a.dim + (k - a.H - a.G) * a.vdim : k * a.dim;
   u.channel_row = u.is_q ? 0 : (u.is_v ? a.G * a.dim + (k - a.H - a.G) * a.vdim : (k - a.H) * a.dim);   // place inside a cached row
@@ -64,7 +64,7 @@ template <typename T, int TAPS, int N>
 __global__ void __launch_bounds__(256, 2)
 conv_prep_kernel(const VbConvPrep a, int L) {
   constexpr int VEC = 8, PAST = TAPS - 1;
-  const int lane = threadIdx.x & (L - 1), k = blockIdx.y, C = (a.H + a.G) * a.dim + a.G * a.vdim, c = lane * VEC;
+  const int lane = threadIdx.x & (L - 1), k = blockIdx.y, C = (a.H + a.G) * a.dim + a.GV * a.vdim, c = lane * VEC;
   const int t0 = (blockIdx.x * (256 / L) + threadIdx.x / L) * N;
   const ConvUnit un = conv_unit(a, k);
   const bool mine = c < un.n && t0 < a.T, rot = !un.is_v && c < 2 * a.half;
@@ -151,7 +151,7 @@ conv_prep_kernel(const VbConvPrep a, int L) {
         for (int h = 0; h < PAST; ++h) Vec<float, VEC>::store(st + static_cast<long long>(h) * C + un.col + c, past[h]);
       }
     }
-    if (!un.is_v) {                      // the same for the whole block
+    if (!un.is_v && (a.half > 0 || a.norm)) {   // the same for the whole block
       // rotation; the partner of (i, i + half) sits half / 8 lanes away
       if (a.halves) {
 #pragma unroll
@@ -167,14 +167,16 @@ conv_prep_kernel(const VbConvPrep a, int L) {
           v[i + 1] = z * cs[i] + y * sn[i];
         }
       }
-      float ss = 0.f;
+      if (a.norm) {
+        float ss = 0.f;
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) ss += v[i] * v[i];
-      if (c >= un.n) ss = 0.f;
-      for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
-      const float f = rsqrtf(ss * inv_n + a.eps);
+        for (int i = 0; i < VEC; ++i) ss += v[i] * v[i];
+        if (c >= un.n) ss = 0.f;
+        for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+        const float f = rsqrtf(ss * inv_n + a.eps);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v[i] *= f;
+        for (int i = 0; i < VEC; ++i) v[i] *= f;
+      }
     }
     if (!ok) continue;
     if (un.is_q) {
@@ -185,7 +187,7 @@ conv_prep_kernel(const VbConvPrep a, int L) {
         const long long sl = a.page_slot[t];
         if (sl >= 0 && sl < a.num_slots) {
           const unsigned blk = static_cast<unsigned>(sl) / static_cast<unsigned>(a.block_size), at = static_cast<unsigned>(sl) - blk * a.block_size;
-          Vec<T, VEC>::store(reinterpret_cast<T*>(a.pages) + blk * a.page_stride + static_cast<long long>(at) * (a.G * (a.dim + a.vdim)) + un.channel_row + c, v);
+          Vec<T, VEC>::store(reinterpret_cast<T*>(a.pages) + blk * a.page_stride + static_cast<long long>(at) * (a.G * a.dim + a.GV * a.vdim) + un.channel_row + c, v);
         }
       }
     }
@@ -197,7 +199,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 conv_prep_any_kernel(const VbConvPrep a, long long units) {
   extern __shared__ float sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, per = a.H + 2 * a.G, C = (a.H + a.G) * a.dim + a.G * a.vdim, past = a.taps - 1;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, per = a.H + a.G + a.GV, C = (a.H + a.G) * a.dim + a.GV * a.vdim, past = a.taps - 1;
   const long long u = blockIdx.x * 4ll + warp;
   if (u >= units) return;
   float* row = sm + warp * max(a.dim, a.vdim);
@@ -245,7 +247,7 @@ conv_prep_any_kernel(const VbConvPrep a, long long units) {
     const float v = turned(c);
     ss += v * v;
   }
-  const float f = un.is_v ? 1.f : 1.f / sqrtf(warp_sum(ss) / un.n + a.eps);
+  const float f = un.is_v || !a.norm ? 1.f : 1.f / sqrtf(warp_sum(ss) / un.n + a.eps);
   T *d0 = nullptr, *d1 = nullptr;
   if (un.is_q) {
     d0 = reinterpret_cast<T*>(a.q) + (t * a.H + k) * a.dim;
@@ -254,7 +256,7 @@ conv_prep_any_kernel(const VbConvPrep a, long long units) {
     if (a.pages != nullptr) {
       const long long sl = a.page_slot[t];
       if (sl >= 0 && sl < a.num_slots)
-        d1 = reinterpret_cast<T*>(a.pages) + (sl / a.block_size) * a.page_stride + (sl % a.block_size) * (a.G * (a.dim + a.vdim)) + un.channel_row;
+        d1 = reinterpret_cast<T*>(a.pages) + (sl / a.block_size) * a.page_stride + (sl % a.block_size) * (a.G * a.dim + a.GV * a.vdim) + un.channel_row;
     }
   }
   for (int c = lane; c < un.n; c += 32) {
@@ -286,7 +288,7 @@ using namespace vb;
 extern "C" int vb_conv_prep(int dtype, const VbConvPrep* p, cudaStream_t s) {
   if (p->T <= 0) return 0;
   auto mis = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) != 0; };
-  const int C = (p->H + p->G) * p->dim + p->G * p->vdim, per = p->H + 2 * p->G, most = p->dim > p->vdim ? p->dim : p->vdim;
+  const int C = (p->H + p->G) * p->dim + p->GV * p->vdim, per = p->H + p->G + p->GV, most = p->dim > p->vdim ? p->dim : p->vdim;
   const bool vec = p->num_slots < (1ll << 31) && per <= 65535 && p->dim % 8 == 0 && p->vdim % 8 == 0 && most <= 256 && p->taps <= 4 && p->ldp % 8 == 0 && p->ldr % 8 == 0 && p->page_stride % 8 == 0 &&
                    p->slot_stride % 4 == 0 && (!p->halves || p->half % 8 == 0) && !mis(p->p) && !mis(p->q) && !mis(p->rows) && !mis(p->pages) && !mis(p->state) &&
                    !mis(p->cos_t) && !mis(p->sin_t) && !mis(p->conv);

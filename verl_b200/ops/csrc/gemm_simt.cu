@@ -70,12 +70,18 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, int M, int N,
         case VB_EPI_GELU: D[m * e.ldd + n] = from_f<T>(gelu_erf(v)); break;
         case VB_EPI_BIAS: D[m * e.ldd + n] = from_f<T>(v + to_f(reinterpret_cast<const T*>(e.nb)[n])); break;
         case VB_EPI_SILU: D[m * e.ldd + n] = from_f<T>(n < e.n0 ? v * sigmoid_f(v) : v); break;
+        case VB_EPI_BIAS_RELU2: {
+          const float z = fmaxf(v + to_f(reinterpret_cast<const T*>(e.nb)[n]), 0.f);
+          D[m * e.ldd + n] = from_f<T>(z * z); break;
+        }
+        case VB_EPI_TANH: D[m * e.ldd + n] = from_f<T>(n < e.n0 ? v : tanhf(v)); break;
         case VB_EPI_SPLIT:
           if (n < e.n0) D[m * e.ldd + n] = from_f<T>(v);
           else e.D2[m * e.ldd2 + n - e.n0] = v;
           break;
         default: {
           if (e.pw != nullptr) v = tanhf(palpha * v) * to_f(reinterpret_cast<const T*>(e.pw)[n]) + to_f(reinterpret_cast<const T*>(e.pb)[n]);
+          else if (e.pb != nullptr) v += to_f(reinterpret_cast<const T*>(e.pb)[n]);
           const float x = e.X[m * e.ldx + n] + v;
           e.X[m * e.ldx + n] = x;
           if (e.D != nullptr)

@@ -644,11 +644,11 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
             const int cc = col0 + (lane & 7) * 4;
             if (cc < p.N) {
               float w4[4], b4[4], pw4[4], pb4[4];
-              const bool post = p.mix.pw != nullptr;
-              if (post) {
+              const bool post = p.mix.pw != nullptr, shift = !post && p.mix.pb != nullptr;
+              if (post || shift) {
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
-                  const float2 a = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(p.mix.pw)[cc / 2 + i]);
+                  const float2 a = post ? __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(p.mix.pw)[cc / 2 + i]) : make_float2(0.f, 0.f);
                   const float2 b = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(p.mix.pb)[cc / 2 + i]);
                   pw4[2 * i] = a.x; pw4[2 * i + 1] = a.y; pb4[2 * i] = b.x; pb4[2 * i + 1] = b.y;
                 }
@@ -671,6 +671,8 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
                     a.y = tanh_full(mix_palpha * a.y) * pw4[1] + pb4[1];
                     a.z = tanh_full(mix_palpha * a.z) * pw4[2] + pb4[2];
                     a.w = tanh_full(mix_palpha * a.w) * pw4[3] + pb4[3];
+                  } else if (shift) {
+                    a.x += pb4[0]; a.y += pb4[1]; a.z += pb4[2]; a.w += pb4[3];
                   }
                   a.x += xs[u].x; a.y += xs[u].y; a.z += xs[u].z; a.w += xs[u].w;
                   *reinterpret_cast<float4*>(p.mix.X + static_cast<long long>(rr) * p.mix.ldx + cc) = a;

@@ -6,7 +6,9 @@
 // heads are the M dimension of m16n8k16 MMAs: like every decode attention the kernel is bound by the stream, not by the
 // tensor pipe. Each of four warps owns 16 of a tile's tokens and keeps its own online softmax; warps and key splits are merged
 // at the end, where the sink (one more score without a value) joins the denominator. Scores may be capped
-// (cap * tanh(score / cap)). Only the tiles of the window and of the kept first tokens are loaded. Compiled without fast math.
+// (cap * tanh(score / cap)). Only the tiles of the window (or chunk) and of the kept first tokens are loaded. Differential attention: the
+// two key maps of a head are one key of twice the size, a query row is zero in the other map's half, so the stream is read once; the
+// merge forms the normed difference. Compiled without fast math.
 #include "mixer_epilogue.cuh"
 #include "mixers.h"
 #include "mixer_common.cuh"
@@ -30,8 +32,12 @@ struct GroupedDecodeParams {
   __nv_bfloat16* out;       // [S, H, vdim]
   float* part_o;            // [S, H, nsplit, vdim] when nsplit > 1
   float* part_ml;           // [S, H, nsplit, 2]
-  int H, share, chunks, dim, vdim, window, keep, nsplit;   // chunks: groups of 16 query heads per key head
+  int H, share, chunks, dim, vdim, window, keep, chunk, nsplit;   // chunks: groups of 16 query heads per key head
   float scale_log2, cap_z, cap_log2;
+  // differential attention: H and share count maps, dim spans both key maps of a head; a query row fills its map's half
+  int maps, map_dim;
+  const __nv_bfloat16* diff_vec;   // four vectors of map_dim
+  float diff, eps;
   int* status;
 };
 
@@ -46,6 +52,16 @@ __device__ __forceinline__ void gd_ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
 __device__ __forceinline__ void gd_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// lambda = exp(x0 . x1) - exp(x2 . x3) + diff, every lane of the warp gets it
+__device__ __forceinline__ float gd_lambda(const __nv_bfloat16* x, int n, float diff) {
+  float a = 0.f, b = 0.f;
+  for (int i = threadIdx.x & 31; i < n; i += 32) {
+    a = fmaf(__bfloat162float(x[i]), __bfloat162float(x[n + i]), a);
+    b = fmaf(__bfloat162float(x[2 * n + i]), __bfloat162float(x[3 * n + i]), b);
+  }
+  return expf(warp_sum(a)) - expf(warp_sum(b)) + diff;
 }
 
 template <int PK, int PV>
@@ -75,7 +91,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_con
   const int h0 = kvh * p.share + h_in, nh = min(GD_HEADS, p.share - h_in);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mi = lane >> 3, r8 = lane & 7;
   const int len = min(p.ctx_len[b], p.max_blocks * p.block_size);
-  const int first = (p.window > 0 && len > p.window) ? len - p.window : 0;
+  const int first = (p.window > 0 && len > p.window) ? len - p.window : (p.chunk > 0 && len > 0) ? (len - 1) / p.chunk * p.chunk : 0;
   const int tile_a = first / GD_TOK, tile_b = (len + GD_TOK - 1) / GD_TOK;
   // the list of tiles: those of the kept tokens that lie in front of the window's, then the window's
   const int nkeep = min((p.keep + GD_TOK - 1) / GD_TOK, tile_a), listed = nkeep + max(0, tile_b - tile_a);
@@ -96,7 +112,8 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_con
   for (int i = threadIdx.x; i < GD_HEADS * PK * 8; i += GD_THREADS) {
     const int g = i / (PK * 8), c = i % (PK * 8);
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (g < nh && c * 8 < p.dim) v = *reinterpret_cast<const uint4*>(p.q + b * p.ldq + static_cast<long long>(h0 + g) * p.hq + c * 8);
+    const int at = c * 8 - (p.maps > 1 && (g & 1) ? p.map_dim : 0);   // heads start at even rows
+    if (g < nh && at >= 0 && at < p.map_dim) v = *reinterpret_cast<const uint4*>(p.q + b * p.ldq + static_cast<long long>(h0 + g) * p.hq + at);
     *reinterpret_cast<uint4*>(sQ + g * L::QPITCH + c * 16) = v;
   }
   __syncthreads();
@@ -216,6 +233,47 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_con
     }
   }
   __syncthreads();
+  if (p.maps > 1 && p.nsplit == 1) {   // a warp per head: both maps merged, their difference normed
+    const float lam = gd_lambda(p.diff_vec, p.map_dim, p.diff);
+    for (int hh = warp; hh < nh / 2; hh += GD_THREADS / 32) {
+      float f[2][4];
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        const float* row = sM + (2 * hh + m) * L::MERGE_LD;
+        float M = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) M = fmaxf(M, row[w * GD_HEADS * L::MERGE_LD + PV * 64]);
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+          const float* rw = row + w * GD_HEADS * L::MERGE_LD;
+          f[m][w] = rw[PV * 64] == -INFINITY ? 0.f : exp2f(rw[PV * 64] - M);
+          l += rw[PV * 64 + 1] * f[m][w];
+        }
+        const float s = len > 0 && l > 0.f ? (m == 0 ? 1.f : -lam) / l : 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) f[m][w] *= s;
+      }
+      float z[PV * 2], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < PV * 2; ++i) {
+        const int d = i * 32 + lane;
+        z[i] = 0.f;
+        if (d < p.vdim) {
+#pragma unroll
+          for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int w = 0; w < 4; ++w) z[i] += sM[(w * GD_HEADS + 2 * hh + m) * L::MERGE_LD + d] * f[m][w];
+        }
+        ss += z[i] * z[i];
+      }
+      const float r = (1.f - p.diff) / sqrtf(warp_sum(ss) / p.vdim + p.eps);
+      __nv_bfloat16* o = p.out + (static_cast<long long>(b) * (p.H / 2) + h0 / 2 + hh) * p.vdim;
+#pragma unroll
+      for (int i = 0; i < PV * 2; ++i)
+        if (i * 32 + lane < p.vdim) o[i * 32 + lane] = __float2bfloat16(z[i] * r);
+    }
+    return;
+  }
   for (int idx = threadIdx.x; idx < nh * p.vdim; idx += GD_THREADS) {
     const int g = idx / p.vdim, d = idx % p.vdim;
     const float* row = sM + g * L::MERGE_LD;
@@ -261,14 +319,43 @@ __global__ void grouped_decode_merge_kernel(const float* __restrict__ po, const 
   }
 }
 
+// Joins the key splits of both maps of one (sequence, head) and finishes the difference. One warp per head.
+__global__ void __launch_bounds__(32)
+grouped_decode_merge_diff_kernel(const float* __restrict__ po, const float* __restrict__ ml, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
+                                 const __nv_bfloat16* __restrict__ vec, int map_dim, float diff, float eps, int heads, int nsplit, int vdim) {
+  const long long row = blockIdx.x;
+  const int lane = threadIdx.x;
+  const float lam = gd_lambda(vec, map_dim, diff);
+  float z[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, ss = 0.f;
+  for (int m = 0; m < 2; ++m) {
+    const long long at = (row * 2 + m) * nsplit;
+    float M = -INFINITY, l = 0.f;
+    for (int s = 0; s < nsplit; ++s) M = fmaxf(M, ml[2 * (at + s)]);
+    for (int s = 0; s < nsplit; ++s) l += ml[2 * (at + s)] == -INFINITY ? 0.f : exp2f(ml[2 * (at + s)] - M) * ml[2 * (at + s) + 1];
+    const float inv = (l > 0.f && ctx_len[row / heads] > 0) ? (m == 0 ? 1.f : -lam) / l : 0.f;
+    for (int s = 0; s < nsplit; ++s) {
+      const float f = ml[2 * (at + s)] == -INFINITY ? 0.f : exp2f(ml[2 * (at + s)] - M) * inv;
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i * 32 + lane < vdim) z[i] += f * po[(at + s) * vdim + i * 32 + lane];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss += z[i] * z[i];
+  const float r = (1.f - diff) / sqrtf(warp_sum(ss) / vdim + eps);
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (i * 32 + lane < vdim) out[row * vdim + i * 32 + lane] = __float2bfloat16(z[i] * r);
+}
+
 }  // namespace vb
 
 using namespace vb;
 
 // Key splits (0: the sizes are not served). max_keys: most keys a sequence can see.
 extern "C" int vb_grouped_decode_splits(const VbLatentAttn* a, int max_keys) {
-  const int share = a->kv_group > 1 ? a->kv_group : 1, bs = a->block_size;
-  if (a->du < 8 || a->du > 256 || a->du % 8 || a->dv < 8 || a->dv > 256 || a->dv % 8 || a->H % share) return 0;
+  const int maps = a->maps > 1 ? a->maps : 1, share = (a->kv_group > 1 ? a->kv_group : 1) * maps, bs = a->block_size;
+  if (a->du < 8 || a->du * maps > 256 || a->du % 8 || a->dv < 8 || a->dv > 256 || a->dv % 8 || a->H % share) return 0;
   if (bs % 8 || !(bs % GD_TOK == 0 || GD_TOK % bs == 0)) return 0;
   const int ctas = a->B * (a->H / share) * ((share + GD_HEADS - 1) / GD_HEADS), tiles = (max_keys + GD_TOK - 1) / GD_TOK;
   int s = 2 * num_sms() / (ctas > 0 ? ctas : 1);
@@ -276,14 +363,18 @@ extern "C" int vb_grouped_decode_splits(const VbLatentAttn* a, int max_keys) {
   return s < 1 ? 1 : (s > 32 ? 32 : s);
 }
 
-// Keys at ku (row stride ku_row inside a page, head stride ku_head), values at v; out [B, H, dv] contiguous. Returns -1 for strides
+// Keys at ku (row stride ku_row inside a page, head stride ku_head; two maps are neighbours), values at v; out [B, H, dv]
+// contiguous ([B, H / 2, dv] with two maps). Returns -1 for strides
 // and alignments it does not serve.
 extern "C" int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, int nsplit, float* part_o, float* part_ml, cudaStream_t stream) {
   if (a->B == 0) return 0;
   if (a->hq % 8 || a->ldq % 8 || a->page_stride % 8 || a->ku_row % 8 || a->ku_head % 8 || a->v_row % 8 || a->v_head % 8) return -1;
   if ((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->ku) | reinterpret_cast<uintptr_t>(a->v)) & 15) return -1;
   GroupedDecodeParams p{};
-  p.share = a->kv_group > 1 ? a->kv_group : 1;
+  p.maps = a->maps > 1 ? a->maps : 1;
+  p.share = (a->kv_group > 1 ? a->kv_group : 1) * p.maps;
+  const int dk = a->du * p.maps;     // a head's key maps lie behind each other
+  if (p.maps > 1 && (a->maps != 2 || a->ku_head != a->du || a->sink != nullptr)) return -1;
   p.chunks = (p.share + GD_HEADS - 1) / GD_HEADS;
   const int kv_heads = a->H / p.share;
   p.box_rows = a->block_size < GD_TOK ? a->block_size : GD_TOK;
@@ -291,7 +382,7 @@ extern "C" int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, in
   const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const uint64_t G = kv_heads, bs = a->block_size, nb = num_blocks, ps = a->page_stride;
   const uint32_t rows = p.box_rows;
-  if (!make_tmap_4d(&tk, a->ku, bf, 2, {(uint64_t)a->du, G, bs, nb}, {(uint64_t)a->ku_head, (uint64_t)a->ku_row, ps}, {64, 1, rows, 1}, CU_TENSOR_MAP_SWIZZLE_128B) ||
+  if (!make_tmap_4d(&tk, a->ku, bf, 2, {(uint64_t)dk, G, bs, nb}, {(uint64_t)a->ku_head * p.maps, (uint64_t)a->ku_row, ps}, {64, 1, rows, 1}, CU_TENSOR_MAP_SWIZZLE_128B) ||
       !make_tmap_4d(&tv, a->v, bf, 2, {(uint64_t)a->dv, G, bs, nb}, {(uint64_t)a->v_head, (uint64_t)a->v_row, ps}, {64, 1, rows, 1}, CU_TENSOR_MAP_SWIZZLE_128B))
     return -1;
   static int* status = nullptr;
@@ -299,7 +390,8 @@ extern "C" int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, in
   p.q = reinterpret_cast<const __nv_bfloat16*>(a->q); p.ldq = a->ldq; p.hq = a->hq;
   p.block_table = a->block_table; p.max_blocks = a->max_blocks; p.block_size = a->block_size; p.num_blocks = num_blocks; p.ctx_len = a->ctx_len;
   p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink); p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.part_o = part_o; p.part_ml = part_ml;
-  p.H = a->H; p.dim = a->du; p.vdim = a->dv; p.window = a->window; p.keep = a->window > 0 ? a->keep_first : 0; p.nsplit = nsplit; p.status = status;
+  p.map_dim = a->du; p.diff_vec = reinterpret_cast<const __nv_bfloat16*>(a->diff_vec); p.diff = a->diff; p.eps = a->eps; p.chunk = a->chunk;
+  p.H = a->H; p.dim = dk; p.vdim = a->dv; p.window = a->window; p.keep = a->window > 0 ? a->keep_first : 0; p.nsplit = nsplit; p.status = status;
   p.scale_log2 = a->scale * 1.4426950408889634f;
   if (a->softcap > 0.f) { p.cap_z = a->scale / a->softcap; p.cap_log2 = a->softcap * 1.4426950408889634f; }
   const dim3 grid(a->B, kv_heads * p.chunks, nsplit);
@@ -309,7 +401,7 @@ extern "C" int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, in
     kern<<<grid, GD_THREADS, smem, stream>>>(tk, tv, p);
     return static_cast<int>(cudaGetLastError());
   };
-  const int pk = (a->du + 63) / 64, pv = (a->dv + 63) / 64;
+  const int pk = (dk + 63) / 64, pv = (a->dv + 63) / 64;
   int rc;
   if (pk == 1 && pv == 1) rc = go(grouped_decode_kernel<1, 1>, GDSmem<1, 1>::TOTAL);
   else if (pk == 1 && pv == 2) rc = go(grouped_decode_kernel<1, 2>, GDSmem<1, 2>::TOTAL);
@@ -318,7 +410,11 @@ extern "C" int vb_grouped_decode(const VbLatentAttn* a, long long num_blocks, in
   else if (pk <= 3 && pv <= 2) rc = go(grouped_decode_kernel<3, 2>, GDSmem<3, 2>::TOTAL);
   else if (pk <= 2 && pv <= 4) rc = go(grouped_decode_kernel<2, 4>, GDSmem<2, 4>::TOTAL);
   else rc = go(grouped_decode_kernel<4, 4>, GDSmem<4, 4>::TOTAL);
-  if (rc == 0 && nsplit > 1) {
+  if (rc == 0 && nsplit > 1 && p.maps > 1) {
+    grouped_decode_merge_diff_kernel<<<a->B * (a->H / 2), 32, 0, stream>>>(part_o, part_ml, a->ctx_len, p.out, p.diff_vec, p.map_dim, p.diff, p.eps, a->H / 2, nsplit,
+                                                                           p.vdim);
+    rc = static_cast<int>(cudaGetLastError());
+  } else if (rc == 0 && nsplit > 1) {
     grouped_decode_merge_kernel<<<a->B * a->H, 128, 0, stream>>>(part_o, part_ml, a->ctx_len, p.out, a->H, nsplit, p.vdim);
     rc = static_cast<int>(cudaGetLastError());
   }

@@ -1,4 +1,4 @@
-// Prompt attention of the mixer stacks on tcgen05 tensor cores: causal, windowed (with kept first keys), with a sink, capped scores
+// Prompt attention of the mixer stacks on tcgen05 tensor cores: causal, windowed (with kept first keys) or chunked, with a sink, capped scores
 // and an output gate.
 // Latent attention, or grouped-query attention with query / key and value sizes of its own (no rotated part, kv_group query
 // heads per key head).
@@ -15,6 +15,9 @@
 //   warps 2 + 4t  softmax of tile t: thread == query row; the running maximum starts at the sink (weight 1, no value); O is
 //   .. 5 + 4t     rescaled only when a row's maximum grew by more than 2^8
 // Epilogue: O / l * sigmoid(gate) -> bf16 [T, H, dv].
+// Differential attention (PAIR): the two tiles are the two maps of the same 128 query rows; their key blocks stand behind each other in
+// a stage, the value blocks are shared. The epilogue forms the difference of the maps and norms it: a row's columns are divided
+// between its two threads (one per map), which exchange denominators and sums of squares through shared memory.
 #include "mixers.h"
 #include "tcgen05_common.cuh"
 
@@ -27,7 +30,7 @@ constexpr int LP_BQ = 128, LP_BK = 64;
 struct LatentPrefillParams {
   const int* cu_q;
   const int* cu_k;
-  int num_seqs, dv, window, keep, kv_group, pu, pr, pv, su, sr;  // panels of 64 columns (unrotated, rotated, value), k steps of 16
+  int num_seqs, dv, window, keep, chunk, kv_group, pu, pr, pv, su, sr;  // panels of 64 columns (unrotated, rotated, value), k steps of 16
   const __nv_bfloat16* sink;
   const float* gate;
   long long ldg;
@@ -39,6 +42,9 @@ struct LatentPrefillParams {
   float cap_z, cap_log2, cap_near, cap_poly[5];
   int tmem_cols;
   int* status;
+  const __nv_bfloat16* diff_vec;   // PAIR: four vectors of du entries
+  int du, key_maps;                // key_maps 2: key heads are maps, two per value head
+  float diff, eps;
 };
 
 __device__ int g_latent_prefill_status[1];
@@ -67,7 +73,65 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
   return r;
 }
 
-template <int NT, bool CAP>
+// Columns of a row of both maps' products -> (1 - diff) rms_norm(a0 - lambda a1). Threads (t = 0, 1; r) share row r: they take every
+// second group of 32 columns. The query tiles' place in shared memory, long read, holds what they exchange.
+__device__ __forceinline__ void pair_epilogue(const LatentPrefillParams& p, uint8_t* smem, uint32_t o_base, int t, int r, int lane, float inv_l, bool row_ok,
+                                              long long tok, int head) {
+  float *s_inv = reinterpret_cast<float*>(smem), *s_sum = s_inv + 2 * LP_BQ;
+  float x = 0.f, y = 0.f;
+  for (int i = lane; i < p.du; i += 32) {
+    x = fmaf(__bfloat162float(p.diff_vec[i]), __bfloat162float(p.diff_vec[p.du + i]), x);
+    y = fmaf(__bfloat162float(p.diff_vec[2 * p.du + i]), __bfloat162float(p.diff_vec[3 * p.du + i]), y);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    x += __shfl_xor_sync(0xffffffffu, x, o);
+    y += __shfl_xor_sync(0xffffffffu, y, o);
+  }
+  const float lam = expf(x) - expf(y) + p.diff;
+  s_inv[t * LP_BQ + r] = inv_l;
+  tc_fence_before();
+  asm volatile("bar.sync 1, 256;" ::: "memory");   // the softmax warps of both maps: both products are complete
+  tc_fence_after();
+  const float f0 = s_inv[r], f1 = -lam * s_inv[LP_BQ + r];
+  float ss = 0.f;
+  for (int c = t; c < p.pv * 2; c += 2) {
+    uint32_t a[32], b[32];
+    tmem_ld_32x32(o_base + c * 32, a);
+    tmem_ld_32x32(o_base + p.pv * 64 + c * 32, b);
+    tmem_ld_wait();
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      const float z = fmaf(__uint_as_float(a[i]), f0, __uint_as_float(b[i]) * f1);
+      ss = fmaf(z, z, ss);                          // columns past dv are zero
+    }
+  }
+  s_sum[t * LP_BQ + r] = ss;
+  asm volatile("bar.sync 1, 256;" ::: "memory");
+  const float g = (1.f - p.diff) * rsqrtf((s_sum[r] + s_sum[LP_BQ + r]) / p.dv + p.eps);
+  for (int c = t; c < p.pv * 2; c += 2) {
+    uint32_t a[32], b[32];
+    tmem_ld_32x32(o_base + c * 32, a);
+    tmem_ld_32x32(o_base + p.pv * 64 + c * 32, b);
+    tmem_ld_wait();
+    if (!row_ok) continue;
+    __nv_bfloat16* dst = p.out + tok * p.ldo + static_cast<long long>(head) * p.dv + c * 32;
+#pragma unroll
+    for (int i = 0; i < 32; i += 8) {
+      if (c * 32 + i < p.dv) {
+        uint32_t v[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int j = i + 2 * k;
+          v[k] = pack_bf16x2(g * fmaf(__uint_as_float(a[j]), f0, __uint_as_float(b[j]) * f1), g * fmaf(__uint_as_float(a[j + 1]), f0, __uint_as_float(b[j + 1]) * f1));
+        }
+        *reinterpret_cast<uint4*>(dst + i) = make_uint4(v[0], v[1], v[2], v[3]);
+      }
+    }
+  }
+}
+
+template <int NT, bool CAP, bool PAIR>
 __global__ void __launch_bounds__(64 + 128 * NT, 3 - NT)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_constant__ CUtensorMap tm_qr, const __grid_constant__ CUtensorMap tm_ku,
                       const __grid_constant__ CUtensorMap tm_kr, const __grid_constant__ CUtensorMap tm_v, const LatentPrefillParams p) {
@@ -77,8 +141,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
     if (threadIdx.x == 0) atomicExch(p.status, 9);
     return;
   }
+  constexpr int RT = PAIR ? 1 : NT;   // row tiles
   const int qp = p.pu + p.pr;
-  const int q_bytes = qp * (LP_BQ * 128), k_bytes = qp * (LP_BK * 128), v_bytes = p.pv * (LP_BK * 128);
+  const int q_bytes = qp * (LP_BQ * 128), map_bytes = qp * (LP_BK * 128), k_bytes = (PAIR ? 2 : 1) * map_bytes, v_bytes = p.pv * (LP_BK * 128);
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + NT * q_bytes;
   uint8_t* sV = sK + 2 * k_bytes;
@@ -89,13 +154,14 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
   uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bar_o + NT);
   int* s_tile = reinterpret_cast<int*>(tmem_holder + 2);  // query start, first row, queries, key start, keys, found
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y, kvh = head / p.kv_group;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y, kvh = head / p.kv_group;   // of the values; keys: kh
+  const int kh = PAIR ? 2 * kvh : p.key_maps > 1 ? 2 * kvh + (head & 1) : kvh;
   if (threadIdx.x == 0) {
     int t = blockIdx.x, found = 0, qs = 0, q0 = 0, nq = 0, ks = 0, nk = 0;
     for (int s = 0; s < p.num_seqs; ++s) {
-      const int a = p.cu_q[s], b = p.cu_q[s + 1], nt = (b - a + NT * LP_BQ - 1) / (NT * LP_BQ);
+      const int a = p.cu_q[s], b = p.cu_q[s + 1], nt = (b - a + RT * LP_BQ - 1) / (RT * LP_BQ);
       if (t < nt) {
-        qs = a; nq = b - a; q0 = (nt - 1 - t) * NT * LP_BQ; ks = p.cu_k[s]; nk = p.cu_k[s + 1] - ks; found = 1;
+        qs = a; nq = b - a; q0 = (nt - 1 - t) * RT * LP_BQ; ks = p.cu_k[s]; nk = p.cu_k[s + 1] - ks; found = 1;
         break;
       }
       t -= nt;
@@ -126,13 +192,14 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
   const int seq_q = s_tile[0], q0 = s_tile[1], nq = s_tile[2], seq_k = s_tile[3], nk = s_tile[4];
   const bool valid = s_tile[5] != 0;
   const int off = nk - nq;  // position of query row 0 among the sequence's keys
+  auto first_key = [&](int pos) { return p.window > 0 ? max(0, pos - p.window + 1) : p.chunk > 0 ? pos / p.chunk * p.chunk : 0; };
   // key blocks: entry j of the list holds keys [block_at(j) * 64, + 64); tile t uses j in [ja[t], jz[t]). Blocks of kept keys in front
   // of the window's come first; every tile walks the list from its start then.
   int jb0 = 0, nkeep = 0, ja[NT], jz[NT], nblk = 0;
 #pragma unroll
   for (int t = 0; t < NT; ++t) {
-    const int r0 = q0 + t * LP_BQ;
-    const int lo = p.window > 0 ? max(0, r0 + off - p.window + 1) : 0;
+    const int r0 = q0 + (PAIR ? 0 : t) * LP_BQ;
+    const int lo = first_key(r0 + off);
     if (t == 0) {
       jb0 = lo / LP_BK;
       nkeep = min((p.keep + LP_BK - 1) / LP_BK, jb0);
@@ -149,8 +216,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
     if (lane == 0 && valid) {
       mbar_expect_tx(q_full, static_cast<uint32_t>(NT * q_bytes));
       for (int t = 0; t < NT; ++t) {
-        const int row = seq_q + q0 + t * LP_BQ;
-        for (int c = 0; c < p.pu; ++c) tma_load_3d(sQ + t * q_bytes + c * (LP_BQ * 128), &tm_qu, q_full, 64 * c, head, row);
+        const int row = seq_q + q0 + (PAIR ? 0 : t) * LP_BQ;
+        for (int c = 0; c < p.pu; ++c) tma_load_3d(sQ + t * q_bytes + c * (LP_BQ * 128), &tm_qu, q_full, 64 * c, PAIR ? 2 * head + t : head, row);
         for (int c = 0; c < p.pr; ++c) tma_load_3d(sQ + t * q_bytes + (p.pu + c) * (LP_BQ * 128), &tm_qr, q_full, 64 * c, head, row);
       }
       for (int j = 0; j < nblk; ++j) {
@@ -158,7 +225,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         const uint32_t ph = ((j >> 1) & 1) ^ 1;
         if (!mbar_wait(&k_empty[st], ph)) { atomicExch(p.status, ST_TIMEOUT_PRODUCER); break; }
         mbar_expect_tx(&k_full[st], static_cast<uint32_t>(k_bytes));
-        for (int c = 0; c < p.pu; ++c) tma_load_3d(sK + st * k_bytes + c * (LP_BK * 128), &tm_ku, &k_full[st], 64 * c, kvh, row);
+        for (int c = 0; c < p.pu; ++c) tma_load_3d(sK + st * k_bytes + c * (LP_BK * 128), &tm_ku, &k_full[st], 64 * c, kh, row);
+        if constexpr (PAIR)
+          for (int c = 0; c < p.pu; ++c) tma_load_3d(sK + st * k_bytes + map_bytes + c * (LP_BK * 128), &tm_ku, &k_full[st], 64 * c, kh + 1, row);
         for (int c = 0; c < p.pr; ++c) tma_load_2d(sK + st * k_bytes + (p.pu + c) * (LP_BK * 128), &tm_kr, &k_full[st], 64 * c, row);
         if (!mbar_wait(&v_empty[st], ph)) { atomicExch(p.status, ST_TIMEOUT_PRODUCER); break; }
         mbar_expect_tx(&v_full[st], static_cast<uint32_t>(v_bytes));
@@ -178,7 +247,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
           if (j < ja[t] || j >= jz[t]) continue;
           const int jj = j - ja[t];
           const uint32_t d = tmem_base + (t * 2 + (jj & 1)) * LP_BK;
-          const uint32_t aq = smem_u32(sQ + t * q_bytes), bk = smem_u32(sK + st * k_bytes);
+          const uint32_t aq = smem_u32(sQ + t * q_bytes), bk = smem_u32(sK + st * k_bytes + (PAIR ? t * map_bytes : 0));
           for (int k = 0; k < p.su; ++k)
             tc_mma_f16_ss(d, make_smem_desc_sw128(aq + (k >> 2) * (LP_BQ * 128) + (k & 3) * 32, 16, 1024),
                           make_smem_desc_sw128(bk + (k >> 2) * (LP_BK * 128) + (k & 3) * 32, 16, 1024), idesc_s, k > 0 ? 1u : 0u);
@@ -224,11 +293,12 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
     const int n = z - a;
     if (n > 0) {
       const int quad = warp & 3, r = quad * 32 + lane;
-      const int row = q0 + t * LP_BQ + r;      // row inside the sequence's queries
+      const int row = q0 + (PAIR ? 0 : t) * LP_BQ + r;      // row inside the sequence's queries
       const int pos = row + off;               // its position among the keys
-      const int tile_lo = q0 + t * LP_BQ + off, tile_hi = tile_lo + LP_BQ - 1;
+      const int tile_lo = q0 + (PAIR ? 0 : t) * LP_BQ + off, tile_hi = tile_lo + LP_BQ - 1;
       const uint32_t lane_off = static_cast<uint32_t>(quad * 32) << 16;
       const uint32_t o_base = tmem_base + tm_o + t * p.pv * 64 + lane_off;
+      const int row_first = first_key(pos);    // without a window
       float m_run = -INFINITY, l_run = 0.f;
       if (p.sink != nullptr) { m_run = __bfloat162float(p.sink[head]) * 1.4426950408889634f; l_run = 1.f; }
       bool ok = true;
@@ -240,9 +310,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         tmem_ld_32x32(tmem_base + (t * 2 + (jj & 1)) * LP_BK + 32 + lane_off, x1);
         tmem_ld_wait();
         const int col0 = block_at(a + jj) * LP_BK;
-        const bool need_mask = col0 + LP_BK - 1 > tile_lo || (p.window > 0 && tile_hi - col0 >= p.window);
+        const bool need_mask = col0 + LP_BK - 1 > tile_lo || (p.window > 0 && tile_hi - col0 >= p.window) || (p.chunk > 0 && first_key(tile_hi) > col0);
         // visible: first_c <= c <= last_c, or c < keep_c and c <= last_c
-        const int last_c = pos - col0, first_c = p.window > 0 ? pos - p.window + 1 - col0 : -1, keep_c = p.keep - col0;
+        const int last_c = pos - col0, first_c = p.window > 0 ? pos - p.window + 1 - col0 : row_first - col0, keep_c = p.keep - col0;
         float mx = -INFINITY;
         if constexpr (CAP) {
           float most = 0.f;
@@ -332,9 +402,13 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
         if (lane == 0) mbar_arrive(&bar_p[t]);
       }
       if (ok) ok = mbar_wait(&bar_o[t], (n - 1) & 1);
-      if (!ok) {
-        if (lane == 0) atomicExch(p.status, ST_TIMEOUT_EPILOGUE);
-      } else {
+      if (!ok && lane == 0) atomicExch(p.status, ST_TIMEOUT_EPILOGUE);
+      if constexpr (PAIR) {
+        // every softmax warp comes here, also one that gave up: both maps walk the same blocks
+        tc_fence_after();
+        pair_epilogue(p, smem_raw, tmem_base + tm_o + lane_off, t, r, lane, l_run > 0.f ? 1.f / l_run : 0.f, ok && row < nq,
+                      static_cast<long long>(seq_q) + row, head);
+      } else if (ok) {
         tc_fence_after();
         const bool row_ok = row < nq;
         const long long tok = static_cast<long long>(seq_q) + row;
@@ -370,8 +444,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qu, const __grid_co
   }
 }
 
-static int latent_prefill_smem(int nt, int qp, int pv) {
-  return nt * qp * LP_BQ * 128 + 2 * qp * LP_BK * 128 + 2 * pv * LP_BK * 128 + nt * LP_BQ * LP_BK * 2 + 192;
+static int latent_prefill_smem(int nt, int qp, int pv, int maps = 1) {
+  return nt * qp * LP_BQ * 128 + 2 * maps * qp * LP_BK * 128 + 2 * pv * LP_BK * 128 + nt * LP_BQ * LP_BK * 2 + 192;
 }
 
 }  // namespace vb
@@ -385,19 +459,22 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
   if (a->du < 8 || a->dr < 0 || a->du % 8 || a->dr % 8 || a->dv % 8 || a->hq % 8 || a->ldq % 8 || a->ku_head % 8 || a->ku_row % 8 || a->kr_row % 8 ||
       a->v_head % 8 || a->v_row % 8 || a->ldo % 8 || mis(a->q) || mis(a->ku) || (a->dr > 0 && mis(a->kr)) || mis(a->v) || mis(a->out) || pv > 4)
     return -1;
-  const int limit = 232448, qp = pu + pr;
+  const int limit = 232448, qp = pu + pr, maps = a->maps > 1 ? a->maps : 1;
+  if (maps > 1 && (maps != 2 || pv > 2 || pr > 0 || a->gate != nullptr || a->sink != nullptr || a->softcap > 0.f || latent_prefill_smem(2, qp, pv, 2) > limit)) return -1;
   const bool pair = pv <= 2 && 2 * (latent_prefill_smem(1, qp, pv) + 1024) <= 228 * 1024;   // two CTAs of one tile (and 256 TMEM columns each)
-  const int nt = (!pair && pv <= 2 && latent_prefill_smem(2, qp, pv) <= limit) ? 2 : 1;
-  const int smem = latent_prefill_smem(nt, qp, pv);
+  const int nt = maps == 2 ? 2 : (!pair && pv <= 2 && latent_prefill_smem(2, qp, pv) <= limit) ? 2 : 1;
+  const int smem = latent_prefill_smem(nt, qp, pv, maps), rows_cta = (maps == 2 ? 1 : nt) * LP_BQ;
   if (smem > limit) return -1;
   const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const auto sw = CU_TENSOR_MAP_SWIZZLE_128B;
   CUtensorMap tqu, tqr, tku, tkr, tv;
   const char* qr = reinterpret_cast<const char*>(a->q) + 2 * a->du;
   if (a->dr > 0 && mis(qr)) return -1;
-  const int kv_group = a->kv_group > 1 ? a->kv_group : 1, kv_heads = a->H / kv_group;
+  // a PAIR's heads count once; split maps are heads of their own, two of which share values
+  const int key_maps = maps == 2 || a->split_maps ? 2 : 1, kv_group = (a->kv_group > 1 ? a->kv_group : 1) * (a->split_maps ? 2 : 1);
+  const int kv_heads = a->H / maps / kv_group;
   if (!make_tmap_3d(&tqu, a->q, bf, 2, a->du, a->H, a->T, a->hq, a->ldq, 64, 1, LP_BQ, sw) ||
-      !make_tmap_3d(&tku, a->ku, bf, 2, a->du, kv_heads, Tk, a->ku_head, a->ku_row, 64, 1, LP_BK, sw) ||
+      !make_tmap_3d(&tku, a->ku, bf, 2, a->du, kv_heads * key_maps, Tk, a->ku_head, a->ku_row, 64, 1, LP_BK, sw) ||
       !make_tmap_3d(&tv, a->v, bf, 2, a->dv, kv_heads, Tk, a->v_head, a->v_row, 64, 1, LP_BK, sw))
     return -1;
   if (a->dr > 0) {
@@ -411,7 +488,7 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
   static int* status = nullptr;
   if (status == nullptr) cudaGetSymbolAddress(reinterpret_cast<void**>(&status), g_latent_prefill_status);
   LatentPrefillParams p{};
-  p.cu_q = a->cu_q; p.cu_k = a->cu_k; p.num_seqs = a->B; p.dv = a->dv; p.window = a->window; p.keep = a->window > 0 ? a->keep_first : 0; p.kv_group = kv_group; p.pu = pu; p.pr = pr; p.pv = pv;
+  p.cu_q = a->cu_q; p.cu_k = a->cu_k; p.num_seqs = a->B; p.dv = a->dv; p.window = a->window; p.keep = a->window > 0 ? a->keep_first : 0; p.chunk = a->chunk; p.kv_group = kv_group; p.pu = pu; p.pr = pr; p.pv = pv;
   p.su = (a->du + 15) / 16; p.sr = (a->dr + 15) / 16;
   p.sink = reinterpret_cast<const __nv_bfloat16*>(a->sink); p.gate = a->gate; p.ldg = a->ldg;
   p.out = reinterpret_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo; p.scale_log2 = a->scale * 1.4426950408889634f; p.status = status;
@@ -427,15 +504,17 @@ extern "C" int vb_latent_prefill(const VbLatentAttn* a, int Tk, cudaStream_t str
   }
   p.tmem_cols = 128;
   while (p.tmem_cols < nt * (2 * LP_BK + pv * 64)) p.tmem_cols *= 2;
-  const dim3 grid((a->T + nt * LP_BQ - 1) / (nt * LP_BQ) + a->B, a->H);
+  p.diff_vec = reinterpret_cast<const __nv_bfloat16*>(a->diff_vec); p.du = a->du; p.key_maps = key_maps; p.diff = a->diff; p.eps = a->eps;
+  const dim3 grid((a->T + rows_cta - 1) / rows_cta + a->B, a->H / maps);
   auto go = [&](auto kern) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
     if (e != cudaSuccess) return static_cast<int>(e);
     kern<<<grid, 64 + 128 * nt, smem, stream>>>(tqu, tqr, tku, tkr, tv, p);
     return static_cast<int>(cudaGetLastError());
   };
-  if (a->softcap > 0.f) return nt == 2 ? go(latent_prefill_kernel<2, true>) : go(latent_prefill_kernel<1, true>);
-  return nt == 2 ? go(latent_prefill_kernel<2, false>) : go(latent_prefill_kernel<1, false>);
+  if (maps == 2) return go(latent_prefill_kernel<2, false, true>);
+  if (a->softcap > 0.f) return nt == 2 ? go(latent_prefill_kernel<2, true, false>) : go(latent_prefill_kernel<1, true, false>);
+  return nt == 2 ? go(latent_prefill_kernel<2, false, false>) : go(latent_prefill_kernel<1, false, false>);
 }
 
 extern "C" int vb_latent_prefill_status() {

@@ -18,6 +18,7 @@ __device__ __forceinline__ float tanh_full(float x) {
 __device__ __forceinline__ float gelu_erf_full(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
 __device__ __forceinline__ float silu_full(float z) { return z / (1.f + __expf(-z)); }
+__device__ __forceinline__ float relu2(float z) { return fmaxf(z, 0.f) * fmaxf(z, 0.f); }
 
 struct EpiColumn { float w, b, pw, pb; };  // weight and bias of an output column: of the norm of the stream, of the norm of the product
 __device__ __forceinline__ EpiColumn epi_column(const VbEpiArgs& e, int col) {
@@ -30,7 +31,8 @@ __device__ __forceinline__ EpiColumn epi_column(const VbEpiArgs& e, int col) {
     c.pw = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.pw)[col]);
     c.pb = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.pb)[col]);
   }
-  if (e.mode == VB_EPI_BIAS) c.b = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.nb)[col]);
+  if (e.mode == VB_EPI_RESID && e.pw == nullptr && e.pb != nullptr) c.pb = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.pb)[col]);
+  if (e.mode == VB_EPI_BIAS || e.mode == VB_EPI_BIAS_RELU2) c.b = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(e.nb)[col]);
   return c;
 }
 __device__ __forceinline__ float epi_palpha(const VbEpiArgs& e) {
@@ -53,13 +55,17 @@ __device__ __forceinline__ void epi_store1(const VbEpiArgs& e, long long row, in
     if (col < e.n0) D[row * e.ldd + col] = __float2bfloat16(v);
     else e.D2[row * e.ldd2 + col - e.n0] = v;
   } else if (e.mode == VB_EPI_RESID) {
-    const float x = e.X[row * e.ldx + col] + (e.pw != nullptr ? tanh_full(palpha * v) * c.pw + c.pb : v);
+    const float x = e.X[row * e.ldx + col] + (e.pw != nullptr ? tanh_full(palpha * v) * c.pw + c.pb : v + c.pb);
     e.X[row * e.ldx + col] = x;
     if (D != nullptr) D[row * e.ldd + col] = __float2bfloat16(tanh_full(alpha * x) * c.w + c.b);
   } else if (e.mode == VB_EPI_BIAS) {
     D[row * e.ldd + col] = __float2bfloat16(v + c.b);
   } else if (e.mode == VB_EPI_SILU) {
     D[row * e.ldd + col] = __float2bfloat16(col < e.n0 ? silu_full(v) : v);
+  } else if (e.mode == VB_EPI_BIAS_RELU2) {
+    D[row * e.ldd + col] = __float2bfloat16(relu2(v + c.b));
+  } else if (e.mode == VB_EPI_TANH) {
+    D[row * e.ldd + col] = __float2bfloat16(col < e.n0 ? v : tanh_full(v));
   } else {
     D[row * e.ldd + col] = __float2bfloat16(v);
   }
@@ -105,6 +111,10 @@ __device__ __forceinline__ void epi_store_row(const VbEpiArgs& e, long long row,
       const __nv_bfloat16* b = reinterpret_cast<const __nv_bfloat16*>(e.pb) + col;
 #pragma unroll
       for (int i = 0; i < NV; ++i) o[i] = tanh_full(palpha * v[i]) * __bfloat162float(w[i]) + __bfloat162float(b[i]);
+    } else if (e.pb != nullptr) {
+      const __nv_bfloat16* b = reinterpret_cast<const __nv_bfloat16*>(e.pb) + col;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) o[i] += __bfloat162float(b[i]);
     }
 #pragma unroll
     for (int i = 0; i < NV; i += 4) {
@@ -119,11 +129,25 @@ __device__ __forceinline__ void epi_store_row(const VbEpiArgs& e, long long row,
       for (int i = 0; i < NV; ++i) o[i] = tanh_full(alpha * o[i]) * __bfloat162float(w[i]) + __bfloat162float(b[i]);
       put16(o);
     }
-  } else if (e.mode == VB_EPI_BIAS) {
+  } else if (e.mode == VB_EPI_BIAS || e.mode == VB_EPI_BIAS_RELU2) {
     const __nv_bfloat16* b = reinterpret_cast<const __nv_bfloat16*>(e.nb) + col;
     float o[NV];
 #pragma unroll
     for (int i = 0; i < NV; ++i) o[i] = v[i] + __bfloat162float(b[i]);
+    if (e.mode == VB_EPI_BIAS_RELU2) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) o[i] = relu2(o[i]);
+    }
+    put16(o);
+  } else if (e.mode == VB_EPI_TANH) {
+    float o[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] = v[i];
+    if (col + NV > e.n0) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (col + i >= e.n0) o[i] = tanh_full(v[i]);
+    }
     put16(o);
   } else if (e.mode == VB_EPI_SILU) {
     float o[NV];

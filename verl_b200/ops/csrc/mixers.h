@@ -11,11 +11,13 @@ enum VbEpi : int {
   VB_EPI_STORE_F32 = 1, // D = acc as fp32
   VB_EPI_GELU = 2,      // D = erf-gelu(acc) in the operands' type
   VB_EPI_SPLIT = 3,     // columns [0, n0) -> D in the operands' type, columns [n0, N) -> D2 as fp32
-  VB_EPI_RESID = 4,     // X += acc, or tanh(palpha acc) pw + pb when pw is given (fp32 residual stream); D = tanh(alpha X) nw + nb in the
+  VB_EPI_RESID = 4,     // X += acc (+ pb when given), or tanh(palpha acc) pw + pb when pw is given (fp32 residual stream); D = tanh(alpha X) nw + nb in the
                         // operands' type when D is given
   VB_EPI_SOFTCAP = 5,   // D = cap * tanh(acc / cap) in the operands' type
   VB_EPI_BIAS = 6,      // D = acc + nb in the operands' type
   VB_EPI_SILU = 7,      // D = silu(acc) in columns [0, n0), acc in the others, in the operands' type
+  VB_EPI_BIAS_RELU2 = 8,// D = max(acc + nb, 0)^2 in the operands' type
+  VB_EPI_TANH = 9,      // D = acc in columns [0, n0), tanh(acc) in the others, in the operands' type
 };
 
 struct VbEpiArgs {
@@ -33,7 +35,7 @@ struct VbEpiArgs {
   float cap;
   const float* gate;  // batched products: batch z of row m is multiplied by sigmoid(gate[m * ldg + z]) when given
   long long ldg;
-  const void* palpha; // VB_EPI_RESID: norm of the product (scalar, [N], [N]), or null
+  const void* palpha; // VB_EPI_RESID: norm of the product (scalar, [N], [N]), or null; pb alone: a bias
   const void* pw;
   const void* pb;
 };
@@ -60,6 +62,14 @@ struct VbLatentAttn {
   int kv_group;             // query heads per key / value head (0 or 1: one)
   float softcap;            // score = softcap * tanh(score / softcap); 0: off
   int keep_first;           // with a window: the sequence's first keys that every query sees besides
+  int chunk;                // > 0: a query sees the keys from its chunk's start on; the sequence's first key row starts a chunk
+  // maps = 2: differential attention. H counts maps (query map m of head h is 2h + m, key map m of head g is 2g + m) and kv_group the
+  // query heads per value head, maps not counted; out [T, H / 2, dv]: (1 - diff) rms_norm(a1 - lambda a2), lambda from the
+  // four vectors of du entries at diff_vec (exp(x0 . x1) - exp(x2 . x3) + diff)
+  int maps;
+  int split_maps;           // vb_latent_prefill: every query head is a map (key head as with maps = 2, maps apart in out [T, H, dv])
+  const void* diff_vec;
+  float diff, eps;
 };
 
 // x += mult * rms_norm(Y) * nw;  Y = [sigmoid(gate)] sum of `splits` planes of y + sum_j rows[slot[t, j]]
@@ -105,7 +115,7 @@ struct VbResidDyt {
   int T, W;
 };
 
-// Row p[t] = [q of H heads | k of G heads | v of G heads]: causal convolution per channel, rotation of q and k, norm without weight.
+// Row p[t] = [q of H heads | k of G heads | v of GV heads]: causal convolution per channel, rotation of q and k, norm without weight.
 struct VbConvPrep {
   const void* p; long long ldp;
   const void* conv; int taps;         // [channels, taps], last tap = the token itself (null: no convolution, taps = 1)
@@ -115,10 +125,50 @@ struct VbConvPrep {
   const uint8_t* active;              // steps: row t is slot t
   const int* pos; const float *cos_t, *sin_t; int half, max_pos, halves;
   void* q;                            // [T, H, dim]
+  void* rows; long long ldr;          // [T, G dim + GV vdim] or null
+  void* pages; long long page_stride; int block_size; long long num_slots; const long long* page_slot;
+  int T, H, G, GV, dim, vdim, norm;   // norm 0: none
+  float eps;
+};
+
+// Row p[t] = [q | k | v]: weighted RMS norms over all query and over all key columns, queries times temp of their head.
+struct VbWholeNorm {
+  const void* p; long long ldp;
+  const void *qn, *kn, *temp;         // [H dim], [G dim], [H]
+  void* q;                            // [T, H dim]
   void* rows; long long ldr;          // [T, G (dim + vdim)] or null
   void* pages; long long page_stride; int block_size; long long num_slots; const long long* page_slot;
   int T, H, G, dim, vdim;
   float eps;
+};
+
+// h = rms_norm(x) nw, plus its causal convolution over time with `conv` [W, taps] when given (last tap: the token itself).
+struct VbRmsConv {
+  float* x;                           // [T, W]; first x += sum of `splits` planes of y (+ bias) when given (steps only)
+  const void* y; int y_f32, splits; long long split_stride, ldy;
+  const void *bias, *nw, *conv;
+  int taps;
+  const int* cu; int B;               // portions; null: one token per slot
+  float* state; long long slot_stride;// last taps - 1 rows of a sequence, [taps - 1, W], oldest first
+  const int *slots, *fresh;
+  const uint8_t* active;
+  void* h;                            // [T, W]
+  int T, W;
+  float eps;
+};
+
+// Generalized delta rule over rows p[t] = [r | k | v | za | g | ...] (H d columns each): S = diag(w) S - (a u)(u^T S) + k v^T, o = S^T r with
+// w = exp(-exp(-1/2) sigmoid(zw + w0)), a = sigmoid(za + ab), u = k / sqrt(k . k + 1e-6).
+struct VbDelta {
+  const void* p; long long ldp;
+  const void* zw; long long ldz;      // [T, H d]
+  const void *ab, *w0;                // [H d]
+  float* state; long long slot_stride;// [slots, H, d, d] or null
+  const int *slots, *fresh, *cu;      // portions
+  const uint8_t* active;              // steps: row t is slot t
+  const void* norm; float eps;        // steps: out = rms_norm(o) norm sigmoid(g)
+  void* out; long long ldo;           // [T, H d]
+  int T, B, H, d;
 };
 
 // Recurrence S = decay S + k v^T, o = S^T q per head over rows p[t] = [q | k | v | ...].
@@ -167,7 +217,19 @@ int vb_embed_rms(int dtype, const long long* ids, const void* w, float scale, co
 int vb_residual_rms(int dtype, const VbResidRms* p, cudaStream_t s);
 int vb_gated_silu(int dtype, const void* gu, long long ldg, const float* row_scale, float clip, void* out, int T, int I, cudaStream_t s);
 int vb_residual_dyt(int dtype, const VbResidDyt* p, cudaStream_t s);
-int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W, cudaStream_t s);
+// W = heads * size: statistics over each head's columns
+int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W, int heads,
+                 cudaStream_t s);
+int vb_whole_norm(int dtype, const VbWholeNorm* p, cudaStream_t s);
+// a [T, 2 H, dv] -> out [T, H, dv], see VbLatentAttn::maps
+int vb_diff_combine(int dtype, const void* a, int a_f32, const void* vec, int dim, float diff, float eps, void* out, int T, int H, int dv, cudaStream_t s);
+// rms_conv.cu
+int vb_embed_rows(int dtype, const long long* ids, const void* w, float scale, float* x, int T, int W, int V, cudaStream_t s);
+int vb_rms_conv(int dtype, const VbRmsConv* p, cudaStream_t s);
+// delta_rule.cu / delta_chunk.cu
+int vb_delta_decode(int dtype, const VbDelta* p, cudaStream_t s);
+int vb_delta_scan(int dtype, const VbDelta* p, cudaStream_t s);
+int vb_delta_chunk(const VbDelta* p, cudaStream_t s);
 // conv_prep.cu
 int vb_conv_prep(int dtype, const VbConvPrep* p, cudaStream_t s);
 // lightning.cu / lightning_tcgen05.cu (d <= 128) / lightning_chunk.cu; nseg > 1: workspace of B (nseg - 1) H d e floats
@@ -222,5 +284,6 @@ int vb_headwise(const VbHeadwise* p, cudaStream_t s);
 int vb_latent_decode_splits(int S, int H, int rank, int width, int block_size, int max_keys);
 int vb_latent_decode(const VbLatentAttn* a, long long num_blocks, int nsplit, float* part_o, float* part_ml, cudaStream_t s);
 // latent_attention_simt.cu
-int vb_latent_attn_simt(int dtype, const VbLatentAttn* a, cudaStream_t s);
+// out_f32: out is fp32 whatever the operands' type
+int vb_latent_attn_simt(int dtype, const VbLatentAttn* a, int out_f32, cudaStream_t s);
 }

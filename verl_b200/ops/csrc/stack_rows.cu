@@ -1,7 +1,7 @@
 // Row kernels of stacks with norms on the sublayers' outputs: normed embedding, residual add of a normed sublayer output (which
 // also adds up split-K partial products and the rows of chosen experts; RMS or Dynamic Tanh), gated activations, gated RMS norm
-// of a row, and the preparation of grouped-query attention (norm and rotation of query and key heads, value mixing, append to
-// the paged cache).
+// of a row or of its heads, and the preparation of grouped-query attention (norm and rotation of query and key heads, or norms over whole
+// projections, value mixing, append to the paged cache), and the normed difference of two attention maps.
 // Statistics, angles and the residual stream are fp32; compiled without fast math.
 #include "mixers.h"
 #include "mixer_common.cuh"
@@ -215,6 +215,126 @@ static int gated_rms(const void* o, long long ldo, const void* g, long long ldg,
   return -1;
 }
 
+// --------------------------------------------------------------------------------------------- the same with one norm per head
+// L lanes share a head row of one token (n <= 32 VEC ITEMS columns).
+template <typename T, int VEC, int ITEMS>
+__global__ void __launch_bounds__(256)
+gated_rms_heads_kernel(const T* __restrict__ o, long long ldo, const T* __restrict__ g, long long ldg, const T* __restrict__ norm, float eps, T* __restrict__ out,
+                       int n, int heads, int L, long long units) {
+  const long long u = (blockIdx.x * 256ll + threadIdx.x) / L;
+  const int lane = threadIdx.x & (L - 1);
+  const bool live = u < units;
+  const long long t = live ? u / heads : 0;
+  const int col = live ? static_cast<int>(u % heads) * n : 0;
+  float v[ITEMS][VEC], z[ITEMS][VEC], w[VEC], ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int c = (it * L + lane) * VEC;
+    if (!live || c >= n) continue;
+    Vec<T, VEC>::load(o + t * ldo + col + c, v[it]);
+    Vec<T, VEC>::load(g + t * ldg + col + c, z[it]);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) ss += v[it][k] * v[it][k];
+  }
+  for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+  const float r = 1.f / sqrtf(ss / n + eps);
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int c = (it * L + lane) * VEC;
+    if (!live || c >= n) continue;
+    Vec<T, VEC>::load(norm + col + c, w);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[it][k] = v[it][k] * r * w[k] * sigmoid_f(z[it][k]);
+    Vec<T, VEC>::store(out + t * (static_cast<long long>(heads) * n) + col + c, v[it]);
+  }
+}
+
+template <typename T, int VEC>
+static int gated_rms_heads(const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T_, int n, int heads, cudaStream_t s) {
+  int L = 1;
+  while (L < 32 && L * VEC < n) L *= 2;
+  const int items = (n + L * VEC - 1) / (L * VEC);
+  const long long units = static_cast<long long>(T_) * heads;
+  auto go = [&](auto kern) {
+    kern<<<static_cast<unsigned>((units * L + 255) / 256), 256, 0, s>>>((const T*)o, ldo, (const T*)g, ldg, (const T*)norm, eps, (T*)out, n, heads, L, units);
+    return static_cast<int>(cudaGetLastError());
+  };
+  if (items == 1) return go(gated_rms_heads_kernel<T, VEC, 1>);
+  if (items <= 4) return go(gated_rms_heads_kernel<T, VEC, 4>);
+  if (items <= 16) return go(gated_rms_heads_kernel<T, VEC, 16>);
+  return -1;
+}
+
+// --------------------------------------------------------------------------------------------- difference of two attention maps
+// One warp per (token, head): a [T, 2 H, dv] -> (1 - diff) rms_norm(a0 - lambda a1).
+template <typename A, typename T>
+__global__ void __launch_bounds__(128)
+diff_combine_kernel(const A* __restrict__ a, const T* __restrict__ vec, int dim, float diff, float eps, T* __restrict__ out, long long rows, int dv) {
+  const int lane = threadIdx.x & 31;
+  const long long u = blockIdx.x * 4ll + (threadIdx.x >> 5);
+  if (u >= rows) return;
+  float x = 0.f, y = 0.f;
+  for (int i = lane; i < dim; i += 32) {
+    x += to_f(vec[i]) * to_f(vec[dim + i]);
+    y += to_f(vec[2 * dim + i]) * to_f(vec[3 * dim + i]);
+  }
+  const float lam = expf(warp_sum(x)) - expf(warp_sum(y)) + diff;
+  const A *a0 = a + 2 * u * dv, *a1 = a0 + dv;
+  float ss = 0.f;
+  for (int c = lane; c < dv; c += 32) {
+    const float z = to_f(a0[c]) - lam * to_f(a1[c]);
+    ss += z * z;
+  }
+  const float r = (1.f - diff) / sqrtf(warp_sum(ss) / dv + eps);
+  for (int c = lane; c < dv; c += 32) out[u * dv + c] = from_f<T>((to_f(a0[c]) - lam * to_f(a1[c])) * r);
+}
+
+// --------------------------------------------------------------------------------------------- norms over whole query and key projections
+// One CTA per token.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+whole_norm_kernel(const VbWholeNorm a) {
+  __shared__ float red[33];
+  const long long t = blockIdx.x;
+  const int nq = a.H * a.dim, nk = a.G * a.dim, nv = a.G * a.vdim;
+  const T* p = reinterpret_cast<const T*>(a.p) + t * a.ldp;
+  float v[VEC], w[VEC], sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * VEC; c < nq + nk; c += 256 * VEC) {
+    Vec<T, VEC>::load(p + c, v);
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s += v[i] * v[i];
+    if (c < nq) sq += s; else sk += s;
+  }
+  const float rq = 1.f / sqrtf(block_sum(sq, red) / nq + a.eps), rk = 1.f / sqrtf(block_sum(sk, red) / nk + a.eps);
+  T* q = reinterpret_cast<T*>(a.q) + t * nq;
+  T* d0 = a.rows != nullptr ? reinterpret_cast<T*>(a.rows) + t * a.ldr : nullptr;
+  T* d1 = nullptr;
+  if (a.pages != nullptr) {
+    const long long sl = a.page_slot[t];
+    if (sl >= 0 && sl < a.num_slots) d1 = reinterpret_cast<T*>(a.pages) + (sl / a.block_size) * a.page_stride + (sl % a.block_size) * (nk + nv);
+  }
+  for (int c = threadIdx.x * VEC; c < nq + nk + nv; c += 256 * VEC) {
+    Vec<T, VEC>::load(p + c, v);
+    if (c < nq) {
+      const float f = rq * to_f(reinterpret_cast<const T*>(a.temp)[c / a.dim]);
+      Vec<T, VEC>::load(reinterpret_cast<const T*>(a.qn) + c, w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = v[i] * f * w[i];
+      Vec<T, VEC>::store(q + c, v);
+      continue;
+    }
+    const int at = c - nq;
+    if (at < nk) {
+      Vec<T, VEC>::load(reinterpret_cast<const T*>(a.kn) + at, w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = v[i] * rk * w[i];
+    }
+    if (d0 != nullptr) Vec<T, VEC>::store(d0 + at, v);
+    if (d1 != nullptr) Vec<T, VEC>::store(d1 + at, v);
+  }
+}
+
 // --------------------------------------------------------------------------------------------- silu(r g) * (r u), or the clipped form
 template <typename T, int VEC>
 __global__ void gated_silu_kernel(const T* __restrict__ gu, long long ldg, const float* __restrict__ row_scale, float clip, T* __restrict__ out, int I,
@@ -383,9 +503,39 @@ extern "C" int vb_residual_dyt(int dtype, const VbResidDyt* p, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W,
+extern "C" int vb_whole_norm(int dtype, const VbWholeNorm* p, cudaStream_t s) {
+  if (p->T <= 0) return 0;
+  const bool vec = p->dim % 8 == 0 && p->vdim % 8 == 0 && p->ldp % 8 == 0 && p->ldr % 8 == 0 && p->page_stride % 8 == 0 && !mis16(p->p) && !mis16(p->qn) &&
+                   !mis16(p->kn) && !mis16(p->q) && !mis16(p->rows) && !mis16(p->pages);
+  if (dtype == 0) {
+    if (vec) whole_norm_kernel<float, 8><<<p->T, 256, 0, s>>>(*p);
+    else whole_norm_kernel<float, 1><<<p->T, 256, 0, s>>>(*p);
+  } else {
+    if (vec) whole_norm_kernel<bf16, 8><<<p->T, 256, 0, s>>>(*p);
+    else whole_norm_kernel<bf16, 1><<<p->T, 256, 0, s>>>(*p);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int vb_diff_combine(int dtype, const void* a, int a_f32, const void* vec, int dim, float diff, float eps, void* out, int T, int H, int dv, cudaStream_t s) {
+  const long long rows = static_cast<long long>(T) * H;
+  if (rows <= 0) return 0;
+  const unsigned grid = static_cast<unsigned>((rows + 3) / 4);
+  if (dtype == 0) diff_combine_kernel<float, float><<<grid, 128, 0, s>>>((const float*)a, (const float*)vec, dim, diff, eps, (float*)out, rows, dv);
+  else if (a_f32) diff_combine_kernel<float, bf16><<<grid, 128, 0, s>>>((const float*)a, (const bf16*)vec, dim, diff, eps, (bf16*)out, rows, dv);
+  else diff_combine_kernel<bf16, bf16><<<grid, 128, 0, s>>>((const bf16*)a, (const bf16*)vec, dim, diff, eps, (bf16*)out, rows, dv);
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W, int heads,
                             cudaStream_t s) {
   if (T <= 0 || W <= 0) return 0;
+  if (heads > 1) {
+    const int n = W / heads;
+    const bool v8 = n % 8 == 0 && ldo % 8 == 0 && ldg % 8 == 0 && !mis16(o) && !mis16(g) && !mis16(norm) && !mis16(out);
+    if (dtype == 0) return v8 ? gated_rms_heads<float, 8>(o, ldo, g, ldg, norm, eps, out, T, n, heads, s) : gated_rms_heads<float, 1>(o, ldo, g, ldg, norm, eps, out, T, n, heads, s);
+    return v8 ? gated_rms_heads<bf16, 8>(o, ldo, g, ldg, norm, eps, out, T, n, heads, s) : gated_rms_heads<bf16, 1>(o, ldo, g, ldg, norm, eps, out, T, n, heads, s);
+  }
   const bool vec = W % 8 == 0 && ldo % 8 == 0 && ldg % 8 == 0 && !mis16(o) && !mis16(g) && !mis16(norm) && !mis16(out);
   if (dtype == 0) return vec ? gated_rms<float, 8>(o, ldo, g, ldg, norm, eps, out, T, W, s) : gated_rms<float, 1>(o, ldo, g, ldg, norm, eps, out, T, W, s);
   return vec ? gated_rms<bf16, 8>(o, ldo, g, ldg, norm, eps, out, T, W, s) : gated_rms<bf16, 1>(o, ldo, g, ldg, norm, eps, out, T, W, s);
