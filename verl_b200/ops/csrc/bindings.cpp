@@ -158,6 +158,7 @@ int64_t gemm_status() {
   if (b == 0) b = vb_grouped_decode_status();
   if (b == 0) b = vb_latent_prefill_status();
   if (b == 0) b = vb_lightning_status();
+  if (b == 0) b = vb_delta_chunk_status();
   const int c = vb_pd_status();
   return a != 0 ? a : (b != 0 ? 100 + b : (c != 0 ? 200 + c : 0));
 }

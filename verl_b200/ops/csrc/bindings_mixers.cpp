@@ -861,10 +861,19 @@ Tensor delta_prefill(const Tensor& p, const Tensor& zw, const Tensor& ab, const 
     a.slots = slots->data_ptr<int>(); a.fresh = fresh->data_ptr<int>();
   }
   if (a.T == 0 || a.B == 0) return out;
+  const int nseg = dt == 1 ? vb_delta_chunk_segments(&a) : 0;
+  if (nseg > 0) {
+    Tensor ws;
+    if (nseg > 1) ws = at::empty({(int64_t)a.B * nseg * a.H * 2 * a.d * a.d}, p.options().dtype(at::kFloat));
+    const int rc = vb_delta_chunk(&a, nseg, nseg > 1 ? ws.data_ptr<float>() : nullptr, cur_stream());
+    if (rc >= 0) {
+      verl_count_launches(nseg > 1 ? 3 : 1);
+      CHECK_RC(rc, "vb_delta_chunk");
+      return out;
+    }
+  }
   verl_count_launches(1);
-  int rc = dt == 1 ? vb_delta_chunk(&a, cur_stream()) : -1;
-  if (rc < 0) rc = vb_delta_scan(dt, &a, cur_stream());
-  CHECK_RC(rc, "delta_prefill");
+  CHECK_RC(vb_delta_scan(dt, &a, cur_stream()), "vb_delta_scan");
   return out;
 }
 

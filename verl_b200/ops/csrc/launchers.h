@@ -130,6 +130,7 @@ int vb_latent_decode_status();
 int vb_grouped_decode_status();
 int vb_latent_prefill_status();
 int vb_lightning_status();
+int vb_delta_chunk_status();
 // moe_kernels.cu
 int vb_moe_route_topk(const void* logits, long long ld, int T, int E, int k, int renorm, float* weights, int* experts, int* counts,
                       cudaStream_t s);

@@ -229,7 +229,8 @@ int vb_rms_conv(int dtype, const VbRmsConv* p, cudaStream_t s);
 // delta_rule.cu / delta_chunk.cu
 int vb_delta_decode(int dtype, const VbDelta* p, cudaStream_t s);
 int vb_delta_scan(int dtype, const VbDelta* p, cudaStream_t s);
-int vb_delta_chunk(const VbDelta* p, cudaStream_t s);
+int vb_delta_chunk_segments(const VbDelta* p);
+int vb_delta_chunk(const VbDelta* p, int nseg, float* ws, cudaStream_t s);
 // conv_prep.cu
 int vb_conv_prep(int dtype, const VbConvPrep* p, cudaStream_t s);
 // lightning.cu / lightning_tcgen05.cu (d <= 128) / lightning_chunk.cu; nseg > 1: workspace of B (nseg - 1) H d e floats
