@@ -67,7 +67,7 @@ def parse_args():
     p.add_argument("--offload", default="auto", choices=["auto", "on", "off"],
                    help="second Adam moment in pinned host memory (optimizer_offload), which leaves the GPU's memory to activations "
                         "instead of recomputation; auto = on one GPU, where the whole unsharded optimizer state would sit on it")
-    p.add_argument("--design", default=None, choices=["zorelorn", "tofinex", "luzitar"],
+    p.add_argument("--design", default=None, choices=["zorelorn", "tofinex", "luzitar", "fusazen"],
                    help="instead of the GRPO step: prefill and decode throughput of this mixer-stack design at a few sizes, beside the uniform "
                         "decoder of equal size (one JSON line per size and model)")
     p.add_argument("--kernels", action="store_true", help="with --design: the kernels of both models, each against its roofline")

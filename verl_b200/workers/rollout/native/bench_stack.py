@@ -4,6 +4,7 @@
     python bench.py --design zorelorn --kernels  # the kernels behind them, each against its roofline
     python bench.py --design tofinex [--kernels]
     python bench.py --design luzitar [--kernels]
+    python bench.py --design fusazen [--kernels]
 
 Random weights and tokens. Prefill runs packed prompts through the engine's prompt path into the cache, decode replays the
 captured decode step over all slots; CUDA events around every timed region, after warm-up, on inputs larger than L2. One
@@ -44,6 +45,14 @@ LUZITAR_SIZES = {
                          ctx=16384),
     "moe4096": dict(width=4096, heads=32, kv_heads=8, window=2048, keep=64, ff=1536, experts=32, top=2, groups=4, group_keep=2, layers=4, prompts=4, prompt_len=4096, slots=128,
                     ctx=4096),
+}
+
+# layers in turn: delta rule, differential attention, attention with norms over whole projections, differential attention over the rows of the one
+# before; the decode steps run at the end of a chunk
+FUSAZEN_SIZES = {
+    "dense2048": dict(width=2048, heads=16, kv_heads=4, delta_dim=64, rank=64, chunk=1024, ff=8192, layers=12, prompts=8, prompt_len=2048, slots=256, ctx=2016),
+    "dense2048-long": dict(width=2048, heads=16, kv_heads=4, delta_dim=64, rank=64, chunk=8192, ff=8192, layers=12, prompts=1, prompt_len=16384, slots=32, ctx=16352),
+    "dense4096": dict(width=4096, heads=32, kv_heads=8, delta_dim=128, rank=128, chunk=2048, ff=16384, layers=8, prompts=4, prompt_len=4096, slots=128, ctx=4064),
 }
 
 
@@ -103,10 +112,29 @@ def closest_to_luzitar(s: dict, params: int) -> ModelConfig:
                        attention_bias=False, tie_word_embeddings=False, num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"])
 
 
+def fusazen_config(s: dict) -> ModelConfig:
+    H, G, layers = s["heads"], s["kv_heads"], []
+    two = dict(heads=H, kv_heads=G, dim=64, vdim=128, diff=0.5, scale=64 ** -0.5, mask={"size": s["chunk"]}, rot=dict(base=500000.0, dims=64))
+    for i in range(0, s["layers"], 4):
+        layers += [("general_delta", dict(heads=s["width"] // s["delta_dim"], dim=s["delta_dim"], decay_rank=s["rank"])), ("attention", two),
+                   ("attention_2", dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask={"size": s["chunk"]})), ("attention", {**two, "kv_from": i + 1})]
+    return ModelConfig.from_hf_dict({"architecture": "Fusazen", "canon": {"taps": 4}, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "vocab": VOCAB, "width": s["width"],
+                                     "layers": [{"type": t, "mixer": m, "mlp": {"kind": "dense", "ff": s["ff"]}} for t, m in layers[: s["layers"]]]})
+
+
+def closest_to_fusazen(s: dict, params: int) -> ModelConfig:
+    """Qwen3-type decoder: full attention of the same head sizes in every layer; its MLP is sized so that the parameters agree."""
+    mk = lambda ff: ModelConfig(model_type="qwen3", vocab_size=VOCAB, hidden_size=s["width"], intermediate_size=ff, num_hidden_layers=s["layers"], num_attention_heads=s["heads"],
+                                num_key_value_heads=s["kv_heads"], head_dim=128, rope_theta=500000.0, max_position_embeddings=1 << 15, qk_norm=True, attention_bias=False,
+                                tie_word_embeddings=False)
+    return mk(max(256, round((params - mk(0).num_parameters()) / (3 * s["width"] * s["layers"]) / 256) * 256))
+
+
 # design -> (sizes, its configuration, label and configuration of the closest existing model)
 DESIGNS = {"zorelorn": (SIZES, zorelorn_config, "uniform decoder of equal size", uniform_config),
            "tofinex": (TOFINEX_SIZES, tofinex_config, "closest existing decoder", closest_to_tofinex),
-           "luzitar": (LUZITAR_SIZES, luzitar_config, "closest existing decoder", closest_to_luzitar)}
+           "luzitar": (LUZITAR_SIZES, luzitar_config, "closest existing decoder", closest_to_luzitar),
+           "fusazen": (FUSAZEN_SIZES, fusazen_config, "closest existing decoder", closest_to_fusazen)}
 
 
 def _events(fn, steps: int) -> float:
@@ -538,9 +566,144 @@ def run_luzitar_kernels(iters: int = 20, only=None, sizes=None) -> None:
     native.check_status()
 
 
+def run_fusazen_kernels(iters: int = 20, only=None, sizes=None) -> None:
+    """The like kernels are those of the closest decoder; those of the delta rule the lightning recurrence's."""
+    dev = torch.device("cuda", torch.cuda.current_device())
+    timer = Timer(dev, iters, 3)
+    r = lambda *sh, sc=1.0, dt=torch.bfloat16: (torch.randn(*sh, device=dev) * sc).to(dt)
+    case = _kernel_reporter("fusazen", "like kernel", timer, only)
+    mm = lambda m, n, k: (2.0 * m * n * k, 2.0 * (m * k + n * k + m * n))
+    for name, s in FUSAZEN_SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        W, H, G, dd, rank, chunk, ff = (s[k] for k in ("width", "heads", "kv_heads", "delta_dim", "rank", "chunk", "ff"))
+        HD, d, e, taps = W // dd, 64, 128, 4
+        Q, scale = H * e, d ** -0.5
+        cos, sin = F.rope_table(1 << 15, 64, 5e5, dev)
+        cos2, sin2 = F.rope_table(1 << 15, 128, 5e5, dev)
+        nw, conv = r(W), r(W, taps, sc=0.4)
+        for phase, T in (("prefill", s["prompts"] * s["prompt_len"]), ("decode", s["slots"])):
+            pre = phase == "prefill"
+            n, L, S, ctx, bs = s["prompts"], s["prompt_len"], s["slots"], s["ctx"], 64
+            h, x, att = r(T, W), torch.randn(T, W, device=dev), r(T, Q)
+            pos = torch.arange(T, device=dev, dtype=torch.int32) % L if pre else torch.full((T,), ctx, device=dev, dtype=torch.int32)
+            cu = torch.arange(n + 1, device=dev, dtype=torch.int32) * L
+            slots, fresh = torch.arange(n, device=dev, dtype=torch.int32), torch.ones(n, device=dev, dtype=torch.int32)
+            active = torch.ones(S, dtype=torch.bool, device=dev)
+            seen = ctx % chunk + 1                    # keys a step sees at position ctx
+            per = -(-(ctx + 64) // bs)
+            table = torch.arange(S * per, device=dev, dtype=torch.int32).view(S, per) if not pre else None
+            cl = torch.full((S,), ctx + 1, device=dev, dtype=torch.int32)
+            pairs = n * (sum(i % chunk + 1 for i in range(L)))
+            # ---- stream
+            ids, emb = torch.randint(0, VOCAB, (T,), device=dev), r(VOCAB, W)
+            case(name, phase, "embed_rows", lambda: X.embed_rows(ids, emb, 1.0), 0, 6.0 * T * W, True)
+            case(name, phase, "embedding", lambda: F.embedding(ids, emb), 0, 4.0 * T * W, False)
+            state = torch.zeros(max(n, S), (taps - 1) * W, device=dev)
+            if pre:
+                case(name, phase, "rms_conv (norm, convolution)", lambda: X.rms_conv(x, nw, 1e-6, conv=conv, cu=cu, state=state, slots=slots, fresh=fresh), 0,
+                     6.0 * T * W + 4.0 * n * (taps - 1) * W, True)
+                case(name, phase, "rms_conv (norm)", lambda: X.rms_conv(x, nw, 1e-6), 0, 6.0 * T * W, True)
+            else:
+                y, bias = X.linear_partial(att, r(W, Q, sc=0.02)), r(W)
+                planes = 4.0 * y.numel() if y.dim() == 3 else 2.0 * y.numel()
+                case(name, phase, "rms_conv (partial products, norm, convolution)", lambda: X.rms_conv(x, nw, 1e-6, y, bias, conv, state=state, active=active), 0,
+                     10.0 * T * W + planes + 8.0 * T * (taps - 1) * W, True)
+                case(name, phase, "rms_conv (partial products, norm)", lambda: X.rms_conv(x, nw, 1e-6, y), 0, 10.0 * T * W + planes, True)
+                del y
+            res = r(T, W)
+            case(name, phase, "rmsnorm with residual", lambda: F.rms_norm(h, nw, 1e-6, residual=res), 0, 8.0 * T * W, False)
+            # ---- delta rule
+            rows = 5 * W + rank
+            w = r(rows, W, sc=0.02)
+            f, b = mm(T, rows, W)
+            case(name, phase, "linear_tanh (r, k, v, a, g, decay)", lambda: X.linear_tanh(h, w, 5 * W), f, b, True)
+            case(name, phase, "gemm (r, k, v, a, g, decay)", lambda: F.gemm(h, w), f, b, False)
+            p, w2 = r(T, rows), r(W, rank, sc=0.1)
+            f, b = mm(T, W, rank)
+            case(name, phase, "linear_act (decay, few columns)", lambda: X.linear_act(p[:, 5 * W :], w2), f, b, True)
+            pc = p[:, 5 * W :].contiguous()
+            case(name, phase, "gemm (decay, few columns)", lambda: F.gemm(pc, w2), f, b, False)
+            zw, ab, w0, nm = r(T, W), r(W), r(W), r(W)
+            mem = torch.zeros(max(n, S), W * dd, device=dev)
+            decay = torch.tensor([1.0 - 2.0 ** (-2.0 - 6.0 * i / HD) for i in range(HD)], device=dev)
+            if pre:
+                case(name, phase, "delta_prefill", lambda: X.delta_prefill(p, zw, ab, w0, HD, cu, mem, slots, fresh), 10.0 * T * W * dd, 12.0 * T * W + 4.0 * n * W * dd, True)
+                case(name, phase, "lightning_prefill", lambda: X.lightning_prefill(p, decay, dd, dd, cu, mem, slots, fresh, True), 4.0 * T * W * dd, 8.0 * T * W + 4.0 * n * W * dd, False)
+                case(name, phase, "gated_rms (norm of every head, gate)", lambda: X.gated_rms(h, p[:, 4 * W : 5 * W], nm, 1e-6, HD), 0, 6.0 * T * W, True)
+            else:
+                case(name, phase, "delta_decode (with norm and gate)", lambda: X.delta_decode(p, zw, ab, w0, HD, nm, 1e-6, mem, active), 0, 14.0 * T * W + 8.0 * T * W * dd, True)
+                case(name, phase, "lightning_decode", lambda: X.lightning_decode(p, decay, dd, dd, mem, active), 0, 8.0 * T * W + 8.0 * T * W * dd, False)
+            del w, p, pc, zw, mem, w2
+            # ---- differential attention
+            vec = r(4 * d, sc=0.05)
+            diff = (vec, 0.5, 1e-6)
+            cols = 2 * H * d + G * (2 * d + e)
+            w = r(cols, W, sc=0.02)
+            f, b = mm(T, cols, W)
+            case(name, phase, "linear_act (query and key maps, values)", lambda: X.linear_act(h, w), f, b, True)
+            case(name, phase, "gemm (query and key maps, values)", lambda: F.gemm(h, w), f, b, False)
+            p = r(T, cols)
+            kw = dict(cu=cu) if pre else dict(active=active)
+            case(name, phase, "conv_qkv_prep (rotation of the maps, rows)", lambda: X.conv_qkv_prep(p, None, 0.0, pos, cos, sin, 2 * H, 2 * G, d, e, True, want_rows=True, norm=False, v_heads=G,
+                                                                                                     **kw), 0, 4.0 * T * cols, True)
+            pq = r(T, 2 * H * d)
+            case(name, phase, "conv_qkv_prep (rotation of the query maps alone)", lambda: X.conv_qkv_prep(pq, None, 0.0, pos, cos, sin, 2 * H, 0, d, e, True, norm=False, v_heads=0, **kw), 0,
+                 8.0 * T * H * d, True)
+            q = r(T, H, e)
+            case(name, phase, "rope (query rotation)", lambda: F.apply_rope_(q, pos, cos2, sin2), 0, 4.0 * T * Q, False)
+            k, v, q2, k2 = r(T, G, e), r(T, G, e), r(T, 2 * H, d), r(T, 2 * G, d)
+            if pre:
+                case(name, phase, "grouped_attention_prefill (differential)", lambda: X.grouped_attention_prefill(q2, k2, v, cu, cu, 0, scale, chunk=chunk, diff=diff),
+                     4.0 * pairs * H * (d + e), 2.0 * T * (H * (2 * d + e) + G * (2 * d + e)), True)
+                case(name, phase, "attention_varlen", lambda: F.attention_varlen(q, k, v, cu, L), 4.0 * n * L * (L + 1) / 2 * Q, 2.0 * T * (2 * Q + 2 * G * e), False)
+            else:
+                pages = r(S * per, bs, 2 * G * e, sc=0.5)
+                case(name, phase, "grouped_attention_decode (differential)", lambda: X.grouped_attention_decode(q2, pages, table, cl, G, e, 0, scale, chunk=chunk, diff=diff),
+                     4.0 * S * seen * H * (d + e), 2.0 * S * seen * G * (2 * d + e), True)
+                few = -(-seen // bs)
+                kc, vc, ct = r(S * few, bs, G, e, sc=0.5), r(S * few, bs, G, e, sc=0.5), torch.arange(S * few, device=dev, dtype=torch.int32).view(S, few)
+                case(name, phase, "paged_decode_attention (as many keys)", lambda: F.paged_decode_attention(q, kc, vc, ct, cl.clamp(max=seen)), 4.0 * S * seen * Q, 4.0 * S * seen * G * e, False)
+                del kc, vc, ct
+            # ---- attention with norms over whole projections
+            cols = (H + 2 * G) * e
+            w, p, qn, kn, temp = r(cols, W, sc=0.02), r(T, cols), r(Q), r(G * e), r(H)
+            f, b = mm(T, cols, W)
+            case(name, phase, "linear_act (q, k, v)", lambda: X.linear_act(h, w), f, b, True)
+            case(name, phase, "gemm (q, k, v)", lambda: F.gemm(h, w), f, b, False)
+            case(name, phase, "whole_norm_prep (norms, rows)", lambda: X.whole_norm_prep(p, qn, kn, temp, 1e-6, H, G, e, want_rows=True), 0, 4.0 * T * cols, True)
+            if pre:
+                case(name, phase, "grouped_attention_prefill (chunks)", lambda: X.grouped_attention_prefill(q, k, v, cu, cu, 0, scale, chunk=chunk), 4.0 * pairs * Q, 2.0 * T * (2 * Q + 2 * G * e),
+                     True)
+            else:
+                case(name, phase, "grouped_attention_decode (chunks)", lambda: X.grouped_attention_decode(q, pages, table, cl, G, e, 0, scale, chunk=chunk), 4.0 * S * seen * Q,
+                     4.0 * S * seen * G * e, True)
+                del pages
+            del w, p, q, k, v, q2, k2, pq
+            # ---- output projection, feed-forward
+            wo, wu, wd, bu, bd, act = r(W, Q, sc=0.02), r(ff, W, sc=0.02), r(W, ff, sc=0.02), r(ff), r(W), r(T, ff)
+            for label, a, w, bias in (("output projection", att, wo, None), ("down projection", act, wd, bd)):
+                f, b = mm(T, W, a.shape[1])
+                if pre:
+                    case(name, phase, f"linear_residual ({label})", lambda: X.linear_residual_(a, w, x, bias=bias), f, b + 6.0 * T * W, True)
+                else:
+                    case(name, phase, f"linear_partial ({label})", lambda: X.linear_partial(a, w), f, b, True)
+                case(name, phase, f"gemm ({label})", lambda: F.gemm(a, w), f, b, False)
+            f, b = mm(T, ff, W)
+            case(name, phase, "linear_bias (up projection, squared relu)", lambda: X.linear_bias(h, wu, bu, "relu2"), f, b, True)
+            case(name, phase, "gemm (up projection)", lambda: F.gemm(h, wu), f, b, False)
+            if not pre:
+                f, b = mm(T, VOCAB, W)
+                case(name, phase, "linear_act (logits)", lambda: X.linear_act(h, emb), f, b, True)
+                case(name, phase, "gemm (logits)", lambda: F.gemm(h, emb), f, b, False)
+            del wo, wu, wd, act, emb, h, x, att, res
+            torch.cuda.empty_cache()
+    native.check_status()
+
+
 def main(args) -> None:
     native.load()
     if args.kernels:
-        {"zorelorn": run_kernels, "tofinex": run_tofinex_kernels, "luzitar": run_luzitar_kernels}[args.design]()
+        {"zorelorn": run_kernels, "tofinex": run_tofinex_kernels, "luzitar": run_luzitar_kernels, "fusazen": run_fusazen_kernels}[args.design]()
     else:
         run_models(args.design, args.steps if args.steps > 2 else 5, args.warmup)
