@@ -45,6 +45,9 @@ void run_gemm(const Tensor& a, const Tensor& w, const VbEpiArgs& e) {
         rc = vb_gemm_skinny_epi(a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), w.stride(0), &e, s, s > 1 ? ws.data_ptr<float>() : nullptr, cur_stream());
       }
     }
+    if (rc < 0 && e.mode == VB_EPI_STORE && e.gate == nullptr && M > 1024 && N % 8 == 0 && K % 8 == 0 && a.stride(0) % 8 == 0 && w.stride(0) % 8 == 0 && e.ldd % 8 == 0 &&
+        !((reinterpret_cast<uintptr_t>(a.data_ptr()) | reinterpret_cast<uintptr_t>(w.data_ptr()) | reinterpret_cast<uintptr_t>(e.D)) & 15))
+      rc = vb_gemm_bf16(a.data_ptr(), w.data_ptr(), e.D, nullptr, M, N, K, a.stride(0), w.stride(0), e.ldd, 0, 0, 0, 0, 0, cur_stream());
     if (rc < 0) rc = vb_gemm_bf16_epi(a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), w.stride(0), &e, cur_stream());
   }
   if (rc < 0) rc = vb_gemm_simt(dt, a.data_ptr(), w.data_ptr(), M, N, K, a.stride(0), w.stride(0), 0, 1, 0, 0, 0, &e, cur_stream());
@@ -88,10 +91,17 @@ Tensor linear_bias(const Tensor& a, const Tensor& w, const Tensor& b, bool relu2
 Tensor linear_tanh(const Tensor& a, const Tensor& w, int64_t n0) {
   const c10::cuda::CUDAGuard guard(a.device());
   Tensor d = at::empty({a.size(0), w.size(0)}, a.options());
+  TORCH_CHECK(n0 >= 0 && n0 <= w.size(0), "linear_tanh: 0 <= n0 <= N");
   VbEpiArgs e{};
-  e.mode = VB_EPI_TANH;
+  // few tokens: the plain product of the decode kernel and a small launch for the few columns beat its epilogue with a function
+  const bool apart = dtype_of(a) == 1 && a.size(0) <= 1024 && n0 >= w.size(0) / 2;
+  e.mode = apart ? VB_EPI_STORE : VB_EPI_TANH;
   e.D = d.data_ptr(); e.ldd = d.stride(0); e.n0 = (int)n0;
   run_gemm(a, w, e);
+  if (apart && n0 < w.size(0)) {
+    verl_count_launches(1);
+    CHECK_RC(vb_tanh_cols(1, reinterpret_cast<char*>(d.data_ptr()) + n0 * d.element_size(), d.stride(0), (int)d.size(0), (int)(w.size(0) - n0), cur_stream()), "vb_tanh_cols");
+  }
   return d;
 }
 

@@ -30,62 +30,60 @@ delta_decode_kernel(const VbDelta p, int RG) {
     for (int c = tid; c < d; c += blockDim.x) orow[c] = from_f<T>(0.f);
     return;
   }
-  float *sr = sm, *sk = sr + d, *su = sk + d, *sw = su + d, *sb = sw + d, *part = sb + d;   // [d] each, then [RG][d]
-  const int cg = d / VEC, rg = tid / cg, ct = tid % cg;
+  float *sr = sm, *sk = sr + d, *sw = sk + d, *sb = sw + d, *part = sb + d, *part2 = part + RG * d;   // [d] each, then [RG][d] twice
+  const int cg = d / VEC, rg = tid / cg, ct = tid % cg, lane = tid & 31;
   const bool on = rg < RG;
   float* S = p.state + t * p.slot_stride + static_cast<long long>(h) * d * d + ct * VEC;
-  float s[ROWS][VEC];
+  const T* row = reinterpret_cast<const T*>(p.p) + t * p.ldp + col0;
+  const T* zw = reinterpret_cast<const T*>(p.zw) + t * p.ldz + col0;
+  float s[ROWS][VEC], v[VEC] = {}, gate[VEC] = {}, nrm[VEC] = {};
   if (on) {
 #pragma unroll
     for (int i = 0; i < ROWS; ++i)
       if (i * RG + rg < d) Vec<float, VEC>::load(S + static_cast<long long>(i * RG + rg) * d, s[i]);
+    Vec<T, VEC>::load(row + 2 * W + ct * VEC, v);
+    if (rg == 0) {
+      Vec<T, VEC>::load(row + 4 * W + ct * VEC, gate);
+      Vec<T, VEC>::load(reinterpret_cast<const T*>(p.norm) + col0 + ct * VEC, nrm);
+    }
   }
-  const T* row = reinterpret_cast<const T*>(p.p) + t * p.ldp + col0;
-  const T* zw = reinterpret_cast<const T*>(p.zw) + t * p.ldz + col0;
-  float kk = 0.f;
+  float kk = 0.f;                                    // every warp sums up the whole key
+  for (int c = lane; c < d; c += 32) {
+    const float k = to_f(row[W + c]);
+    kk += k * k;
+  }
   for (int c = tid; c < d; c += blockDim.x) {
+    const float k = to_f(row[W + c]);
     sr[c] = to_f(row[c]);
-    sk[c] = to_f(row[W + c]);
+    sk[c] = k;
     sw[c] = dr_decay(to_f(zw[c]) + to_f(reinterpret_cast<const T*>(p.w0)[col0 + c]));
-    kk += sk[c] * sk[c];
+    sb[c] = sigmoid_f(to_f(row[3 * W + c]) + to_f(reinterpret_cast<const T*>(p.ab)[col0 + c])) * k;
   }
-  const float iu = 1.f / sqrtf(block_sum(kk, red) + 1e-6f);
-  for (int c = tid; c < d; c += blockDim.x) {
-    const float u = sk[c] * iu;
-    su[c] = u;
-    sb[c] = sigmoid_f(to_f(row[3 * W + c]) + to_f(reinterpret_cast<const T*>(p.ab)[col0 + c])) * u;
-  }
+  const float iu2 = 1.f / (warp_sum(kk) + 1e-6f);    // both factors of the removal carry the key's length
   __syncthreads();
-  auto reduce = [&](float (&acc)[VEC]) {           // over the row groups; every thread of a column gets the sum
-    if (on) {
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) part[rg * d + ct * VEC + k] = acc[k];
-    }
-    __syncthreads();
-#pragma unroll
-    for (int k = 0; k < VEC; ++k) acc[k] = 0.f;
-    if (on) {
-      for (int g = 0; g < RG; ++g)
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) acc[k] += part[g * d + ct * VEC + k];
-    }
-    __syncthreads();
-  };
-  float held[VEC] = {}, o[VEC] = {}, v[VEC] = {};
+  float held[VEC] = {}, o[VEC] = {};
   if (on) {
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
       const int r = i * RG + rg;
       if (r < d) {
-        const float u = su[r];
+        const float k_ = sk[r];
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) held[k] = fmaf(u, s[i][k], held[k]);
+        for (int k = 0; k < VEC; ++k) held[k] = fmaf(k_, s[i][k], held[k]);
       }
     }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) part[rg * d + ct * VEC + k] = held[k];
   }
-  reduce(held);
+  __syncthreads();
   if (on) {
-    Vec<T, VEC>::load(row + 2 * W + ct * VEC, v);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) held[k] = 0.f;
+    for (int g = 0; g < RG; ++g)
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) held[k] += part[g * d + ct * VEC + k];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) held[k] *= iu2;
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
       const int r = i * RG + rg;
@@ -99,20 +97,30 @@ delta_decode_kernel(const VbDelta p, int RG) {
         Vec<float, VEC>::store(S + static_cast<long long>(r) * d, s[i]);
       }
     }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) part2[rg * d + ct * VEC + k] = o[k];
   }
-  reduce(o);
+  __syncthreads();
   float ss = 0.f;
   if (on && rg == 0) {
 #pragma unroll
+    for (int k = 0; k < VEC; ++k) o[k] = 0.f;
+    for (int g = 0; g < RG; ++g)
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) o[k] += part2[g * d + ct * VEC + k];
+#pragma unroll
     for (int k = 0; k < VEC; ++k) ss += o[k] * o[k];
   }
-  const float r = 1.f / sqrtf(block_sum(ss, red) / d + p.eps);
+  if (cg <= 32) {                                    // the columns' threads are one warp
+    if (tid >= 32) return;
+    ss = warp_sum(ss);
+  } else {
+    ss = block_sum(ss, red);
+  }
+  const float r = 1.f / sqrtf(ss / d + p.eps);
   if (on && rg == 0) {
-    float g[VEC], n[VEC];
-    Vec<T, VEC>::load(row + 4 * W + ct * VEC, g);
-    Vec<T, VEC>::load(reinterpret_cast<const T*>(p.norm) + col0 + ct * VEC, n);
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) orow[ct * VEC + k] = from_f<T>(o[k] * r * n[k] * sigmoid_f(g[k]));
+    for (int k = 0; k < VEC; ++k) orow[ct * VEC + k] = from_f<T>(o[k] * r * nrm[k] * sigmoid_f(gate[k]));
   }
 }
 
@@ -184,9 +192,12 @@ template <typename T, int VEC>
 static int delta_decode(const VbDelta* p, cudaStream_t s) {
   const int cg = p->d / VEC;
   if (cg > 256) return -1;
-  int RG = 256 / cg;
+  int RG = (p->d + 15) / 16;                         // sixteen rows of a thread: small CTAs, many of them
+  if (RG * cg < 64) RG = 64 / cg;
+  if (RG * cg > 256) RG = 256 / cg;
   if (RG > p->d) RG = p->d;
-  const int rows = (p->d + RG - 1) / RG, smem = (5 * p->d + RG * p->d) * 4;
+  if (RG < 1) RG = 1;
+  const int rows = (p->d + RG - 1) / RG, smem = (4 * p->d + 2 * RG * p->d) * 4;
   auto go = [&](auto kern) {
     const int rc = dr_smem(kern, smem);
     if (rc != 0) return rc;

@@ -252,9 +252,22 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
           if (EPI == SK_MIX && direct) {
             const int col = w.out_col0 + nl;
             const EpiColumn ec = epi_column(p.mix, col);
+            const int mode = p.mix.mode;
+            const bool square = mode == VB_EPI_BIAS_RELU2;
+            if (square || mode == VB_EPI_BIAS || (mode == VB_EPI_TANH && col < p.mix.n0) || (mode == VB_EPI_SILU && col >= p.mix.n0)) {
+              // columns without a function: no switch over the modes per element
+              __nv_bfloat16* d = reinterpret_cast<__nv_bfloat16*>(p.mix.D) + static_cast<long long>(tok0 + c * 32) * p.mix.ldd + col;
 #pragma unroll
-            for (int j = 0; j < 32; ++j)
-              if (j < mrem) epi_store1(p.mix, tok0 + c * 32 + j, col, __uint_as_float(r[j]), mix_alpha, mix_palpha, ec);
+              for (int j = 0; j < 32; ++j)
+                if (j < mrem) {
+                  const float v = __uint_as_float(r[j]) + ec.b;
+                  d[j * p.mix.ldd] = __float2bfloat16(square ? relu2(v) : v);
+                }
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (j < mrem) epi_store1(p.mix, tok0 + c * 32 + j, col, __uint_as_float(r[j]), mix_alpha, mix_palpha, ec);
+            }
           } else if (direct) {
 #pragma unroll
             for (int j = 0; j < 32; ++j)
@@ -307,6 +320,17 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
             b4.x = __bfloat162float(bp[0]); b4.y = __bfloat162float(bp[1]);
             b4.z = __bfloat162float(bp[2]); b4.w = __bfloat162float(bp[3]);
           }
+          bool plain = EPI != SK_MIX, square = false;   // without a function of the mode's that needs the whole switch
+          if constexpr (EPI == SK_MIX) {
+            const int mode = p.mix.mode;
+            square = mode == VB_EPI_BIAS_RELU2;
+            const bool bias = square || mode == VB_EPI_BIAS;
+            plain = bias || (mode == VB_EPI_TANH && col + 4 <= p.mix.n0) || (mode == VB_EPI_SILU && col >= p.mix.n0);
+            if (bias) {
+              const __nv_bfloat16* bp = reinterpret_cast<const __nv_bfloat16*>(p.mix.nb) + col;
+              b4 = make_float4(__bfloat162float(bp[0]), __bfloat162float(bp[1]), __bfloat162float(bp[2]), __bfloat162float(bp[3]));
+            }
+          }
           const float* __restrict__ src = p.ws + col;
           const long long split_stride = p.ws_split_stride;
           constexpr int RB = 4;  // rows in flight per thread
@@ -330,7 +354,13 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
 #pragma unroll
             for (int u = 0; u < RB; ++u) {
               const int mm = m + 4 * u;
-              if (EPI == SK_MIX) {
+              if (EPI == SK_MIX && plain) {
+                if (mm < r1) {
+                  if (square) { a[u].x = relu2(a[u].x); a[u].y = relu2(a[u].y); a[u].z = relu2(a[u].z); a[u].w = relu2(a[u].w); }
+                  *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.mix.D) + static_cast<long long>(mm) * p.mix.ldd + col) =
+                      make_uint2(pack_bf16x2(a[u].x, a[u].y), pack_bf16x2(a[u].z, a[u].w));
+                }
+              } else if (EPI == SK_MIX) {
                 if (mm < r1) {
                   const float v4[4] = {a[u].x, a[u].y, a[u].z, a[u].w};
                   epi_store_row<4>(p.mix, mm, col, v4, mix_alpha, mix_palpha);

@@ -220,6 +220,8 @@ int vb_residual_dyt(int dtype, const VbResidDyt* p, cudaStream_t s);
 // W = heads * size: statistics over each head's columns
 int vb_gated_rms(int dtype, const void* o, long long ldo, const void* g, long long ldg, const void* norm, float eps, void* out, int T, int W, int heads,
                  cudaStream_t s);
+// x[t, c] = tanh(x[t, c]) for c < n
+int vb_tanh_cols(int dtype, void* x, long long ld, int T, int n, cudaStream_t s);
 int vb_whole_norm(int dtype, const VbWholeNorm* p, cudaStream_t s);
 // a [T, 2 H, dv] -> out [T, H, dv], see VbLatentAttn::maps
 int vb_diff_combine(int dtype, const void* a, int a_f32, const void* vec, int dim, float diff, float eps, void* out, int T, int H, int dv, cudaStream_t s);

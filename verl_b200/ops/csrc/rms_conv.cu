@@ -1,8 +1,8 @@
 // Row kernels of stacks with RMS norms in front of the sublayers: embedding, and norm of the residual stream with an optional causal
 // convolution of its output over time, h + conv(h). A decode step's kernel also adds the partial products of the GEMM in front of it
-// (and a bias) to the stream, takes the convolution's past from the slot's state and moves it on. Prompts: a CTA takes a run of
-// consecutive tokens; statistics first (a warp per row), then every thread walks its columns through the run with the window of normed
-// rows in registers. What a sequence keeps (fp32) is written by a second small launch. Compiled without fast math.
+// (and a bias) to the stream, takes the convolution's past from the slot's state and moves it on. Prompts: a CTA walks a run of
+// consecutive tokens, four at a time (the next four on their way), and keeps the window of normed rows in registers; rows too wide for
+// that are read twice (statistics first, a warp per row). What a sequence keeps (fp32) is written by a second small launch. Compiled without fast math.
 #include "mixers.h"
 #include "mixer_common.cuh"
 
@@ -139,6 +139,7 @@ __device__ __forceinline__ float rc_scale(const float* x, int W, float eps) {
   return 1.f / sqrtf(warp_sum(ss) / W + eps);
 }
 
+// Rows too wide for the kernel below, and columns one at a time.
 constexpr int RC_RUN = 16;   // tokens of a CTA
 template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(256)
@@ -216,6 +217,166 @@ rms_conv_kernel(const VbRmsConv a) {
   }
 }
 
+// two floats in a register pair: one instruction for both
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("{\n.reg .b64 a, b, c, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmov.b64 c, {%6, %7};\nfma.rn.f32x2 d, a, b, c;\nmov.b64 {%0, %1}, d;\n}"
+      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+  return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+  float2 d;
+  asm("{\n.reg .b64 a, b, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmul.rn.f32x2 d, a, b;\nmov.b64 {%0, %1}, d;\n}" : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+  return d;
+}
+
+// The same with every row read once: a thread owns eight columns (W <= 8 blockDim), four tokens share a reduction, the rows of the next
+// eight are on their way to shared memory (every thread fetches and reads its own columns).
+constexpr int RW_RUN = 16, RW_N = 4, RW_STAGES = 3, RW_VEC = 8;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(512)
+rms_conv_once_kernel(const VbRmsConv a) {
+  constexpr int PAST = TAPS - 1, H = RW_VEC / 2;
+  extern __shared__ __align__(16) float ring[];      // [stage][token][thread][8]
+  __shared__ float part[2][16][RW_N];
+  const int t0 = blockIdx.x * RW_RUN, t1 = min(a.T, t0 + RW_RUN), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, c = threadIdx.x * RW_VEC;
+  const bool on = c < a.W;
+  const int first = max(0, t0 - PAST);               // rows t0 - PAST .. are normed too
+  float* mine = ring + threadIdx.x * RW_VEC;
+  const int row = blockDim.x * RW_VEC;
+  auto fetch = [&](int n) {                          // batch n
+#pragma unroll
+    for (int u = 0; u < RW_N; ++u) {
+      const int t = first + n * RW_N + u;
+      if (t < t1) {
+        const uint32_t dst = static_cast<uint32_t>(__cvta_generic_to_shared(mine + (n % RW_STAGES * RW_N + u) * row));
+        const float* src = a.x + static_cast<long long>(t) * a.W + (on ? c : 0);
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + 16), "l"(src + 4), "r"(on ? 16 : 0) : "memory");
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll
+  for (int n = 0; n < RW_STAGES - 1; ++n) fetch(n);
+  float2 g[H] = {}, w[TAPS][H] = {}, rows[PAST + RW_N][H];   // the window, then the batch's rows
+  if (on) {
+    float v[RW_VEC];
+    Vec<T, RW_VEC>::load(reinterpret_cast<const T*>(a.nw) + c, v);
+#pragma unroll
+    for (int i = 0; i < H; ++i) g[i] = make_float2(v[2 * i], v[2 * i + 1]);
+    const T* conv = reinterpret_cast<const T*>(a.conv) + static_cast<long long>(c) * TAPS;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < H; ++i)
+        w[j][i] = make_float2(to_f(conv[2 * i * TAPS + j]) + (j == PAST ? 1.f : 0.f), to_f(conv[(2 * i + 1) * TAPS + j]) + (j == PAST ? 1.f : 0.f));
+  }
+#pragma unroll
+  for (int k = 0; k < PAST; ++k)
+#pragma unroll
+    for (int i = 0; i < H; ++i) rows[k][i] = make_float2(0.f, 0.f);
+  int b = rc_sequence(a, first), end = a.cu[b + 1];
+  auto kept = [&](int k, int slot) {                 // row `slot` of what sequence b kept -> window row k
+    const float* st = rc_past(a, b);
+#pragma unroll
+    for (int i = 0; i < H; ++i) rows[k][i] = on && st != nullptr ? *reinterpret_cast<const float2*>(st + static_cast<long long>(slot) * a.W + c + 2 * i) : make_float2(0.f, 0.f);
+  };
+  {  // a list that starts within PAST rows of a portion's start: what the sequence kept stands in front
+    const int back = first - a.cu[b];
+#pragma unroll
+    for (int k = 0; k < PAST; ++k)
+      if (back + k < PAST) kept(k, back + k);        // only looked at when the list starts with the portion
+  }
+  const int batches = (t1 - first + RW_N - 1) / RW_N;
+  for (int n = 0; n < batches; ++n) {
+    const int t = first + n * RW_N;
+    asm volatile("cp.async.wait_group %0;" ::"n"(RW_STAGES - 2) : "memory");
+    float ss[RW_N];
+#pragma unroll
+    for (int u = 0; u < RW_N; ++u) {
+      const float4* src = reinterpret_cast<const float4*>(mine + (n % RW_STAGES * RW_N + u) * row);
+      const float4 x = t + u < t1 ? src[0] : make_float4(0.f, 0.f, 0.f, 0.f), y = t + u < t1 ? src[1] : make_float4(0.f, 0.f, 0.f, 0.f);
+      rows[PAST + u][0] = make_float2(x.x, x.y);
+      rows[PAST + u][1] = make_float2(x.z, x.w);
+      rows[PAST + u][2] = make_float2(y.x, y.y);
+      rows[PAST + u][3] = make_float2(y.z, y.w);
+      float2 q = mul2(rows[PAST + u][0], rows[PAST + u][0]);
+#pragma unroll
+      for (int i = 1; i < H; ++i) q = fma2(rows[PAST + u][i], rows[PAST + u][i], q);
+      ss[u] = q.x + q.y;
+    }
+    if (n + RW_STAGES - 1 < batches) fetch(n + RW_STAGES - 1);   // into the stage that was read one batch ago
+    else asm volatile("cp.async.commit_group;" ::: "memory");
+    {  // four sums at once: after two steps a lane is in charge of one token
+      const bool up16 = (lane & 16) != 0, up8 = (lane & 8) != 0;
+      const float y0 = (up16 ? ss[2] : ss[0]) + __shfl_xor_sync(0xffffffffu, up16 ? ss[0] : ss[2], 16);
+      const float y1 = (up16 ? ss[3] : ss[1]) + __shfl_xor_sync(0xffffffffu, up16 ? ss[1] : ss[3], 16);
+      float y = (up8 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up8 ? y0 : y1, 8);
+      y += __shfl_xor_sync(0xffffffffu, y, 4);
+      y += __shfl_xor_sync(0xffffffffu, y, 2);
+      y += __shfl_xor_sync(0xffffffffu, y, 1);
+      if ((lane & 7) == 0) part[n & 1][warp][lane >> 3] = y;
+    }
+    __syncthreads();
+    float sum[RW_N] = {};
+    for (int k = 0; k < nw; ++k) {
+      const float4 v = *reinterpret_cast<const float4*>(part[n & 1][k]);
+      sum[0] += v.x; sum[1] += v.y; sum[2] += v.z; sum[3] += v.w;
+    }
+#pragma unroll
+    for (int u = 0; u < RW_N; ++u) {
+      const float r = rsqrtf(sum[u] / a.W + a.eps);
+#pragma unroll
+      for (int i = 0; i < H; ++i) rows[PAST + u][i] = mul2(mul2(rows[PAST + u][i], make_float2(r, r)), g[i]);
+    }
+    auto put = [&](int u, const float2 (&o)[H]) {
+      if (!on || t + u < t0 || t + u >= t1) return;
+      const float v[RW_VEC] = {o[0].x, o[0].y, o[1].x, o[1].y, o[2].x, o[2].y, o[3].x, o[3].y};
+      Vec<T, RW_VEC>::store(reinterpret_cast<T*>(a.h) + static_cast<long long>(t + u) * a.W + c, v);
+    };
+    if (min(t + RW_N, t1) <= end) {                  // one portion (the same for the whole CTA)
+#pragma unroll
+      for (int u = 0; u < RW_N; ++u) {
+        float2 o[H];
+#pragma unroll
+        for (int i = 0; i < H; ++i) {
+          o[i] = mul2(w[PAST][i], rows[PAST + u][i]);
+#pragma unroll
+          for (int k = 0; k < PAST; ++k) o[i] = fma2(w[k][i], rows[u + k][i], o[i]);
+        }
+        put(u, o);
+      }
+#pragma unroll
+      for (int k = 0; k < PAST; ++k)
+#pragma unroll
+        for (int i = 0; i < H; ++i) rows[k][i] = rows[RW_N + k][i];
+    } else {
+#pragma unroll
+      for (int u = 0; u < RW_N; ++u) {
+        if (t + u >= t1) break;
+        if (t + u >= end) {                          // the next portion
+          while (t + u >= end) { ++b; end = a.cu[b + 1]; }
+#pragma unroll
+          for (int k = 0; k < PAST; ++k) kept(k, k);
+        }
+        float2 o[H];
+#pragma unroll
+        for (int i = 0; i < H; ++i) {
+          o[i] = mul2(w[PAST][i], rows[PAST + u][i]);
+#pragma unroll
+          for (int k = 0; k < PAST; ++k) o[i] = fma2(w[k][i], rows[k][i], o[i]);
+        }
+        put(u, o);
+#pragma unroll
+        for (int k = 0; k < PAST; ++k)
+#pragma unroll
+          for (int i = 0; i < H; ++i) rows[k][i] = k + 1 < PAST ? rows[k + 1 < PAST ? k + 1 : k][i] : rows[PAST + u][i];
+      }
+    }
+  }
+}
+
 // Any number of taps: one CTA per token, the rows of the window are normed again.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -243,7 +404,7 @@ rms_conv_any_kernel(const VbRmsConv a) {
 }
 
 // The last taps - 1 normed rows of every portion (a portion shorter than that moves older ones up). One CTA per sequence.
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 rms_conv_state_kernel(const VbRmsConv a) {
   extern __shared__ float inv[];                     // [taps - 1]
@@ -253,17 +414,26 @@ rms_conv_state_kernel(const VbRmsConv a) {
   const bool zero = a.fresh != nullptr && a.fresh[b] != 0;
   for (int j = warp; j < past; j += 8) {
     const int at = n - past + j;
-    const float f = at >= 0 ? rc_scale<1>(a.x + static_cast<long long>(s0 + at) * a.W, a.W, a.eps) : 0.f;
+    const float f = at >= 0 ? rc_scale<VEC>(a.x + static_cast<long long>(s0 + at) * a.W, a.W, a.eps) : 0.f;
     if ((threadIdx.x & 31) == 0) inv[j] = f;
   }
   __syncthreads();
   float* st = a.state + static_cast<long long>(a.slots[b]) * a.slot_stride;
-  for (int c = threadIdx.x; c < a.W; c += 256) {
-    const float g = to_f(reinterpret_cast<const T*>(a.nw)[c]);
+  for (int c = threadIdx.x * VEC; c < a.W; c += 256 * VEC) {
+    float g[VEC], v[VEC];
+    Vec<T, VEC>::load(reinterpret_cast<const T*>(a.nw) + c, g);
     for (int j = 0; j < past; ++j) {
       const int at = n - past + j;                   // reads ahead of what it writes
-      st[static_cast<long long>(j) * a.W + c] = at >= 0 ? a.x[static_cast<long long>(s0 + at) * a.W + c] * inv[j] * g
-                                                        : (zero ? 0.f : st[static_cast<long long>(at + past) * a.W + c]);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+      if (at >= 0) {
+        Vec<float, VEC>::load(a.x + static_cast<long long>(s0 + at) * a.W + c, v);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] *= inv[j] * g[i];
+      } else if (!zero) {
+        Vec<float, VEC>::load(st + static_cast<long long>(at + past) * a.W + c, v);
+      }
+      Vec<float, VEC>::store(st + static_cast<long long>(j) * a.W + c, v);
     }
   }
 }
@@ -271,7 +441,17 @@ rms_conv_state_kernel(const VbRmsConv a) {
 template <typename T, int VEC>
 static int rms_conv_run(const VbRmsConv* p, cudaStream_t s) {
   const unsigned grid = static_cast<unsigned>((p->T + RC_RUN - 1) / RC_RUN);
-  if (p->taps == 1) rms_conv_kernel<T, VEC, 1><<<grid, 256, 0, s>>>(*p);
+  const int threads = ((p->W + VEC - 1) / VEC + 31) / 32 * 32;
+  if (VEC == RW_VEC && threads <= 512 && p->taps <= 4) {
+    const int smem = RW_STAGES * RW_N * threads * RW_VEC * 4;
+    auto go = [&](auto kern) {
+      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+      if (e != cudaSuccess) return static_cast<int>(e);
+      kern<<<static_cast<unsigned>((p->T + RW_RUN - 1) / RW_RUN), threads, smem, s>>>(*p);
+      return static_cast<int>(cudaGetLastError());
+    };
+    return p->taps == 1 ? go(rms_conv_once_kernel<T, 1>) : p->taps == 2 ? go(rms_conv_once_kernel<T, 2>) : p->taps == 3 ? go(rms_conv_once_kernel<T, 3>) : go(rms_conv_once_kernel<T, 4>);
+  } else if (p->taps == 1) rms_conv_kernel<T, VEC, 1><<<grid, 256, 0, s>>>(*p);
   else if (p->taps == 2) rms_conv_kernel<T, VEC, 2><<<grid, 256, 0, s>>>(*p);
   else if (p->taps == 3) rms_conv_kernel<T, VEC, 3><<<grid, 256, 0, s>>>(*p);
   else if (p->taps == 4) rms_conv_kernel<T, VEC, 4><<<grid, 256, 0, s>>>(*p);
@@ -313,8 +493,8 @@ extern "C" int vb_rms_conv(int dtype, const VbRmsConv* p, cudaStream_t s) {
   if (dtype == 0) rc = vec ? rms_conv_run<float, 8>(p, s) : rms_conv_run<float, 1>(p, s);
   else rc = vec ? rms_conv_run<bf16, 8>(p, s) : rms_conv_run<bf16, 1>(p, s);
   if (rc == 0 && p->state != nullptr && p->slots != nullptr && p->taps > 1) {
-    if (dtype == 0) rms_conv_state_kernel<float><<<p->B, 256, p->taps * 4, s>>>(*p);
-    else rms_conv_state_kernel<bf16><<<p->B, 256, p->taps * 4, s>>>(*p);
+    if (dtype == 0) vec ? rms_conv_state_kernel<float, 8><<<p->B, 256, p->taps * 4, s>>>(*p) : rms_conv_state_kernel<float, 1><<<p->B, 256, p->taps * 4, s>>>(*p);
+    else vec ? rms_conv_state_kernel<bf16, 8><<<p->B, 256, p->taps * 4, s>>>(*p) : rms_conv_state_kernel<bf16, 1><<<p->B, 256, p->taps * 4, s>>>(*p);
     rc = static_cast<int>(cudaGetLastError());
   }
   return rc;

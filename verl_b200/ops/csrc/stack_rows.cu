@@ -444,6 +444,15 @@ qkv_prep_kernel(const VbQkvPrep a, int L, long long units) {
   }
 }
 
+// --------------------------------------------------------------------------------------------- tanh of some columns, in place
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_cols_kernel(T* __restrict__ x, long long ld, int n, long long total) {
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= total) return;
+  T* at = x + i / n * ld + i % n;
+  *at = from_f<T>(tanhf(to_f(*at)));
+}
+
 static bool mis16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) != 0; }
 
 }  // namespace vb
@@ -500,6 +509,15 @@ extern "C" int vb_residual_dyt(int dtype, const VbResidDyt* p, cudaStream_t s) {
     if (vec) residual_dyt_kernel<bf16, 8><<<grid, 256, 0, s>>>(*p, total);
     else residual_dyt_kernel<bf16, 1><<<grid, 256, 0, s>>>(*p, total);
   }
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int vb_tanh_cols(int dtype, void* x, long long ld, int T, int n, cudaStream_t s) {
+  const long long total = static_cast<long long>(T) * n;
+  if (total <= 0) return 0;
+  const unsigned grid = static_cast<unsigned>((total + 255) / 256);
+  if (dtype == 0) tanh_cols_kernel<float><<<grid, 256, 0, s>>>((float*)x, ld, n, total);
+  else tanh_cols_kernel<bf16><<<grid, 256, 0, s>>>((bf16*)x, ld, n, total);
   return static_cast<int>(cudaGetLastError());
 }
 
