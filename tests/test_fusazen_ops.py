@@ -288,7 +288,7 @@ def plain_delta(p, zw, ab, w0, H):
     return torch.cat([plain.delta_rule(r[:, h], k[:, h], v[:, h], w[:, h], a[:, h]) for h in range(H)], -1)
 
 
-DELTA = [(2, 8), (3, 32), (1, 40), (4, 64), (2, 96), (2, 128), (3, 10), (2, 7), (1, 136), (1, 1)]
+DELTA = [(2, 8), (3, 32), (1, 40), (4, 64), (2, 96), (2, 128), (3, 10), (2, 7), (1, 136), (1, 250), (1, 260), (1, 1)]
 
 
 @pytest.mark.parametrize("H,d", DELTA)

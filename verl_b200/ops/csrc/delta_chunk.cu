@@ -409,7 +409,7 @@ delta_chunk_kernel(const VbDelta P, int nseg, float* __restrict__ ws, int* statu
         for (int u = 0; u < 2; ++u)
 #pragma unroll
           for (int i = 0; i < 4; ++i) x[u][i] = 0.f;
-        constexpr int KB = RP > 0 && RP < 72 ? 1 : 2;
+        constexpr int KB = SW < 2 ? 1 : 2;
 #pragma unroll
         for (int k0 = 0; k0 < SW; k0 += KB) {
           uint32_t ah[KB][4], al[KB][4], bh[KB][4], bl[KB][4];
@@ -627,7 +627,7 @@ extern "C" int vb_delta_chunk(const VbDelta* p, int nseg, float* ws, cudaStream_
     rc = static_cast<int>(cudaGetLastError());
     if (rc != 0) return rc;
   }
-  return p->d <= 32 ? VB_DC(32, 2, 4, 3, 0, 0, true) : p->d <= 64 ? VB_DC(64, 2, 4, 2, 96, 72, true) : p->d <= 96 ? VB_DC(96, 1, 4, 1, 0, 0, true) : VB_DC(128, 2, 4, 1, 128, 56, true);
+  return p->d <= 32 ? VB_DC(32, 2, 4, 3, 0, 0, true) : p->d <= 64 ? VB_DC(64, 2, 4, 2, 96, 72, true) : p->d <= 96 ? VB_DC(96, 1, 4, 1, 0, 0, true) : VB_DC(128, 2, 4, 1, 112, 64, true);
 #undef VB_DC
 }
 

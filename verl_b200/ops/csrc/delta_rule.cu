@@ -124,6 +124,52 @@ delta_decode_kernel(const VbDelta p, int RG) {
   }
 }
 
+// Heads too large for registers: a thread owns every 256th column and reads its part of the state twice.
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_decode_any_kernel(const VbDelta p) {
+  extern __shared__ float sm[];
+  __shared__ float red[33];
+  const int h = blockIdx.x, tid = threadIdx.x, d = p.d, W = p.H * d, col0 = h * d;
+  const long long t = blockIdx.y;
+  T* orow = reinterpret_cast<T*>(p.out) + t * p.ldo + col0;
+  if (!p.active[t]) {
+    for (int c = tid; c < d; c += 256) orow[c] = from_f<T>(0.f);
+    return;
+  }
+  float *sr = sm, *sk = sr + d, *sw = sk + d, *sb = sw + d, *so = sb + d;   // [d] each
+  float* S = p.state + t * p.slot_stride + static_cast<long long>(h) * d * d;
+  const T* row = reinterpret_cast<const T*>(p.p) + t * p.ldp + col0;
+  const T* zw = reinterpret_cast<const T*>(p.zw) + t * p.ldz + col0;
+  float kk = 0.f;
+  for (int c = tid; c < d; c += 256) {
+    const float k = to_f(row[W + c]);
+    sr[c] = to_f(row[c]);
+    sk[c] = k;
+    sw[c] = dr_decay(to_f(zw[c]) + to_f(reinterpret_cast<const T*>(p.w0)[col0 + c]));
+    sb[c] = sigmoid_f(to_f(row[3 * W + c]) + to_f(reinterpret_cast<const T*>(p.ab)[col0 + c])) * k;
+    kk += k * k;
+  }
+  const float iu2 = 1.f / (block_sum(kk, red) + 1e-6f);
+  float ss = 0.f;
+  for (int c = tid; c < d; c += 256) {
+    float held = 0.f, o = 0.f;
+    const float v = to_f(row[2 * W + c]);
+    for (int r = 0; r < d; ++r) held = fmaf(sk[r], S[static_cast<long long>(r) * d + c], held);
+    held *= iu2;
+    for (int r = 0; r < d; ++r) {
+      float* at = S + static_cast<long long>(r) * d + c;
+      const float s = fmaf(sw[r], *at, fmaf(sk[r], v, -sb[r] * held));
+      *at = s;
+      o = fmaf(sr[r], s, o);
+    }
+    so[c] = o;
+    ss += o * o;
+  }
+  const float f = 1.f / sqrtf(block_sum(ss, red) / d + p.eps);
+  for (int c = tid; c < d; c += 256) orow[c] = from_f<T>(so[c] * f * to_f(reinterpret_cast<const T*>(p.norm)[col0 + c]) * sigmoid_f(to_f(row[4 * W + c])));
+}
+
 // Token-by-token scan of a portion: one CTA = one (sequence, head, 32 columns of v); the state columns live in shared memory.
 constexpr int DS_COLS = 32, DS_ROWS = 8;
 template <typename T>
@@ -191,13 +237,18 @@ static int dr_smem(K kern, int bytes) {
 template <typename T, int VEC>
 static int delta_decode(const VbDelta* p, cudaStream_t s) {
   const int cg = p->d / VEC;
-  if (cg > 256) return -1;
   int RG = (p->d + 15) / 16;                         // sixteen rows of a thread: small CTAs, many of them
   if (RG * cg < 64) RG = 64 / cg;
   if (RG * cg > 256) RG = 256 / cg;
   if (RG > p->d) RG = p->d;
-  if (RG < 1) RG = 1;
-  const int rows = (p->d + RG - 1) / RG, smem = (4 * p->d + 2 * RG * p->d) * 4;
+  const int rows = RG > 0 ? (p->d + RG - 1) / RG : p->d;
+  if (RG < 1 || rows > 64) {
+    const int smem = 5 * p->d * 4, rc = dr_smem(delta_decode_any_kernel<T>, smem);
+    if (rc != 0) return rc;
+    delta_decode_any_kernel<T><<<dim3(p->H, p->T), 256, smem, s>>>(*p);
+    return static_cast<int>(cudaGetLastError());
+  }
+  const int smem = (4 * p->d + 2 * RG * p->d) * 4;
   auto go = [&](auto kern) {
     const int rc = dr_smem(kern, smem);
     if (rc != 0) return rc;
@@ -207,8 +258,7 @@ static int delta_decode(const VbDelta* p, cudaStream_t s) {
   if (rows <= 4) return go(delta_decode_kernel<T, VEC, 4>);
   if (rows <= 8) return go(delta_decode_kernel<T, VEC, 8>);
   if (rows <= 16) return go(delta_decode_kernel<T, VEC, 16>);
-  if (rows <= 64) return go(delta_decode_kernel<T, VEC, 64>);
-  return -1;
+  return go(delta_decode_kernel<T, VEC, 64>);
 }
 
 template <typename T>
